@@ -92,10 +92,8 @@ __device__ __forceinline__ void tmem_st_wait() {
 }
 
 // The softmax warps are bound by instruction issue (one slot per sub-partition and clock), so the
-// exponent path uses the cheapest encodings the ISA has: packed two-lane fp32 FMA / ADD
-// (fma.rn.f32x2, add.rn.f32x2 — one issue slot for two elements) and the bare ex2.approx.ftz
-// (exp2f() wraps it in a denormal-range rescue of three more instructions; the arguments here are
-// <= 8 and flush-to-zero at the bottom is exactly what a softmax tail wants).
+// exponent path uses packed two-lane fp32 FMA / ADD (fma.rn.f32x2, add.rn.f32x2) and the PTX
+// instruction ex2.approx.ftz (the arguments are <= 8, and flushing the softmax tail to zero is fine).
 __device__ __forceinline__ uint64_t pack_f32x2(uint32_t lo, uint32_t hi) {
   uint64_t r;
   asm("mov.b64 %0, {%1, %2};" : "=l"(r) : "r"(lo), "r"(hi));
