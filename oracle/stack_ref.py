@@ -1,0 +1,143 @@
+"""ORACLE (test infrastructure only — never imported by the product path).
+
+Plain, slow restatement of the mechanisms that layer-stack designs are made of (Bekopel: latent
+attention with a sliding window and a sink, generalized delta rule, PolyNorm feed-forward, norms on
+both sides of each sublayer).  One function per mechanism; torch on the CPU, in the dtype of its
+inputs (the tests use float64, rounding weights only).  A whole sequence is computed at once, token by
+token where there is a recurrence, with no cache: what a cache, a batch or a cut of the prompt could get
+wrong is absent here by construction.
+
+Every function works on one sequence; x is [tokens, width].
+"""
+from __future__ import annotations
+
+import math
+
+import torch
+
+
+def rms_norm(x, eps, weight=None):
+    y = x / torch.sqrt((x * x).mean(-1, keepdim=True) + eps)
+    return y if weight is None else y * weight
+
+
+def poly_norm(z, coef, eps):
+    a, b, c, e = coef
+    return a * rms_norm(z, eps) + b * rms_norm(z ** 2, eps) + c * rms_norm(z ** 3, eps) + e
+
+
+def rotate(x, positions, dims, base):
+    """Rotate-half over the first `dims` entries of the last axis; x is [tokens, ..., n]."""
+    half = dims // 2
+    f = torch.tensor([float(base) ** (-2.0 * i / dims) for i in range(half)], dtype=torch.float64)
+    ang = positions.to(torch.float64)[:, None] * f[None, :]
+    cos, sin = ang.cos().to(x.dtype), ang.sin().to(x.dtype)
+    shape = (x.shape[0],) + (1,) * (x.dim() - 2) + (half,)
+    cos, sin = cos.view(shape), sin.view(shape)
+    u, v = x[..., :half], x[..., half:dims]
+    return torch.cat([u * cos - v * sin, v * cos + u * sin, x[..., dims:]], dim=-1)
+
+
+def window_visible(n, size):
+    """[query, key] boolean: 0 <= i - j < size (size 0: plain causal)."""
+    i, j = torch.arange(n)[:, None], torch.arange(n)[None, :]
+    ok = j <= i
+    return ok & (i - j < size) if size else ok
+
+
+def softmax_with_sink(scores, visible, sink=None):
+    """Weights over the visible keys; exp(sink) joins the denominator.  scores [heads, q, k], sink [heads]."""
+    s = scores.masked_fill(~visible, -math.inf)
+    top = s.max(-1, keepdim=True).values
+    if sink is not None:
+        top = torch.maximum(top, sink[:, None, None])
+    p = torch.exp(s - top)
+    den = p.sum(-1, keepdim=True)
+    if sink is not None:
+        den = den + torch.exp(sink[:, None, None] - top)
+    return p / den
+
+
+def latent_kv(h, w_dkv, norm_w, kv_rank, rot_dims, base, eps, positions):
+    """(latent [t, kv_rank], rotated key part [t, rot_dim]) of a layer with its own down-projection."""
+    down = h @ w_dkv.T
+    return rms_norm(down[:, :kv_rank], eps, norm_w), rotate(down[:, kv_rank:], positions, rot_dims, base)
+
+
+def latent_attention(h, latent, k_rot, w, m, positions):
+    """m: dict(heads, dim, rot_dim, vdim, scale, window, rot_dims, base); w: dict(q, uk, uv, o, sink)."""
+    t, H = h.shape[0], m["heads"]
+    q = (h @ w["q"].T).view(t, H, m["dim"] + m["rot_dim"])
+    qn, qr = q[..., :m["dim"]], rotate(q[..., m["dim"]:], positions, m["rot_dims"], m["base"])
+    kn = (latent @ w["uk"].T).view(t, H, m["dim"])
+    v = (latent @ w["uv"].T).view(t, H, m["vdim"])
+    s = (torch.einsum("ihd,jhd->hij", qn, kn) + torch.einsum("ihd,jd->hij", qr, k_rot)) * m["scale"]
+    p = softmax_with_sink(s, window_visible(t, m["window"]), w.get("sink"))
+    o = torch.einsum("hij,jhd->ihd", p, v).reshape(t, H * m["vdim"])
+    return o @ w["o"].T
+
+
+def delta_gates(h, w):
+    """(decay, removal rate), both [t, heads * dim]."""
+    decay = torch.exp(-math.exp(-0.5) * torch.sigmoid(torch.tanh(h @ w["w1"].T) @ w["w2"].T + w["w0"]))
+    return decay, torch.sigmoid(h @ w["a"].T + w["a.b"])
+
+
+def delta_scan(r, k, v, decay, rate, state=None):
+    """Token-by-token recurrence; all inputs [t, heads, dim].  Returns (o [t, heads, dim], state)."""
+    t, H, D = r.shape
+    S = torch.zeros(H, D, D, dtype=r.dtype) if state is None else state.clone()
+    out = []
+    for i in range(t):
+        u = k[i] / torch.sqrt((k[i] ** 2).sum(-1, keepdim=True) + 1e-6)
+        seen = torch.einsum("hd,hde->he", u, S)
+        S = decay[i][:, :, None] * S - (rate[i] * u)[:, :, None] * seen[:, None, :] + k[i][:, :, None] * v[i][:, None, :]
+        out.append(torch.einsum("hde,hd->he", S, r[i]))
+    return torch.stack(out), S
+
+
+def general_delta(h, w, heads, dim, eps):
+    t = h.shape[0]
+    split = lambda x: x.reshape(t, heads, dim)
+    decay, rate = delta_gates(h, w)
+    o, _ = delta_scan(split(h @ w["r"].T), split(h @ w["k"].T), split(h @ w["v"].T), split(decay), split(rate))
+    o = rms_norm(o, eps).reshape(t, heads * dim) * w["norm"]
+    return (o * torch.sigmoid(h @ w["g"].T)) @ w["o"].T
+
+
+def feed_forward(h, w, eps):
+    return poly_norm(h @ w["up"].T, [float(c) for c in w["act"]], eps) @ w["down"].T
+
+
+def forward(config, tensors, tokens, collect=None, dtype=torch.float64):
+    """Logits [tokens, vocab] of one sequence.  `config` is the parsed config.json, `tensors` name -> tensor.
+    `collect`: a list that receives the residual stream after every layer."""
+    eps = float(config["norm"]["eps"])
+    T = {n: x.to(dtype) if x.is_floating_point() else x for n, x in tensors.items()}
+    pos = torch.arange(len(tokens))
+    x = T["embed"][torch.as_tensor(tokens, dtype=torch.long)]
+    kv = {}
+    for i, layer in enumerate(config["layers"]):
+        p, mix = f"l{i}.", layer["mixer"]
+        sub = lambda kind: {n[len(p + kind) + 1:]: t for n, t in T.items() if n.startswith(p + kind + ".")}
+        w = sub("mix")
+        h = rms_norm(x, eps, T[p + "norm1"])
+        if layer["type"] == "latent_attention":
+            rot, src = mix["rot"], mix.get("kv_from")
+            if src is None:
+                kv[i] = latent_kv(h, w["dkv"], w["dkv.norm"], mix["kv_rank"], rot["dims"], rot["base"], eps, pos)
+            c, kr = kv[i if src is None else src]
+            m = dict(heads=mix["heads"], dim=mix["dim"], rot_dim=mix["rot_dim"], vdim=mix["vdim"], scale=mix["scale"],
+                     window=mix["mask"]["size"], rot_dims=rot["dims"], base=rot["base"])
+            y = latent_attention(h, c, kr, w, m, pos)
+        elif layer["type"] == "general_delta":
+            y = general_delta(h, w, mix["heads"], mix["dim"], eps)
+        else:
+            raise ValueError(f"unknown mixer {layer['type']!r}")
+        x = x + rms_norm(y, eps, T[p + "norm1b"])
+        if layer.get("mlp"):
+            y = feed_forward(rms_norm(x, eps, T[p + "norm2"]), sub("mlp"), eps)
+            x = x + rms_norm(y, eps, T[p + "norm2b"])
+        if collect is not None:
+            collect.append(x.clone())
+    return rms_norm(x, eps, T["final.norm"]) @ T["head"].T
