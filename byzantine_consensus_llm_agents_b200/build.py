@@ -31,6 +31,12 @@ SOURCES = [
     "model_step.cu",
     "tp_comm.cu",
     "tp_reduce_norm.cu",
+    "stack_norm.cu",
+    "gemm_simt.cu",
+    "latent_attn.cu",
+    "latent_prefill.cu",
+    "delta_scan.cu",
+    "stack_step.cu",
 ]
 
 NVCC_FLAGS = [

@@ -59,6 +59,7 @@ void set_last_error(const char* what, const char* detail) {
 int model_prefill(const bcg_model* m, const bcg_workspace* ws, const int* ids, const int* positions,
                   const int* slot_map, const int* block_table, int max_blocks, const int* tile_info,
                   int n_tiles, const int* last_rows, int n_seqs, int T, cudaStream_t st);
+int model_head(const bcg_model* m, const bcg_workspace* ws, const int* rows, int n, int row0, cudaStream_t st);
 int model_decode(const bcg_model* m, const bcg_workspace* ws, const int* ids, const int* positions,
                  const int* slot_map, const int* seq_lens, const int* block_table, int max_blocks,
                  int B, int flags, cudaStream_t st);
@@ -194,12 +195,55 @@ int bcg_model_prefill(const bcg_model* m, const bcg_workspace* ws, const int* id
                        n_tiles, last_rows, n_seqs, T, S(stream));
 }
 
+int bcg_model_head(const bcg_model* m, const bcg_workspace* ws, const int* rows, int n, int row0, void* stream) {
+  return model_head(m, ws, rows, n, row0, S(stream));
+}
+
 int bcg_model_decode(const bcg_model* m, const bcg_workspace* ws, const int* ids,
                      const int* positions, const int* slot_map, const int* seq_lens,
                      const int* block_table, int max_blocks_per_seq, int B, int flags,
                      void* stream) {
   return model_decode(m, ws, ids, positions, slot_map, seq_lens, block_table, max_blocks_per_seq, B,
                       flags, S(stream));
+}
+
+int bcg_stack_step(const bcg_stack* m, const bcg_stack_ws* ws, const bcg_step_batch* b, void* stream) {
+  return stack_step(m, ws, b, S(stream));
+}
+
+int bcg_stack_head(const bcg_stack* m, const bcg_stack_ws* ws, const int* rows, int n, int row0, int flags,
+                   void* stream) {
+  return stack_head(m, ws, rows, n, row0, flags, S(stream));
+}
+
+int bcg_gemm_any(const void* X, int x_dtype, const void* W, float* out, int M, int N, int K, long long ldx,
+                 long long ldw, long long ldo, void* stream) {
+  return gemm_any(X, x_dtype, W, out, M, N, K, ldx, ldw, ldo, S(stream));
+}
+
+int bcg_sandwich_norm(float* residual, const float* delta, int n_partials, long long partial_stride,
+                      const float* w_post, const float* w_next, void* xn, int act_dtype, int T, int d, float eps,
+                      void* stream) {
+  return sandwich_norm(residual, delta, n_partials, partial_stride, w_post, w_next, xn, act_dtype, T, d, eps,
+                       S(stream));
+}
+
+int bcg_poly_norm(const float* z, int n_partials, long long partial_stride, const float* coef, void* out,
+                  int act_dtype, int T, int ff, float eps, void* stream) {
+  return poly_norm(z, n_partials, partial_stride, coef, out, act_dtype, T, ff, eps, S(stream));
+}
+
+int bcg_delta_scan(const bcg_layer* l, const float* proj, int n_partials, long long partial_stride, long long ld,
+                   const float* decay, int decay_partials, long long decay_stride, const int* positions,
+                   const int* slot_map, const int* seq_start, const int* state_slots, int n_seqs, void* out,
+                   int act_dtype, float eps, void* stream) {
+  return delta_scan(l, proj, n_partials, partial_stride, ld, decay, decay_partials, decay_stride, positions, slot_map,
+                    seq_start, state_slots, n_seqs, seq_start == nullptr, out, act_dtype, eps, S(stream));
+}
+
+int bcg_latent_attention(const bcg_stack* m, const bcg_stack_ws* ws, const bcg_step_batch* b, int layer, int mode,
+                         void* stream) {
+  return latent_attention(m, ws, b, layer, mode, S(stream));
 }
 
 }  // extern "C"

@@ -62,6 +62,40 @@ int prefill_attn_paged(const void* q, const void* kv_cache, const int* block_tab
 
 int mask_sample(const bcg_sampler_args* a, cudaStream_t stream);
 
+// layer stacks (stack_*.cu, latent_*.cu, delta_scan.cu, gemm_simt.cu); act_dtype = BCG_DT_*
+int embed_norm(const int* ids, const void* embed, const float* w, float* residual, void* xn, int act_dtype, int T,
+               int d, float eps, cudaStream_t stream);
+int rows_norm(const float* residual, const int* rows, const float* w, void* xn, int act_dtype, int n, int d,
+              float eps, cudaStream_t stream);
+int sandwich_norm(float* residual, const float* delta, int n_partials, long long partial_stride,
+                  const float* w_post, const float* w_next, void* xn, int act_dtype, int T, int d, float eps,
+                  cudaStream_t stream);
+int poly_norm(const float* z, int n_partials, long long partial_stride, const float* coef, void* out, int act_dtype,
+              int T, int ff, float eps, cudaStream_t stream);
+int gemm_any(const void* X, int x_dtype, const void* W, float* out, int M, int N, int K, long long ldx,
+             long long ldw, long long ldo, cudaStream_t stream);
+int latent_qkv(const bcg_layer* l, const float* proj, int n_partials, long long pstride, const int* positions,
+               const int* slot_map, void* q, int act_dtype, int T, float eps, cudaStream_t stream);
+int latent_plain(const bcg_layer* l, const void* q, void* out, const bcg_step_batch* b, const int* rows, int n,
+                 int page_size, int act_dtype, cudaStream_t stream);
+bool latent_decode_ok(const bcg_layer* l);
+int latent_decode(const bcg_layer* l, const bcg_stack_ws* ws, const bcg_step_batch* b, int page_size,
+                  cudaStream_t stream);
+int latent_gather(const void* cache, const int* slots, void* out, int n, int crow, cudaStream_t stream);
+bool latent_prefill_ok(const bcg_layer* l);
+int latent_prefill(const bcg_layer* l, const bcg_stack_ws* ws, const bcg_step_batch* b, cudaStream_t stream);
+int delta_low(const bcg_layer* l, const float* proj, int n_partials, long long pstride, void* low, int act_dtype,
+              int T, cudaStream_t stream);
+int delta_scan(const bcg_layer* l, const float* proj, int n_partials, long long pstride, long long ld,
+               const float* decay, int d_partials, long long dstride, const int* positions, const int* slot_map,
+               const int* seq_start, const int* state_slots, int n_seqs, int one_token, void* out, int act_dtype,
+               float eps, cudaStream_t stream);
+int latent_attention(const bcg_stack* m, const bcg_stack_ws* ws, const bcg_step_batch* b, int layer, int mode,
+                     cudaStream_t stream);
+int stack_step(const bcg_stack* m, const bcg_stack_ws* ws, const bcg_step_batch* b, cudaStream_t stream);
+int stack_head(const bcg_stack* m, const bcg_stack_ws* ws, const int* rows, int n, int row0, int flags,
+               cudaStream_t stream);
+
 // tensor parallelism (tp_comm.cu)
 int tp_unique_id(void* out128);
 int tp_init(const void* id128, int rank, int size);

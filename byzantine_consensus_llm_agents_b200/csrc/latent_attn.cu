@@ -1,0 +1,554 @@
+// Latent (compressed-KV) attention over paged latents, sliding window and softmax sink.
+//
+// A cache row holds one token's latent c [kv_rank] and the rotated key part shared by all heads [rot_dim].
+// A head's key is (W_uk c, k_rot) and its value W_uv c, so with q~ = W_uk^T q the score is q~ . c + q_rot . k_rot
+// and the output W_uv (sum_j p_j c_j): attention can run in latent space, where all heads share the keys.
+//   latent_qkv        projection slabs -> rotated queries; latent norm + rotation -> cache row
+//   latent_plain      one CTA per (token, head), latent space, any sizes, fp32 or bf16: the fp32 engine's
+//                     kernel, and the bf16 one's for sizes the kernels below do not take
+//   latent_absorb     q~ for single tokens (decode), W_uk tile staged ahead of the dependency wait
+//   latent_decode     split-KV: one CTA per (key chunk, token), mma.sync over 32-head groups
+//   latent_up         chunks combined, then W_uv
+//   latent_gather     cache rows -> contiguous rows for the expanded (prefill) form, latent_prefill.cu
+#include "stack_common.cuh"
+#include "kernels.h"
+
+namespace bcg {
+
+// ------------------------------------------------------------------------------------------- q, k, v
+constexpr int kQkvThreads = 256;
+
+// grid (T, head groups of 8 [+ 1 for the cache row]); a warp per head.
+template <typename T>
+__global__ void __launch_bounds__(kQkvThreads)
+latent_qkv_kernel(const float* __restrict__ proj, int n_partials, long long pstride, long long ld,
+                  const int* __restrict__ positions, const int* __restrict__ slot_map,
+                  const float* __restrict__ cos_sin, const float* __restrict__ latent_norm, T* __restrict__ q,
+                  T* __restrict__ cache, int heads, int dim, int rot_dim, int rot_dims, int q_row, int kv_rank,
+                  int q_groups, float eps) {
+  extern __shared__ float stage[];    // latent
+  __shared__ RowSum<kQkvThreads, 1, 1> sh;
+  pdl_launch_dependents();
+  pdl_wait();
+  const long long t = blockIdx.x;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const float* row = proj + t * ld;
+  const float* cs = cos_sin + static_cast<long long>(positions[t]) * rot_dims;
+  const int half = rot_dims >> 1;
+  auto rotated = [&](const float* x, int i) {   // element i of the rotated part whose first element is x
+    const float a = slab_sum(x + i, n_partials, pstride);
+    if (i >= rot_dims) return a;
+    const int f = i < half ? i : i - half;
+    const float b = slab_sum(x + (i < half ? i + half : i - half), n_partials, pstride);
+    const float c = cs[f], s = cs[half + f];
+    return i < half ? a * c - b * s : a * c + b * s;
+  };
+  if (static_cast<int>(blockIdx.y) < q_groups) {
+    const int h = blockIdx.y * (kQkvThreads / 32) + warp;
+    if (h >= heads) return;
+    const float* x = row + static_cast<long long>(h) * (dim + rot_dim);
+    T* dst = q + (t * heads + h) * q_row;
+    for (int i = lane; i < q_row; i += 32) {
+      float v = 0.f;
+      if (i < dim) v = slab_sum(x + i, n_partials, pstride);
+      else if (i < dim + rot_dim) v = rotated(x + dim, i - dim);
+      dst[i] = from_f32<T>(v);
+    }
+    return;
+  }
+  const int slot = slot_map[t];
+  if (slot < 0) return;
+  const float* x = row + static_cast<long long>(heads) * (dim + rot_dim);
+  float ss[1] = {0.f};
+  for (int i = threadIdx.x; i < kv_rank; i += kQkvThreads) {
+    const float v = slab_sum(x + i, n_partials, pstride);
+    stage[i] = v;
+    ss[0] += v * v;
+  }
+  row_sum<kQkvThreads, 1, 1>(sh, ss, 0);
+  const float inv = rsqrtf(ss[0] / static_cast<float>(kv_rank) + eps);
+  T* dst = cache + static_cast<long long>(slot) * (kv_rank + rot_dim);
+  for (int i = threadIdx.x; i < kv_rank; i += kQkvThreads) dst[i] = from_f32<T>(stage[i] * inv * latent_norm[i]);
+  for (int i = threadIdx.x; i < rot_dim; i += kQkvThreads) dst[kv_rank + i] = from_f32<T>(rotated(x + kv_rank, i));
+}
+
+int latent_qkv(const bcg_layer* l, const float* proj, int n_partials, long long pstride, const int* positions,
+               const int* slot_map, void* q, int act_dtype, int T, float eps, cudaStream_t st) {
+  const int groups = (l->heads + kQkvThreads / 32 - 1) / (kQkvThreads / 32);
+  const int q_row = l->q_ld > 0 ? l->q_ld : l->dim + l->rot_dim;
+  const dim3 grid(T, groups + (l->owns_cache ? 1 : 0));
+  const size_t sm = static_cast<size_t>(l->kv_rank) * 4;
+  if (act_dtype == BCG_DT_F32)
+    BCG_CUDA_CHECK(launch_k(latent_qkv_kernel<float>, grid, dim3(kQkvThreads), sm, st, proj, n_partials, pstride,
+                            static_cast<long long>(l->n_in), positions, slot_map, l->cos_sin, l->latent_norm,
+                            static_cast<float*>(q), static_cast<float*>(l->cache), l->heads, l->dim, l->rot_dim,
+                            l->rot_dims, q_row, l->kv_rank, groups, eps));
+  else
+    BCG_CUDA_CHECK(launch_k(latent_qkv_kernel<__nv_bfloat16>, grid, dim3(kQkvThreads), sm, st, proj, n_partials,
+                            pstride, static_cast<long long>(l->n_in), positions, slot_map, l->cos_sin,
+                            l->latent_norm, static_cast<__nv_bfloat16*>(q), static_cast<__nv_bfloat16*>(l->cache),
+                            l->heads, l->dim, l->rot_dim, l->rot_dims, q_row, l->kv_rank, groups, eps));
+  return BCG_OK;
+}
+
+// ------------------------------------------------------------------------------------------- plain
+constexpr int kPlainThreads = 128;
+constexpr int kPlainKeys = 256;
+
+template <typename T>
+__global__ void __launch_bounds__(kPlainThreads)
+latent_plain_kernel(const T* __restrict__ q, const T* __restrict__ cache, const __nv_bfloat16* __restrict__ w_uk,
+                    const __nv_bfloat16* __restrict__ w_uv, const float* __restrict__ sink,
+                    const int* __restrict__ rows, const int* __restrict__ positions, const int* __restrict__ row_seq,
+                    const int* __restrict__ block_table, int max_blocks, int page_size, T* __restrict__ out,
+                    int heads, int dim, int rot_dim, int vdim, int kv_rank, int q_row, int window, float scale) {
+  extern __shared__ float sm[];
+  __shared__ float red[kPlainThreads / 32];
+  const int crow = kv_rank + rot_dim;
+  float* qa = sm;                 // [kv_rank | rot_dim] query in latent space
+  float* oc = qa + crow;          // [kv_rank]
+  float* qs = oc + kv_rank;       // [dim]
+  float* p = qs + dim;            // [kPlainKeys]
+  pdl_launch_dependents();
+  pdl_wait();
+  const long long t = rows ? rows[blockIdx.x] : blockIdx.x;
+  const int h = blockIdx.y;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int pos = positions[t];
+  const int* bt = block_table + static_cast<long long>(row_seq ? row_seq[t] : t) * max_blocks;
+  const T* qh = q + (t * heads + h) * q_row;
+  for (int i = threadIdx.x; i < dim; i += kPlainThreads) qs[i] = to_f32<T>(qh[i]);
+  for (int i = threadIdx.x; i < rot_dim; i += kPlainThreads) qa[kv_rank + i] = to_f32<T>(qh[dim + i]);
+  __syncthreads();
+  for (int r = threadIdx.x; r < kv_rank; r += kPlainThreads) {
+    float acc = 0.f;
+    const __nv_bfloat16* w = w_uk + static_cast<long long>(h) * dim * kv_rank + r;
+    for (int i = 0; i < dim; ++i) acc = fmaf(qs[i], __bfloat162float(w[static_cast<long long>(i) * kv_rank]), acc);
+    qa[r] = acc;
+    oc[r] = 0.f;
+  }
+  float m = sink ? sink[h] : -INFINITY, l = sink ? 1.0f : 0.0f;
+  const int lo = window > 0 ? max(0, pos - window + 1) : 0;
+  for (int j0 = lo; j0 <= pos; j0 += kPlainKeys) {
+    const int n = min(kPlainKeys, pos + 1 - j0);
+    __syncthreads();
+    float mx = -INFINITY;
+    for (int j = warp; j < n; j += kPlainThreads / 32) {
+      const int key = j0 + j;
+      const T* c = cache + (static_cast<long long>(bt[key / page_size]) * page_size + key % page_size) * crow;
+      float s = 0.f;
+      for (int i = lane; i < crow; i += 32) s = fmaf(qa[i], to_f32<T>(c[i]), s);
+      s = warp_sum(s) * scale;
+      if (lane == 0) p[j] = s;
+      mx = fmaxf(mx, s);
+    }
+    if (lane == 0) red[warp] = mx;
+    __syncthreads();
+#pragma unroll
+    for (int i = 0; i < kPlainThreads / 32; ++i) mx = fmaxf(mx, red[i]);
+    const float m_new = fmaxf(m, mx);
+    const float corr = expf(m - m_new);
+    float sum = 0.f;
+    for (int j = threadIdx.x; j < n; j += kPlainThreads) {
+      const float e = expf(p[j] - m_new);
+      p[j] = e;
+      sum += e;
+    }
+    sum = warp_sum(sum);
+    __syncthreads();
+    if (lane == 0) red[warp] = sum;
+    __syncthreads();
+    sum = 0.f;
+#pragma unroll
+    for (int i = 0; i < kPlainThreads / 32; ++i) sum += red[i];
+    l = l * corr + sum;
+    m = m_new;
+    for (int r = threadIdx.x; r < kv_rank; r += kPlainThreads) {
+      float acc = oc[r] * corr;
+      for (int j = 0; j < n; ++j) {
+        const int key = j0 + j;
+        acc = fmaf(p[j], to_f32<T>(cache[(static_cast<long long>(bt[key / page_size]) * page_size + key % page_size) * crow + r]), acc);
+      }
+      oc[r] = acc;
+    }
+  }
+  __syncthreads();
+  const float inv = 1.0f / l;
+  for (int v = warp; v < vdim; v += kPlainThreads / 32) {
+    const __nv_bfloat16* w = w_uv + (static_cast<long long>(h) * vdim + v) * kv_rank;
+    float acc = 0.f;
+    for (int r = lane; r < kv_rank; r += 32) acc = fmaf(__bfloat162float(w[r]), oc[r], acc);
+    acc = warp_sum(acc);
+    if (lane == 0) out[(t * heads + h) * vdim + v] = from_f32<T>(acc * inv);
+  }
+}
+
+int latent_plain(const bcg_layer* l, const void* q, void* out, const bcg_step_batch* b, const int* rows, int n,
+                 int page_size, int act_dtype, cudaStream_t st) {
+  const int q_row = l->q_ld > 0 ? l->q_ld : l->dim + l->rot_dim;
+  const int sm = (2 * l->kv_rank + l->rot_dim + l->dim + kPlainKeys) * 4;
+  const auto* uk = static_cast<const __nv_bfloat16*>(l->w_uk);
+  const auto* uv = static_cast<const __nv_bfloat16*>(l->w_uv);
+  const dim3 grid(n, l->heads);
+  if (act_dtype == BCG_DT_F32) {
+    BCG_TRY(ensure_dynamic_smem(reinterpret_cast<const void*>(latent_plain_kernel<float>), 64 * 1024));
+    BCG_CUDA_CHECK(launch_k(latent_plain_kernel<float>, grid, dim3(kPlainThreads), sm, st, static_cast<const float*>(q),
+                            static_cast<const float*>(l->cache), uk, uv, l->sink, rows, b->positions, b->row_seq,
+                            b->block_table, b->max_blocks, page_size, static_cast<float*>(out), l->heads, l->dim,
+                            l->rot_dim, l->vdim, l->kv_rank, q_row, l->window, l->scale));
+  } else {
+    BCG_TRY(ensure_dynamic_smem(reinterpret_cast<const void*>(latent_plain_kernel<__nv_bfloat16>), 64 * 1024));
+    BCG_CUDA_CHECK(launch_k(latent_plain_kernel<__nv_bfloat16>, grid, dim3(kPlainThreads), sm, st,
+                            static_cast<const __nv_bfloat16*>(q), static_cast<const __nv_bfloat16*>(l->cache), uk, uv,
+                            l->sink, rows, b->positions, b->row_seq, b->block_table, b->max_blocks, page_size,
+                            static_cast<__nv_bfloat16*>(out), l->heads, l->dim, l->rot_dim, l->vdim, l->kv_rank,
+                            q_row, l->window, l->scale));
+  }
+  return BCG_OK;
+}
+
+// ------------------------------------------------------------------------------------------- absorb
+// q_latent[i, h] = (W_uk^T q_unrotated, q_rotated) for single token i = rows[i].
+constexpr int kAbCols = 128;    // latent columns per CTA
+constexpr int kAbRows = 8;      // tokens per pass
+
+__global__ void __launch_bounds__(128)
+latent_absorb_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __restrict__ w_uk,
+                     const int* __restrict__ rows, int n, __nv_bfloat16* __restrict__ q_latent, int heads, int dim,
+                     int rot_dim, int kv_rank, int q_row) {
+  extern __shared__ __align__(16) uint8_t ab_raw[];
+  __nv_bfloat16* wt = reinterpret_cast<__nv_bfloat16*>(ab_raw);                       // [dim][128]
+  float* qs = reinterpret_cast<float*>(ab_raw + static_cast<size_t>(dim) * kAbCols * 2);   // [8][dim]
+  pdl_launch_dependents();
+  const int h = blockIdx.x, c0 = blockIdx.y * kAbCols;
+  const int crow = kv_rank + rot_dim;
+  for (int i = threadIdx.x; i < dim * (kAbCols / 8); i += 128) {
+    const int d = i / (kAbCols / 8), c = c0 + (i % (kAbCols / 8)) * 8;
+    uint4 v = make_uint4(0, 0, 0, 0);
+    if (c < kv_rank) v = *reinterpret_cast<const uint4*>(w_uk + (static_cast<long long>(h) * dim + d) * kv_rank + c);
+    reinterpret_cast<uint4*>(wt)[i] = v;
+  }
+  pdl_wait();
+  for (int r0 = 0; r0 < n; r0 += kAbRows) {
+    const int nr = min(kAbRows, n - r0);
+    __syncthreads();
+    for (int i = threadIdx.x; i < nr * dim; i += 128) {
+      const int r = i / dim, d = i - r * dim;
+      const long long t = rows ? rows[r0 + r] : r0 + r;
+      qs[i] = __bfloat162float(q[(t * heads + h) * q_row + d]);
+    }
+    __syncthreads();
+    // thread = 2 columns x half of the pass's tokens
+    const int c = (threadIdx.x & 63) * 2, rh = (threadIdx.x >> 6) * (kAbRows / 2);
+    float acc[kAbRows / 2][2] = {};
+    for (int d = 0; d < dim; ++d) {
+      const uint32_t w = *reinterpret_cast<const uint32_t*>(wt + d * kAbCols + c);
+      const float w0 = bf16lo(w), w1 = bf16hi(w);
+#pragma unroll
+      for (int r = 0; r < kAbRows / 2; ++r) {
+        const float x = qs[min(rh + r, nr - 1) * dim + d];
+        acc[r][0] = fmaf(x, w0, acc[r][0]);
+        acc[r][1] = fmaf(x, w1, acc[r][1]);
+      }
+    }
+#pragma unroll
+    for (int r = 0; r < kAbRows / 2; ++r)
+      if (rh + r < nr && c0 + c < kv_rank)
+        *reinterpret_cast<uint32_t*>(q_latent + (static_cast<long long>(r0 + rh + r) * heads + h) * crow + c0 + c) =
+            pack_bf16(acc[r][0], acc[r][1]);
+    if (blockIdx.y == 0) {
+      for (int i = threadIdx.x; i < nr * rot_dim; i += 128) {
+        const int r = i / rot_dim, d = i - r * rot_dim;
+        const long long t = rows ? rows[r0 + r] : r0 + r;
+        q_latent[(static_cast<long long>(r0 + r) * heads + h) * crow + kv_rank + d] = q[(t * heads + h) * q_row + dim + d];
+      }
+    }
+  }
+}
+
+// ------------------------------------------------------------------------------------------- decode
+// grid (chunks, tokens, head groups of 32).  Chunk c of a token covers keys [c * 64, c * 64 + 64) counted
+// from the chunk-aligned start of its window.
+constexpr int kLdKeys = 64, kLdHeads = 32, kLdThreads = 128;
+
+__device__ __forceinline__ void cp_async16(void* dst, const void* src) {
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(smem_u32(dst)), "l"(src) : "memory");
+}
+__device__ __forceinline__ void cp_async_wait_all() { asm volatile("cp.async.wait_all;" ::: "memory"); }
+__device__ __forceinline__ void ldsm_x4(uint32_t (&r)[4], const void* p) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0, %1, %2, %3}, [%4];"
+               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3])
+               : "r"(smem_u32(p)));
+}
+__device__ __forceinline__ void ldsm_x4_trans(uint32_t (&r)[4], const void* p) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0, %1, %2, %3}, [%4];"
+               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3])
+               : "r"(smem_u32(p)));
+}
+__device__ __forceinline__ void mma_bf16_16816(float (&d)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
+  asm volatile(
+      "mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0, %1, %2, %3}, {%4, %5, %6, %7}, {%8, %9}, "
+      "{%0, %1, %2, %3};"
+      : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3])
+      : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
+}
+
+__host__ __device__ constexpr int latent_decode_smem(int crow) {
+  return (kLdKeys + kLdHeads) * (crow + 8) * 2 + kLdHeads * (kLdKeys + 4) * 4 + kLdHeads * (kLdKeys + 8) * 2;
+}
+
+__global__ void __launch_bounds__(kLdThreads)
+latent_decode_kernel(const __nv_bfloat16* __restrict__ q_latent, const __nv_bfloat16* __restrict__ cache,
+                     const int* __restrict__ rows, const int* __restrict__ positions,
+                     const int* __restrict__ row_seq, const int* __restrict__ block_table, int max_blocks,
+                     int page_size, float* __restrict__ part_o, float* __restrict__ part_ml, int heads, int kv_rank,
+                     int rot_dim, int window, float scale) {
+  extern __shared__ __align__(16) uint8_t ld_raw[];
+  const int crow = kv_rank + rot_dim, srow = crow + 8;     // +16 bytes: ldmatrix rows on different banks
+  __nv_bfloat16* ks = reinterpret_cast<__nv_bfloat16*>(ld_raw);   // [64][srow]
+  __nv_bfloat16* qs = ks + kLdKeys * srow;                        // [32][srow]
+  float* ss = reinterpret_cast<float*>(qs + kLdHeads * srow);     // [32][68]
+  __nv_bfloat16* ps = reinterpret_cast<__nv_bfloat16*>(ss + kLdHeads * (kLdKeys + 4));   // [32][72]
+  constexpr int kSs = kLdKeys + 4, kPs = kLdKeys + 8;
+  pdl_launch_dependents();
+  pdl_wait();
+  const int i_tok = blockIdx.y, h0 = blockIdx.z * kLdHeads;
+  const int t = rows ? rows[i_tok] : i_tok;
+  const int pos = positions[t];
+  const int lo = window > 0 ? max(0, pos - window + 1) : 0;
+  const int base = (lo / kLdKeys + blockIdx.x) * kLdKeys;
+  if (base > pos) return;
+  const int nh = min(kLdHeads, heads - h0);
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int* bt = block_table + static_cast<long long>(row_seq ? row_seq[t] : t) * max_blocks;
+  const int vec = crow >> 3;
+  for (int k = warp; k < kLdKeys; k += kLdThreads / 32) {
+    const int key = base + k;
+    __nv_bfloat16* dst = ks + k * srow;
+    if (key >= lo && key <= pos) {
+      const __nv_bfloat16* src = cache + (static_cast<long long>(bt[key / page_size]) * page_size + key % page_size) * crow;
+      for (int i = lane; i < vec; i += 32) cp_async16(dst + i * 8, src + i * 8);
+    } else {   // outside the window or not written: finite zeros, masked below
+      for (int i = lane; i < vec; i += 32) *reinterpret_cast<uint4*>(dst + i * 8) = make_uint4(0, 0, 0, 0);
+    }
+  }
+  const __nv_bfloat16* qsrc = q_latent + (static_cast<long long>(i_tok) * heads + h0) * crow;
+  for (int r = warp; r < kLdHeads; r += kLdThreads / 32)
+    for (int i = lane; i < vec; i += 32) {
+      if (r < nh) cp_async16(qs + r * srow + i * 8, qsrc + static_cast<long long>(r) * crow + i * 8);
+      else *reinterpret_cast<uint4*>(qs + r * srow + i * 8) = make_uint4(0, 0, 0, 0);
+    }
+  cp_async_wait_all();
+  __syncthreads();
+  const int mt = nh > 16 ? 2 : 1;
+  {   // scores: each warp 16 keys x all heads of the group
+    float acc[2][2][4] = {};
+    const int kr = warp * 16 + (lane & 7) + ((lane >> 4) << 3), kc = ((lane >> 3) & 1) * 8;
+    const int ar = lane & 15, ac = (lane >> 4) * 8;
+    for (int k = 0; k < crow; k += 16) {
+      uint32_t bq[4], a0[4], a1[4];
+      ldsm_x4(bq, ks + kr * srow + k + kc);
+      ldsm_x4(a0, qs + ar * srow + k + ac);
+      mma_bf16_16816(acc[0][0], a0, bq[0], bq[1]);
+      mma_bf16_16816(acc[0][1], a0, bq[2], bq[3]);
+      if (mt == 2) {
+        ldsm_x4(a1, qs + (16 + ar) * srow + k + ac);
+        mma_bf16_16816(acc[1][0], a1, bq[0], bq[1]);
+        mma_bf16_16816(acc[1][1], a1, bq[2], bq[3]);
+      }
+    }
+#pragma unroll
+    for (int m = 0; m < 2; ++m)
+#pragma unroll
+      for (int n = 0; n < 2; ++n)
+#pragma unroll
+        for (int e = 0; e < 4; ++e)
+          ss[(m * 16 + (lane >> 2) + (e >> 1) * 8) * kSs + warp * 16 + n * 8 + (lane & 3) * 2 + (e & 1)] = acc[m][n][e] * scale;
+  }
+  __syncthreads();
+  const long long chunk = static_cast<long long>(i_tok) * gridDim.x + blockIdx.x;
+  for (int r = warp; r < kLdHeads; r += kLdThreads / 32) {   // softmax of the chunk, one warp per head
+    const int k0 = base + lane, k1 = k0 + 32;
+    const bool ok0 = k0 >= lo && k0 <= pos, ok1 = k1 >= lo && k1 <= pos;
+    const float s0 = ok0 ? ss[r * kSs + lane] : -INFINITY, s1 = ok1 ? ss[r * kSs + lane + 32] : -INFINITY;
+    const float m = warp_max(fmaxf(s0, s1));     // some key of [base, base + 64) is visible, so m is finite
+    const float p0 = ok0 ? __expf(s0 - m) : 0.f, p1 = ok1 ? __expf(s1 - m) : 0.f;
+    ps[r * kPs + lane] = __float2bfloat16(p0);
+    ps[r * kPs + lane + 32] = __float2bfloat16(p1);
+    const float l = warp_sum(p0 + p1);
+    if (lane == 0 && r < nh) {
+      part_ml[(chunk * heads + h0 + r) * 2] = m;
+      part_ml[(chunk * heads + h0 + r) * 2 + 1] = l;
+    }
+  }
+  __syncthreads();
+  uint32_t pa[2][4][4];
+#pragma unroll
+  for (int m = 0; m < 2; ++m)
+#pragma unroll
+    for (int k = 0; k < 4; ++k)
+      ldsm_x4(pa[m][k], ps + (m * 16 + (lane & 15)) * kPs + k * 16 + (lane >> 4) * 8);
+  for (int n0 = warp * 16; n0 < kv_rank; n0 += (kLdThreads / 32) * 16) {   // 16 latent columns per turn
+    float acc[2][2][4] = {};
+#pragma unroll
+    for (int k = 0; k < 4; ++k) {
+      uint32_t bv[4];
+      ldsm_x4_trans(bv, ks + (k * 16 + (lane & 15)) * srow + n0 + (lane >> 4) * 8);
+      mma_bf16_16816(acc[0][0], pa[0][k], bv[0], bv[1]);
+      mma_bf16_16816(acc[0][1], pa[0][k], bv[2], bv[3]);
+      if (mt == 2) {
+        mma_bf16_16816(acc[1][0], pa[1][k], bv[0], bv[1]);
+        mma_bf16_16816(acc[1][1], pa[1][k], bv[2], bv[3]);
+      }
+    }
+#pragma unroll
+    for (int m = 0; m < 2; ++m)
+#pragma unroll
+      for (int n = 0; n < 2; ++n)
+#pragma unroll
+        for (int e = 0; e < 2; ++e) {
+          const int r = m * 16 + (lane >> 2) + e * 8;
+          if (r < nh)
+            *reinterpret_cast<float2*>(part_o + (chunk * heads + h0 + r) * kv_rank + n0 + n * 8 + (lane & 3) * 2) =
+                make_float2(acc[m][n][2 * e], acc[m][n][2 * e + 1]);
+        }
+  }
+}
+
+// o_latent[i, h] = sum over chunks (and the sink's share of the denominator), bf16.  grid (tokens, heads).
+__global__ void __launch_bounds__(128)
+latent_combine_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml,
+                      const float* __restrict__ sink, const int* __restrict__ rows,
+                      const int* __restrict__ positions, __nv_bfloat16* __restrict__ o_latent, int chunks, int heads,
+                      int kv_rank, int window) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const int i_tok = blockIdx.x, h = blockIdx.y;
+  const int pos = positions[rows ? rows[i_tok] : i_tok];
+  const int lo = window > 0 ? max(0, pos - window + 1) : 0;
+  const int n = min(chunks, pos / kLdKeys - lo / kLdKeys + 1);
+  const float* ml = part_ml + (static_cast<long long>(i_tok) * chunks * heads + h) * 2;
+  float m = sink ? sink[h] : -INFINITY;
+  for (int c = 0; c < n; ++c) m = fmaxf(m, ml[static_cast<long long>(c) * heads * 2]);
+  float l = sink ? __expf(sink[h] - m) : 0.f;
+  for (int c = 0; c < n; ++c)
+    l += __expf(ml[static_cast<long long>(c) * heads * 2] - m) * ml[static_cast<long long>(c) * heads * 2 + 1];
+  const float inv = 1.0f / l;
+  for (int r = threadIdx.x; r < kv_rank; r += 128) {
+    float acc = 0.f;
+#pragma unroll 4
+    for (int c = 0; c < n; ++c)
+      acc = fmaf(__expf(ml[static_cast<long long>(c) * heads * 2] - m),
+                 part_o[((static_cast<long long>(i_tok) * chunks + c) * heads + h) * kv_rank + r], acc);
+    o_latent[(static_cast<long long>(i_tok) * heads + h) * kv_rank + r] = __float2bfloat16(acc * inv);
+  }
+}
+
+// out[t, h, v] = W_uv o_latent.  grid (heads, v tiles of 32); the weight tile is staged ahead of the wait.
+constexpr int kUpRows = 32;
+
+__global__ void __launch_bounds__(128)
+latent_up_kernel(const __nv_bfloat16* __restrict__ o_latent, const __nv_bfloat16* __restrict__ w_uv,
+                 const int* __restrict__ rows, int n, __nv_bfloat16* __restrict__ out, int heads, int vdim,
+                 int kv_rank) {
+  extern __shared__ __align__(16) uint8_t up_raw[];
+  __nv_bfloat16* wt = reinterpret_cast<__nv_bfloat16*>(up_raw);   // [32][kv_rank]
+  pdl_launch_dependents();
+  const int h = blockIdx.x, v0 = blockIdx.y * kUpRows;
+  const int nv = min(kUpRows, vdim - v0);
+  const uint4* src = reinterpret_cast<const uint4*>(w_uv + (static_cast<long long>(h) * vdim + v0) * kv_rank);
+  for (int i = threadIdx.x; i < nv * (kv_rank / 8); i += 128) reinterpret_cast<uint4*>(wt)[i] = src[i];
+  pdl_wait();
+  __syncthreads();
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  for (int i = warp; i < n; i += 4) {          // a warp per token, lanes across the latent
+    const long long t = rows ? rows[i] : i;
+    const __nv_bfloat16* o = o_latent + (static_cast<long long>(i) * heads + h) * kv_rank;
+    float mine = 0.f;
+    for (int vb = 0; vb < nv; vb += 8) {
+      float acc[8] = {};
+      for (int r = lane * 2; r < kv_rank; r += 64) {
+        const uint32_t ow = *reinterpret_cast<const uint32_t*>(o + r);
+        const float o0 = bf16lo(ow), o1 = bf16hi(ow);
+#pragma unroll
+        for (int v = 0; v < 8; ++v) {
+          const uint32_t w = *reinterpret_cast<const uint32_t*>(wt + min(vb + v, nv - 1) * kv_rank + r);
+          acc[v] = fmaf(bf16lo(w), o0, fmaf(bf16hi(w), o1, acc[v]));
+        }
+      }
+#pragma unroll
+      for (int v = 0; v < 8; ++v) {
+        const float s = warp_sum(acc[v]);
+        if (lane == vb + v) mine = s;
+      }
+    }
+    if (lane < nv) out[(t * heads + h) * vdim + v0 + lane] = __float2bfloat16(mine);
+  }
+}
+
+// Sizes the latent-space tensor-core path takes.
+bool latent_decode_ok(const bcg_layer* l) {
+  const int crow = l->kv_rank + l->rot_dim;
+  return l->kv_rank % 16 == 0 && crow % 16 == 0 && l->rot_dim % 8 == 0 && latent_decode_smem(crow) <= 220 * 1024 &&
+         l->dim * kAbCols * 2 + kAbRows * l->dim * 4 <= 200 * 1024 && kUpRows * l->kv_rank * 2 <= 200 * 1024;
+}
+
+int latent_decode_chunks(const bcg_layer* l, int max_context) {
+  const int span = l->window > 0 && l->window < max_context ? l->window : max_context;
+  return span / kLdKeys + 2 < (max_context + kLdKeys - 1) / kLdKeys ? span / kLdKeys + 2
+                                                                    : (max_context + kLdKeys - 1) / kLdKeys;
+}
+
+int latent_decode(const bcg_layer* l, const bcg_stack_ws* ws, const bcg_step_batch* b, int page_size,
+                  cudaStream_t st) {
+  const int n = b->single_rows ? b->n_single : b->T;
+  const int crow = l->kv_rank + l->rot_dim;
+  const int q_row = l->q_ld > 0 ? l->q_ld : l->dim + l->rot_dim;
+  const int chunks = latent_decode_chunks(l, b->max_context);
+  if (n > ws->D_max || n > 65535 || static_cast<long long>(n) * chunks * l->heads * l->kv_rank > ws->part_floats) {
+    set_last_error("bcg_latent_attention", "single tokens x chunks exceed the decode scratch");
+    return BCG_ERR_TOO_LARGE;
+  }
+  auto* ql = static_cast<__nv_bfloat16*>(ws->q_latent);
+  auto* ol = static_cast<__nv_bfloat16*>(ws->o_latent);
+  const size_t sm_a = static_cast<size_t>(l->dim) * kAbCols * 2 + kAbRows * l->dim * 4;
+  const size_t sm_u = static_cast<size_t>(kUpRows) * l->kv_rank * 2;
+  BCG_TRY(ensure_dynamic_smem(reinterpret_cast<const void*>(latent_absorb_kernel), 200 * 1024));
+  BCG_TRY(ensure_dynamic_smem(reinterpret_cast<const void*>(latent_decode_kernel), 220 * 1024));
+  BCG_TRY(ensure_dynamic_smem(reinterpret_cast<const void*>(latent_up_kernel), 200 * 1024));
+  BCG_CUDA_CHECK(launch_k(latent_absorb_kernel, dim3(l->heads, (l->kv_rank + kAbCols - 1) / kAbCols), dim3(128), sm_a,
+                          st, static_cast<const __nv_bfloat16*>(ws->q), static_cast<const __nv_bfloat16*>(l->w_uk),
+                          b->single_rows, n, ql, l->heads, l->dim, l->rot_dim, l->kv_rank, q_row));
+  BCG_CUDA_CHECK(launch_k(latent_decode_kernel, dim3(chunks, n, (l->heads + kLdHeads - 1) / kLdHeads), dim3(kLdThreads),
+                          latent_decode_smem(crow), st, ql, static_cast<const __nv_bfloat16*>(l->cache),
+                          b->single_rows, b->positions, b->row_seq, b->block_table, b->max_blocks, page_size,
+                          ws->part_o, ws->part_ml, l->heads, l->kv_rank, l->rot_dim, l->window, l->scale));
+  BCG_CUDA_CHECK(launch_k(latent_combine_kernel, dim3(n, l->heads), dim3(128), 0, st, ws->part_o, ws->part_ml, l->sink,
+                          b->single_rows, b->positions, ol, chunks, l->heads, l->kv_rank, l->window));
+  BCG_CUDA_CHECK(launch_k(latent_up_kernel, dim3(l->heads, (l->vdim + kUpRows - 1) / kUpRows), dim3(128), sm_u, st, ol,
+                          static_cast<const __nv_bfloat16*>(l->w_uv), b->single_rows, n,
+                          static_cast<__nv_bfloat16*>(ws->mix), l->heads, l->vdim, l->kv_rank));
+  return BCG_OK;
+}
+
+// ------------------------------------------------------------------------------------------- gather
+__global__ void __launch_bounds__(128)
+latent_gather_kernel(const __nv_bfloat16* __restrict__ cache, const int* __restrict__ slots,
+                     __nv_bfloat16* __restrict__ out, int n, int crow) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const long long r = static_cast<long long>(blockIdx.x) * 4 + warp;
+  if (r >= n) return;
+  const uint4* src = reinterpret_cast<const uint4*>(cache + static_cast<long long>(slots[r]) * crow);
+  uint4* dst = reinterpret_cast<uint4*>(out + r * crow);
+  for (int i = lane; i < crow / 8; i += 32) dst[i] = src[i];
+}
+
+int latent_gather(const void* cache, const int* slots, void* out, int n, int crow, cudaStream_t st) {
+  BCG_CUDA_CHECK(launch_k(latent_gather_kernel, dim3((n + 3) / 4), dim3(128), 0, st,
+                          static_cast<const __nv_bfloat16*>(cache), slots, static_cast<__nv_bfloat16*>(out), n, crow));
+  return BCG_OK;
+}
+
+}  // namespace bcg

@@ -25,6 +25,22 @@ static int check_model(const bcg_model* m, const bcg_workspace* ws) {
   return BCG_OK;
 }
 
+// Final norm + lm_head of `n` tokens of the prefill step just run, into logits rows row0.. .
+int model_head(const bcg_model* m, const bcg_workspace* ws, const int* rows, int n, int row0, cudaStream_t st) {
+  BCG_TRY(check_model(m, ws));
+  if (!rows || !ws->delta || n <= 0 || row0 < 0 || row0 + n > ws->B_max) {
+    set_last_error("bcg_model_head", "rows exceed the logits buffer");
+    return BCG_ERR_TOO_LARGE;
+  }
+  const int d = m->d_model;
+  BCG_TRY(add_rmsnorm(ws->residual, ws->delta, 1, 1, 0, m->final_norm, ws->xn_last, rows, n, d, m->rms_eps, st));
+  // With tensor parallelism m->vocab is this rank's shard and the logits stay sharded: the sampler
+  // exchanges one candidate per row instead (bcg_sampler_args.tp_size).
+  BCG_TRY(gemm_bf16_tn(ws->xn_last, m->lm_head, ws->logits + static_cast<long long>(row0) * m->vocab, n, m->vocab, d, d,
+                       d, m->vocab, BCG_EPI_F32, 1, 0, st));
+  return BCG_OK;
+}
+
 int model_prefill(const bcg_model* m, const bcg_workspace* ws, const int* ids, const int* positions,
                   const int* slot_map, const int* block_table, int max_blocks, const int* tile_info,
                   int n_tiles, const int* last_rows, int n_seqs, int T, cudaStream_t st) {
@@ -67,13 +83,7 @@ int model_prefill(const bcg_model* m, const bcg_workspace* ws, const int* ids, c
                          BCG_EPI_F32, 1, 0, st));
     if (tp > 1) BCG_TRY(tp_all_reduce_f32(ws->delta, static_cast<long long>(T) * d, st));
   }
-  BCG_TRY(add_rmsnorm(ws->residual, ws->delta, 1, 1, 0, m->final_norm, ws->xn_last, last_rows,
-                      n_seqs, d, m->rms_eps, st));
-  // With tensor parallelism m->vocab is this rank's shard and the logits stay sharded: the sampler
-  // exchanges one candidate per row instead (bcg_sampler_args.tp_size).
-  BCG_TRY(gemm_bf16_tn(ws->xn_last, m->lm_head, ws->logits, n_seqs, m->vocab, d, d, d, m->vocab,
-                       BCG_EPI_F32, 1, 0, st));
-  return BCG_OK;
+  return model_head(m, ws, last_rows, n_seqs, 0, st);
 }
 
 int model_decode(const bcg_model* m, const bcg_workspace* ws, const int* ids, const int* positions,

@@ -1,0 +1,153 @@
+// One step of a layer stack: whatever tokens the batch brings (whole prompts, portions, single decoded
+// tokens, mixed), launched from C++ on one stream.  Generation, trace replay and the captured decode graph
+// all go through stack_step; only the work lists differ.
+#include "stack_common.cuh"
+#include "kernels.h"
+
+namespace bcg {
+
+static int check_stack(const bcg_stack* m, const bcg_stack_ws* ws) {
+  if (!m || !ws || m->n_layers <= 0 || m->d_model <= 0 || (m->d_model % 4) || !m->embed || !m->lm_head ||
+      !m->final_norm || !m->layers || !ws->residual || !ws->xn || !ws->proj || !ws->logits ||
+      (m->act_dtype != BCG_DT_BF16 && m->act_dtype != BCG_DT_F32) || m->page_size <= 0) {
+    set_last_error("bcg_stack", "incomplete model / workspace description (d_model must be a multiple of 4)");
+    return BCG_ERR_ARG;
+  }
+  return BCG_OK;
+}
+
+// The tensor-core GEMM where TMA can address the operands, the CUDA-core one otherwise (and for fp32).
+static bool tensor_gemm(int act_dtype, int M, int N, int K) {
+  return act_dtype == BCG_DT_BF16 && K % 8 == 0 && (M <= 128 || N % 16 == 0);
+}
+// Rows of up to 128 tokens split K into slabs (a function of N and K only); larger launches do not.
+int stack_splits(int act_dtype, int M, int N, int K) {
+  return tensor_gemm(act_dtype, M, N, K) && M <= 128 ? gemm_splits_for(M, N, K) : 1;
+}
+static int project(const bcg_stack* m, const void* x, const void* w, float* out, long long cap, int M, int N, int K,
+                   int* splits, cudaStream_t st) {
+  *splits = stack_splits(m->act_dtype, M, N, K);
+  if (static_cast<long long>(*splits) * M * N > cap) {
+    set_last_error("bcg_stack_step", "projection scratch too small");
+    return BCG_ERR_TOO_LARGE;
+  }
+  if (tensor_gemm(m->act_dtype, M, N, K))
+    return gemm_bf16_tn(x, w, out, M, N, K, K, K, N, BCG_EPI_F32, *splits, launch_flags() & BCG_GEMM_PDL, st);
+  return gemm_any(x, m->act_dtype, w, out, M, N, K, K, K, N, st);
+}
+
+struct FlagScope {
+  int saved;
+  explicit FlagScope(int f) : saved(launch_flags()) { launch_flags() = f; }
+  ~FlagScope() { launch_flags() = saved; }
+};
+
+// Attention of one layer over the step's queries; `gathered` remembers whose cache rows ws->latents holds.
+static int attention(const bcg_stack* m, const bcg_stack_ws* ws, const bcg_step_batch* b, const bcg_layer* l,
+                     int mode, const void** gathered, cudaStream_t st) {
+  const int n_single = b->single_rows ? b->n_single : (b->n_tiles > 0 ? 0 : b->T);
+  const bool bf16 = m->act_dtype == BCG_DT_BF16 && mode == 0;
+  const bool fast_single = bf16 && latent_decode_ok(l), fast_tiles = bf16 && latent_prefill_ok(l);
+  if (!fast_single && !fast_tiles) return latent_plain(l, ws->q, ws->mix, b, nullptr, b->T, m->page_size, m->act_dtype, st);
+  if (b->n_tiles > 0) {
+    if (fast_tiles) {
+      if (b->n_gather > ws->K_max || !ws->latents || !ws->expanded) {
+        set_last_error("bcg_latent_attention", "gathered keys exceed the workspace");
+        return BCG_ERR_TOO_LARGE;
+      }
+      if (*gathered != l->cache) {
+        BCG_TRY(latent_gather(l->cache, b->gather, ws->latents, b->n_gather, l->kv_rank + l->rot_dim, st));
+        *gathered = l->cache;
+      }
+      BCG_TRY(latent_prefill(l, ws, b, st));
+    } else {   // single tokens are recomputed here too, which is harmless
+      BCG_TRY(latent_plain(l, ws->q, ws->mix, b, nullptr, b->T, m->page_size, m->act_dtype, st));
+    }
+  }
+  if (n_single > 0) {
+    if (fast_single) BCG_TRY(latent_decode(l, ws, b, m->page_size, st));
+    else BCG_TRY(latent_plain(l, ws->q, ws->mix, b, b->single_rows, n_single, m->page_size, m->act_dtype, st));
+  }
+  return BCG_OK;
+}
+
+int latent_attention(const bcg_stack* m, const bcg_stack_ws* ws, const bcg_step_batch* b, int layer, int mode,
+                     cudaStream_t st) {
+  BCG_TRY(check_stack(m, ws));
+  if (!b || layer < 0 || layer >= m->n_layers || m->layers[layer].mixer != BCG_MIXER_LATENT_ATTN) {
+    set_last_error("bcg_latent_attention", "not a latent attention layer");
+    return BCG_ERR_ARG;
+  }
+  const void* gathered = nullptr;
+  return attention(m, ws, b, &m->layers[layer], mode, &gathered, st);
+}
+
+int stack_step(const bcg_stack* m, const bcg_stack_ws* ws, const bcg_step_batch* b, cudaStream_t st) {
+  BCG_TRY(check_stack(m, ws));
+  if (!b || b->T <= 0 || b->T > ws->T_max || b->n_seqs <= 0 || !b->ids || !b->positions || !b->slot_map ||
+      !b->block_table || (!b->row_seq != !b->seq_start)) {
+    set_last_error("bcg_stack_step", "bad batch (T within the workspace, row_seq and seq_start together)");
+    return BCG_ERR_ARG;
+  }
+  FlagScope scope(b->flags & BCG_GEMM_PDL);
+  const int T = b->T, d = m->d_model, dt = m->act_dtype;
+  const void* gathered = nullptr;
+  BCG_TRY(embed_norm(b->ids, m->embed, m->layers[0].norm1, ws->residual, ws->xn, dt, T, d, m->eps, st));
+  for (int i = 0; i < m->n_layers; ++i) {
+    const bcg_layer* l = &m->layers[i];
+    const float* next = i + 1 < m->n_layers ? m->layers[i + 1].norm1 : m->final_norm;
+    int s = 1, mix_out = 0;
+    BCG_TRY(project(m, ws->xn, l->w_in, ws->proj, ws->proj_floats, T, l->n_in, d, &s, st));
+    const long long in_stride = static_cast<long long>(T) * l->n_in;
+    if (l->mixer == BCG_MIXER_LATENT_ATTN) {
+      mix_out = l->heads * l->vdim;
+      BCG_TRY(latent_qkv(l, ws->proj, s, in_stride, b->positions, b->slot_map, ws->q, dt, T, m->eps, st));
+      if (gathered == l->cache && l->owns_cache) gathered = nullptr;
+      BCG_TRY(attention(m, ws, b, l, 0, &gathered, st));
+    } else if (l->mixer == BCG_MIXER_GENERAL_DELTA) {
+      mix_out = l->heads * l->dim;
+      int sd = 1;
+      BCG_TRY(delta_low(l, ws->proj, s, in_stride, ws->low, dt, T, st));
+      BCG_TRY(project(m, ws->low, l->w_decay, ws->decay, ws->decay_floats, T, mix_out, l->decay_rank, &sd, st));
+      BCG_TRY(delta_scan(l, ws->proj, s, in_stride, l->n_in, ws->decay, sd, static_cast<long long>(T) * mix_out,
+                         b->positions, b->slot_map, b->seq_start, b->state_slots, b->n_seqs, T == b->n_seqs, ws->mix,
+                         dt, m->eps, st));
+    } else {
+      set_last_error("bcg_stack_step", "unknown mixer");
+      return BCG_ERR_UNSUPPORTED;
+    }
+    BCG_TRY(project(m, ws->mix, l->w_out, ws->proj, ws->proj_floats, T, d, mix_out, &s, st));
+    BCG_TRY(sandwich_norm(ws->residual, ws->proj, s, static_cast<long long>(T) * d, l->norm1b, l->ff ? l->norm2 : next,
+                          ws->xn, dt, T, d, m->eps, st));
+    if (l->ff) {
+      BCG_TRY(project(m, ws->xn, l->w_up, ws->proj, ws->proj_floats, T, l->ff, d, &s, st));
+      BCG_TRY(poly_norm(ws->proj, s, static_cast<long long>(T) * l->ff, l->act_coef, ws->act, dt, T, l->ff, m->eps, st));
+      BCG_TRY(project(m, ws->act, l->w_down, ws->proj, ws->proj_floats, T, d, l->ff, &s, st));
+      BCG_TRY(sandwich_norm(ws->residual, ws->proj, s, static_cast<long long>(T) * d, l->norm2b, next, ws->xn, dt, T, d,
+                            m->eps, st));
+    }
+  }
+  return BCG_OK;
+}
+
+int stack_head(const bcg_stack* m, const bcg_stack_ws* ws, const int* rows, int n, int row0, int flags,
+               cudaStream_t st) {
+  BCG_TRY(check_stack(m, ws));
+  if (n <= 0 || row0 < 0 || row0 + n > ws->B_max || (rows && !ws->xn_rows)) {
+    set_last_error("bcg_stack_head", "rows exceed the logits buffer");
+    return BCG_ERR_TOO_LARGE;
+  }
+  FlagScope scope(flags & BCG_GEMM_PDL);
+  const void* x = ws->xn;
+  if (rows) {
+    BCG_TRY(rows_norm(ws->residual, rows, m->final_norm, ws->xn_rows, m->act_dtype, n, m->d_model, m->eps, st));
+    x = ws->xn_rows;
+  }
+  float* out = ws->logits + static_cast<long long>(row0) * m->vocab_ld;
+  const int d = m->d_model, V = m->vocab_ld;
+  if (tensor_gemm(m->act_dtype, n, V, d))
+    return gemm_bf16_tn(x, m->lm_head, out, n, V, d, d, d, V, BCG_EPI_F32, 1, launch_flags() & BCG_GEMM_PDL, st);
+  return gemm_any(x, m->act_dtype, m->lm_head, out, n, V, d, d, d, V, st);
+}
+
+}  // namespace bcg

@@ -33,16 +33,13 @@ import torch
 
 from . import grammar as G
 from . import lib as L
-from .model import ModelConfig, ModelHandle, Weights
+from .executors import PAGE, PREFILL_TILE, SPLIT_TOKENS, Entry, make_executor
+from .model import ModelConfig, Weights
 from .tokenizer import CachedEncoder
 
-PAGE = 16
-SPLIT_TOKENS = 256
 MAX_GRAMMARS = 64
 POLL_EVERY = 8      # tensor-parallel engines: steps between two synchronised looks at the active-row count
 IN_FLIGHT = 2       # single-GPU engines: decode steps queued ahead of the one whose result the host has seen
-# query rows per prefill-attention CTA (bcg_prefill_attn_paged)
-PREFILL_TILE = 128
 
 
 def row_seed(base_seed: int, call_index: int, row: int):
@@ -145,16 +142,43 @@ class PagePool:
                 self.free.append(p)
 
 
+class SlotPool:
+    """State slots of recurrent layers.  A slot is not cleared when it changes hands: a sequence's first token
+    (position 0) starts from a zero state, whatever the slot holds."""
+
+    def __init__(self, n: int):
+        self.n = n
+        self.free = list(range(n - 1, -1, -1))
+
+    def alloc(self) -> int:
+        if not self.free:
+            raise MemoryError("state slots exhausted")
+        return self.free.pop()
+
+    def release(self, slot: int) -> None:
+        self.free.append(slot)
+
+
+@dataclass
+class LiveSequence:
+    """A live sequence of the step interface (Engine.open / step / close)."""
+    length: int = 0
+    pages: List[int] = field(default_factory=list)
+    slot: int = 0
+
+
 class Engine:
     def __init__(self, cfg: ModelConfig, weights: Weights, tokenizer, *, max_model_len: int = 8192,
                  max_rows: int = 64, prefill_tokens: int = 16384, kv_pages: Optional[int] = None,
                  gpu_memory_utilization: float = 0.9, base_seed: int = 0, device: str = "cuda:0",
                  enable_prefix_cache: bool = True, use_cuda_graph: bool = True, pdl: bool = True,
                  fused_norm: bool = False, deferred_norm: Optional[bool] = None,
-                 fused_rope: bool = False,
+                 fused_rope: bool = False, state_slots: Optional[int] = None, logit_rows: int = 0,
                  tp_rank: int = 0, tp_size: int = 1, tp_fused_allreduce: bool = True, tp_group=None):
-        """`cfg` is the FULL architecture; with tp_size > 1 `weights` must be this rank's shard
-        (Weights.shard / random_init_sharded) and bcg_tp_init must have been called (collective)."""
+        """`cfg` is the FULL architecture (a ModelConfig, or a StackConfig with StackWeights).  `tokenizer` may be
+        None for an engine that only steps given tokens (open / step / close_sequence).  With tp_size > 1 `weights` must
+        be this rank's shard (Weights.shard / random_init_sharded) and bcg_tp_init must have been called
+        (collective)."""
         if not torch.cuda.is_available():
             raise L.BcgError("the engine needs a CUDA device (sm_100a); there is no CPU fallback")
         self.lib = L.load()
@@ -172,7 +196,6 @@ class Engine:
         self.T_max = max(prefill_tokens, self.max_model_len)
         self.base_seed = base_seed
         self.calls = 0
-        self.enable_prefix_cache = enable_prefix_cache
         self.use_cuda_graph = use_cuda_graph
         # How decode runs the residual add + RMSNorm between projections (include/bcg_b200.h,
         # bcg_model_decode).  Default on one GPU: statistics kernel + 1/RMS in the next GEMM's epilogue
@@ -187,54 +210,23 @@ class Engine:
         self.max_blocks = (self.max_model_len + PAGE - 1) // PAGE
         self.max_steps = self.max_model_len
 
-        d, B, T = cfg.d_model, self.max_rows, self.T_max
-        bf, f32, i32 = torch.bfloat16, torch.float32, torch.int32
-        z = lambda *s, dt=bf: torch.zeros(*s, dtype=dt, device=self.dev)
-        # ---- workspace (include/bcg_b200.h bcg_workspace)
-        self.max_splits_cap = (self.max_model_len + SPLIT_TOKENS - 1) // SPLIT_TOKENS
-        lc = lcfg
-        splits = [L.splits_for(1, n, k) for n, k in ((lc.qkv_dim, d), (d, lc.n_heads * 128),
-                                                      (2 * lc.d_ff, d), (d, lc.d_ff))]
-        pf = max(splits[0] * B * lc.qkv_dim, splits[1] * B * d,
-                 (splits[2] * B * 2 * lc.d_ff) if splits[2] > 1 else 0, splits[3] * B * d)
-        self.buf = dict(
-            residual=z(T, d, dt=f32), xn=z(T, d), qkv=z(T, lc.qkv_dim, dt=f32), q=z(T, lc.n_heads * 128),
-            attn=z(T, lc.n_heads * 128), act=z(T, lc.d_ff), delta=z(T, d, dt=f32), partials=z(pf, dt=f32),
-            so=z(B * lc.n_heads * self.max_splits_cap * 128, dt=f32),
-            sml=z(B * lc.n_heads * self.max_splits_cap * 2, dt=f32),
-            attn_counters=z(B * lc.n_kv_heads, dt=i32),
-            row_sumsq=z(2 * max((d + 127) // 128, 8) * 128, dt=f32), tile_counters=z((d + 127) // 128, dt=i32),
-            # under tensor parallelism the logits stay sharded: [B, vocab / tp] per rank
-            logits=z(B, lc.vocab, dt=f32), xn_last=z(B, d))
-        ws = L.Workspace()
-        b = self.buf
-        ws.residual, ws.xn, ws.qkv, ws.q = b["residual"].data_ptr(), b["xn"].data_ptr(), b["qkv"].data_ptr(), b["q"].data_ptr()
-        ws.attn, ws.act, ws.delta = b["attn"].data_ptr(), b["act"].data_ptr(), b["delta"].data_ptr()
-        ws.partials, ws.partials_floats = b["partials"].data_ptr(), pf
-        ws.attn_scratch_o, ws.attn_scratch_ml = b["so"].data_ptr(), b["sml"].data_ptr()
-        ws.attn_counters = b["attn_counters"].data_ptr()
-        ws.max_splits = self.max_splits_cap
-        ws.logits, ws.xn_last, ws.T_max, ws.B_max = b["logits"].data_ptr(), b["xn_last"].data_ptr(), T, B
-        ws.logits_local = None
-        # tables for the deferred / fused norm (row sums of squares; tile counters for fused_norm=True)
-        ws.row_sumsq = b["row_sumsq"].data_ptr()
-        ws.tile_counters = b["tile_counters"].data_ptr() if (tp_size == 1 and d % 128 == 0) else None
-        ws.tp_region_floats = 0
-        if tp_size > 1:
-            # The symmetric buffer (cudaIpc over NVLink) carries the sampler's candidate exchange
-            # and, with tp_fused_allreduce, the decode step's all-reduces (bcg_tp_add_norm_stats).
-            from . import tp as _tp
-            region = B * d if tp_fused_allreduce else 0
-            _tp.setup_symmetric(int(self.lib.bcg_tp_symm_bytes_for(region, tp_size)), tp_rank, tp_size, tp_group)
-            ws.tp_region_floats = region
-        self.ws = ws
-        # ---- KV pages
-        page_bytes = 2 * lc.n_kv_heads * PAGE * 128 * 2 * cfg.n_layers
+        B = self.max_rows
+        f32, i32 = torch.float32, torch.int32
+        z = lambda *s, dt=torch.bfloat16: torch.zeros(*s, dtype=dt, device=self.dev)
+        self.exec = make_executor(cfg, lcfg, weights, self.dev, max_rows=B, T_max=self.T_max,
+                                  max_model_len=self.max_model_len, logit_rows=logit_rows, flags=self.flags,
+                                  tp_rank=tp_rank, tp_size=tp_size, tp_fused_allreduce=tp_fused_allreduce,
+                                  tp_group=tp_group)
+        self.buf, self.ws = self.exec.buf, self.exec.ws
+        # ---- state slots and KV pages
+        self.slots = SlotPool(state_slots or B)
+        page_bytes = self.exec.page_bytes
         if kv_pages is None:
             free_b, total_b = torch.cuda.mem_get_info(self.dev)
-            budget = int(total_b * gpu_memory_utilization) - (total_b - free_b)
+            budget = int(total_b * gpu_memory_utilization) - (total_b - free_b) \
+                - self.slots.n * self.exec.state_slot_bytes
             want = self.max_rows * self.max_blocks * 2
-            kv_pages = max(self.max_blocks + 8, min(want, budget // page_bytes))
+            kv_pages = max(self.max_blocks + 8, min(want, budget // max(page_bytes, 1)))
             if tp_size > 1:
                 # every rank must run the SAME page pool (eviction, cache hits and prefill sizes are
                 # decided per rank and have to agree): take the smallest budget of the replica
@@ -242,14 +234,16 @@ class Engine:
                 t = torch.tensor([kv_pages], dtype=torch.int64)
                 dist.all_reduce(t, op=dist.ReduceOp.MIN, group=tp_group)
                 kv_pages = int(t.item())
-        self.kv_layers = [z(kv_pages, 2, lc.n_kv_heads, PAGE, 128) for _ in range(cfg.n_layers)]
+        self.exec.alloc_cache(kv_pages, self.slots.n)
+        self.kv_layers, self.model = self.exec.kv_layers, self.exec.model
         self.pool = PagePool(kv_pages)
-        self.model = ModelHandle(weights, self.kv_layers, PAGE, tp_size)
+        # pages alone restore a prefix only where no layer carries a recurrent state
+        self.enable_prefix_cache = enable_prefix_cache and not self.exec.has_state
         # ---- per-row device state (bcg_sampler_args).  Everything the host writes at the start of a
         # call lives in ONE int32 block with a pinned host mirror, so a call costs one H2D copy
         # instead of one per field.
         fields = [("grammar_id", 1), ("state", 1), ("temperature", 1), ("seed", 2), ("max_tokens", 1),
-                  ("n_out", 1), ("finished", 1), ("seq_lens", 1), ("block_table", self.max_blocks)]
+                  ("n_out", 1), ("finished", 1), ("seq_lens", 1), ("state_slot", 1), ("block_table", self.max_blocks)]
         words = sum(w for _, w in fields) * B
         self._state_dev = z(words, dt=i32)
         self._state_host = torch.zeros(words, dtype=i32).pin_memory()
@@ -270,19 +264,19 @@ class Engine:
         # HOST memory (mapped into the device's address space), so the host reads it without a copy.
         self.n_active_host = torch.zeros(1, dtype=i32).pin_memory()
         self.row["n_active"] = self.n_active_host
-        # ---- prefill staging: ids | positions | slots | last rows | tiles | block table, one copy per group
-        self._pf_cap = (3 * self.T_max, B, 4 * (self.T_max // PREFILL_TILE + B), B * self.max_blocks, 32)
-        self._pf_dev = z(sum(self._pf_cap), dt=i32)
-        self._pf_host = torch.zeros(sum(self._pf_cap), dtype=i32).pin_memory()
+        # ---- staging of a ragged step's arrays (ids, positions, slots, work lists, block table), one copy each
+        self._pf_dev = z(self.exec.staging_words, dt=i32)
+        self._pf_host = torch.zeros(self.exec.staging_words, dtype=i32).pin_memory()
         # ---- tokenizer / grammar tables on the device
-        tok_bytes = G.grammar_token_bytes(tokenizer)
-        lens = np.fromiter((len(x) for x in tok_bytes), np.int64, count=cfg.vocab)
-        offs = np.zeros(cfg.vocab + 1, np.int32)
-        offs[1:] = np.cumsum(lens)
-        blob = np.frombuffer(b"".join(tok_bytes) or b"\0", dtype=np.uint8).copy()
-        self.tok_bytes = torch.from_numpy(blob).to(self.dev)
-        self.tok_offsets = torch.from_numpy(offs).to(self.dev)
-        self.mask_words = (cfg.vocab + 31) // 32
+        if tokenizer is not None:
+            tok_bytes = G.grammar_token_bytes(tokenizer)
+            lens = np.fromiter((len(x) for x in tok_bytes), np.int64, count=cfg.vocab)
+            offs = np.zeros(cfg.vocab + 1, np.int32)
+            offs[1:] = np.cumsum(lens)
+            blob = np.frombuffer(b"".join(tok_bytes) or b"\0", dtype=np.uint8).copy()
+            self.tok_bytes = torch.from_numpy(blob).to(self.dev)
+            self.tok_offsets = torch.from_numpy(offs).to(self.dev)
+            self.mask_words = (cfg.vocab + 31) // 32
         self.grammars: Dict[str, int] = {}
         self.grammar_objs: List[G.CompiledGrammar] = []
         self._gram_dev = []
@@ -293,7 +287,7 @@ class Engine:
                           decode_steps=0, generated_tokens=0, prefill_s=0.0, decode_s=0.0, host_s=0.0,
                           gpu_launches=0, h2d_bytes=0, d2h_bytes=0)
         self._capture_stream = torch.cuda.Stream(self.dev)
-        self._encode = CachedEncoder(tokenizer)    # retries resubmit identical prompts
+        self._encode = CachedEncoder(tokenizer) if tokenizer is not None else None    # retries resubmit identical prompts
         # parity tests: when set to a list, the logits of every step are appended (forces the
         # eager, graph-less decode loop)
         self.debug_logits: Optional[list] = None
@@ -345,20 +339,11 @@ class Engine:
         L.check(self.lib.bcg_mask_sample(C.byref(a), L.stream_ptr()), "bcg_mask_sample")
 
     def _decode_step(self, B: int, max_splits: int, use_forced: bool) -> None:
-        r = self.row
-        self.ws.max_splits = max_splits
-        L.check(self.lib.bcg_model_decode(C.byref(self.model.struct), C.byref(self.ws),
-                                          r["next_ids"].data_ptr(), r["positions"].data_ptr(),
-                                          r["slot_map"].data_ptr(), r["seq_lens"].data_ptr(),
-                                          r["block_table"].data_ptr(), self.max_blocks, B, self.flags,
-                                          L.stream_ptr()), "bcg_model_decode")
+        self.exec.decode(self.row, B, max_splits)
         self._sample(B, use_forced)
 
     def launches_per_decode_step(self, B: int) -> int:
-        cfg = self.cfg
-        s_gu = L.splits_for(B, 2 * cfg.d_ff, cfg.d_model)
-        per_layer = 8 + (1 if s_gu > 1 else 0)   # norm, qkv, rope, attn, o, norm, gate_up(+reduce), down
-        return cfg.n_layers * per_layer + 2 + 2  # final norm + lm_head + sampler + active count
+        return self.exec.launches_per_decode_step(B) + 2     # sampler + active count
 
     def _graph_for(self, B: int, max_splits: int, use_forced: bool):
         key = (B, max_splits, use_forced)
@@ -374,6 +359,10 @@ class Engine:
 
     # ------------------------------------------------------------------ generation
     def generate(self, requests: List[Request]) -> List[Result]:
+        if self.tk is None:
+            raise L.BcgError("an engine without a tokenizer only steps given tokens (open / step / close_sequence)")
+        if self.lcfg.vocab % 4:
+            raise L.BcgError(f"the sampler needs a vocabulary that is a multiple of 4 (got {self.lcfg.vocab})")
         out: List[Result] = []
         for i in range(0, len(requests), self.max_rows):
             out.extend(self._generate_wave(requests[i:i + self.max_rows], i))
@@ -385,7 +374,7 @@ class Engine:
         t_host0 = time.perf_counter()
         cfg, B = self.cfg, len(reqs)
         r = self.row
-        ids_list, cached, pages_of, hashes_of = [], [], [], []
+        ids_list, cached, pages_of, hashes_of, slots_of = [], [], [], [], []
         use_forced = any(q.forced is not None for q in reqs)
         for q in reqs:
             ids = list(q.prompt_ids) if q.prompt_ids is not None else self._encode(q.prompt)
@@ -420,21 +409,26 @@ class Engine:
                 pages_of.append(pages)
                 hashes_of.append(hs)
                 cached.append(hit * PAGE)
+                slots_of.append(self.slots.alloc() if self.exec.has_state else 0)
         except Exception:
-            for pages in pages_of:
-                for p in pages:
-                    self.pool.release(p)
+            self._release(pages_of, slots_of)
             raise
 
         try:
-            results = self._run(reqs, ids_list, cached, pages_of, hashes_of, use_forced, row0, t_host0)
+            results = self._run(reqs, ids_list, cached, pages_of, hashes_of, slots_of, use_forced, row0, t_host0)
         finally:
-            for pages in pages_of:
-                for p in pages:
-                    self.pool.release(p)
+            self._release(pages_of, slots_of)
         return results
 
-    def _run(self, reqs, ids_list, cached, pages_of, hashes_of, use_forced, row0, t_host0):
+    def _release(self, pages_of, slots_of) -> None:
+        for pages in pages_of:
+            for p in pages:
+                self.pool.release(p)
+        if self.exec.has_state:
+            for s in slots_of:
+                self.slots.release(s)
+
+    def _run(self, reqs, ids_list, cached, pages_of, hashes_of, slots_of, use_forced, row0, t_host0):
         cfg, B, r, dev = self.cfg, len(reqs), self.row, self.dev
         i32 = torch.int32
         bt = np.zeros((B, self.max_blocks), np.int32)
@@ -453,6 +447,7 @@ class Engine:
         h["n_out"][:B] = 0
         h["finished"][:B] = 0
         h["seq_lens"][:B] = [len(x) for x in ids_list]
+        h["state_slot"][:B] = slots_of
         h["seed"][:B] = seeds.view(np.int32).reshape(B, 2)
         h["block_table"][:B] = bt
         self._state_dev.copy_(self._state_host, non_blocking=True)     # ONE copy for all per-row state
@@ -465,17 +460,15 @@ class Engine:
             r["forced"][:B].copy_(torch.from_numpy(f))
             self.stats["h2d_bytes"] += f.nbytes
 
-        # ---- prefill in groups of <= T_max new tokens
+        # ---- prefill: the uncached part of every prompt, in groups that fit a launch
         ev0, ev1, ev2 = (torch.cuda.Event(enable_timing=True) for _ in range(3))
         ev0.record()
+        entries = [Entry(ids[c:], c, bt[b], slots_of[b], (len(ids) - c - 1,))
+                   for b, (ids, c) in enumerate(zip(ids_list, cached))]
         b0 = 0
-        while b0 < B:
-            b1, T = b0, 0
-            while b1 < B and T + (len(ids_list[b1]) - cached[b1]) <= self.T_max:
-                T += len(ids_list[b1]) - cached[b1]
-                b1 += 1
-            self._prefill_group(b0, b1, ids_list, cached, bt)
-            b0 = b1
+        for group in self._groups(entries):
+            self._launch_group(group, b0)       # last-token logits go straight to the rows of these prompts
+            b0 += len(group)
         # publish freshly written full prompt pages for later calls
         if self.enable_prefix_cache:
             for b in range(B):
@@ -579,57 +572,91 @@ class Engine:
         """[B, V] logits of the current step (parity tests only; under TP the vocabulary shards are
         gathered over the control group — the product path never moves logits between ranks)."""
         if self.tp_size == 1:
-            return self.buf["logits"][:B].clone()
+            return self.buf["logits"][:B, :self.cfg.vocab].clone()
         import torch.distributed as dist
         mine = self.buf["logits"][:B].cpu()
         parts = [torch.empty_like(mine) for _ in range(self.tp_size)]
         dist.all_gather(parts, mine, group=self.tp_group)
         return torch.cat(parts, dim=1).to(self.dev)
 
-    def _prefill_group(self, b0, b1, ids_list, cached, bt) -> None:
-        cfg, dev = self.cfg, self.dev
-        ids, pos, slots, tiles, last = [], [], [], [], []
-        row = 0
-        for b in range(b0, b1):
-            c, n = cached[b], len(ids_list[b]) - cached[b]
-            ids.extend(ids_list[b][c:])
-            p = np.arange(c, c + n)
-            pos.append(p)
-            slots.append(bt[b, p // PAGE] * PAGE + p % PAGE)
-            for q0 in range(0, n, PREFILL_TILE):
-                tiles.append((b - b0, row + q0, c + q0, min(PREFILL_TILE, n - q0)))
-            row += n
-            last.append(row - 1)
-        T, n_seqs = row, b1 - b0
-        # one pinned staging block, one H2D copy per group: ids | positions | slots | last | tiles | bt.
-        # A group's copy must have left the pinned block before the next group refills it.
+    # ------------------------------------------------------------------ ragged steps
+    def _groups(self, entries: List[Entry]):
+        """Consecutive entries that fit one launch (tokens, gathered keys, rows)."""
+        group, T, K = [], 0, 0
+        for e in entries:
+            t, k = self.exec.cost(e)
+            if group and (T + t > self.T_max or K + k > max(self.exec.K_max, 0) and k or len(group) >= self.max_rows):
+                yield group
+                group, T, K = [], 0, 0
+            group.append(e)
+            T, K = T + t, K + k
+        if group:
+            yield group
+
+    def _launch_group(self, entries: List[Entry], row0: int):
+        """Stage and launch one ragged step; wanted logits from logits row `row0`.  Returns (plan, device
+        views, how many wanted logits that left in the buffer)."""
+        plan = self.exec.plan(entries)
+        # one pinned staging block, one H2D copy per launch.  A launch's copy must have left the pinned
+        # block before the next one refills it.
         if getattr(self, "_pf_event", None) is not None:
             self._pf_event.synchronize()
-        hs, o0 = self._pf_host.numpy(), 0
-        views = []
-        for arr in (ids, np.concatenate(pos), np.concatenate(slots), last, np.array(tiles).reshape(-1),
-                    bt[b0:b1].reshape(-1)):
+        hs, o0, views = self._pf_host.numpy(), 0, {}
+        for name, arr in plan.arrays.items():
             a = np.asarray(arr, dtype=np.int32)
             hs[o0:o0 + a.size] = a
-            views.append(self._pf_dev[o0:o0 + a.size])
+            views[name] = self._pf_dev[o0:o0 + a.size]
             o0 += (a.size + 3) // 4 * 4        # keep every array 16-byte aligned
         self._pf_dev[:o0].copy_(self._pf_host[:o0], non_blocking=True)
         self._pf_event = torch.cuda.Event()
         self._pf_event.record()
-        d_ids, d_pos, d_slots, d_last, d_tiles, d_bt = views
         self.stats["h2d_bytes"] += o0 * 4
-        # this group's last-token logits go straight to rows b0..b1 of the row-indexed buffer
-        base = self.buf["logits"].data_ptr()
-        self.ws.logits = base + b0 * self.lcfg.vocab * 4
-        try:
-            L.check(self.lib.bcg_model_prefill(C.byref(self.model.struct), C.byref(self.ws),
-                                               d_ids.data_ptr(), d_pos.data_ptr(), d_slots.data_ptr(),
-                                               d_bt.data_ptr(), self.max_blocks, d_tiles.data_ptr(),
-                                               len(tiles), d_last.data_ptr(), n_seqs, T, L.stream_ptr()),
-                    "bcg_model_prefill")
-        finally:
-            self.ws.logits = base
-        self.stats["gpu_launches"] += cfg.n_layers * 8 + 2
+        done = self.exec.launch(plan, views, row0)
+        self.stats["gpu_launches"] += self.exec.launches_prefill()
+        return plan, views, done
+
+    # The step interface: the caller brings the tokens, the engine keeps pages and states.  The same launches
+    # as generate(): a batch of single tokens is a decode step, anything else a ragged step.
+    def open(self) -> LiveSequence:
+        return LiveSequence(slot=self.slots.alloc() if self.exec.has_state else 0)
+
+    def close_sequence(self, seq: LiveSequence) -> None:
+        """Gives a sequence's pages and state slot back."""
+        self._release([seq.pages], [seq.slot])
+        seq.pages, seq.length = [], 0
+
+    def step(self, work) -> torch.Tensor:
+        """work: [(LiveSequence, token ids, places among them whose logits are wanted)], one batch.  Returns the
+        wanted logits [n, vocab] (fp32, on the device) in that order."""
+        entries: List[Entry] = []
+        for seq, tokens, want in work:
+            end = seq.length + len(tokens)
+            if not tokens:
+                raise L.BcgError("a step's entry needs at least one token")
+            if end > self.max_model_len:
+                raise L.BcgError(f"sequence of {end} tokens exceeds max_model_len ({self.max_model_len})")
+            while len(seq.pages) * PAGE < end:
+                seq.pages.append(self.pool.alloc())
+            row = np.zeros(self.max_blocks, np.int32)
+            row[:len(seq.pages)] = seq.pages
+            done = 0
+            while done < len(tokens):           # a portion longer than a launch takes is cut
+                n = min(len(tokens) - done, self.exec.max_tokens_of(seq.length + done))
+                entries.append(Entry(tokens[done:done + n], seq.length + done, row, seq.slot,
+                                     [w - done for w in want if done <= w < done + n]))
+                done += n
+        out = []
+        for group in self._groups(entries):
+            plan, views, done = self._launch_group(group, 0)
+            out.append(self.buf["logits"][:done, :self.lcfg.vocab].clone())
+            while done < plan.n_want:
+                n = min(plan.n_want - done, self.exec.B_max)
+                self.exec.head(views, done, n, 0)
+                out.append(self.buf["logits"][:n, :self.lcfg.vocab].clone())
+                done += n
+        for seq, tokens, _ in work:
+            seq.length += len(tokens)
+        return torch.cat(out)
 
     # ------------------------------------------------------------------ misc
     def reset_prefix_cache(self) -> None:

@@ -18,6 +18,9 @@ STEP_FUSED_NORM = 0x20000   # bcg_model_decode: fold add+RMSNorm into the GEMMs 
 STEP_FUSED_ROPE = 0x80000     # bcg_model_decode: qk-norm/RoPE/KV-write folded into decode attention
 STEP_DEFERRED_NORM = 0x40000  # bcg_model_decode: norm statistics kernel + 1/RMS in the next GEMM's epilogue
 
+DT_BF16, DT_F32 = 0, 1                          # activation dtype of a layer stack
+MIXER_LATENT_ATTN, MIXER_GENERAL_DELTA = 1, 2
+
 c_int_p = C.POINTER(C.c_int)
 c_float_p = C.POINTER(C.c_float)
 vp = C.c_void_p
@@ -77,6 +80,45 @@ class Workspace(C.Structure):
     ]
 
 
+class Layer(C.Structure):
+    _fields_ = [
+        ("mixer", C.c_int), ("heads", C.c_int), ("dim", C.c_int), ("rot_dim", C.c_int),
+        ("rot_dims", C.c_int), ("vdim", C.c_int), ("kv_rank", C.c_int), ("window", C.c_int),
+        ("scale", C.c_float), ("q_ld", C.c_int), ("v_ld", C.c_int), ("owns_cache", C.c_int),
+        ("n_in", C.c_int), ("decay_rank", C.c_int), ("ff", C.c_int), ("norm1", vp), ("norm1b", vp),
+        ("norm2", vp), ("norm2b", vp), ("w_in", vp), ("w_out", vp), ("latent_norm", vp), ("sink", vp),
+        ("cos_sin", vp), ("w_uk", vp), ("w_uv", vp), ("w_expand", vp), ("decay_bias", vp), ("rate_bias", vp),
+        ("out_norm", vp), ("w_decay", vp), ("w_up", vp), ("w_down", vp), ("act_coef", vp), ("cache", vp),
+    ]
+
+
+class Stack(C.Structure):
+    _fields_ = [
+        ("n_layers", C.c_int), ("d_model", C.c_int), ("vocab_ld", C.c_int), ("act_dtype", C.c_int),
+        ("page_size", C.c_int), ("eps", C.c_float), ("embed", vp), ("lm_head", vp), ("final_norm", vp),
+        ("layers", C.POINTER(Layer)),
+    ]
+
+
+class StackWs(C.Structure):
+    _fields_ = [
+        ("residual", vp), ("xn", vp), ("proj", vp), ("proj_floats", C.c_longlong), ("decay", vp),
+        ("decay_floats", C.c_longlong), ("q", vp), ("mix", vp), ("act", vp), ("low", vp), ("latents", vp),
+        ("expanded", vp), ("q_latent", vp), ("o_latent", vp), ("part_o", vp), ("part_floats", C.c_longlong),
+        ("part_ml", vp), ("xn_rows", vp), ("logits", vp), ("T_max", C.c_int), ("K_max", C.c_int),
+        ("D_max", C.c_int), ("B_max", C.c_int),
+    ]
+
+
+class StepBatch(C.Structure):
+    _fields_ = [
+        ("T", C.c_int), ("n_seqs", C.c_int), ("ids", vp), ("positions", vp), ("slot_map", vp),
+        ("row_seq", vp), ("seq_start", vp), ("block_table", vp), ("max_blocks", C.c_int),
+        ("state_slots", vp), ("max_context", C.c_int), ("single_rows", vp), ("n_single", C.c_int),
+        ("tiles", vp), ("n_tiles", C.c_int), ("gather", vp), ("n_gather", C.c_int), ("flags", C.c_int),
+    ]
+
+
 _SIGS = {
     "bcg_abi_version": (C.c_int, []),
     "bcg_last_error": (C.c_char_p, []),
@@ -114,8 +156,20 @@ _SIGS = {
     "bcg_tp_symm_open": (C.c_int, [vp, C.c_int, C.c_int]),
     "bcg_model_prefill": (C.c_int, [C.POINTER(Model), C.POINTER(Workspace), vp, vp, vp, vp, C.c_int,
                                     vp, C.c_int, vp, C.c_int, C.c_int, vp]),
+    "bcg_model_head": (C.c_int, [C.POINTER(Model), C.POINTER(Workspace), vp, C.c_int, C.c_int, vp]),
     "bcg_model_decode": (C.c_int, [C.POINTER(Model), C.POINTER(Workspace), vp, vp, vp, vp, vp,
                                    C.c_int, C.c_int, C.c_int, vp]),
+    "bcg_stack_step": (C.c_int, [C.POINTER(Stack), C.POINTER(StackWs), C.POINTER(StepBatch), vp]),
+    "bcg_stack_head": (C.c_int, [C.POINTER(Stack), C.POINTER(StackWs), vp, C.c_int, C.c_int, C.c_int, vp]),
+    "bcg_gemm_any": (C.c_int, [vp, C.c_int, vp, vp, C.c_int, C.c_int, C.c_int, C.c_longlong, C.c_longlong,
+                               C.c_longlong, vp]),
+    "bcg_sandwich_norm": (C.c_int, [vp, vp, C.c_int, C.c_longlong, vp, vp, vp, C.c_int, C.c_int, C.c_int, C.c_float,
+                                    vp]),
+    "bcg_poly_norm": (C.c_int, [vp, C.c_int, C.c_longlong, vp, vp, C.c_int, C.c_int, C.c_int, C.c_float, vp]),
+    "bcg_delta_scan": (C.c_int, [C.POINTER(Layer), vp, C.c_int, C.c_longlong, C.c_longlong, vp, C.c_int,
+                                 C.c_longlong, vp, vp, vp, vp, C.c_int, vp, C.c_int, C.c_float, vp]),
+    "bcg_latent_attention": (C.c_int, [C.POINTER(Stack), C.POINTER(StackWs), C.POINTER(StepBatch), C.c_int, C.c_int,
+                                       vp]),
 }
 
 EXPORTED = tuple(_SIGS)

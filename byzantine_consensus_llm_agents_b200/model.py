@@ -14,6 +14,7 @@ from dataclasses import dataclass, field
 import torch
 
 from . import lib as L
+from . import stack
 
 
 @dataclass(frozen=True)
@@ -75,6 +76,9 @@ PRESETS = {
     # Mistral-Small-Instruct-2409's config.json: rms_norm_eps 1e-05 (Qwen3's is 1e-06)
     "mistral-22b": ModelConfig("mistral-22b", 56, 6144, 48, 8, 16384, 32768, rms_eps=1e-5, qk_norm=False,
                                family="mistral"),
+    # layer stacks (stack.py) at the widths of the dense presets beside them
+    "bekopel-1b": stack.bekopel_preset("bekopel-1b", 16, 2048, 8192, 151936, heads=16),
+    "bekopel-8b": stack.bekopel_preset("bekopel-8b", 36, 4096, 18432, 151936),
 }
 
 _HF_NAMES = {
@@ -86,7 +90,12 @@ _HF_NAMES = {
 }
 
 
-def config_for(model_name: str) -> ModelConfig:
+def weights_for(cfg):
+    """The weights class (from_safetensors_dir, random_init) that goes with a configuration."""
+    return stack.StackWeights if isinstance(cfg, stack.StackConfig) else Weights
+
+
+def config_for(model_name: str):
     key = model_name.lower()
     if key in PRESETS:
         return PRESETS[key]
@@ -95,13 +104,16 @@ def config_for(model_name: str) -> ModelConfig:
     raise KeyError(f"no architecture known for model {model_name!r}")
 
 
-def config_from_dir(model_dir: str) -> ModelConfig:
-    """ModelConfig from a local HuggingFace model directory's config.json (the file vLLM reads when
+def config_from_dir(model_dir: str):
+    """The configuration of a local model directory: a StackConfig where config.json's "architecture" names a
+    layer-stack design (stack.DESIGNS), else a ModelConfig from a HuggingFace model directory's config.json (the file vLLM reads when
     the reference names a model, vllm_agent.py:126-144).  Dense Qwen3 / Qwen2 / Llama / Mistral-style
     decoders with head_dim 128 are what the kernels support."""
     import json
     from pathlib import Path
     c = json.loads((Path(model_dir) / "config.json").read_text())
+    if c.get("architecture") in stack.DESIGNS:
+        return stack.config_from_dir(model_dir, c)
     mt = str(c.get("model_type", "")).lower()
     heads = int(c["num_attention_heads"])
     head_dim = int(c.get("head_dim") or c["hidden_size"] // heads)

@@ -1,0 +1,423 @@
+"""Layer stacks: models whose layers differ in kind, described by composable specs.
+
+A `StackConfig` lists layers; each has a mixer spec (`LatentAttention`, `GeneralDelta`), optionally a
+feed-forward spec (`DenseMlp`), and norms before and after every sublayer.  Which design a model directory
+holds is decided by config.json's "architecture" (`DESIGNS`, consulted by model.config_from_dir); a design is
+a reader from its config.json to specs, everything below the specs is shared.  `StackWeights` loads and packs
+the tensors for the kernels (include/bcg_b200.h, bcg_layer); there is nothing model-specific in the engine.
+
+The reference has no counterpart: its engine only ever meets uniform dense decoders (config.py:20-25).
+"""
+from __future__ import annotations
+
+import ctypes as C
+import json
+from dataclasses import dataclass, field, replace
+from pathlib import Path
+from typing import Callable, Dict, Optional, Tuple
+
+import torch
+
+from . import lib as L
+
+
+def _up(n: int, m: int) -> int:
+    return (n + m - 1) // m * m
+
+
+# ------------------------------------------------------------------------------------------ specs
+@dataclass(frozen=True)
+class Rotary:
+    """Rotate-half over the first `dims` entries of the rotated part, frequencies base^(-2i/dims)."""
+    base: float
+    dims: int
+
+
+@dataclass(frozen=True)
+class LatentAttention:
+    """Attention over a compressed cache row (latent, shared rotated key part)."""
+    heads: int
+    dim: int
+    rot_dim: int
+    vdim: int
+    kv_rank: int
+    scale: float
+    rot: Rotary
+    window: int = 0                 # keys a query sees, itself included; 0 = all
+    kv_from: Optional[int] = None   # layer whose cache rows this one reads; None = its own
+    sink: bool = True
+
+    @property
+    def cache_row(self) -> int:
+        return self.kv_rank + self.rot_dim
+
+    @property
+    def out_dim(self) -> int:
+        return self.heads * self.vdim
+
+    @property
+    def q_ld(self) -> int:
+        """Padded q/k head size of the expanded form, 0 when the sizes are not for it."""
+        n = _up(self.dim + self.rot_dim, 64)
+        return n if n <= 256 and self.v_pad and self.vdim % 8 == 0 and self.cache_row % 8 == 0 and self.scale > 0 else 0
+
+    @property
+    def v_pad(self) -> int:
+        return next((v for v in (64, 128, 256) if self.vdim <= v), 0)
+
+    @property
+    def v_ld(self) -> int:
+        return self.v_pad if self.q_ld else 0
+
+    @property
+    def q_row(self) -> int:
+        return self.q_ld or self.dim + self.rot_dim
+
+    def in_rows(self) -> int:
+        return self.heads * (self.dim + self.rot_dim) + (self.cache_row if self.kv_from is None else 0)
+
+    def tensors(self, d: int) -> Dict[str, tuple]:
+        t = {"q": (self.heads * (self.dim + self.rot_dim), d), "uk": (self.heads * self.dim, self.kv_rank),
+             "uv": (self.heads * self.vdim, self.kv_rank), "o": (d, self.out_dim)}
+        if self.sink:
+            t["sink"] = (self.heads,)
+        if self.kv_from is None:
+            t.update({"dkv": (self.cache_row, d), "dkv.norm": (self.kv_rank,)})
+        return t
+
+
+@dataclass(frozen=True)
+class GeneralDelta:
+    """Generalized delta rule: a [dim, dim] fp32 state per head, decay and removal rate per key channel."""
+    heads: int
+    dim: int
+    decay_rank: int
+
+    @property
+    def out_dim(self) -> int:
+        return self.heads * self.dim
+
+    @property
+    def rank_ld(self) -> int:
+        return _up(self.decay_rank, 8)
+
+    def in_rows(self) -> int:
+        return 5 * self.out_dim + self.rank_ld
+
+    def tensors(self, d: int) -> Dict[str, tuple]:
+        n = self.out_dim
+        return {"r": (n, d), "k": (n, d), "v": (n, d), "g": (n, d), "a": (n, d), "a.b": (n,), "w1": (self.decay_rank, d),
+                "w2": (n, self.decay_rank), "w0": (n,), "norm": (n,), "o": (d, n)}
+
+
+@dataclass(frozen=True)
+class DenseMlp:
+    """down(PolyNorm(up(x))); the activation's four numbers are weights."""
+    ff: int
+
+    def tensors(self, d: int) -> Dict[str, tuple]:
+        return {"up": (self.ff, d), "down": (d, self.ff), "act": (4,)}
+
+
+@dataclass(frozen=True)
+class LayerSpec:
+    mixer: object
+    mlp: Optional[DenseMlp] = None
+
+
+@dataclass(frozen=True)
+class StackConfig:
+    name: str
+    d_model: int
+    vocab: int
+    layers: Tuple[LayerSpec, ...]
+    rms_eps: float = 1e-5
+    act_dtype: str = "bfloat16"      # or "float32": everything in true fp32
+    family: str = "qwen3"            # tokenizer / chat-template family
+    max_pos: int = 131072
+
+    def __post_init__(self):
+        if self.d_model % 4 or any(l.mlp and l.mlp.ff % 4 for l in self.layers):
+            raise ValueError(f"{self.name}: width and feed-forward sizes must be multiples of 4")
+        if self.act_dtype not in ("bfloat16", "float32"):
+            raise ValueError(f"act_dtype {self.act_dtype!r}")
+        for i, l in enumerate(self.layers):
+            m = l.mixer
+            if isinstance(m, GeneralDelta) and m.dim > 256:
+                raise ValueError(f"{self.name}: layer {i}: the delta-rule kernel takes up to 256 channels per head")
+            if isinstance(m, LatentAttention):
+                if m.rot.dims % 2 or m.rot.dims > m.rot_dim:
+                    raise ValueError(f"{self.name}: layer {i}: rotary dims {m.rot.dims} of {m.rot_dim}")
+                if m.kv_from is not None:
+                    src = self.layers[m.kv_from].mixer if 0 <= m.kv_from < i else None
+                    if not isinstance(src, LatentAttention) or src.kv_from is not None or src.kv_rank != m.kv_rank \
+                            or src.rot_dim != m.rot_dim:
+                        raise ValueError(f"{self.name}: layer {i} cannot read layer {m.kv_from}'s cache")
+
+    @property
+    def n_layers(self) -> int:
+        return len(self.layers)
+
+    @property
+    def vocab_ld(self) -> int:
+        return _up(self.vocab, 4)
+
+    @property
+    def has_state(self) -> bool:
+        """True when a prefix's cache pages alone do not restore it (recurrent layers)."""
+        return any(isinstance(l.mixer, GeneralDelta) for l in self.layers)
+
+    @property
+    def max_window(self) -> int:
+        """Largest attention window of the stack, 0 = unbounded."""
+        w = [l.mixer.window for l in self.layers if isinstance(l.mixer, LatentAttention)]
+        return 0 if not w or 0 in w else max(w)
+
+    @property
+    def torch_dtype(self):
+        return torch.float32 if self.act_dtype == "float32" else torch.bfloat16
+
+    @property
+    def itemsize(self) -> int:
+        return 4 if self.act_dtype == "float32" else 2
+
+    @property
+    def kv_bytes_per_token(self) -> int:
+        return sum(l.mixer.cache_row for l in self.layers
+                   if isinstance(l.mixer, LatentAttention) and l.mixer.kv_from is None) * self.itemsize
+
+    @property
+    def state_bytes_per_row(self) -> int:
+        return sum(4 * l.mixer.heads * l.mixer.dim ** 2 for l in self.layers if isinstance(l.mixer, GeneralDelta))
+
+    def in_rows(self, i: int) -> int:
+        """Rows of layer i's fused input projection, padded for the 256-wide GEMM tiles when it is large."""
+        n = self.layers[i].mixer.in_rows()
+        return _up(n, 256 if n >= 2048 else 16)
+
+    def tensor_shapes(self) -> Dict[str, tuple]:
+        """Every tensor of the checkpoint, name -> shape."""
+        d = self.d_model
+        out = {"embed": (self.vocab, d), "final.norm": (d,), "head": (self.vocab, d)}
+        for i, l in enumerate(self.layers):
+            out.update({f"l{i}.norm1": (d,), f"l{i}.norm1b": (d,)})
+            out.update({f"l{i}.mix.{n}": s for n, s in l.mixer.tensors(d).items()})
+            if l.mlp:
+                out.update({f"l{i}.norm2": (d,), f"l{i}.norm2b": (d,)})
+                out.update({f"l{i}.mlp.{n}": s for n, s in l.mlp.tensors(d).items()})
+        return out
+
+    def decode_weight_bytes(self) -> int:
+        """bf16 bytes of matrices streamed per decode step."""
+        return 2 * sum(s[0] * s[1] for n, s in self.tensor_shapes().items() if len(s) == 2 and n != "embed")
+
+    def shard(self, tp_size: int) -> "StackConfig":
+        if tp_size != 1:
+            raise ValueError(f"{self.name}: tensor parallelism is not implemented for layer stacks")
+        return self
+
+
+# ------------------------------------------------------------------------------------------ designs
+def _bekopel(c: dict, shape: Callable[[str], tuple], name: str) -> StackConfig:
+    """config.json of the Bekopel design; `shape(tensor)` gives what only the checkpoint states."""
+    layers = []
+    for i, e in enumerate(c["layers"]):
+        m, kind = e["mixer"], e["type"]
+        if kind == "latent_attention":
+            mixer = LatentAttention(heads=int(m["heads"]), dim=int(m["dim"]), rot_dim=int(m["rot_dim"]),
+                                    vdim=int(m["vdim"]), kv_rank=int(m["kv_rank"]), scale=float(m["scale"]),
+                                    rot=Rotary(float(m["rot"]["base"]), int(m["rot"]["dims"])),
+                                    window=int(m["mask"]["size"]),
+                                    kv_from=None if m.get("kv_from") is None else int(m["kv_from"]))
+        elif kind == "general_delta":
+            mixer = GeneralDelta(heads=int(m["heads"]), dim=int(m["dim"]), decay_rank=int(shape(f"l{i}.mix.w1")[0]))
+        else:
+            raise ValueError(f"{name}: layer {i}: unknown mixer {kind!r}")
+        f = e.get("mlp")
+        if f is not None and f.get("kind") != "dense":
+            raise ValueError(f"{name}: layer {i}: unknown feed-forward {f.get('kind')!r}")
+        layers.append(LayerSpec(mixer, DenseMlp(int(f["ff"])) if f is not None else None))
+    return StackConfig(name=name, d_model=int(c["width"]), vocab=int(c["vocab"]), layers=tuple(layers),
+                       rms_eps=float(c["norm"]["eps"]))
+
+
+DESIGNS: Dict[str, Callable] = {"Bekopel": _bekopel}
+
+
+def safetensors_shapes(path) -> Dict[str, tuple]:
+    """Tensor shapes from a safetensors header (the data is not read)."""
+    with open(path, "rb") as f:
+        n = int.from_bytes(f.read(8), "little")
+        head = json.loads(f.read(n))
+    return {k: tuple(v["shape"]) for k, v in head.items() if k != "__metadata__"}
+
+
+def config_from_dir(model_dir, c: dict) -> StackConfig:
+    """StackConfig of a model directory whose config.json `c` names a design in DESIGNS."""
+    path = Path(model_dir) / "model.safetensors"
+    shapes: Dict[str, tuple] = {}
+
+    def shape(n):
+        if not shapes:
+            shapes.update(safetensors_shapes(path))
+        return shapes[n]
+    return DESIGNS[c["architecture"]](c, shape, Path(model_dir).name)
+
+
+def bekopel_preset(name: str, n_layers: int, d_model: int, ff: int, vocab: int, heads: int = 32, dim: int = 128,
+                   rot_dim: int = 64, kv_rank: int = 512, window: int = 1024, decay_rank: int = 128,
+                   max_pos: int = 32768) -> StackConfig:
+    """Bekopel at sizes of a real model's layers (random-init presets, bench): groups of delta, latent attention,
+    latent attention on the same cache, delta."""
+    delta = GeneralDelta(d_model // 128, 128, decay_rank)
+    layers = []
+    for i in range(n_layers):
+        if i % 4 in (1, 2):
+            m = LatentAttention(heads, dim, rot_dim, dim, kv_rank, (dim + rot_dim) ** -0.5, Rotary(1e6, rot_dim), window,
+                                None if i % 4 == 1 else i - 1)
+        else:
+            m = delta
+        layers.append(LayerSpec(m, DenseMlp(ff)))
+    return StackConfig(name, d_model, vocab, tuple(layers), max_pos=max_pos)
+
+
+# ------------------------------------------------------------------------------------------ weights
+def rope_table(rot: Rotary, n_pos: int, device) -> torch.Tensor:
+    """[n_pos, dims] fp32: cos of the dims/2 angles, then sin (angles formed in fp64, rounded once)."""
+    half = rot.dims // 2
+    f = rot.base ** (-2.0 * torch.arange(half, dtype=torch.float64) / rot.dims)
+    ang = torch.arange(n_pos, dtype=torch.float64)[:, None] * f[None, :]
+    return torch.cat([ang.cos(), ang.sin()], dim=1).float().contiguous().to(device)
+
+
+@dataclass
+class StackWeights:
+    """Tensors packed for the kernels: per layer a dict of device tensors named after bcg_layer's fields."""
+    cfg: StackConfig
+    embed: torch.Tensor
+    lm_head: torch.Tensor
+    final_norm: torch.Tensor
+    layers: list = field(default_factory=list)
+
+    @staticmethod
+    def from_tensors(cfg: StackConfig, get: Callable[[str], torch.Tensor], device) -> "StackWeights":
+        """`get(name)` returns a checkpoint tensor (CPU or device, any float dtype)."""
+        want = cfg.tensor_shapes()
+
+        def raw(n):
+            t = get(n)
+            if tuple(t.shape) != want[n]:
+                raise ValueError(f"{cfg.name}: tensor {n} has shape {tuple(t.shape)}, expected {want[n]}")
+            return t.detach().to(device)
+
+        bf = lambda t: t.to(torch.bfloat16).contiguous()
+        f32 = lambda t: t.float().contiguous()
+
+        def rows(t, n):
+            return t if t.shape[0] == n else torch.cat([t, t.new_zeros(n - t.shape[0], *t.shape[1:])])
+
+        w = StackWeights(cfg, bf(raw("embed")), bf(rows(raw("head"), cfg.vocab_ld)), f32(raw("final.norm")))
+        for i, l in enumerate(cfg.layers):
+            m, g = l.mixer, lambda n: raw(f"l{i}.mix.{n}")
+            t = {"norm1": f32(raw(f"l{i}.norm1")), "norm1b": f32(raw(f"l{i}.norm1b")), "w_out": bf(g("o"))}
+            if isinstance(m, LatentAttention):
+                own = m.kv_from is None
+                t["w_in"] = bf(rows(torch.cat([g("q"), g("dkv")]) if own else g("q"), cfg.in_rows(i)))
+                if own:
+                    t["latent_norm"] = f32(g("dkv.norm"))
+                if m.sink:
+                    t["sink"] = f32(g("sink"))
+                t["w_uk"], t["w_uv"] = bf(g("uk")), bf(g("uv"))
+                if m.q_ld and cfg.act_dtype == "bfloat16":
+                    t["w_expand"] = StackWeights.expansion(m, t["w_uk"], t["w_uv"])
+            else:
+                w1 = rows(g("w1"), m.rank_ld)
+                t["w_in"] = bf(rows(torch.cat([g("r"), g("k"), g("v"), g("g"), g("a"), w1]), cfg.in_rows(i)))
+                w2 = g("w2")
+                t["w_decay"] = bf(torch.cat([w2, w2.new_zeros(w2.shape[0], m.rank_ld - m.decay_rank)], dim=1))
+                t["decay_bias"], t["rate_bias"], t["out_norm"] = f32(g("w0")), f32(g("a.b")), f32(g("norm"))
+            if l.mlp:
+                t.update(norm2=f32(raw(f"l{i}.norm2")), norm2b=f32(raw(f"l{i}.norm2b")), w_up=bf(raw(f"l{i}.mlp.up")),
+                         w_down=bf(raw(f"l{i}.mlp.down")), act_coef=f32(raw(f"l{i}.mlp.act")))
+            w.layers.append(t)
+        return w
+
+    @staticmethod
+    def expansion(m: LatentAttention, uk: torch.Tensor, uv: torch.Tensor) -> torch.Tensor:
+        """[heads * (q_ld + v_ld), cache_row]: cache row -> every head's key (up-projected latent, the rotated
+        part through an identity block, zero padding), then every head's value."""
+        k = uk.new_zeros(m.heads, m.q_ld, m.cache_row)
+        k[:, :m.dim, :m.kv_rank] = uk.view(m.heads, m.dim, m.kv_rank)
+        k[:, m.dim:m.dim + m.rot_dim, m.kv_rank:] = torch.eye(m.rot_dim, dtype=uk.dtype, device=uk.device)
+        v = uv.new_zeros(m.heads, m.v_ld, m.cache_row)
+        v[:, :m.vdim, :m.kv_rank] = uv.view(m.heads, m.vdim, m.kv_rank)
+        return torch.cat([k.flatten(0, 1), v.flatten(0, 1)]).contiguous()
+
+    @staticmethod
+    def from_safetensors_dir(cfg: StackConfig, model_dir, device) -> "StackWeights":
+        from safetensors import safe_open
+        with safe_open(str(Path(model_dir) / "model.safetensors"), "pt") as f:
+            return StackWeights.from_tensors(cfg, f.get_tensor, device)
+
+    @staticmethod
+    def random_init(cfg: StackConfig, device, seed: int = 0) -> "StackWeights":
+        """N(0, 0.02) matrices, unit norms, zero biases and sinks, identity-like activation; made on the device."""
+        g = torch.Generator(device=device)
+        g.manual_seed(seed)
+        shapes = cfg.tensor_shapes()
+
+        def get(n):
+            s = shapes[n]
+            if n.endswith(".act"):
+                return torch.tensor([1.0, 0.5, 0.25, 0.0], device=device)
+            if len(s) == 2:
+                return torch.empty(*s, dtype=torch.bfloat16, device=device).normal_(0.0, 0.02, generator=g)
+            leaf = n.rsplit(".", 1)[-1]
+            return (torch.ones if leaf.startswith("norm") else torch.zeros)(*s, device=device)
+        return StackWeights.from_tensors(cfg, get, device)
+
+    def nbytes(self) -> int:
+        ts = [self.embed, self.lm_head] + [t for l in self.layers for t in l.values()]
+        return sum(t.numel() * t.element_size() for t in ts)
+
+
+# ------------------------------------------------------------------------------------------ handle
+class StackHandle:
+    """Host-side bcg_stack (include/bcg_b200.h) over StackWeights, caches and states.
+
+    caches[i]: the latent pages [pages, page, cache_row] or the states [slots, heads, dim, dim] of layer i
+    (None where the layer reads another layer's cache)."""
+
+    def __init__(self, w: StackWeights, caches: list, n_pos: int, page_size: int):
+        cfg = w.cfg
+        self.w, self.caches = w, caches
+        dev = w.embed.device
+        self._rope: Dict[Rotary, torch.Tensor] = {}
+        arr = (L.Layer * cfg.n_layers)()
+        for i, (spec, t) in enumerate(zip(cfg.layers, w.layers)):
+            a, m = arr[i], spec.mixer
+            a.heads, a.dim, a.n_in = m.heads, m.dim, cfg.in_rows(i)
+            src = i
+            if isinstance(m, LatentAttention):
+                a.mixer = L.MIXER_LATENT_ATTN
+                a.rot_dim, a.rot_dims, a.vdim, a.kv_rank = m.rot_dim, m.rot.dims, m.vdim, m.kv_rank
+                a.window, a.scale, a.owns_cache = m.window, m.scale, int(m.kv_from is None)
+                if "w_expand" in t:
+                    a.q_ld, a.v_ld = m.q_ld, m.v_ld
+                src = i if m.kv_from is None else m.kv_from
+                if m.rot not in self._rope:
+                    self._rope[m.rot] = rope_table(m.rot, n_pos, dev)
+                a.cos_sin = self._rope[m.rot].data_ptr()
+            else:
+                a.mixer, a.decay_rank = L.MIXER_GENERAL_DELTA, m.rank_ld
+            a.ff = spec.mlp.ff if spec.mlp else 0
+            for n, x in t.items():
+                setattr(a, n, x.data_ptr())
+            a.cache = caches[src].data_ptr()
+        self._layers = arr
+        s = L.Stack()
+        s.n_layers, s.d_model, s.vocab_ld, s.page_size, s.eps = cfg.n_layers, cfg.d_model, cfg.vocab_ld, page_size, cfg.rms_eps
+        s.act_dtype = L.DT_F32 if cfg.act_dtype == "float32" else L.DT_BF16
+        s.embed, s.lm_head, s.final_norm = w.embed.data_ptr(), w.lm_head.data_ptr(), w.final_norm.data_ptr()
+        s.layers = C.cast(arr, C.POINTER(L.Layer))
+        self.struct = s

@@ -98,13 +98,13 @@ class B200LLM:
             # what the reference gets when vLLM resolves the model name (vllm_agent.py:126-144)
             from .tokenizer import LocalTokenizer
             cfg = M.config_from_dir(model_name)
-            factory = lambda c, dev: M.Weights.from_safetensors_dir(c, model_name, dev)
+            factory = lambda c, dev: M.weights_for(c).from_safetensors_dir(c, model_name, dev)
             if os.path.exists(os.path.join(model_name, "tokenizer.json")):
                 tokenizer = LocalTokenizer(model_name, cfg.vocab, cfg.family)
         else:
             cfg = M.config_for(model_name)
             seed = int(model_config.get("weight_seed", os.environ.get("BCG_B200_WEIGHT_SEED", 0)))
-            factory = lambda c, dev: M.Weights.random_init(c, dev, seed=seed)
+            factory = lambda c, dev: M.weights_for(c).random_init(c, dev, seed=seed)
         device = model_config.get("device", "cuda:0")
         self.cfg = cfg
         self.tokenizer = tokenizer or get_tokenizer(cfg.family, cfg.vocab)

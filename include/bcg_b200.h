@@ -22,7 +22,7 @@
 extern "C" {
 #endif
 
-#define BCG_ABI_VERSION 2
+#define BCG_ABI_VERSION 3
 
 /* status codes */
 #define BCG_STATUS_OK 0
@@ -281,7 +281,7 @@ int bcg_tp_add_norm_stats(float* residual, const float* partials, int n_partials
                           int d, void* stream);
 
 /* Whole-model steps: the layer stack launched from C++ on one stream so a decode step is one
- * host call (captured into a CUDA graph by the engine).  See DESIGN.md §4. */
+ * host call (captured into a CUDA graph by the engine). */
 typedef struct bcg_model {
   /* With tensor parallelism n_heads, n_kv_heads, d_ff and vocab are THIS RANK's shard sizes
    * (column-parallel qkv / gate_up, row-parallel o / down, vocab-parallel lm_head). */
@@ -336,6 +336,9 @@ int bcg_model_prefill(const bcg_model* m, const bcg_workspace* ws, const int* id
                       const int* positions, const int* slot_map, const int* block_table,
                       int max_blocks_per_seq, const int* tile_info, int n_tiles,
                       const int* last_rows, int n_seqs, int T, void* stream);
+/* Logits of `n` more tokens (device list `rows`) of the prefill step just run, into ws->logits rows
+ * row0.. (stands in for vLLM's LogitsProcessor over chosen positions). */
+int bcg_model_head(const bcg_model* m, const bcg_workspace* ws, const int* rows, int n, int row0, void* stream);
 /* One decode step for B rows: ids/positions/slot_map/seq_lens are the arrays bcg_mask_sample
  * maintains; logits land in ws->logits[0..B).  Stands in for one decode step of the same vLLM
  * forward.  flags: BCG_GEMM_PDL, plus how the residual add + RMSNorm between two
@@ -343,7 +346,7 @@ int bcg_model_prefill(const bcg_model* m, const bcg_workspace* ws, const int* id
  *   default                   bcg_add_rmsnorm kernels (complete norm, then the projection)
  *   BCG_STEP_DEFERRED_NORM    bcg_add_norm_stats + 1/RMS applied in the next projection's epilogue
  *   BCG_STEP_FUSED_NORM       the producing projection finishes the residual itself
- *                             (bcg_gemm_bf16_tn_fused producer half; measured slower, DESIGN.md 8) */
+ *                             (bcg_gemm_bf16_tn_fused producer half; measured slower) */
 #define BCG_STEP_FUSED_NORM 0x20000
 #define BCG_STEP_DEFERRED_NORM 0x40000
 #define BCG_STEP_FUSED_ROPE 0x80000 /* bcg_decode_attn_paged_qkv instead of rope kernel + attention */
@@ -351,6 +354,147 @@ int bcg_model_decode(const bcg_model* m, const bcg_workspace* ws, const int* ids
                      const int* positions, const int* slot_map, const int* seq_lens,
                      const int* block_table, int max_blocks_per_seq, int B, int flags,
                      void* stream);
+
+/* ---------------------------------------------------------------------------------------------
+ * Layer stacks: models whose layers differ in kind (the reference has no counterpart; its engine
+ * only meets uniform dense decoders).  Every layer is a mixer and, optionally, a feed-forward, each
+ * with a norm before and a norm after it:  x += norm1b(mixer(norm1(x))),  x += norm2b(ff(norm2(x))).
+ * `act_dtype` selects the activations that feed matrix products, the latent cache and the attention
+ * operands: BCG_DT_BF16 (tensor-core kernels, fp32 accumulation) or BCG_DT_F32 (true fp32
+ * throughout, CUDA-core kernels).  Weights are bf16 in both; the residual, norms, scores, gates and
+ * recurrent states are fp32 in both. */
+#define BCG_DT_BF16 0
+#define BCG_DT_F32 1
+#define BCG_MIXER_LATENT_ATTN 1
+#define BCG_MIXER_GENERAL_DELTA 2
+
+typedef struct bcg_layer {
+  int mixer;               /* BCG_MIXER_* */
+  int heads, dim;          /* latent attention: unrotated q/k dims per head; delta: channels per head */
+  int rot_dim, rot_dims;   /* rotated q/k dims per head, and how many of them rotate (rotate-half) */
+  int vdim, kv_rank;
+  int window;              /* keys a query sees, itself included; 0 = all earlier ones */
+  float scale;
+  int q_ld, v_ld;          /* padded q/k and v head sizes of the expanded form (multiples of 64), 0 = none */
+  int owns_cache;          /* 0: the layer reads `cache`, which an earlier layer writes */
+  int n_in;                /* rows of w_in */
+  int decay_rank;          /* columns of w_decay */
+  int ff;                  /* 0 = no feed-forward */
+  const float* norm1;      /* [d] */
+  const float* norm1b;
+  const float* norm2;
+  const float* norm2b;
+  const void* w_in;        /* bf16 [n_in, d]: latent attention q | down-projection (owners only);
+                              delta r | k | v | g | rate | decay-in; zero rows after */
+  const void* w_out;       /* bf16 [d, heads * (vdim or dim)] */
+  const float* latent_norm; /* [kv_rank] */
+  const float* sink;       /* [heads] or NULL */
+  const float* cos_sin;    /* [max_pos][rot_dims]: cos of the rot_dims/2 angles, then sin */
+  const void* w_uk;        /* bf16 [heads * dim, kv_rank] */
+  const void* w_uv;        /* bf16 [heads * vdim, kv_rank] */
+  const void* w_expand;    /* bf16 [heads * (q_ld + v_ld), kv_rank + rot_dim]: cache row -> all heads' keys
+                              (w_uk rows, then the identity on the rotated part, then zero rows), then
+                              all heads' values; NULL = no expanded form */
+  const float* decay_bias; /* [heads * dim] */
+  const float* rate_bias;  /* [heads * dim] */
+  const float* out_norm;   /* [heads * dim] */
+  const void* w_decay;     /* bf16 [heads * dim, decay_rank] */
+  const void* w_up;        /* bf16 [ff, d] */
+  const void* w_down;      /* bf16 [d, ff] */
+  const float* act_coef;   /* PolyNorm's four numbers (device) */
+  void* cache;             /* latent pages [pages][page_size][kv_rank + rot_dim], or state
+                              fp32 [slots][heads][dim][dim] */
+} bcg_layer;
+
+typedef struct bcg_stack {
+  int n_layers, d_model, vocab_ld; /* vocab_ld: rows of lm_head (vocabulary, padded to a multiple of 4) */
+  int act_dtype, page_size;
+  float eps;
+  const void* embed;        /* bf16 [vocab, d] */
+  const void* lm_head;      /* bf16 [vocab_ld, d] */
+  const float* final_norm;
+  const bcg_layer* layers;  /* host array */
+} bcg_stack;
+
+typedef struct bcg_stack_ws {
+  float* residual;  /* [T_max, d] */
+  void* xn;         /* act [T_max, d]; after a step: the final norm of every row */
+  float* proj;      /* fp32 projection outputs / split-K slabs */
+  long long proj_floats;
+  float* decay;     /* fp32 [T_max, heads * dim] slabs of w_decay */
+  long long decay_floats;
+  void* q;          /* act [T_max, heads * q_row] */
+  void* mix;        /* act [T_max, heads * (vdim or dim)] */
+  void* act;        /* act [T_max, ff] */
+  void* low;        /* act [T_max, decay_rank] */
+  void* latents;    /* bf16 [K_max, kv_rank + rot_dim] gathered cache rows */
+  void* expanded;   /* bf16 [K_max, heads * (q_ld + v_ld)] */
+  void* q_latent;   /* bf16 [D_max, heads, kv_rank + rot_dim]: queries in latent space */
+  void* o_latent;   /* bf16 [D_max, heads, kv_rank] */
+  float* part_o;    /* fp32 decode partials [D_max, chunks, heads, kv_rank], part_floats long */
+  long long part_floats;
+  float* part_ml;   /* fp32 [D_max, chunks, heads, 2] */
+  void* xn_rows;    /* act [B_max, d] */
+  float* logits;    /* fp32 [B_max, vocab_ld] */
+  int T_max, K_max, D_max, B_max;
+} bcg_stack_ws;
+
+/* A step: T new tokens of n_seqs sequences, portions of prompts beside single decoded tokens.  All
+ * pointers are device int32. */
+typedef struct bcg_step_batch {
+  int T, n_seqs;
+  const int* ids;          /* [T] */
+  const int* positions;    /* [T] */
+  const int* slot_map;     /* [T] cache row of each token (< 0: writes nothing, keeps the state) */
+  const int* row_seq;      /* [T] sequence of each token, NULL = token t belongs to sequence t */
+  const int* seq_start;    /* [n_seqs + 1] first token of each sequence, NULL = one token each */
+  const int* block_table;  /* [n_seqs, max_blocks] */
+  int max_blocks;
+  const int* state_slots;  /* [n_seqs] */
+  int max_context;         /* upper bound on positions + 1 of the single tokens (sizes the grid) */
+  /* attention work lists of the bf16 kernels */
+  const int* single_rows;  /* [n_single] tokens attended one by one in latent space, NULL = all T */
+  int n_single;
+  const int* tiles;        /* [n_tiles][8] {first token, its position, tokens (<= 128), expanded row of
+                              key position k0, k0, 0, 0, 0} */
+  int n_tiles;
+  const int* gather;       /* [n_gather] cache row behind every expanded row */
+  int n_gather;
+  int flags;               /* BCG_GEMM_PDL */
+} bcg_step_batch;
+
+/* Runs the layers over a step's tokens: caches and states advanced, ws->residual and ws->xn (final norm)
+ * filled.  One call = prefill, decode or a mixture; the reference has no counterpart (vLLM's
+ * GPUModelRunner.execute_model is the nearest relative). */
+int bcg_stack_step(const bcg_stack* m, const bcg_stack_ws* ws, const bcg_step_batch* b, void* stream);
+/* Logits of `n` tokens of the step just run, in ws->logits rows row0..: rows = device list of token
+ * indices, or NULL = tokens 0..n-1.  The reference has no counterpart of its own (vLLM LogitsProcessor). */
+int bcg_stack_head(const bcg_stack* m, const bcg_stack_ws* ws, const int* rows, int n, int row0, int flags,
+                   void* stream);
+
+/* The mechanisms one by one (what bcg_stack_step launches; the reference has no counterpart).
+ * `in` arguments with n_partials slabs are fp32 split-K outputs added in index order. */
+/* out fp32 [M, ldo] = X [M, ldx] (act_dtype) * W bf16 [N, ldw]^T on CUDA cores, any shape. */
+int bcg_gemm_any(const void* X, int x_dtype, const void* W, float* out, int M, int N, int K, long long ldx,
+                 long long ldw, long long ldo, void* stream);
+/* No counterpart in the reference: residual += w_post ? rmsnorm(delta) * w_post : delta, then
+ * xn = rmsnorm(residual) * w_next (NULL: skipped). */
+int bcg_sandwich_norm(float* residual, const float* delta, int n_partials, long long partial_stride,
+                      const float* w_post, const float* w_next, void* xn, int act_dtype, int T, int d, float eps,
+                      void* stream);
+/* No counterpart in the reference: a N(z) + b N(z^2) + c N(z^3) + e with N = division by the row's RMS. */
+int bcg_poly_norm(const float* z, int n_partials, long long partial_stride, const float* coef, void* out,
+                  int act_dtype, int T, int ff, float eps, void* stream);
+/* No counterpart in the reference: generalized delta rule over ragged sequences; proj rows are
+ * r | k | v | g | rate (heads * dim each, row pitch ld), decay the fp32 pre-activation without its bias. */
+int bcg_delta_scan(const bcg_layer* l, const float* proj, int n_partials, long long partial_stride, long long ld,
+                   const float* decay, int decay_partials, long long decay_stride, const int* positions,
+                   const int* slot_map, const int* seq_start, const int* state_slots, int n_seqs, void* out,
+                   int act_dtype, float eps, void* stream);
+/* No counterpart in the reference: attention of a step's queries (ws->q) over the latent pages.
+ * mode 0: what bcg_stack_step picks; 1: the plain kernel; ws->mix receives the heads' values. */
+int bcg_latent_attention(const bcg_stack* m, const bcg_stack_ws* ws, const bcg_step_batch* b, int layer, int mode,
+                         void* stream);
 
 #ifdef __cplusplus
 }
