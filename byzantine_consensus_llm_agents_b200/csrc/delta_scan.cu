@@ -114,7 +114,9 @@ delta_scan_kernel(const DeltaArgs a, T* __restrict__ out) {
         const int i = q * 32 + lane;
         float w = 0.f, rate = 0.f, v = 0.f;
         if (i < D) {
-          w = expf(-kDecayGain * sigmoid_f32(slab_sum(pd + i, a.d_partials, a.dstride) + a.decay_bias[h * D + i]));
+          // 1 + expm1: rounded once near 1, where channels that remember for long live (an error of one
+          // unit there, repeated at every token, is a drift of the whole memory)
+          w = 1.0f + expm1f(-kDecayGain * sigmoid_f32(slab_sum(pd + i, a.d_partials, a.dstride) + a.decay_bias[h * D + i]));
           rate = sigmoid_f32(slab_sum(p + 4ll * HD + i, a.n_partials, a.pstride) + a.rate_bias[h * D + i]);
           v = slab_sum(p + 2ll * HD + i, a.n_partials, a.pstride);
         }
