@@ -1,0 +1,79 @@
+"""Small random layer-stack models for the tests: config.json dicts of the Bekopel design, their tensors, and
+model directories.  Weights are scaled so that every mechanism moves the logits: scores spread over several
+units, sinks that take a visible share, decays from fast to almost none, all four activation numbers set."""
+import json
+
+import torch
+
+
+def attn(heads=3, dim=16, rot_dim=8, vdim=24, kv_rank=32, window=20, base=1e4, scale=None, kv_from=None, ff=96):
+    m = {"heads": heads, "dim": dim, "rot_dim": rot_dim, "vdim": vdim, "kv_rank": kv_rank, "mask": {"size": window},
+         "rot": {"base": base, "dims": rot_dim}, "scale": scale or 2.0 * (dim + rot_dim) ** -0.5}
+    if kv_from is not None:
+        m["kv_from"] = kv_from
+    return {"type": "latent_attention", "mixer": m, "mlp": {"kind": "dense", "ff": ff} if ff else None}
+
+
+def delta(heads=2, dim=24, ff=96):
+    return {"type": "general_delta", "mixer": {"heads": heads, "dim": dim},
+            "mlp": {"kind": "dense", "ff": ff} if ff else None}
+
+
+def config(layers, width=80, vocab=200, eps=1e-5):
+    return {"architecture": "Bekopel", "layers": layers, "norm": {"eps": eps}, "vocab": vocab, "width": width}
+
+
+def tensors(cfg, seed=0, decay_rank=12):
+    """name -> bf16 tensor, as a checkpoint of the design holds them."""
+    g = torch.Generator().manual_seed(seed)
+    rnd = lambda *s, std=1.0, mean=0.0: (torch.randn(*s, generator=g) * std + mean).to(torch.bfloat16)
+    d, V = cfg["width"], cfg["vocab"]
+    lin = lambda n, k, gain=1.0: rnd(n, k, std=gain * k ** -0.5)
+    t = {"embed": rnd(V, d), "final.norm": rnd(d, std=0.1, mean=1.0), "head": lin(V, d)}
+    for i, l in enumerate(cfg["layers"]):
+        p, m = f"l{i}.", l["mixer"]
+        for n in ("norm1", "norm1b") + (("norm2", "norm2b") if l["mlp"] else ()):
+            t[p + n] = rnd(d, std=0.1, mean=1.0)
+        p += "mix."
+        if l["type"] == "latent_attention":
+            H, qk = m["heads"], m["dim"] + m["rot_dim"]
+            t.update({p + "q": lin(H * qk, d), p + "uk": lin(H * m["dim"], m["kv_rank"]),
+                      p + "uv": lin(H * m["vdim"], m["kv_rank"]), p + "o": lin(d, H * m["vdim"]), p + "sink": rnd(H, mean=1.0)})
+            if "kv_from" not in m:
+                t.update({p + "dkv": lin(m["kv_rank"] + m["rot_dim"], d), p + "dkv.norm": rnd(m["kv_rank"], std=0.1, mean=1.0)})
+        else:
+            n = m["heads"] * m["dim"]
+            t.update({p + x: lin(n, d) for x in ("r", "k", "v", "g", "a")})
+            t.update({p + "a.b": rnd(n, mean=-1.0), p + "w1": lin(decay_rank, d, 2.0), p + "w2": lin(n, decay_rank, 2.0),
+                      p + "w0": rnd(n, std=2.0, mean=-3.0), p + "norm": rnd(n, std=0.1, mean=1.0), p + "o": lin(d, n)})
+        if l["mlp"]:
+            ff = l["mlp"]["ff"]
+            q = f"l{i}.mlp."
+            t.update({q + "up": lin(ff, d), q + "down": lin(d, ff), q + "act": torch.tensor([0.8, 0.6, -0.4, 0.3]).to(torch.bfloat16)})
+    return t
+
+
+def save(cfg, t, path):
+    from safetensors.torch import save_file
+    path.mkdir(parents=True, exist_ok=True)
+    (path / "config.json").write_text(json.dumps(cfg))
+    save_file(t, str(path / "model.safetensors"))
+    return path
+
+
+def stack_config(cfg, t, dtype="bfloat16", name="tiny-stack"):
+    import dataclasses
+
+    from byzantine_consensus_llm_agents_b200 import stack
+    c = stack.DESIGNS[cfg["architecture"]](cfg, lambda n: tuple(t[n].shape), name)
+    return dataclasses.replace(c, act_dtype=dtype)
+
+
+def engine(cfg, t, dtype="bfloat16", tokens=512, rows=4, tokenizer=None, **kw):
+    """Engine over a tiny model; its pages hold `tokens` tokens."""
+    from byzantine_consensus_llm_agents_b200.engine import Engine
+    from byzantine_consensus_llm_agents_b200.stack import StackWeights
+    c = stack_config(cfg, t, dtype)
+    w = StackWeights.from_tensors(c, t.__getitem__, torch.device("cuda:0"))
+    kw = {"max_model_len": tokens, "max_rows": rows, "prefill_tokens": tokens, "kv_pages": tokens // 16, **kw}
+    return Engine(c, w, tokenizer, **kw)

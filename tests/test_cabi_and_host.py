@@ -77,6 +77,9 @@ def test_ctypes_structs_mirror_header():
     assert fields("bcg_sampler_args") == [f[0] for f in L.SamplerArgs._fields_]
     assert fields("bcg_model") == [f[0] for f in L.Model._fields_]
     assert fields("bcg_workspace") == [f[0] for f in L.Workspace._fields_]
+    for name, cls in (("bcg_layer", L.Layer), ("bcg_stack", L.Stack), ("bcg_stack_ws", L.StackWs),
+                      ("bcg_step_batch", L.StepBatch)):
+        assert fields(name) == [f[0] for f in cls._fields_], name
 
 
 def test_missing_library_is_loud(monkeypatch, tmp_path):

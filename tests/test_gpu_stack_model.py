@@ -1,0 +1,298 @@
+"""Layer-stack models through the engine: whole prompts, token by token, portions, mixed batches, reused pages
+and slots, long decoding, greedy generation and trace replay — against the plain oracle."""
+import json
+import subprocess
+import sys
+from pathlib import Path
+
+import numpy as np
+import pytest
+import torch
+
+from oracle import stack_ref as R
+
+import stack_models as SM
+
+pytestmark = pytest.mark.gpu
+ROOT = Path(__file__).resolve().parent.parent
+# rms logit error over rms logit: of 95 % of the positions, and of every one.  (A head whose recurrent output
+# nearly cancels is divided by its own small root mean square: such positions amplify bf16 rounding.)
+TOL = {"float32": 3e-4, "bfloat16": 3e-2}
+WORST = {"float32": 3e-4, "bfloat16": 0.2}
+
+CONFIGS = {
+    # attention first, a cache read by two layers with other windows and head counts, a layer without feed-forward
+    "mixed": SM.config([SM.attn(), SM.delta(), SM.attn(kv_from=0, window=45, heads=5, dim=12, ff=None),
+                        SM.attn(kv_from=0, window=3, vdim=8), SM.delta(heads=3, dim=36, ff=None)]),
+    # everything on the tensor-core kernels, two caches, wide heads
+    "tensor": SM.config([SM.delta(heads=3, dim=64, ff=256), SM.attn(4, 48, 16, 64, 112, 33, ff=256),
+                         SM.attn(8, 32, 32, 32, 96, 70, base=1e6), SM.attn(2, 80, 16, 96, 112, 16, kv_from=1)], width=192, vocab=320),
+    "attention-only": SM.config([SM.attn(window=1), SM.attn(2, 32, 32, 40, 32, 100)], width=64, vocab=101),
+    "delta-only": SM.config([SM.delta(1, 8, ff=None), SM.delta(2, 128)], width=100, vocab=64, eps=1e-3),
+    "one-each": SM.config([SM.attn(1, 8, 8, 8, 16, 5, ff=20)], width=36, vocab=36),
+}
+
+
+class Model:
+    def __init__(self, name, dtype, **kw):
+        self.cfg = CONFIGS[name]
+        self.t = SM.tensors(self.cfg, seed=len(name))
+        self.dtype = dtype
+        self.eng = SM.engine(self.cfg, self.t, dtype, **kw)
+
+    def tokens(self, n, seed=0):
+        return torch.randint(0, self.cfg["vocab"], (n,), generator=torch.Generator().manual_seed(seed)).tolist()
+
+    def oracle(self, toks):
+        return R.forward(self.cfg, self.t, toks)
+
+    def check(self, got, want):
+        got, want = got.double().cpu(), want.double()
+        assert got.shape == want.shape and torch.isfinite(got).all()
+        d = got - want
+        err = (d - d.mean(-1, keepdim=True)).pow(2).mean(-1).sqrt() / want.std(-1).mean()
+        assert err.max().item() < WORST[self.dtype], (err.max().item(), int(err.argmax()))
+        assert err.quantile(0.95).item() < TOL[self.dtype], err.quantile(0.95).item()
+
+    def feed(self, toks, sizes):
+        """Logits of all tokens, fed in portions of the given sizes (the last size repeats)."""
+        s, out, i, k = self.eng.open(), [], 0, 0
+        while i < len(toks):
+            n = min(sizes[min(k, len(sizes) - 1)], len(toks) - i)
+            out.append(self.eng.step([(s, toks[i:i + n], list(range(n)))]))
+            i, k = i + n, k + 1
+        self.eng.close_sequence(s)
+        return torch.cat(out)
+
+
+@pytest.mark.parametrize("dtype", TOL)
+@pytest.mark.parametrize("name", CONFIGS)
+def test_prompt_tokens_and_portions(name, dtype):
+    m = Model(name, dtype)
+    toks = m.tokens(210)
+    want = m.oracle(toks)
+    for sizes in ([210], [1], [2], [130, 1], [1, 3, 2, 17, 64, 5, 16, 31], [7, 150, 4, 1]):
+        m.check(m.feed(toks, sizes), want)
+    assert len(m.eng.pool.free) == m.eng.pool.n_pages and len(m.eng.slots.free) == m.eng.slots.n
+
+
+@pytest.mark.parametrize("name", ["mixed", "tensor"])
+def test_residual_after_every_depth(name):
+    """The residual stream after each layer, by running the first layers only."""
+    full, t = CONFIGS[name], SM.tensors(CONFIGS[name], seed=3)
+    toks = torch.randint(0, full["vocab"], (60,), generator=torch.Generator().manual_seed(1)).tolist()
+    layers = []
+    R.forward(full, t, toks, collect=layers)
+    for k in range(1, len(full["layers"]) + 1):
+        cfg = {**full, "layers": full["layers"][:k]}
+        eng = SM.engine(cfg, {n: x for n, x in t.items() if not n.startswith("l") or int(n[1:n.index(".")]) < k}, "float32")
+        eng.step([(eng.open(), toks, [])])
+        got = eng.buf["residual"][:60 * full["width"]].view(60, -1).double().cpu()
+        assert (got - layers[k - 1]).abs().max() < 2e-4 * layers[k - 1].abs().max(), k
+
+
+@pytest.mark.parametrize("dtype", TOL)
+@pytest.mark.parametrize("name", ["mixed", "tensor"])
+def test_unequal_requests_in_one_batch_equal_each_alone(name, dtype):
+    """Four live requests, portions beside single tokens; pages and slots of finished ones are used again."""
+    m = Model(name, dtype, tokens=448)
+    rng = np.random.default_rng(7)
+    todo = [(m.tokens(n, seed=n), m) for n in (100, 1, 37, 64, 129, 16, 17, 2, 80)]
+    want = {len(t): m.oracle(t) for t, _ in todo}
+    live, got, queue = {}, {}, [t for t, _ in todo]
+    while queue or live:
+        while queue and len(live) < 4:
+            t = queue.pop(0)
+            live[len(t)] = [m.eng.open(), t, 0]
+            got[len(t)] = []
+        work, order = [], []
+        for n, (s, t, at) in live.items():
+            if len(live) > 1 and rng.random() < 0.25:
+                continue                                             # left out of this step, goes on later
+            k = min(int(rng.choice([1, 1, 2, 5, 33, 64])), n - at)
+            work.append((s, t[at:at + k], list(range(k))))
+            order.append((n, k))
+        if not work:
+            continue
+        out = m.eng.step(work)
+        for n, k in order:
+            got[n].append(out[:k])
+            out = out[k:]
+            live[n][2] += k
+            if live[n][2] == n:
+                m.eng.close_sequence(live.pop(n)[0])
+    for n, parts in got.items():
+        m.check(torch.cat(parts), want[n])
+    assert len(m.eng.pool.free) == m.eng.pool.n_pages and len(m.eng.slots.free) == m.eng.slots.n
+
+
+def test_wanted_places_only_and_in_order():
+    m = Model("mixed", "float32", logit_rows=3)           # fewer logit rows than wanted: several head launches
+    a, b = m.tokens(50, 1), m.tokens(30, 2)
+    sa, sb = m.eng.open(), m.eng.open()
+    out = m.eng.step([(sa, a, [0, 49, 7, 8, 9]), (sb, b, [29, 3])])
+    want = torch.cat([m.oracle(a)[[0, 49, 7, 8, 9]], m.oracle(b)[[29, 3]]])
+    m.check(out, want)
+    assert m.eng.step([(sa, [1, 2], [])]).shape == (0, m.cfg["vocab"])
+
+
+def test_step_longer_than_a_launch_is_cut():
+    m = Model("tensor", "float32", tokens=256, kv_pages=48)
+    a, b = m.tokens(250, 1), m.tokens(200, 2)
+    sa, sb = m.eng.open(), m.eng.open()
+    out = m.eng.step([(sa, a, [249]), (sb, b, [0, 199])])
+    m.check(out, torch.cat([m.oracle(a)[[249]], m.oracle(b)[[0, 199]]]))
+
+
+def test_pool_is_as_large_as_asked_and_says_when_it_is_full():
+    m = Model("mixed", "bfloat16", tokens=64)
+    s = m.eng.open()
+    m.eng.step([(s, m.tokens(64), [])])
+    with pytest.raises(Exception, match="max_model_len"):
+        m.eng.step([(s, [1], [])])
+    with pytest.raises(MemoryError):
+        m.eng.step([(m.eng.open(), [1], [])])
+    m.eng.close_sequence(s)
+    m.eng.step([(m.eng.open(), m.tokens(64), [])])
+
+
+@pytest.mark.parametrize("dtype", TOL)
+def test_long_decoding(dtype):
+    """Windows pass over decoded tokens many times over; the state is carried through every one of them."""
+    m = Model("mixed", dtype)
+    toks = m.tokens(400, 9)
+    m.check(m.feed(toks, [3, 1]), m.oracle(toks))
+
+
+@pytest.mark.parametrize("dtype", ["float32"])
+def test_a_far_token_is_remembered(dtype):
+    """Slow decays: logits hundreds of tokens later depend on the first ones (a lost state would show)."""
+    m = Model("mixed", dtype)
+    for n in ("l1.mix.w0", "l4.mix.w0"):
+        m.t[n] -= 6.0
+    m.eng = SM.engine(m.cfg, m.t, dtype)
+    toks = m.tokens(300, 4)
+    want = m.oracle(toks)
+    other = m.oracle(m.tokens(8, 5) + toks[8:])
+    assert (want[-1] - other[-1]).std() / want[-1].std() > 50 * TOL[dtype]
+    for sizes in ([300], [90, 2, 1]):
+        m.check(m.feed(toks, sizes), want)
+
+
+# ------------------------------------------------------------------------------------------ generation
+GEN = SM.config([SM.delta(heads=2, dim=32), SM.attn(4, 32, 32, 32, 64, 24), SM.attn(2, 32, 32, 64, 64, 40, kv_from=1), SM.delta(2, 40)],
+                width=128, vocab=1024)
+
+
+def _greedy(t, ids, n, out):
+    """The oracle's greedy continuation, following `out` where two logits are within rounding of each other."""
+    lg = R.forward(GEN, t, ids + out[:-1])[len(ids) - 1:]
+    for i, tok in enumerate(out):
+        top = lg[i].max()
+        assert top - lg[i][tok] < 0.15 * lg[i].std(), (i, tok, int(lg[i].argmax()))
+    return [int(x.argmax()) for x in lg]
+
+
+@pytest.mark.parametrize("graph", [False, True])
+@pytest.mark.parametrize("dtype", TOL)
+def test_greedy_generation_through_the_scheduler(dtype, graph):
+    from byzantine_consensus_llm_agents_b200.engine import Request
+    from byzantine_consensus_llm_agents_b200.tokenizer import get_tokenizer
+    t = SM.tensors(GEN, seed=2)
+    tk = get_tokenizer("qwen3", GEN["vocab"])
+    eng = SM.engine(GEN, t, dtype, tokens=256, rows=3, tokenizer=tk, kv_pages=64, use_cuda_graph=graph)
+    g = torch.Generator().manual_seed(0)
+    prompts = [torch.randint(0, 700, (n,), generator=g).tolist() for n in (70, 1, 16, 33, 5)]    # two waves of rows
+    res = eng.generate([Request("", prompt_ids=p, max_tokens=m) for p, m in zip(prompts, (40, 60, 25, 30, 64))])
+    again = eng.generate([Request("", prompt_ids=prompts[3], max_tokens=30)])[0]
+    same = 0
+    for p, r in zip(prompts, res):
+        assert r.token_ids and r.finish in ("length", "stop")
+        want = _greedy(t, p, len(r.token_ids), r.token_ids)
+        same += sum(a == b for a, b in zip(want, r.token_ids))
+    total = sum(len(r.token_ids) for r in res)
+    assert same >= total * (0.995 if dtype == "float32" else 0.9), (same, total)
+    if dtype == "float32":
+        assert again.token_ids == res[3].token_ids
+    assert len(eng.slots.free) == eng.slots.n and len(eng.pool.free) == eng.pool.n_pages
+
+
+def test_adapter_generates_from_a_model_directory(tmp_path):
+    """The agents' entry point: a directory as model name, a JSON schema, greedy."""
+    from byzantine_consensus_llm_agents_b200 import vllm_agent as VA
+    from byzantine_consensus_llm_agents_b200.stack import StackWeights
+    t = SM.tensors(GEN, seed=2)
+    d = SM.save(GEN, t, tmp_path / "stack-model")
+    schema = {"type": "object", "properties": {"decision": {"type": "string", "enum": ["stop", "continue"]}},
+              "required": ["decision"], "additionalProperties": False}
+    mc = {"max_model_len": 512, "gpu_memory_utilization": 0.5, "kv_pages": 200, "engine_max_rows": 4,
+          "tensor_parallel_size": 1, "max_num_seqs": 4, "seed": 3}
+    rows = [("You are agent_%d." % i, "Vote now.", schema if i % 2 else None) for i in range(6)]
+
+    def play(name):
+        a = VA.VLLMAgent("agent_0", name, mc)
+        out = [a.generate_json("Vote now.", schema, temperature=0.0, max_tokens=40, system_prompt="You are agent_0.")]
+        out += a.batch_generate_json([r for r in rows if r[2]], temperature=0.7, max_tokens=40)
+        return out + a.batch_generate([s + u for s, u, _ in rows], temperature=0.0, max_tokens=20)
+    try:
+        from_dir = play(str(d))
+        assert all("raw" not in r or r["raw"].startswith("{") for r in from_dir if isinstance(r, dict))
+        VA.register_model("test/stack", SM.stack_config(GEN, t),
+                          lambda cfg, dev: StackWeights.from_tensors(cfg, t.__getitem__, dev))
+        assert play("test/stack") == from_dir
+    finally:
+        VA.VLLMAgent.shutdown()
+
+
+# ------------------------------------------------------------------------------------------ trace replay
+@pytest.mark.parametrize("dtype", TOL)
+def test_trace_replay_program(tmp_path, dtype):
+    cfg = CONFIGS["tensor"]
+    t = SM.tensors(cfg, seed=11)
+    d, out = SM.save(cfg, t, tmp_path / "m"), tmp_path / "out"
+    out.mkdir()
+    toks = {i: torch.randint(0, cfg["vocab"], (n,), generator=torch.Generator().manual_seed(n)).tolist()
+            for i, n in (("a", 90), ("b", 40), ("c", 64), ("d", 120))}
+    plan = [([("a", 60, [0, 59]), ("b", 40, [39])], ["b"]), ([("a", 1, [0]), ("c", 64, [])], ["c"]),
+            ([("a", 1, []), ("d", 20, [3])], []), ([("d", 2, [1])], []), ([("a", 28, [27]), ("d", 98, [97, 0])], ["a", "d"])]
+    at, lines, want = {}, [], {}
+    for n, (entries, end) in enumerate(plan):
+        e = []
+        for i, k, w in entries:
+            lo = at.get(i, 0)
+            e.append({"id": i, "tokens": toks[i][lo:lo + k], "want": w})
+            want.setdefault(n, []).extend((i, lo + x) for x in w)
+            at[i] = lo + k
+        lines.append(json.dumps({"step": n, "entries": e, "end": end}))
+    p = subprocess.run([str(ROOT / "bin" / "trace_run"), "--model", str(d), "--dtype", dtype, "--out", str(out),
+                        "--max-tokens", "256"], input="\n".join(lines) + "\n", capture_output=True, text=True, timeout=300)
+    assert p.returncode == 0, p.stderr[-2000:]
+    assert [x for x in p.stdout.splitlines() if x.startswith("done")] == [f"done {n}" for n in range(len(plan))]
+    ref = {i: R.forward(cfg, t, x) for i, x in toks.items()}
+    for n, w in want.items():
+        f = out / f"{n}.f32"
+        assert f.exists() == bool(w)
+        if w:
+            got = torch.from_numpy(np.fromfile(f, "<f4")).view(len(w), cfg["vocab"]).double()
+            exp = torch.stack([ref[i][k] for i, k in w])
+            assert ((got - exp).pow(2).mean(-1).sqrt() / exp.std(-1)).max() < WORST[dtype]
+
+
+def test_dense_models_step_and_refuse_float32(tmp_path):
+    """The step interface over a uniform dense decoder: portions and mixed batches equal whole prompts."""
+    from byzantine_consensus_llm_agents_b200 import trace
+    from byzantine_consensus_llm_agents_b200.engine import Engine
+    from byzantine_consensus_llm_agents_b200.model import ModelConfig, Weights
+    from oracle.model import build_hf_model, full_logits
+    cfg = ModelConfig("dense", n_layers=2, d_model=256, n_heads=4, n_kv_heads=2, d_ff=512, vocab=4096)
+    hf = build_hf_model(cfg, seed=0)
+    w = Weights.from_hf_state_dict(cfg, hf.state_dict(), torch.device("cuda:0"))
+    eng = Engine(cfg, w, None, max_model_len=256, max_rows=4, prefill_tokens=256, kv_pages=40)
+    a, b = list(range(5, 155)), list(range(900, 960))
+    sa, sb = eng.open(), eng.open()
+    out = [eng.step([(sa, a[:70], [69, 3])]), eng.step([(sa, a[70:71], [0]), (sb, b, list(range(60)))]), eng.step([(sa, a[71:], [78])])]
+    ra, rb = full_logits(hf, a), full_logits(hf, b)
+    want = torch.cat([ra[[69, 3]], ra[[70]], rb, ra[[149]]])
+    assert (torch.cat(out).cpu() - want).abs().max() < 2e-2
+    hf.save_pretrained(str(tmp_path / "hf"), safe_serialization=True)
+    assert trace.build_engine(str(tmp_path / "hf"), "float32", 256) is None

@@ -1,0 +1,148 @@
+"""Layer stacks, host side (no GPU): reading a design's configuration, packing weights, the oracle's own
+consistency, work lists of ragged steps, pools."""
+import numpy as np
+import pytest
+import torch
+
+from byzantine_consensus_llm_agents_b200 import model as M
+from byzantine_consensus_llm_agents_b200 import stack as S
+from byzantine_consensus_llm_agents_b200.engine import SlotPool
+from byzantine_consensus_llm_agents_b200.executors import Entry, StackExecutor
+from oracle import stack_ref as R
+
+import stack_models as SM
+
+CFG = SM.config([SM.delta(), SM.attn(), SM.attn(kv_from=1, window=33, heads=2, ff=None), SM.delta(heads=1, dim=40, ff=None)])
+
+
+def test_config_comes_from_the_directory(tmp_path):
+    t = SM.tensors(CFG)
+    c = M.config_from_dir(str(SM.save(CFG, t, tmp_path / "m")))
+    assert isinstance(c, S.StackConfig) and M.weights_for(c) is S.StackWeights
+    assert set(c.tensor_shapes()) == set(t)
+    assert all(tuple(t[n].shape) == s for n, s in c.tensor_shapes().items())
+    assert [type(l.mixer).__name__ for l in c.layers] == ["GeneralDelta", "LatentAttention", "LatentAttention", "GeneralDelta"]
+    assert c.layers[2].mixer.kv_from == 1 and c.layers[2].mixer.window == 33 and c.layers[2].mlp is None
+    assert c.layers[0].mixer.decay_rank == 12          # stated by the checkpoint only
+    assert c.has_state and c.max_window == 33
+    assert c.kv_bytes_per_token == 2 * (32 + 8)        # one cache for both attention layers
+    assert c.state_bytes_per_row == 4 * (2 * 24 * 24 + 40 * 40)
+
+
+@pytest.mark.parametrize("spoil, words", [
+    (lambda c: c["layers"][0].update(type="other"), "unknown mixer"),
+    (lambda c: c["layers"][0]["mlp"].update(kind="moe"), "unknown feed-forward"),
+    (lambda c: c["layers"][2]["mixer"].update(kv_from=0), "cannot read"),
+    (lambda c: c["layers"][2]["mixer"].update(kv_rank=64), "cannot read"),
+    (lambda c: c["layers"][1]["mixer"]["rot"].update(dims=10), "rotary"),
+    (lambda c: c.update(width=81), "multiples of 4"),
+])
+def test_bad_configurations_are_refused(spoil, words):
+    import copy
+    c = copy.deepcopy(CFG)
+    spoil(c)
+    with pytest.raises(ValueError, match=words):
+        SM.stack_config(c, SM.tensors(CFG))
+
+
+def test_wrong_tensor_shape_is_refused():
+    t = SM.tensors(CFG)
+    c = SM.stack_config(CFG, t)
+    t["l1.mix.uk"] = t["l1.mix.uk"][:-1]
+    with pytest.raises(ValueError, match="l1.mix.uk"):
+        S.StackWeights.from_tensors(c, t.__getitem__, "cpu")
+
+
+def test_expansion_matrix_builds_keys_and_values():
+    m = S.LatentAttention(heads=3, dim=20, rot_dim=12, vdim=40, kv_rank=28, scale=1.0, rot=S.Rotary(1e4, 12))
+    uk, uv, row = torch.randn(60, 28), torch.randn(120, 28), torch.randn(5, 40)
+    e = (row @ S.StackWeights.expansion(m, uk, uv).T)
+    k, v = e[:, :3 * m.q_ld].view(5, 3, m.q_ld), e[:, 3 * m.q_ld:].view(5, 3, m.v_ld)
+    assert torch.allclose(k[..., :20].flatten(1), row[:, :28] @ uk.T, atol=1e-5)
+    assert torch.equal(k[..., 20:32], row[:, None, 28:].expand(5, 3, 12)) and not k[..., 32:].any()
+    assert torch.allclose(v[..., :40].flatten(1), row[:, :28] @ uv.T, atol=1e-5) and not v[..., 40:].any()
+
+
+def test_packed_rows_are_padded_with_zeros():
+    t = SM.tensors(CFG)
+    w = S.StackWeights.from_tensors(SM.stack_config(CFG, t), t.__getitem__, "cpu")
+    l0, n = w.layers[0], 2 * 24
+    assert l0["w_in"].shape[0] % 16 == 0 and torch.equal(l0["w_in"][5 * n:5 * n + 12], t["l0.mix.w1"])
+    assert not l0["w_in"][5 * n + 12:].any() and l0["w_decay"].shape == (n, 16) and not l0["w_decay"][:, 12:].any()
+    assert "latent_norm" not in w.layers[2] and w.layers[2]["w_in"].shape[0] == 48
+
+
+def test_preset_resolves_by_name():
+    c = M.config_for("bekopel-8b")
+    assert isinstance(c, S.StackConfig) and c.d_model == M.PRESETS["qwen3-8b"].d_model
+    with pytest.raises(ValueError, match="tensor parallelism"):
+        c.shard(2)
+
+
+# ---------------------------------------------------------------------------------------- work lists
+def _exec(history=10, D_max=4, K_max=1 << 20):
+    x = StackExecutor.__new__(StackExecutor)
+    x.history, x.D_max, x.K_max, x.T_max = history, D_max, K_max, 512
+    return x
+
+
+def test_plan_separates_portions_from_single_tokens():
+    rows = np.arange(3 * 20, dtype=np.int32).reshape(3, 20)
+    p = _exec().plan([Entry([7], 40, rows[0], 2, [0]), Entry(list(range(150)), 25, rows[1], 0, [0, 149]),
+                      Entry([1, 2], 0, rows[2], 1, [])])
+    a = p.arrays
+    assert p.T == 153 and p.n_seqs == 3 and p.n_want == 3 and list(a["rows"]) == [0, 1, 150]
+    assert list(a["seq_start"]) == [0, 1, 151, 153] and list(a["state_slots"]) == [2, 0, 1]
+    assert list(a["singles"]) == [0, 151, 152] and p.extra["context"] == 41
+    t = a["tiles"].reshape(-1, 8)
+    assert [list(x[:5]) for x in t] == [[1, 25, 128, 0, 15], [129, 153, 22, 0, 15]]
+    keys = np.arange(15, 175)                       # window history of ten keys, then the portion itself
+    assert list(a["gather"]) == list(rows[1][keys // 16] * 16 + keys % 16)
+    assert list(a["slots"][:2]) == [rows[0][2] * 16 + 8, rows[1][1] * 16 + 9]
+
+
+def test_plan_keeps_a_place_for_every_single_token():
+    rows = np.zeros((4, 20), np.int32)
+    p = _exec(D_max=4).plan([Entry([1, 2, 3], 0, rows[i], i) for i in range(2)] + [Entry([1], 0, rows[i], i) for i in (2, 3)])
+    assert len(p.arrays["singles"]) <= 4 and p.extra["n_tiles"] == 2
+
+
+def test_slot_pool_reuses_and_refuses():
+    p = SlotPool(2)
+    a, b = p.alloc(), p.alloc()
+    with pytest.raises(MemoryError):
+        p.alloc()
+    p.release(a)
+    assert p.alloc() == a and a != b
+
+
+# ---------------------------------------------------------------------------------------- oracle
+def test_oracle_window_and_sink():
+    v = R.window_visible(6, 3)
+    assert v[5].tolist() == [False, False, False, True, True, True] and v[0].tolist() == [True] + [False] * 5
+    s = torch.zeros(1, 2, 2, dtype=torch.float64)
+    p = R.softmax_with_sink(s, R.window_visible(2, 2), torch.tensor([0.0], dtype=torch.float64))
+    assert torch.allclose(p[0], torch.tensor([[0.5, 0.0], [1 / 3, 1 / 3]], dtype=torch.float64))
+
+
+def test_oracle_delta_state_can_be_carried():
+    g = torch.Generator().manual_seed(1)
+    r, k, v = (torch.randn(9, 2, 5, generator=g, dtype=torch.float64) for _ in range(3))
+    w, a = (torch.rand(9, 2, 5, generator=g, dtype=torch.float64) for _ in range(2))
+    whole, s = R.delta_scan(r, k, v, w, a)
+    o1, s1 = R.delta_scan(r[:4], k[:4], v[:4], w[:4], a[:4])
+    o2, s2 = R.delta_scan(r[4:], k[4:], v[4:], w[4:], a[4:], s1)
+    assert torch.allclose(whole, torch.cat([o1, o2])) and torch.allclose(s, s2)
+    # one step by hand: removal uses the unit key and the old state
+    u = k[4] / torch.sqrt((k[4] ** 2).sum(-1, keepdim=True) + 1e-6)
+    seen = (u[:, :, None] * s1).sum(1)
+    want = w[4][:, :, None] * s1 - (a[4] * u)[:, :, None] * seen[:, None] + k[4][:, :, None] * v[4][:, None]
+    assert torch.allclose(R.delta_scan(r[4:5], k[4:5], v[4:5], w[4:5], a[4:5], s1)[1], want)
+
+
+def test_oracle_rotation_turns_pairs():
+    x = torch.tensor([[1.0, 0.0, 0.0, 2.0, 9.0]], dtype=torch.float64)
+    y = R.rotate(x, torch.tensor([3]), 4, 100.0)
+    c, s = np.cos(3.0), np.sin(3.0)
+    c2, s2 = np.cos(0.3), np.sin(0.3)
+    assert torch.allclose(y, torch.tensor([[c, -2 * s2, s, 2 * c2, 9.0]], dtype=torch.float64))
