@@ -5,20 +5,24 @@
 //
 // Columns of S evolve independently given (r, k, w, a, u), so a head is spread over threads by columns: a
 // lane holds DIM/8 rows of CPT columns in registers (rows interleaved by fours over the warp's eight row
-// groups), a warp 4*CPT columns, a CTA 32*CPT columns and a cluster of CL CTAs the whole head.  Few (sequence,
-// head) pairs take the many-CTA shape, many take the one-CTA shape.  Tokens are worked off in chunks: all
-// gates, unit keys and the two scalars below are prepared for a chunk in parallel, then the recurrence runs
-// over the chunk without a barrier.  Both products of a step read the old state,
+// groups), a warp 4*CPT columns, and the scan warps of a CTA - or of a cluster of CL CTAs - the whole head.
+// Both products of a step read the old state,
 //     o = (r*w)^T S - (r . (a*u)) (u^T S) + (r . k) v,
 // so their reductions overlap and the state update is off the critical path.  Everything is fp32 FMA.
+//
+// Two kernels share this core:
+//   delta_token   one token per sequence (decode): streams the state through registers; the state is
+//                 requested before the dependency wait
+//   delta_scan    portions of prompts: scan warps run the recurrence over a chunk of tokens without a barrier
+//                 while preparation warps turn the next chunk's projections into operands (unit keys, gates,
+//                 the two scalars) and finish the previous chunk's outputs.  Few (sequence, head) pairs take
+//                 the many-CTA shape, many take the one-CTA shape.
 #include "attn_tcgen05.cuh"
 #include "stack_common.cuh"
 #include "kernels.h"
 
 namespace bcg {
 
-constexpr int kDsThreads = 256;
-constexpr int kDsChunk = 16;
 constexpr float kDecayGain = 0.60653065971263342f;   // exp(-1/2)
 
 struct DeltaArgs {
@@ -31,7 +35,7 @@ struct DeltaArgs {
   const float *decay_bias, *rate_bias, *out_norm;
   const int *positions, *slot_map, *seq_start, *state_slots;
   float* state;
-  int heads, dim, chunk;
+  int heads, dim;
   float eps;
 };
 
@@ -48,226 +52,434 @@ delta_low_kernel(const float* __restrict__ proj, int n_partials, long long pstri
   low[i] = from_f32<T>(tanhf(slab_sum(proj + t * ld + col0 + (i - t * rank), n_partials, pstride)));
 }
 
-template <typename T, int DP, int CPT>
-__global__ void __launch_bounds__(kDsThreads)
-delta_scan_kernel(const DeltaArgs a, T* __restrict__ out) {
-  constexpr int kCols = kDsThreads / 32 * 4 * CPT;     // columns per CTA
-  constexpr int CL = DP / kCols;
-  constexpr int kQ = DP / 32;                           // float4 groups of rows per lane
-  extern __shared__ float4 ds_raw[];
-  __shared__ float ra_s[kDsChunk], rk_s[kDsChunk], part_s[2][kDsChunk];
-  float* su = reinterpret_cast<float*>(ds_raw);         // [chunk][DP] each
-  const int C = a.chunk, D = a.dim, HD = a.heads * a.dim;
-  float* srw = su + C * DP;
-  float* sw = srw + C * DP;
-  float* sau = sw + C * DP;
-  float* sk = sau + C * DP;
-  float* sv = sk + C * DP;
-  float* so = sv + C * DP;                              // [chunk][kCols]
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const int rg = lane >> 2;
-  const int cta = CL > 1 ? static_cast<int>(blockIdx.x) : 0;
-  const int h = blockIdx.y, s = blockIdx.z;
-  pdl_launch_dependents();
-  pdl_wait();
-  const int t0 = a.seq_start ? a.seq_start[s] : s;
-  const int t1 = a.seq_start ? a.seq_start[s + 1] : s + 1;
-  if (t1 <= t0 || a.slot_map[t0] < 0) return;           // nothing to do (the same for the whole cluster)
-  const bool fresh = a.positions[t0] == 0;
-  const int lcol = warp * 4 * CPT + (lane & 3) * CPT;   // first column within the CTA
-  const int col = cta * kCols + lcol;
-  float* st = a.state + (static_cast<long long>(a.state_slots[s]) * a.heads + h) * D * D;
-  uint64_t S[CPT][kQ * 2];
-#pragma unroll
-  for (int q = 0; q < kQ; ++q)
-#pragma unroll
-    for (int e = 0; e < 2; ++e) {
-      const int i = q * 32 + rg * 4 + e * 2;
-#pragma unroll
-      for (int c = 0; c < CPT; ++c) {
-        float x = 0.f, y = 0.f;
-        if (!fresh && col + c < D) {
-          if (i < D) x = st[static_cast<long long>(i) * D + col + c];
-          if (i + 1 < D) y = st[static_cast<long long>(i + 1) * D + col + c];
-        }
-        S[c][q * 2 + e] = pack_f32x2(__float_as_uint(x), __float_as_uint(y));
-      }
-    }
+// ------------------------------------------------------------------------------------------- core
+// One lane's share of a head's state: rows q*32 + rg*4 + {0..3}, q < DP/32, of columns col .. col + CPT - 1.
+template <int DP, int CPT>
+struct StateTile {
+  static constexpr int kQ = DP / 32;
+  uint64_t s[CPT][kQ * 2];
 
-  auto prepare = [&](int tb, int n) {
-    for (int j = warp; j < n; j += kDsThreads / 32) {
-      const long long t = tb + j;
-      const float* p = a.proj + t * a.ld + static_cast<long long>(h) * D;
-      const float* pd = a.decay + t * HD + static_cast<long long>(h) * D;
-      float kk[kQ], ss = 0.f, r[kQ], au[kQ];
+  __device__ __forceinline__ void zero() {
 #pragma unroll
-      for (int q = 0; q < kQ; ++q) {
-        const int i = q * 32 + lane;
-        kk[q] = i < D ? slab_sum(p + HD + i, a.n_partials, a.pstride) : 0.f;
-        r[q] = i < D ? slab_sum(p + i, a.n_partials, a.pstride) : 0.f;
-        ss += kk[q] * kk[q];
-      }
-      const float inv = rsqrtf(warp_sum(ss) + 1e-6f);
-      float ra = 0.f, rk = 0.f;
+    for (int c = 0; c < CPT; ++c)
 #pragma unroll
-      for (int q = 0; q < kQ; ++q) {
-        const int i = q * 32 + lane;
-        float w = 0.f, rate = 0.f, v = 0.f;
-        if (i < D) {
-          // 1 + expm1: rounded once near 1, where channels that remember for long live (an error of one
-          // unit there, repeated at every token, is a drift of the whole memory)
-          w = 1.0f + expm1f(-kDecayGain * sigmoid_f32(slab_sum(pd + i, a.d_partials, a.dstride) + a.decay_bias[h * D + i]));
-          rate = sigmoid_f32(slab_sum(p + 4ll * HD + i, a.n_partials, a.pstride) + a.rate_bias[h * D + i]);
-          v = slab_sum(p + 2ll * HD + i, a.n_partials, a.pstride);
-        }
-        const float u = kk[q] * inv;
-        au[q] = rate * u;
-        ra = fmaf(r[q], au[q], ra);
-        rk = fmaf(r[q], kk[q], rk);
-        su[j * DP + i] = u;
-        srw[j * DP + i] = r[q] * w;
-        sw[j * DP + i] = w;
-        sau[j * DP + i] = au[q];
-        sk[j * DP + i] = kk[q];
-        sv[j * DP + i] = v;
-      }
-      ra = warp_sum(ra);
-      rk = warp_sum(rk);
-      if (lane == 0) {
-        ra_s[j] = ra;
-        rk_s[j] = rk;
-      }
-    }
-  };
-
-  prepare(t0, min(C, t1 - t0));
-  __syncthreads();
-  for (int tb = t0, par = 0; tb < t1; tb += C, par ^= 1) {
-    const int n = min(C, t1 - tb);
-    for (int j = 0; j < n; ++j) {
-      uint64_t d2[CPT], o2[CPT];
-#pragma unroll
-      for (int c = 0; c < CPT; ++c) d2[c] = o2[c] = 0ull;
-#pragma unroll
-      for (int q = 0; q < kQ; ++q) {
-        const ulonglong2 u = *reinterpret_cast<const ulonglong2*>(su + j * DP + q * 32 + rg * 4);
-        const ulonglong2 rw = *reinterpret_cast<const ulonglong2*>(srw + j * DP + q * 32 + rg * 4);
-#pragma unroll
-        for (int c = 0; c < CPT; ++c) {
-          d2[c] = fma_f32x2(u.x, S[c][q * 2], d2[c]);
-          o2[c] = fma_f32x2(rw.x, S[c][q * 2], o2[c]);
-          d2[c] = fma_f32x2(u.y, S[c][q * 2 + 1], d2[c]);
-          o2[c] = fma_f32x2(rw.y, S[c][q * 2 + 1], o2[c]);
-        }
-      }
-      float d[CPT], o[CPT];
-#pragma unroll
-      for (int c = 0; c < CPT; ++c) {
-        float x, y;
-        unpack_f32x2(d2[c], x, y);
-        d[c] = x + y;
-        unpack_f32x2(o2[c], x, y);
-        o[c] = x + y;
-      }
-#pragma unroll
-      for (int m = 4; m < 32; m <<= 1)
-#pragma unroll
-        for (int c = 0; c < CPT; ++c) {
-          d[c] += __shfl_xor_sync(0xffffffffu, d[c], m);
-          o[c] += __shfl_xor_sync(0xffffffffu, o[c], m);
-        }
-      uint64_t v2[CPT], nd2[CPT];
-#pragma unroll
-      for (int c = 0; c < CPT; ++c) {
-        const float v = sv[j * DP + col + c];
-        if (rg == 0) so[j * kCols + lcol + c] = fmaf(rk_s[j], v, fmaf(-ra_s[j], d[c], o[c]));
-        v2[c] = pack_f32x2(__float_as_uint(v), __float_as_uint(v));
-        nd2[c] = pack_f32x2(__float_as_uint(-d[c]), __float_as_uint(-d[c]));
-      }
-#pragma unroll
-      for (int q = 0; q < kQ; ++q) {
-        const ulonglong2 w = *reinterpret_cast<const ulonglong2*>(sw + j * DP + q * 32 + rg * 4);
-        const ulonglong2 au = *reinterpret_cast<const ulonglong2*>(sau + j * DP + q * 32 + rg * 4);
-        const ulonglong2 k = *reinterpret_cast<const ulonglong2*>(sk + j * DP + q * 32 + rg * 4);
-#pragma unroll
-        for (int c = 0; c < CPT; ++c) {
-          S[c][q * 2] = fma_f32x2(w.x, S[c][q * 2], fma_f32x2(au.x, nd2[c], mul_f32x2(k.x, v2[c])));
-          S[c][q * 2 + 1] = fma_f32x2(w.y, S[c][q * 2 + 1], fma_f32x2(au.y, nd2[c], mul_f32x2(k.y, v2[c])));
-        }
-      }
-    }
-    __syncthreads();
-    // this chunk's outputs, and the next chunk's operands, between the same two barriers
-    if constexpr (CL > 1) {
-      for (int j = warp; j < n; j += kDsThreads / 32) {
-        float ss = 0.f;
-        for (int i = lane; i < kCols; i += 32) ss += cta * kCols + i < D ? so[j * kCols + i] * so[j * kCols + i] : 0.f;
-        ss = warp_sum(ss);
-        if (lane == 0) part_s[par][j] = ss;
-      }
-      cooperative_groups::this_cluster().sync();
-    }
-    for (int j = warp; j < n; j += kDsThreads / 32) {
-      float ss = 0.f;
-      if constexpr (CL > 1) {
-        auto cluster = cooperative_groups::this_cluster();
-#pragma unroll
-        for (int k = 0; k < CL; ++k) ss += *cluster.map_shared_rank(&part_s[par][j], k);
-      } else {
-        for (int i = lane; i < kCols; i += 32) ss += i < D ? so[j * kCols + i] * so[j * kCols + i] : 0.f;
-        ss = warp_sum(ss);
-      }
-      const float inv = rsqrtf(ss / static_cast<float>(D) + a.eps);
-      const long long t = tb + j;
-      for (int i = lane; i < kCols; i += 32) {
-        const int ch = cta * kCols + i;
-        if (ch < D) {
-          const float g = slab_sum(a.proj + t * a.ld + 3ll * HD + static_cast<long long>(h) * D + ch, a.n_partials, a.pstride);
-          out[t * HD + static_cast<long long>(h) * D + ch] =
-              from_f32<T>(so[j * kCols + i] * inv * a.out_norm[h * D + ch] * sigmoid_f32(g));
-        }
-      }
-    }
-    if (tb + C < t1) prepare(tb + C, min(C, t1 - tb - C));
-    __syncthreads();
+      for (int i = 0; i < kQ * 2; ++i) s[c][i] = 0ull;
   }
+  // st: the head's [D, D] state; vec: D is a multiple of CPT and rows are aligned for vector access
+  __device__ __forceinline__ void load(const float* st, int D, int rg, int col) {
 #pragma unroll
-  for (int q = 0; q < kQ; ++q)
+    for (int q = 0; q < kQ; ++q)
 #pragma unroll
-    for (int e = 0; e < 2; ++e) {
-      const int i = q * 32 + rg * 4 + e * 2;
+      for (int e = 0; e < 2; ++e) {
+        float x[2][CPT];
 #pragma unroll
-      for (int c = 0; c < CPT; ++c) {
-        float x, y;
-        unpack_f32x2(S[c][q * 2 + e], x, y);
-        if (col + c < D) {
-          if (i < D) st[static_cast<long long>(i) * D + col + c] = x;
-          if (i + 1 < D) st[static_cast<long long>(i + 1) * D + col + c] = y;
+        for (int k = 0; k < 2; ++k) {
+          const int i = q * 32 + rg * 4 + e * 2 + k;
+          const float* p = st + static_cast<long long>(i) * D + col;
+          if (i < D && col + CPT <= D && D % CPT == 0) {
+            if constexpr (CPT == 4) {
+              const float4 v = *reinterpret_cast<const float4*>(p);
+              x[k][0] = v.x; x[k][1] = v.y; x[k][2] = v.z; x[k][3] = v.w;
+            } else if constexpr (CPT == 2) {
+              const float2 v = *reinterpret_cast<const float2*>(p);
+              x[k][0] = v.x; x[k][1] = v.y;
+            } else {
+              x[k][0] = *p;
+            }
+          } else {
+#pragma unroll
+            for (int c = 0; c < CPT; ++c) x[k][c] = (i < D && col + c < D) ? p[c] : 0.f;
+          }
+        }
+#pragma unroll
+        for (int c = 0; c < CPT; ++c)
+          s[c][q * 2 + e] = pack_f32x2(__float_as_uint(x[0][c]), __float_as_uint(x[1][c]));
+      }
+  }
+  __device__ __forceinline__ void store(float* st, int D, int rg, int col) const {
+#pragma unroll
+    for (int q = 0; q < kQ; ++q)
+#pragma unroll
+      for (int e = 0; e < 2; ++e) {
+        float x[2][CPT];
+#pragma unroll
+        for (int c = 0; c < CPT; ++c) unpack_f32x2(s[c][q * 2 + e], x[0][c], x[1][c]);
+#pragma unroll
+        for (int k = 0; k < 2; ++k) {
+          const int i = q * 32 + rg * 4 + e * 2 + k;
+          float* p = st + static_cast<long long>(i) * D + col;
+          if (i < D && col + CPT <= D && D % CPT == 0) {
+            if constexpr (CPT == 4) *reinterpret_cast<float4*>(p) = make_float4(x[k][0], x[k][1], x[k][2], x[k][3]);
+            else if constexpr (CPT == 2) *reinterpret_cast<float2*>(p) = make_float2(x[k][0], x[k][1]);
+            else *p = x[k][0];
+          } else {
+#pragma unroll
+            for (int c = 0; c < CPT; ++c)
+              if (i < D && col + c < D) p[c] = x[k][c];
+          }
         }
       }
+  }
+  // One token: op = its operands u, r*w, w, a*u, k, v [DP each, `pitch` floats apart]; ra = r.(a*u), rk = r.k.
+  // o[c] is complete in every lane of a column's row groups.
+  __device__ __forceinline__ void token(const float* op, int pitch, float ra, float rk, int rg, int col,
+                                        float (&o)[CPT]) {
+    uint64_t d2[CPT], o2[CPT];
+#pragma unroll
+    for (int c = 0; c < CPT; ++c) d2[c] = o2[c] = 0ull;
+#pragma unroll
+    for (int q = 0; q < kQ; ++q) {
+      const ulonglong2 u = *reinterpret_cast<const ulonglong2*>(op + q * 32 + rg * 4);
+      const ulonglong2 rw = *reinterpret_cast<const ulonglong2*>(op + pitch + q * 32 + rg * 4);
+#pragma unroll
+      for (int c = 0; c < CPT; ++c) {
+        d2[c] = fma_f32x2(u.x, s[c][q * 2], d2[c]);
+        o2[c] = fma_f32x2(rw.x, s[c][q * 2], o2[c]);
+        d2[c] = fma_f32x2(u.y, s[c][q * 2 + 1], d2[c]);
+        o2[c] = fma_f32x2(rw.y, s[c][q * 2 + 1], o2[c]);
+      }
     }
-  if constexpr (CL > 1) cooperative_groups::this_cluster().sync();
+    float d[CPT];
+#pragma unroll
+    for (int c = 0; c < CPT; ++c) {
+      float x, y;
+      unpack_f32x2(d2[c], x, y);
+      d[c] = x + y;
+      unpack_f32x2(o2[c], x, y);
+      o[c] = x + y;
+    }
+#pragma unroll
+    for (int m = 4; m < 32; m <<= 1)
+#pragma unroll
+      for (int c = 0; c < CPT; ++c) {
+        d[c] += __shfl_xor_sync(0xffffffffu, d[c], m);
+        o[c] += __shfl_xor_sync(0xffffffffu, o[c], m);
+      }
+    uint64_t v2[CPT], nd2[CPT];
+#pragma unroll
+    for (int c = 0; c < CPT; ++c) {
+      const float v = op[5 * pitch + col + c];
+      o[c] = fmaf(rk, v, fmaf(-ra, d[c], o[c]));
+      v2[c] = pack_f32x2(__float_as_uint(v), __float_as_uint(v));
+      nd2[c] = pack_f32x2(__float_as_uint(-d[c]), __float_as_uint(-d[c]));
+    }
+#pragma unroll
+    for (int q = 0; q < kQ; ++q) {
+      const ulonglong2 w = *reinterpret_cast<const ulonglong2*>(op + 2 * pitch + q * 32 + rg * 4);
+      const ulonglong2 au = *reinterpret_cast<const ulonglong2*>(op + 3 * pitch + q * 32 + rg * 4);
+      const ulonglong2 k = *reinterpret_cast<const ulonglong2*>(op + 4 * pitch + q * 32 + rg * 4);
+#pragma unroll
+      for (int c = 0; c < CPT; ++c) {
+        s[c][q * 2] = fma_f32x2(w.x, s[c][q * 2], fma_f32x2(au.x, nd2[c], mul_f32x2(k.x, v2[c])));
+        s[c][q * 2 + 1] = fma_f32x2(w.y, s[c][q * 2 + 1], fma_f32x2(au.y, nd2[c], mul_f32x2(k.y, v2[c])));
+      }
+    }
+  }
+};
+
+// One token's operands from its raw projections (x: r, k, v, g, rate, decay, DP floats each, in shared
+// memory), by one warp: op = u, r*w, w, a*u, k, v, sigmoid(g), `pitch` apart; scalars[0..1] = r.(a*u), r.k.
+template <int DP>
+__device__ __forceinline__ void prepare_token(const DeltaArgs& a, int h, const float* x, float* op, int pitch,
+                                              float* scalars) {
+  constexpr int kQ = DP / 32;
+  const int lane = threadIdx.x & 31, D = a.dim;
+  float kk[kQ], ss = 0.f;
+#pragma unroll
+  for (int q = 0; q < kQ; ++q) {
+    const int i = q * 32 + lane;
+    kk[q] = i < D ? x[DP + i] : 0.f;
+    ss += kk[q] * kk[q];
+  }
+  const float inv = rsqrtf(warp_sum(ss) + 1e-6f);
+  float ra = 0.f, rk = 0.f;
+#pragma unroll
+  for (int q = 0; q < kQ; ++q) {
+    const int i = q * 32 + lane;
+    float r = 0.f, w = 0.f, rate = 0.f, v = 0.f, g = 0.f;
+    if (i < D) {
+      // 1 + expm1: rounded once near 1, where channels that remember for long live (an error of one
+      // unit there, repeated at every token, is a drift of the whole memory)
+      w = 1.0f + expm1f(-kDecayGain * sigmoid_f32(x[5 * DP + i] + a.decay_bias[h * D + i]));
+      rate = sigmoid_f32(x[4 * DP + i] + a.rate_bias[h * D + i]);
+      r = x[i];
+      v = x[2 * DP + i];
+      g = sigmoid_f32(x[3 * DP + i]);
+    }
+    const float u = kk[q] * inv, au = rate * u;
+    ra = fmaf(r, au, ra);
+    rk = fmaf(r, kk[q], rk);
+    op[i] = u;
+    op[pitch + i] = r * w;
+    op[2 * pitch + i] = w;
+    op[3 * pitch + i] = au;
+    op[4 * pitch + i] = kk[q];
+    op[5 * pitch + i] = v;
+    op[6 * pitch + i] = g;
+  }
+  ra = warp_sum(ra);
+  rk = warp_sum(rk);
+  if (lane == 0) {
+    scalars[0] = ra;
+    scalars[1] = rk;
+  }
+}
+
+// element `i` of raw projection `kind` (r, k, v, g, rate, decay) of token t, head h
+__device__ __forceinline__ const float* raw_ptr(const DeltaArgs& a, long long t, int h, int kind, int i) {
+  const int HD = a.heads * a.dim;
+  return kind < 5 ? a.proj + t * a.ld + static_cast<long long>(kind) * HD + h * a.dim + i : a.decay + t * HD + h * a.dim + i;
+}
+
+// ------------------------------------------------------------------------------------------- one token each
+constexpr int kTokThreads = 256;
+
+template <typename T, int DP, int CPT>
+__global__ void __launch_bounds__(kTokThreads)
+delta_token_kernel(const DeltaArgs a, T* __restrict__ out) {
+  constexpr int kCols = kTokThreads / 32 * 4 * CPT, CL = DP / kCols;
+  __shared__ __align__(16) float raw[6 * DP];
+  __shared__ __align__(16) float op[7 * DP];
+  __shared__ float so[kCols], sc[2];
+  __shared__ RowSum<kTokThreads, CL, 1> sh;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, rg = lane >> 2, D = a.dim, HD = a.heads * a.dim;
+  const int cta = CL > 1 ? static_cast<int>(blockIdx.x) : 0;
+  const int h = blockIdx.y, t = blockIdx.z;
+  pdl_launch_dependents();
+  // Positions, slots and the state were written by earlier steps, which are complete before any kernel of
+  // this step starts (a step's first launch follows the sampler's bookkeeping kernel or a copy, neither of
+  // which lets its successor start early), so the state is on its way while the projections are finished.
+  const bool idle = a.slot_map[t] < 0;
+  const bool fresh = a.positions[t] == 0;
+  const int lcol = warp * 4 * CPT + (lane & 3) * CPT, col = cta * kCols + lcol;
+  float* st = a.state + (static_cast<long long>(a.state_slots[t]) * a.heads + h) * D * D;
+  StateTile<DP, CPT> S;
+  if (idle || fresh) S.zero();
+  else S.load(st, D, rg, col);
+  pdl_wait();
+  if (idle) return;                                     // the same for the whole cluster
+  for (int e = threadIdx.x; e < 6 * D; e += kTokThreads) {
+    const int kind = e / D, i = e - kind * D;
+    raw[kind * DP + i] = kind < 5 ? slab_sum(raw_ptr(a, t, h, kind, i), a.n_partials, a.pstride)
+                                  : slab_sum(raw_ptr(a, t, h, kind, i), a.d_partials, a.dstride);
+  }
+  __syncthreads();
+  if (warp == 0) prepare_token<DP>(a, h, raw, op, DP, sc);
+  __syncthreads();
+  float o[CPT];
+  S.token(op, DP, sc[0], sc[1], rg, col, o);
+  S.store(st, D, rg, col);
+  float ss[1] = {0.f};
+#pragma unroll
+  for (int c = 0; c < CPT; ++c)
+    if (rg == 0) {
+      so[lcol + c] = o[c];
+      if (col + c < D) ss[0] += o[c] * o[c];
+    }
+  row_sum<kTokThreads, CL, 1>(sh, ss, 0);               // also orders `so`
+  const float inv = rsqrtf(ss[0] / static_cast<float>(D) + a.eps);
+  for (int i = threadIdx.x; i < kCols; i += kTokThreads) {
+    const int ch = cta * kCols + i;
+    if (ch < D)
+      out[static_cast<long long>(t) * HD + h * D + ch] = from_f32<T>(so[i] * inv * a.out_norm[h * D + ch] * op[6 * DP + ch]);
+  }
+  row_sum_exit<CL>();
 }
 
 template <typename T, int DP, int CPT>
-static int launch_scan(const DeltaArgs& a, void* out, int n_seqs, cudaStream_t st) {
-  constexpr int kCols = kDsThreads / 32 * 4 * CPT, CL = DP / kCols;
-  const size_t sm = static_cast<size_t>(a.chunk) * (6 * DP + kCols) * 4;
-  BCG_TRY(ensure_dynamic_smem(reinterpret_cast<const void*>(delta_scan_kernel<T, DP, CPT>),
-                              kDsChunk * (6 * DP + kCols) * 4));
-  BCG_CUDA_CHECK(launch_cluster(delta_scan_kernel<T, DP, CPT>, dim3(CL, a.heads, n_seqs), dim3(kDsThreads), CL, sm, st, a,
+static int launch_token(const DeltaArgs& a, void* out, int n, cudaStream_t st) {
+  constexpr int CL = DP / (kTokThreads / 32 * 4 * CPT);
+  BCG_CUDA_CHECK(launch_cluster(delta_token_kernel<T, DP, CPT>, dim3(CL, a.heads, n), dim3(kTokThreads), CL, 0, st, a,
                                 static_cast<T*>(out)));
+  return BCG_OK;
+}
+template <typename T>
+static int dispatch_token(const DeltaArgs& a, void* out, int n, cudaStream_t st) {
+  if (a.dim <= 32) return launch_token<T, 32, 1>(a, out, n, st);
+  if (a.dim <= 64) return launch_token<T, 64, 2>(a, out, n, st);
+  if (a.dim <= 128) return launch_token<T, 128, 4>(a, out, n, st);
+  return launch_token<T, 256, 2>(a, out, n, st);
+}
+
+// ------------------------------------------------------------------------------------------- portions
+// SW scan warps, PW preparation warps; a chunk is PW tokens, one per preparation warp.
+template <int DP, int CPT, int SW, int PW>
+struct DsCfg {
+  static constexpr int kCols = SW * 4 * CPT, CL = DP / kCols, kThreads = (SW + PW) * 32, kChunk = PW;
+  static constexpr int kOps = 7 * DP;                    // operands of one token
+  static constexpr int kFloats = 2 * kChunk * kOps + 2 * kChunk * kCols + kChunk * 6 * DP;
+};
+
+// wait for a cluster-wide phase; a phase that never comes traps instead of hanging
+__device__ __forceinline__ void mbar_wait_cluster(uint64_t* bar, uint32_t parity) {
+  uint32_t ok = 0, spins = 0;
+  while (!ok) {
+    asm volatile(
+        "{\n"
+        ".reg .pred p;\n"
+        "mbarrier.try_wait.parity.acquire.cluster.shared::cta.b64 p, [%1], %2;\n"
+        "selp.b32 %0, 1, 0, p;\n"
+        "}\n"
+        : "=r"(ok)
+        : "r"(smem_u32(bar)), "r"(parity)
+        : "memory");
+    if (++spins > (1u << 26)) __trap();
+  }
+}
+__device__ __forceinline__ uint32_t peer_smem(const void* p, int rank) {
+  uint32_t r;
+  asm("mapa.shared::cluster.u32 %0, %1, %2;" : "=r"(r) : "r"(smem_u32(p)), "r"(rank));
+  return r;
+}
+
+template <typename T, int DP, int CPT, int SW, int PW>
+__global__ void __launch_bounds__((SW + PW) * 32, 1)
+delta_scan_kernel(const DeltaArgs a, T* __restrict__ out) {
+  using C = DsCfg<DP, CPT, SW, PW>;
+  constexpr int CL = C::CL;
+  extern __shared__ float4 ds_raw[];
+  float* ops = reinterpret_cast<float*>(ds_raw);          // [2][chunk][7][DP]
+  float* so = ops + 2 * C::kChunk * C::kOps;              // [2][chunk][kCols]
+  float* raw = so + 2 * C::kChunk * C::kCols;             // [chunk][6][DP]
+  __shared__ float sc[2][C::kChunk][2];
+  __shared__ float part[2][C::kChunk][CL];                // sums of squares of the cluster's column blocks
+  __shared__ uint64_t part_bar[2];
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, D = a.dim, HD = a.heads * a.dim;
+  const int cta = CL > 1 ? static_cast<int>(blockIdx.x) : 0;
+  const int h = blockIdx.y, s = blockIdx.z;
+  pdl_launch_dependents();
+  if (CL > 1 && threadIdx.x == 0) {
+    mbar_init(&part_bar[0], CL * C::kChunk);
+    mbar_init(&part_bar[1], CL * C::kChunk);
+    fence_barrier_init();
+  }
+  pdl_wait();
+  if constexpr (CL > 1) cooperative_groups::this_cluster().sync();   // barriers ready before any peer arrives
+  const int t0 = a.seq_start ? a.seq_start[s] : s;
+  const int t1 = a.seq_start ? a.seq_start[s + 1] : s + 1;
+  if (t1 <= t0 || a.slot_map[t0] < 0) return;             // nothing to do (the same for the whole cluster)
+  const bool fresh = a.positions[t0] == 0;
+  float* st = a.state + (static_cast<long long>(a.state_slots[s]) * a.heads + h) * D * D;
+  const int n_chunks = (t1 - t0 + C::kChunk - 1) / C::kChunk;
+  const bool copies = a.n_partials == 1 && a.d_partials == 1;
+  const bool wide = copies && (D & 3) == 0 && (a.ld & 3) == 0;
+
+  // the raw projections of one token into raw[j], by one warp: asynchronous copies, or sums of slabs
+  auto fetch = [&](int j, long long t) {
+    float* dst = raw + j * 6 * DP;
+#pragma unroll
+    for (int kind = 0; kind < 6; ++kind) {
+      const float* src = raw_ptr(a, t, h, kind, 0);
+      if (wide) {
+        for (int i = lane * 4; i < D; i += 128)
+          asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(smem_u32(dst + kind * DP + i)), "l"(src + i) : "memory");
+      } else if (copies) {
+        for (int i = lane; i < D; i += 32)
+          asm volatile("cp.async.ca.shared.global [%0], [%1], 4;" ::"r"(smem_u32(dst + kind * DP + i)), "l"(src + i) : "memory");
+      } else {
+        for (int i = lane; i < D; i += 32)
+          dst[kind * DP + i] = kind < 5 ? slab_sum(src + i, a.n_partials, a.pstride) : slab_sum(src + i, a.d_partials, a.dstride);
+      }
+    }
+  };
+  auto prepare = [&](int c, int j) {      // token j of chunk c, by its warp; then the copy of its next token
+    const int t = t0 + c * C::kChunk + j;
+    if (t < t1) {
+      asm volatile("cp.async.wait_all;" ::: "memory");
+      __syncwarp();
+      prepare_token<DP>(a, h, raw + j * 6 * DP, ops + ((c & 1) * C::kChunk + j) * C::kOps, DP, sc[c & 1][j]);
+      __syncwarp();
+      if (t + C::kChunk < t1) fetch(j, t + C::kChunk);
+    }
+  };
+  auto finish = [&](int c, int j) {       // output of token j of chunk c, by its warp
+    const int t = t0 + c * C::kChunk + j, b = c & 1;
+    const float* o = so + (b * C::kChunk + j) * C::kCols;
+    float ss = 0.f;
+    if (t < t1)
+      for (int i = lane; i < C::kCols; i += 32) ss += cta * C::kCols + i < D ? o[i] * o[i] : 0.f;
+    ss = warp_sum(ss);
+    if constexpr (CL > 1) {
+      // every CTA of the cluster gets every block's sum; tokens past the end arrive too, so that a phase is
+      // always CL * chunk arrivals
+      if (lane < CL) {
+        asm volatile("st.relaxed.cluster.shared::cluster.f32 [%0], %1;" ::"r"(peer_smem(&part[b][j][cta], lane)), "f"(ss) : "memory");
+        asm volatile("mbarrier.arrive.release.cluster.shared::cluster.b64 _, [%0];" ::"r"(peer_smem(&part_bar[b], lane)) : "memory");
+      }
+      __syncwarp();
+      mbar_wait_cluster(&part_bar[b], (c >> 1) & 1);
+      ss = 0.f;
+#pragma unroll
+      for (int k = 0; k < CL; ++k) ss += part[b][j][k];
+    }
+    if (t < t1) {
+      const float inv = rsqrtf(ss / static_cast<float>(D) + a.eps);
+      const float* g = ops + (b * C::kChunk + j) * C::kOps + 6 * DP;
+      for (int i = lane; i < C::kCols; i += 32) {
+        const int ch = cta * C::kCols + i;
+        if (ch < D)
+          out[static_cast<long long>(t) * HD + h * D + ch] = from_f32<T>(o[i] * inv * a.out_norm[h * D + ch] * g[ch]);
+      }
+    }
+    __syncwarp();
+  };
+
+  if (warp < SW) {
+    // ------------------------------ scan warps ------------------------------
+    const int rg = lane >> 2;
+    const int lcol = warp * 4 * CPT + (lane & 3) * CPT, col = cta * C::kCols + lcol;
+    StateTile<DP, CPT> S;
+    if (fresh) S.zero();
+    else S.load(st, D, rg, col);
+    __syncthreads();
+    for (int c = 0; c < n_chunks; ++c) {
+      const int n = min(C::kChunk, t1 - t0 - c * C::kChunk), b = c & 1;
+      const float* op = ops + b * C::kChunk * C::kOps;
+      float* o_row = so + b * C::kChunk * C::kCols;
+      for (int j = 0; j < n; ++j, op += C::kOps, o_row += C::kCols) {
+        float o[CPT];
+        S.token(op, DP, sc[b][j][0], sc[b][j][1], rg, col, o);
+        if (rg == 0) {
+#pragma unroll
+          for (int k = 0; k < CPT; ++k) o_row[lcol + k] = o[k];
+        }
+      }
+      __syncthreads();
+    }
+    S.store(st, D, rg, col);
+  } else {
+    // ------------------------------ preparation warps ------------------------
+    const int j = warp - SW;
+    if (t0 + j < t1) fetch(j, t0 + j);
+    prepare(0, j);
+    __syncthreads();
+    for (int c = 0; c < n_chunks; ++c) {
+      if (c > 0) finish(c - 1, j);        // before its operands (the gate) are overwritten
+      if (c + 1 < n_chunks) prepare(c + 1, j);
+      __syncthreads();
+    }
+    finish(n_chunks - 1, j);
+  }
+  if constexpr (CL > 1) cooperative_groups::this_cluster().sync();   // no peer writes into a CTA that has left
+}
+
+template <typename T, int DP, int CPT, int SW, int PW>
+static int launch_scan(const DeltaArgs& a, void* out, int n_seqs, cudaStream_t st) {
+  using C = DsCfg<DP, CPT, SW, PW>;
+  BCG_TRY(ensure_dynamic_smem(reinterpret_cast<const void*>(delta_scan_kernel<T, DP, CPT, SW, PW>), C::kFloats * 4));
+  BCG_CUDA_CHECK(launch_cluster(delta_scan_kernel<T, DP, CPT, SW, PW>, dim3(C::CL, a.heads, n_seqs), dim3(C::kThreads),
+                                C::CL, C::kFloats * 4, st, a, static_cast<T*>(out)));
   return BCG_OK;
 }
 
 template <typename T>
 static int dispatch_scan(const DeltaArgs& a, void* out, int n_seqs, cudaStream_t st) {
-  const bool many = static_cast<long long>(n_seqs) * a.heads >= 148;   // enough heads to fill the GPU one CTA each
-  if (a.dim <= 32) return launch_scan<T, 32, 1>(a, out, n_seqs, st);
-  if (a.dim <= 64) return many ? launch_scan<T, 64, 2>(a, out, n_seqs, st) : launch_scan<T, 64, 1>(a, out, n_seqs, st);
+  const bool many = static_cast<long long>(n_seqs) * a.heads >= 96;   // heads enough for most SMs, one CTA each
+  if (a.dim <= 32) return launch_scan<T, 32, 1, 8, 8>(a, out, n_seqs, st);
+  if (a.dim <= 64) return launch_scan<T, 64, 1, 16, 8>(a, out, n_seqs, st);
   if (a.dim <= 128)
-    return many ? launch_scan<T, 128, 4>(a, out, n_seqs, st) : launch_scan<T, 128, 1>(a, out, n_seqs, st);
-  return launch_scan<T, 256, 2>(a, out, n_seqs, st);
+    return many ? launch_scan<T, 128, 2, 16, 8>(a, out, n_seqs, st) : launch_scan<T, 128, 1, 8, 16>(a, out, n_seqs, st);
+  return launch_scan<T, 256, 1, 16, 8>(a, out, n_seqs, st);
 }
 
 int delta_low(const bcg_layer* l, const float* proj, int n_partials, long long pstride, void* low, int act_dtype,
@@ -293,8 +505,10 @@ int delta_scan(const bcg_layer* l, const float* proj, int n_partials, long long 
     return BCG_ERR_ARG;
   }
   DeltaArgs a = {proj, n_partials, pstride, ld, decay, d_partials, dstride, l->decay_bias, l->rate_bias, l->out_norm,
-                 positions, slot_map, seq_start, state_slots, static_cast<float*>(l->cache), l->heads, l->dim,
-                 one_token ? 1 : kDsChunk, eps};
+                 positions, slot_map, seq_start, state_slots, static_cast<float*>(l->cache), l->heads, l->dim, eps};
+  if (one_token)
+    return act_dtype == BCG_DT_F32 ? dispatch_token<float>(a, out, n_seqs, st)
+                                   : dispatch_token<__nv_bfloat16>(a, out, n_seqs, st);
   return act_dtype == BCG_DT_F32 ? dispatch_scan<float>(a, out, n_seqs, st)
                                  : dispatch_scan<__nv_bfloat16>(a, out, n_seqs, st);
 }

@@ -282,7 +282,8 @@ class StackExecutor:
 
     def _batch(self, T, n_seqs) -> L.StepBatch:
         b = L.StepBatch()
-        b.T, b.n_seqs, b.max_blocks, b.flags = T, n_seqs, self.max_blocks, self.flags & L.GEMM_PDL
+        # programmatic dependent launch pays for short kernels; long ones only occupy SMs while they wait
+        b.T, b.n_seqs, b.max_blocks, b.flags = T, n_seqs, self.max_blocks, self.flags & L.GEMM_PDL if T <= 128 else 0
         return b
 
     def _run(self, b: L.StepBatch) -> None:
