@@ -120,22 +120,23 @@ struct StateTile {
         }
       }
   }
-  // One token: op = its operands u, r*w, w, a*u, k, v [DP each, `pitch` floats apart]; ra = r.(a*u), rk = r.k.
-  // o[c] is complete in every lane of a column's row groups.
-  __device__ __forceinline__ void token(const float* op, int pitch, float ra, float rk, int rg, int col,
+  // One token: op = its operands k, r*w, w, a*u, v [DP each, `pitch` floats apart]; sc = 1/|k|, r.(a*u),
+  // r.k.  (u^T S is formed as (k^T S)/|k|: four vectors per token instead of five - a lane's share of them, read
+  // from shared memory, is what the loop is bound by when CPT is small.)  o[c] is complete in every lane of a column's row groups.
+  __device__ __forceinline__ void token(const float* op, int pitch, const float* sc, int rg, int col,
                                         float (&o)[CPT]) {
     uint64_t d2[CPT], o2[CPT];
 #pragma unroll
     for (int c = 0; c < CPT; ++c) d2[c] = o2[c] = 0ull;
 #pragma unroll
     for (int q = 0; q < kQ; ++q) {
-      const ulonglong2 u = *reinterpret_cast<const ulonglong2*>(op + q * 32 + rg * 4);
+      const ulonglong2 k = *reinterpret_cast<const ulonglong2*>(op + q * 32 + rg * 4);
       const ulonglong2 rw = *reinterpret_cast<const ulonglong2*>(op + pitch + q * 32 + rg * 4);
 #pragma unroll
       for (int c = 0; c < CPT; ++c) {
-        d2[c] = fma_f32x2(u.x, s[c][q * 2], d2[c]);
+        d2[c] = fma_f32x2(k.x, s[c][q * 2], d2[c]);
         o2[c] = fma_f32x2(rw.x, s[c][q * 2], o2[c]);
-        d2[c] = fma_f32x2(u.y, s[c][q * 2 + 1], d2[c]);
+        d2[c] = fma_f32x2(k.y, s[c][q * 2 + 1], d2[c]);
         o2[c] = fma_f32x2(rw.y, s[c][q * 2 + 1], o2[c]);
       }
     }
@@ -158,8 +159,9 @@ struct StateTile {
     uint64_t v2[CPT], nd2[CPT];
 #pragma unroll
     for (int c = 0; c < CPT; ++c) {
-      const float v = op[5 * pitch + col + c];
-      o[c] = fmaf(rk, v, fmaf(-ra, d[c], o[c]));
+      const float v = op[4 * pitch + col + c];
+      d[c] *= sc[0];
+      o[c] = fmaf(sc[2], v, fmaf(-sc[1], d[c], o[c]));
       v2[c] = pack_f32x2(__float_as_uint(v), __float_as_uint(v));
       nd2[c] = pack_f32x2(__float_as_uint(-d[c]), __float_as_uint(-d[c]));
     }
@@ -167,7 +169,7 @@ struct StateTile {
     for (int q = 0; q < kQ; ++q) {
       const ulonglong2 w = *reinterpret_cast<const ulonglong2*>(op + 2 * pitch + q * 32 + rg * 4);
       const ulonglong2 au = *reinterpret_cast<const ulonglong2*>(op + 3 * pitch + q * 32 + rg * 4);
-      const ulonglong2 k = *reinterpret_cast<const ulonglong2*>(op + 4 * pitch + q * 32 + rg * 4);
+      const ulonglong2 k = *reinterpret_cast<const ulonglong2*>(op + q * 32 + rg * 4);
 #pragma unroll
       for (int c = 0; c < CPT; ++c) {
         s[c][q * 2] = fma_f32x2(w.x, s[c][q * 2], fma_f32x2(au.x, nd2[c], mul_f32x2(k.x, v2[c])));
@@ -178,7 +180,7 @@ struct StateTile {
 };
 
 // One token's operands from its raw projections (x: r, k, v, g, rate, decay, DP floats each, in shared
-// memory), by one warp: op = u, r*w, w, a*u, k, v, sigmoid(g), `pitch` apart; scalars[0..1] = r.(a*u), r.k.
+// memory), by one warp: op = k, r*w, w, a*u, v, sigmoid(g), `pitch` apart; scalars = 1/|k|, r.(a*u), r.k.
 template <int DP>
 __device__ __forceinline__ void prepare_token(const DeltaArgs& a, int h, const float* x, float* op, int pitch,
                                               float* scalars) {
@@ -206,22 +208,22 @@ __device__ __forceinline__ void prepare_token(const DeltaArgs& a, int h, const f
       v = x[2 * DP + i];
       g = sigmoid_f32(x[3 * DP + i]);
     }
-    const float u = kk[q] * inv, au = rate * u;
+    const float au = rate * (kk[q] * inv);
     ra = fmaf(r, au, ra);
     rk = fmaf(r, kk[q], rk);
-    op[i] = u;
+    op[i] = kk[q];
     op[pitch + i] = r * w;
     op[2 * pitch + i] = w;
     op[3 * pitch + i] = au;
-    op[4 * pitch + i] = kk[q];
-    op[5 * pitch + i] = v;
-    op[6 * pitch + i] = g;
+    op[4 * pitch + i] = v;
+    op[5 * pitch + i] = g;
   }
   ra = warp_sum(ra);
   rk = warp_sum(rk);
   if (lane == 0) {
-    scalars[0] = ra;
-    scalars[1] = rk;
+    scalars[0] = inv;
+    scalars[1] = ra;
+    scalars[2] = rk;
   }
 }
 
@@ -239,8 +241,8 @@ __global__ void __launch_bounds__(kTokThreads)
 delta_token_kernel(const DeltaArgs a, T* __restrict__ out) {
   constexpr int kCols = kTokThreads / 32 * 4 * CPT, CL = DP / kCols;
   __shared__ __align__(16) float raw[6 * DP];
-  __shared__ __align__(16) float op[7 * DP];
-  __shared__ float so[kCols], sc[2];
+  __shared__ __align__(16) float op[6 * DP];
+  __shared__ float so[kCols], sc[3];
   __shared__ RowSum<kTokThreads, CL, 1> sh;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, rg = lane >> 2, D = a.dim, HD = a.heads * a.dim;
   const int cta = CL > 1 ? static_cast<int>(blockIdx.x) : 0;
@@ -267,7 +269,7 @@ delta_token_kernel(const DeltaArgs a, T* __restrict__ out) {
   if (warp == 0) prepare_token<DP>(a, h, raw, op, DP, sc);
   __syncthreads();
   float o[CPT];
-  S.token(op, DP, sc[0], sc[1], rg, col, o);
+  S.token(op, DP, sc, rg, col, o);
   S.store(st, D, rg, col);
   float ss[1] = {0.f};
 #pragma unroll
@@ -281,7 +283,7 @@ delta_token_kernel(const DeltaArgs a, T* __restrict__ out) {
   for (int i = threadIdx.x; i < kCols; i += kTokThreads) {
     const int ch = cta * kCols + i;
     if (ch < D)
-      out[static_cast<long long>(t) * HD + h * D + ch] = from_f32<T>(so[i] * inv * a.out_norm[h * D + ch] * op[6 * DP + ch]);
+      out[static_cast<long long>(t) * HD + h * D + ch] = from_f32<T>(so[i] * inv * a.out_norm[h * D + ch] * op[5 * DP + ch]);
   }
   row_sum_exit<CL>();
 }
@@ -306,7 +308,7 @@ static int dispatch_token(const DeltaArgs& a, void* out, int n, cudaStream_t st)
 template <int DP, int CPT, int SW, int PW>
 struct DsCfg {
   static constexpr int kCols = SW * 4 * CPT, CL = DP / kCols, kThreads = (SW + PW) * 32, kChunk = PW;
-  static constexpr int kOps = 7 * DP;                    // operands of one token
+  static constexpr int kOps = 6 * DP;                    // operands of one token
   static constexpr int kFloats = 2 * kChunk * kOps + 2 * kChunk * kCols + kChunk * 6 * DP;
 };
 
@@ -338,10 +340,10 @@ delta_scan_kernel(const DeltaArgs a, T* __restrict__ out) {
   using C = DsCfg<DP, CPT, SW, PW>;
   constexpr int CL = C::CL;
   extern __shared__ float4 ds_raw[];
-  float* ops = reinterpret_cast<float*>(ds_raw);          // [2][chunk][7][DP]
+  float* ops = reinterpret_cast<float*>(ds_raw);          // [2][chunk][6][DP]
   float* so = ops + 2 * C::kChunk * C::kOps;              // [2][chunk][kCols]
   float* raw = so + 2 * C::kChunk * C::kCols;             // [chunk][6][DP]
-  __shared__ float sc[2][C::kChunk][2];
+  __shared__ float sc[2][C::kChunk][4];
   __shared__ float part[2][C::kChunk][CL];                // sums of squares of the cluster's column blocks
   __shared__ uint64_t part_bar[2];
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, D = a.dim, HD = a.heads * a.dim;
@@ -414,7 +416,7 @@ delta_scan_kernel(const DeltaArgs a, T* __restrict__ out) {
     }
     if (t < t1) {
       const float inv = rsqrtf(ss / static_cast<float>(D) + a.eps);
-      const float* g = ops + (b * C::kChunk + j) * C::kOps + 6 * DP;
+      const float* g = ops + (b * C::kChunk + j) * C::kOps + 5 * DP;
       for (int i = lane; i < C::kCols; i += 32) {
         const int ch = cta * C::kCols + i;
         if (ch < D)
@@ -438,7 +440,7 @@ delta_scan_kernel(const DeltaArgs a, T* __restrict__ out) {
       float* o_row = so + b * C::kChunk * C::kCols;
       for (int j = 0; j < n; ++j, op += C::kOps, o_row += C::kCols) {
         float o[CPT];
-        S.token(op, DP, sc[b][j][0], sc[b][j][1], rg, col, o);
+        S.token(op, DP, sc[b][j], rg, col, o);
         if (rg == 0) {
 #pragma unroll
           for (int k = 0; k < CPT; ++k) o_row[lcol + k] = o[k];
@@ -475,11 +477,11 @@ static int launch_scan(const DeltaArgs& a, void* out, int n_seqs, cudaStream_t s
 template <typename T>
 static int dispatch_scan(const DeltaArgs& a, void* out, int n_seqs, cudaStream_t st) {
   const bool many = static_cast<long long>(n_seqs) * a.heads >= 96;   // heads enough for most SMs, one CTA each
-  if (a.dim <= 32) return launch_scan<T, 32, 1, 8, 8>(a, out, n_seqs, st);
-  if (a.dim <= 64) return launch_scan<T, 64, 1, 16, 8>(a, out, n_seqs, st);
+  if (a.dim <= 32) return launch_scan<T, 32, 2, 4, 8>(a, out, n_seqs, st);
+  if (a.dim <= 64) return launch_scan<T, 64, 2, 8, 8>(a, out, n_seqs, st);
   if (a.dim <= 128)
-    return many ? launch_scan<T, 128, 2, 16, 8>(a, out, n_seqs, st) : launch_scan<T, 128, 1, 8, 16>(a, out, n_seqs, st);
-  return launch_scan<T, 256, 1, 16, 8>(a, out, n_seqs, st);
+    return many ? launch_scan<T, 128, 4, 8, 8>(a, out, n_seqs, st) : launch_scan<T, 128, 2, 4, 16>(a, out, n_seqs, st);
+  return launch_scan<T, 256, 2, 8, 8>(a, out, n_seqs, st);
 }
 
 int delta_low(const bcg_layer* l, const float* proj, int n_partials, long long pstride, void* low, int act_dtype,
