@@ -260,10 +260,36 @@ delta_token_kernel(const DeltaArgs a, T* __restrict__ out) {
   else S.load(st, D, rg, col);
   pdl_wait();
   if (idle) return;                                     // the same for the whole cluster
-  for (int e = threadIdx.x; e < 6 * D; e += kTokThreads) {
-    const int kind = e / D, i = e - kind * D;
-    raw[kind * DP + i] = kind < 5 ? slab_sum(raw_ptr(a, t, h, kind, i), a.n_partials, a.pstride)
-                                  : slab_sum(raw_ptr(a, t, h, kind, i), a.d_partials, a.dstride);
+  {   // raw projections: a thread's elements and up to four slabs of each in flight together
+    constexpr int kE = (6 * DP + kTokThreads - 1) / kTokThreads;
+    const float* src[kE];
+    long long stride[kE];
+    float acc[kE];
+    const int n = max(a.n_partials, a.d_partials);
+#pragma unroll
+    for (int k = 0; k < kE; ++k) {
+      const int e = threadIdx.x + k * kTokThreads, kind = min(e / DP, 5), i = min(e % DP, D - 1);
+      src[k] = raw_ptr(a, t, h, kind, i);
+      stride[k] = kind < 5 ? a.pstride : a.dstride;
+      acc[k] = 0.f;
+    }
+    for (int s0 = 0; s0 < n; s0 += 4) {
+      float v[kE][4];
+#pragma unroll
+      for (int k = 0; k < kE; ++k)
+#pragma unroll
+        for (int q = 0; q < 4; ++q) {
+          const int np = threadIdx.x + k * kTokThreads < 5 * DP ? a.n_partials : a.d_partials;
+          v[k][q] = s0 + q < np ? src[k][(s0 + q) * stride[k]] : 0.f;
+        }
+#pragma unroll
+      for (int k = 0; k < kE; ++k)
+#pragma unroll
+        for (int q = 0; q < 4; ++q) acc[k] += v[k][q];
+    }
+#pragma unroll
+    for (int k = 0; k < kE; ++k)
+      if (threadIdx.x + k * kTokThreads < 6 * DP) raw[threadIdx.x + k * kTokThreads] = acc[k];
   }
   __syncthreads();
   if (warp == 0) prepare_token<DP>(a, h, raw, op, DP, sc);

@@ -7,8 +7,8 @@
 //   latent_plain      one CTA per (token, head), latent space, any sizes, fp32 or bf16: the fp32 engine's
 //                     kernel, and the bf16 one's for sizes the kernels below do not take
 //   latent_absorb     q~ for single tokens (decode), W_uk tile staged ahead of the dependency wait
-//   latent_decode     split-KV: one CTA per (key chunk, token), mma.sync over 32-head groups
-//   latent_up         chunks combined, then W_uv
+//   latent_decode     split-KV: one CTA per (span of keys, token), mma.sync over 32-head groups
+//   latent_combine    spans -> latent-space output;  latent_up: W_uv
 //   latent_gather     cache rows -> contiguous rows for the expanded (prefill) form, latent_prefill.cu
 #include "stack_common.cuh"
 #include "kernels.h"
@@ -208,73 +208,16 @@ int latent_plain(const bcg_layer* l, const void* q, void* out, const bcg_step_ba
 }
 
 // ------------------------------------------------------------------------------------------- absorb
-// q_latent[i, h] = (W_uk^T q_unrotated, q_rotated) for single token i = rows[i].
-constexpr int kAbCols = 128;    // latent columns per CTA
-constexpr int kAbRows = 8;      // tokens per pass
-
-__global__ void __launch_bounds__(128)
-latent_absorb_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __restrict__ w_uk,
-                     const int* __restrict__ rows, int n, __nv_bfloat16* __restrict__ q_latent, int heads, int dim,
-                     int rot_dim, int kv_rank, int q_row) {
-  extern __shared__ __align__(16) uint8_t ab_raw[];
-  __nv_bfloat16* wt = reinterpret_cast<__nv_bfloat16*>(ab_raw);                       // [dim][128]
-  float* qs = reinterpret_cast<float*>(ab_raw + static_cast<size_t>(dim) * kAbCols * 2);   // [8][dim]
-  pdl_launch_dependents();
-  const int h = blockIdx.x, c0 = blockIdx.y * kAbCols;
-  const int crow = kv_rank + rot_dim;
-  for (int i = threadIdx.x; i < dim * (kAbCols / 8); i += 128) {
-    const int d = i / (kAbCols / 8), c = c0 + (i % (kAbCols / 8)) * 8;
-    uint4 v = make_uint4(0, 0, 0, 0);
-    if (c < kv_rank) v = *reinterpret_cast<const uint4*>(w_uk + (static_cast<long long>(h) * dim + d) * kv_rank + c);
-    reinterpret_cast<uint4*>(wt)[i] = v;
-  }
-  pdl_wait();
-  for (int r0 = 0; r0 < n; r0 += kAbRows) {
-    const int nr = min(kAbRows, n - r0);
-    __syncthreads();
-    for (int i = threadIdx.x; i < nr * dim; i += 128) {
-      const int r = i / dim, d = i - r * dim;
-      const long long t = rows ? rows[r0 + r] : r0 + r;
-      qs[i] = __bfloat162float(q[(t * heads + h) * q_row + d]);
-    }
-    __syncthreads();
-    // thread = 2 columns x half of the pass's tokens
-    const int c = (threadIdx.x & 63) * 2, rh = (threadIdx.x >> 6) * (kAbRows / 2);
-    float acc[kAbRows / 2][2] = {};
-    for (int d = 0; d < dim; ++d) {
-      const uint32_t w = *reinterpret_cast<const uint32_t*>(wt + d * kAbCols + c);
-      const float w0 = bf16lo(w), w1 = bf16hi(w);
-#pragma unroll
-      for (int r = 0; r < kAbRows / 2; ++r) {
-        const float x = qs[min(rh + r, nr - 1) * dim + d];
-        acc[r][0] = fmaf(x, w0, acc[r][0]);
-        acc[r][1] = fmaf(x, w1, acc[r][1]);
-      }
-    }
-#pragma unroll
-    for (int r = 0; r < kAbRows / 2; ++r)
-      if (rh + r < nr && c0 + c < kv_rank)
-        *reinterpret_cast<uint32_t*>(q_latent + (static_cast<long long>(r0 + rh + r) * heads + h) * crow + c0 + c) =
-            pack_bf16(acc[r][0], acc[r][1]);
-    if (blockIdx.y == 0) {
-      for (int i = threadIdx.x; i < nr * rot_dim; i += 128) {
-        const int r = i / rot_dim, d = i - r * rot_dim;
-        const long long t = rows ? rows[r0 + r] : r0 + r;
-        q_latent[(static_cast<long long>(r0 + r) * heads + h) * crow + kv_rank + d] = q[(t * heads + h) * q_row + dim + d];
-      }
-    }
-  }
-}
-
-// ------------------------------------------------------------------------------------------- decode
-// grid (chunks, tokens, head groups of 32).  Chunk c of a token covers keys [c * 64, c * 64 + 64) counted
-// from the chunk-aligned start of its window.
-constexpr int kLdKeys = 64, kLdHeads = 32, kLdThreads = 128;
+// q_latent[i, h] = (W_uk^T q_unrotated, q_rotated) for single token i = rows[i].  grid (heads, 128-column
+// tiles of the latent); the weight tile is staged ahead of the dependency wait; mma.sync over 16 tokens a pass.
+constexpr int kAbCols = 128, kAbThreads = 128;
 
 __device__ __forceinline__ void cp_async16(void* dst, const void* src) {
   asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(smem_u32(dst)), "l"(src) : "memory");
 }
-__device__ __forceinline__ void cp_async_wait_all() { asm volatile("cp.async.wait_all;" ::: "memory"); }
+__device__ __forceinline__ void cp_async_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
+template <int N>
+__device__ __forceinline__ void cp_async_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory"); }
 __device__ __forceinline__ void ldsm_x4(uint32_t (&r)[4], const void* p) {
   asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0, %1, %2, %3}, [%4];"
                : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3])
@@ -292,241 +235,388 @@ __device__ __forceinline__ void mma_bf16_16816(float (&d)[4], const uint32_t (&a
       : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3])
       : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
 }
-
-__host__ __device__ constexpr int latent_decode_smem(int crow) {
-  return (kLdKeys + kLdHeads) * (crow + 8) * 2 + kLdHeads * (kLdKeys + 4) * 4 + kLdHeads * (kLdKeys + 8) * 2;
+__host__ __device__ constexpr int up16(int n) { return (n + 15) / 16 * 16; }
+__host__ __device__ constexpr int absorb_smem(int dim) {
+  return (up16(dim) * (kAbCols + 8) + 16 * (up16(dim) + 8)) * 2;
 }
 
-__global__ void __launch_bounds__(kLdThreads)
+__global__ void __launch_bounds__(kAbThreads)
+latent_absorb_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __restrict__ w_uk,
+                     const int* __restrict__ rows, int n, __nv_bfloat16* __restrict__ q_latent, int heads, int dim,
+                     int rot_dim, int kv_rank, int q_row) {
+  extern __shared__ __align__(16) uint8_t ab_raw[];
+  const int kd = up16(dim), srow = kd + 8;
+  constexpr int wrow = kAbCols + 8;
+  __nv_bfloat16* wt = reinterpret_cast<__nv_bfloat16*>(ab_raw);   // [kd][wrow]
+  __nv_bfloat16* qs = wt + kd * wrow;                             // [16][srow]
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int h = blockIdx.x, c0 = blockIdx.y * kAbCols, crow = kv_rank + rot_dim;
+  pdl_launch_dependents();
+  for (int i = threadIdx.x; i < kd * (kAbCols / 8); i += kAbThreads) {
+    const int d = i / (kAbCols / 8), c = (i % (kAbCols / 8)) * 8;
+    if (d < dim && c0 + c < kv_rank)
+      cp_async16(wt + d * wrow + c, w_uk + (static_cast<long long>(h) * dim + d) * kv_rank + c0 + c);
+    else
+      *reinterpret_cast<uint4*>(wt + d * wrow + c) = make_uint4(0, 0, 0, 0);
+  }
+  cp_async_commit();
+  pdl_wait();
+  for (int r0 = 0; r0 < n; r0 += 16) {
+    __syncthreads();                       // the pass before has read its queries
+    for (int r = warp; r < 16; r += kAbThreads / 32) {
+      const long long t = r0 + r < n ? (rows ? rows[r0 + r] : r0 + r) : -1;
+      const __nv_bfloat16* src = q + (t * heads + h) * q_row;
+      for (int d = lane; d < kd; d += 32) qs[r * srow + d] = (t >= 0 && d < dim) ? src[d] : __float2bfloat16(0.f);
+      if (blockIdx.y == 0 && t >= 0)
+        for (int d = lane; d < rot_dim; d += 32)
+          q_latent[(static_cast<long long>(r0 + r) * heads + h) * crow + kv_rank + d] = src[dim + d];
+    }
+    cp_async_wait<0>();
+    __syncthreads();
+    float acc[4][4] = {};
+    for (int k = 0; k < kd; k += 16) {
+      uint32_t a[4], b[4];
+      ldsm_x4(a, qs + (lane & 15) * srow + k + (lane >> 4) * 8);
+#pragma unroll
+      for (int g = 0; g < 2; ++g) {
+        ldsm_x4_trans(b, wt + (k + (lane & 15)) * wrow + warp * 32 + g * 16 + (lane >> 4) * 8);
+        mma_bf16_16816(acc[g * 2], a, b[0], b[1]);
+        mma_bf16_16816(acc[g * 2 + 1], a, b[2], b[3]);
+      }
+    }
+#pragma unroll
+    for (int g = 0; g < 4; ++g)
+#pragma unroll
+      for (int e = 0; e < 2; ++e) {
+        const int r = r0 + (lane >> 2) + e * 8, c = c0 + warp * 32 + g * 8 + (lane & 3) * 2;
+        if (r < n && c < kv_rank)
+          *reinterpret_cast<uint32_t*>(q_latent + (static_cast<long long>(r) * heads + h) * crow + c) =
+              pack_bf16(acc[g][2 * e], acc[g][2 * e + 1]);
+      }
+  }
+}
+
+// ------------------------------------------------------------------------------------------- decode
+// grid (spans, tokens, head groups of 32).  A token's visible keys, from the 64-aligned start of its window,
+// are cut into spans of `tiles` 64-key tiles; a CTA works one span off with a running softmax (two tiles in
+// shared memory, the next one in flight) and leaves an unnormalised partial.
+constexpr int kLdKeys = 64, kLdHeads = 32, kLdThreads = 256, kLdMaxRank = 512;
+
+__host__ __device__ constexpr int latent_decode_smem(int crow) {
+  return (2 * kLdKeys + kLdHeads) * (crow + 8) * 2 + kLdHeads * (kLdKeys + 4) * 4 + kLdHeads * (kLdKeys + 8) * 2 +
+         3 * kLdHeads * 4;
+}
+
+__global__ void __launch_bounds__(kLdThreads, 1)
 latent_decode_kernel(const __nv_bfloat16* __restrict__ q_latent, const __nv_bfloat16* __restrict__ cache,
                      const int* __restrict__ rows, const int* __restrict__ positions,
                      const int* __restrict__ row_seq, const int* __restrict__ block_table, int max_blocks,
                      int page_size, float* __restrict__ part_o, float* __restrict__ part_ml, int heads, int kv_rank,
-                     int rot_dim, int window, float scale) {
+                     int rot_dim, int window, int tiles, float scale) {
   extern __shared__ __align__(16) uint8_t ld_raw[];
+  constexpr int kSs = kLdKeys + 4, kPs = kLdKeys + 8, kWarps = kLdThreads / 32;
   const int crow = kv_rank + rot_dim, srow = crow + 8;     // +16 bytes: ldmatrix rows on different banks
-  __nv_bfloat16* ks = reinterpret_cast<__nv_bfloat16*>(ld_raw);   // [64][srow]
-  __nv_bfloat16* qs = ks + kLdKeys * srow;                        // [32][srow]
-  float* ss = reinterpret_cast<float*>(qs + kLdHeads * srow);     // [32][68]
-  __nv_bfloat16* ps = reinterpret_cast<__nv_bfloat16*>(ss + kLdHeads * (kLdKeys + 4));   // [32][72]
-  constexpr int kSs = kLdKeys + 4, kPs = kLdKeys + 8;
+  __nv_bfloat16* ks = reinterpret_cast<__nv_bfloat16*>(ld_raw);   // [2][64][srow]
+  __nv_bfloat16* qs = ks + 2 * kLdKeys * srow;                    // [32][srow]
+  float* ss = reinterpret_cast<float*>(qs + kLdHeads * srow);     // [32][kSs]
+  __nv_bfloat16* ps = reinterpret_cast<__nv_bfloat16*>(ss + kLdHeads * kSs);   // [32][kPs]
+  float* m_run = reinterpret_cast<float*>(ps + kLdHeads * kPs);
+  float* l_run = m_run + kLdHeads;
+  float* corr = l_run + kLdHeads;
   pdl_launch_dependents();
   pdl_wait();
   const int i_tok = blockIdx.y, h0 = blockIdx.z * kLdHeads;
   const int t = rows ? rows[i_tok] : i_tok;
   const int pos = positions[t];
   const int lo = window > 0 ? max(0, pos - window + 1) : 0;
-  const int base = (lo / kLdKeys + blockIdx.x) * kLdKeys;
-  if (base > pos) return;
+  const int base0 = (lo / kLdKeys + blockIdx.x * tiles) * kLdKeys;
+  if (base0 > pos) return;
+  const int n_tiles = min(tiles, (pos - base0) / kLdKeys + 1);
   const int nh = min(kLdHeads, heads - h0);
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int* bt = block_table + static_cast<long long>(row_seq ? row_seq[t] : t) * max_blocks;
   const int vec = crow >> 3;
-  for (int k = warp; k < kLdKeys; k += kLdThreads / 32) {
-    const int key = base + k;
-    __nv_bfloat16* dst = ks + k * srow;
-    if (key >= lo && key <= pos) {
-      const __nv_bfloat16* src = cache + (static_cast<long long>(bt[key / page_size]) * page_size + key % page_size) * crow;
-      for (int i = lane; i < vec; i += 32) cp_async16(dst + i * 8, src + i * 8);
-    } else {   // outside the window or not written: finite zeros, masked below
-      for (int i = lane; i < vec; i += 32) *reinterpret_cast<uint4*>(dst + i * 8) = make_uint4(0, 0, 0, 0);
-    }
-  }
-  const __nv_bfloat16* qsrc = q_latent + (static_cast<long long>(i_tok) * heads + h0) * crow;
-  for (int r = warp; r < kLdHeads; r += kLdThreads / 32)
-    for (int i = lane; i < vec; i += 32) {
-      if (r < nh) cp_async16(qs + r * srow + i * 8, qsrc + static_cast<long long>(r) * crow + i * 8);
-      else *reinterpret_cast<uint4*>(qs + r * srow + i * 8) = make_uint4(0, 0, 0, 0);
-    }
-  cp_async_wait_all();
-  __syncthreads();
-  const int mt = nh > 16 ? 2 : 1;
-  {   // scores: each warp 16 keys x all heads of the group
-    float acc[2][2][4] = {};
-    const int kr = warp * 16 + (lane & 7) + ((lane >> 4) << 3), kc = ((lane >> 3) & 1) * 8;
-    const int ar = lane & 15, ac = (lane >> 4) * 8;
-    for (int k = 0; k < crow; k += 16) {
-      uint32_t bq[4], a0[4], a1[4];
-      ldsm_x4(bq, ks + kr * srow + k + kc);
-      ldsm_x4(a0, qs + ar * srow + k + ac);
-      mma_bf16_16816(acc[0][0], a0, bq[0], bq[1]);
-      mma_bf16_16816(acc[0][1], a0, bq[2], bq[3]);
-      if (mt == 2) {
-        ldsm_x4(a1, qs + (16 + ar) * srow + k + ac);
-        mma_bf16_16816(acc[1][0], a1, bq[0], bq[1]);
-        mma_bf16_16816(acc[1][1], a1, bq[2], bq[3]);
+  auto load_tile = [&](int i) {
+    for (int k = warp; k < kLdKeys; k += kWarps) {
+      const int key = base0 + i * kLdKeys + k;
+      __nv_bfloat16* dst = ks + ((i & 1) * kLdKeys + k) * srow;
+      if (key >= lo && key <= pos) {
+        const __nv_bfloat16* src = cache + (static_cast<long long>(bt[key / page_size]) * page_size + key % page_size) * crow;
+        for (int v = lane; v < vec; v += 32) cp_async16(dst + v * 8, src + v * 8);
+      } else {   // outside the window or not written: finite zeros, masked below
+        for (int v = lane; v < vec; v += 32) *reinterpret_cast<uint4*>(dst + v * 8) = make_uint4(0, 0, 0, 0);
       }
     }
+    cp_async_commit();
+  };
+  const __nv_bfloat16* qsrc = q_latent + (static_cast<long long>(i_tok) * heads + h0) * crow;
+  for (int r = warp; r < kLdHeads; r += kWarps)
+    for (int v = lane; v < vec; v += 32) {
+      if (r < nh) cp_async16(qs + r * srow + v * 8, qsrc + static_cast<long long>(r) * crow + v * 8);
+      else *reinterpret_cast<uint4*>(qs + r * srow + v * 8) = make_uint4(0, 0, 0, 0);
+    }
+  load_tile(0);
+  if (threadIdx.x < kLdHeads) {
+    m_run[threadIdx.x] = -INFINITY;
+    l_run[threadIdx.x] = 0.f;
+  }
+  float o[4][2][2][4] = {};      // up to four 16-column tiles of the latent x (2 x 16 heads) x (2 x 8 columns)
+  for (int i = 0; i < n_tiles; ++i) {
+    if (i + 1 < n_tiles) {
+      load_tile(i + 1);
+      cp_async_wait<1>();
+    } else {
+      cp_async_wait<0>();
+    }
+    __syncthreads();
+    const __nv_bfloat16* kt = ks + (i & 1) * kLdKeys * srow;
+    {   // scores: warp = 16 heads x 16 keys
+      const int m0 = (warp & 1) * 16, n0 = (warp >> 1) * 16;
+      float acc[2][4] = {};
+      const __nv_bfloat16* kp = kt + (n0 + (lane & 7) + ((lane >> 4) << 3)) * srow + ((lane >> 3) & 1) * 8;
+      const __nv_bfloat16* qp = qs + (m0 + (lane & 15)) * srow + (lane >> 4) * 8;
+#pragma unroll 4
+      for (int k = 0; k < crow; k += 16) {
+        uint32_t b[4], a[4];
+        ldsm_x4(b, kp + k);
+        ldsm_x4(a, qp + k);
+        mma_bf16_16816(acc[0], a, b[0], b[1]);
+        mma_bf16_16816(acc[1], a, b[2], b[3]);
+      }
 #pragma unroll
-    for (int m = 0; m < 2; ++m)
-#pragma unroll
-      for (int n = 0; n < 2; ++n)
+      for (int g = 0; g < 2; ++g)
 #pragma unroll
         for (int e = 0; e < 4; ++e)
-          ss[(m * 16 + (lane >> 2) + (e >> 1) * 8) * kSs + warp * 16 + n * 8 + (lane & 3) * 2 + (e & 1)] = acc[m][n][e] * scale;
-  }
-  __syncthreads();
-  const long long chunk = static_cast<long long>(i_tok) * gridDim.x + blockIdx.x;
-  for (int r = warp; r < kLdHeads; r += kLdThreads / 32) {   // softmax of the chunk, one warp per head
-    const int k0 = base + lane, k1 = k0 + 32;
-    const bool ok0 = k0 >= lo && k0 <= pos, ok1 = k1 >= lo && k1 <= pos;
-    const float s0 = ok0 ? ss[r * kSs + lane] : -INFINITY, s1 = ok1 ? ss[r * kSs + lane + 32] : -INFINITY;
-    const float m = warp_max(fmaxf(s0, s1));     // some key of [base, base + 64) is visible, so m is finite
-    const float p0 = ok0 ? __expf(s0 - m) : 0.f, p1 = ok1 ? __expf(s1 - m) : 0.f;
-    ps[r * kPs + lane] = __float2bfloat16(p0);
-    ps[r * kPs + lane + 32] = __float2bfloat16(p1);
-    const float l = warp_sum(p0 + p1);
-    if (lane == 0 && r < nh) {
-      part_ml[(chunk * heads + h0 + r) * 2] = m;
-      part_ml[(chunk * heads + h0 + r) * 2 + 1] = l;
+          ss[(m0 + (lane >> 2) + (e >> 1) * 8) * kSs + n0 + g * 8 + (lane & 3) * 2 + (e & 1)] = acc[g][e] * scale;
     }
-  }
-  __syncthreads();
-  uint32_t pa[2][4][4];
-#pragma unroll
-  for (int m = 0; m < 2; ++m)
-#pragma unroll
-    for (int k = 0; k < 4; ++k)
-      ldsm_x4(pa[m][k], ps + (m * 16 + (lane & 15)) * kPs + k * 16 + (lane >> 4) * 8);
-  for (int n0 = warp * 16; n0 < kv_rank; n0 += (kLdThreads / 32) * 16) {   // 16 latent columns per turn
-    float acc[2][2][4] = {};
-#pragma unroll
-    for (int k = 0; k < 4; ++k) {
-      uint32_t bv[4];
-      ldsm_x4_trans(bv, ks + (k * 16 + (lane & 15)) * srow + n0 + (lane >> 4) * 8);
-      mma_bf16_16816(acc[0][0], pa[0][k], bv[0], bv[1]);
-      mma_bf16_16816(acc[0][1], pa[0][k], bv[2], bv[3]);
-      if (mt == 2) {
-        mma_bf16_16816(acc[1][0], pa[1][k], bv[0], bv[1]);
-        mma_bf16_16816(acc[1][1], pa[1][k], bv[2], bv[3]);
+    __syncthreads();
+    const int k0 = base0 + i * kLdKeys + lane, k1 = k0 + 32;
+    const bool ok0 = k0 >= lo && k0 <= pos, ok1 = k1 >= lo && k1 <= pos;
+    for (int r = warp; r < kLdHeads; r += kWarps) {   // softmax of the tile, one warp per head
+      const float s0 = ok0 ? ss[r * kSs + lane] : -INFINITY, s1 = ok1 ? ss[r * kSs + lane + 32] : -INFINITY;
+      const float m_old = m_run[r];
+      const float m = fmaxf(m_old, warp_max(fmaxf(s0, s1)));     // every tile has a visible key: m is finite
+      const float p0 = ok0 ? __expf(s0 - m) : 0.f, p1 = ok1 ? __expf(s1 - m) : 0.f;
+      ps[r * kPs + lane] = __float2bfloat16(p0);
+      ps[r * kPs + lane + 32] = __float2bfloat16(p1);
+      const float l = warp_sum(p0 + p1);
+      if (lane == 0) {
+        const float c = __expf(m_old - m);
+        corr[r] = c;
+        m_run[r] = m;
+        l_run[r] = fmaf(l_run[r], c, l);
       }
     }
+    __syncthreads();
+    uint32_t pa[2][4][4];
 #pragma unroll
     for (int m = 0; m < 2; ++m)
 #pragma unroll
-      for (int n = 0; n < 2; ++n)
+      for (int k = 0; k < 4; ++k)
+        ldsm_x4(pa[m][k], ps + (m * 16 + (lane & 15)) * kPs + k * 16 + (lane >> 4) * 8);
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+      const int n0 = (warp + j * kWarps) * 16;
+      if (n0 < kv_rank) {
+        if (i > 0) {
+#pragma unroll
+          for (int m = 0; m < 2; ++m)
+#pragma unroll
+            for (int e = 0; e < 2; ++e) {
+              const float c = corr[m * 16 + (lane >> 2) + e * 8];
+#pragma unroll
+              for (int g = 0; g < 2; ++g) {
+                o[j][m][g][2 * e] *= c;
+                o[j][m][g][2 * e + 1] *= c;
+              }
+            }
+        }
+#pragma unroll
+        for (int k = 0; k < 4; ++k) {
+          uint32_t bv[4];
+          ldsm_x4_trans(bv, kt + (k * 16 + (lane & 15)) * srow + n0 + (lane >> 4) * 8);
+#pragma unroll
+          for (int m = 0; m < 2; ++m) {
+            mma_bf16_16816(o[j][m][0], pa[m][k], bv[0], bv[1]);
+            mma_bf16_16816(o[j][m][1], pa[m][k], bv[2], bv[3]);
+          }
+        }
+      }
+    }
+    __syncthreads();     // the tile and the probabilities may be overwritten
+  }
+  const long long span = static_cast<long long>(i_tok) * gridDim.x + blockIdx.x;
+#pragma unroll
+  for (int j = 0; j < 4; ++j) {
+    const int n0 = (warp + j * kWarps) * 16;
+    if (n0 < kv_rank) {
+#pragma unroll
+      for (int m = 0; m < 2; ++m)
 #pragma unroll
         for (int e = 0; e < 2; ++e) {
           const int r = m * 16 + (lane >> 2) + e * 8;
           if (r < nh)
-            *reinterpret_cast<float2*>(part_o + (chunk * heads + h0 + r) * kv_rank + n0 + n * 8 + (lane & 3) * 2) =
-                make_float2(acc[m][n][2 * e], acc[m][n][2 * e + 1]);
+#pragma unroll
+            for (int g = 0; g < 2; ++g)
+              *reinterpret_cast<float2*>(part_o + (span * heads + h0 + r) * kv_rank + n0 + g * 8 + (lane & 3) * 2) =
+                  make_float2(o[j][m][g][2 * e], o[j][m][g][2 * e + 1]);
         }
+    }
+  }
+  if (threadIdx.x < nh) {
+    part_ml[(span * heads + h0 + threadIdx.x) * 2] = m_run[threadIdx.x];
+    part_ml[(span * heads + h0 + threadIdx.x) * 2 + 1] = l_run[threadIdx.x];
   }
 }
 
-// o_latent[i, h] = sum over chunks (and the sink's share of the denominator), bf16.  grid (tokens, heads).
+// o_latent[i, h] = sum over spans (and the sink's share of the denominator), bf16.  grid (tokens, heads), a
+// warp per 128 columns.
 __global__ void __launch_bounds__(128)
 latent_combine_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml,
                       const float* __restrict__ sink, const int* __restrict__ rows,
-                      const int* __restrict__ positions, __nv_bfloat16* __restrict__ o_latent, int chunks, int heads,
-                      int kv_rank, int window) {
+                      const int* __restrict__ positions, __nv_bfloat16* __restrict__ o_latent, int spans, int tiles,
+                      int heads, int kv_rank, int window) {
   pdl_launch_dependents();
   pdl_wait();
-  const int i_tok = blockIdx.x, h = blockIdx.y;
+  const int i_tok = blockIdx.x, h = blockIdx.y, lane = threadIdx.x & 31;
   const int pos = positions[rows ? rows[i_tok] : i_tok];
   const int lo = window > 0 ? max(0, pos - window + 1) : 0;
-  const int n = min(chunks, pos / kLdKeys - lo / kLdKeys + 1);
-  const float* ml = part_ml + (static_cast<long long>(i_tok) * chunks * heads + h) * 2;
-  float m = sink ? sink[h] : -INFINITY;
-  for (int c = 0; c < n; ++c) m = fmaxf(m, ml[static_cast<long long>(c) * heads * 2]);
-  float l = sink ? __expf(sink[h] - m) : 0.f;
-  for (int c = 0; c < n; ++c)
-    l += __expf(ml[static_cast<long long>(c) * heads * 2] - m) * ml[static_cast<long long>(c) * heads * 2 + 1];
+  const int n = min(spans, (pos / kLdKeys - lo / kLdKeys) / tiles + 1);
+  const float2* ml = reinterpret_cast<const float2*>(part_ml) + static_cast<long long>(i_tok) * spans * heads + h;
+  const float s0 = sink ? sink[h] : -INFINITY;
+  float m = -INFINITY, l = 0.f;
+  for (int c = lane; c < n; c += 32) {       // a lane's spans, then across lanes
+    const float2 v = ml[static_cast<long long>(c) * heads];
+    const float mn = fmaxf(m, v.x);
+    l = l * __expf(m - mn) + v.y * __expf(v.x - mn);
+    m = mn;
+  }
+  const float top = fmaxf(warp_max(m), s0);
+  l = warp_sum(m == -INFINITY ? 0.f : l * __expf(m - top)) + (sink ? __expf(s0 - top) : 0.f);
   const float inv = 1.0f / l;
-  for (int r = threadIdx.x; r < kv_rank; r += 128) {
-    float acc = 0.f;
-#pragma unroll 4
-    for (int c = 0; c < n; ++c)
-      acc = fmaf(__expf(ml[static_cast<long long>(c) * heads * 2] - m),
-                 part_o[((static_cast<long long>(i_tok) * chunks + c) * heads + h) * kv_rank + r], acc);
-    o_latent[(static_cast<long long>(i_tok) * heads + h) * kv_rank + r] = __float2bfloat16(acc * inv);
+  const float* src = part_o + (static_cast<long long>(i_tok) * spans * heads + h) * kv_rank;
+  const long long pitch = static_cast<long long>(heads) * kv_rank;
+  for (int r = threadIdx.x * 4; r < kv_rank; r += 512) {
+    float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
+    for (int c0 = 0; c0 < n; c0 += 8) {
+      float4 v[8];
+      float w[8];
+#pragma unroll
+      for (int k = 0; k < 8; ++k) {
+        const int c = min(c0 + k, n - 1);
+        v[k] = *reinterpret_cast<const float4*>(src + c * pitch + r);
+        w[k] = ml[static_cast<long long>(c) * heads].x;
+      }
+#pragma unroll
+      for (int k = 0; k < 8; ++k)
+        if (c0 + k < n) {
+          const float e = __expf(w[k] - top);
+          acc.x = fmaf(e, v[k].x, acc.x);
+          acc.y = fmaf(e, v[k].y, acc.y);
+          acc.z = fmaf(e, v[k].z, acc.z);
+          acc.w = fmaf(e, v[k].w, acc.w);
+        }
+    }
+    store4(o_latent + (static_cast<long long>(i_tok) * heads + h) * kv_rank + r, acc.x * inv, acc.y * inv, acc.z * inv,
+           acc.w * inv);
   }
 }
 
-// out[t, h, v] = W_uv o_latent.  grid (heads, v tiles of 32); the weight tile is staged ahead of the wait.
-constexpr int kUpRows = 32;
+// out[t, h, v] = W_uv o_latent.  grid (heads, v tiles of 32); the weight tile is staged ahead of the wait,
+// 16 tokens a pass, a warp per 8 values.
+constexpr int kUpV = 32, kUpThreads = 128;
+__host__ __device__ constexpr int up_row(int kv_rank) { return (kv_rank + 31) / 32 * 32 + 8; }
+__host__ __device__ constexpr int up_smem(int kv_rank) { return (kUpV + 16) * up_row(kv_rank) * 2; }
 
-__global__ void __launch_bounds__(128)
+__global__ void __launch_bounds__(kUpThreads)
 latent_up_kernel(const __nv_bfloat16* __restrict__ o_latent, const __nv_bfloat16* __restrict__ w_uv,
                  const int* __restrict__ rows, int n, __nv_bfloat16* __restrict__ out, int heads, int vdim,
                  int kv_rank) {
   extern __shared__ __align__(16) uint8_t up_raw[];
-  __nv_bfloat16* wt = reinterpret_cast<__nv_bfloat16*>(up_raw);   // [32][kv_rank]
-  pdl_launch_dependents();
-  const int h = blockIdx.x, v0 = blockIdx.y * kUpRows;
-  const int nv = min(kUpRows, vdim - v0);
-  const uint4* src = reinterpret_cast<const uint4*>(w_uv + (static_cast<long long>(h) * vdim + v0) * kv_rank);
-  for (int i = threadIdx.x; i < nv * (kv_rank / 8); i += 128) reinterpret_cast<uint4*>(wt)[i] = src[i];
-  pdl_wait();
-  __syncthreads();
+  const int srow = up_row(kv_rank), kd = srow - 8;
+  __nv_bfloat16* wt = reinterpret_cast<__nv_bfloat16*>(up_raw);   // [32][srow]
+  __nv_bfloat16* os = wt + kUpV * srow;                           // [16][srow]
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  for (int i = warp; i < n; i += 4) {          // a warp per token, lanes across the latent
-    const long long t = rows ? rows[i] : i;
-    const __nv_bfloat16* o = o_latent + (static_cast<long long>(i) * heads + h) * kv_rank;
-    float mine = 0.f;
-    for (int vb = 0; vb < nv; vb += 8) {
-      float acc[8] = {};
-      for (int r = lane * 2; r < kv_rank; r += 64) {
-        const uint32_t ow = *reinterpret_cast<const uint32_t*>(o + r);
-        const float o0 = bf16lo(ow), o1 = bf16hi(ow);
+  const int h = blockIdx.x, v0 = blockIdx.y * kUpV;
+  pdl_launch_dependents();
+  auto stage = [&](__nv_bfloat16* dst, const __nv_bfloat16* src, bool there) {   // one row, by a warp
+    for (int c = lane * 8; c < kd; c += 256) {
+      if (there && c < kv_rank) cp_async16(dst + c, src + c);
+      else *reinterpret_cast<uint4*>(dst + c) = make_uint4(0, 0, 0, 0);
+    }
+  };
+  for (int r = warp; r < kUpV; r += kUpThreads / 32)
+    stage(wt + r * srow, w_uv + (static_cast<long long>(h) * vdim + v0 + r) * kv_rank, v0 + r < vdim);
+  pdl_wait();
+  for (int r0 = 0; r0 < n; r0 += 16) {
+    __syncthreads();
+    for (int r = warp; r < 16; r += kUpThreads / 32)
+      stage(os + r * srow, o_latent + (static_cast<long long>(r0 + r) * heads + h) * kv_rank, r0 + r < n);
+    cp_async_commit();
+    cp_async_wait<0>();
+    __syncthreads();
+    float acc[2][4] = {};
+    const __nv_bfloat16* wp = wt + (warp * 8 + (lane & 7)) * srow + (lane >> 3) * 8;
+    const __nv_bfloat16* op = os + (lane & 15) * srow + (lane >> 4) * 8;
+#pragma unroll 4
+    for (int k = 0; k < kd; k += 32) {
+      uint32_t b[4], a0[4], a1[4];
+      ldsm_x4(b, wp + k);
+      ldsm_x4(a0, op + k);
+      ldsm_x4(a1, op + k + 16);
+      mma_bf16_16816(acc[0], a0, b[0], b[1]);
+      mma_bf16_16816(acc[1], a1, b[2], b[3]);
+    }
 #pragma unroll
-        for (int v = 0; v < 8; ++v) {
-          const uint32_t w = *reinterpret_cast<const uint32_t*>(wt + min(vb + v, nv - 1) * kv_rank + r);
-          acc[v] = fmaf(bf16lo(w), o0, fmaf(bf16hi(w), o1, acc[v]));
-        }
-      }
-#pragma unroll
-      for (int v = 0; v < 8; ++v) {
-        const float s = warp_sum(acc[v]);
-        if (lane == vb + v) mine = s;
+    for (int e = 0; e < 4; ++e) {
+      const int r = r0 + (lane >> 2) + (e >> 1) * 8, v = v0 + warp * 8 + (lane & 3) * 2 + (e & 1);
+      if (r < n && v < vdim) {
+        const long long t = rows ? rows[r] : r;
+        out[(t * heads + h) * vdim + v] = __float2bfloat16(acc[0][e] + acc[1][e]);
       }
     }
-    if (lane < nv) out[(t * heads + h) * vdim + v0 + lane] = __float2bfloat16(mine);
   }
 }
 
 // Sizes the latent-space tensor-core path takes.
 bool latent_decode_ok(const bcg_layer* l) {
   const int crow = l->kv_rank + l->rot_dim;
-  return l->kv_rank % 16 == 0 && crow % 16 == 0 && l->rot_dim % 8 == 0 && latent_decode_smem(crow) <= 220 * 1024 &&
-         l->dim * kAbCols * 2 + kAbRows * l->dim * 4 <= 200 * 1024 && kUpRows * l->kv_rank * 2 <= 200 * 1024;
+  return l->kv_rank % 16 == 0 && l->kv_rank <= kLdMaxRank && crow % 16 == 0 &&
+         latent_decode_smem(crow) <= 220 * 1024 && absorb_smem(l->dim) <= 200 * 1024 && up_smem(l->kv_rank) <= 200 * 1024;
 }
 
-int latent_decode_chunks(const bcg_layer* l, int max_context) {
-  const int span = l->window > 0 && l->window < max_context ? l->window : max_context;
-  return span / kLdKeys + 2 < (max_context + kLdKeys - 1) / kLdKeys ? span / kLdKeys + 2
-                                                                    : (max_context + kLdKeys - 1) / kLdKeys;
-}
+// Key tiles per span: a CTA per tile while that does not fill the GPU, longer spans (fewer partials) when it
+// more than does.
+static int span_tiles(int n) { return n <= 16 ? 1 : n <= 32 ? 2 : 4; }
 
 int latent_decode(const bcg_layer* l, const bcg_stack_ws* ws, const bcg_step_batch* b, int page_size,
                   cudaStream_t st) {
   const int n = b->single_rows ? b->n_single : b->T;
   const int crow = l->kv_rank + l->rot_dim;
   const int q_row = l->q_ld > 0 ? l->q_ld : l->dim + l->rot_dim;
-  const int chunks = latent_decode_chunks(l, b->max_context);
-  if (n > ws->D_max || n > 65535 || static_cast<long long>(n) * chunks * l->heads * l->kv_rank > ws->part_floats) {
-    set_last_error("bcg_latent_attention", "single tokens x chunks exceed the decode scratch");
+  const int reach = l->window > 0 && l->window < b->max_context ? l->window + kLdKeys : b->max_context;
+  const int tiles = span_tiles(n), spans = ((reach + kLdKeys - 1) / kLdKeys + tiles - 1) / tiles;
+  if (n > ws->D_max || n > 65535 || static_cast<long long>(n) * spans * l->heads * l->kv_rank > ws->part_floats) {
+    set_last_error("bcg_latent_attention", "single tokens x key spans exceed the decode scratch");
     return BCG_ERR_TOO_LARGE;
   }
   auto* ql = static_cast<__nv_bfloat16*>(ws->q_latent);
   auto* ol = static_cast<__nv_bfloat16*>(ws->o_latent);
-  const size_t sm_a = static_cast<size_t>(l->dim) * kAbCols * 2 + kAbRows * l->dim * 4;
-  const size_t sm_u = static_cast<size_t>(kUpRows) * l->kv_rank * 2;
   BCG_TRY(ensure_dynamic_smem(reinterpret_cast<const void*>(latent_absorb_kernel), 200 * 1024));
   BCG_TRY(ensure_dynamic_smem(reinterpret_cast<const void*>(latent_decode_kernel), 220 * 1024));
   BCG_TRY(ensure_dynamic_smem(reinterpret_cast<const void*>(latent_up_kernel), 200 * 1024));
-  BCG_CUDA_CHECK(launch_k(latent_absorb_kernel, dim3(l->heads, (l->kv_rank + kAbCols - 1) / kAbCols), dim3(128), sm_a,
-                          st, static_cast<const __nv_bfloat16*>(ws->q), static_cast<const __nv_bfloat16*>(l->w_uk),
-                          b->single_rows, n, ql, l->heads, l->dim, l->rot_dim, l->kv_rank, q_row));
-  BCG_CUDA_CHECK(launch_k(latent_decode_kernel, dim3(chunks, n, (l->heads + kLdHeads - 1) / kLdHeads), dim3(kLdThreads),
+  BCG_CUDA_CHECK(launch_k(latent_absorb_kernel, dim3(l->heads, (l->kv_rank + kAbCols - 1) / kAbCols), dim3(kAbThreads),
+                          absorb_smem(l->dim), st, static_cast<const __nv_bfloat16*>(ws->q),
+                          static_cast<const __nv_bfloat16*>(l->w_uk), b->single_rows, n, ql, l->heads, l->dim,
+                          l->rot_dim, l->kv_rank, q_row));
+  BCG_CUDA_CHECK(launch_k(latent_decode_kernel, dim3(spans, n, (l->heads + kLdHeads - 1) / kLdHeads), dim3(kLdThreads),
                           latent_decode_smem(crow), st, ql, static_cast<const __nv_bfloat16*>(l->cache),
                           b->single_rows, b->positions, b->row_seq, b->block_table, b->max_blocks, page_size,
-                          ws->part_o, ws->part_ml, l->heads, l->kv_rank, l->rot_dim, l->window, l->scale));
+                          ws->part_o, ws->part_ml, l->heads, l->kv_rank, l->rot_dim, l->window, tiles, l->scale));
   BCG_CUDA_CHECK(launch_k(latent_combine_kernel, dim3(n, l->heads), dim3(128), 0, st, ws->part_o, ws->part_ml, l->sink,
-                          b->single_rows, b->positions, ol, chunks, l->heads, l->kv_rank, l->window));
-  BCG_CUDA_CHECK(launch_k(latent_up_kernel, dim3(l->heads, (l->vdim + kUpRows - 1) / kUpRows), dim3(128), sm_u, st, ol,
-                          static_cast<const __nv_bfloat16*>(l->w_uv), b->single_rows, n,
+                          b->single_rows, b->positions, ol, spans, tiles, l->heads, l->kv_rank, l->window));
+  BCG_CUDA_CHECK(launch_k(latent_up_kernel, dim3(l->heads, (l->vdim + kUpV - 1) / kUpV), dim3(kUpThreads),
+                          up_smem(l->kv_rank), st, ol, static_cast<const __nv_bfloat16*>(l->w_uv), b->single_rows, n,
                           static_cast<__nv_bfloat16*>(ws->mix), l->heads, l->vdim, l->kv_rank));
   return BCG_OK;
 }
