@@ -244,6 +244,7 @@ delta_token_kernel(const DeltaArgs a, T* __restrict__ out) {
   __shared__ __align__(16) float op[6 * DP];
   __shared__ float so[kCols], sc[3];
   __shared__ RowSum<kTokThreads, CL, 1> sh;
+  __shared__ RowSum<kTokThreads, 1, 3> sums;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, rg = lane >> 2, D = a.dim, HD = a.heads * a.dim;
   const int cta = CL > 1 ? static_cast<int>(blockIdx.x) : 0;
   const int h = blockIdx.y, t = blockIdx.z;
@@ -292,7 +293,35 @@ delta_token_kernel(const DeltaArgs a, T* __restrict__ out) {
       if (threadIdx.x + k * kTokThreads < 6 * DP) raw[threadIdx.x + k * kTokThreads] = acc[k];
   }
   __syncthreads();
-  if (warp == 0) prepare_token<DP>(a, h, raw, op, DP, sc);
+  {   // prepare_token with a thread per channel: a single token's latency is on the critical path
+    const int i = threadIdx.x;
+    float r = 0.f, kx = 0.f, w = 0.f, rate = 0.f, v = 0.f, g = 0.f;
+    if (i < D) {
+      r = raw[i];
+      kx = raw[DP + i];
+      v = raw[2 * DP + i];
+      g = sigmoid_f32(raw[3 * DP + i]);
+      rate = sigmoid_f32(raw[4 * DP + i] + a.rate_bias[h * D + i]);
+      w = 1.0f + expm1f(-kDecayGain * sigmoid_f32(raw[5 * DP + i] + a.decay_bias[h * D + i]));
+    }
+    // sums of k^2, r.(a*k), r.k; the unit key's factor is applied to the sums
+    float part[3] = {kx * kx, r * (rate * kx), r * kx};
+    row_sum<kTokThreads, 1, 3>(sums, part, 0);
+    const float inv = rsqrtf(part[0] + 1e-6f);
+    if (i < DP) {
+      op[i] = kx;
+      op[DP + i] = r * w;
+      op[2 * DP + i] = w;
+      op[3 * DP + i] = rate * (kx * inv);
+      op[4 * DP + i] = v;
+      op[5 * DP + i] = g;
+    }
+    if (i == 0) {
+      sc[0] = inv;
+      sc[1] = part[1] * inv;
+      sc[2] = part[2];
+    }
+  }
   __syncthreads();
   float o[CPT];
   S.token(op, DP, sc, rg, col, o);

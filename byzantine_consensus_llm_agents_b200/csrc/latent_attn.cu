@@ -209,7 +209,7 @@ int latent_plain(const bcg_layer* l, const void* q, void* out, const bcg_step_ba
 
 // ------------------------------------------------------------------------------------------- absorb
 // q_latent[i, h] = (W_uk^T q_unrotated, q_rotated) for single token i = rows[i].  grid (heads, 128-column
-// tiles of the latent); the weight tile is staged ahead of the dependency wait; mma.sync over 16 tokens a pass.
+// tiles of the latent, groups of 16 tokens); the weight tile is staged ahead of the dependency wait.
 constexpr int kAbCols = 128, kAbThreads = 128;
 
 __device__ __forceinline__ void cp_async16(void* dst, const void* src) {
@@ -261,39 +261,47 @@ latent_absorb_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* _
   }
   cp_async_commit();
   pdl_wait();
-  for (int r0 = 0; r0 < n; r0 += 16) {
-    __syncthreads();                       // the pass before has read its queries
-    for (int r = warp; r < 16; r += kAbThreads / 32) {
-      const long long t = r0 + r < n ? (rows ? rows[r0 + r] : r0 + r) : -1;
-      const __nv_bfloat16* src = q + (t * heads + h) * q_row;
+  const int r0 = blockIdx.z * 16;
+  const bool wide = (dim & 7) == 0 && (q_row & 7) == 0;
+  for (int r = warp; r < 16; r += kAbThreads / 32) {
+    const long long t = r0 + r < n ? (rows ? rows[r0 + r] : r0 + r) : -1;
+    const __nv_bfloat16* src = q + (t * heads + h) * q_row;
+    if (wide && t >= 0) {
+      for (int d = lane * 8; d < kd; d += 256) {
+        if (d < dim) cp_async16(qs + r * srow + d, src + d);
+        else *reinterpret_cast<uint4*>(qs + r * srow + d) = make_uint4(0, 0, 0, 0);
+      }
+    } else {
       for (int d = lane; d < kd; d += 32) qs[r * srow + d] = (t >= 0 && d < dim) ? src[d] : __float2bfloat16(0.f);
-      if (blockIdx.y == 0 && t >= 0)
-        for (int d = lane; d < rot_dim; d += 32)
-          q_latent[(static_cast<long long>(r0 + r) * heads + h) * crow + kv_rank + d] = src[dim + d];
     }
-    cp_async_wait<0>();
-    __syncthreads();
-    float acc[4][4] = {};
-    for (int k = 0; k < kd; k += 16) {
-      uint32_t a[4], b[4];
-      ldsm_x4(a, qs + (lane & 15) * srow + k + (lane >> 4) * 8);
-#pragma unroll
-      for (int g = 0; g < 2; ++g) {
-        ldsm_x4_trans(b, wt + (k + (lane & 15)) * wrow + warp * 32 + g * 16 + (lane >> 4) * 8);
-        mma_bf16_16816(acc[g * 2], a, b[0], b[1]);
-        mma_bf16_16816(acc[g * 2 + 1], a, b[2], b[3]);
-      }
-    }
-#pragma unroll
-    for (int g = 0; g < 4; ++g)
-#pragma unroll
-      for (int e = 0; e < 2; ++e) {
-        const int r = r0 + (lane >> 2) + e * 8, c = c0 + warp * 32 + g * 8 + (lane & 3) * 2;
-        if (r < n && c < kv_rank)
-          *reinterpret_cast<uint32_t*>(q_latent + (static_cast<long long>(r) * heads + h) * crow + c) =
-              pack_bf16(acc[g][2 * e], acc[g][2 * e + 1]);
-      }
+    if (blockIdx.y == 0 && t >= 0)
+      for (int d = lane; d < rot_dim; d += 32)
+        q_latent[(static_cast<long long>(r0 + r) * heads + h) * crow + kv_rank + d] = src[dim + d];
   }
+  cp_async_commit();
+  cp_async_wait<0>();
+  __syncthreads();
+  float acc[4][4] = {};
+#pragma unroll 4
+  for (int k = 0; k < kd; k += 16) {
+    uint32_t a[4], b[4];
+    ldsm_x4(a, qs + (lane & 15) * srow + k + (lane >> 4) * 8);
+#pragma unroll
+    for (int g = 0; g < 2; ++g) {
+      ldsm_x4_trans(b, wt + (k + (lane & 15)) * wrow + warp * 32 + g * 16 + (lane >> 4) * 8);
+      mma_bf16_16816(acc[g * 2], a, b[0], b[1]);
+      mma_bf16_16816(acc[g * 2 + 1], a, b[2], b[3]);
+    }
+  }
+#pragma unroll
+  for (int g = 0; g < 4; ++g)
+#pragma unroll
+    for (int e = 0; e < 2; ++e) {
+      const int r = r0 + (lane >> 2) + e * 8, c = c0 + warp * 32 + g * 8 + (lane & 3) * 2;
+      if (r < n && c < kv_rank)
+        *reinterpret_cast<uint32_t*>(q_latent + (static_cast<long long>(r) * heads + h) * crow + c) =
+            pack_bf16(acc[g][2 * e], acc[g][2 * e + 1]);
+    }
 }
 
 // ------------------------------------------------------------------------------------------- decode
@@ -337,11 +345,16 @@ latent_decode_kernel(const __nv_bfloat16* __restrict__ q_latent, const __nv_bflo
   const int* bt = block_table + static_cast<long long>(row_seq ? row_seq[t] : t) * max_blocks;
   const int vec = crow >> 3;
   auto load_tile = [&](int i) {
-    for (int k = warp; k < kLdKeys; k += kWarps) {
-      const int key = base0 + i * kLdKeys + k;
-      __nv_bfloat16* dst = ks + ((i & 1) * kLdKeys + k) * srow;
-      if (key >= lo && key <= pos) {
-        const __nv_bfloat16* src = cache + (static_cast<long long>(bt[key / page_size]) * page_size + key % page_size) * crow;
+    // a warp loads eight keys; their cache rows are looked up by eight lanes at once
+    const int mine = base0 + i * kLdKeys + warp * 8 + (lane & 7);
+    long long at = -1;
+    if (mine >= lo && mine <= pos) at = (static_cast<long long>(bt[mine / page_size]) * page_size + mine % page_size) * crow;
+#pragma unroll
+    for (int k = 0; k < 8; ++k) {
+      __nv_bfloat16* dst = ks + ((i & 1) * kLdKeys + warp * 8 + k) * srow;
+      const long long row = __shfl_sync(0xffffffffu, at, k);
+      if (row >= 0) {
+        const __nv_bfloat16* src = cache + row;
         for (int v = lane; v < vec; v += 32) cp_async16(dst + v * 8, src + v * 8);
       } else {   // outside the window or not written: finite zeros, masked below
         for (int v = lane; v < vec; v += 32) *reinterpret_cast<uint4*>(dst + v * 8) = make_uint4(0, 0, 0, 0);
@@ -392,19 +405,42 @@ latent_decode_kernel(const __nv_bfloat16* __restrict__ q_latent, const __nv_bflo
     __syncthreads();
     const int k0 = base0 + i * kLdKeys + lane, k1 = k0 + 32;
     const bool ok0 = k0 >= lo && k0 <= pos, ok1 = k1 >= lo && k1 <= pos;
-    for (int r = warp; r < kLdHeads; r += kWarps) {   // softmax of the tile, one warp per head
-      const float s0 = ok0 ? ss[r * kSs + lane] : -INFINITY, s1 = ok1 ? ss[r * kSs + lane + 32] : -INFINITY;
-      const float m_old = m_run[r];
-      const float m = fmaxf(m_old, warp_max(fmaxf(s0, s1)));     // every tile has a visible key: m is finite
-      const float p0 = ok0 ? __expf(s0 - m) : 0.f, p1 = ok1 ? __expf(s1 - m) : 0.f;
-      ps[r * kPs + lane] = __float2bfloat16(p0);
-      ps[r * kPs + lane + 32] = __float2bfloat16(p1);
-      const float l = warp_sum(p0 + p1);
-      if (lane == 0) {
-        const float c = __expf(m_old - m);
+    constexpr int kR = kLdHeads / kWarps;             // softmax of the tile: a warp's heads side by side
+    float p0[kR], p1[kR], m[kR], l[kR], m_old[kR];
+#pragma unroll
+    for (int x = 0; x < kR; ++x) {
+      const int r = warp + x * kWarps;
+      p0[x] = ok0 ? ss[r * kSs + lane] : -INFINITY;
+      p1[x] = ok1 ? ss[r * kSs + lane + 32] : -INFINITY;
+      m_old[x] = m_run[r];
+      m[x] = fmaxf(p0[x], p1[x]);
+    }
+#pragma unroll
+    for (int off = 16; off > 0; off >>= 1)
+#pragma unroll
+      for (int x = 0; x < kR; ++x) m[x] = fmaxf(m[x], __shfl_xor_sync(0xffffffffu, m[x], off));
+#pragma unroll
+    for (int x = 0; x < kR; ++x) {                    // every tile has a visible key: m is finite
+      const int r = warp + x * kWarps;
+      m[x] = fmaxf(m[x], m_old[x]);
+      p0[x] = ok0 ? __expf(p0[x] - m[x]) : 0.f;
+      p1[x] = ok1 ? __expf(p1[x] - m[x]) : 0.f;
+      ps[r * kPs + lane] = __float2bfloat16(p0[x]);
+      ps[r * kPs + lane + 32] = __float2bfloat16(p1[x]);
+      l[x] = p0[x] + p1[x];
+    }
+#pragma unroll
+    for (int off = 16; off > 0; off >>= 1)
+#pragma unroll
+      for (int x = 0; x < kR; ++x) l[x] += __shfl_xor_sync(0xffffffffu, l[x], off);
+    if (lane == 0) {
+#pragma unroll
+      for (int x = 0; x < kR; ++x) {
+        const int r = warp + x * kWarps;
+        const float c = __expf(m_old[x] - m[x]);
         corr[r] = c;
-        m_run[r] = m;
-        l_run[r] = fmaf(l_run[r], c, l);
+        m_run[r] = m[x];
+        l_run[r] = fmaf(l_run[r], c, l[x]);
       }
     }
     __syncthreads();
@@ -522,8 +558,8 @@ latent_combine_kernel(const float* __restrict__ part_o, const float* __restrict_
   }
 }
 
-// out[t, h, v] = W_uv o_latent.  grid (heads, v tiles of 32); the weight tile is staged ahead of the wait,
-// 16 tokens a pass, a warp per 8 values.
+// out[t, h, v] = W_uv o_latent.  grid (heads, v tiles of 32, groups of 16 tokens); the weight tile is staged
+// ahead of the wait, a warp per 8 values.
 constexpr int kUpV = 32, kUpThreads = 128;
 __host__ __device__ constexpr int up_row(int kv_rank) { return (kv_rank + 31) / 32 * 32 + 8; }
 __host__ __device__ constexpr int up_smem(int kv_rank) { return (kUpV + 16) * up_row(kv_rank) * 2; }
@@ -548,32 +584,30 @@ latent_up_kernel(const __nv_bfloat16* __restrict__ o_latent, const __nv_bfloat16
   for (int r = warp; r < kUpV; r += kUpThreads / 32)
     stage(wt + r * srow, w_uv + (static_cast<long long>(h) * vdim + v0 + r) * kv_rank, v0 + r < vdim);
   pdl_wait();
-  for (int r0 = 0; r0 < n; r0 += 16) {
-    __syncthreads();
-    for (int r = warp; r < 16; r += kUpThreads / 32)
-      stage(os + r * srow, o_latent + (static_cast<long long>(r0 + r) * heads + h) * kv_rank, r0 + r < n);
-    cp_async_commit();
-    cp_async_wait<0>();
-    __syncthreads();
-    float acc[2][4] = {};
-    const __nv_bfloat16* wp = wt + (warp * 8 + (lane & 7)) * srow + (lane >> 3) * 8;
-    const __nv_bfloat16* op = os + (lane & 15) * srow + (lane >> 4) * 8;
+  const int r0 = blockIdx.z * 16;
+  for (int r = warp; r < 16; r += kUpThreads / 32)
+    stage(os + r * srow, o_latent + (static_cast<long long>(r0 + r) * heads + h) * kv_rank, r0 + r < n);
+  cp_async_commit();
+  cp_async_wait<0>();
+  __syncthreads();
+  float acc[2][4] = {};
+  const __nv_bfloat16* wp = wt + (warp * 8 + (lane & 7)) * srow + (lane >> 3) * 8;
+  const __nv_bfloat16* op = os + (lane & 15) * srow + (lane >> 4) * 8;
 #pragma unroll 4
-    for (int k = 0; k < kd; k += 32) {
-      uint32_t b[4], a0[4], a1[4];
-      ldsm_x4(b, wp + k);
-      ldsm_x4(a0, op + k);
-      ldsm_x4(a1, op + k + 16);
-      mma_bf16_16816(acc[0], a0, b[0], b[1]);
-      mma_bf16_16816(acc[1], a1, b[2], b[3]);
-    }
+  for (int k = 0; k < kd; k += 32) {
+    uint32_t b[4], a0[4], a1[4];
+    ldsm_x4(b, wp + k);
+    ldsm_x4(a0, op + k);
+    ldsm_x4(a1, op + k + 16);
+    mma_bf16_16816(acc[0], a0, b[0], b[1]);
+    mma_bf16_16816(acc[1], a1, b[2], b[3]);
+  }
 #pragma unroll
-    for (int e = 0; e < 4; ++e) {
-      const int r = r0 + (lane >> 2) + (e >> 1) * 8, v = v0 + warp * 8 + (lane & 3) * 2 + (e & 1);
-      if (r < n && v < vdim) {
-        const long long t = rows ? rows[r] : r;
-        out[(t * heads + h) * vdim + v] = __float2bfloat16(acc[0][e] + acc[1][e]);
-      }
+  for (int e = 0; e < 4; ++e) {
+    const int r = r0 + (lane >> 2) + (e >> 1) * 8, v = v0 + warp * 8 + (lane & 3) * 2 + (e & 1);
+    if (r < n && v < vdim) {
+      const long long t = rows ? rows[r] : r;
+      out[(t * heads + h) * vdim + v] = __float2bfloat16(acc[0][e] + acc[1][e]);
     }
   }
 }
@@ -605,7 +639,7 @@ int latent_decode(const bcg_layer* l, const bcg_stack_ws* ws, const bcg_step_bat
   BCG_TRY(ensure_dynamic_smem(reinterpret_cast<const void*>(latent_absorb_kernel), 200 * 1024));
   BCG_TRY(ensure_dynamic_smem(reinterpret_cast<const void*>(latent_decode_kernel), 220 * 1024));
   BCG_TRY(ensure_dynamic_smem(reinterpret_cast<const void*>(latent_up_kernel), 200 * 1024));
-  BCG_CUDA_CHECK(launch_k(latent_absorb_kernel, dim3(l->heads, (l->kv_rank + kAbCols - 1) / kAbCols), dim3(kAbThreads),
+  BCG_CUDA_CHECK(launch_k(latent_absorb_kernel, dim3(l->heads, (l->kv_rank + kAbCols - 1) / kAbCols, (n + 15) / 16), dim3(kAbThreads),
                           absorb_smem(l->dim), st, static_cast<const __nv_bfloat16*>(ws->q),
                           static_cast<const __nv_bfloat16*>(l->w_uk), b->single_rows, n, ql, l->heads, l->dim,
                           l->rot_dim, l->kv_rank, q_row));
@@ -615,7 +649,7 @@ int latent_decode(const bcg_layer* l, const bcg_stack_ws* ws, const bcg_step_bat
                           ws->part_o, ws->part_ml, l->heads, l->kv_rank, l->rot_dim, l->window, tiles, l->scale));
   BCG_CUDA_CHECK(launch_k(latent_combine_kernel, dim3(n, l->heads), dim3(128), 0, st, ws->part_o, ws->part_ml, l->sink,
                           b->single_rows, b->positions, ol, spans, tiles, l->heads, l->kv_rank, l->window));
-  BCG_CUDA_CHECK(launch_k(latent_up_kernel, dim3(l->heads, (l->vdim + kUpV - 1) / kUpV), dim3(kUpThreads),
+  BCG_CUDA_CHECK(launch_k(latent_up_kernel, dim3(l->heads, (l->vdim + kUpV - 1) / kUpV, (n + 15) / 16), dim3(kUpThreads),
                           up_smem(l->kv_rank), st, ol, static_cast<const __nv_bfloat16*>(l->w_uv), b->single_rows, n,
                           static_cast<__nv_bfloat16*>(ws->mix), l->heads, l->vdim, l->kv_rank));
   return BCG_OK;
