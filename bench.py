@@ -363,8 +363,20 @@ def main():
                     help="1: qk-norm / RoPE / KV write inside decode attention (one launch fewer per layer)")
     ap.add_argument("--pdl", type=int, default=int(os.environ.get("BCG_B200_PDL", "1")),
                     help="programmatic dependent launch for the decode step (1 = on)")
+    ap.add_argument("--design", default=None,
+                    help="instead of the default workload: throughput of a layer-stack design (bekopel) beside a "
+                         "dense model of equal size, one JSON line")
+    ap.add_argument("--design-sizes", default=None, help="comma-separated subset of the sizes of --design")
     a = ap.parse_args()
 
+    if a.design:
+        from byzantine_consensus_llm_agents_b200 import design_bench
+        hbm, tf, kind = load_peaks()
+        clk = ClockSampler(0)
+        line = design_bench.run(a.design, hbm, tf, kind, a.design_sizes.split(",") if a.design_sizes else None)
+        line["clocks"] = clk.stop()
+        print(json.dumps(line))
+        return
     if os.environ.get("BCG_BENCH_WATCHDOG_S"):
         # a hung collective must not eat a GPU lease: dump every thread's stack and exit
         import faulthandler
