@@ -308,10 +308,10 @@ latent_absorb_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* _
 // grid (spans, tokens, head groups of 32).  A token's visible keys, from the 64-aligned start of its window,
 // are cut into spans of `tiles` 64-key tiles; a CTA works one span off with a running softmax (two tiles in
 // shared memory, the next one in flight) and leaves an unnormalised partial.
-constexpr int kLdKeys = 64, kLdHeads = 32, kLdThreads = 256, kLdMaxRank = 512;
+constexpr int kLdKeys = 64, kLdHeads = 32, kLdThreads = 512, kLdMaxRank = 512;
 
 __host__ __device__ constexpr int latent_decode_smem(int crow) {
-  return (2 * kLdKeys + kLdHeads) * (crow + 8) * 2 + kLdHeads * (kLdKeys + 4) * 4 + kLdHeads * (kLdKeys + 8) * 2 +
+  return (2 * kLdKeys + kLdHeads) * (crow + 8) * 2 + 2 * kLdHeads * (kLdKeys + 4) * 4 + kLdHeads * (kLdKeys + 8) * 2 +
          3 * kLdHeads * 4;
 }
 
@@ -326,8 +326,8 @@ latent_decode_kernel(const __nv_bfloat16* __restrict__ q_latent, const __nv_bflo
   const int crow = kv_rank + rot_dim, srow = crow + 8;     // +16 bytes: ldmatrix rows on different banks
   __nv_bfloat16* ks = reinterpret_cast<__nv_bfloat16*>(ld_raw);   // [2][64][srow]
   __nv_bfloat16* qs = ks + 2 * kLdKeys * srow;                    // [32][srow]
-  float* ss = reinterpret_cast<float*>(qs + kLdHeads * srow);     // [32][kSs]
-  __nv_bfloat16* ps = reinterpret_cast<__nv_bfloat16*>(ss + kLdHeads * kSs);   // [32][kPs]
+  float* ss = reinterpret_cast<float*>(qs + kLdHeads * srow);     // [2][32][kSs]: halves of the dot product
+  __nv_bfloat16* ps = reinterpret_cast<__nv_bfloat16*>(ss + 2 * kLdHeads * kSs);   // [32][kPs]
   float* m_run = reinterpret_cast<float*>(ps + kLdHeads * kPs);
   float* l_run = m_run + kLdHeads;
   float* corr = l_run + kLdHeads;
@@ -345,13 +345,14 @@ latent_decode_kernel(const __nv_bfloat16* __restrict__ q_latent, const __nv_bflo
   const int* bt = block_table + static_cast<long long>(row_seq ? row_seq[t] : t) * max_blocks;
   const int vec = crow >> 3;
   auto load_tile = [&](int i) {
-    // a warp loads eight keys; their cache rows are looked up by eight lanes at once
-    const int mine = base0 + i * kLdKeys + warp * 8 + (lane & 7);
+    // a warp loads four keys; their cache rows are looked up by four lanes at once
+    constexpr int kPer = kLdKeys / kWarps;
+    const int mine = base0 + i * kLdKeys + warp * kPer + (lane & (kPer - 1));
     long long at = -1;
     if (mine >= lo && mine <= pos) at = (static_cast<long long>(bt[mine / page_size]) * page_size + mine % page_size) * crow;
 #pragma unroll
-    for (int k = 0; k < 8; ++k) {
-      __nv_bfloat16* dst = ks + ((i & 1) * kLdKeys + warp * 8 + k) * srow;
+    for (int k = 0; k < kPer; ++k) {
+      __nv_bfloat16* dst = ks + ((i & 1) * kLdKeys + warp * kPer + k) * srow;
       const long long row = __shfl_sync(0xffffffffu, at, k);
       if (row >= 0) {
         const __nv_bfloat16* src = cache + row;
@@ -373,7 +374,8 @@ latent_decode_kernel(const __nv_bfloat16* __restrict__ q_latent, const __nv_bflo
     m_run[threadIdx.x] = -INFINITY;
     l_run[threadIdx.x] = 0.f;
   }
-  float o[4][2][2][4] = {};      // up to four 16-column tiles of the latent x (2 x 16 heads) x (2 x 8 columns)
+  constexpr int kJ = kLdMaxRank / 16 / kWarps;
+  float o[kJ][2][2][4] = {};     // 16-column tiles of the latent x (2 x 16 heads) x (2 x 8 columns)
   for (int i = 0; i < n_tiles; ++i) {
     if (i + 1 < n_tiles) {
       load_tile(i + 1);
@@ -383,13 +385,14 @@ latent_decode_kernel(const __nv_bfloat16* __restrict__ q_latent, const __nv_bflo
     }
     __syncthreads();
     const __nv_bfloat16* kt = ks + (i & 1) * kLdKeys * srow;
-    {   // scores: warp = 16 heads x 16 keys
-      const int m0 = (warp & 1) * 16, n0 = (warp >> 1) * 16;
+    {   // scores: warp = 16 heads x 16 keys x half of the dot product
+      const int m0 = (warp & 1) * 16, n0 = ((warp >> 1) & 3) * 16, half = warp >> 3;
+      const int steps = crow / 16, kb = half ? (steps / 2) * 16 : 0, ke = half ? crow : (steps / 2) * 16;
       float acc[2][4] = {};
       const __nv_bfloat16* kp = kt + (n0 + (lane & 7) + ((lane >> 4) << 3)) * srow + ((lane >> 3) & 1) * 8;
       const __nv_bfloat16* qp = qs + (m0 + (lane & 15)) * srow + (lane >> 4) * 8;
-#pragma unroll 4
-      for (int k = 0; k < crow; k += 16) {
+#pragma unroll 6
+      for (int k = kb; k < ke; k += 16) {
         uint32_t b[4], a[4];
         ldsm_x4(b, kp + k);
         ldsm_x4(a, qp + k);
@@ -399,8 +402,9 @@ latent_decode_kernel(const __nv_bfloat16* __restrict__ q_latent, const __nv_bflo
 #pragma unroll
       for (int g = 0; g < 2; ++g)
 #pragma unroll
-        for (int e = 0; e < 4; ++e)
-          ss[(m0 + (lane >> 2) + (e >> 1) * 8) * kSs + n0 + g * 8 + (lane & 3) * 2 + (e & 1)] = acc[g][e] * scale;
+        for (int e = 0; e < 2; ++e)
+          *reinterpret_cast<float2*>(ss + (half * kLdHeads + m0 + (lane >> 2) + e * 8) * kSs + n0 + g * 8 + (lane & 3) * 2) =
+              make_float2(acc[g][2 * e], acc[g][2 * e + 1]);
     }
     __syncthreads();
     const int k0 = base0 + i * kLdKeys + lane, k1 = k0 + 32;
@@ -410,8 +414,10 @@ latent_decode_kernel(const __nv_bfloat16* __restrict__ q_latent, const __nv_bflo
 #pragma unroll
     for (int x = 0; x < kR; ++x) {
       const int r = warp + x * kWarps;
-      p0[x] = ok0 ? ss[r * kSs + lane] : -INFINITY;
-      p1[x] = ok1 ? ss[r * kSs + lane + 32] : -INFINITY;
+      const float* s0 = ss + r * kSs + lane;
+      const float* s1 = s0 + kLdHeads * kSs;
+      p0[x] = ok0 ? (s0[0] + s1[0]) * scale : -INFINITY;
+      p1[x] = ok1 ? (s0[32] + s1[32]) * scale : -INFINITY;
       m_old[x] = m_run[r];
       m[x] = fmaxf(p0[x], p1[x]);
     }
@@ -451,7 +457,7 @@ latent_decode_kernel(const __nv_bfloat16* __restrict__ q_latent, const __nv_bflo
       for (int k = 0; k < 4; ++k)
         ldsm_x4(pa[m][k], ps + (m * 16 + (lane & 15)) * kPs + k * 16 + (lane >> 4) * 8);
 #pragma unroll
-    for (int j = 0; j < 4; ++j) {
+    for (int j = 0; j < kJ; ++j) {
       const int n0 = (warp + j * kWarps) * 16;
       if (n0 < kv_rank) {
         if (i > 0) {
@@ -483,7 +489,7 @@ latent_decode_kernel(const __nv_bfloat16* __restrict__ q_latent, const __nv_bflo
   }
   const long long span = static_cast<long long>(i_tok) * gridDim.x + blockIdx.x;
 #pragma unroll
-  for (int j = 0; j < 4; ++j) {
+  for (int j = 0; j < kJ; ++j) {
     const int n0 = (warp + j * kWarps) * 16;
     if (n0 < kv_rank) {
 #pragma unroll
@@ -619,9 +625,21 @@ bool latent_decode_ok(const bcg_layer* l) {
          latent_decode_smem(crow) <= 220 * 1024 && absorb_smem(l->dim) <= 200 * 1024 && up_smem(l->kv_rank) <= 200 * 1024;
 }
 
-// Key tiles per span: a CTA per tile while that does not fill the GPU, longer spans (fewer partials) when it
-// more than does.
-static int span_tiles(int n) { return n <= 16 ? 1 : n <= 32 ? 2 : 4; }
+// Key tiles per span, for `rows` (token, head group) pairs of up to `total` tiles each: the choice that needs
+// the fewest tile times on 148 SMs (a span costs about two tiles of start-up).
+static int span_tiles(int rows, int total) {
+  int best = 1;
+  long long best_cost = -1;
+  for (int t = 1; t <= total; ++t) {
+    const long long ctas = static_cast<long long>(rows) * ((total + t - 1) / t);
+    const long long cost = ((ctas + 147) / 148) * (t + 2);
+    if (best_cost < 0 || cost < best_cost) {
+      best_cost = cost;
+      best = t;
+    }
+  }
+  return best;
+}
 
 int latent_decode(const bcg_layer* l, const bcg_stack_ws* ws, const bcg_step_batch* b, int page_size,
                   cudaStream_t st) {
@@ -629,7 +647,8 @@ int latent_decode(const bcg_layer* l, const bcg_stack_ws* ws, const bcg_step_bat
   const int crow = l->kv_rank + l->rot_dim;
   const int q_row = l->q_ld > 0 ? l->q_ld : l->dim + l->rot_dim;
   const int reach = l->window > 0 && l->window < b->max_context ? l->window + kLdKeys : b->max_context;
-  const int tiles = span_tiles(n), spans = ((reach + kLdKeys - 1) / kLdKeys + tiles - 1) / tiles;
+  const int total = (reach + kLdKeys - 1) / kLdKeys, groups = (l->heads + kLdHeads - 1) / kLdHeads;
+  const int tiles = span_tiles(n * groups, total), spans = (total + tiles - 1) / tiles;
   if (n > ws->D_max || n > 65535 || static_cast<long long>(n) * spans * l->heads * l->kv_rank > ws->part_floats) {
     set_last_error("bcg_latent_attention", "single tokens x key spans exceed the decode scratch");
     return BCG_ERR_TOO_LARGE;
@@ -643,7 +662,7 @@ int latent_decode(const bcg_layer* l, const bcg_stack_ws* ws, const bcg_step_bat
                           absorb_smem(l->dim), st, static_cast<const __nv_bfloat16*>(ws->q),
                           static_cast<const __nv_bfloat16*>(l->w_uk), b->single_rows, n, ql, l->heads, l->dim,
                           l->rot_dim, l->kv_rank, q_row));
-  BCG_CUDA_CHECK(launch_k(latent_decode_kernel, dim3(spans, n, (l->heads + kLdHeads - 1) / kLdHeads), dim3(kLdThreads),
+  BCG_CUDA_CHECK(launch_k(latent_decode_kernel, dim3(spans, n, groups), dim3(kLdThreads),
                           latent_decode_smem(crow), st, ql, static_cast<const __nv_bfloat16*>(l->cache),
                           b->single_rows, b->positions, b->row_seq, b->block_table, b->max_blocks, page_size,
                           ws->part_o, ws->part_ml, l->heads, l->kv_rank, l->rot_dim, l->window, tiles, l->scale));
