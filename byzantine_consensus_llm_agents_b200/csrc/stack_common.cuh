@@ -42,15 +42,57 @@ __device__ __forceinline__ float slab_sum(const float* p, int n, long long strid
   }
   return acc;
 }
-__device__ __forceinline__ float4 slab_sum4(const float* p, int n, long long stride) {
-  float4 acc = *reinterpret_cast<const float4*>(p);
-  for (int s = 1; s < n; s += 8) {
-    float4 v[8];
+// V consecutive floats: 4 (vector access, widths that are multiples of 4) or 1 (any width).
+template <int V>
+struct Vec {
+  float x[V];
+  __device__ __forceinline__ float sumsq() const {
+    float s = 0.f;
 #pragma unroll
-    for (int i = 0; i < 8; ++i) v[i] = *reinterpret_cast<const float4*>(p + min(s + i, n - 1) * stride);
+    for (int i = 0; i < V; ++i) s += x[i] * x[i];
+    return s;
+  }
+};
+template <int V>
+__device__ __forceinline__ Vec<V> load_vec(const float* p) {
+  Vec<V> v;
+  if constexpr (V == 4) {
+    const float4 f = *reinterpret_cast<const float4*>(p);
+    v.x[0] = f.x; v.x[1] = f.y; v.x[2] = f.z; v.x[3] = f.w;
+  } else {
+    v.x[0] = *p;
+  }
+  return v;
+}
+template <int V>
+__device__ __forceinline__ Vec<V> load_vec(const __nv_bfloat16* p) {
+  Vec<V> v;
+  if constexpr (V == 4) {
+    const uint2 raw = *reinterpret_cast<const uint2*>(p);
+    v.x[0] = bf16lo(raw.x); v.x[1] = bf16hi(raw.x); v.x[2] = bf16lo(raw.y); v.x[3] = bf16hi(raw.y);
+  } else {
+    v.x[0] = __bfloat162float(*p);
+  }
+  return v;
+}
+template <int V, typename T>
+__device__ __forceinline__ void store_vec(T* p, const Vec<V>& v) {
+  if constexpr (V == 4) store4(p, v.x[0], v.x[1], v.x[2], v.x[3]);
+  else *p = from_f32<T>(v.x[0]);
+}
+template <int V>
+__device__ __forceinline__ Vec<V> slab_sum_vec(const float* p, int n, long long stride) {
+  Vec<V> acc = load_vec<V>(p);
+  for (int s = 1; s < n; s += 8) {
+    Vec<V> v[8];
+#pragma unroll
+    for (int i = 0; i < 8; ++i) v[i] = load_vec<V>(p + min(s + i, n - 1) * stride);
 #pragma unroll
     for (int i = 0; i < 8; ++i)
-      if (s + i < n) { acc.x += v[i].x; acc.y += v[i].y; acc.z += v[i].z; acc.w += v[i].w; }
+      if (s + i < n) {
+#pragma unroll
+        for (int k = 0; k < V; ++k) acc.x[k] += v[i].x[k];
+      }
   }
   return acc;
 }

@@ -15,7 +15,7 @@ constexpr int kRowT = 256;          // threads per CTA
 constexpr int kRowCluster = 8;
 constexpr int kClusterMaxRows = 128;
 
-template <typename T>
+template <typename T, int V>
 __global__ void __launch_bounds__(kRowT)
 embed_norm_kernel(const int* __restrict__ ids, const __nv_bfloat16* __restrict__ embed, const float* __restrict__ w,
                   float* __restrict__ residual, T* __restrict__ xn, int d, float eps) {
@@ -23,42 +23,42 @@ embed_norm_kernel(const int* __restrict__ ids, const __nv_bfloat16* __restrict__
   pdl_launch_dependents();
   pdl_wait();
   const long long t = blockIdx.x, row = ids[t];
-  const int nvec = d >> 2;
   float ss[1] = {0.f};
-  for (int v = threadIdx.x; v < nvec; v += kRowT) {
-    const uint2 raw = *reinterpret_cast<const uint2*>(embed + row * d + v * 4);
-    const float4 x = make_float4(bf16lo(raw.x), bf16hi(raw.x), bf16lo(raw.y), bf16hi(raw.y));
-    *reinterpret_cast<float4*>(residual + t * d + v * 4) = x;
-    ss[0] += x.x * x.x + x.y * x.y + x.z * x.z + x.w * x.w;
+  for (int v = threadIdx.x * V; v < d; v += kRowT * V) {
+    const Vec<V> x = load_vec<V>(embed + row * d + v);
+    store_vec<V>(residual + t * d + v, x);
+    ss[0] += x.sumsq();
   }
   row_sum<kRowT, 1, 1>(sh, ss, 0);
   const float inv = rsqrtf(ss[0] / static_cast<float>(d) + eps);
-  for (int v = threadIdx.x; v < nvec; v += kRowT) {
-    const uint2 raw = *reinterpret_cast<const uint2*>(embed + row * d + v * 4);
-    const float4 ww = *reinterpret_cast<const float4*>(w + v * 4);
-    store4(xn + t * d + v * 4, bf16lo(raw.x) * inv * ww.x, bf16hi(raw.x) * inv * ww.y, bf16lo(raw.y) * inv * ww.z,
-           bf16hi(raw.y) * inv * ww.w);
+  for (int v = threadIdx.x * V; v < d; v += kRowT * V) {
+    Vec<V> x = load_vec<V>(embed + row * d + v);
+    const Vec<V> ww = load_vec<V>(w + v);
+#pragma unroll
+    for (int k = 0; k < V; ++k) x.x[k] *= inv * ww.x[k];
+    store_vec<V>(xn + t * d + v, x);
   }
 }
 
-template <typename T, int CL>
+template <typename T, int V, int CL>
 __global__ void __launch_bounds__(kRowT)
 sandwich_norm_kernel(float* __restrict__ residual, const float* __restrict__ delta, int n_partials,
                      long long partial_stride, const float* __restrict__ w_post, const float* __restrict__ w_next,
                      T* __restrict__ xn, int d, float eps) {
-  extern __shared__ float4 stage[];   // this CTA's part of the row
+  extern __shared__ float4 stage_raw[];   // this CTA's part of the row
+  float* stage = reinterpret_cast<float*>(stage_raw);
   __shared__ RowSum<kRowT, CL, 1> sh;
   pdl_launch_dependents();
   pdl_wait();
   const long long t = CL > 1 ? blockIdx.y : blockIdx.x;
-  const int nvec = d >> 2, per = (nvec + CL - 1) / CL;
-  const int v0 = (CL > 1 ? static_cast<int>(blockIdx.x) : 0) * per, v1 = min(nvec, v0 + per);
+  const int per = (d / V + CL - 1) / CL * V;
+  const int v0 = (CL > 1 ? static_cast<int>(blockIdx.x) : 0) * per, v1 = min(d, v0 + per);
   const float inv_d = 1.0f / static_cast<float>(d);
   float ss[1] = {0.f};
-  for (int v = v0 + threadIdx.x; v < v1; v += kRowT) {
-    const float4 y = slab_sum4(delta + t * d + v * 4, n_partials, partial_stride);
-    stage[v - v0] = y;
-    ss[0] += y.x * y.x + y.y * y.y + y.z * y.z + y.w * y.w;
+  for (int v = v0 + threadIdx.x * V; v < v1; v += kRowT * V) {
+    const Vec<V> y = slab_sum_vec<V>(delta + t * d + v, n_partials, partial_stride);
+    store_vec<V>(stage + v - v0, y);
+    ss[0] += y.sumsq();
   }
   float inv = 1.0f;
   if (w_post) {
@@ -66,31 +66,36 @@ sandwich_norm_kernel(float* __restrict__ residual, const float* __restrict__ del
     inv = rsqrtf(ss[0] * inv_d + eps);
   }
   ss[0] = 0.f;
-  for (int v = v0 + threadIdx.x; v < v1; v += kRowT) {
-    float4 y = stage[v - v0];
+  for (int v = v0 + threadIdx.x * V; v < v1; v += kRowT * V) {
+    const Vec<V> y = load_vec<V>(stage + v - v0);
+    Vec<V> x = load_vec<V>(residual + t * d + v);
     if (w_post) {
-      const float4 ww = *reinterpret_cast<const float4*>(w_post + v * 4);
-      y.x *= inv * ww.x; y.y *= inv * ww.y; y.z *= inv * ww.z; y.w *= inv * ww.w;
+      const Vec<V> ww = load_vec<V>(w_post + v);
+#pragma unroll
+      for (int k = 0; k < V; ++k) x.x[k] = fmaf(y.x[k], inv * ww.x[k], x.x[k]);
+    } else {
+#pragma unroll
+      for (int k = 0; k < V; ++k) x.x[k] += y.x[k];
     }
-    float4 x = *reinterpret_cast<const float4*>(residual + t * d + v * 4);
-    x.x += y.x; x.y += y.y; x.z += y.z; x.w += y.w;
-    *reinterpret_cast<float4*>(residual + t * d + v * 4) = x;
-    stage[v - v0] = x;
-    ss[0] += x.x * x.x + x.y * x.y + x.z * x.z + x.w * x.w;
+    store_vec<V>(residual + t * d + v, x);
+    store_vec<V>(stage + v - v0, x);
+    ss[0] += x.sumsq();
   }
   if (w_next) {
     row_sum<kRowT, CL, 1>(sh, ss, 1);
     const float inv2 = rsqrtf(ss[0] * inv_d + eps);
-    for (int v = v0 + threadIdx.x; v < v1; v += kRowT) {
-      const float4 x = stage[v - v0];
-      const float4 ww = *reinterpret_cast<const float4*>(w_next + v * 4);
-      store4(xn + t * d + v * 4, x.x * inv2 * ww.x, x.y * inv2 * ww.y, x.z * inv2 * ww.z, x.w * inv2 * ww.w);
+    for (int v = v0 + threadIdx.x * V; v < v1; v += kRowT * V) {
+      Vec<V> x = load_vec<V>(stage + v - v0);
+      const Vec<V> ww = load_vec<V>(w_next + v);
+#pragma unroll
+      for (int k = 0; k < V; ++k) x.x[k] *= inv2 * ww.x[k];
+      store_vec<V>(xn + t * d + v, x);
     }
   }
   row_sum_exit<CL>();
 }
 
-template <typename T>
+template <typename T, int V>
 __global__ void __launch_bounds__(kRowT)
 rows_norm_kernel(const float* __restrict__ residual, const int* __restrict__ rows, const float* __restrict__ w,
                  T* __restrict__ xn, int d, float eps) {
@@ -98,122 +103,143 @@ rows_norm_kernel(const float* __restrict__ residual, const int* __restrict__ row
   pdl_launch_dependents();
   pdl_wait();
   const long long t = blockIdx.x, src = rows[t];
-  const int nvec = d >> 2;
   float ss[1] = {0.f};
-  for (int v = threadIdx.x; v < nvec; v += kRowT) {
-    const float4 x = *reinterpret_cast<const float4*>(residual + src * d + v * 4);
-    ss[0] += x.x * x.x + x.y * x.y + x.z * x.z + x.w * x.w;
-  }
+  for (int v = threadIdx.x * V; v < d; v += kRowT * V) ss[0] += load_vec<V>(residual + src * d + v).sumsq();
   row_sum<kRowT, 1, 1>(sh, ss, 0);
   const float inv = rsqrtf(ss[0] / static_cast<float>(d) + eps);
-  for (int v = threadIdx.x; v < nvec; v += kRowT) {
-    const float4 x = *reinterpret_cast<const float4*>(residual + src * d + v * 4);
-    const float4 ww = *reinterpret_cast<const float4*>(w + v * 4);
-    store4(xn + t * d + v * 4, x.x * inv * ww.x, x.y * inv * ww.y, x.z * inv * ww.z, x.w * inv * ww.w);
+  for (int v = threadIdx.x * V; v < d; v += kRowT * V) {
+    Vec<V> x = load_vec<V>(residual + src * d + v);
+    const Vec<V> ww = load_vec<V>(w + v);
+#pragma unroll
+    for (int k = 0; k < V; ++k) x.x[k] *= inv * ww.x[k];
+    store_vec<V>(xn + t * d + v, x);
   }
 }
 
-template <typename T, int CL>
+template <typename T, int V, int CL>
 __global__ void __launch_bounds__(kRowT)
 poly_norm_kernel(const float* __restrict__ z, int n_partials, long long partial_stride,
                  const float* __restrict__ coef, T* __restrict__ out, int ff, float eps) {
-  extern __shared__ float4 stage[];
+  extern __shared__ float4 stage_raw[];
+  float* stage = reinterpret_cast<float*>(stage_raw);
   __shared__ RowSum<kRowT, CL, 3> sh;
   pdl_launch_dependents();
   pdl_wait();
   const long long t = CL > 1 ? blockIdx.y : blockIdx.x;
-  const int nvec = ff >> 2, per = (nvec + CL - 1) / CL;
-  const int v0 = (CL > 1 ? static_cast<int>(blockIdx.x) : 0) * per, v1 = min(nvec, v0 + per);
+  const int per = (ff / V + CL - 1) / CL * V;
+  const int v0 = (CL > 1 ? static_cast<int>(blockIdx.x) : 0) * per, v1 = min(ff, v0 + per);
   float s[3] = {0.f, 0.f, 0.f};   // sums of z^2, z^4, z^6
-  auto add = [&](float x) {
-    const float x2 = x * x, x4 = x2 * x2;
-    s[0] += x2;
-    s[1] += x4;
-    s[2] = fmaf(x4, x2, s[2]);
-  };
-  for (int v = v0 + threadIdx.x; v < v1; v += kRowT) {
-    const float4 x = slab_sum4(z + t * ff + v * 4, n_partials, partial_stride);
-    stage[v - v0] = x;
-    add(x.x); add(x.y); add(x.z); add(x.w);
+  for (int v = v0 + threadIdx.x * V; v < v1; v += kRowT * V) {
+    const Vec<V> x = slab_sum_vec<V>(z + t * ff + v, n_partials, partial_stride);
+    store_vec<V>(stage + v - v0, x);
+#pragma unroll
+    for (int k = 0; k < V; ++k) {
+      const float x2 = x.x[k] * x.x[k], x4 = x2 * x2;
+      s[0] += x2;
+      s[1] += x4;
+      s[2] = fmaf(x4, x2, s[2]);
+    }
   }
   row_sum<kRowT, CL, 3>(sh, s, 0);
   const float inv_f = 1.0f / static_cast<float>(ff);
   const float a = coef[0] * rsqrtf(s[0] * inv_f + eps), b = coef[1] * rsqrtf(s[1] * inv_f + eps),
               c = coef[2] * rsqrtf(s[2] * inv_f + eps), e = coef[3];
-  auto act = [&](float x) { return fmaf(x, fmaf(x, fmaf(x, c, b), a), e); };
-  for (int v = v0 + threadIdx.x; v < v1; v += kRowT) {
-    const float4 x = stage[v - v0];
-    store4(out + t * ff + v * 4, act(x.x), act(x.y), act(x.z), act(x.w));
+  for (int v = v0 + threadIdx.x * V; v < v1; v += kRowT * V) {
+    Vec<V> x = load_vec<V>(stage + v - v0);
+#pragma unroll
+    for (int k = 0; k < V; ++k) x.x[k] = fmaf(x.x[k], fmaf(x.x[k], fmaf(x.x[k], c, b), a), e);
+    store_vec<V>(out + t * ff + v, x);
   }
   row_sum_exit<CL>();
 }
 
-int embed_norm(const int* ids, const void* embed, const float* w, float* residual, void* xn, int act_dtype, int T,
-               int d, float eps, cudaStream_t st) {
-  const auto* e = static_cast<const __nv_bfloat16*>(embed);
-  if (act_dtype == BCG_DT_F32)
-    BCG_CUDA_CHECK(launch_k(embed_norm_kernel<float>, dim3(T), dim3(kRowT), 0, st, ids, e, w, residual,
-                            static_cast<float*>(xn), d, eps));
-  else
-    BCG_CUDA_CHECK(launch_k(embed_norm_kernel<__nv_bfloat16>, dim3(T), dim3(kRowT), 0, st, ids, e, w, residual,
-                            static_cast<__nv_bfloat16*>(xn), d, eps));
-  return BCG_OK;
-}
-
-int rows_norm(const float* residual, const int* rows, const float* w, void* xn, int act_dtype, int n, int d,
-              float eps, cudaStream_t st) {
-  if (act_dtype == BCG_DT_F32)
-    BCG_CUDA_CHECK(launch_k(rows_norm_kernel<float>, dim3(n), dim3(kRowT), 0, st, residual, rows, w,
-                            static_cast<float*>(xn), d, eps));
-  else
-    BCG_CUDA_CHECK(launch_k(rows_norm_kernel<__nv_bfloat16>, dim3(n), dim3(kRowT), 0, st, residual, rows, w,
-                            static_cast<__nv_bfloat16*>(xn), d, eps));
-  return BCG_OK;
-}
-
-// One row per cluster (decode) or per CTA; KERNEL is a template over <T, CL>.
-#define BCG_LAUNCH_ROWS(KERNEL, T_ROWS, WIDTH, TYPE, ...)                                                           \
-  do {                                                                                                              \
-    if ((T_ROWS) <= kClusterMaxRows && (WIDTH) >= 1024) {                                                           \
-      const size_t _sm = static_cast<size_t>(((WIDTH) / 4 + kRowCluster - 1) / kRowCluster) * 16;                   \
-      BCG_CUDA_CHECK(launch_cluster(KERNEL<TYPE, kRowCluster>, dim3(kRowCluster, T_ROWS), dim3(kRowT), kRowCluster, \
-                                    _sm, st, __VA_ARGS__));                                                         \
-    } else {                                                                                                        \
-      const size_t _sm = static_cast<size_t>(WIDTH) * 4;                                                            \
-      BCG_TRY(ensure_dynamic_smem(reinterpret_cast<const void*>(KERNEL<TYPE, 1>), 200 * 1024));                     \
-      BCG_CUDA_CHECK(launch_k(KERNEL<TYPE, 1>, dim3(T_ROWS), dim3(kRowT), _sm, st, __VA_ARGS__));                   \
-    }                                                                                                               \
+// calls FN<type, vector width>(...) for the activation dtype and the row width
+#define BCG_BY_TYPE(FN, WIDTH, DTYPE, ...)                                   \
+  do {                                                                       \
+    if ((DTYPE) == BCG_DT_F32)                                               \
+      return (WIDTH) % 4 ? FN<float, 1>(__VA_ARGS__) : FN<float, 4>(__VA_ARGS__); \
+    return (WIDTH) % 4 ? FN<__nv_bfloat16, 1>(__VA_ARGS__) : FN<__nv_bfloat16, 4>(__VA_ARGS__); \
   } while (0)
 
+template <typename T, int V>
+static int embed_t(const int* ids, const void* embed, const float* w, float* residual, void* xn, int T_rows, int d,
+                   float eps, cudaStream_t st) {
+  BCG_CUDA_CHECK(launch_k(embed_norm_kernel<T, V>, dim3(T_rows), dim3(kRowT), 0, st, ids,
+                          static_cast<const __nv_bfloat16*>(embed), w, residual, static_cast<T*>(xn), d, eps));
+  return BCG_OK;
+}
+int embed_norm(const int* ids, const void* embed, const float* w, float* residual, void* xn, int act_dtype, int T,
+               int d, float eps, cudaStream_t st) {
+  BCG_BY_TYPE(embed_t, d, act_dtype, ids, embed, w, residual, xn, T, d, eps, st);
+}
+
+template <typename T, int V>
+static int rows_t(const float* residual, const int* rows, const float* w, void* xn, int n, int d, float eps,
+                  cudaStream_t st) {
+  BCG_CUDA_CHECK(launch_k(rows_norm_kernel<T, V>, dim3(n), dim3(kRowT), 0, st, residual, rows, w, static_cast<T*>(xn),
+                          d, eps));
+  return BCG_OK;
+}
+int rows_norm(const float* residual, const int* rows, const float* w, void* xn, int act_dtype, int n, int d,
+              float eps, cudaStream_t st) {
+  BCG_BY_TYPE(rows_t, d, act_dtype, residual, rows, w, xn, n, d, eps, st);
+}
+
+// One row per cluster (decode) or per CTA; shared memory stages a CTA's part of the row.
+static bool row_cluster(int rows, int width) { return rows <= kClusterMaxRows && width >= 1024; }
+static size_t row_stage(bool cluster, int width, int v) {
+  return static_cast<size_t>(cluster ? (width / v + kRowCluster - 1) / kRowCluster * v : width) * 4;
+}
+
+template <typename T, int V>
+static int sandwich_t(float* residual, const float* delta, int n_partials, long long stride, const float* w_post,
+                      const float* w_next, void* xn, int T_rows, int d, float eps, cudaStream_t st) {
+  const bool cl = row_cluster(T_rows, d);
+  const size_t sm = row_stage(cl, d, V);
+  T* x = static_cast<T*>(xn);
+  if (cl) {
+    BCG_CUDA_CHECK(launch_cluster(sandwich_norm_kernel<T, V, kRowCluster>, dim3(kRowCluster, T_rows), dim3(kRowT),
+                                  kRowCluster, sm, st, residual, delta, n_partials, stride, w_post, w_next, x, d, eps));
+  } else {
+    BCG_TRY(ensure_dynamic_smem(reinterpret_cast<const void*>(sandwich_norm_kernel<T, V, 1>), 200 * 1024));
+    BCG_CUDA_CHECK(launch_k(sandwich_norm_kernel<T, V, 1>, dim3(T_rows), dim3(kRowT), sm, st, residual, delta, n_partials,
+                            stride, w_post, w_next, x, d, eps));
+  }
+  return BCG_OK;
+}
 int sandwich_norm(float* residual, const float* delta, int n_partials, long long partial_stride,
                   const float* w_post, const float* w_next, void* xn, int act_dtype, int T, int d, float eps,
                   cudaStream_t st) {
-  if (!residual || !delta || T <= 0 || d <= 0 || (d % 4) || d > 51200 || n_partials < 1 || (w_next && !xn)) {
-    set_last_error("bcg_sandwich_norm", "bad argument (d must be a multiple of 4, <= 51200)");
+  if (!residual || !delta || T <= 0 || d <= 0 || d > 51200 || n_partials < 1 || (w_next && !xn)) {
+    set_last_error("bcg_sandwich_norm", "bad argument (d <= 51200)");
     return BCG_ERR_ARG;
   }
-  if (act_dtype == BCG_DT_F32)
-    BCG_LAUNCH_ROWS(sandwich_norm_kernel, T, d, float, residual, delta, n_partials, partial_stride, w_post, w_next,
-                    static_cast<float*>(xn), d, eps);
-  else
-    BCG_LAUNCH_ROWS(sandwich_norm_kernel, T, d, __nv_bfloat16, residual, delta, n_partials, partial_stride, w_post,
-                    w_next, static_cast<__nv_bfloat16*>(xn), d, eps);
-  return BCG_OK;
+  BCG_BY_TYPE(sandwich_t, d, act_dtype, residual, delta, n_partials, partial_stride, w_post, w_next, xn, T, d, eps, st);
 }
 
+template <typename T, int V>
+static int poly_t(const float* z, int n_partials, long long stride, const float* coef, void* out, int T_rows, int ff,
+                  float eps, cudaStream_t st) {
+  const bool cl = row_cluster(T_rows, ff);
+  const size_t sm = row_stage(cl, ff, V);
+  T* o = static_cast<T*>(out);
+  if (cl) {
+    BCG_CUDA_CHECK(launch_cluster(poly_norm_kernel<T, V, kRowCluster>, dim3(kRowCluster, T_rows), dim3(kRowT), kRowCluster,
+                                  sm, st, z, n_partials, stride, coef, o, ff, eps));
+  } else {
+    BCG_TRY(ensure_dynamic_smem(reinterpret_cast<const void*>(poly_norm_kernel<T, V, 1>), 200 * 1024));
+    BCG_CUDA_CHECK(launch_k(poly_norm_kernel<T, V, 1>, dim3(T_rows), dim3(kRowT), sm, st, z, n_partials, stride, coef, o,
+                            ff, eps));
+  }
+  return BCG_OK;
+}
 int poly_norm(const float* z, int n_partials, long long partial_stride, const float* coef, void* out, int act_dtype,
               int T, int ff, float eps, cudaStream_t st) {
-  if (!z || !coef || !out || T <= 0 || ff <= 0 || (ff % 4) || ff > 51200 || n_partials < 1) {
-    set_last_error("bcg_poly_norm", "bad argument (ff must be a multiple of 4, <= 51200)");
+  if (!z || !coef || !out || T <= 0 || ff <= 0 || ff > 51200 || n_partials < 1) {
+    set_last_error("bcg_poly_norm", "bad argument (ff <= 51200)");
     return BCG_ERR_ARG;
   }
-  if (act_dtype == BCG_DT_F32)
-    BCG_LAUNCH_ROWS(poly_norm_kernel, T, ff, float, z, n_partials, partial_stride, coef, static_cast<float*>(out), ff,
-                    eps);
-  else
-    BCG_LAUNCH_ROWS(poly_norm_kernel, T, ff, __nv_bfloat16, z, n_partials, partial_stride, coef,
-                    static_cast<__nv_bfloat16*>(out), ff, eps);
-  return BCG_OK;
+  BCG_BY_TYPE(poly_t, ff, act_dtype, z, n_partials, partial_stride, coef, out, T, ff, eps, st);
 }
 
 }  // namespace bcg

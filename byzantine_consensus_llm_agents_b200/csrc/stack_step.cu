@@ -7,10 +7,10 @@
 namespace bcg {
 
 static int check_stack(const bcg_stack* m, const bcg_stack_ws* ws) {
-  if (!m || !ws || m->n_layers <= 0 || m->d_model <= 0 || (m->d_model % 4) || !m->embed || !m->lm_head ||
+  if (!m || !ws || m->n_layers <= 0 || m->d_model <= 0 || !m->embed || !m->lm_head ||
       !m->final_norm || !m->layers || !ws->residual || !ws->xn || !ws->proj || !ws->logits ||
       (m->act_dtype != BCG_DT_BF16 && m->act_dtype != BCG_DT_F32) || m->page_size <= 0) {
-    set_last_error("bcg_stack", "incomplete model / workspace description (d_model must be a multiple of 4)");
+    set_last_error("bcg_stack", "incomplete model / workspace description");
     return BCG_ERR_ARG;
   }
   return BCG_OK;

@@ -25,7 +25,7 @@ from .tokenizer import get_tokenizer
 # name -> (width, dense ff, stack ff, layers): widths and feed-forward sizes of 1-2B / 8B class models; the stack's ff
 # makes its layers (no gate matrix, five mixer projections) the dense layers' size.  Fewer layers than a whole
 # model (layers repeat; throughput per layer is what is compared), the same vocabulary.
-SIZES = {"2k": (2048, 6144, 8192, 8), "4k": (4096, 12288, 18432, 8)}
+SIZES = {"2k": (2048, 6144, 7424, 8), "4k": (4096, 12288, 14592, 8)}
 VOCAB, CTX, PROMPT, PROMPTS = 32768, 1600, 1536, 8
 FP32_FMA = 148 * 128 * 1.965e9       # nominal
 

@@ -77,8 +77,8 @@ PRESETS = {
     "mistral-22b": ModelConfig("mistral-22b", 56, 6144, 48, 8, 16384, 32768, rms_eps=1e-5, qk_norm=False,
                                family="mistral"),
     # layer stacks (stack.py) at the widths of the dense presets beside them
-    "bekopel-1b": stack.bekopel_preset("bekopel-1b", 16, 2048, 8192, 151936, heads=16),
-    "bekopel-8b": stack.bekopel_preset("bekopel-8b", 36, 4096, 18432, 151936),
+    "bekopel-1b": stack.bekopel_preset("bekopel-1b", 16, 2048, 7424, 151936, heads=16),
+    "bekopel-8b": stack.bekopel_preset("bekopel-8b", 36, 4096, 14592, 151936),
 }
 
 _HF_NAMES = {

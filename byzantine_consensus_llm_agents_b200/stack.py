@@ -137,8 +137,6 @@ class StackConfig:
     max_pos: int = 131072
 
     def __post_init__(self):
-        if self.d_model % 4 or any(l.mlp and l.mlp.ff % 4 for l in self.layers):
-            raise ValueError(f"{self.name}: width and feed-forward sizes must be multiples of 4")
         if self.act_dtype not in ("bfloat16", "float32"):
             raise ValueError(f"act_dtype {self.act_dtype!r}")
         for i, l in enumerate(self.layers):

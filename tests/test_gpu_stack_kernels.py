@@ -44,7 +44,8 @@ def test_gemm_any(dtype, M, N, K):
 
 
 @pytest.mark.parametrize("dtype", DT)
-@pytest.mark.parametrize("T,d,parts", [(1, 4, 1), (3, 80, 2), (5, 2048, 5), (128, 1028, 1), (200, 1536, 1), (2, 16384, 9)])
+@pytest.mark.parametrize("T,d,parts", [(1, 4, 1), (3, 80, 2), (5, 2048, 5), (128, 1028, 1), (200, 1536, 1), (2, 16384, 9),
+                                        (3, 77, 2), (2, 1501, 3)])
 def test_sandwich_norm(dtype, T, d, parts):
     code, td, tol = DT[dtype]
     g = gen(T + d)
@@ -64,7 +65,7 @@ def test_sandwich_norm(dtype, T, d, parts):
 
 
 @pytest.mark.parametrize("dtype", DT)
-@pytest.mark.parametrize("T,ff,parts", [(1, 8, 1), (3, 96, 3), (4, 4096, 2), (150, 1280, 1)])
+@pytest.mark.parametrize("T,ff,parts", [(1, 8, 1), (3, 96, 3), (4, 4096, 2), (150, 1280, 1), (3, 99, 2), (5, 1155, 2)])
 def test_poly_norm(dtype, T, ff, parts):
     code, td, tol = DT[dtype]
     g = gen(T + ff)

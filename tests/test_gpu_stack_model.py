@@ -29,6 +29,9 @@ CONFIGS = {
                          SM.attn(8, 32, 32, 32, 96, 70, base=1e6), SM.attn(2, 80, 16, 96, 112, 16, kv_from=1)], width=192, vocab=320),
     "attention-only": SM.config([SM.attn(window=1), SM.attn(2, 32, 32, 40, 32, 100)], width=64, vocab=101),
     "delta-only": SM.config([SM.delta(1, 8, ff=None), SM.delta(2, 128)], width=100, vocab=64, eps=1e-3),
+    # sizes no vector load or tensor-core tile likes
+    "odd": SM.config([SM.delta(3, 7, ff=45), SM.attn(3, 9, 6, 11, 13, 19, ff=51), SM.attn(5, 10, 6, 7, 13, 40, kv_from=1, ff=None)],
+                     width=61, vocab=83),
     "one-each": SM.config([SM.attn(1, 8, 8, 8, 16, 5, ff=20)], width=36, vocab=36),
 }
 

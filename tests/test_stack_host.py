@@ -35,7 +35,7 @@ def test_config_comes_from_the_directory(tmp_path):
     (lambda c: c["layers"][2]["mixer"].update(kv_from=0), "cannot read"),
     (lambda c: c["layers"][2]["mixer"].update(kv_rank=64), "cannot read"),
     (lambda c: c["layers"][1]["mixer"]["rot"].update(dims=10), "rotary"),
-    (lambda c: c.update(width=81), "multiples of 4"),
+    (lambda c: c["layers"][3]["mixer"].update(dim=300), "256 channels"),
 ])
 def test_bad_configurations_are_refused(spoil, words):
     import copy
