@@ -128,11 +128,6 @@ int model_decode(const bcg_model* m, const bcg_workspace* ws, const int* ids, co
     return BCG_ERR_TOO_LARGE;
   }
   const int gf = flags & BCG_GEMM_PDL;
-  // profiling aids (tools/step_ablation.py): leave one kernel family out of the step to read its
-  // in-pipeline cost off the step time.  Results are garbage with any of these set.
-  const bool skip_attn = flags & 0x100, skip_norm = flags & 0x200, skip_rope = flags & 0x400;
-  const bool skip_qkv = flags & 0x1000, skip_o = flags & 0x2000, skip_gu = flags & 0x4000,
-             skip_dn = flags & 0x8000, skip_lm = flags & 0x10000;
   struct FlagScope {
     int saved;
     explicit FlagScope(int f) : saved(launch_flags()) { launch_flags() = f; }
@@ -140,7 +135,7 @@ int model_decode(const bcg_model* m, const bcg_workspace* ws, const int* ids, co
   } scope(gf);
   float* P = ws->partials;
   // qk-norm / RoPE / KV-write folded into decode attention (bcg_decode_attn_paged_qkv)
-  const bool fuse_rope = (flags & BCG_STEP_FUSED_ROPE) && !skip_rope;
+  const bool fuse_rope = (flags & BCG_STEP_FUSED_ROPE);
   // Norm fusion (single GPU, opt-in with BCG_STEP_FUSED_NORM): the o / down projections finish the
   // residual add and leave bf16(residual * w) plus per-tile sums of squares; the projection that
   // follows applies 1/RMS in its epilogue.  No add_rmsnorm kernel runs after layer 0's embedding
@@ -148,11 +143,11 @@ int model_decode(const bcg_model* m, const bcg_workspace* ws, const int* ids, co
   // 5.93 ms per step): the fence + counter + reload chain at the end of the o / down GEMMs runs
   // while HBM is saturated and costs 7-10 us, the stand-alone norm 4-5 us on an idle memory system.
   const bool nf = tp == 1 && ws->row_sumsq && ws->tile_counters && (d % 128) == 0 && s_o <= 16 &&
-                  s_dn <= 16 && (flags & BCG_STEP_FUSED_NORM) && !skip_norm;
+                  s_dn <= 16 && (flags & BCG_STEP_FUSED_NORM);
   // Deferred norm (single GPU, opt-in with BCG_STEP_DEFERRED_NORM): bcg_add_norm_stats finishes the
   // residual and writes bf16(residual * w) + 8 segment sums per row; the projection that follows
   // applies 1/RMS in its epilogue, so the row-wide reduction leaves the critical path.
-  const bool dn = !nf && tp == 1 && ws->row_sumsq && B <= 128 && (flags & BCG_STEP_DEFERRED_NORM) && !skip_norm;
+  const bool dn = !nf && tp == 1 && ws->row_sumsq && B <= 128 && (flags & BCG_STEP_DEFERRED_NORM);
   const bool scaled = nf || dn || fused;   // the consuming projection applies 1/RMS in its epilogue
   const int n_tiles_d = (dn || fused) ? 8 : d / 128;
   const int table_floats = (d / 128 > 8 ? d / 128 : 8) * 128;
@@ -186,17 +181,16 @@ int model_decode(const bcg_model* m, const bcg_workspace* ws, const int* ids, co
     } else if (fused) {
       BCG_TRY(tp_add_norm_stats(ws->residual, P, s_dn, static_cast<long long>(B) * d, m->ln1[l], ws->xn,
                                 sumsq_mlp, 1, ws->tp_region_floats, B, d, st));
-    } else if (!skip_norm) {
+    } else {
       BCG_TRY(add_rmsnorm(ws->residual, P, 1, s_dn, static_cast<long long>(B) * d, m->ln1[l], ws->xn,
                           nullptr, B, d, m->rms_eps, st));
     }
-    if (!skip_qkv) {
+    {
       const bcg_gemm_fusion f = consumer(sumsq_mlp);
       BCG_TRY(gemm_bf16_tn_fused(ws->xn, m->w_qkv[l], P, B, qkv_dim, d, d, d, qkv_dim, BCG_EPI_F32, s_qkv,
                                  gf, (scaled && l > 0) ? &f : nullptr, st));
     }
     if (fuse_rope) {
-      if (!skip_attn)
       BCG_TRY(decode_attn_paged_qkv(P, s_qkv, static_cast<long long>(B) * qkv_dim, qkv_dim,
                                     m->q_norm ? static_cast<const float*>(m->q_norm[l]) : nullptr,
                                     m->k_norm ? static_cast<const float*>(m->k_norm[l]) : nullptr,
@@ -205,12 +199,10 @@ int model_decode(const bcg_model* m, const bcg_workspace* ws, const int* ids, co
                                     ws->attn_scratch_o, ws->attn_scratch_ml, ws->attn_counters, B, hq, hkv,
                                     m->page_size, ws->max_splits, scale, st));
     } else {
-    if (!skip_rope)
     BCG_TRY(qknorm_rope_kvwrite(P, 1, s_qkv, static_cast<long long>(B) * qkv_dim, qkv_dim,
                                 m->q_norm ? m->q_norm[l] : nullptr,
                                 m->k_norm ? m->k_norm[l] : nullptr, m->cos_sin, positions, slot_map,
                                 ws->q, m->kv_cache[l], B, hq, hkv, m->page_size, m->rms_eps, st));
-    if (!skip_attn)
     BCG_TRY(decode_attn_paged(ws->q, m->kv_cache[l], block_table, max_blocks, seq_lens, ws->attn,
                               ws->attn_scratch_o, ws->attn_scratch_ml, ws->attn_counters, B, hq, hkv,
                               m->page_size, ws->max_splits, scale, st));
@@ -222,11 +214,9 @@ int model_decode(const bcg_model* m, const bcg_workspace* ws, const int* ids, co
                                 sumsq_attn, 0, ws->tp_region_floats, B, d, st));
     } else if (nf) {
       const bcg_gemm_fusion f = producer(sumsq_attn, m->ln2[l], ws->xn);
-      if (!skip_o)
       BCG_TRY(gemm_bf16_tn_fused(ws->attn, m->w_o[l], P, B, d, hq * 128, hq * 128, hq * 128, d, BCG_EPI_F32,
                                  s_o, gf, &f, st));
     } else {
-    if (!skip_o)
     BCG_TRY(gemm_bf16_tn(ws->attn, m->w_o[l], P, B, d, hq * 128, hq * 128, hq * 128, d, BCG_EPI_F32,
                          s_o, gf, st));
     // row-parallel projection: sum the split-K slabs over the ranks in place (slab s of every rank
@@ -235,13 +225,13 @@ int model_decode(const bcg_model* m, const bcg_workspace* ws, const int* ids, co
     if (dn) {
       BCG_TRY(add_norm_stats(ws->residual, P, 1, s_o, static_cast<long long>(B) * d, m->ln2[l], ws->xn,
                              sumsq_attn, B, d, st));
-    } else if (!skip_norm)
-    BCG_TRY(add_rmsnorm(ws->residual, P, 1, s_o, static_cast<long long>(B) * d, m->ln2[l], ws->xn,
-                        nullptr, B, d, m->rms_eps, st));
+    } else {
+      BCG_TRY(add_rmsnorm(ws->residual, P, 1, s_o, static_cast<long long>(B) * d, m->ln2[l], ws->xn,
+                          nullptr, B, d, m->rms_eps, st));
+    }
     }
     const bcg_gemm_fusion f_gu = consumer(sumsq_attn);
-    if (skip_gu) {
-    } else if (s_gu == 1) {
+    if (s_gu == 1) {
       BCG_TRY(gemm_bf16_tn_fused(ws->xn, m->w_gate_up[l], ws->act, B, 2 * ff, d, d, d, ff, BCG_EPI_SWIGLU, 1,
                                  gf, scaled ? &f_gu : nullptr, st));
     } else {
@@ -255,10 +245,8 @@ int model_decode(const bcg_model* m, const bcg_workspace* ws, const int* ids, co
       const bool last = (l + 1 == m->n_layers);
       const bcg_gemm_fusion f = producer(sumsq_mlp, last ? m->final_norm : m->ln1[l + 1],
                                          last ? ws->xn_last : ws->xn);
-      if (!skip_dn)
       BCG_TRY(gemm_bf16_tn_fused(ws->act, m->w_down[l], P, B, d, ff, ff, ff, d, BCG_EPI_F32, s_dn, gf, &f, st));
     } else {
-      if (!skip_dn)
       BCG_TRY(gemm_bf16_tn(ws->act, m->w_down[l], P, B, d, ff, ff, ff, d, BCG_EPI_F32, s_dn, gf, st));
       if (tp > 1) BCG_TRY(tp_all_reduce_f32(P, static_cast<long long>(s_dn) * B * d, st));
     }
@@ -275,7 +263,7 @@ int model_decode(const bcg_model* m, const bcg_workspace* ws, const int* ids, co
     BCG_TRY(add_rmsnorm(ws->residual, P, 1, s_dn, static_cast<long long>(B) * d, m->final_norm,
                         ws->xn_last, nullptr, B, d, m->rms_eps, st));
   }
-  if (!skip_lm) {
+  {
     // (tensor parallelism: m->vocab is this rank's shard; the logits stay sharded for the sampler)
     const bcg_gemm_fusion f = consumer(sumsq_mlp);
     BCG_TRY(gemm_bf16_tn_fused(ws->xn_last, m->lm_head, ws->logits, B, m->vocab, d, d, d, m->vocab,

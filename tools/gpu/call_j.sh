@@ -11,6 +11,6 @@ run "BCG_GEMM_2SM_HINT_A=0 BCG_GEMM_2SM_HINT_B=0"
 run "BCG_X=0"
 grep "==\|layer total" $O/gemm_variants.log
 for c in 1600 1780 1800 1900; do
-  timeout 200 python tools/step_ablation.py --period-only --ctx $c --sustain-steps 240 2>&1 | grep "full step\|1 token\|replays" >> $O/period_vs_ctx.txt
+  timeout 200 python tools/step_period.py --ctx $c --sustain-steps 240 2>&1 | grep "full step\|1 token\|replays" >> $O/period_vs_ctx.txt
 done
 cat $O/period_vs_ctx.txt

@@ -1,10 +1,7 @@
 #!/usr/bin/env python
-"""In-pipeline cost of each kernel family of the decode step (dev tool).
-
-Times the real decode step (CUDA graph, optional PDL) and the same step with one kernel family
-left out (bcg_model_decode profiling flags); the difference is what that family costs INSIDE the
-pipeline, overlap included — unlike isolated kernel timings.
-    python tools/step_ablation.py [--model qwen3-14b] [--rows 10] [--ctx 1600] [--pdl 1]
+"""Period of the decode step (dev tool): the real step as a CUDA graph, alone and with the sampler, for a
+few tokens and for seconds of back-to-back replays.
+    python tools/step_period.py [--model qwen3-14b] [--rows 10] [--ctx 1600] [--pdl 1]
 """
 import argparse
 import ctypes as C
@@ -20,9 +17,6 @@ from byzantine_consensus_llm_agents_b200.engine import Engine  # noqa: E402
 from byzantine_consensus_llm_agents_b200.model import PRESETS, Weights  # noqa: E402
 from byzantine_consensus_llm_agents_b200.tokenizer import get_tokenizer  # noqa: E402
 
-SKIPS = {"attention": 0x100, "add_rmsnorm": 0x200, "qknorm_rope_kvwrite": 0x400, "qkv GEMM": 0x1000,
-         "o GEMM": 0x2000, "gate_up GEMM": 0x4000, "down GEMM": 0x8000, "lm_head GEMM": 0x10000}
-
 
 def main():
     ap = argparse.ArgumentParser()
@@ -32,7 +26,6 @@ def main():
     ap.add_argument("--pdl", type=int, default=1)
     ap.add_argument("--sustain-steps", type=int, default=1500)
     ap.add_argument("--max-splits", type=int, default=0, help="attention grid width (default: what --ctx needs)")
-    ap.add_argument("--period-only", action="store_true", help="skip the per-kernel ablation")
     ap.add_argument("--base-flags", type=lambda x: int(x, 0), default=0,
                     help="extra bcg_model_decode flags for every run, e.g. 0x20000 = norm folded into the GEMMs")
     a = ap.parse_args()
@@ -134,14 +127,6 @@ def main():
 
     out["token_period_ms_sustained"] = sustained(a.sustain_steps)
     print(f"  step + sampler, {a.sustain_steps} replays back to back: {out['token_period_ms_sustained']:.3f} ms per token")
-    if a.period_only:
-        print(json.dumps(out))
-        return
-    for name, bit in SKIPS.items():
-        t = time_step(bit)
-        out[name] = full - t
-        per = (full - t) * 1e3 / (1 if name.startswith("lm_head") else cfg.n_layers)
-        print(f"  without {name:22s} {t:7.3f} ms   -> costs {full - t:6.3f} ms/step = {per:6.2f} us/launch-group")
     print(json.dumps(out))
 
 
