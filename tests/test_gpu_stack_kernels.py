@@ -179,7 +179,7 @@ def test_delta_scan_keeps_a_long_memory():
 
 # ------------------------------------------------------------------------------------------ latent attention
 SIZES = {   # heads, dim, rot_dim, vdim, kv_rank
-    "plain": (3, 10, 6, 20, 20), "small": (5, 16, 16, 24, 48), "even": (8, 32, 32, 32, 64), "wide-v": (2, 48, 16, 200, 112),
+    "plain": (3, 10, 6, 20, 20), "small": (5, 16, 16, 24, 48), "even": (6, 32, 32, 40, 80), "wide-v": (2, 48, 16, 200, 112),
     "large": (33, 128, 64, 128, 512), "max": (2, 192, 64, 256, 128), "one": (1, 8, 8, 8, 16), "tall": (40, 64, 64, 64, 64)}
 
 
