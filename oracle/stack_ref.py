@@ -2,7 +2,9 @@
 
 Plain, slow restatement of the mechanisms that layer-stack designs are made of (Bekopel: latent
 attention with a sliding window and a sink, generalized delta rule, PolyNorm feed-forward, norms on
-both sides of each sublayer).  One function per mechanism; torch on the CPU, in the dtype of its
+both sides of each sublayer; Lerazen: grouped-query attention with a linear distance bias, a query
+temperature and values mixed with an earlier layer's, squared-relu and mixture-of-experts
+feed-forwards, parallel sublayers, learned positions).  One function per mechanism; torch on the CPU, in the dtype of its
 inputs (the tests use float64, rounding weights only).  A whole sequence is computed at once, token by
 token where there is a recurrence, with no cache: what a cache, a batch or a cut of the prompt could get
 wrong is absent here by construction.
@@ -109,11 +111,107 @@ def feed_forward(h, w, eps):
     return poly_norm(h @ w["up"].T, [float(c) for c in w["act"]], eps) @ w["down"].T
 
 
+def squared_relu(z):
+    return torch.clamp(z, min=0) ** 2
+
+
+def dense_ff(h, w):
+    return squared_relu(h @ w["up"].T) @ w["down"].T
+
+
+def head_slopes(heads):
+    """Distance slope of every head: 2^-8 for the last one, a geometric series from 2^(-8 / heads)."""
+    return torch.tensor([2.0 ** (-8.0 * (h + 1) / heads) for h in range(heads)], dtype=torch.float64)
+
+
+def query_temperature(positions, coef, every):
+    return 1 + coef * torch.log(torch.floor((positions.to(torch.float64) + 1) / every) + 1)
+
+
+def mix_values(v, v_first, weight):
+    return (1 - weight) * v + weight * v_first
+
+
+def grouped_values(h, w):
+    return h @ w["v"].T + w["v.b"]
+
+
+def grouped_attention(h, v, w, m, positions):
+    """m: dict(heads, kv_heads, dim, vdim, scale, window, coef, every); v: the layer's (mixed) values
+    [t, kv_heads * vdim]; w: dict(q, q.b, k, k.b, o, o.b)."""
+    t, H, G = h.shape[0], m["heads"], m["kv_heads"]
+    q = (h @ w["q"].T + w["q.b"]).view(t, H, m["dim"])
+    q = q * query_temperature(positions, m["coef"], m["every"]).to(q.dtype)[:, None, None]
+    k = (h @ w["k"].T + w["k.b"]).view(t, G, m["dim"])
+    v = v.view(t, G, m["vdim"])
+    mine = torch.arange(H) // (H // G)                      # the key/value head of each query head
+    s = torch.einsum("ihd,jhd->hij", q, k[:, mine]) * m["scale"]
+    away = (positions[:, None] - positions[None, :]).to(s.dtype)
+    s = s - head_slopes(H).to(s.dtype)[:, None, None] * away
+    p = softmax_with_sink(s, window_visible(t, m["window"]))
+    o = torch.einsum("hij,jhd->ihd", p, v[:, mine]).reshape(t, H * m["vdim"])
+    return o @ w["o"].T + w["o.b"]
+
+
+def route(h, router, top):
+    """(experts [t, top], weights [t, top]): the experts with the largest sigmoid scores and those scores."""
+    s = torch.sigmoid(h @ router.T)
+    best = torch.topk(s, top, dim=-1)
+    return best.indices, best.values
+
+
+def clamped_glu(g, u, limit):
+    g, u = torch.clamp(g, max=limit), torch.clamp(u, -limit, limit)
+    return g * torch.sigmoid(1.702 * g) * (u + 1)
+
+
+def mixture(h, w, top, limit):
+    """The routing weight scales an expert's input."""
+    experts, weights = route(h, w["router"], top)
+    out = torch.zeros_like(h)
+    for t in range(h.shape[0]):
+        for e, s in zip(experts[t].tolist(), weights[t]):
+            x = s * h[t]
+            y = clamped_glu(w[f"e{e}.gate"] @ x, w[f"e{e}.up"] @ x, limit)
+            out[t] += w[f"e{e}.down"] @ y
+    return out
+
+
+def _lerazen(config, T, tokens, collect):
+    eps, pos = float(config["norm"]["eps"]), torch.arange(len(tokens))
+    x = T["embed"][torch.as_tensor(tokens, dtype=torch.long)] + T["pos"][pos]
+    v_first = None
+    for i, layer in enumerate(config["layers"]):
+        p, mix, mlp = f"l{i}.", layer["mixer"], layer.get("mlp")
+        sub = lambda kind: {n[len(p + kind) + 1:]: t for n, t in T.items() if n.startswith(p + kind + ".")}
+        w = sub("mix")
+        h = rms_norm(x, eps, T[p + "norm1"])
+        v = grouped_values(h, w)
+        if mix.get("v_mix"):
+            if v_first is None:
+                v_first = v
+            else:
+                v = mix_values(v, v_first, w["vmix"])
+        m = dict(heads=mix["heads"], kv_heads=mix["kv_heads"], dim=mix["dim"], vdim=mix["vdim"], scale=mix["scale"],
+                 window=mix["mask"]["size"], coef=mix["q_temp"]["coef"], every=mix["q_temp"]["every"])
+        y = grouped_attention(h, v, w, m, pos)
+        if mlp and mlp["kind"] == "moe":
+            y = y + mixture(h, sub("mlp"), mlp["router"]["top"], mlp["expert"]["limit"])
+        elif mlp:
+            y = y + dense_ff(h, sub("mlp"))
+        x = x + y
+        if collect is not None:
+            collect.append(x.clone())
+    return rms_norm(x, eps, T["final.norm"]) @ T["head"].T
+
+
 def forward(config, tensors, tokens, collect=None, dtype=torch.float64):
     """Logits [tokens, vocab] of one sequence.  `config` is the parsed config.json, `tensors` name -> tensor.
     `collect`: a list that receives the residual stream after every layer."""
     eps = float(config["norm"]["eps"])
     T = {n: x.to(dtype) if x.is_floating_point() else x for n, x in tensors.items()}
+    if config["architecture"] == "Lerazen":
+        return _lerazen(config, T, tokens, collect)
     pos = torch.arange(len(tokens))
     x = T["embed"][torch.as_tensor(tokens, dtype=torch.long)]
     kv = {}
