@@ -35,6 +35,8 @@ SOURCES = [
     "gemm_simt.cu",
     "latent_attn.cu",
     "latent_prefill.cu",
+    "grouped_attn.cu",
+    "moe.cu",
     "delta_scan.cu",
     "stack_step.cu",
 ]

@@ -224,7 +224,21 @@ int bcg_gemm_any(const void* X, int x_dtype, const void* W, float* out, int M, i
 int bcg_sandwich_norm(float* residual, const float* delta, int n_partials, long long partial_stride,
                       const float* w_post, const float* w_next, void* xn, int act_dtype, int T, int d, float eps,
                       void* stream) {
-  return sandwich_norm(residual, delta, n_partials, partial_stride, w_post, w_next, xn, act_dtype, T, d, eps,
+  return sandwich_norm(residual, delta, n_partials, partial_stride, w_post, w_next, xn, act_dtype, T, d, eps, {},
+                       S(stream));
+}
+
+int bcg_residual_norm(float* residual, const float* delta, int n_partials, long long partial_stride, const float* bias,
+                      const float* rows, const int* index, int per_row, int row_partials, long long row_stride,
+                      const float* w_next, void* xn, int act_dtype, int T, int d, float eps, void* stream) {
+  NormExtra extra;
+  extra.bias = bias;
+  extra.rows = rows;
+  extra.index = index;
+  extra.per_row = rows && index ? per_row : 0;
+  extra.n_partials = row_partials;
+  extra.partial_stride = row_stride;
+  return sandwich_norm(residual, delta, n_partials, partial_stride, nullptr, w_next, xn, act_dtype, T, d, eps, extra,
                        S(stream));
 }
 
@@ -244,6 +258,20 @@ int bcg_delta_scan(const bcg_layer* l, const float* proj, int n_partials, long l
 int bcg_latent_attention(const bcg_stack* m, const bcg_stack_ws* ws, const bcg_step_batch* b, int layer, int mode,
                          void* stream) {
   return latent_attention(m, ws, b, layer, mode, S(stream));
+}
+
+int bcg_grouped_in(const bcg_stack* m, const bcg_stack_ws* ws, const bcg_step_batch* b, int layer, int n_partials,
+                   long long partial_stride, long long ld, int with_act, void* stream) {
+  return grouped_in_step(m, ws, b, layer, n_partials, partial_stride, ld, with_act, S(stream));
+}
+
+int bcg_grouped_attention(const bcg_stack* m, const bcg_stack_ws* ws, const bcg_step_batch* b, int layer, int mode,
+                          void* stream) {
+  return grouped_attention_step(m, ws, b, layer, mode, S(stream));
+}
+
+int bcg_experts(const bcg_stack* m, const bcg_stack_ws* ws, int layer, int T, int* splits, void* stream) {
+  return experts_step(m, ws, layer, T, splits, S(stream));
 }
 
 }  // extern "C"

@@ -284,6 +284,14 @@ gemm2sm_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_
           } else {
             __nv_bfloat16* o = reinterpret_cast<__nv_bfloat16*>(args.out);
             uint32_t p[16];
+            if (args.epi == BCG_EPI_RELU2) {
+#pragma unroll
+              for (int j = 0; j < 16; ++j) {
+                const float x0 = fmaxf(__uint_as_float(v0[j]), 0.f), x1 = fmaxf(__uint_as_float(v1[j]), 0.f);
+                v0[j] = __float_as_uint(x0 * x0);
+                v1[j] = __float_as_uint(x1 * x1);
+              }
+            }
 #pragma unroll
             for (int j = 0; j < 8; ++j) {
               p[j] = pack_bf16(__uint_as_float(v0[2 * j]), __uint_as_float(v0[2 * j + 1]));
@@ -318,7 +326,8 @@ gemm2sm_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_
 // single-CTA kernel).
 int gemm2sm_bf16_tn(const void* X, const void* W, void* out, int M, int N, int K, long long ldx, long long ldw,
                     long long ld_out, int epi, cudaStream_t stream) {
-  if (M < 512 || (N % k2BlockN) != 0) return BCG_ERR_UNSUPPORTED;
+  // the last column tile may be partial (the epilogue stores 32 columns at a time), where that wastes little
+  if (M < 512 || (N % 32) != 0 || (N % k2BlockN != 0 && N < 8 * k2BlockN)) return BCG_ERR_UNSUPPORTED;
   static const bool off = getenv("BCG_GEMM_2SM") && atoi(getenv("BCG_GEMM_2SM")) == 0;   // tuning knob
   if (off) return BCG_ERR_UNSUPPORTED;
   Gemm2Args a = {};
@@ -326,7 +335,7 @@ int gemm2sm_bf16_tn(const void* X, const void* W, void* out, int M, int N, int K
   a.N = N;
   a.K = K;
   a.tiles_m = (M + 255) / 256;
-  a.tiles_n = N / k2BlockN;
+  a.tiles_n = (N + k2BlockN - 1) / k2BlockN;
   a.k_blocks = (K + k2BlockK - 1) / k2BlockK;
   static const int group = getenv("BCG_GEMM_2SM_GROUP") ? atoi(getenv("BCG_GEMM_2SM_GROUP")) : 12;   // tuning knobs
   static const int stages = getenv("BCG_GEMM_2SM_STAGES") ? atoi(getenv("BCG_GEMM_2SM_STAGES")) : 7;

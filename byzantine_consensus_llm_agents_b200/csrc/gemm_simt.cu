@@ -1,5 +1,7 @@
 // out fp32 [M, ldo] = X [M, ldx] * W bf16 [N, ldw]^T on CUDA cores, fp32 FMA throughout: the product of
 // fp32 activations, and of bf16 ones whose shape TMA cannot address.  64 x 64 tiles, 4 x 4 per thread.
+// With row counts: rows sorted by group, blockIdx.z = group, W = the groups' matrices one after another.
+#include "moe.cuh"
 #include "stack_common.cuh"
 #include "kernels.h"
 
@@ -10,10 +12,18 @@ constexpr int kSgT = 64, kSgK = 16;
 template <typename T>
 __global__ void __launch_bounds__(256)
 gemm_simt_kernel(const T* __restrict__ X, const __nv_bfloat16* __restrict__ W, float* __restrict__ out, int M, int N,
-                 int K, long long ldx, long long ldw, long long ldo) {
+                 int K, long long ldx, long long ldw, long long ldo, const int* __restrict__ counts) {
   __shared__ float xs[kSgK][kSgT + 4], wsm[kSgK][kSgT + 4];
   pdl_launch_dependents();
   pdl_wait();
+  if (counts) {
+    M = counts[blockIdx.z];
+    if (static_cast<int>(blockIdx.y) * kSgT >= M) return;
+    const long long row0 = expert_offset(counts, blockIdx.z, threadIdx.x & 31);
+    X += row0 * ldx;
+    out += row0 * ldo;
+    W += static_cast<long long>(blockIdx.z) * N * ldw;
+  }
   const int n0 = blockIdx.x * kSgT, m0 = blockIdx.y * kSgT;
   const int tx = threadIdx.x & 15, ty = threadIdx.x >> 4;
   const int lk = threadIdx.x & 15, lr = threadIdx.x >> 4;   // loader: k within the slice, row (four turns)
@@ -56,10 +66,28 @@ int gemm_any(const void* X, int x_dtype, const void* W, float* out, int M, int N
   const auto* w = static_cast<const __nv_bfloat16*>(W);
   if (x_dtype == BCG_DT_F32)
     BCG_CUDA_CHECK(launch_k(gemm_simt_kernel<float>, grid, dim3(256), 0, st, static_cast<const float*>(X), w, out, M,
-                            N, K, ldx, ldw, ldo));
+                            N, K, ldx, ldw, ldo, nullptr));
   else
     BCG_CUDA_CHECK(launch_k(gemm_simt_kernel<__nv_bfloat16>, grid, dim3(256), 0, st,
-                            static_cast<const __nv_bfloat16*>(X), w, out, M, N, K, ldx, ldw, ldo));
+                            static_cast<const __nv_bfloat16*>(X), w, out, M, N, K, ldx, ldw, ldo, nullptr));
+  return BCG_OK;
+}
+
+int gemm_any_grouped(const void* X, int x_dtype, const void* W, float* out, int N, int K, const GemmGroups& g,
+                     cudaStream_t st) {
+  if (!X || !W || !out || N <= 0 || K <= 0 || !g.counts || g.n_groups <= 0 || g.n_groups > 65535 || g.max_rows <= 0 ||
+      (g.max_rows + kSgT - 1) / kSgT > 65535) {
+    set_last_error("bcg_gemm_any", "bad grouped product");
+    return BCG_ERR_ARG;
+  }
+  const dim3 grid((N + kSgT - 1) / kSgT, (g.max_rows + kSgT - 1) / kSgT, g.n_groups);
+  const auto* w = static_cast<const __nv_bfloat16*>(W);
+  if (x_dtype == BCG_DT_F32)
+    BCG_CUDA_CHECK(launch_k(gemm_simt_kernel<float>, grid, dim3(256), 0, st, static_cast<const float*>(X), w, out, 0, N, K,
+                            K, K, N, g.counts));
+  else
+    BCG_CUDA_CHECK(launch_k(gemm_simt_kernel<__nv_bfloat16>, grid, dim3(256), 0, st, static_cast<const __nv_bfloat16*>(X),
+                            w, out, 0, N, K, K, K, N, g.counts));
   return BCG_OK;
 }
 

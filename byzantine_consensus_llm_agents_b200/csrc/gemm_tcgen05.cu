@@ -11,6 +11,9 @@
 //     fp32 [split][M][N] and summed in a FIXED order by the consumer kernel
 //     (add_rmsnorm / qknorm_rope / swiglu_reduce): deterministic, batch-invariant.
 //
+// GROUPED: rows sorted by group (mixture of experts), W = the groups' matrices one after another; a tile belongs to
+// one group.  How many rows a group has is read on the device, so the list of work items is too.
+//
 // Roles (192 threads): warp 0 = TMA producer, warp 1 = TMEM alloc + MMA issuer,
 // warps 2..5 = epilogue (TMEM -> registers -> global).  smem ring of STAGES
 // {A 128x64, B BNx64} bf16 tiles in the 128B-swizzled K-major layout shared by TMA and
@@ -65,13 +68,49 @@ struct GemmArgs {
   __nv_bfloat16* red_xn;     // [M][N]
   float* red_sumsq;          // [tiles_a][kSumsqStride]
   int* red_counters;         // [tiles_a], zero on entry, zero again on exit
+  GemmGroups groups;         // GROUPED only; M = rows of all groups, N = weight rows of one
 };
 
+__device__ __forceinline__ uint32_t relu_squared(uint32_t v) {
+  const float r = fmaxf(__uint_as_float(v), 0.f);
+  return __float_as_uint(r * r);
+}
 __device__ __forceinline__ float silu_mul(float g, float u) {
   return g * (1.0f / (1.0f + __expf(-g))) * u;
 }
 
-template <int BN, int STAGES>
+// First item, row tile and row of every group, from the groups' row counts (one warp).
+__device__ __forceinline__ void scan_groups(const GemmGroups& g, int tile_rows, int* first_tile, int* first_row, int lane) {
+  int tiles = 0, rows = 0;
+  for (int e0 = 0; e0 < g.n_groups; e0 += 32) {
+    const int c = e0 + lane < g.n_groups ? g.counts[e0 + lane] : 0;
+    int ct = (c + tile_rows - 1) / tile_rows, cr = c;
+#pragma unroll
+    for (int o = 1; o < 32; o <<= 1) {
+      const int t = __shfl_up_sync(0xffffffffu, ct, o), r = __shfl_up_sync(0xffffffffu, cr, o);
+      if (lane >= o) {
+        ct += t;
+        cr += r;
+      }
+    }
+    if (e0 + lane < g.n_groups) {
+      first_tile[e0 + lane + 1] = tiles + ct;
+      first_row[e0 + lane + 1] = rows + cr;
+    }
+    tiles += __shfl_sync(0xffffffffu, ct, 31);
+    rows += __shfl_sync(0xffffffffu, cr, 31);
+  }
+  if (lane == 0) first_tile[0] = first_row[0] = 0;
+}
+
+// gate clamped from above, linear part from both sides (mixture of experts)
+__device__ __forceinline__ float glu_clamp(float g, float u, float limit, float alpha) {
+  g = fminf(g, limit);
+  u = fminf(fmaxf(u, -limit), limit);
+  return __fdividef(g, 1.0f + __expf(-alpha * g)) * (u + 1.0f);
+}
+
+template <int BN, int STAGES, bool GROUPED>
 __global__ void __launch_bounds__(kGemmThreads, two_cta(BN, STAGES) ? 2 : 1)
 gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_a,
                     const __grid_constant__ CUtensorMap tmap_b, const GemmArgs args) {
@@ -92,6 +131,7 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_a,
   uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(tmem_empty + 2);
   __shared__ float row_scale[kSumsqStride];
   __shared__ int red_last;
+  __shared__ int first_tile[GROUPED ? kMaxGroups + 1 : 1], first_row[GROUPED ? kMaxGroups + 1 : 1];
 
   const int warp = threadIdx.x >> 5;
   const int lane = threadIdx.x & 31;
@@ -120,10 +160,37 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_a,
   tc_fence_after();
   const uint32_t tmem_base = *tmem_slot;
 
-  const int total_items = args.tiles_a * args.tiles_b * args.splits;
+  // tiles along the weights (GROUPED: of one group)
+  const int w_tiles = args.swap ? args.tiles_a : args.tiles_b;
+  int total_items = args.tiles_a * args.tiles_b * args.splits;
+  if constexpr (GROUPED) {
+    pdl_wait();
+    if (warp == 0) scan_groups(args.groups, args.swap ? BN : kBlockA, first_tile, first_row, lane);
+    __syncthreads();
+    total_items = first_tile[args.groups.n_groups] * w_tiles * args.splits;
+  }
   const int group_tiles = args.group_a * args.tiles_b;
 
-  auto decode_item = [&](int item, int& ta, int& tb, int& split, int& kb0, int& kb1) {
+  // GROUPED: ta / tb are tiles inside group `e`
+  auto decode_item = [&](int item, int& ta, int& tb, int& split, int& kb0, int& kb1, int& e) {
+    e = 0;
+    if constexpr (GROUPED) {
+      const int unit = item / (w_tiles * args.splits);
+      int hi = args.groups.n_groups;      // first_tile[e] <= unit < first_tile[hi]
+      while (hi - e > 1) {
+        const int mid = (e + hi) >> 1;
+        if (first_tile[mid] <= unit) e = mid;
+        else hi = mid;
+      }
+      const int local = item - first_tile[e] * w_tiles * args.splits, rt = first_tile[e + 1] - first_tile[e];
+      split = local % args.splits;
+      const int tile = local / args.splits, w = tile / rt, r = tile - w * rt;
+      ta = args.swap ? w : r;
+      tb = args.swap ? r : w;
+      kb0 = static_cast<int>((static_cast<long long>(split) * args.k_blocks) / args.splits);
+      kb1 = static_cast<int>((static_cast<long long>(split + 1) * args.k_blocks) / args.splits);
+      return;
+    }
     split = item % args.splits;
     const int t = item / args.splits;
     const int g = t / group_tiles;
@@ -148,12 +215,12 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_a,
       // cp.async.bulk.prefetch made the step monotonically slower, 6.16 -> 6.93 ms at 64 tiles.)
       int n_pre = 0;
       if (args.pdl_wait_b) {
-        if (args.swap) {
+        if (!GROUPED && args.swap) {
           constexpr int pre = STAGES < kPreWaitStages ? STAGES : kPreWaitStages;
           int idx = 0;
           for (int item = blockIdx.x; item < total_items && idx < pre; item += gridDim.x) {
-            int ta, tb, split, kb0, kb1;
-            decode_item(item, ta, tb, split, kb0, kb1);
+            int ta, tb, split, kb0, kb1, e;
+            decode_item(item, ta, tb, split, kb0, kb1, e);
             for (int kb = kb0; kb < kb1 && idx < pre; ++kb, ++idx) {
               mbar_arrive_expect_tx(&full_bar[idx], STAGE_BYTES);
               tma_load_2d(smem + idx * STAGE_BYTES, &tmap_a, &full_bar[idx], kb * kBlockK,
@@ -169,17 +236,21 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_a,
       uint32_t phase = 0;
       int idx = 0;
       for (int item = blockIdx.x; item < total_items; item += gridDim.x) {
-        int ta, tb, split, kb0, kb1;
-        decode_item(item, ta, tb, split, kb0, kb1);
+        int ta, tb, split, kb0, kb1, e;
+        decode_item(item, ta, tb, split, kb0, kb1, e);
+        int row_a = ta * kBlockA, row_b = tb * BN;
+        if constexpr (GROUPED) {
+          row_a += args.swap ? e * args.N : first_row[e];
+          row_b += args.swap ? first_row[e] : e * args.N;
+        }
         for (int kb = kb0; kb < kb1; ++kb, ++idx) {
           uint8_t* sa = smem + stage * STAGE_BYTES;
           if (idx >= n_pre) {
             mbar_wait(&empty_bar[stage], phase ^ 1);
             mbar_arrive_expect_tx(&full_bar[stage], STAGE_BYTES);
-            tma_load_2d(sa, &tmap_a, &full_bar[stage], kb * kBlockK, ta * kBlockA, args.hint_a);
+            tma_load_2d(sa, &tmap_a, &full_bar[stage], kb * kBlockK, row_a, args.hint_a);
           }
-          tma_load_2d(sa + A_BYTES, &tmap_b, &full_bar[stage], kb * kBlockK, tb * BN,
-                      args.hint_b);
+          tma_load_2d(sa + A_BYTES, &tmap_b, &full_bar[stage], kb * kBlockK, row_b, args.hint_b);
           if (++stage == STAGES) {
             stage = 0;
             phase ^= 1;
@@ -195,8 +266,8 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_a,
     int acc = 0;
     uint32_t acc_phase = 0;
     for (int item = blockIdx.x; item < total_items; item += gridDim.x) {
-      int ta, tb, split, kb0, kb1;
-      decode_item(item, ta, tb, split, kb0, kb1);
+      int ta, tb, split, kb0, kb1, e;
+      decode_item(item, ta, tb, split, kb0, kb1, e);
       mbar_wait(&tmem_empty[acc], acc_phase ^ 1);
       tc_fence_after();
       const uint32_t tmem_d = tmem_base + static_cast<uint32_t>(acc * BN);
@@ -250,11 +321,15 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_a,
     }
     int acc = 0;
     uint32_t acc_phase = 0;
-    const int M = args.M, N = args.N;
+    const int N = args.N;
     const long long ld = args.ld_out;
+    const long long slab = static_cast<long long>(args.M) * ld;
     for (int item = blockIdx.x; item < total_items; item += gridDim.x) {
-      int ta, tb, split, kb0, kb1;
-      decode_item(item, ta, tb, split, kb0, kb1);
+      int ta, tb, split, kb0, kb1, e;
+      decode_item(item, ta, tb, split, kb0, kb1, e);
+      // rows this tile may store: M of them from row `base` of the output
+      const int M = GROUPED ? first_row[e + 1] - first_row[e] : args.M;
+      const long long base = GROUPED ? first_row[e] * ld : 0;
       mbar_wait(&tmem_full[acc], acc_phase);
       tc_fence_after();
       const uint32_t taddr = tmem_base + (static_cast<uint32_t>(q * 32) << 16) +
@@ -274,7 +349,7 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_a,
               v[j] = __float_as_uint(__uint_as_float(v[j]) * row_scale[(m0 + c + j) & (kSumsqStride - 1)]);
           }
           if (args.epi == BCG_EPI_F32) {
-            float* o = reinterpret_cast<float*>(args.out) + static_cast<long long>(split) * M * ld;
+            float* o = reinterpret_cast<float*>(args.out) + split * slab + base;
 #pragma unroll
             for (int j = 0; j < 16; ++j) {
               const int m = m0 + c + j;
@@ -303,8 +378,10 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_a,
         // lanes = activation rows (m), columns = weight rows (n)
         const int m = ta * kBlockA + row;
         const int n0 = tb * BN;
-        if (args.epi == BCG_EPI_SWIGLU) {
-          __nv_bfloat16* o = reinterpret_cast<__nv_bfloat16*>(args.out);
+        if (args.epi == BCG_EPI_SWIGLU || (GROUPED && args.epi == BCG_EPI_GLU)) {
+          __nv_bfloat16* o = reinterpret_cast<__nv_bfloat16*>(args.out) + base;
+          float weight = 1.f;
+          if (GROUPED && m < M) weight = args.groups.row_weight[first_row[e] + m];
 #pragma unroll 1
           for (int c = 0; c < BN; c += 32) {
             uint32_t g[16], u[16];
@@ -314,8 +391,13 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_a,
             uint32_t p[8];
 #pragma unroll
             for (int j = 0; j < 8; ++j) {
-              p[j] = pack_bf16(silu_mul(__uint_as_float(g[2 * j]), __uint_as_float(u[2 * j])),
-                               silu_mul(__uint_as_float(g[2 * j + 1]), __uint_as_float(u[2 * j + 1])));
+              const float g0 = __uint_as_float(g[2 * j]), g1 = __uint_as_float(g[2 * j + 1]);
+              const float u0 = __uint_as_float(u[2 * j]), u1 = __uint_as_float(u[2 * j + 1]);
+              if constexpr (GROUPED)
+                p[j] = pack_bf16(glu_clamp(weight * g0, weight * u0, args.groups.glu_limit, args.groups.glu_alpha),
+                                 glu_clamp(weight * g1, weight * u1, args.groups.glu_limit, args.groups.glu_alpha));
+              else
+                p[j] = pack_bf16(silu_mul(g0, u0), silu_mul(g1, u1));
             }
             if (m < M && n0 + c < N) {
               uint4* dst = reinterpret_cast<uint4*>(o + m * ld + (n0 + c) / 2);
@@ -331,8 +413,7 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_a,
             tmem_ld_x16(taddr + c + 16, v1);
             tmem_ld_wait();
             if (args.epi == BCG_EPI_F32) {
-              float* o = reinterpret_cast<float*>(args.out) +
-                         static_cast<long long>(split) * M * ld;
+              float* o = reinterpret_cast<float*>(args.out) + split * slab + base;
               if (m < M) {
                 float4* dst = reinterpret_cast<float4*>(o + m * ld + n0 + c);
                 if (n0 + c < N) {
@@ -349,8 +430,15 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_a,
                 }
               }
             } else {
-              __nv_bfloat16* o = reinterpret_cast<__nv_bfloat16*>(args.out);
+              __nv_bfloat16* o = reinterpret_cast<__nv_bfloat16*>(args.out) + base;
               uint32_t p[16];
+              if (args.epi == BCG_EPI_RELU2) {
+#pragma unroll
+                for (int j = 0; j < 16; ++j) {
+                  v0[j] = relu_squared(v0[j]);
+                  v1[j] = relu_squared(v1[j]);
+                }
+              }
 #pragma unroll
               for (int j = 0; j < 8; ++j) {
                 p[j] = pack_bf16(__uint_as_float(v0[2 * j]), __uint_as_float(v0[2 * j + 1]));
@@ -395,7 +483,6 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_a,
           const int n = ta * kBlockA + lane * 4;
           const float4 wv = *reinterpret_cast<const float4*>(args.red_w + n);
           const float* P = reinterpret_cast<const float*>(args.out);
-          const long long slab = static_cast<long long>(M) * ld;
           for (int m = e; m < M; m += 4) {
             float4 p[16];
             // unconditional (clamped) loads so that all of them are in flight before the first add
@@ -486,14 +573,14 @@ static int num_sms() {
   return n;
 }
 
-template <int BN, int STAGES>
+template <int BN, int STAGES, bool GROUPED = false>
 static int launch_gemm(const CUtensorMap& ta, const CUtensorMap& tb, const GemmArgs& a, int pdl,
                        cudaStream_t stream) {
   constexpr int STAGE_BYTES = kBlockA * kBlockK * 2 + BN * kBlockK * 2;
   constexpr int SMEM = STAGES * STAGE_BYTES + 1024 + 256;
-  if (const int rc = ensure_dynamic_smem(reinterpret_cast<const void*>(gemm_tcgen05_kernel<BN, STAGES>), SMEM))
+  if (const int rc = ensure_dynamic_smem(reinterpret_cast<const void*>(gemm_tcgen05_kernel<BN, STAGES, GROUPED>), SMEM))
     return rc;
-  const int total = a.tiles_a * a.tiles_b * a.splits;
+  const int total = GROUPED ? a.group_a : a.tiles_a * a.tiles_b * a.splits;   // GROUPED: the most items there can be
   cudaLaunchConfig_t cfg = {};
   const int slots = two_cta(BN, STAGES) ? 2 * num_sms() : num_sms();
   cfg.gridDim = dim3(static_cast<unsigned>(total < slots ? total : slots));
@@ -505,7 +592,7 @@ static int launch_gemm(const CUtensorMap& ta, const CUtensorMap& tb, const GemmA
   attr[0].val.programmaticStreamSerializationAllowed = pdl ? 1 : 0;
   cfg.attrs = attr;
   cfg.numAttrs = 1;
-  BCG_CUDA_CHECK(cudaLaunchKernelEx(&cfg, gemm_tcgen05_kernel<BN, STAGES>, ta, tb, a));
+  BCG_CUDA_CHECK(cudaLaunchKernelEx(&cfg, gemm_tcgen05_kernel<BN, STAGES, GROUPED>, ta, tb, a));
   return BCG_OK;
 }
 
@@ -566,6 +653,10 @@ int gemm_bf16_tn_fused(const void* X, const void* W, void* out, int M, int N, in
     return BCG_ERR_ARG;
   }
   const bool swap = (M <= 128);
+  if (epi < 0 || epi > BCG_EPI_RELU2 || (epi == BCG_EPI_RELU2 && (swap || N % 16))) {
+    set_last_error("bcg_gemm_bf16_tn", "unknown epilogue, or squared relu with M <= 128 or N % 16");
+    return BCG_ERR_ARG;
+  }
   if (!swap && ((epi == BCG_EPI_SWIGLU ? (ld_out % 8) : (epi == BCG_EPI_F32 ? (ld_out % 4) : (ld_out % 8))))) {
     set_last_error("bcg_gemm_bf16_tn", "ld_out must keep 16-byte row alignment");
     return BCG_ERR_ARG;
@@ -653,6 +744,56 @@ int gemm_bf16_tn_fused(const void* X, const void* W, void* out, int M, int N, in
     case 128: return swap ? launch_gemm<128, 3>(tma, tmb, a, pdl, stream)  // decode, 65-128 rows: two CTAs per SM
                           : launch_gemm<128, 6>(tma, tmb, a, pdl, stream);
     default: return launch_gemm<256, 4>(tma, tmb, a, pdl, stream);
+  }
+}
+
+// Rows sorted by group: X [rows, K], W [n_groups * N, K]; every group's rows against its own N weight rows.
+// max_rows bounds the rows of one group; up to 128 of them run as the decode form (weights on the TMEM lanes).
+int gemm_grouped(const void* X, const void* W, void* out, int rows, int N, int K, int epi, int splits, const GemmGroups& g,
+                 cudaStream_t stream) {
+  const bool swap = g.max_rows <= 128;
+  if (!X || !W || !out || rows <= 0 || N <= 0 || K <= 0 || K % 8 || g.n_groups <= 0 || g.n_groups > kMaxGroups ||
+      !g.counts || splits < 1 || (splits > 1 && !swap) || (epi != BCG_EPI_F32 && (epi != BCG_EPI_GLU || swap || N % 32)) ||
+      (!swap && N % 16) || (epi == BCG_EPI_GLU && !g.row_weight) ||
+      ((reinterpret_cast<uintptr_t>(X) | reinterpret_cast<uintptr_t>(W) | reinterpret_cast<uintptr_t>(out)) & 15)) {
+    set_last_error("bcg_gemm_grouped", "bad argument (K % 8, N % 16 beyond 128 rows, at most 512 groups, alignment)");
+    return BCG_ERR_ARG;
+  }
+  GemmArgs a = {};
+  a.M = rows;
+  a.N = N;
+  a.K = K;
+  a.k_blocks = (K + kBlockK - 1) / kBlockK;
+  a.splits = splits > a.k_blocks ? a.k_blocks : splits;
+  a.swap = swap ? 1 : 0;
+  a.epi = epi;
+  a.out = out;
+  a.ld_out = epi == BCG_EPI_GLU ? N / 2 : N;
+  a.groups = g;
+  a.pdl_wait_b = (launch_flags() & BCG_GEMM_PDL) ? 1 : 0;
+  const int bn = swap ? (g.max_rows <= 16 ? 16 : g.max_rows <= 32 ? 32 : g.max_rows <= 64 ? 64 : 128)
+                      : (N % 256 == 0 ? 256 : 128);
+  const int tile_rows = swap ? bn : kBlockA, w_tiles = swap ? (N + kBlockA - 1) / kBlockA : (N + bn - 1) / bn;
+  a.tiles_a = swap ? w_tiles : 1;
+  a.tiles_b = swap ? 1 : w_tiles;
+  const long long units = (g.n_groups < rows ? g.n_groups : rows) + static_cast<long long>(rows) / tile_rows;
+  const long long items = units * w_tiles * a.splits;
+  a.group_a = items > (1 << 30) ? (1 << 30) : static_cast<int>(items);
+  a.hint_a = swap ? kEvictFirst : kEvictNormal;
+  a.hint_b = swap ? kEvictLast : kEvictNormal;
+  CUtensorMap wm, xm;
+  int rc;
+  if ((rc = make_tmap_bf16_sw128(&wm, W, static_cast<long long>(g.n_groups) * N, K, K, swap ? kBlockA : bn)) != BCG_OK) return rc;
+  if ((rc = make_tmap_bf16_sw128(&xm, X, rows, K, K, swap ? bn : kBlockA)) != BCG_OK) return rc;
+  const CUtensorMap &ta = swap ? wm : xm, &tb = swap ? xm : wm;
+  const int pdl = a.pdl_wait_b;
+  switch (bn) {
+    case 16: return launch_gemm<16, 5, true>(ta, tb, a, pdl, stream);
+    case 32: return launch_gemm<32, 5, true>(ta, tb, a, pdl, stream);
+    case 64: return launch_gemm<64, 4, true>(ta, tb, a, pdl, stream);
+    case 128: return swap ? launch_gemm<128, 3, true>(ta, tb, a, pdl, stream)
+                          : launch_gemm<128, 6, true>(ta, tb, a, pdl, stream);
+    default: return launch_gemm<256, 4, true>(ta, tb, a, pdl, stream);
   }
 }
 

@@ -1,0 +1,572 @@
+// Grouped-query attention with a linear distance bias, sliding window and query temperature over paged keys and
+// values.
+//
+// A layer's cache is two pools of 16-token pages, keys [page][kv head][16][q_ld] and values [page][kv head][16][v_ld];
+// heads are padded to q_ld / v_ld columns, the padding is zero and stays so.
+//   grouped_in      projection slabs -> queries (bias, temperature), keys and values (bias, value mixing) into the
+//                   pages, squared-relu activations of a parallel feed-forward, routing of a parallel mixture
+//   grouped_plain   one CTA per (token, head), any sizes, fp32 or bf16: the fp32 engine's kernel, and the bf16
+//                   one's for head sizes the kernels below do not take
+//   grouped_decode  single tokens: a cluster per (token, kv head) shares the key pages, a ring of TMA loads and a
+//                   running softmax per warp, partial results merged through distributed shared memory
+//   prompts run on the tcgen05 window attention kernel (attn_window.cuh), reading pages directly
+#include "attn_window.cuh"
+#include "mma_sync.cuh"
+#include "moe.cuh"
+
+namespace bcg {
+
+constexpr float kLog2e = 1.4426950408889634f;
+
+// ------------------------------------------------------------------------------------------- inputs
+constexpr int kInThreads = 256;
+
+struct GroupedIn {
+  const float* proj;          // [n_partials][T][ld]
+  int n_partials;
+  long long pstride, ld;
+  const int *positions, *slot_map;
+  const float* bias;          // [q + k + v columns]
+  void *q, *k_cache, *v_cache, *act;
+  float* v_first;             // [T][kv_heads * vdim]
+  int heads, kv_heads, dim, vdim, q_ld, v_ld, page_size;
+  float temp_coef, temp_every;
+  int v_role;
+  float v_mix;
+  int ff, act_from;           // squared-relu columns of proj (ff = 0: none)
+  long long act_ld;
+  int blocks;                 // CTAs per token that share the columns
+  MoeRoute route;             // experts = 0: none
+};
+
+// grid (T, blocks [+ 1 routes]).  Columns go to their destination four at a time (V = 4) or one by one.
+template <typename T, int V>
+__global__ void __launch_bounds__(kInThreads)
+grouped_in_kernel(const GroupedIn a) {
+  extern __shared__ float scores[];   // routing: one logit per expert
+  pdl_launch_dependents();
+  pdl_wait();
+  const long long t = blockIdx.x;
+  const float* row = a.proj + t * a.ld;
+  if (static_cast<int>(blockIdx.y) == a.blocks) {
+    route_token<kInThreads>(a.route, row, a.n_partials, a.pstride, static_cast<int>(t), scores);
+    return;
+  }
+  const int pos = a.positions[t], slot = a.slot_map[t];
+  const float temp = 1.0f + a.temp_coef * logf(floorf(static_cast<float>(pos + 1) / a.temp_every) + 1.0f);
+  const int nq = a.heads * a.dim, nk = nq + a.kv_heads * a.dim, nv = nk + a.kv_heads * a.vdim;
+  const long long page = slot >= 0 ? slot / a.page_size : 0;
+  const int in_page = slot >= 0 ? slot % a.page_size : 0;
+  const int step = a.blocks * kInThreads * V;
+  for (int c = (blockIdx.y * kInThreads + threadIdx.x) * V; c < nv; c += step) {
+    Vec<V> x = slab_sum_vec<V>(row + c, a.n_partials, a.pstride);
+    const Vec<V> b = load_vec<V>(a.bias + c);
+#pragma unroll
+    for (int i = 0; i < V; ++i) x.x[i] += b.x[i];
+    if (c < nq) {
+      const int h = c / a.dim, i = c - h * a.dim;
+#pragma unroll
+      for (int k = 0; k < V; ++k) x.x[k] *= temp;
+      store_vec<V>(static_cast<T*>(a.q) + (t * a.heads + h) * a.q_ld + i, x);
+    } else if (c < nk) {
+      const int g = (c - nq) / a.dim, i = c - nq - g * a.dim;
+      if (slot >= 0)
+        store_vec<V>(static_cast<T*>(a.k_cache) + ((page * a.kv_heads + g) * a.page_size + in_page) * a.q_ld + i, x);
+    } else {
+      const int o = c - nk, g = o / a.vdim, i = o - g * a.vdim;
+      float* first = a.v_first + t * (nv - nk) + o;
+      if (a.v_role == BCG_VALUES_FIRST) {
+        store_vec<V>(first, x);
+      } else if (a.v_role == BCG_VALUES_MIX) {
+        const Vec<V> f = load_vec<V>(first);
+#pragma unroll
+        for (int k = 0; k < V; ++k) x.x[k] = (1.0f - a.v_mix) * x.x[k] + a.v_mix * f.x[k];
+      }
+      if (slot >= 0)
+        store_vec<V>(static_cast<T*>(a.v_cache) + ((page * a.kv_heads + g) * a.page_size + in_page) * a.v_ld + i, x);
+    }
+  }
+  for (int c = (blockIdx.y * kInThreads + threadIdx.x) * V; c < a.ff; c += step) {
+    Vec<V> x = slab_sum_vec<V>(row + a.act_from + c, a.n_partials, a.pstride);
+#pragma unroll
+    for (int k = 0; k < V; ++k) {
+      const float r = fmaxf(x.x[k], 0.f);
+      x.x[k] = r * r;
+    }
+    store_vec<V>(static_cast<T*>(a.act) + t * a.act_ld + c, x);
+  }
+}
+
+template <typename T>
+static int grouped_in_t(const GroupedIn& a, int n_tokens, cudaStream_t st) {
+  const bool wide = ((a.dim | a.vdim | a.ff | a.act_from) & 3) == 0 && a.ld % 4 == 0 && a.pstride % 4 == 0;
+  const dim3 grid(n_tokens, a.blocks + (a.route.experts > 0 ? 1 : 0));
+  const size_t sm = static_cast<size_t>(a.route.experts) * 4;
+  if (wide) BCG_CUDA_CHECK(launch_k(grouped_in_kernel<T, 4>, grid, dim3(kInThreads), sm, st, a));
+  else BCG_CUDA_CHECK(launch_k(grouped_in_kernel<T, 1>, grid, dim3(kInThreads), sm, st, a));
+  return BCG_OK;
+}
+
+// with_act: the activations of the feed-forward are columns l->n_qkv.. of proj (else the GEMM made them)
+int grouped_in(const bcg_stack* m, const bcg_layer* l, const bcg_stack_ws* ws, const bcg_step_batch* b, int n_partials,
+               long long pstride, long long ld, bool with_act, cudaStream_t st) {
+  const size_t act_bytes = m->act_dtype == BCG_DT_F32 ? 4 : 2;
+  GroupedIn a = {};
+  a.proj = ws->proj;
+  a.n_partials = n_partials;
+  a.pstride = pstride;
+  a.ld = ld;
+  a.positions = b->positions;
+  a.slot_map = b->slot_map;
+  a.bias = l->in_bias;
+  a.q = ws->q;
+  a.k_cache = l->cache;
+  a.v_cache = l->cache_v;
+  a.v_first = ws->v_first;
+  a.heads = l->heads;
+  a.kv_heads = l->kv_heads;
+  a.dim = l->dim;
+  a.vdim = l->vdim;
+  a.q_ld = l->q_ld;
+  a.v_ld = l->v_ld;
+  a.page_size = m->page_size;
+  a.temp_coef = l->temp_coef;
+  a.temp_every = l->temp_every;
+  a.v_role = l->v_role;
+  a.v_mix = l->v_mix;
+  a.ff = with_act ? l->ff : 0;
+  a.act_from = with_act ? l->n_qkv : 0;
+  a.act = static_cast<char*>(ws->mix) + l->act_col * act_bytes;
+  a.act_ld = l->mix_ld;
+  if (l->experts > 0) a.route = moe_route(l, ws);
+  const int cols = l->heads * l->dim + l->kv_heads * (l->dim + l->vdim);
+  a.blocks = b->T <= 128 ? max(1, ((cols > a.ff ? cols : a.ff) + kInThreads * 4 - 1) / (kInThreads * 4)) : 1;
+  return m->act_dtype == BCG_DT_F32 ? grouped_in_t<float>(a, b->T, st) : grouped_in_t<__nv_bfloat16>(a, b->T, st);
+}
+
+// ------------------------------------------------------------------------------------------- plain
+constexpr int kGpThreads = 128, kGpKeys = 256;
+
+struct GroupedAttn {
+  const void *q, *k_cache, *v_cache;
+  const float* slopes;
+  const int *rows, *positions, *row_seq, *block_table;
+  int max_blocks, page_size;
+  void* out;
+  long long out_ld;
+  int heads, kv_heads, dim, vdim, q_ld, v_ld, window;
+  float scale;
+};
+
+template <typename T>
+__global__ void __launch_bounds__(kGpThreads)
+grouped_plain_kernel(const GroupedAttn a) {
+  extern __shared__ float sm[];
+  __shared__ float red[kGpThreads / 32];
+  float* qs = sm;             // [dim]
+  float* oc = qs + a.dim;     // [vdim]
+  float* p = oc + a.vdim;     // [kGpKeys]
+  pdl_launch_dependents();
+  pdl_wait();
+  const long long t = a.rows ? a.rows[blockIdx.x] : blockIdx.x;
+  const int h = blockIdx.y, g = h / (a.heads / a.kv_heads);
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int pos = a.positions[t];
+  const int* bt = a.block_table + static_cast<long long>(a.row_seq ? a.row_seq[t] : t) * a.max_blocks;
+  const T* qh = static_cast<const T*>(a.q) + (t * a.heads + h) * a.q_ld;
+  const float slope = a.slopes ? a.slopes[h] : 0.f;
+  auto row_of = [&](int key) {
+    return (static_cast<long long>(bt[key / a.page_size]) * a.kv_heads + g) * a.page_size + key % a.page_size;
+  };
+  for (int i = threadIdx.x; i < a.dim; i += kGpThreads) qs[i] = to_f32<T>(qh[i]);
+  for (int i = threadIdx.x; i < a.vdim; i += kGpThreads) oc[i] = 0.f;
+  float m = -INFINITY, l = 0.f;
+  const int lo = a.window > 0 ? max(0, pos - a.window + 1) : 0;
+  for (int j0 = lo; j0 <= pos; j0 += kGpKeys) {
+    const int n = min(kGpKeys, pos + 1 - j0);
+    __syncthreads();
+    float mx = -INFINITY;
+    for (int j = warp; j < n; j += kGpThreads / 32) {
+      const int key = j0 + j;
+      const T* k = static_cast<const T*>(a.k_cache) + row_of(key) * a.q_ld;
+      float s = 0.f;
+      for (int i = lane; i < a.dim; i += 32) s = fmaf(qs[i], to_f32<T>(k[i]), s);
+      s = warp_sum(s) * a.scale - slope * static_cast<float>(pos - key);
+      if (lane == 0) p[j] = s;
+      mx = fmaxf(mx, s);
+    }
+    if (lane == 0) red[warp] = mx;
+    __syncthreads();
+#pragma unroll
+    for (int i = 0; i < kGpThreads / 32; ++i) mx = fmaxf(mx, red[i]);
+    const float m_new = fmaxf(m, mx);
+    const float corr = expf(m - m_new);
+    float sum = 0.f;
+    for (int j = threadIdx.x; j < n; j += kGpThreads) {
+      const float e = expf(p[j] - m_new);
+      p[j] = e;
+      sum += e;
+    }
+    sum = warp_sum(sum);
+    __syncthreads();
+    if (lane == 0) red[warp] = sum;
+    __syncthreads();
+    sum = 0.f;
+#pragma unroll
+    for (int i = 0; i < kGpThreads / 32; ++i) sum += red[i];
+    l = l * corr + sum;
+    m = m_new;
+    for (int r = threadIdx.x; r < a.vdim; r += kGpThreads) {
+      float acc = oc[r] * corr;
+      for (int j = 0; j < n; ++j)
+        acc = fmaf(p[j], to_f32<T>(static_cast<const T*>(a.v_cache)[row_of(j0 + j) * a.v_ld + r]), acc);
+      oc[r] = acc;
+    }
+  }
+  __syncthreads();
+  const float inv = 1.0f / l;
+  T* dst = static_cast<T*>(a.out) + t * a.out_ld + static_cast<long long>(h) * a.vdim;
+  for (int r = threadIdx.x; r < a.vdim; r += kGpThreads) dst[r] = from_f32<T>(oc[r] * inv);
+}
+
+static GroupedAttn attn_args(const bcg_stack* m, const bcg_layer* l, const bcg_stack_ws* ws, const bcg_step_batch* b,
+                             const int* rows) {
+  GroupedAttn a = {};
+  a.q = ws->q;
+  a.k_cache = l->cache;
+  a.v_cache = l->cache_v;
+  a.slopes = l->slopes;
+  a.rows = rows;
+  a.positions = b->positions;
+  a.row_seq = b->row_seq;
+  a.block_table = b->block_table;
+  a.max_blocks = b->max_blocks;
+  a.page_size = m->page_size;
+  a.out = ws->mix;
+  a.out_ld = l->mix_ld;
+  a.heads = l->heads;
+  a.kv_heads = l->kv_heads;
+  a.dim = l->dim;
+  a.vdim = l->vdim;
+  a.q_ld = l->q_ld;
+  a.v_ld = l->v_ld;
+  a.window = l->window;
+  a.scale = l->scale;
+  return a;
+}
+
+static int grouped_plain(const bcg_stack* m, const bcg_layer* l, const bcg_stack_ws* ws, const bcg_step_batch* b,
+                         const int* rows, int n, cudaStream_t st) {
+  const GroupedAttn a = attn_args(m, l, ws, b, rows);
+  const int sm = (l->dim + l->vdim + kGpKeys) * 4;
+  const dim3 grid(n, l->heads);
+  if (m->act_dtype == BCG_DT_F32) {
+    BCG_TRY(ensure_dynamic_smem(reinterpret_cast<const void*>(grouped_plain_kernel<float>), 64 * 1024));
+    BCG_CUDA_CHECK(launch_k(grouped_plain_kernel<float>, grid, dim3(kGpThreads), sm, st, a));
+  } else {
+    BCG_TRY(ensure_dynamic_smem(reinterpret_cast<const void*>(grouped_plain_kernel<__nv_bfloat16>), 64 * 1024));
+    BCG_CUDA_CHECK(launch_k(grouped_plain_kernel<__nv_bfloat16>, grid, dim3(kGpThreads), sm, st, a));
+  }
+  return BCG_OK;
+}
+
+// ------------------------------------------------------------------------------------------- decode
+// grid (cluster, tokens, kv heads x groups of 16 query heads), 4 warps.  The visible pages of a token are dealt
+// round-robin to the cluster's warps; a warp keeps `stages` pages in flight, each a stage of its own ring.
+constexpr int kGdWarps = 4, kGdThreads = kGdWarps * 32, kGdHeads = 16, kGdPage = 16, kGdMaxCluster = 8;
+
+template <int QD, int VD>
+struct GdCfg {
+  static constexpr int kK = kGdPage * QD * 2, kV = kGdPage * VD * 2, kStage = kK + kV;
+  static constexpr int kFit = 96 * 1024 / (kGdWarps * kStage);
+  static constexpr int kStages = kFit < 2 ? 2 : kFit > 6 ? 6 : kFit;
+  static constexpr int kRing = kStages * kStage;                      // a warp's ring; later its partial output
+  static constexpr int kQRow = QD + 8;
+  static constexpr int kOffQ = kGdWarps * kRing;
+  static constexpr int kOffMl = kOffQ + kGdHeads * kQRow * 2;         // [5][16] (maximum, denominator)
+  static constexpr int kOffBar = kOffMl + (kGdWarps + 1) * kGdHeads * 8;
+  static constexpr int kSmem = kOffBar + kGdWarps * kStages * 8 + 1024;
+  static_assert(kGdHeads * VD * 4 <= kRing, "a warp's partial output fits its ring");
+};
+
+// 16 x D tile of D / 64 boxes of [16 rows][128 bytes], 128B-swizzled: address of 16-byte chunk `chunk` of a row
+__device__ __forceinline__ const void* swizzled(const uint8_t* tile, int row, int chunk) {
+  return tile + (chunk >> 3) * (kGdPage * 128) + row * 128 + (((chunk & 7) ^ (row & 7)) << 4);
+}
+
+template <int QD, int VD>
+__global__ void __launch_bounds__(kGdThreads)
+grouped_decode_kernel(const __grid_constant__ CUtensorMap k_map, const __grid_constant__ CUtensorMap v_map,
+                      const GroupedAttn a) {
+  using C = GdCfg<QD, VD>;
+  namespace cg = cooperative_groups;
+  extern __shared__ __align__(16) uint8_t gd_raw[];
+  uint8_t* smem = gd_raw + ((1024u - (smem_u32(gd_raw) & 1023u)) & 1023u);
+  __nv_bfloat16* qs = reinterpret_cast<__nv_bfloat16*>(smem + C::kOffQ);
+  float2* ml = reinterpret_cast<float2*>(smem + C::kOffMl);   // [warp][16], then the CTA's
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  uint64_t* full = reinterpret_cast<uint64_t*>(smem + C::kOffBar) + warp * C::kStages;
+  uint8_t* ring = smem + warp * C::kRing;
+  pdl_launch_dependents();
+  if (lane == 0) {
+    tma_prefetch_desc(&k_map);
+    tma_prefetch_desc(&v_map);
+    for (int s = 0; s < C::kStages; ++s) mbar_init(&full[s], 1);
+    fence_barrier_init();
+  }
+  __syncwarp();
+  pdl_wait();
+  cg::cluster_group cluster = cg::this_cluster();
+  const int rank = blockIdx.x, n_cta = gridDim.x;
+  const int i_tok = blockIdx.y, g = blockIdx.z % a.kv_heads, group = a.heads / a.kv_heads;
+  const int h0 = g * group + blockIdx.z / a.kv_heads * kGdHeads;
+  const int nh = min(kGdHeads, (g + 1) * group - h0);
+  const int t = a.rows ? a.rows[i_tok] : i_tok;
+  const int pos = a.positions[t];
+  const int lo = a.window > 0 ? max(0, pos - a.window + 1) : 0;
+  const int* bt = a.block_table + static_cast<long long>(a.row_seq ? a.row_seq[t] : t) * a.max_blocks;
+  const int first = lo / kGdPage + rank * kGdWarps + warp, stride = n_cta * kGdWarps;
+  const int n = pos / kGdPage >= first ? (pos / kGdPage - first) / stride + 1 : 0;
+  auto load = [&](int i) {    // lane 0
+    const int st = i % C::kStages;
+    const int row = (bt[first + i * stride] * a.kv_heads + g) * kGdPage;
+    uint8_t* dst = ring + st * C::kStage;
+    mbar_arrive_expect_tx(&full[st], C::kStage);
+#pragma unroll
+    for (int c = 0; c < QD / 64; ++c)
+      tma_load_2d(dst + c * kGdPage * 128, &k_map, &full[st], c * 64, row, kEvictNormal);
+#pragma unroll
+    for (int c = 0; c < VD / 64; ++c)
+      tma_load_2d(dst + C::kK + c * kGdPage * 128, &v_map, &full[st], c * 64, row, kEvictNormal);
+  };
+  if (lane == 0)
+    for (int i = 0; i < C::kStages && i < n; ++i) load(i);
+  const __nv_bfloat16* qsrc = static_cast<const __nv_bfloat16*>(a.q) + (static_cast<long long>(t) * a.heads + h0) * a.q_ld;
+  for (int i = threadIdx.x; i < kGdHeads * (QD / 8); i += kGdThreads) {
+    const int r = i / (QD / 8), c = i % (QD / 8) * 8;
+    *reinterpret_cast<uint4*>(qs + r * C::kQRow + c) =
+        r < nh ? *reinterpret_cast<const uint4*>(qsrc + static_cast<long long>(r) * a.q_ld + c) : make_uint4(0, 0, 0, 0);
+  }
+  __syncthreads();
+  const float scale2 = a.scale * kLog2e;
+  float slope[2], m[2] = {-INFINITY, -INFINITY}, l[2] = {0.f, 0.f};
+#pragma unroll
+  for (int e = 0; e < 2; ++e) {
+    const int r = (lane >> 2) + e * 8;
+    slope[e] = (a.slopes && r < nh) ? a.slopes[h0 + r] * kLog2e : 0.f;
+  }
+  float o[VD / 8][4] = {};
+  for (int i = 0; i < n; ++i) {
+    const int st = i % C::kStages;
+    const uint8_t* kt = ring + st * C::kStage;
+    const uint8_t* vt = kt + C::kK;
+    mbar_wait(&full[st], (i / C::kStages) & 1);
+    float s[2][4] = {};
+#pragma unroll
+    for (int k = 0; k < QD / 16; ++k) {
+      uint32_t qa[4], kb[4];
+      ldsm_x4(qa, qs + (lane & 15) * C::kQRow + k * 16 + (lane >> 4) * 8);
+      ldsm_x4(kb, swizzled(kt, (lane & 7) + ((lane >> 4) << 3), k * 2 + ((lane >> 3) & 1)));
+      mma_bf16_16816(s[0], qa, kb[0], kb[1]);
+      mma_bf16_16816(s[1], qa, kb[2], kb[3]);
+    }
+    const int key0 = (first + i * stride) * kGdPage + (lane & 3) * 2;
+    float corr[2];
+#pragma unroll
+    for (int e = 0; e < 2; ++e) {
+      float mx = -INFINITY;
+#pragma unroll
+      for (int c = 0; c < 4; ++c) {      // keys key0, key0 + 1, key0 + 8, key0 + 9
+        const int key = key0 + (c >> 1) * 8 + (c & 1);
+        float& x = s[c >> 1][2 * e + (c & 1)];
+        x = key >= lo && key <= pos ? fmaf(x, scale2, slope[e] * static_cast<float>(key - pos)) : -INFINITY;
+        mx = fmaxf(mx, x);
+      }
+      mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 1));
+      mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 2));
+      const float m_new = fmaxf(m[e], mx);       // every page has a visible key: finite
+      corr[e] = ex2_approx(m[e] - m_new);
+      m[e] = m_new;
+      float sum = 0.f;
+#pragma unroll
+      for (int c = 0; c < 4; ++c) {
+        float& x = s[c >> 1][2 * e + (c & 1)];
+        x = ex2_approx(x - m_new);
+        sum += x;
+      }
+      l[e] = l[e] * corr[e] + sum;
+    }
+    const uint32_t pa[4] = {pack_bf16(s[0][0], s[0][1]), pack_bf16(s[0][2], s[0][3]), pack_bf16(s[1][0], s[1][1]),
+                            pack_bf16(s[1][2], s[1][3])};
+    if (__any_sync(0xffffffffu, corr[0] != 1.0f || corr[1] != 1.0f)) {
+#pragma unroll
+      for (int j = 0; j < VD / 8; ++j) {
+        o[j][0] *= corr[0];
+        o[j][1] *= corr[0];
+        o[j][2] *= corr[1];
+        o[j][3] *= corr[1];
+      }
+    }
+#pragma unroll
+    for (int j = 0; j < VD / 16; ++j) {
+      uint32_t vb[4];
+      ldsm_x4_trans(vb, swizzled(vt, lane & 15, j * 2 + (lane >> 4)));
+      mma_bf16_16816(o[2 * j], pa, vb[0], vb[1]);
+      mma_bf16_16816(o[2 * j + 1], pa, vb[2], vb[3]);
+    }
+    __syncwarp();                        // everybody has read the page: its stage may be filled again
+    if (lane == 0 && i + C::kStages < n) load(i + C::kStages);
+  }
+  // ---- merge: the warps of a CTA, then the CTAs of the cluster
+  float* part = reinterpret_cast<float*>(ring);      // [16][VD]
+#pragma unroll
+  for (int e = 0; e < 2; ++e) {
+    l[e] += __shfl_xor_sync(0xffffffffu, l[e], 1);
+    l[e] += __shfl_xor_sync(0xffffffffu, l[e], 2);
+    const int r = (lane >> 2) + e * 8;
+    if ((lane & 3) == 0) ml[warp * kGdHeads + r] = make_float2(m[e], l[e]);
+#pragma unroll
+    for (int j = 0; j < VD / 8; ++j)
+      *reinterpret_cast<float2*>(part + r * VD + j * 8 + (lane & 3) * 2) = make_float2(o[j][2 * e], o[j][2 * e + 1]);
+  }
+  __syncthreads();
+  auto weight = [](float mine, float top) { return mine == -INFINITY ? 0.f : ex2_approx(mine - top); };
+  float* mine = reinterpret_cast<float*>(smem);      // the CTA's result takes warp 0's place
+  for (int i = threadIdx.x; i < nh * VD; i += kGdThreads) {
+    const int r = i / VD;
+    float top = -INFINITY, x = 0.f, den = 0.f;
+#pragma unroll
+    for (int w = 0; w < kGdWarps; ++w) top = fmaxf(top, ml[w * kGdHeads + r].x);
+#pragma unroll
+    for (int w = 0; w < kGdWarps; ++w) {
+      const float f = weight(ml[w * kGdHeads + r].x, top);
+      x = fmaf(f, reinterpret_cast<const float*>(smem + w * C::kRing)[i], x);
+      den = fmaf(f, ml[w * kGdHeads + r].y, den);
+    }
+    mine[i] = x;                                     // element i is read and written by this thread only
+    if (i % VD == 0) ml[kGdWarps * kGdHeads + r] = make_float2(top, den);
+  }
+  if (n_cta > 1) cluster.sync();
+  else __syncthreads();
+  auto* dst = static_cast<__nv_bfloat16*>(a.out) + static_cast<long long>(t) * a.out_ld + static_cast<long long>(h0) * a.vdim;
+  for (int i = rank * kGdThreads + threadIdx.x; i < nh * VD; i += n_cta * kGdThreads) {
+    const int r = i / VD, c = i % VD;
+    if (c >= a.vdim) continue;
+    float top = -INFINITY, x = 0.f, den = 0.f;
+    for (int q = 0; q < n_cta; ++q) {
+      const float2 other = *cluster.map_shared_rank(ml + kGdWarps * kGdHeads + r, q);
+      const float val = cluster.map_shared_rank(mine, q)[i];
+      const float up = fmaxf(top, other.x);
+      const float f0 = weight(top, up), f1 = weight(other.x, up);
+      x = x * f0 + val * f1;
+      den = den * f0 + other.y * f1;
+      top = up;
+    }
+    dst[static_cast<long long>(r) * a.vdim + c] = __float2bfloat16(x / den);
+  }
+  if (n_cta > 1) cluster.sync();                     // nobody leaves while its shared memory is being read
+}
+
+template <int QD, int VD>
+static int launch_decode(const CUtensorMap& km, const CUtensorMap& vm, const GroupedAttn& a, dim3 grid, cudaStream_t st) {
+  using C = GdCfg<QD, VD>;
+  BCG_TRY(ensure_dynamic_smem(reinterpret_cast<const void*>(grouped_decode_kernel<QD, VD>), C::kSmem));
+  BCG_CUDA_CHECK(launch_cluster(grouped_decode_kernel<QD, VD>, grid, dim3(kGdThreads), static_cast<int>(grid.x), C::kSmem,
+                                st, km, vm, a));
+  return BCG_OK;
+}
+
+static bool padded_head(int q_ld, int v_ld) {
+  return q_ld % 64 == 0 && q_ld >= 64 && q_ld <= 256 && (v_ld == 64 || v_ld == 128 || v_ld == 256);
+}
+
+// CTAs per (token, kv head): the choice with the fewest page times on 148 SMs with two CTAs each (a CTA costs
+// about four pages of start-up).
+static int decode_cluster(int rows, int pages) {
+  int best = 1;
+  long long best_cost = -1;
+  for (int c = 1; c <= kGdMaxCluster; c *= 2) {
+    if (c > 1 && pages < c * kGdWarps) break;
+    const long long waves = (static_cast<long long>(rows) * c + 295) / 296;
+    const long long cost = waves * ((pages + c * kGdWarps - 1) / (c * kGdWarps) + 4);
+    if (best_cost < 0 || cost < best_cost) {
+      best_cost = cost;
+      best = c;
+    }
+  }
+  return best;
+}
+
+static int grouped_decode(const bcg_stack* m, const bcg_layer* l, const bcg_stack_ws* ws, const bcg_step_batch* b,
+                          cudaStream_t st) {
+  const int n = b->single_rows ? b->n_single : b->T;
+  const int reach = l->window > 0 && l->window < b->max_context ? l->window + kGdPage - 1 : b->max_context;
+  const int pages = (reach + kGdPage - 1) / kGdPage;
+  const int groups = l->kv_heads * ((l->heads / l->kv_heads + kGdHeads - 1) / kGdHeads);
+  if (n > 65535 || groups > 65535) {
+    set_last_error("bcg_grouped_attention", "too many single tokens or heads");
+    return BCG_ERR_TOO_LARGE;
+  }
+  const dim3 grid(decode_cluster(n * groups, pages), n, groups);
+  CUtensorMap km, vm;
+  BCG_TRY(make_tmap_bf16_sw128(&km, l->cache, 1ll << 30, l->q_ld, l->q_ld, kGdPage));
+  BCG_TRY(make_tmap_bf16_sw128(&vm, l->cache_v, 1ll << 30, l->v_ld, l->v_ld, kGdPage));
+  const GroupedAttn a = attn_args(m, l, ws, b, b->single_rows);
+#define BCG_GD(Q, V) \
+  if (l->q_ld == Q && l->v_ld == V) return launch_decode<Q, V>(km, vm, a, grid, st)
+  BCG_GD(64, 64);
+  BCG_GD(64, 128);
+  BCG_GD(64, 256);
+  BCG_GD(128, 64);
+  BCG_GD(128, 128);
+  BCG_GD(128, 256);
+  BCG_GD(192, 64);
+  BCG_GD(192, 128);
+  BCG_GD(192, 256);
+  BCG_GD(256, 64);
+  BCG_GD(256, 128);
+  BCG_GD(256, 256);
+#undef BCG_GD
+  set_last_error("bcg_grouped_attention", "no decode kernel for this head size");
+  return BCG_ERR_UNSUPPORTED;
+}
+
+// ------------------------------------------------------------------------------------------- prompts
+static int grouped_prefill(const bcg_layer* l, const bcg_stack_ws* ws, const bcg_step_batch* b, cudaStream_t st) {
+  CUtensorMap qm, km, vm;
+  const long long q_cols = static_cast<long long>(l->heads) * l->q_ld;
+  BCG_TRY(make_tmap_bf16_sw128(&qm, ws->q, b->T, q_cols, q_cols, kWaBM));
+  BCG_TRY(make_tmap_bf16_sw128(&km, l->cache, 1ll << 30, l->q_ld, l->q_ld, kWaPage));
+  BCG_TRY(make_tmap_bf16_sw128(&vm, l->cache_v, 1ll << 30, l->v_ld, l->v_ld, kWaPage));
+  WindowAttn a = {};
+  a.tiles = b->tiles;
+  a.n_tiles = b->n_tiles;
+  a.slopes = l->slopes;
+  a.block_table = b->block_table;
+  a.max_blocks = b->max_blocks;
+  a.page_heads = l->kv_heads;
+  a.group = l->heads / l->kv_heads;
+  a.out = static_cast<__nv_bfloat16*>(ws->mix);
+  a.out_ld = l->mix_ld;
+  a.heads = l->heads;
+  a.vdim = l->vdim;
+  a.window = l->window;
+  a.scale_log2e = l->scale * kLog2e;
+  return window_attn<true, true>(l->q_ld, l->v_ld, qm, km, vm, a, st);
+}
+
+int grouped_attention(const bcg_stack* m, const bcg_stack_ws* ws, const bcg_step_batch* b, const bcg_layer* l, int mode,
+                      cudaStream_t st) {
+  const int n_single = b->single_rows ? b->n_single : (b->n_tiles > 0 ? 0 : b->T);
+  const bool tensor = m->act_dtype == BCG_DT_BF16 && mode == 0 && m->page_size == kGdPage && padded_head(l->q_ld, l->v_ld);
+  if (!tensor) return grouped_plain(m, l, ws, b, nullptr, b->T, st);
+  if (b->n_tiles > 0) {
+    // the prompt kernel stores 16 bytes at a time and wants slopes
+    if (l->slopes && l->vdim % 8 == 0 && l->mix_ld % 8 == 0) BCG_TRY(grouped_prefill(l, ws, b, st));
+    else BCG_TRY(grouped_plain(m, l, ws, b, nullptr, b->T, st));   // single tokens are recomputed below: harmless
+  }
+  if (n_single > 0) BCG_TRY(grouped_decode(m, l, ws, b, st));
+  return BCG_OK;
+}
+
+}  // namespace bcg

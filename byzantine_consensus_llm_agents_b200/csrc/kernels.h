@@ -16,6 +16,20 @@ int gemm_bf16_tn_fused(const void* X, const void* W, void* out, int M, int N, in
                        long long ldw, long long ld_out, int epi, int splits, int flags,
                        const bcg_gemm_fusion* fusion, cudaStream_t stream);
 int gemm_splits_for(int M, int N, int K);
+// Rows sorted by group (mixture of experts); internal epilogue BCG_EPI_GLU: columns interleaved [16 gate | 16 up],
+// each row's accumulators times its weight, clamped gated unit, bf16 [rows, N / 2]
+constexpr int BCG_EPI_GLU = 16;
+constexpr int kMaxGroups = 512;
+struct GemmGroups {
+  const int* counts;         // device [n_groups]: rows of every group
+  int n_groups, max_rows;    // max_rows: host-side bound on the rows of one group
+  const float* row_weight;   // [rows]
+  float glu_limit, glu_alpha;
+};
+int gemm_grouped(const void* X, const void* W, void* out, int rows, int N, int K, int epi, int splits, const GemmGroups& g,
+                 cudaStream_t stream);
+int gemm_any_grouped(const void* X, int x_dtype, const void* W, float* out, int N, int K, const GemmGroups& g,
+                     cudaStream_t stream);
 // Prefill shapes on CTA pairs (tcgen05.mma.cta_group::2); BCG_ERR_UNSUPPORTED = not a shape for it
 int gemm2sm_bf16_tn(const void* X, const void* W, void* out, int M, int N, int K, long long ldx, long long ldw,
                     long long ld_out, int epi, cudaStream_t stream);
@@ -62,14 +76,24 @@ int prefill_attn_paged(const void* q, const void* kv_cache, const int* block_tab
 
 int mask_sample(const bcg_sampler_args* a, cudaStream_t stream);
 
+// Further summands of sandwich_norm's delta: a bias, and `per_row` rows of a second set of slabs.
+struct NormExtra {
+  const float* bias = nullptr;      // [d]
+  const float* rows = nullptr;      // [n_partials][any][d]
+  const int* index = nullptr;       // [T][per_row] rows of it
+  int per_row = 0, n_partials = 1;
+  long long partial_stride = 0;
+};
 // layer stacks (stack_*.cu, latent_*.cu, delta_scan.cu, gemm_simt.cu); act_dtype = BCG_DT_*
-int embed_norm(const int* ids, const void* embed, const float* w, float* residual, void* xn, int act_dtype, int T,
-               int d, float eps, cudaStream_t stream);
+// pos_embed (bf16 [n_pos, d]) may be NULL; zero[0..n_zero) is set to zero on the way
+int embed_norm(const int* ids, const void* embed, const int* positions, const void* pos_embed, int n_pos, const float* w,
+               float* residual, void* xn, int act_dtype, int T, int d, float eps, int* zero, int n_zero,
+               cudaStream_t stream);
 int rows_norm(const float* residual, const int* rows, const float* w, void* xn, int act_dtype, int n, int d,
               float eps, cudaStream_t stream);
 int sandwich_norm(float* residual, const float* delta, int n_partials, long long partial_stride,
                   const float* w_post, const float* w_next, void* xn, int act_dtype, int T, int d, float eps,
-                  cudaStream_t stream);
+                  const NormExtra& extra, cudaStream_t stream);
 int poly_norm(const float* z, int n_partials, long long partial_stride, const float* coef, void* out, int act_dtype,
               int T, int ff, float eps, cudaStream_t stream);
 int gemm_any(const void* X, int x_dtype, const void* W, float* out, int M, int N, int K, long long ldx,
@@ -92,6 +116,18 @@ int delta_scan(const bcg_layer* l, const float* proj, int n_partials, long long 
                float eps, cudaStream_t stream);
 int latent_attention(const bcg_stack* m, const bcg_stack_ws* ws, const bcg_step_batch* b, int layer, int mode,
                      cudaStream_t stream);
+int grouped_in(const bcg_stack* m, const bcg_layer* l, const bcg_stack_ws* ws, const bcg_step_batch* b, int n_partials,
+               long long pstride, long long ld, bool with_act, cudaStream_t stream);
+int grouped_attention(const bcg_stack* m, const bcg_stack_ws* ws, const bcg_step_batch* b, const bcg_layer* l, int mode,
+                      cudaStream_t stream);
+// ws->xn through the layer's experts into ws->moe_out (*splits slabs), rows ws->moe_row
+int experts(const bcg_stack* m, const bcg_layer* l, const bcg_stack_ws* ws, int T, int* splits, cudaStream_t stream);
+int moe_splits(int T, int top, int N, int K);
+int grouped_in_step(const bcg_stack* m, const bcg_stack_ws* ws, const bcg_step_batch* b, int layer, int n_partials,
+                    long long pstride, long long ld, int with_act, cudaStream_t stream);
+int grouped_attention_step(const bcg_stack* m, const bcg_stack_ws* ws, const bcg_step_batch* b, int layer, int mode,
+                           cudaStream_t stream);
+int experts_step(const bcg_stack* m, const bcg_stack_ws* ws, int layer, int T, int* splits, cudaStream_t stream);
 int stack_step(const bcg_stack* m, const bcg_stack_ws* ws, const bcg_step_batch* b, cudaStream_t stream);
 int stack_head(const bcg_stack* m, const bcg_stack_ws* ws, const int* rows, int n, int row0, int flags,
                cudaStream_t stream);

@@ -52,6 +52,10 @@ struct Vec {
     for (int i = 0; i < V; ++i) s += x[i] * x[i];
     return s;
   }
+  __device__ __forceinline__ void add(const Vec& o) {
+#pragma unroll
+    for (int i = 0; i < V; ++i) x[i] += o.x[i];
+  }
 };
 template <int V>
 __device__ __forceinline__ Vec<V> load_vec(const float* p) {

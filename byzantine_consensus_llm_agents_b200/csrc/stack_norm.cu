@@ -1,6 +1,7 @@
 // Row-wise kernels of layer stacks:
-//   embed_norm      x = E[ids];  xn = rmsnorm(x) * w
+//   embed_norm      x = E[ids] (+ P[positions]);  xn = rmsnorm(x) * w
 //   sandwich_norm   x += rmsnorm(delta) * w_post (or += delta);  xn = rmsnorm(x) * w_next
+//                   delta may have a bias and rows of a second source (a token's experts) added
 //   rows_norm       xn[i] = rmsnorm(x[rows[i]]) * w
 //   poly_norm       PolyNorm activation: a N(z) + b N(z^2) + c N(z^3) + e, N = division by the row's RMS
 // `delta` and `z` arrive as fp32 split-K slabs of the projection in front.  Decode-sized launches spread a
@@ -17,22 +18,36 @@ constexpr int kClusterMaxRows = 128;
 
 template <typename T, int V>
 __global__ void __launch_bounds__(kRowT)
-embed_norm_kernel(const int* __restrict__ ids, const __nv_bfloat16* __restrict__ embed, const float* __restrict__ w,
-                  float* __restrict__ residual, T* __restrict__ xn, int d, float eps) {
+embed_norm_kernel(const int* __restrict__ ids, const __nv_bfloat16* __restrict__ embed,
+                  const int* __restrict__ positions, const __nv_bfloat16* __restrict__ pos_embed, int n_pos,
+                  const float* __restrict__ w, float* __restrict__ residual, T* __restrict__ xn, int d, float eps,
+                  int* __restrict__ zero, int n_zero) {
   __shared__ RowSum<kRowT, 1, 1> sh;
   pdl_launch_dependents();
   pdl_wait();
   const long long t = blockIdx.x, row = ids[t];
+  for (int i = blockIdx.x * kRowT + threadIdx.x; i < n_zero; i += gridDim.x * kRowT) zero[i] = 0;
+  const __nv_bfloat16* pos = nullptr;
+  if (pos_embed) pos = pos_embed + static_cast<long long>(min(positions[t], n_pos - 1)) * d;
+  auto token = [&](int v) {
+    Vec<V> x = load_vec<V>(embed + row * d + v);
+    if (pos) {
+      const Vec<V> p = load_vec<V>(pos + v);
+#pragma unroll
+      for (int k = 0; k < V; ++k) x.x[k] += p.x[k];
+    }
+    return x;
+  };
   float ss[1] = {0.f};
   for (int v = threadIdx.x * V; v < d; v += kRowT * V) {
-    const Vec<V> x = load_vec<V>(embed + row * d + v);
+    const Vec<V> x = token(v);
     store_vec<V>(residual + t * d + v, x);
     ss[0] += x.sumsq();
   }
   row_sum<kRowT, 1, 1>(sh, ss, 0);
   const float inv = rsqrtf(ss[0] / static_cast<float>(d) + eps);
   for (int v = threadIdx.x * V; v < d; v += kRowT * V) {
-    Vec<V> x = load_vec<V>(embed + row * d + v);
+    Vec<V> x = token(v);
     const Vec<V> ww = load_vec<V>(w + v);
 #pragma unroll
     for (int k = 0; k < V; ++k) x.x[k] *= inv * ww.x[k];
@@ -44,7 +59,7 @@ template <typename T, int V, int CL>
 __global__ void __launch_bounds__(kRowT)
 sandwich_norm_kernel(float* __restrict__ residual, const float* __restrict__ delta, int n_partials,
                      long long partial_stride, const float* __restrict__ w_post, const float* __restrict__ w_next,
-                     T* __restrict__ xn, int d, float eps) {
+                     T* __restrict__ xn, int d, float eps, const NormExtra extra) {
   extern __shared__ float4 stage_raw[];   // this CTA's part of the row
   float* stage = reinterpret_cast<float*>(stage_raw);
   __shared__ RowSum<kRowT, CL, 1> sh;
@@ -56,7 +71,11 @@ sandwich_norm_kernel(float* __restrict__ residual, const float* __restrict__ del
   const float inv_d = 1.0f / static_cast<float>(d);
   float ss[1] = {0.f};
   for (int v = v0 + threadIdx.x * V; v < v1; v += kRowT * V) {
-    const Vec<V> y = slab_sum_vec<V>(delta + t * d + v, n_partials, partial_stride);
+    Vec<V> y = slab_sum_vec<V>(delta + t * d + v, n_partials, partial_stride);
+    if (extra.bias) y.add(load_vec<V>(extra.bias + v));
+    for (int k = 0; k < extra.per_row; ++k)
+      y.add(slab_sum_vec<V>(extra.rows + static_cast<long long>(extra.index[t * extra.per_row + k]) * d + v,
+                            extra.n_partials, extra.partial_stride));
     store_vec<V>(stage + v - v0, y);
     ss[0] += y.sumsq();
   }
@@ -162,15 +181,20 @@ poly_norm_kernel(const float* __restrict__ z, int n_partials, long long partial_
   } while (0)
 
 template <typename T, int V>
-static int embed_t(const int* ids, const void* embed, const float* w, float* residual, void* xn, int T_rows, int d,
-                   float eps, cudaStream_t st) {
+static int embed_t(const int* ids, const void* embed, const int* positions, const void* pos_embed, int n_pos,
+                   const float* w, float* residual, void* xn, int T_rows, int d, float eps, int* zero, int n_zero,
+                   cudaStream_t st) {
   BCG_CUDA_CHECK(launch_k(embed_norm_kernel<T, V>, dim3(T_rows), dim3(kRowT), 0, st, ids,
-                          static_cast<const __nv_bfloat16*>(embed), w, residual, static_cast<T*>(xn), d, eps));
+                          static_cast<const __nv_bfloat16*>(embed), positions,
+                          static_cast<const __nv_bfloat16*>(pos_embed), n_pos, w, residual, static_cast<T*>(xn), d, eps,
+                          zero, n_zero));
   return BCG_OK;
 }
-int embed_norm(const int* ids, const void* embed, const float* w, float* residual, void* xn, int act_dtype, int T,
-               int d, float eps, cudaStream_t st) {
-  BCG_BY_TYPE(embed_t, d, act_dtype, ids, embed, w, residual, xn, T, d, eps, st);
+int embed_norm(const int* ids, const void* embed, const int* positions, const void* pos_embed, int n_pos, const float* w,
+               float* residual, void* xn, int act_dtype, int T, int d, float eps, int* zero, int n_zero,
+               cudaStream_t st) {
+  BCG_BY_TYPE(embed_t, d, act_dtype, ids, embed, positions, pos_embed, n_pos, w, residual, xn, T, d, eps, zero, n_zero,
+              st);
 }
 
 template <typename T, int V>
@@ -193,28 +217,30 @@ static size_t row_stage(bool cluster, int width, int v) {
 
 template <typename T, int V>
 static int sandwich_t(float* residual, const float* delta, int n_partials, long long stride, const float* w_post,
-                      const float* w_next, void* xn, int T_rows, int d, float eps, cudaStream_t st) {
+                      const float* w_next, void* xn, int T_rows, int d, float eps, const NormExtra& extra,
+                      cudaStream_t st) {
   const bool cl = row_cluster(T_rows, d);
   const size_t sm = row_stage(cl, d, V);
   T* x = static_cast<T*>(xn);
   if (cl) {
     BCG_CUDA_CHECK(launch_cluster(sandwich_norm_kernel<T, V, kRowCluster>, dim3(kRowCluster, T_rows), dim3(kRowT),
-                                  kRowCluster, sm, st, residual, delta, n_partials, stride, w_post, w_next, x, d, eps));
+                                  kRowCluster, sm, st, residual, delta, n_partials, stride, w_post, w_next, x, d, eps, extra));
   } else {
     BCG_TRY(ensure_dynamic_smem(reinterpret_cast<const void*>(sandwich_norm_kernel<T, V, 1>), 200 * 1024));
     BCG_CUDA_CHECK(launch_k(sandwich_norm_kernel<T, V, 1>, dim3(T_rows), dim3(kRowT), sm, st, residual, delta, n_partials,
-                            stride, w_post, w_next, x, d, eps));
+                            stride, w_post, w_next, x, d, eps, extra));
   }
   return BCG_OK;
 }
 int sandwich_norm(float* residual, const float* delta, int n_partials, long long partial_stride,
                   const float* w_post, const float* w_next, void* xn, int act_dtype, int T, int d, float eps,
-                  cudaStream_t st) {
+                  const NormExtra& extra, cudaStream_t st) {
   if (!residual || !delta || T <= 0 || d <= 0 || d > 51200 || n_partials < 1 || (w_next && !xn)) {
     set_last_error("bcg_sandwich_norm", "bad argument (d <= 51200)");
     return BCG_ERR_ARG;
   }
-  BCG_BY_TYPE(sandwich_t, d, act_dtype, residual, delta, n_partials, partial_stride, w_post, w_next, xn, T, d, eps, st);
+  BCG_BY_TYPE(sandwich_t, d, act_dtype, residual, delta, n_partials, partial_stride, w_post, w_next, xn, T, d, eps, extra,
+              st);
 }
 
 template <typename T, int V>

@@ -42,8 +42,8 @@ struct FlagScope {
   ~FlagScope() { launch_flags() = saved; }
 };
 
-// Attention of one layer over the step's queries; `gathered` remembers whose cache rows ws->latents holds.
-static int attention(const bcg_stack* m, const bcg_stack_ws* ws, const bcg_step_batch* b, const bcg_layer* l,
+// Latent attention of one layer over the step's queries; `gathered` remembers whose cache rows ws->latents holds.
+static int latent_mix(const bcg_stack* m, const bcg_stack_ws* ws, const bcg_step_batch* b, const bcg_layer* l,
                      int mode, const void** gathered, cudaStream_t st) {
   const int n_single = b->single_rows ? b->n_single : (b->n_tiles > 0 ? 0 : b->T);
   const bool bf16 = m->act_dtype == BCG_DT_BF16 && mode == 0;
@@ -79,7 +79,69 @@ int latent_attention(const bcg_stack* m, const bcg_stack_ws* ws, const bcg_step_
     return BCG_ERR_ARG;
   }
   const void* gathered = nullptr;
-  return attention(m, ws, b, &m->layers[layer], mode, &gathered, st);
+  return latent_mix(m, ws, b, &m->layers[layer], mode, &gathered, st);
+}
+
+static const bcg_layer* layer_of(const bcg_stack* m, int layer, bool fits, const char* what) {
+  if (!fits || layer < 0 || layer >= m->n_layers || m->layers[layer].mixer != BCG_MIXER_GROUPED_ATTN) {
+    set_last_error(what, "not a grouped attention layer");
+    return nullptr;
+  }
+  return &m->layers[layer];
+}
+
+int grouped_in_step(const bcg_stack* m, const bcg_stack_ws* ws, const bcg_step_batch* b, int layer, int n_partials,
+                    long long pstride, long long ld, int with_act, cudaStream_t st) {
+  BCG_TRY(check_stack(m, ws));
+  const bcg_layer* l = layer_of(m, layer, b && b->T > 0 && b->T <= ws->T_max && n_partials > 0, "bcg_grouped_in");
+  return l ? grouped_in(m, l, ws, b, n_partials, pstride, ld, with_act != 0, st) : static_cast<int>(BCG_ERR_ARG);
+}
+
+int grouped_attention_step(const bcg_stack* m, const bcg_stack_ws* ws, const bcg_step_batch* b, int layer, int mode,
+                           cudaStream_t st) {
+  BCG_TRY(check_stack(m, ws));
+  const bcg_layer* l = layer_of(m, layer, b && b->T > 0 && b->T <= ws->T_max, "bcg_grouped_attention");
+  return l ? grouped_attention(m, ws, b, l, mode, st) : static_cast<int>(BCG_ERR_ARG);
+}
+
+int experts_step(const bcg_stack* m, const bcg_stack_ws* ws, int layer, int T, int* splits, cudaStream_t st) {
+  BCG_TRY(check_stack(m, ws));
+  const bcg_layer* l = layer_of(m, layer, T > 0 && T <= ws->T_max && splits, "bcg_experts");
+  if (l && l->experts <= 0) set_last_error("bcg_experts", "the layer has no experts");
+  return l && l->experts > 0 ? experts(m, l, ws, T, splits, st) : static_cast<int>(BCG_ERR_ARG);
+}
+
+// A parallel layer: attention and feed-forward read one norm, their outputs meet in one residual addition.  The
+// input projection holds q | k | v (| router) and, behind them, a dense feed-forward's up rows; attention output and
+// activations lie side by side in ws->mix, so that one product applies both output matrices.
+static int parallel_layer(const bcg_stack* m, const bcg_stack_ws* ws, const bcg_step_batch* b, const bcg_layer* l,
+                          const float* next, cudaStream_t st) {
+  const int T = b->T, d = m->d_model, dt = m->act_dtype;
+  const size_t size = dt == BCG_DT_F32 ? 4 : 2;
+  int s = 1;
+  // long launches: the squared relu is the up product's epilogue
+  const int n_up = l->n_in - l->n_qkv;
+  const bool apart = l->ff > 0 && T > 128 && tensor_gemm(dt, T, n_up, d) && tensor_gemm(dt, T, l->n_qkv, d);
+  const int n_in = apart ? l->n_qkv : l->n_in;
+  BCG_TRY(project(m, ws->xn, l->w_in, ws->proj, ws->proj_floats, T, n_in, d, &s, st));
+  if (apart)
+    BCG_TRY(gemm_bf16_tn(ws->xn, static_cast<const char*>(l->w_in) + static_cast<size_t>(l->n_qkv) * d * 2,
+                         static_cast<char*>(ws->mix) + l->act_col * size, T, n_up, d, d, d, l->mix_ld, BCG_EPI_RELU2, 1,
+                         launch_flags() & BCG_GEMM_PDL, st));
+  BCG_TRY(grouped_in(m, l, ws, b, s, static_cast<long long>(T) * n_in, n_in, !apart, st));
+  NormExtra extra;
+  extra.bias = l->out_bias;
+  if (l->experts > 0) {
+    BCG_TRY(experts(m, l, ws, T, &extra.n_partials, st));
+    extra.rows = ws->moe_out;
+    extra.index = ws->moe_row;
+    extra.per_row = l->top;
+    extra.partial_stride = static_cast<long long>(T) * l->top * d;
+  }
+  BCG_TRY(grouped_attention(m, ws, b, l, 0, st));
+  BCG_TRY(project(m, ws->mix, l->w_out, ws->proj, ws->proj_floats, T, d, l->mix_ld, &s, st));
+  return sandwich_norm(ws->residual, ws->proj, s, static_cast<long long>(T) * d, nullptr, next, ws->xn, dt, T, d, m->eps,
+                       extra, st);
 }
 
 int stack_step(const bcg_stack* m, const bcg_stack_ws* ws, const bcg_step_batch* b, cudaStream_t st) {
@@ -92,10 +154,19 @@ int stack_step(const bcg_stack* m, const bcg_stack_ws* ws, const bcg_step_batch*
   FlagScope scope(b->flags & BCG_GEMM_PDL);
   const int T = b->T, d = m->d_model, dt = m->act_dtype;
   const void* gathered = nullptr;
-  BCG_TRY(embed_norm(b->ids, m->embed, m->layers[0].norm1, ws->residual, ws->xn, dt, T, d, m->eps, st));
+  BCG_TRY(embed_norm(b->ids, m->embed, b->positions, m->pos_embed, m->n_pos, m->layers[0].norm1, ws->residual, ws->xn, dt,
+                     T, d, m->eps, ws->moe_counts, ws->moe_counts_n, st));
   for (int i = 0; i < m->n_layers; ++i) {
     const bcg_layer* l = &m->layers[i];
     const float* next = i + 1 < m->n_layers ? m->layers[i + 1].norm1 : m->final_norm;
+    if (l->parallel) {
+      if (l->mixer != BCG_MIXER_GROUPED_ATTN) {
+        set_last_error("bcg_stack_step", "parallel layers have grouped attention");
+        return BCG_ERR_UNSUPPORTED;
+      }
+      BCG_TRY(parallel_layer(m, ws, b, l, next, st));
+      continue;
+    }
     int s = 1, mix_out = 0;
     BCG_TRY(project(m, ws->xn, l->w_in, ws->proj, ws->proj_floats, T, l->n_in, d, &s, st));
     const long long in_stride = static_cast<long long>(T) * l->n_in;
@@ -103,7 +174,7 @@ int stack_step(const bcg_stack* m, const bcg_stack_ws* ws, const bcg_step_batch*
       mix_out = l->heads * l->vdim;
       BCG_TRY(latent_qkv(l, ws->proj, s, in_stride, b->positions, b->slot_map, ws->q, dt, T, m->eps, st));
       if (gathered == l->cache && l->owns_cache) gathered = nullptr;
-      BCG_TRY(attention(m, ws, b, l, 0, &gathered, st));
+      BCG_TRY(latent_mix(m, ws, b, l, 0, &gathered, st));
     } else if (l->mixer == BCG_MIXER_GENERAL_DELTA) {
       mix_out = l->heads * l->dim;
       int sd = 1;
@@ -118,13 +189,13 @@ int stack_step(const bcg_stack* m, const bcg_stack_ws* ws, const bcg_step_batch*
     }
     BCG_TRY(project(m, ws->mix, l->w_out, ws->proj, ws->proj_floats, T, d, mix_out, &s, st));
     BCG_TRY(sandwich_norm(ws->residual, ws->proj, s, static_cast<long long>(T) * d, l->norm1b, l->ff ? l->norm2 : next,
-                          ws->xn, dt, T, d, m->eps, st));
+                          ws->xn, dt, T, d, m->eps, {}, st));
     if (l->ff) {
       BCG_TRY(project(m, ws->xn, l->w_up, ws->proj, ws->proj_floats, T, l->ff, d, &s, st));
       BCG_TRY(poly_norm(ws->proj, s, static_cast<long long>(T) * l->ff, l->act_coef, ws->act, dt, T, l->ff, m->eps, st));
       BCG_TRY(project(m, ws->act, l->w_down, ws->proj, ws->proj_floats, T, d, l->ff, &s, st));
       BCG_TRY(sandwich_norm(ws->residual, ws->proj, s, static_cast<long long>(T) * d, l->norm2b, next, ws->xn, dt, T, d,
-                            m->eps, st));
+                            m->eps, {}, st));
     }
   }
   return BCG_OK;

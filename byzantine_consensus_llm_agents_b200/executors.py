@@ -24,7 +24,7 @@ import torch
 
 from . import lib as L
 from .model import ModelHandle
-from .stack import GeneralDelta, LatentAttention, StackHandle
+from .stack import GeneralDelta, GroupedAttention, LatentAttention, MoeMlp, StackHandle
 
 PAGE = 16
 SPLIT_TOKENS = 256
@@ -181,7 +181,7 @@ class DenseExecutor:
 
 
 class StackExecutor:
-    """Layer stacks: latent pages for attention layers, fp32 state slots for recurrent ones."""
+    """Layer stacks: latent or key/value pages for attention layers, fp32 state slots for recurrent ones."""
 
     def __init__(self, cfg, weights, dev, *, max_rows: int, T_max: int, max_model_len: int, logit_rows: int, flags: int):
         self.lib, self.cfg, self.lcfg, self.dev, self.flags = L.load(), cfg, cfg, dev, flags
@@ -192,25 +192,41 @@ class StackExecutor:
         act, f32, bf = cfg.torch_dtype, torch.float32, torch.bfloat16
         T, D, d = T_max, max_rows, cfg.d_model
         attn = [l.mixer for l in cfg.layers if isinstance(l.mixer, LatentAttention)]
+        grouped = [l.mixer for l in cfg.layers if isinstance(l.mixer, GroupedAttention)]
         delta = [l.mixer for l in cfg.layers if isinstance(l.mixer, GeneralDelta)]
-        mlps = [l.mlp for l in cfg.layers if l.mlp]
+        mlps = [l.mlp for l in cfg.layers if l.mlp and not l.parallel]
+        moes = [l.mlp for l in cfg.layers if isinstance(l.mlp, MoeMlp)]
         top = lambda xs: max([8, *xs])
         self.history = min(cfg.max_window - 1 if cfg.max_window else max_model_len, max_model_len)
         expanded = [m for m in attn if m.q_ld and cfg.act_dtype == "bfloat16"]
         self.K_max = T + min(T, max_rows * self.history) if expanded else 0
         wide = act == bf
         shapes = [(cfg.in_rows(i), d) for i in range(cfg.n_layers)]
-        for l in cfg.layers:
-            shapes += [(d, l.mixer.out_dim)] + ([(l.mlp.ff, d), (d, l.mlp.ff)] if l.mlp else [])
+        for i, l in enumerate(cfg.layers):
+            shapes += [(d, cfg.mix_cols(i)[1])] + ([(l.mlp.ff, d), (d, l.mlp.ff)] if l.mlp in mlps else [])
         slabs = lambda n, k: min(T, 128) * n * (L.splits_for(1, n, k) if wide else 1)
         proj = max([T * n for n, _ in shapes] + [slabs(n, k) for n, k in shapes])
         dec = max([8] + [max(T * m.out_dim, slabs(m.out_dim, m.rank_ld)) for m in delta])
         chunks = lambda m: min((min(m.window or max_model_len, max_model_len)) // 64 + 2, (max_model_len + 63) // 64)
         part = top(D * chunks(m) * m.heads * m.kv_rank for m in attn) if wide else 8
+        # experts: rows are (token, choice) pairs; long bf16 launches keep gate and up in the GEMM's epilogue
+        choices = max([m.top for m in moes], default=0)
+        cut = lambda m, n, k: min(T, 128) * m.top * n * (L.splits_for(1, m.top * n, k) if wide else 1)
+        moe_in = top([cut(m, 2 * m.ff_ld, d) for m in moes] + [T * m.top * 2 * m.ff_ld for m in moes
+                                                             if not (wide and d % 8 == 0 and m.experts <= L.MAX_GROUPS)])
+        moe_out = top([max(T * m.top * d, cut(m, d, m.ff_ld)) for m in moes])
+        counts = sum(m.experts for m in moes)
         z = lambda n, dt: torch.zeros(int(n), dtype=dt, device=dev)
         self.buf = b = dict(
             residual=z(T * d, f32), xn=z(T * d, act), proj=z(proj, f32), decay=z(dec, f32),
-            q=z(T * top(m.heads * m.q_row for m in attn), act), mix=z(T * top(l.mixer.out_dim for l in cfg.layers), act),
+            q=z(T * top(m.heads * m.q_row for m in attn + grouped), act),
+            mix=z(T * top(cfg.mix_cols(i)[1] for i in range(cfg.n_layers)), act),
+            v_first=z(T * top(m.kv_heads * m.vdim for m in grouped if m.v_mix), f32),
+            moe_x=z(max(8, T * choices * d), act), moe_h=z(max(8, T * top(m.top * m.ff_ld for m in moes)), act),
+            moe_proj=z(moe_in, f32), moe_out=z(moe_out, f32), moe_expert=z(T * choices + 8, torch.int32),
+            moe_rank=z(T * choices + 8, torch.int32), moe_weight=z(T * choices + 8, f32),
+            moe_row=z(T * choices + 8, torch.int32), moe_row_weight=z(T * choices + 8, f32),
+            moe_counts=z(counts + 8, torch.int32),
             act=z(T * top(m.ff for m in mlps), act), low=z(T * top(m.rank_ld for m in delta), act),
             latents=z(max(8, self.K_max * top(m.cache_row for m in expanded)), bf),
             expanded=z(max(8, self.K_max * top(m.heads * (m.q_ld + m.v_ld) for m in expanded)), bf),
@@ -222,6 +238,7 @@ class StackExecutor:
         for n in b:
             setattr(ws, n, b[n].data_ptr())
         ws.proj_floats, ws.decay_floats, ws.part_floats = proj, dec, part
+        ws.moe_proj_floats, ws.moe_out_floats, ws.moe_counts_n, ws.moe_rows_max = moe_in, moe_out, counts, T * choices
         ws.T_max, ws.K_max, ws.D_max, ws.B_max = T, self.K_max, D, self.B_max
         self.ws = ws
         self.page_bytes = PAGE * cfg.kv_bytes_per_token
@@ -236,6 +253,9 @@ class StackExecutor:
             m = l.mixer
             if isinstance(m, GeneralDelta):
                 t = torch.zeros(slots, m.heads, m.dim, m.dim, dtype=torch.float32, device=self.dev)
+            elif isinstance(m, GroupedAttention):
+                t = tuple(torch.zeros(pages, m.kv_heads, PAGE, n, dtype=self.cfg.torch_dtype, device=self.dev)
+                          for n in (m.q_ld, m.v_ld))
             else:
                 t = torch.zeros(pages, PAGE, m.cache_row, dtype=self.cfg.torch_dtype, device=self.dev) \
                     if m.kv_from is None else None
@@ -270,7 +290,7 @@ class StackExecutor:
                 continue
             k0 = max(0, e.start - self.history)
             for q0 in range(0, n, PREFILL_TILE):
-                tiles.append((starts[s] + q0, e.start + q0, min(PREFILL_TILE, n - q0), n_gather, k0, 0, 0, 0))
+                tiles.append((starts[s] + q0, e.start + q0, min(PREFILL_TILE, n - q0), n_gather, k0, s, 0, 0))
             keys = np.arange(k0, e.start + n)
             gather.append(e.block_row[keys // PAGE].astype(np.int64) * PAGE + keys % PAGE)
             n_gather += len(keys)
@@ -313,6 +333,9 @@ class StackExecutor:
     def _launches_per_step(self) -> int:
         n = 1
         for l in self.cfg.layers:
+            if l.parallel:   # input projection, its split, attention, output projection, norm; scatter, two products, gate
+                n += 5 + (4 if isinstance(l.mlp, MoeMlp) else 0)
+                continue
             # input projection, mixer (delta: low rank, decay projection, scan; attention: qkv, absorb, decode,
             # combine, up), output projection, norm; feed-forward: up, activation, down, norm
             n += (6 if isinstance(l.mixer, GeneralDelta) else 8) + (4 if l.mlp else 0)

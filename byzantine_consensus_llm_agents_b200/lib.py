@@ -12,14 +12,16 @@ from pathlib import Path
 PKG = Path(__file__).resolve().parent
 LIB_PATH = PKG / "_lib" / "libbcg_b200.so"
 
-EPI_BF16, EPI_F32, EPI_SWIGLU = 0, 1, 2
+EPI_BF16, EPI_F32, EPI_SWIGLU, EPI_RELU2 = 0, 1, 2, 3
 GEMM_PDL = 1
 STEP_FUSED_NORM = 0x20000   # bcg_model_decode: fold add+RMSNorm into the GEMMs (opt-in, slower)
 STEP_FUSED_ROPE = 0x80000     # bcg_model_decode: qk-norm/RoPE/KV-write folded into decode attention
 STEP_DEFERRED_NORM = 0x40000  # bcg_model_decode: norm statistics kernel + 1/RMS in the next GEMM's epilogue
 
 DT_BF16, DT_F32 = 0, 1                          # activation dtype of a layer stack
-MIXER_LATENT_ATTN, MIXER_GENERAL_DELTA = 1, 2
+MIXER_LATENT_ATTN, MIXER_GENERAL_DELTA, MIXER_GROUPED_ATTN = 1, 2, 3
+MAX_GROUPS = 512                                # experts the grouped tensor-core GEMM takes
+VALUES_FIRST, VALUES_MIX = 1, 2                 # Layer.v_role
 
 c_int_p = C.POINTER(C.c_int)
 c_float_p = C.POINTER(C.c_float)
@@ -89,6 +91,11 @@ class Layer(C.Structure):
         ("norm2", vp), ("norm2b", vp), ("w_in", vp), ("w_out", vp), ("latent_norm", vp), ("sink", vp),
         ("cos_sin", vp), ("w_uk", vp), ("w_uv", vp), ("w_expand", vp), ("decay_bias", vp), ("rate_bias", vp),
         ("out_norm", vp), ("w_decay", vp), ("w_up", vp), ("w_down", vp), ("act_coef", vp), ("cache", vp),
+        ("parallel", C.c_int), ("kv_heads", C.c_int), ("temp_coef", C.c_float), ("temp_every", C.c_float),
+        ("v_role", C.c_int), ("v_mix", C.c_float), ("n_qkv", C.c_int), ("act_col", C.c_int), ("mix_ld", C.c_int),
+        ("router_col", C.c_int), ("experts", C.c_int), ("top", C.c_int), ("expert_ld", C.c_int),
+        ("glu_limit", C.c_float), ("glu_alpha", C.c_float), ("moe_counts_at", C.c_int), ("slopes", vp),
+        ("in_bias", vp), ("out_bias", vp), ("w_experts_in", vp), ("w_experts_out", vp), ("cache_v", vp),
     ]
 
 
@@ -96,7 +103,7 @@ class Stack(C.Structure):
     _fields_ = [
         ("n_layers", C.c_int), ("d_model", C.c_int), ("vocab_ld", C.c_int), ("act_dtype", C.c_int),
         ("page_size", C.c_int), ("eps", C.c_float), ("embed", vp), ("lm_head", vp), ("final_norm", vp),
-        ("layers", C.POINTER(Layer)),
+        ("layers", C.POINTER(Layer)), ("pos_embed", vp), ("n_pos", C.c_int),
     ]
 
 
@@ -106,7 +113,10 @@ class StackWs(C.Structure):
         ("decay_floats", C.c_longlong), ("q", vp), ("mix", vp), ("act", vp), ("low", vp), ("latents", vp),
         ("expanded", vp), ("q_latent", vp), ("o_latent", vp), ("part_o", vp), ("part_floats", C.c_longlong),
         ("part_ml", vp), ("xn_rows", vp), ("logits", vp), ("T_max", C.c_int), ("K_max", C.c_int),
-        ("D_max", C.c_int), ("B_max", C.c_int),
+        ("D_max", C.c_int), ("B_max", C.c_int), ("v_first", vp), ("moe_x", vp), ("moe_h", vp), ("moe_proj", vp),
+        ("moe_proj_floats", C.c_longlong), ("moe_out", vp), ("moe_out_floats", C.c_longlong), ("moe_expert", vp),
+        ("moe_rank", vp), ("moe_weight", vp), ("moe_row", vp), ("moe_row_weight", vp), ("moe_counts", vp),
+        ("moe_counts_n", C.c_int), ("moe_rows_max", C.c_int),
     ]
 
 
@@ -165,11 +175,18 @@ _SIGS = {
                                C.c_longlong, vp]),
     "bcg_sandwich_norm": (C.c_int, [vp, vp, C.c_int, C.c_longlong, vp, vp, vp, C.c_int, C.c_int, C.c_int, C.c_float,
                                     vp]),
+    "bcg_residual_norm": (C.c_int, [vp, vp, C.c_int, C.c_longlong, vp, vp, vp, C.c_int, C.c_int, C.c_longlong, vp, vp,
+                                    C.c_int, C.c_int, C.c_int, C.c_float, vp]),
     "bcg_poly_norm": (C.c_int, [vp, C.c_int, C.c_longlong, vp, vp, C.c_int, C.c_int, C.c_int, C.c_float, vp]),
     "bcg_delta_scan": (C.c_int, [C.POINTER(Layer), vp, C.c_int, C.c_longlong, C.c_longlong, vp, C.c_int,
                                  C.c_longlong, vp, vp, vp, vp, C.c_int, vp, C.c_int, C.c_float, vp]),
     "bcg_latent_attention": (C.c_int, [C.POINTER(Stack), C.POINTER(StackWs), C.POINTER(StepBatch), C.c_int, C.c_int,
                                        vp]),
+    "bcg_grouped_in": (C.c_int, [C.POINTER(Stack), C.POINTER(StackWs), C.POINTER(StepBatch), C.c_int, C.c_int,
+                                 C.c_longlong, C.c_longlong, C.c_int, vp]),
+    "bcg_grouped_attention": (C.c_int, [C.POINTER(Stack), C.POINTER(StackWs), C.POINTER(StepBatch), C.c_int, C.c_int,
+                                        vp]),
+    "bcg_experts": (C.c_int, [C.POINTER(Stack), C.POINTER(StackWs), C.c_int, C.c_int, c_int_p, vp]),
 }
 
 EXPORTED = tuple(_SIGS)

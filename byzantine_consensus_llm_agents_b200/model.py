@@ -79,6 +79,9 @@ PRESETS = {
     # layer stacks (stack.py) at the widths of the dense presets beside them
     "bekopel-1b": stack.bekopel_preset("bekopel-1b", 16, 2048, 7424, 151936, heads=16),
     "bekopel-8b": stack.bekopel_preset("bekopel-8b", 36, 4096, 14592, 151936),
+    "lerazen-8b": stack.lerazen_preset("lerazen-8b", 36, 4096, 18432, 151936),
+    "lerazen-30b-a3b": stack.lerazen_preset("lerazen-30b-a3b", 48, 2048, 6144, 151936, kv_heads=4, experts=128, top=8,
+                                            expert_ff=768),
 }
 
 _HF_NAMES = {

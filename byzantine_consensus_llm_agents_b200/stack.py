@@ -1,7 +1,8 @@
 """Layer stacks: models whose layers differ in kind, described by composable specs.
 
-A `StackConfig` lists layers; each has a mixer spec (`LatentAttention`, `GeneralDelta`), optionally a
-feed-forward spec (`DenseMlp`), and norms before and after every sublayer.  Which design a model directory
+A `StackConfig` lists layers; each has a mixer spec (`LatentAttention`, `GeneralDelta`, `GroupedAttention`),
+optionally a feed-forward spec (`DenseMlp`, `MoeMlp`), and either norms before and after every sublayer or, in a
+parallel layer, one norm in front of both.  Which design a model directory
 holds is decided by config.json's "architecture" (`DESIGNS`, consulted by model.config_from_dir); a design is
 a reader from its config.json to specs, everything below the specs is shared.  `StackWeights` loads and packs
 the tensors for the kernels (include/bcg_b200.h, bcg_layer); there is nothing model-specific in the engine.
@@ -111,18 +112,93 @@ class GeneralDelta:
 
 
 @dataclass(frozen=True)
-class DenseMlp:
-    """down(PolyNorm(up(x))); the activation's four numbers are weights."""
-    ff: int
+class GroupedAttention:
+    """Grouped-query attention without rotation: a linear distance bias per head, biased projections, queries
+    scaled by 1 + temp_coef * ln(floor((position + 1) / temp_every) + 1)."""
+    heads: int
+    kv_heads: int
+    dim: int
+    vdim: int
+    scale: float
+    window: int = 0                 # keys a query sees, itself included; 0 = all
+    temp_coef: float = 0.0
+    temp_every: float = 1.0
+    v_mix: bool = False             # the first such layer's values are mixed into the later ones'
+    slopes: bool = True             # distance slope 2^(-8 (h + 1) / heads) of head h
+
+    @property
+    def out_dim(self) -> int:
+        return self.heads * self.vdim
+
+    @property
+    def q_ld(self) -> int:
+        """Columns of a head in the query buffer and the key pages."""
+        return _up(self.dim, 64) if self.dim <= 256 else _up(self.dim, 8)
+
+    @property
+    def v_ld(self) -> int:
+        return next((v for v in (64, 128, 256) if self.vdim <= v), _up(self.vdim, 8))
+
+    q_row = q_ld
+
+    @property
+    def cache_row(self) -> int:
+        """Cache elements of one token."""
+        return self.kv_heads * (self.q_ld + self.v_ld)
+
+    @property
+    def in_dim(self) -> int:
+        return self.heads * self.dim + self.kv_heads * (self.dim + self.vdim)
 
     def tensors(self, d: int) -> Dict[str, tuple]:
-        return {"up": (self.ff, d), "down": (d, self.ff), "act": (4,)}
+        out = {}
+        for n, rows, cols in (("q", self.heads * self.dim, d), ("k", self.kv_heads * self.dim, d),
+                              ("v", self.kv_heads * self.vdim, d), ("o", d, self.out_dim)):
+            out.update({n: (rows, cols), n + ".b": (rows,)})
+        if self.v_mix:
+            out["vmix"] = ()
+        return out
+
+
+@dataclass(frozen=True)
+class DenseMlp:
+    """down(act(up(x))); act is PolyNorm, whose four numbers are weights, or the square of relu."""
+    ff: int
+    act: str = "poly_norm"          # or "relu2"
+
+    def tensors(self, d: int) -> Dict[str, tuple]:
+        t = {"up": (self.ff, d), "down": (d, self.ff)}
+        if self.act == "poly_norm":
+            t["act"] = (4,)
+        return t
+
+
+@dataclass(frozen=True)
+class MoeMlp:
+    """`experts` gated units (gate clamped from above, linear part from both sides, sigmoid(alpha * gate)), of which
+    a token uses the `top` with the largest sigmoid scores; a score scales its expert's input."""
+    experts: int
+    top: int
+    ff: int
+    limit: float
+    alpha: float = 1.702
+
+    @property
+    def ff_ld(self) -> int:
+        return _up(self.ff, 16)
+
+    def tensors(self, d: int) -> Dict[str, tuple]:
+        t = {"router": (self.experts, d)}
+        for e in range(self.experts):
+            t.update({f"e{e}.gate": (self.ff, d), f"e{e}.up": (self.ff, d), f"e{e}.down": (d, self.ff)})
+        return t
 
 
 @dataclass(frozen=True)
 class LayerSpec:
     mixer: object
-    mlp: Optional[DenseMlp] = None
+    mlp: object = None
+    parallel: bool = False          # x += mixer(h) + ff(h) with one norm h of x
 
 
 @dataclass(frozen=True)
@@ -135,12 +211,26 @@ class StackConfig:
     act_dtype: str = "bfloat16"      # or "float32": everything in true fp32
     family: str = "qwen3"            # tokenizer / chat-template family
     max_pos: int = 131072
+    learned_pos: bool = False        # max_pos position vectors are added to the embedding
 
     def __post_init__(self):
         if self.act_dtype not in ("bfloat16", "float32"):
             raise ValueError(f"act_dtype {self.act_dtype!r}")
         for i, l in enumerate(self.layers):
             m = l.mixer
+            if l.parallel != isinstance(m, GroupedAttention) or isinstance(l.mlp, MoeMlp) and not l.parallel:
+                raise ValueError(f"{self.name}: layer {i}: grouped attention and experts come in parallel layers, and only there")
+            if l.mlp and isinstance(l.mlp, DenseMlp) and (l.mlp.act == "relu2") != l.parallel:
+                raise ValueError(f"{self.name}: layer {i}: activation {l.mlp.act!r} in this kind of layer")
+            if isinstance(l.mlp, MoeMlp) and not 0 < l.mlp.top <= l.mlp.experts:
+                raise ValueError(f"{self.name}: layer {i}: {l.mlp.top} of {l.mlp.experts} experts")
+            if isinstance(m, GroupedAttention):
+                if m.heads % m.kv_heads:
+                    raise ValueError(f"{self.name}: layer {i}: {m.heads} query heads on {m.kv_heads} key/value heads")
+                if m.v_mix:
+                    f = self.layers[self.v_first].mixer
+                    if (f.kv_heads, f.vdim) != (m.kv_heads, m.vdim):
+                        raise ValueError(f"{self.name}: layer {i} cannot mix in values of layer {self.v_first}")
             if isinstance(m, GeneralDelta) and m.dim > 256:
                 raise ValueError(f"{self.name}: layer {i}: the delta-rule kernel takes up to 256 channels per head")
             if isinstance(m, LatentAttention):
@@ -157,6 +247,11 @@ class StackConfig:
         return len(self.layers)
 
     @property
+    def v_first(self) -> Optional[int]:
+        """The layer whose values later layers mix in."""
+        return next((i for i, l in enumerate(self.layers) if getattr(l.mixer, "v_mix", False)), None)
+
+    @property
     def vocab_ld(self) -> int:
         return _up(self.vocab, 4)
 
@@ -168,7 +263,7 @@ class StackConfig:
     @property
     def max_window(self) -> int:
         """Largest attention window of the stack, 0 = unbounded."""
-        w = [l.mixer.window for l in self.layers if isinstance(l.mixer, LatentAttention)]
+        w = [l.mixer.window for l in self.layers if not isinstance(l.mixer, GeneralDelta)]
         return 0 if not w or 0 in w else max(w)
 
     @property
@@ -182,7 +277,7 @@ class StackConfig:
     @property
     def kv_bytes_per_token(self) -> int:
         return sum(l.mixer.cache_row for l in self.layers
-                   if isinstance(l.mixer, LatentAttention) and l.mixer.kv_from is None) * self.itemsize
+                   if not isinstance(l.mixer, GeneralDelta) and getattr(l.mixer, "kv_from", None) is None) * self.itemsize
 
     @property
     def state_bytes_per_row(self) -> int:
@@ -190,24 +285,51 @@ class StackConfig:
 
     def in_rows(self, i: int) -> int:
         """Rows of layer i's fused input projection, padded for the 256-wide GEMM tiles when it is large."""
+        if self.layers[i].parallel:
+            return self.qkv_rows(i) + self.up_rows(i)
         n = self.layers[i].mixer.in_rows()
         return _up(n, 256 if n >= 2048 else 16)
+
+    def qkv_rows(self, i: int) -> int:
+        """Parallel layers: padded rows of q | k | v | router."""
+        f = self.layers[i].mlp
+        n = self.layers[i].mixer.in_dim + (f.experts if isinstance(f, MoeMlp) else 0)
+        return _up(n, 32 if n >= 2048 else 16)
+
+    def up_rows(self, i: int) -> int:
+        """Parallel layers: padded rows of a dense feed-forward's up matrix, behind the rows above."""
+        f = self.layers[i].mlp
+        return _up(f.ff, 32 if f.ff >= 2048 else 16) if isinstance(f, DenseMlp) else 0
+
+    def mix_cols(self, i: int) -> Tuple[int, int]:
+        """(first activation column, columns) of what layer i's output projection reads."""
+        n = self.layers[i].mixer.out_dim
+        return (_up(n, 8), _up(n, 8) + self.up_rows(i)) if self.layers[i].parallel else (n, n)
 
     def tensor_shapes(self) -> Dict[str, tuple]:
         """Every tensor of the checkpoint, name -> shape."""
         d = self.d_model
         out = {"embed": (self.vocab, d), "final.norm": (d,), "head": (self.vocab, d)}
+        if self.learned_pos:
+            out["pos"] = (self.max_pos, d)
         for i, l in enumerate(self.layers):
-            out.update({f"l{i}.norm1": (d,), f"l{i}.norm1b": (d,)})
+            norms = ("norm1",) if l.parallel else ("norm1", "norm1b") + (("norm2", "norm2b") if l.mlp else ())
+            out.update({f"l{i}.{n}": (d,) for n in norms})
             out.update({f"l{i}.mix.{n}": s for n, s in l.mixer.tensors(d).items()})
             if l.mlp:
-                out.update({f"l{i}.norm2": (d,), f"l{i}.norm2b": (d,)})
                 out.update({f"l{i}.mlp.{n}": s for n, s in l.mlp.tensors(d).items()})
         return out
 
-    def decode_weight_bytes(self) -> int:
-        """bf16 bytes of matrices streamed per decode step."""
-        return 2 * sum(s[0] * s[1] for n, s in self.tensor_shapes().items() if len(s) == 2 and n != "embed")
+    def decode_weight_bytes(self, rows: Optional[int] = None) -> int:
+        """bf16 bytes of matrices streamed per decode step of `rows` tokens: experts by the number that so many tokens
+        use on average when they choose at random (None: all of them)."""
+        total = 0.0
+        for n, s in self.tensor_shapes().items():
+            if len(s) == 2 and n not in ("embed", "pos"):
+                f = self.layers[int(n[1:n.index(".")])].mlp if ".mlp.e" in n else None
+                used = 1.0 - (1.0 - f.top / f.experts) ** rows if f and rows is not None else 1.0
+                total += 2 * s[0] * s[1] * used
+        return round(total)
 
     def shard(self, tp_size: int) -> "StackConfig":
         if tp_size != 1:
@@ -239,7 +361,33 @@ def _bekopel(c: dict, shape: Callable[[str], tuple], name: str) -> StackConfig:
                        rms_eps=float(c["norm"]["eps"]))
 
 
-DESIGNS: Dict[str, Callable] = {"Bekopel": _bekopel}
+def _lerazen(c: dict, shape: Callable[[str], tuple], name: str) -> StackConfig:
+    """config.json of the Lerazen design."""
+    layers = []
+    for i, e in enumerate(c["layers"]):
+        m, kind = e["mixer"], e["type"]
+        if kind != "attention":
+            raise ValueError(f"{name}: layer {i}: unknown mixer {kind!r}")
+        temp = m.get("q_temp") or {"coef": 0.0, "every": 1}
+        mixer = GroupedAttention(heads=int(m["heads"]), kv_heads=int(m["kv_heads"]), dim=int(m["dim"]), vdim=int(m["vdim"]),
+                                 scale=float(m["scale"]), window=int((m.get("mask") or {"size": 0})["size"]),
+                                 temp_coef=float(temp["coef"]), temp_every=float(temp["every"]),
+                                 v_mix=bool(m.get("v_mix", False)))
+        f = e.get("mlp")
+        if f is None:
+            mlp = None
+        elif f.get("kind") == "dense":
+            mlp = DenseMlp(int(f["ff"]), "relu2")
+        elif f.get("kind") == "moe":
+            mlp = MoeMlp(int(f["router"]["experts"]), int(f["router"]["top"]), int(f["expert"]["ff"]), float(f["expert"]["limit"]))
+        else:
+            raise ValueError(f"{name}: layer {i}: unknown feed-forward {f.get('kind')!r}")
+        layers.append(LayerSpec(mixer, mlp, parallel=True))
+    return StackConfig(name=name, d_model=int(c["width"]), vocab=int(c["vocab"]), layers=tuple(layers),
+                       rms_eps=float(c["norm"]["eps"]), max_pos=int(c["max_positions"]), learned_pos=True)
+
+
+DESIGNS: Dict[str, Callable] = {"Bekopel": _bekopel, "Lerazen": _lerazen}
 
 
 def safetensors_shapes(path) -> Dict[str, tuple]:
@@ -279,7 +427,25 @@ def bekopel_preset(name: str, n_layers: int, d_model: int, ff: int, vocab: int, 
     return StackConfig(name, d_model, vocab, tuple(layers), max_pos=max_pos)
 
 
+def lerazen_preset(name: str, n_layers: int, d_model: int, ff: int, vocab: int, heads: int = 32, kv_heads: int = 8,
+                   dim: int = 128, window: int = 1024, experts: int = 0, top: int = 4, expert_ff: int = 1024,
+                   max_pos: int = 32768) -> StackConfig:
+    """Lerazen at sizes of a real model's layers (random-init presets, bench): dense feed-forwards, or, with
+    `experts`, a dense one in the first layer and experts in the others."""
+    m = GroupedAttention(heads, kv_heads, dim, dim, dim ** -0.5, window, 0.1, 8192, True)
+    dense = DenseMlp(ff, "relu2")
+    moe = MoeMlp(experts, top, expert_ff, 7.0) if experts else dense
+    layers = tuple(LayerSpec(m, moe if i else dense, True) for i in range(n_layers))
+    return StackConfig(name, d_model, vocab, layers, max_pos=max_pos, learned_pos=True)
+
+
 # ------------------------------------------------------------------------------------------ weights
+def head_slopes(heads: int, device) -> torch.Tensor:
+    """[heads] fp32 distance slopes 2^(-8 (h + 1) / heads)."""
+    h = torch.arange(1, heads + 1, dtype=torch.float64)
+    return torch.exp2(-8.0 * h / heads).float().to(device)
+
+
 def rope_table(rot: Rotary, n_pos: int, device) -> torch.Tensor:
     """[n_pos, dims] fp32: cos of the dims/2 angles, then sin (angles formed in fp64, rounded once)."""
     half = rot.dims // 2
@@ -296,6 +462,7 @@ class StackWeights:
     lm_head: torch.Tensor
     final_norm: torch.Tensor
     layers: list = field(default_factory=list)
+    pos_embed: Optional[torch.Tensor] = None
 
     @staticmethod
     def from_tensors(cfg: StackConfig, get: Callable[[str], torch.Tensor], device) -> "StackWeights":
@@ -315,8 +482,13 @@ class StackWeights:
             return t if t.shape[0] == n else torch.cat([t, t.new_zeros(n - t.shape[0], *t.shape[1:])])
 
         w = StackWeights(cfg, bf(raw("embed")), bf(rows(raw("head"), cfg.vocab_ld)), f32(raw("final.norm")))
+        if cfg.learned_pos:
+            w.pos_embed = bf(raw("pos"))
         for i, l in enumerate(cfg.layers):
             m, g = l.mixer, lambda n: raw(f"l{i}.mix.{n}")
+            if l.parallel:
+                w.layers.append(StackWeights._parallel(cfg, i, raw, bf, f32, rows))
+                continue
             t = {"norm1": f32(raw(f"l{i}.norm1")), "norm1b": f32(raw(f"l{i}.norm1b")), "w_out": bf(g("o"))}
             if isinstance(m, LatentAttention):
                 own = m.kv_from is None
@@ -339,6 +511,37 @@ class StackWeights:
                          w_down=bf(raw(f"l{i}.mlp.down")), act_coef=f32(raw(f"l{i}.mlp.act")))
             w.layers.append(t)
         return w
+
+    @staticmethod
+    def _parallel(cfg: StackConfig, i: int, raw, bf, f32, rows) -> dict:
+        """A parallel layer: q | k | v | router, then the up rows, in one matrix; o and down side by side in another;
+        experts one after another, gate and up rows interleaved by 16."""
+        l, d = cfg.layers[i], cfg.d_model
+        m, f, dense = l.mixer, l.mlp, isinstance(l.mlp, DenseMlp)
+        g, ffn = lambda n: raw(f"l{i}.mix.{n}"), lambda n: raw(f"l{i}.mlp.{n}")
+        top = [g("q"), g("k"), g("v")] + ([ffn("router")] if isinstance(f, MoeMlp) else [])
+        w_in = rows(torch.cat(top), cfg.qkv_rows(i))
+        act_col, cols = cfg.mix_cols(i)
+        w_out = torch.zeros(d, cols, dtype=torch.bfloat16, device=w_in.device)
+        w_out[:, :m.out_dim] = bf(g("o"))
+        if dense:
+            w_in = torch.cat([w_in, rows(ffn("up"), cfg.up_rows(i))])
+            w_out[:, act_col:act_col + f.ff] = bf(ffn("down"))
+        t = {"norm1": f32(raw(f"l{i}.norm1")), "w_in": bf(w_in), "w_out": w_out, "out_bias": f32(g("o.b")),
+             "in_bias": f32(torch.cat([g("q.b"), g("k.b"), g("v.b")]))}
+        if m.slopes:
+            t["slopes"] = head_slopes(m.heads, w_in.device)
+        if m.v_mix:
+            t["vmix"] = f32(g("vmix"))
+        if isinstance(f, MoeMlp):
+            n = f.ff_ld
+            t["w_experts_in"] = torch.zeros(f.experts, 2 * n, d, dtype=torch.bfloat16, device=w_in.device)
+            t["w_experts_out"] = torch.zeros(f.experts, d, n, dtype=torch.bfloat16, device=w_in.device)
+            for e in range(f.experts):
+                pair = torch.stack([rows(bf(ffn(f"e{e}.{x}")), n).view(n // 16, 16, d) for x in ("gate", "up")], dim=1)
+                t["w_experts_in"][e] = pair.reshape(2 * n, d)
+                t["w_experts_out"][e, :, :f.ff] = bf(ffn(f"e{e}.down"))
+        return t
 
     @staticmethod
     def expansion(m: LatentAttention, uk: torch.Tensor, uv: torch.Tensor) -> torch.Tensor:
@@ -368,6 +571,8 @@ class StackWeights:
             s = shapes[n]
             if n.endswith(".act"):
                 return torch.tensor([1.0, 0.5, 0.25, 0.0], device=device)
+            if n.endswith(".vmix"):
+                return torch.tensor(0.5, device=device)
             if len(s) == 2:
                 return torch.empty(*s, dtype=torch.bfloat16, device=device).normal_(0.0, 0.02, generator=g)
             leaf = n.rsplit(".", 1)[-1]
@@ -375,7 +580,7 @@ class StackWeights:
         return StackWeights.from_tensors(cfg, get, device)
 
     def nbytes(self) -> int:
-        ts = [self.embed, self.lm_head] + [t for l in self.layers for t in l.values()]
+        ts = [self.embed, self.lm_head] + ([self.pos_embed] if self.pos_embed is not None else []) + [t for l in self.layers for t in l.values()]
         return sum(t.numel() * t.element_size() for t in ts)
 
 
@@ -384,7 +589,8 @@ class StackHandle:
     """Host-side bcg_stack (include/bcg_b200.h) over StackWeights, caches and states.
 
     caches[i]: the latent pages [pages, page, cache_row] or the states [slots, heads, dim, dim] of layer i
-    (None where the layer reads another layer's cache)."""
+    (None where the layer reads another layer's cache); for grouped attention a pair (keys [pages, kv_heads, page,
+    q_ld], values [pages, kv_heads, page, v_ld])."""
 
     def __init__(self, w: StackWeights, caches: list, n_pos: int, page_size: int):
         cfg = w.cfg
@@ -392,11 +598,21 @@ class StackHandle:
         dev = w.embed.device
         self._rope: Dict[Rotary, torch.Tensor] = {}
         arr = (L.Layer * cfg.n_layers)()
+        counts = 0
         for i, (spec, t) in enumerate(zip(cfg.layers, w.layers)):
             a, m = arr[i], spec.mixer
             a.heads, a.dim, a.n_in = m.heads, m.dim, cfg.in_rows(i)
             src = i
-            if isinstance(m, LatentAttention):
+            if isinstance(m, GroupedAttention):
+                a.mixer, a.kv_heads, a.vdim, a.q_ld, a.v_ld = L.MIXER_GROUPED_ATTN, m.kv_heads, m.vdim, m.q_ld, m.v_ld
+                a.window, a.scale, a.owns_cache = m.window, m.scale, 1
+                a.temp_coef, a.temp_every = m.temp_coef, m.temp_every
+                if m.v_mix:
+                    a.v_role = L.VALUES_FIRST if i == cfg.v_first else L.VALUES_MIX
+                    a.v_mix = float(t["vmix"])
+                a.parallel, a.n_qkv, a.router_col = 1, cfg.qkv_rows(i), m.in_dim
+                a.act_col, a.mix_ld = cfg.mix_cols(i)
+            elif isinstance(m, LatentAttention):
                 a.mixer = L.MIXER_LATENT_ATTN
                 a.rot_dim, a.rot_dims, a.vdim, a.kv_rank = m.rot_dim, m.rot.dims, m.vdim, m.kv_rank
                 a.window, a.scale, a.owns_cache = m.window, m.scale, int(m.kv_from is None)
@@ -408,14 +624,26 @@ class StackHandle:
                 a.cos_sin = self._rope[m.rot].data_ptr()
             else:
                 a.mixer, a.decay_rank = L.MIXER_GENERAL_DELTA, m.rank_ld
-            a.ff = spec.mlp.ff if spec.mlp else 0
+            if isinstance(spec.mlp, MoeMlp):
+                f = spec.mlp
+                a.experts, a.top, a.expert_ld, a.glu_limit, a.glu_alpha = f.experts, f.top, f.ff_ld, f.limit, f.alpha
+                a.moe_counts_at = counts
+                counts += f.experts
+            else:
+                a.ff = spec.mlp.ff if spec.mlp else 0
             for n, x in t.items():
-                setattr(a, n, x.data_ptr())
-            a.cache = caches[src].data_ptr()
+                if n != "vmix":
+                    setattr(a, n, x.data_ptr())
+            if isinstance(m, GroupedAttention):
+                a.cache, a.cache_v = (c.data_ptr() for c in caches[i])
+            else:
+                a.cache = caches[src].data_ptr()
         self._layers = arr
         s = L.Stack()
         s.n_layers, s.d_model, s.vocab_ld, s.page_size, s.eps = cfg.n_layers, cfg.d_model, cfg.vocab_ld, page_size, cfg.rms_eps
         s.act_dtype = L.DT_F32 if cfg.act_dtype == "float32" else L.DT_BF16
         s.embed, s.lm_head, s.final_norm = w.embed.data_ptr(), w.lm_head.data_ptr(), w.final_norm.data_ptr()
+        if w.pos_embed is not None:
+            s.pos_embed, s.n_pos = w.pos_embed.data_ptr(), w.pos_embed.shape[0]
         s.layers = C.cast(arr, C.POINTER(L.Layer))
         self.struct = s

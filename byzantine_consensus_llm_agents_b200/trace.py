@@ -37,7 +37,8 @@ def build_engine(model_dir: str, dtype: str, max_tokens: int, device: str = "cud
     cfg = M.config_from_dir(model_dir)
     pages = max(1, -(-max_tokens // PAGE))
     if isinstance(cfg, stack.StackConfig):
-        cfg = dataclasses.replace(cfg, act_dtype=dtype, max_pos=max(cfg.max_pos, max_tokens))
+        reach = cfg.max_pos if cfg.learned_pos else max(cfg.max_pos, max_tokens)
+        cfg = dataclasses.replace(cfg, act_dtype=dtype, max_pos=reach)
     elif dtype != "bfloat16":
         return None
     weights = M.weights_for(cfg).from_safetensors_dir(cfg, model_dir, torch.device(device))

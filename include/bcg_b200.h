@@ -35,6 +35,7 @@ extern "C" {
 #define BCG_EPI_BF16 0   /* out bf16 [M, ld_out]                                         */
 #define BCG_EPI_F32 1    /* out fp32 [splits][M, ld_out] (split-K partials, or logits)   */
 #define BCG_EPI_SWIGLU 2 /* W rows interleaved [16 gate | 16 up]; out bf16 [M, N/2]      */
+#define BCG_EPI_RELU2 3  /* out bf16 [M, ld_out] = max(y, 0)^2 (M > 128, N % 16 == 0)    */
 /* GEMM flags */
 #define BCG_GEMM_PDL 1   /* programmatic dependent launch: weights prefetch before the wait */
 
@@ -358,7 +359,8 @@ int bcg_model_decode(const bcg_model* m, const bcg_workspace* ws, const int* ids
 /* ---------------------------------------------------------------------------------------------
  * Layer stacks: models whose layers differ in kind (the reference has no counterpart; its engine
  * only meets uniform dense decoders).  Every layer is a mixer and, optionally, a feed-forward, each
- * with a norm before and a norm after it:  x += norm1b(mixer(norm1(x))),  x += norm2b(ff(norm2(x))).
+ * with a norm before and a norm after it:  x += norm1b(mixer(norm1(x))),  x += norm2b(ff(norm2(x))),
+ * or, `parallel`, both behind one norm:  h = norm1(x),  x += mixer(h) + ff(h).
  * `act_dtype` selects the activations that feed matrix products, the latent cache and the attention
  * operands: BCG_DT_BF16 (tensor-core kernels, fp32 accumulation) or BCG_DT_F32 (true fp32
  * throughout, CUDA-core kernels).  Weights are bf16 in both; the residual, norms, scores, gates and
@@ -367,6 +369,9 @@ int bcg_model_decode(const bcg_model* m, const bcg_workspace* ws, const int* ids
 #define BCG_DT_F32 1
 #define BCG_MIXER_LATENT_ATTN 1
 #define BCG_MIXER_GENERAL_DELTA 2
+#define BCG_MIXER_GROUPED_ATTN 3
+#define BCG_VALUES_FIRST 1   /* bcg_layer.v_role: the layer's values are what later layers mix in */
+#define BCG_VALUES_MIX 2     /* values are (1 - v_mix) of its own and v_mix of those */
 
 typedef struct bcg_layer {
   int mixer;               /* BCG_MIXER_* */
@@ -403,7 +408,28 @@ typedef struct bcg_layer {
   const void* w_down;      /* bf16 [d, ff] */
   const float* act_coef;   /* PolyNorm's four numbers (device) */
   void* cache;             /* latent pages [pages][page_size][kv_rank + rot_dim], or state
-                              fp32 [slots][heads][dim][dim] */
+                              fp32 [slots][heads][dim][dim]; grouped attention: keys
+                              [pages][kv_heads][page_size][q_ld], columns past dim zero */
+  /* grouped attention (parallel layers) and their feed-forward */
+  int parallel;
+  int kv_heads;            /* query head h reads key/value head h / (heads / kv_heads) */
+  float temp_coef, temp_every; /* queries times 1 + temp_coef * ln(floor((position + 1) / temp_every) + 1) */
+  int v_role;              /* 0 or BCG_VALUES_* */
+  float v_mix;
+  int n_qkv;               /* rows of w_in in front of the up rows: q | k | v | router; zero rows after */
+  int act_col, mix_ld;     /* rows of ws->mix: heads * vdim attention columns, ff activations (squared relu) from act_col
+                              on; mix_ld columns of w_out */
+  int router_col;          /* first router row of w_in */
+  int experts, top;        /* mixture of experts; experts = 0: none */
+  int expert_ld;           /* an expert's inner size, padded to a multiple of 16 */
+  float glu_limit, glu_alpha;
+  int moe_counts_at;       /* the layer's place in ws->moe_counts */
+  const float* slopes;     /* [heads] slope * (query position - key position) is taken off the score; NULL = none */
+  const float* in_bias;    /* [q + k + v rows] */
+  const float* out_bias;   /* [d] */
+  const void* w_experts_in;  /* bf16 [experts][2 * expert_ld][d], rows interleaved [16 gate | 16 up] */
+  const void* w_experts_out; /* bf16 [experts][d][expert_ld] */
+  void* cache_v;           /* values [pages][kv_heads][page_size][v_ld], columns past vdim zero */
 } bcg_layer;
 
 typedef struct bcg_stack {
@@ -414,6 +440,8 @@ typedef struct bcg_stack {
   const void* lm_head;      /* bf16 [vocab_ld, d] */
   const float* final_norm;
   const bcg_layer* layers;  /* host array */
+  const void* pos_embed;    /* bf16 [n_pos, d] added to the embedding, or NULL */
+  int n_pos;
 } bcg_stack;
 
 typedef struct bcg_stack_ws {
@@ -437,6 +465,21 @@ typedef struct bcg_stack_ws {
   void* xn_rows;    /* act [B_max, d] */
   float* logits;    /* fp32 [B_max, vocab_ld] */
   int T_max, K_max, D_max, B_max;
+  float* v_first;   /* fp32 [T_max, kv_heads * vdim]: the step's values of the BCG_VALUES_FIRST layer */
+  /* mixture of experts; rows = (token, choice) pairs */
+  void* moe_x;      /* act [moe_rows_max, d] rows sorted by expert */
+  void* moe_h;      /* act [moe_rows_max, expert_ld] */
+  float* moe_proj;  /* fp32 slabs of [rows, 2 * expert_ld] */
+  long long moe_proj_floats;
+  float* moe_out;   /* fp32 slabs of [rows, d] */
+  long long moe_out_floats;
+  int* moe_expert;  /* [T][top] */
+  int* moe_rank;    /* [T][top] */
+  float* moe_weight;     /* [T][top] */
+  int* moe_row;          /* [T][top] sorted row of each choice */
+  float* moe_row_weight; /* [rows] */
+  int* moe_counts;       /* rows per expert, all layers' one after another; cleared at the start of a step */
+  int moe_counts_n, moe_rows_max;
 } bcg_stack_ws;
 
 /* A step: T new tokens of n_seqs sequences, portions of prompts beside single decoded tokens.  All
@@ -456,7 +499,7 @@ typedef struct bcg_step_batch {
   const int* single_rows;  /* [n_single] tokens attended one by one in latent space, NULL = all T */
   int n_single;
   const int* tiles;        /* [n_tiles][8] {first token, its position, tokens (<= 128), expanded row of
-                              key position k0, k0, 0, 0, 0} */
+                              key position k0, k0, sequence, 0, 0} */
   int n_tiles;
   const int* gather;       /* [n_gather] cache row behind every expanded row */
   int n_gather;
@@ -482,6 +525,11 @@ int bcg_gemm_any(const void* X, int x_dtype, const void* W, float* out, int M, i
 int bcg_sandwich_norm(float* residual, const float* delta, int n_partials, long long partial_stride,
                       const float* w_post, const float* w_next, void* xn, int act_dtype, int T, int d, float eps,
                       void* stream);
+/* No counterpart in the reference: the same with further summands and no norm of delta: residual += delta + bias (may be
+ * NULL) + sum over k < per_row of rows[index[t * per_row + k]] (fp32 slabs too); xn = rmsnorm(residual) * w_next. */
+int bcg_residual_norm(float* residual, const float* delta, int n_partials, long long partial_stride, const float* bias,
+                      const float* rows, const int* index, int per_row, int row_partials, long long row_stride,
+                      const float* w_next, void* xn, int act_dtype, int T, int d, float eps, void* stream);
 /* No counterpart in the reference: a N(z) + b N(z^2) + c N(z^3) + e with N = division by the row's RMS. */
 int bcg_poly_norm(const float* z, int n_partials, long long partial_stride, const float* coef, void* out,
                   int act_dtype, int T, int ff, float eps, void* stream);
@@ -495,6 +543,18 @@ int bcg_delta_scan(const bcg_layer* l, const float* proj, int n_partials, long l
  * mode 0: what bcg_stack_step picks; 1: the plain kernel; ws->mix receives the heads' values. */
 int bcg_latent_attention(const bcg_stack* m, const bcg_stack_ws* ws, const bcg_step_batch* b, int layer, int mode,
                          void* stream);
+/* No counterpart in the reference: a grouped attention layer's input projection (ws->proj, row pitch ld) to queries, key
+ * and value pages, activations (with_act: columns n_qkv.. are up rows), and the routing of its experts
+ * (ws->moe_counts must be zero). */
+int bcg_grouped_in(const bcg_stack* m, const bcg_stack_ws* ws, const bcg_step_batch* b, int layer, int n_partials,
+                   long long partial_stride, long long ld, int with_act, void* stream);
+/* No counterpart in the reference: attention of a step's queries (ws->q) over the key and value pages.
+ * mode 0: what bcg_stack_step picks; 1: the plain kernel; columns 0.. of ws->mix receive the heads' values. */
+int bcg_grouped_attention(const bcg_stack* m, const bcg_stack_ws* ws, const bcg_step_batch* b, int layer, int mode,
+                          void* stream);
+/* No counterpart in the reference: ws->xn through the experts that bcg_grouped_in chose; ws->moe_out receives *splits
+ * slabs of [T * top, d], row ws->moe_row[t * top + k] for choice k of token t. */
+int bcg_experts(const bcg_stack* m, const bcg_stack_ws* ws, int layer, int T, int* splits, void* stream);
 
 #ifdef __cplusplus
 }
