@@ -229,7 +229,7 @@ class StackConfig:
                     raise ValueError(f"{self.name}: layer {i}: {m.heads} query heads on {m.kv_heads} key/value heads")
                 if m.v_mix:
                     f = self.layers[self.v_first].mixer
-                    if (f.kv_heads, f.vdim) != (m.kv_heads, m.vdim):
+                    if f.kv_heads * f.vdim != m.kv_heads * m.vdim:
                         raise ValueError(f"{self.name}: layer {i} cannot mix in values of layer {self.v_first}")
             if isinstance(m, GeneralDelta) and m.dim > 256:
                 raise ValueError(f"{self.name}: layer {i}: the delta-rule kernel takes up to 256 channels per head")

@@ -1,6 +1,9 @@
-"""Small random layer-stack models for the tests: config.json dicts of the Bekopel design, their tensors, and
-model directories.  Weights are scaled so that every mechanism moves the logits: scores spread over several
-units, sinks that take a visible share, decays from fast to almost none, all four activation numbers set."""
+"""Small random layer-stack models for the tests: config.json dicts of the Bekopel and Lerazen designs, their
+tensors, and model directories.  Weights are scaled so that every mechanism moves the logits: scores spread over
+several units, sinks that take a visible share, decays from fast to almost none, all four activation numbers set,
+biases and mixed values of the size of what they join.  Routers are decisive: a few coordinates of the stream hold
+a code of the token that no layer touches, and the router reads mostly those, so that rounding does not choose
+another expert."""
 import json
 
 import torch
@@ -19,12 +22,75 @@ def delta(heads=2, dim=24, ff=96):
             "mlp": {"kind": "dense", "ff": ff} if ff else None}
 
 
+def dense(ff):
+    return {"kind": "dense", "ff": ff}
+
+
+def moe(experts=6, top=2, ff=40, limit=1.5):
+    return {"kind": "moe", "expert": {"ff": ff, "limit": limit}, "router": {"experts": experts, "top": top}}
+
+
+def gattn(heads=6, kv_heads=3, dim=24, vdim=40, window=20, coef=0.4, every=23, v_mix=True, scale=None, mlp=None):
+    return {"type": "attention", "mlp": mlp,
+            "mixer": {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "mask": {"size": window},
+                      "q_temp": {"coef": coef, "every": every}, "scale": scale or 2.0 * dim ** -0.5, "v_mix": v_mix}}
+
+
+def parallel_config(layers, width=80, vocab=200, eps=1e-5, positions=512):
+    return {"architecture": "Lerazen", "layers": layers, "norm": {"eps": eps}, "vocab": vocab, "width": width,
+            "max_positions": positions}
+
+
+def parallel_tensors(cfg, seed=0):
+    g = torch.Generator().manual_seed(seed)
+    rnd = lambda *s, std=1.0, mean=0.0: torch.randn(*s, generator=g) * std + mean
+    d, V = cfg["width"], cfg["vocab"]
+    lin = lambda n, k, gain=1.0: rnd(n, k, std=gain * k ** -0.5)
+    routers = [l["mlp"]["router"]["experts"] for l in cfg["layers"] if l["mlp"] and l["mlp"]["kind"] == "moe"]
+    code = max(routers, default=0)               # the last coordinates of the stream
+
+    def out(*s, gain=1.0):                        # output matrices and biases leave the code alone
+        w = lin(*s, gain) if len(s) == 2 else rnd(*s, std=0.3)
+        w[d - code:] = 0
+        return w
+    t = {"embed": rnd(V, d), "pos": rnd(cfg["max_positions"], d, std=0.5), "final.norm": rnd(d, std=0.1, mean=1.0), "head": lin(V, d)}
+    if code:
+        t["pos"][:, d - code:] = 0
+        for v in range(V):
+            t["embed"][v, d - code:] = torch.linspace(-3, 3, code)[torch.randperm(code, generator=g)]
+    for i, l in enumerate(cfg["layers"]):
+        p, m, f = f"l{i}.", l["mixer"], l["mlp"]
+        t[p + "norm1"] = rnd(d, std=0.1, mean=1.0)
+        t[p + "norm1"][d - code:] = 1
+        H, G = m["heads"], m["kv_heads"]
+        for n, rows in (("q", H * m["dim"]), ("k", G * m["dim"]), ("v", G * m["vdim"])):
+            t[p + f"mix.{n}"], t[p + f"mix.{n}.b"] = lin(rows, d), rnd(rows, std=0.5)
+        t[p + "mix.o"], t[p + "mix.o.b"] = out(d, H * m["vdim"], gain=1.5), out(d)
+        if m["v_mix"]:
+            t[p + "mix.vmix"] = torch.rand((), generator=g) * 0.5 + 0.25
+        if f and f["kind"] == "dense":
+            t[p + "mlp.up"], t[p + "mlp.down"] = lin(f["ff"], d), out(d, f["ff"])
+        elif f:
+            E, n = f["router"]["experts"], f["expert"]["ff"]
+            router = lin(E, d, 0.02)
+            router[:, d - code:] = 0
+            for e, c in enumerate(torch.randperm(code, generator=g)[:E]):
+                router[e, d - code + c] = 2.0
+            t[p + "mlp.router"] = router
+            for e in range(E):
+                q = p + f"mlp.e{e}."
+                t.update({q + "gate": lin(n, d, 3.0), q + "up": lin(n, d, 3.0), q + "down": out(d, n, gain=1.5)})
+    return {n: x.to(torch.bfloat16) for n, x in t.items()}
+
+
 def config(layers, width=80, vocab=200, eps=1e-5):
     return {"architecture": "Bekopel", "layers": layers, "norm": {"eps": eps}, "vocab": vocab, "width": width}
 
 
 def tensors(cfg, seed=0, decay_rank=12):
     """name -> bf16 tensor, as a checkpoint of the design holds them."""
+    if cfg["architecture"] == "Lerazen":
+        return parallel_tensors(cfg, seed)
     g = torch.Generator().manual_seed(seed)
     rnd = lambda *s, std=1.0, mean=0.0: (torch.randn(*s, generator=g) * std + mean).to(torch.bfloat16)
     d, V = cfg["width"], cfg["vocab"]

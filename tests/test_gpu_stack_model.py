@@ -33,7 +33,22 @@ CONFIGS = {
     "odd": SM.config([SM.delta(3, 7, ff=45), SM.attn(3, 9, 6, 11, 13, 19, ff=51), SM.attn(5, 10, 6, 7, 13, 40, kv_from=1, ff=None)],
                      width=61, vocab=83),
     "one-each": SM.config([SM.attn(1, 8, 8, 8, 16, 5, ff=20)], width=36, vocab=36),
+    # parallel layers: values mixed from the second layer on, a layer in between without, every kind of feed-forward
+    "parallel": SM.parallel_config([SM.gattn(v_mix=False, mlp=SM.dense(96)), SM.gattn(window=1, mlp=SM.moe()),
+                                    SM.gattn(2, 1, 16, 24, 45, v_mix=False), SM.gattn(3, 3, 40, 40, 400, every=64, mlp=SM.moe(4, 1, 24, 0.7))]),
+    # everything on the tensor-core kernels
+    "parallel-tensor": SM.parallel_config([SM.gattn(8, 2, 64, 32, 33, mlp=SM.moe(8, 3, 64)), SM.gattn(4, 1, 128, 64, 100, mlp=SM.dense(320)),
+                                           SM.gattn(8, 2, 96, 32, 17, coef=-0.1, mlp=SM.moe(8, 2, 96, 3.0)), SM.gattn(2, 1, 256, 200, 70, v_mix=False)],
+                                          width=192, vocab=320),
+    # a group of more than 16 query heads, heads no tensor-core tile takes, one expert out of one
+    "parallel-groups": SM.parallel_config([SM.gattn(20, 1, 16, 16, 64, mlp=SM.moe(1, 1, 16)), SM.gattn(36, 2, 8, 8, 30, mlp=SM.moe(9, 9, 8)),
+                                           SM.gattn(2, 2, 264, 264, 50, v_mix=False)], width=96, vocab=96, eps=1e-3),
+    # sizes no vector load or tile likes
+    "parallel-odd": SM.parallel_config([SM.gattn(3, 1, 7, 11, 19, mlp=SM.dense(45)), SM.gattn(5, 5, 9, 6, 40, v_mix=False, mlp=SM.moe(5, 3, 21)),
+                                        SM.gattn(3, 1, 13, 11, 130, every=1, mlp=SM.dense(51))], width=61, vocab=83),
+    "parallel-one": SM.parallel_config([SM.gattn(1, 1, 8, 8, 5, mlp=SM.dense(20))], width=36, vocab=36, positions=300),
 }
+ATTENTION_MIX = ["mixed", "tensor", "parallel", "parallel-tensor"]
 
 
 class Model:
@@ -48,6 +63,10 @@ class Model:
 
     def oracle(self, toks):
         return R.forward(self.cfg, self.t, toks)
+
+    def given_back(self):
+        e = self.eng
+        return len(e.pool.free) == e.pool.n_pages and len(e.slots.free) == e.slots.n
 
     def check(self, got, want):
         got, want = got.double().cpu(), want.double()
@@ -76,10 +95,10 @@ def test_prompt_tokens_and_portions(name, dtype):
     want = m.oracle(toks)
     for sizes in ([210], [1], [2], [130, 1], [1, 3, 2, 17, 64, 5, 16, 31], [7, 150, 4, 1]):
         m.check(m.feed(toks, sizes), want)
-    assert len(m.eng.pool.free) == m.eng.pool.n_pages and len(m.eng.slots.free) == m.eng.slots.n
+    assert m.given_back()
 
 
-@pytest.mark.parametrize("name", ["mixed", "tensor"])
+@pytest.mark.parametrize("name", ATTENTION_MIX)
 def test_residual_after_every_depth(name):
     """The residual stream after each layer, by running the first layers only."""
     full, t = CONFIGS[name], SM.tensors(CONFIGS[name], seed=3)
@@ -95,7 +114,7 @@ def test_residual_after_every_depth(name):
 
 
 @pytest.mark.parametrize("dtype", TOL)
-@pytest.mark.parametrize("name", ["mixed", "tensor"])
+@pytest.mark.parametrize("name", ATTENTION_MIX)
 def test_unequal_requests_in_one_batch_equal_each_alone(name, dtype):
     """Four live requests, portions beside single tokens; pages and slots of finished ones are used again."""
     m = Model(name, dtype, tokens=448)
@@ -126,7 +145,7 @@ def test_unequal_requests_in_one_batch_equal_each_alone(name, dtype):
                 m.eng.close_sequence(live.pop(n)[0])
     for n, parts in got.items():
         m.check(torch.cat(parts), want[n])
-    assert len(m.eng.pool.free) == m.eng.pool.n_pages and len(m.eng.slots.free) == m.eng.slots.n
+    assert m.given_back()
 
 
 def test_wanted_places_only_and_in_order():
@@ -160,9 +179,10 @@ def test_pool_is_as_large_as_asked_and_says_when_it_is_full():
 
 
 @pytest.mark.parametrize("dtype", TOL)
-def test_long_decoding(dtype):
+@pytest.mark.parametrize("name", ["mixed", "parallel"])
+def test_long_decoding(name, dtype):
     """Windows pass over decoded tokens many times over; the state is carried through every one of them."""
-    m = Model("mixed", dtype)
+    m = Model(name, dtype)
     toks = m.tokens(400, 9)
     m.check(m.feed(toks, [3, 1]), m.oracle(toks))
 
@@ -182,14 +202,55 @@ def test_a_far_token_is_remembered(dtype):
         m.check(m.feed(toks, sizes), want)
 
 
+def test_learned_positions_end_where_the_table_does():
+    m = Model("parallel-one", "float32")                  # 300 positions, pages for 512 tokens
+    toks = m.tokens(301)
+    s = m.eng.open()
+    out = m.eng.step([(s, toks[:300], [0, 299])])
+    m.check(out, m.oracle(toks[:300])[[0, 299]])
+    with pytest.raises(Exception, match="max_model_len"):
+        m.eng.step([(s, toks[300:], [0])])
+
+
+@pytest.mark.parametrize("dtype", TOL)
+def test_prompts_of_many_tiles(dtype):
+    """More tokens than one row tile of the experts' products, several prompt tiles, windows across them."""
+    m = Model("parallel-tensor", dtype, tokens=1024, max_model_len=512)
+    a, b = m.tokens(500, 1), m.tokens(333, 2)
+    sa, sb = m.eng.open(), m.eng.open()
+    out = [m.eng.step([(sa, a[:400], list(range(400))), (sb, b[:3], [0, 1, 2])]),
+           m.eng.step([(sb, b[3:], list(range(330))), (sa, a[400:], list(range(100)))])]
+    want = torch.cat([m.oracle(a)[:400], m.oracle(b), m.oracle(a)[400:]])
+    m.check(torch.cat(out), want)
+
+
+@pytest.mark.parametrize("dtype", TOL)
+def test_one_expert_takes_every_token(dtype):
+    """All rows of a batch on one expert, the others empty."""
+    m = Model("parallel-tensor", dtype)
+    for i in (0, 2):
+        r = m.t[f"l{i}.mlp.router"]
+        r[:, :] = 0.01 * r
+        r[5, -8:] = 0
+        others = [e for e in range(8) if e != 5]
+        r[others, -8:] = torch.eye(8)[others].to(r.dtype)
+        m.t["embed"][:, -8:] = torch.tensor([1.0, -1.0, 0.5, -0.5, 0.0, 0.0, -2.0, -3.0]).to(r.dtype)   # 5's logit: third
+    m.eng = SM.engine(m.cfg, m.t, dtype)
+    toks = m.tokens(200)
+    m.check(m.feed(toks, [160, 1]), m.oracle(toks))
+
+
 # ------------------------------------------------------------------------------------------ generation
 GEN = SM.config([SM.delta(heads=2, dim=32), SM.attn(4, 32, 32, 32, 64, 24), SM.attn(2, 32, 32, 64, 64, 40, kv_from=1), SM.delta(2, 40)],
                 width=128, vocab=1024)
+GENS = {"Bekopel": GEN, "Lerazen": SM.parallel_config([SM.gattn(4, 2, 32, 32, 24, mlp=SM.dense(96)), SM.gattn(4, 1, 64, 64, 40, mlp=SM.moe(8, 2, 48)),
+                                                       SM.gattn(2, 2, 40, 48, 1000, v_mix=False, mlp=SM.moe(4, 1, 32))],
+                                                      width=128, vocab=1024, positions=600)}
 
 
-def _greedy(t, ids, n, out):
+def _greedy(cfg, t, ids, out):
     """The oracle's greedy continuation, following `out` where two logits are within rounding of each other."""
-    lg = R.forward(GEN, t, ids + out[:-1])[len(ids) - 1:]
+    lg = R.forward(cfg, t, ids + out[:-1])[len(ids) - 1:]
     for i, tok in enumerate(out):
         top = lg[i].max()
         assert top - lg[i][tok] < 0.15 * lg[i].std(), (i, tok, int(lg[i].argmax()))
@@ -198,12 +259,14 @@ def _greedy(t, ids, n, out):
 
 @pytest.mark.parametrize("graph", [False, True])
 @pytest.mark.parametrize("dtype", TOL)
-def test_greedy_generation_through_the_scheduler(dtype, graph):
+@pytest.mark.parametrize("design", GENS)
+def test_greedy_generation_through_the_scheduler(design, dtype, graph):
     from byzantine_consensus_llm_agents_b200.engine import Request
     from byzantine_consensus_llm_agents_b200.tokenizer import get_tokenizer
-    t = SM.tensors(GEN, seed=2)
-    tk = get_tokenizer("qwen3", GEN["vocab"])
-    eng = SM.engine(GEN, t, dtype, tokens=256, rows=3, tokenizer=tk, kv_pages=64, use_cuda_graph=graph)
+    cfg = GENS[design]
+    t = SM.tensors(cfg, seed=2)
+    tk = get_tokenizer("qwen3", cfg["vocab"])
+    eng = SM.engine(cfg, t, dtype, tokens=256, rows=3, tokenizer=tk, kv_pages=64, use_cuda_graph=graph)
     g = torch.Generator().manual_seed(0)
     prompts = [torch.randint(0, 700, (n,), generator=g).tolist() for n in (70, 1, 16, 33, 5)]    # two waves of rows
     res = eng.generate([Request("", prompt_ids=p, max_tokens=m) for p, m in zip(prompts, (40, 60, 25, 30, 64))])
@@ -211,19 +274,23 @@ def test_greedy_generation_through_the_scheduler(dtype, graph):
     same = 0
     for p, r in zip(prompts, res):
         assert r.token_ids and r.finish in ("length", "stop")
-        want = _greedy(t, p, len(r.token_ids), r.token_ids)
+        want = _greedy(cfg, t, p, r.token_ids)
         same += sum(a == b for a, b in zip(want, r.token_ids))
     total = sum(len(r.token_ids) for r in res)
     assert same >= total * (0.995 if dtype == "float32" else 0.9), (same, total)
     if dtype == "float32":
         assert again.token_ids == res[3].token_ids
-    assert len(eng.slots.free) == eng.slots.n and len(eng.pool.free) == eng.pool.n_pages
+    # a prefix is taken from its pages where they are all there is to it
+    assert again.cached_tokens == (0 if eng.exec.has_state else 32)
+    assert len(eng.slots.free) == eng.slots.n and len(eng.pool.free) + len(eng.pool.cached) == eng.pool.n_pages
 
 
-def test_adapter_generates_from_a_model_directory(tmp_path):
+@pytest.mark.parametrize("design", GENS)
+def test_adapter_generates_from_a_model_directory(design, tmp_path):
     """The agents' entry point: a directory as model name, a JSON schema, greedy."""
     from byzantine_consensus_llm_agents_b200 import vllm_agent as VA
     from byzantine_consensus_llm_agents_b200.stack import StackWeights
+    GEN = GENS[design]
     t = SM.tensors(GEN, seed=2)
     d = SM.save(GEN, t, tmp_path / "stack-model")
     schema = {"type": "object", "properties": {"decision": {"type": "string", "enum": ["stop", "continue"]}},
@@ -249,8 +316,9 @@ def test_adapter_generates_from_a_model_directory(tmp_path):
 
 # ------------------------------------------------------------------------------------------ trace replay
 @pytest.mark.parametrize("dtype", TOL)
-def test_trace_replay_program(tmp_path, dtype):
-    cfg = CONFIGS["tensor"]
+@pytest.mark.parametrize("name", ["tensor", "parallel-tensor"])
+def test_trace_replay_program(tmp_path, name, dtype):
+    cfg = CONFIGS[name]
     t = SM.tensors(cfg, seed=11)
     d, out = SM.save(cfg, t, tmp_path / "m"), tmp_path / "out"
     out.mkdir()

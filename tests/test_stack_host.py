@@ -72,11 +72,97 @@ def test_packed_rows_are_padded_with_zeros():
     assert "latent_norm" not in w.layers[2] and w.layers[2]["w_in"].shape[0] == 48
 
 
+# ---------------------------------------------------------------------------------------- parallel layers
+PAR = SM.parallel_config([SM.gattn(v_mix=False, mlp=SM.dense(45)), SM.gattn(window=33, mlp=SM.moe(5, 2, 21, 0.75)), SM.gattn(mlp=None)], width=60)
+
+
+def test_parallel_config_comes_from_the_directory(tmp_path):
+    t = SM.tensors(PAR)
+    c = M.config_from_dir(str(SM.save(PAR, t, tmp_path / "m")))
+    assert isinstance(c, S.StackConfig) and set(c.tensor_shapes()) == set(t)
+    assert all(tuple(t[n].shape) == s for n, s in c.tensor_shapes().items())
+    assert all(l.parallel for l in c.layers) and c.v_first == 1 and not c.has_state and c.max_window == 33
+    assert c.layers[0].mlp == S.DenseMlp(45, "relu2") and c.layers[1].mlp == S.MoeMlp(5, 2, 21, 0.75) and c.layers[2].mlp is None
+    m = c.layers[1].mixer
+    assert (m.heads, m.kv_heads, m.dim, m.vdim, m.window, m.temp_coef, m.temp_every) == (6, 3, 24, 40, 33, 0.4, 23.0)
+    assert c.learned_pos and c.max_pos == PAR["max_positions"] and c.kv_bytes_per_token == 3 * 2 * 3 * (64 + 64)
+    w = S.StackWeights.from_safetensors_dir(c, tmp_path / "m", "cpu")
+    assert w.pos_embed.shape == (PAR["max_positions"], 60)
+    # experts are streamed by the number of them that a step's tokens use
+    dense = 2 * (c.decode_weight_bytes(1) - c.decode_weight_bytes(0)) // 2
+    assert dense == 2 * 2 * 3 * 21 * 60 and c.decode_weight_bytes(1000) == c.decode_weight_bytes() > c.decode_weight_bytes(1)
+
+
+def test_parallel_layers_are_packed_side_by_side():
+    t = SM.tensors(PAR)
+    c = SM.stack_config(PAR, t)
+    w = S.StackWeights.from_tensors(c, t.__getitem__, "cpu")
+    m, a, b = c.layers[0].mixer, *w.layers[:2]
+    col, cols = c.mix_cols(0)
+    assert c.qkv_rows(0) % 16 == 0 and a["w_in"].shape == (c.qkv_rows(0) + 48, 60) and a["w_out"].shape == (60, cols)
+    assert torch.equal(a["w_in"][m.in_dim - 120:m.in_dim], t["l0.mix.v"]) and not a["w_in"][m.in_dim:c.qkv_rows(0)].any()
+    assert torch.equal(a["w_in"][c.qkv_rows(0):c.qkv_rows(0) + 45], t["l0.mlp.up"]) and not a["w_in"][c.qkv_rows(0) + 45:].any()
+    assert torch.equal(a["w_out"][:, :240], t["l0.mix.o"]) and torch.equal(a["w_out"][:, col:col + 45], t["l0.mlp.down"])
+    assert not a["w_out"][:, col + 45:].any() and "vmix" not in a and "slopes" in a
+    assert torch.equal(b["w_in"][m.in_dim:m.in_dim + 5], t["l1.mlp.router"]) and b["w_out"].shape == (60, 240)
+    gate, up = b["w_experts_in"][3].view(2, 2, 16, 60).unbind(1)
+    for x, n in ((gate, "gate"), (up, "up")):
+        assert torch.equal(x.reshape(32, 60)[:21], t[f"l1.mlp.e3.{n}"]) and not x.reshape(32, 60)[21:].any()
+    assert torch.equal(b["w_experts_out"][4, :, :21], t["l1.mlp.e4.down"]) and not b["w_experts_out"][:, :, 21:].any()
+    assert torch.allclose(a["slopes"], 2.0 ** (-8 * torch.arange(1, 7) / 6))
+
+
+@pytest.mark.parametrize("spoil, words", [
+    (lambda c: c["layers"][0].update(type="other"), "unknown mixer"),
+    (lambda c: c["layers"][0]["mlp"].update(kind="other"), "unknown feed-forward"),
+    (lambda c: c["layers"][0]["mixer"].update(kv_heads=4), "key/value heads"),
+    (lambda c: c["layers"][2]["mixer"].update(vdim=8), "cannot mix"),
+    (lambda c: c["layers"][1]["mlp"]["router"].update(top=6), "6 of 5 experts"),
+])
+def test_bad_parallel_configurations_are_refused(spoil, words):
+    import copy
+    c = copy.deepcopy(PAR)
+    spoil(c)
+    with pytest.raises(ValueError, match=words):
+        SM.stack_config(c, SM.tensors(PAR))
+
+
+def test_mixed_kinds_of_layers_are_refused():
+    g = S.GroupedAttention(2, 1, 8, 8, 1.0)
+    with pytest.raises(ValueError, match="parallel"):
+        S.StackConfig("x", 16, 16, (S.LayerSpec(g),))
+    with pytest.raises(ValueError, match="activation"):
+        S.StackConfig("x", 16, 16, (S.LayerSpec(g, S.DenseMlp(8), True),))
+
+
+def test_oracle_temperature_slopes_and_mixing():
+    assert torch.allclose(R.head_slopes(4), torch.tensor([2.0 ** -2, 2.0 ** -4, 2.0 ** -6, 2.0 ** -8], dtype=torch.float64))
+    t = R.query_temperature(torch.tensor([0, 2, 3, 4, 8]), 2.0, 4)
+    assert torch.allclose(t, 1 + 2 * torch.log(torch.tensor([1.0, 1, 2, 2, 3], dtype=torch.float64)))
+    v = R.mix_values(torch.tensor([1.0]), torch.tensor([3.0]), 0.25)
+    assert v.item() == 1.5
+
+
+def test_oracle_experts_scale_their_input():
+    g = torch.Generator().manual_seed(0)
+    w = {f"e{e}.{n}": torch.randn(*s, generator=g, dtype=torch.float64) for e in range(3) for n, s in (("gate", (4, 5)), ("up", (4, 5)), ("down", (5, 4)))}
+    w["router"] = torch.tensor([[1.0, 0, 0, 0, 0], [0, 1.0, 0, 0, 0], [0, 0, 1.0, 0, 0]], dtype=torch.float64)
+    h = torch.tensor([[0.3, -2.0, 1.1, 0.4, -0.7]], dtype=torch.float64)
+    s = torch.sigmoid(h[0, :3])
+    y = 0
+    for e in (2, 0):
+        gate, up = torch.clamp(w[f"e{e}.gate"] @ (s[e] * h[0]), max=0.6), torch.clamp(w[f"e{e}.up"] @ (s[e] * h[0]), -0.6, 0.6)
+        y = y + w[f"e{e}.down"] @ (gate * torch.sigmoid(1.702 * gate) * (up + 1))
+    assert torch.allclose(R.mixture(h, w, 2, 0.6)[0], y)
+
+
 def test_preset_resolves_by_name():
     c = M.config_for("bekopel-8b")
     assert isinstance(c, S.StackConfig) and c.d_model == M.PRESETS["qwen3-8b"].d_model
     with pytest.raises(ValueError, match="tensor parallelism"):
         c.shard(2)
+    c = M.config_for("lerazen-30b-a3b")
+    assert c.layers[0].mlp.act == "relu2" and c.layers[1].mlp.experts == 128 and c.v_first == 0
 
 
 # ---------------------------------------------------------------------------------------- work lists
