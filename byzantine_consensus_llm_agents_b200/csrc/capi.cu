@@ -270,6 +270,22 @@ int bcg_grouped_attention(const bcg_stack* m, const bcg_stack_ws* ws, const bcg_
   return grouped_attention_step(m, ws, b, layer, mode, S(stream));
 }
 
+int bcg_gemm_grouped(const void* X, const void* W, void* out, int rows, int N, int K, const int* counts, int n_groups,
+                     int max_rows, int splits, const float* row_weight, float limit, float alpha, int flags, void* stream) {
+  GemmGroups g = {};
+  g.counts = counts;
+  g.n_groups = n_groups;
+  g.max_rows = max_rows;
+  g.row_weight = row_weight;
+  g.glu_limit = limit;
+  g.glu_alpha = alpha;
+  const int saved = launch_flags();
+  launch_flags() = flags & BCG_GEMM_PDL;
+  const int rc = gemm_grouped(X, W, out, rows, N, K, row_weight ? BCG_EPI_GLU : BCG_EPI_F32, splits, g, S(stream));
+  launch_flags() = saved;
+  return rc;
+}
+
 int bcg_experts(const bcg_stack* m, const bcg_stack_ws* ws, int layer, int T, int* splits, void* stream) {
   return experts_step(m, ws, layer, T, splits, S(stream));
 }

@@ -35,34 +35,36 @@ struct GroupedIn {
   float v_mix;
   int ff, act_from;           // squared-relu columns of proj (ff = 0: none)
   long long act_ld;
-  int blocks;                 // CTAs per token that share the columns
+  int n_tokens, blocks;       // blocks: CTAs per token that share the columns
   MoeRoute route;             // experts = 0: none
+  int route_tokens;           // tokens per routing CTA
 };
 
-// grid (T, blocks [+ 1 routes]).  Columns go to their destination four at a time (V = 4) or one by one.
+// grid: `blocks` CTAs per token, then the routing CTAs (`route_tokens` tokens each).  Columns go to their destination four at a
+// time (V = 4) or one by one.
 template <typename T, int V>
 __global__ void __launch_bounds__(kInThreads)
 grouped_in_kernel(const GroupedIn a) {
-  extern __shared__ float scores[];   // routing: one logit per expert
+  extern __shared__ uint32_t route_mem[];   // route_words(experts)
   pdl_launch_dependents();
   pdl_wait();
-  const long long t = blockIdx.x;
-  const float* row = a.proj + t * a.ld;
-  if (static_cast<int>(blockIdx.y) == a.blocks) {
-    route_token<kInThreads>(a.route, row, a.n_partials, a.pstride, static_cast<int>(t), scores);
+  const int split = blockIdx.x - a.n_tokens * a.blocks;
+  if (split >= 0) {
+    const int t0 = split * a.route_tokens;
+    route_tokens<kInThreads>(a.route, a.proj, a.n_partials, a.pstride, a.ld, t0, min(t0 + a.route_tokens, a.n_tokens),
+                             route_mem);
     return;
   }
+  const long long t = blockIdx.x / a.blocks;
+  const int part = blockIdx.x % a.blocks;
+  const float* row = a.proj + t * a.ld;
   const int pos = a.positions[t], slot = a.slot_map[t];
   const float temp = 1.0f + a.temp_coef * logf(floorf(static_cast<float>(pos + 1) / a.temp_every) + 1.0f);
   const int nq = a.heads * a.dim, nk = nq + a.kv_heads * a.dim, nv = nk + a.kv_heads * a.vdim;
   const long long page = slot >= 0 ? slot / a.page_size : 0;
   const int in_page = slot >= 0 ? slot % a.page_size : 0;
   const int step = a.blocks * kInThreads * V;
-  for (int c = (blockIdx.y * kInThreads + threadIdx.x) * V; c < nv; c += step) {
-    Vec<V> x = slab_sum_vec<V>(row + c, a.n_partials, a.pstride);
-    const Vec<V> b = load_vec<V>(a.bias + c);
-#pragma unroll
-    for (int i = 0; i < V; ++i) x.x[i] += b.x[i];
+  auto store = [&](int c, Vec<V>& x) {
     if (c < nq) {
       const int h = c / a.dim, i = c - h * a.dim;
 #pragma unroll
@@ -85,8 +87,13 @@ grouped_in_kernel(const GroupedIn a) {
       if (slot >= 0)
         store_vec<V>(static_cast<T*>(a.v_cache) + ((page * a.kv_heads + g) * a.page_size + in_page) * a.v_ld + i, x);
     }
+  };
+  for (int c = (part * kInThreads + threadIdx.x) * V; c < nv; c += step) {
+    Vec<V> x = slab_sum_vec<V>(row + c, a.n_partials, a.pstride);
+    x.add(load_vec<V>(a.bias + c));
+    store(c, x);
   }
-  for (int c = (blockIdx.y * kInThreads + threadIdx.x) * V; c < a.ff; c += step) {
+  for (int c = (part * kInThreads + threadIdx.x) * V; c < a.ff; c += step) {
     Vec<V> x = slab_sum_vec<V>(row + a.act_from + c, a.n_partials, a.pstride);
 #pragma unroll
     for (int k = 0; k < V; ++k) {
@@ -98,10 +105,14 @@ grouped_in_kernel(const GroupedIn a) {
 }
 
 template <typename T>
-static int grouped_in_t(const GroupedIn& a, int n_tokens, cudaStream_t st) {
+static int grouped_in_t(const GroupedIn& a, cudaStream_t st) {
   const bool wide = ((a.dim | a.vdim | a.ff | a.act_from) & 3) == 0 && a.ld % 4 == 0 && a.pstride % 4 == 0;
-  const dim3 grid(n_tokens, a.blocks + (a.route.experts > 0 ? 1 : 0));
-  const size_t sm = static_cast<size_t>(a.route.experts) * 4;
+  const dim3 grid(a.n_tokens * a.blocks + (a.route.experts > 0 ? (a.n_tokens + a.route_tokens - 1) / a.route_tokens : 0));
+  const size_t sm = static_cast<size_t>(route_words(a.route.experts, kInThreads)) * 4;
+  if (sm > 48 * 1024) {
+    set_last_error("bcg_grouped_in", "too many experts");
+    return BCG_ERR_UNSUPPORTED;
+  }
   if (wide) BCG_CUDA_CHECK(launch_k(grouped_in_kernel<T, 4>, grid, dim3(kInThreads), sm, st, a));
   else BCG_CUDA_CHECK(launch_k(grouped_in_kernel<T, 1>, grid, dim3(kInThreads), sm, st, a));
   return BCG_OK;
@@ -141,7 +152,9 @@ int grouped_in(const bcg_stack* m, const bcg_layer* l, const bcg_stack_ws* ws, c
   if (l->experts > 0) a.route = moe_route(l, ws);
   const int cols = l->heads * l->dim + l->kv_heads * (l->dim + l->vdim);
   a.blocks = b->T <= 128 ? max(1, ((cols > a.ff ? cols : a.ff) + kInThreads * 4 - 1) / (kInThreads * 4)) : 1;
-  return m->act_dtype == BCG_DT_F32 ? grouped_in_t<float>(a, b->T, st) : grouped_in_t<__nv_bfloat16>(a, b->T, st);
+  a.n_tokens = b->T;
+  a.route_tokens = b->T <= 128 ? kInThreads / 32 : kInThreads / 4;
+  return m->act_dtype == BCG_DT_F32 ? grouped_in_t<float>(a, st) : grouped_in_t<__nv_bfloat16>(a, st);
 }
 
 // ------------------------------------------------------------------------------------------- plain

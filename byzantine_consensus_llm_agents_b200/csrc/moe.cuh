@@ -26,41 +26,82 @@ __host__ inline MoeRoute moe_route(const bcg_layer* l, const bcg_stack_ws* ws) {
   return r;
 }
 
-// One CTA, one token: the `top` experts with the largest logits (the sigmoid is monotone; ties go to the lower
-// index), weighted by their sigmoid scores.  scores: shared memory, one float per expert.
-template <int THREADS>
+// fp32 <-> unsigned integers of the same order
+__device__ __forceinline__ uint32_t ordered_bits(float v) {
+  const uint32_t b = __float_as_uint(v);
+  return b & 0x80000000u ? ~b : b | 0x80000000u;
+}
+__device__ __forceinline__ float from_ordered(uint32_t k) {
+  return __uint_as_float(k & 0x80000000u ? k & 0x7fffffffu : ~k);
+}
+
+// Shared memory of route_tokens, in words: a key per expert and warp, two counters per expert.
+__host__ __device__ constexpr int route_words(int experts, int threads) { return experts * (threads / 32 + 2); }
+
+// One warp, one token: the `top` experts with the largest logits (the sigmoid is monotone; ties go to the lower
+// index), weighted by their sigmoid scores.  keys: the warp's shared memory, one word per expert.
+// counters: rows of every expert so far.
 __device__ __forceinline__ void route_token(const MoeRoute& r, const float* row, int n_partials, long long pstride, int t,
-                                            float* scores) {
-  for (int e = threadIdx.x; e < r.experts; e += THREADS) scores[e] = slab_sum(row + r.col + e, n_partials, pstride);
-  __syncthreads();
-  if (threadIdx.x >= 32) return;
-  const int lane = threadIdx.x;
-  for (int k = 0; k < r.top; ++k) {
-    float best = -INFINITY;
-    int at = 0x7fffffff;
+                                            uint32_t* keys, int* counters, int lane) {
+  for (int e = lane; e < r.experts; e += 32) keys[e] = ordered_bits(slab_sum(row + r.col + e, n_partials, pstride));
+  uint32_t best;      // the lane's best expert that is still free (key 0: none)
+  int at;
+  auto scan = [&]() {
+    best = 0;
+    at = lane < r.experts ? lane : 0x7fffffff;
     for (int e = lane; e < r.experts; e += 32)
-      if (scores[e] > best || at == 0x7fffffff) {
-        best = scores[e];
+      if (keys[e] > best) {
+        best = keys[e];
         at = e;
       }
-#pragma unroll
-    for (int o = 16; o > 0; o >>= 1) {
-      const float other = __shfl_xor_sync(0xffffffffu, best, o);
-      const int oat = __shfl_xor_sync(0xffffffffu, at, o);
-      if (other > best || (other == best && oat < at)) {
-        best = other;
-        at = oat;
+  };
+  __syncwarp();
+  scan();
+  int mine = 0;              // lane k keeps choice k: the counters are then touched side by side
+  uint32_t key = 0;
+  for (int k = 0; k < r.top; ++k) {
+    const uint32_t top = __reduce_max_sync(0xffffffffu, best);
+    const int e = __reduce_min_sync(0xffffffffu, best == top ? at : 0x7fffffff);
+    if (e % 32 == lane) {
+      keys[e] = 0;
+      scan();
+    }
+    if (k % 32 == lane) {
+      mine = e;
+      key = top;
+    }
+    if (k % 32 == 31 || k == r.top - 1) {
+      const int i = t * r.top + (k & ~31) + lane;
+      if (lane <= k % 32) {
+        r.expert[i] = mine;
+        r.weight[i] = 1.0f / (1.0f + expf(-from_ordered(key)));
+        r.rank[i] = atomicAdd(counters + mine, 1);
       }
     }
-    if (lane == 0) {
-      const int i = t * r.top + k;
-      r.expert[i] = at;
-      r.rank[i] = atomicAdd(r.counts + at, 1);
-      r.weight[i] = 1.0f / (1.0f + expf(-best));
-      scores[at] = -INFINITY;      // not chosen again: top <= experts leaves another one, or all are taken
-    }
-    __syncwarp();
   }
+}
+
+// One CTA: tokens t0 .. t1.  With more than one token per warp, rows are numbered inside the CTA first, so that a
+// global counter is touched once per CTA.
+template <int THREADS>
+__device__ __forceinline__ void route_tokens(const MoeRoute& r, const float* proj, int n_partials, long long pstride,
+                                             long long ld, int t0, int t1, uint32_t* mem) {
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  if (t1 - t0 <= THREADS / 32) {
+    if (t0 + warp < t1)
+      route_token(r, proj + (t0 + warp) * ld, n_partials, pstride, t0 + warp, mem + warp * r.experts, r.counts, lane);
+    return;
+  }
+  int* local = reinterpret_cast<int*>(mem + THREADS / 32 * r.experts);
+  int* base = local + r.experts;
+  for (int e = threadIdx.x; e < r.experts; e += THREADS) local[e] = 0;
+  __syncthreads();
+  for (int t = t0 + warp; t < t1; t += THREADS / 32)
+    route_token(r, proj + t * ld, n_partials, pstride, t, mem + warp * r.experts, local, lane);
+  __syncthreads();
+  for (int e = threadIdx.x; e < r.experts; e += THREADS) base[e] = local[e] ? atomicAdd(r.counts + e, local[e]) : 0;
+  __syncthreads();
+  for (int i = t0 * r.top + threadIdx.x; i < t1 * r.top; i += THREADS) r.rank[i] += base[r.expert[i]];
 }
 
 // First row of an expert's rows: the counts in front of it.  A whole warp calls this.

@@ -186,6 +186,8 @@ _SIGS = {
                                  C.c_longlong, C.c_longlong, C.c_int, vp]),
     "bcg_grouped_attention": (C.c_int, [C.POINTER(Stack), C.POINTER(StackWs), C.POINTER(StepBatch), C.c_int, C.c_int,
                                         vp]),
+    "bcg_gemm_grouped": (C.c_int, [vp, vp, vp, C.c_int, C.c_int, C.c_int, vp, C.c_int, C.c_int, C.c_int, vp, C.c_float,
+                                   C.c_float, C.c_int, vp]),
     "bcg_experts": (C.c_int, [C.POINTER(Stack), C.POINTER(StackWs), C.c_int, C.c_int, c_int_p, vp]),
 }
 

@@ -222,8 +222,8 @@ class StackConfig:
                 raise ValueError(f"{self.name}: layer {i}: grouped attention and experts come in parallel layers, and only there")
             if l.mlp and isinstance(l.mlp, DenseMlp) and (l.mlp.act == "relu2") != l.parallel:
                 raise ValueError(f"{self.name}: layer {i}: activation {l.mlp.act!r} in this kind of layer")
-            if isinstance(l.mlp, MoeMlp) and not 0 < l.mlp.top <= l.mlp.experts:
-                raise ValueError(f"{self.name}: layer {i}: {l.mlp.top} of {l.mlp.experts} experts")
+            if isinstance(l.mlp, MoeMlp) and not 0 < l.mlp.top <= l.mlp.experts <= 1024:
+                raise ValueError(f"{self.name}: layer {i}: {l.mlp.top} of {l.mlp.experts} experts (at most 1,024)")
             if isinstance(m, GroupedAttention):
                 if m.heads % m.kv_heads:
                     raise ValueError(f"{self.name}: layer {i}: {m.heads} query heads on {m.kv_heads} key/value heads")

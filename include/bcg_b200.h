@@ -552,6 +552,13 @@ int bcg_grouped_in(const bcg_stack* m, const bcg_stack_ws* ws, const bcg_step_ba
  * mode 0: what bcg_stack_step picks; 1: the plain kernel; columns 0.. of ws->mix receive the heads' values. */
 int bcg_grouped_attention(const bcg_stack* m, const bcg_stack_ws* ws, const bcg_step_batch* b, int layer, int mode,
                           void* stream);
+/* No counterpart in the reference (vLLM's fused_moe is the nearest relative): rows sorted by group, X bf16 [rows, K]
+ * times the groups' matrices W bf16 [n_groups * N, K]; counts: device, rows per group, at most max_rows each.  K % 8 == 0,
+ * N % 16 == 0 where max_rows > 128, n_groups <= 512.  row_weight NULL: out fp32 [splits][rows, N] (splits > 1 only where
+ * max_rows <= 128).  Otherwise max_rows > 128, W rows interleaved [16 gate | 16 up], out bf16 [rows, N / 2] =
+ * g * sigmoid(alpha * g) * (u + 1) of the weighted accumulators, g = min(., limit), u clamped to +-limit. */
+int bcg_gemm_grouped(const void* X, const void* W, void* out, int rows, int N, int K, const int* counts, int n_groups,
+                     int max_rows, int splits, const float* row_weight, float limit, float alpha, int flags, void* stream);
 /* No counterpart in the reference: ws->xn through the experts that bcg_grouped_in chose; ws->moe_out receives *splits
  * slabs of [T * top, d], row ws->moe_row[t * top + k] for choice k of token t. */
 int bcg_experts(const bcg_stack* m, const bcg_stack_ws* ws, int layer, int T, int* splits, void* stream);
