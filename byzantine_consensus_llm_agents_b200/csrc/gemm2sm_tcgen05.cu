@@ -50,6 +50,7 @@ struct Gemm2Args {
   int epi;
   void* out;
   long long ld_out;
+  int sector_stores;         // fp32 output rows are 32-byte aligned: whole sectors per store
   uint64_t hint_a, hint_b;   // L2 eviction priority of the activation / weight loads
 };
 
@@ -272,6 +273,13 @@ gemm2sm_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_
             float* o = reinterpret_cast<float*>(args.out);
             if (m < M && n0 + c < N) {
               float4* dst = reinterpret_cast<float4*>(o + m * ld + n0 + c);
+              if (args.sector_stores) {
+                st_v8(dst, v0);
+                st_v8(dst + 2, v0 + 8);
+                st_v8(dst + 4, v1);
+                st_v8(dst + 6, v1 + 8);
+                continue;
+              }
 #pragma unroll
               for (int j = 0; j < 4; ++j)
                 dst[j] = make_float4(__uint_as_float(v0[4 * j]), __uint_as_float(v0[4 * j + 1]),
@@ -352,6 +360,7 @@ int gemm2sm_bf16_tn(const void* X, const void* W, void* out, int M, int N, int K
   a.epi = epi;
   a.out = out;
   a.ld_out = ld_out;
+  a.sector_stores = (reinterpret_cast<uintptr_t>(out) % 32 == 0 && ld_out % 8 == 0) ? 1 : 0;
   CUtensorMap tma, tmb;
   int rc;
   if ((rc = make_tmap_bf16_sw128(&tma, X, M, K, ldx, k2BlockM)) != BCG_OK) return rc;

@@ -52,6 +52,7 @@ struct GemmArgs {
   void* out;
   long long ld_out;         // elements
   uint64_t hint_a, hint_b;
+  int sector_stores;        // fp32 output rows are 32-byte aligned: whole sectors per store
   int pdl_wait_b;           // 1: launched with programmatic stream serialization (see the producer)
   // ---- decode-only fusions of the residual add + RMSNorm that sits between two projections
   // consumer side: the activations are r*w (NOT yet divided by the row's RMS); every output row m is
@@ -416,6 +417,17 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_a,
               float* o = reinterpret_cast<float*>(args.out) + split * slab + base;
               if (m < M) {
                 float4* dst = reinterpret_cast<float4*>(o + m * ld + n0 + c);
+                if (args.sector_stores) {
+                  if (n0 + c < N) {
+                    st_v8(dst, v0);
+                    st_v8(dst + 2, v0 + 8);
+                  }
+                  if (n0 + c + 16 < N) {
+                    st_v8(dst + 4, v1);
+                    st_v8(dst + 6, v1 + 8);
+                  }
+                  continue;
+                }
                 if (n0 + c < N) {
 #pragma unroll
                   for (int j = 0; j < 4; ++j)
@@ -676,6 +688,7 @@ int gemm_bf16_tn_fused(const void* X, const void* W, void* out, int M, int N, in
   a.swap = swap ? 1 : 0;
   a.epi = epi;
   a.out = out;
+  a.sector_stores = (reinterpret_cast<uintptr_t>(out) % 32 == 0 && ld_out % 8 == 0) ? 1 : 0;
   a.ld_out = ld_out;
   a.pdl_wait_b = ((flags | launch_flags()) & BCG_GEMM_PDL) ? 1 : 0;
   if (fu && (fu->scale_sumsq || fu->red_counters)) {
@@ -768,6 +781,7 @@ int gemm_grouped(const void* X, const void* W, void* out, int rows, int N, int K
   a.swap = swap ? 1 : 0;
   a.epi = epi;
   a.out = out;
+  a.sector_stores = (reinterpret_cast<uintptr_t>(out) % 32 == 0 && N % 8 == 0) ? 1 : 0;
   a.ld_out = epi == BCG_EPI_GLU ? N / 2 : N;
   a.groups = g;
   a.pdl_wait_b = (launch_flags() & BCG_GEMM_PDL) ? 1 : 0;
