@@ -197,10 +197,10 @@ def test_distance_bias_decides_between_equal_keys(dtype, portion):
 
 # ------------------------------------------------------------------------------------------ inputs
 @pytest.mark.parametrize("dtype", DT)
-@pytest.mark.parametrize("heads,kv,dim,vdim,ff,experts", [(3, 1, 7, 11, 45, 0), (8, 2, 64, 32, 96, 0), (4, 4, 20, 8, 0, 6), (2, 1, 260, 4, 0, 40)])
+@pytest.mark.parametrize("heads,kv,dim,vdim,ff,experts", [(3, 1, 7, 11, 45, 0), (8, 2, 64, 32, 96, 0), (4, 4, 20, 8, 0, 6), (2, 1, 260, 4, 0, 40), (2, 2, 16, 4, 0, 70)])
 def test_projection_is_split_biased_and_stored(dtype, heads, kv, dim, vdim, ff, experts):
-    mlp = SM.dense(ff) if ff else SM.moe(experts, min(3, experts), 16)
-    o = OneLayer(SM.gattn(heads, kv, dim, vdim, coef=0.7, every=9, mlp=mlp), dtype, seed=dim)
+    mlp = SM.dense(ff) if ff else SM.moe(experts, 45 if experts > 45 else 3, 16)
+    o = OneLayer(SM.gattn(heads, kv, dim, vdim, coef=0.7, every=9, mlp=mlp), dtype, seed=dim, width=96)
     td, tol, l = o.td, (4e-3 if dtype == "bfloat16" else 2e-6), o.layer
     starts = [40, 0, 7]
     entries, lens, used = [], [5, 1, 20], []
