@@ -4,7 +4,8 @@ Plain, slow restatement of the mechanisms that layer-stack designs are made of (
 attention with a sliding window and a sink, generalized delta rule, PolyNorm feed-forward, norms on
 both sides of each sublayer; Lerazen: grouped-query attention with a linear distance bias, a query
 temperature and values mixed with an earlier layer's, squared-relu and mixture-of-experts
-feed-forwards, parallel sublayers, learned positions).  One function per mechanism; torch on the CPU, in the dtype of its
+feed-forwards, parallel sublayers, learned positions; Merulorn: attention with whole-projection query and key
+norms and a gate per head beside a selective state-space mixer, clamped gated units, sinusoidal positions).  One function per mechanism; torch on the CPU, in the dtype of its
 inputs (the tests use float64, rounding weights only).  A whole sequence is computed at once, token by
 token where there is a recurrence, with no cache: what a cache, a batch or a cut of the prompt could get
 wrong is absent here by construction.
@@ -205,6 +206,108 @@ def _lerazen(config, T, tokens, collect):
     return rms_norm(x, eps, T["final.norm"]) @ T["head"].T
 
 
+def sinusoid(positions, width):
+    """[t, width]: sine and cosine of position * 10000^(-2i / width) in turn."""
+    i = torch.arange(width)
+    f = torch.tensor([10000.0 ** (-2.0 * (k // 2) / width) for k in i.tolist()], dtype=torch.float64)
+    ang = positions.to(torch.float64)[:, None] * f[None, :]
+    return torch.where(i % 2 == 0, ang.sin(), ang.cos())
+
+
+def zero_norm(x, eps, w):
+    """RMS norm whose weight is stored around zero."""
+    return rms_norm(x, eps, 1 + w)
+
+
+def gated_attention(h, w, m, positions, eps):
+    """m: dict(heads, kv_heads, dim, vdim, scale, coef, every).  Biased projections; query and key norms span all heads;
+    one output gate per head."""
+    t, H, G = h.shape[0], m["heads"], m["kv_heads"]
+    q = rms_norm(h @ w["q"].T + w["q.b"], eps, w["q.norm"]).view(t, H, m["dim"])
+    k = rms_norm(h @ w["k"].T + w["k.b"], eps, w["k.norm"]).view(t, G, m["dim"])
+    v = (h @ w["v"].T + w["v.b"]).view(t, G, m["vdim"])
+    q = q * query_temperature(positions, m["coef"], m["every"]).to(q.dtype)[:, None, None]
+    mine = torch.arange(H) // (H // G)
+    s = torch.einsum("ihd,jhd->hij", q, k[:, mine]) * m["scale"]
+    p = softmax_with_sink(s, window_visible(t, 0))
+    o = torch.einsum("hij,jhd->ihd", p, v[:, mine]) * torch.sigmoid(h @ w["g"].T)[:, :, None]
+    return o.reshape(t, H * m["vdim"]) @ w["o"].T
+
+
+def causal_conv(x, w, b, before=None):
+    """Per channel: y_t = b + sum over taps k of w[:, k] * x_(t - taps + 1 + k); x [t, channels].  `before`: the taps - 1
+    inputs ahead of x (zeros at the start of a sequence)."""
+    taps = w.shape[1]
+    full = torch.cat([x.new_zeros(taps - 1, x.shape[1]) if before is None else before, x])
+    y = torch.zeros_like(x)
+    for t in range(x.shape[0]):
+        y[t] = b
+        for k in range(taps):
+            y[t] = y[t] + w[:, k] * full[t + k]
+    return y
+
+
+def silu(x):
+    return x * torch.sigmoid(x)
+
+
+def ssm_scan(x, B, C, dt, A_log, D, state=None):
+    """x [t, heads, vdim], B and C [t, groups, n], dt [t, heads] (already positive).  Token by token
+    S = exp(-exp(A_log) dt) S + dt B x^T,  y = S^T C + D x.  Returns (y, S [heads, n, vdim])."""
+    t, H, P = x.shape
+    mine = torch.arange(H) // (H // B.shape[1])
+    S = torch.zeros(H, B.shape[2], P, dtype=x.dtype) if state is None else state.clone()
+    y = []
+    for i in range(t):
+        keep = torch.exp(-torch.exp(A_log) * dt[i])
+        S = keep[:, None, None] * S + dt[i][:, None, None] * B[i][mine][:, :, None] * x[i][:, None, :]
+        y.append(torch.einsum("hnp,hn->hp", S, C[i][mine]) + D[:, None] * x[i])
+    return torch.stack(y), S
+
+
+def part_norm(x, parts, eps, w):
+    """RMS norm of `parts` equal pieces of the last axis, each by its own root mean square."""
+    return rms_norm(x.view(x.shape[0], parts, -1), eps).reshape(x.shape) * w
+
+
+def mamba2(h, w, m, eps):
+    """m: dict(heads, vdim, state, groups, norm_groups); taps from the weight's shape."""
+    t, H, P, N, G = h.shape[0], m["heads"], m["vdim"], m["state"], m["groups"]
+    inner = H * P
+    z, xbc, dt = torch.split(h @ w["in"].T, [inner, inner + 2 * G * N, H], dim=-1)
+    xbc = silu(causal_conv(xbc, w["conv"], w["conv.b"]))
+    x, B, C = torch.split(xbc, [inner, G * N, G * N], dim=-1)
+    dt = torch.nn.functional.softplus(dt + w["dt_bias"], threshold=1e9)
+    y, _ = ssm_scan(x.view(t, H, P), B.view(t, G, N), C.view(t, G, N), dt, w["A_log"], w["D"])
+    return part_norm(y.reshape(t, inner) * silu(z), m["norm_groups"], eps, w["norm"]) @ w["o"].T
+
+
+def _merulorn(config, T, tokens, collect):
+    eps, pos, d = float(config["norm"]["eps"]), torch.arange(len(tokens)), config["width"]
+    x = T["embed"][torch.as_tensor(tokens, dtype=torch.long)]
+    x = x * config["embedding"]["scale"] + sinusoid(pos, d).to(x.dtype)
+    for i, layer in enumerate(config["layers"]):
+        p, mix = f"l{i}.", layer["mixer"]
+        sub = lambda kind: {n[len(p + kind) + 1:]: t for n, t in T.items() if n.startswith(p + kind + ".")}
+        h = zero_norm(x, eps, T[p + "norm1"])
+        if layer["type"] == "parallel":
+            a = mix["left"]
+            m = {**a, "coef": a["q_temp"]["coef"], "every": a["q_temp"]["every"]}
+            y = mix["left_scale"] * gated_attention(h, sub("mix.left"), m, pos, eps) \
+                + mix["right_scale"] * mamba2(h, sub("mix.right"), mix["right"], eps)
+        elif layer["type"] == "mamba2":
+            y = mamba2(h, sub("mix"), mix, eps)
+        else:
+            raise ValueError(f"unknown mixer {layer['type']!r}")
+        x = x + y
+        if layer.get("mlp"):
+            h, w = zero_norm(x, eps, T[p + "norm2"]), sub("mlp")
+            x = x + clamped_glu(h @ w["gate"].T, h @ w["up"].T, layer["mlp"]["limit"]) @ w["down"].T
+        if collect is not None:
+            collect.append(x.clone())
+    return zero_norm(x, eps, T["final.norm"]) @ T["head"].T
+
+
 def forward(config, tensors, tokens, collect=None, dtype=torch.float64):
     """Logits [tokens, vocab] of one sequence.  `config` is the parsed config.json, `tensors` name -> tensor.
     `collect`: a list that receives the residual stream after every layer."""
@@ -212,6 +315,8 @@ def forward(config, tensors, tokens, collect=None, dtype=torch.float64):
     T = {n: x.to(dtype) if x.is_floating_point() else x for n, x in tensors.items()}
     if config["architecture"] == "Lerazen":
         return _lerazen(config, T, tokens, collect)
+    if config["architecture"] == "Merulorn":
+        return _merulorn(config, T, tokens, collect)
     pos = torch.arange(len(tokens))
     x = T["embed"][torch.as_tensor(tokens, dtype=torch.long)]
     kv = {}
