@@ -36,6 +36,8 @@ SOURCES = [
     "latent_attn.cu",
     "latent_prefill.cu",
     "grouped_attn.cu",
+    "grouped_prefill.cu",
+    "state_space.cu",
     "moe.cu",
     "delta_scan.cu",
     "stack_step.cu",

@@ -64,6 +64,7 @@ struct WindowAttn {
   int max_blocks, page_heads;   // page_heads: key/value heads of a page
   int k_col, v_col;         // contiguous rows: columns per head of a key / first column of the values
   int group;                // query heads per key/value head
+  const float* gates;       // [tokens][heads] factors of the outputs, or NULL
   __nv_bfloat16* out;
   long long out_ld;         // row pitch
   int heads, vdim, window;
@@ -303,7 +304,8 @@ window_attn_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_const
     }
     mbar_wait(pv_done, (nb - 1) & 1);
     tc_fence_after();
-    const float inv = l_run > 0.f ? 1.0f / l_run : 0.f;
+    float inv = l_run > 0.f ? 1.0f / l_run : 0.f;
+    if (a.gates && r < n_rows) inv *= a.gates[(static_cast<long long>(row0) + r) * a.heads + head];
     __nv_bfloat16* dst = a.out + (static_cast<long long>(row0) + r) * a.out_ld + static_cast<long long>(head) * a.vdim;
 #pragma unroll
     for (int c = 0; c < VD / 32; ++c) {

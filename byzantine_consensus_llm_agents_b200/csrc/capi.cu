@@ -286,6 +286,21 @@ int bcg_gemm_grouped(const void* X, const void* W, void* out, int rows, int N, i
   return rc;
 }
 
+int bcg_state_space(const bcg_stack* m, const bcg_stack_ws* ws, const bcg_step_batch* b, int layer, int n_partials,
+                    long long partial_stride, long long ld, int mode, void* stream) {
+  return state_space_step(m, ws, b, layer, n_partials, partial_stride, ld, mode, S(stream));
+}
+
+int bcg_clamped_glu(const float* z, int n_partials, long long partial_stride, void* out, int act_dtype, int T, int ff,
+                    float limit, float alpha, void* stream) {
+  return clamped_glu_rows(z, n_partials, partial_stride, nullptr, out, act_dtype, T, ff, limit, alpha, S(stream));
+}
+
+int bcg_gemm_bf16_glu(const void* X, const void* W, void* out, int M, int N, int K, float limit, float alpha, int flags,
+                      void* stream) {
+  return gemm_bf16_glu(X, W, out, M, N, K, limit, alpha, flags, S(stream));
+}
+
 int bcg_experts(const bcg_stack* m, const bcg_stack_ws* ws, int layer, int T, int* splits, void* stream) {
   return experts_step(m, ws, layer, T, splits, S(stream));
 }

@@ -50,6 +50,7 @@ struct Gemm2Args {
   int epi;
   void* out;
   long long ld_out;
+  float glu_limit, glu_alpha;   // BCG_EPI_GLU
   int sector_stores;         // fp32 output rows are 32-byte aligned: whole sectors per store
   uint64_t hint_a, hint_b;   // L2 eviction priority of the activation / weight loads
 };
@@ -113,6 +114,11 @@ __device__ __forceinline__ void mbar_arrive_leader(uint64_t* bar) {
 }
 
 __device__ __forceinline__ float silu_mul2(float g, float u) { return g * (1.0f / (1.0f + __expf(-g))) * u; }
+__device__ __forceinline__ float glu_clamp2(float g, float u, float limit, float alpha) {
+  g = fminf(g, limit);
+  u = fminf(fmaxf(u, -limit), limit);
+  return __fdividef(g, 1.0f + __expf(-alpha * g)) * (u + 1.0f);
+}
 
 template <int k2Stages>
 __global__ void __cluster_dims__(2, 1, 1) __launch_bounds__(k2Threads, 1)
@@ -243,7 +249,7 @@ gemm2sm_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_
       const uint32_t taddr = tmem_base + (static_cast<uint32_t>(q * 32) << 16) + static_cast<uint32_t>(acc * k2BlockN);
       const int m = tm * 256 + static_cast<int>(rank) * k2BlockM + row;
       const int n0 = tn * k2BlockN;
-      if (args.epi == BCG_EPI_SWIGLU) {
+      if (args.epi == BCG_EPI_SWIGLU || args.epi == BCG_EPI_GLU) {
         __nv_bfloat16* o = reinterpret_cast<__nv_bfloat16*>(args.out);
 #pragma unroll 1
         for (int c = 0; c < k2BlockN; c += 32) {
@@ -252,10 +258,18 @@ gemm2sm_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_
           tmem_ld_x16(taddr + c + 16, u);
           tmem_ld_wait();
           uint32_t p[8];
+          if (args.epi == BCG_EPI_GLU) {
 #pragma unroll
-          for (int j = 0; j < 8; ++j)
-            p[j] = pack_bf16(silu_mul2(__uint_as_float(g[2 * j]), __uint_as_float(u[2 * j])),
-                             silu_mul2(__uint_as_float(g[2 * j + 1]), __uint_as_float(u[2 * j + 1])));
+            for (int j = 0; j < 8; ++j)
+              p[j] = pack_bf16(glu_clamp2(__uint_as_float(g[2 * j]), __uint_as_float(u[2 * j]), args.glu_limit, args.glu_alpha),
+                               glu_clamp2(__uint_as_float(g[2 * j + 1]), __uint_as_float(u[2 * j + 1]), args.glu_limit,
+                                          args.glu_alpha));
+          } else {
+#pragma unroll
+            for (int j = 0; j < 8; ++j)
+              p[j] = pack_bf16(silu_mul2(__uint_as_float(g[2 * j]), __uint_as_float(u[2 * j])),
+                               silu_mul2(__uint_as_float(g[2 * j + 1]), __uint_as_float(u[2 * j + 1])));
+          }
           if (m < M && n0 + c < N) {
             uint4* dst = reinterpret_cast<uint4*>(o + m * ld + (n0 + c) / 2);
             dst[0] = make_uint4(p[0], p[1], p[2], p[3]);
@@ -333,7 +347,7 @@ gemm2sm_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_
 // Returns BCG_ERR_UNSUPPORTED when the shape is not for this kernel (the caller then uses the
 // single-CTA kernel).
 int gemm2sm_bf16_tn(const void* X, const void* W, void* out, int M, int N, int K, long long ldx, long long ldw,
-                    long long ld_out, int epi, cudaStream_t stream) {
+                    long long ld_out, int epi, float glu_limit, float glu_alpha, cudaStream_t stream) {
   // the last column tile may be partial (the epilogue stores 32 columns at a time), where that wastes little
   if (M < 512 || (N % 32) != 0 || (N % k2BlockN != 0 && N < 8 * k2BlockN)) return BCG_ERR_UNSUPPORTED;
   static const bool off = getenv("BCG_GEMM_2SM") && atoi(getenv("BCG_GEMM_2SM")) == 0;   // tuning knob
@@ -360,6 +374,8 @@ int gemm2sm_bf16_tn(const void* X, const void* W, void* out, int M, int N, int K
   a.epi = epi;
   a.out = out;
   a.ld_out = ld_out;
+  a.glu_limit = glu_limit;
+  a.glu_alpha = glu_alpha;
   a.sector_stores = (reinterpret_cast<uintptr_t>(out) % 32 == 0 && ld_out % 8 == 0) ? 1 : 0;
   CUtensorMap tma, tmb;
   int rc;

@@ -69,6 +69,7 @@ struct GemmArgs {
   __nv_bfloat16* red_xn;     // [M][N]
   float* red_sumsq;          // [tiles_a][kSumsqStride]
   int* red_counters;         // [tiles_a], zero on entry, zero again on exit
+  float glu_limit, glu_alpha;   // BCG_EPI_GLU
   GemmGroups groups;         // GROUPED only; M = rows of all groups, N = weight rows of one
 };
 
@@ -363,7 +364,7 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_a,
               const int m = m0 + c + j;
               if (m < M && n < N) o[m * ld + n] = __float2bfloat16_rn(__uint_as_float(v[j]));
             }
-          } else {  // SWIGLU: rows interleaved [16 gate | 16 up]
+          } else {  // SWIGLU / GLU: rows interleaved [16 gate | 16 up]
             __nv_bfloat16* o = reinterpret_cast<__nv_bfloat16*>(args.out);
             const int nb = (ta * kBlockA + q * 32) / 2 + lane;
 #pragma unroll
@@ -371,7 +372,8 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_a,
               const float g = __uint_as_float(v[j]);
               const float u = __shfl_down_sync(0xffffffffu, g, 16);
               const int m = m0 + c + j;
-              if (lane < 16 && m < M && n < N) o[m * ld + nb] = __float2bfloat16_rn(silu_mul(g, u));
+              if (lane < 16 && m < M && n < N) o[m * ld + nb] = __float2bfloat16_rn(
+                  args.epi == BCG_EPI_GLU ? glu_clamp(g, u, args.glu_limit, args.glu_alpha) : silu_mul(g, u));
             }
           }
         }
@@ -379,7 +381,7 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_a,
         // lanes = activation rows (m), columns = weight rows (n)
         const int m = ta * kBlockA + row;
         const int n0 = tb * BN;
-        if (args.epi == BCG_EPI_SWIGLU || (GROUPED && args.epi == BCG_EPI_GLU)) {
+        if (args.epi == BCG_EPI_SWIGLU || args.epi == BCG_EPI_GLU) {
           __nv_bfloat16* o = reinterpret_cast<__nv_bfloat16*>(args.out) + base;
           float weight = 1.f;
           if (GROUPED && m < M) weight = args.groups.row_weight[first_row[e] + m];
@@ -394,9 +396,9 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_a,
             for (int j = 0; j < 8; ++j) {
               const float g0 = __uint_as_float(g[2 * j]), g1 = __uint_as_float(g[2 * j + 1]);
               const float u0 = __uint_as_float(u[2 * j]), u1 = __uint_as_float(u[2 * j + 1]);
-              if constexpr (GROUPED)
-                p[j] = pack_bf16(glu_clamp(weight * g0, weight * u0, args.groups.glu_limit, args.groups.glu_alpha),
-                                 glu_clamp(weight * g1, weight * u1, args.groups.glu_limit, args.groups.glu_alpha));
+              if (GROUPED || args.epi == BCG_EPI_GLU)
+                p[j] = pack_bf16(glu_clamp(weight * g0, weight * u0, args.glu_limit, args.glu_alpha),
+                                 glu_clamp(weight * g1, weight * u1, args.glu_limit, args.glu_alpha));
               else
                 p[j] = pack_bf16(silu_mul(g0, u0), silu_mul(g1, u1));
             }
@@ -637,6 +639,10 @@ int gemm_splits_for(int M, int N, int K) {
   return best;
 }
 
+static int gemm_dense(const void* X, const void* W, void* out, int M, int N, int K, long long ldx, long long ldw,
+                      long long ld_out, int epi, int splits, int flags, const bcg_gemm_fusion* fu, float glu_limit,
+                      float glu_alpha, cudaStream_t stream);
+
 int gemm_bf16_tn(const void* X, const void* W, void* out, int M, int N, int K, long long ldx,
                  long long ldw, long long ld_out, int epi, int splits, int flags,
                  cudaStream_t stream) {
@@ -646,6 +652,21 @@ int gemm_bf16_tn(const void* X, const void* W, void* out, int M, int N, int K, l
 int gemm_bf16_tn_fused(const void* X, const void* W, void* out, int M, int N, int K, long long ldx,
                        long long ldw, long long ld_out, int epi, int splits, int flags,
                        const bcg_gemm_fusion* fu, cudaStream_t stream) {
+  if (epi < 0 || epi > BCG_EPI_RELU2) {
+    set_last_error("bcg_gemm_bf16_tn", "unknown epilogue");
+    return BCG_ERR_ARG;
+  }
+  return gemm_dense(X, W, out, M, N, K, ldx, ldw, ld_out, epi, splits, flags, fu, 0.f, 0.f, stream);
+}
+
+int gemm_bf16_glu(const void* X, const void* W, void* out, int M, int N, int K, float limit, float alpha, int flags,
+                  cudaStream_t stream) {
+  return gemm_dense(X, W, out, M, N, K, K, K, N / 2, BCG_EPI_GLU, 1, flags, nullptr, limit, alpha, stream);
+}
+
+static int gemm_dense(const void* X, const void* W, void* out, int M, int N, int K, long long ldx, long long ldw,
+                      long long ld_out, int epi, int splits, int flags, const bcg_gemm_fusion* fu, float glu_limit,
+                      float glu_alpha, cudaStream_t stream) {
   if (!X || !W || !out || M <= 0 || N <= 0 || K <= 0) {
     set_last_error("bcg_gemm_bf16_tn", "null pointer or non-positive dimension");
     return BCG_ERR_ARG;
@@ -660,22 +681,23 @@ int gemm_bf16_tn_fused(const void* X, const void* W, void* out, int M, int N, in
     set_last_error("bcg_gemm_bf16_tn", "split-K needs the fp32 partial epilogue");
     return BCG_ERR_ARG;
   }
-  if (epi == BCG_EPI_SWIGLU && (N % 32)) {
-    set_last_error("bcg_gemm_bf16_tn", "SwiGLU epilogue needs N % 32 == 0");
+  const bool paired = epi == BCG_EPI_SWIGLU || epi == BCG_EPI_GLU;
+  if (paired && (N % 32)) {
+    set_last_error("bcg_gemm_bf16_tn", "gated epilogues need N % 32 == 0");
     return BCG_ERR_ARG;
   }
   const bool swap = (M <= 128);
-  if (epi < 0 || epi > BCG_EPI_RELU2 || (epi == BCG_EPI_RELU2 && (swap || N % 16))) {
-    set_last_error("bcg_gemm_bf16_tn", "unknown epilogue, or squared relu with M <= 128 or N % 16");
+  if (epi == BCG_EPI_RELU2 && (swap || N % 16)) {
+    set_last_error("bcg_gemm_bf16_tn", "squared relu with M <= 128 or N % 16");
     return BCG_ERR_ARG;
   }
-  if (!swap && ((epi == BCG_EPI_SWIGLU ? (ld_out % 8) : (epi == BCG_EPI_F32 ? (ld_out % 4) : (ld_out % 8))))) {
+  if (!swap && ((epi == BCG_EPI_F32 ? (ld_out % 4) : (ld_out % 8)))) {
     set_last_error("bcg_gemm_bf16_tn", "ld_out must keep 16-byte row alignment");
     return BCG_ERR_ARG;
   }
   if (!swap && splits == 1 && !(fu && (fu->scale_sumsq || fu->red_counters))) {
     // prefill-sized: 256x256 tiles on CTA pairs when the shape allows it
-    const int rc2 = gemm2sm_bf16_tn(X, W, out, M, N, K, ldx, ldw, ld_out, epi, stream);
+    const int rc2 = gemm2sm_bf16_tn(X, W, out, M, N, K, ldx, ldw, ld_out, epi, glu_limit, glu_alpha, stream);
     if (rc2 != BCG_ERR_UNSUPPORTED) return rc2;
   }
   GemmArgs a = {};
@@ -690,6 +712,8 @@ int gemm_bf16_tn_fused(const void* X, const void* W, void* out, int M, int N, in
   a.out = out;
   a.sector_stores = (reinterpret_cast<uintptr_t>(out) % 32 == 0 && ld_out % 8 == 0) ? 1 : 0;
   a.ld_out = ld_out;
+  a.glu_limit = glu_limit;
+  a.glu_alpha = glu_alpha;
   a.pdl_wait_b = ((flags | launch_flags()) & BCG_GEMM_PDL) ? 1 : 0;
   if (fu && (fu->scale_sumsq || fu->red_counters)) {
     if (!swap || (fu->red_counters && (N % kBlockA))) {
@@ -784,6 +808,8 @@ int gemm_grouped(const void* X, const void* W, void* out, int rows, int N, int K
   a.sector_stores = (reinterpret_cast<uintptr_t>(out) % 32 == 0 && N % 8 == 0) ? 1 : 0;
   a.ld_out = epi == BCG_EPI_GLU ? N / 2 : N;
   a.groups = g;
+  a.glu_limit = g.glu_limit;
+  a.glu_alpha = g.glu_alpha;
   a.pdl_wait_b = (launch_flags() & BCG_GEMM_PDL) ? 1 : 0;
   const int bn = swap ? (g.max_rows <= 16 ? 16 : g.max_rows <= 32 ? 32 : g.max_rows <= 64 ? 64 : 128)
                       : (N % 256 == 0 ? 256 : 128);

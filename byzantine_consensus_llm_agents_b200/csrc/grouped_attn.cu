@@ -1,10 +1,11 @@
-// Grouped-query attention with a linear distance bias, sliding window and query temperature over paged keys and
-// values.
+// Grouped-query attention over paged keys and values, with what a layer has of: a linear distance bias, a sliding
+// window, a query temperature, query and key norms over all heads at once, an output gate per head.
 //
 // A layer's cache is two pools of 16-token pages, keys [page][kv head][16][q_ld] and values [page][kv head][16][v_ld];
 // heads are padded to q_ld / v_ld columns, the padding is zero and stays so.
 //   grouped_in      projection slabs -> queries (bias, temperature), keys and values (bias, value mixing) into the
-//                   pages, squared-relu activations of a parallel feed-forward, routing of a parallel mixture
+//                   pages, squared-relu activations of a parallel feed-forward, routing of a parallel mixture;
+//                   where there are norms or gates, a CTA or a cluster has a whole token (grouped_norm_in)
 //   grouped_plain   one CTA per (token, head), any sizes, fp32 or bf16: the fp32 engine's kernel, and the bf16
 //                   one's for head sizes the kernels below do not take
 //   grouped_decode  single tokens: a cluster per (token, kv head) shares the key pages, a ring of TMA loads and a
@@ -38,7 +39,54 @@ struct GroupedIn {
   int n_tokens, blocks;       // blocks: CTAs per token that share the columns
   MoeRoute route;             // experts = 0: none
   int route_tokens;           // tokens per routing CTA
+  const float *q_norm, *k_norm;   // [heads * dim], [kv_heads * dim] or NULL
+  float* gates;               // [T][heads] or NULL; logits are columns gate_col.. of proj
+  int gate_col;
+  float gate_scale, eps;
 };
+
+// Where a token's columns go.
+struct InToken {
+  long long t, page;
+  int slot, in_page;
+  float temp;
+  __device__ __forceinline__ InToken(const GroupedIn& a, long long t_) : t(t_) {
+    const int pos = a.positions[t];
+    slot = a.slot_map[t];
+    temp = 1.0f + a.temp_coef * logf(floorf(static_cast<float>(pos + 1) / a.temp_every) + 1.0f);
+    page = slot >= 0 ? slot / a.page_size : 0;
+    in_page = slot >= 0 ? slot % a.page_size : 0;
+  }
+};
+
+// Biased (and normed) columns c.. of q | k | v to the query buffer or the token's place in the pages.
+template <typename T, int V>
+__device__ __forceinline__ void store_columns(const GroupedIn& a, const InToken& tok, int c, Vec<V>& x) {
+  const int nq = a.heads * a.dim, nk = nq + a.kv_heads * a.dim;
+  const long long t = tok.t;
+  if (c < nq) {
+    const int h = c / a.dim, i = c - h * a.dim;
+#pragma unroll
+    for (int k = 0; k < V; ++k) x.x[k] *= tok.temp;
+    store_vec<V>(static_cast<T*>(a.q) + (t * a.heads + h) * a.q_ld + i, x);
+  } else if (c < nk) {
+    const int g = (c - nq) / a.dim, i = c - nq - g * a.dim;
+    if (tok.slot >= 0)
+      store_vec<V>(static_cast<T*>(a.k_cache) + ((tok.page * a.kv_heads + g) * a.page_size + tok.in_page) * a.q_ld + i, x);
+  } else {
+    const int o = c - nk, g = o / a.vdim, i = o - g * a.vdim;
+    float* first = a.v_first + t * (a.kv_heads * a.vdim) + o;
+    if (a.v_role == BCG_VALUES_FIRST) {
+      store_vec<V>(first, x);
+    } else if (a.v_role == BCG_VALUES_MIX) {
+      const Vec<V> f = load_vec<V>(first);
+#pragma unroll
+      for (int k = 0; k < V; ++k) x.x[k] = (1.0f - a.v_mix) * x.x[k] + a.v_mix * f.x[k];
+    }
+    if (tok.slot >= 0)
+      store_vec<V>(static_cast<T*>(a.v_cache) + ((tok.page * a.kv_heads + g) * a.page_size + tok.in_page) * a.v_ld + i, x);
+  }
+}
 
 // grid: `blocks` CTAs per token, then the routing CTAs (`route_tokens` tokens each).  Columns go to their destination four at a
 // time (V = 4) or one by one.
@@ -58,40 +106,13 @@ grouped_in_kernel(const GroupedIn a) {
   const long long t = blockIdx.x / a.blocks;
   const int part = blockIdx.x % a.blocks;
   const float* row = a.proj + t * a.ld;
-  const int pos = a.positions[t], slot = a.slot_map[t];
-  const float temp = 1.0f + a.temp_coef * logf(floorf(static_cast<float>(pos + 1) / a.temp_every) + 1.0f);
-  const int nq = a.heads * a.dim, nk = nq + a.kv_heads * a.dim, nv = nk + a.kv_heads * a.vdim;
-  const long long page = slot >= 0 ? slot / a.page_size : 0;
-  const int in_page = slot >= 0 ? slot % a.page_size : 0;
+  const InToken tok(a, t);
+  const int nv = a.heads * a.dim + a.kv_heads * (a.dim + a.vdim);
   const int step = a.blocks * kInThreads * V;
-  auto store = [&](int c, Vec<V>& x) {
-    if (c < nq) {
-      const int h = c / a.dim, i = c - h * a.dim;
-#pragma unroll
-      for (int k = 0; k < V; ++k) x.x[k] *= temp;
-      store_vec<V>(static_cast<T*>(a.q) + (t * a.heads + h) * a.q_ld + i, x);
-    } else if (c < nk) {
-      const int g = (c - nq) / a.dim, i = c - nq - g * a.dim;
-      if (slot >= 0)
-        store_vec<V>(static_cast<T*>(a.k_cache) + ((page * a.kv_heads + g) * a.page_size + in_page) * a.q_ld + i, x);
-    } else {
-      const int o = c - nk, g = o / a.vdim, i = o - g * a.vdim;
-      float* first = a.v_first + t * (nv - nk) + o;
-      if (a.v_role == BCG_VALUES_FIRST) {
-        store_vec<V>(first, x);
-      } else if (a.v_role == BCG_VALUES_MIX) {
-        const Vec<V> f = load_vec<V>(first);
-#pragma unroll
-        for (int k = 0; k < V; ++k) x.x[k] = (1.0f - a.v_mix) * x.x[k] + a.v_mix * f.x[k];
-      }
-      if (slot >= 0)
-        store_vec<V>(static_cast<T*>(a.v_cache) + ((page * a.kv_heads + g) * a.page_size + in_page) * a.v_ld + i, x);
-    }
-  };
   for (int c = (part * kInThreads + threadIdx.x) * V; c < nv; c += step) {
     Vec<V> x = slab_sum_vec<V>(row + c, a.n_partials, a.pstride);
     x.add(load_vec<V>(a.bias + c));
-    store(c, x);
+    store_columns<T, V>(a, tok, c, x);
   }
   for (int c = (part * kInThreads + threadIdx.x) * V; c < a.ff; c += step) {
     Vec<V> x = slab_sum_vec<V>(row + a.act_from + c, a.n_partials, a.pstride);
@@ -104,9 +125,75 @@ grouped_in_kernel(const GroupedIn a) {
   }
 }
 
+// One token per CTA, or per cluster of CL CTAs that have a range of its columns each: query and key norms span all
+// heads.
+template <typename T, int V, int CL>
+__global__ void __launch_bounds__(kInThreads)
+grouped_norm_in_kernel(const GroupedIn a) {
+  extern __shared__ float4 stage_raw[];
+  float* stage = reinterpret_cast<float*>(stage_raw);
+  __shared__ RowSum<kInThreads, CL, 2> sh;
+  pdl_launch_dependents();
+  pdl_wait();
+  const int cta = CL > 1 ? static_cast<int>(blockIdx.x) : 0;
+  const InToken tok(a, CL > 1 ? blockIdx.y : blockIdx.x);
+  const float* row = a.proj + tok.t * a.ld;
+  const int nq = a.heads * a.dim, nk = nq + a.kv_heads * a.dim, nv = nk + a.kv_heads * a.vdim;
+  const int per = (nv / V + CL - 1) / CL * V;
+  const int c0 = cta * per, c1 = min(nv, c0 + per);
+  float ss[2] = {0.f, 0.f};     // queries, keys
+  for (int c = c0 + threadIdx.x * V; c < c1; c += kInThreads * V) {
+    Vec<V> x = slab_sum_vec<V>(row + c, a.n_partials, a.pstride);
+    x.add(load_vec<V>(a.bias + c));
+    store_vec<V>(stage + c - c0, x);
+    if (c < nq) ss[0] += x.sumsq();
+    else if (c < nk) ss[1] += x.sumsq();
+  }
+  if (a.gates)
+    for (int h = cta * kInThreads + threadIdx.x; h < a.heads; h += CL * kInThreads)
+      a.gates[tok.t * a.heads + h] = a.gate_scale * sigmoid_f32(slab_sum(row + a.gate_col + h, a.n_partials, a.pstride));
+  row_sum<kInThreads, CL, 2>(sh, ss, 0);
+  const float inv_q = rsqrtf(ss[0] / static_cast<float>(nq) + a.eps);
+  const float inv_k = rsqrtf(ss[1] / static_cast<float>(nk - nq) + a.eps);
+  for (int c = c0 + threadIdx.x * V; c < c1; c += kInThreads * V) {
+    Vec<V> x = load_vec<V>(stage + c - c0);
+    const float* w = c < nq ? (a.q_norm ? a.q_norm + c : nullptr) : c < nk ? (a.k_norm ? a.k_norm + c - nq : nullptr) : nullptr;
+    if (w) {
+      const Vec<V> ww = load_vec<V>(w);
+      const float inv = c < nq ? inv_q : inv_k;
+#pragma unroll
+      for (int k = 0; k < V; ++k) x.x[k] = x.x[k] * inv * ww.x[k];
+    }
+    store_columns<T, V>(a, tok, c, x);
+  }
+  row_sum_exit<CL>();
+}
+
+template <typename T, int V>
+static int norm_in_t(const GroupedIn& a, cudaStream_t st) {
+  const int cols = a.heads * a.dim + a.kv_heads * (a.dim + a.vdim);
+  if (a.n_tokens <= 128 && cols >= 1024) {
+    const size_t sm = static_cast<size_t>((cols / V + 7) / 8 * V) * 4;
+    BCG_TRY(ensure_dynamic_smem(reinterpret_cast<const void*>(grouped_norm_in_kernel<T, V, 8>), 48 * 1024));
+    BCG_CUDA_CHECK(launch_cluster(grouped_norm_in_kernel<T, V, 8>, dim3(8, a.n_tokens), dim3(kInThreads), 8, sm, st, a));
+  } else {
+    BCG_TRY(ensure_dynamic_smem(reinterpret_cast<const void*>(grouped_norm_in_kernel<T, V, 1>), 200 * 1024));
+    BCG_CUDA_CHECK(launch_k(grouped_norm_in_kernel<T, V, 1>, dim3(a.n_tokens), dim3(kInThreads), static_cast<size_t>(cols) * 4,
+                            st, a));
+  }
+  return BCG_OK;
+}
+
 template <typename T>
 static int grouped_in_t(const GroupedIn& a, cudaStream_t st) {
   const bool wide = ((a.dim | a.vdim | a.ff | a.act_from) & 3) == 0 && a.ld % 4 == 0 && a.pstride % 4 == 0;
+  if (a.q_norm || a.k_norm || a.gates) {
+    if (a.ff > 0 || a.route.experts > 0 || a.heads * a.dim + a.kv_heads * (a.dim + a.vdim) > 51200) {
+      set_last_error("bcg_grouped_in", "norms and gates: no parallel feed-forward, at most 51,200 columns");
+      return BCG_ERR_UNSUPPORTED;
+    }
+    return wide ? norm_in_t<T, 4>(a, st) : norm_in_t<T, 1>(a, st);
+  }
   const dim3 grid(a.n_tokens * a.blocks + (a.route.experts > 0 ? (a.n_tokens + a.route_tokens - 1) / a.route_tokens : 0));
   const size_t sm = static_cast<size_t>(route_words(a.route.experts, kInThreads)) * 4;
   if (sm > 48 * 1024) {
@@ -149,6 +236,12 @@ int grouped_in(const bcg_stack* m, const bcg_layer* l, const bcg_stack_ws* ws, c
   a.act_from = with_act ? l->n_qkv : 0;
   a.act = static_cast<char*>(ws->mix) + l->act_col * act_bytes;
   a.act_ld = l->mix_ld;
+  a.q_norm = l->q_norm;
+  a.k_norm = l->k_norm;
+  a.gates = l->gated ? ws->gates : nullptr;
+  a.gate_col = l->gate_col;
+  a.gate_scale = l->gate_scale;
+  a.eps = m->eps;
   if (l->experts > 0) a.route = moe_route(l, ws);
   const int cols = l->heads * l->dim + l->kv_heads * (l->dim + l->vdim);
   a.blocks = b->T <= 128 ? max(1, ((cols > a.ff ? cols : a.ff) + kInThreads * 4 - 1) / (kInThreads * 4)) : 1;
@@ -162,7 +255,7 @@ constexpr int kGpThreads = 128, kGpKeys = 256;
 
 struct GroupedAttn {
   const void *q, *k_cache, *v_cache;
-  const float* slopes;
+  const float *slopes, *gates;
   const int *rows, *positions, *row_seq, *block_table;
   int max_blocks, page_size;
   void* out;
@@ -237,7 +330,7 @@ grouped_plain_kernel(const GroupedAttn a) {
     }
   }
   __syncthreads();
-  const float inv = 1.0f / l;
+  const float inv = (a.gates ? a.gates[t * a.heads + h] : 1.0f) / l;
   T* dst = static_cast<T*>(a.out) + t * a.out_ld + static_cast<long long>(h) * a.vdim;
   for (int r = threadIdx.x; r < a.vdim; r += kGpThreads) dst[r] = from_f32<T>(oc[r] * inv);
 }
@@ -249,6 +342,7 @@ static GroupedAttn attn_args(const bcg_stack* m, const bcg_layer* l, const bcg_s
   a.k_cache = l->cache;
   a.v_cache = l->cache_v;
   a.slopes = l->slopes;
+  a.gates = l->gated ? ws->gates : nullptr;
   a.rows = rows;
   a.positions = b->positions;
   a.row_seq = b->row_seq;
@@ -475,6 +569,7 @@ grouped_decode_kernel(const __grid_constant__ CUtensorMap k_map, const __grid_co
       den = den * f0 + other.y * f1;
       top = up;
     }
+    if (a.gates) x *= a.gates[static_cast<long long>(t) * a.heads + h0 + r];
     dst[static_cast<long long>(r) * a.vdim + c] = __float2bfloat16(x / den);
   }
   if (n_cta > 1) cluster.sync();                     // nobody leaves while its shared memory is being read
@@ -555,6 +650,7 @@ static int grouped_prefill(const bcg_layer* l, const bcg_stack_ws* ws, const bcg
   a.tiles = b->tiles;
   a.n_tiles = b->n_tiles;
   a.slopes = l->slopes;
+  a.gates = l->gated ? ws->gates : nullptr;
   a.block_table = b->block_table;
   a.max_blocks = b->max_blocks;
   a.page_heads = l->kv_heads;
@@ -565,7 +661,8 @@ static int grouped_prefill(const bcg_layer* l, const bcg_stack_ws* ws, const bcg
   a.vdim = l->vdim;
   a.window = l->window;
   a.scale_log2e = l->scale * kLog2e;
-  return window_attn<true, true>(l->q_ld, l->v_ld, qm, km, vm, a, st);
+  return l->slopes ? window_attn<true, true>(l->q_ld, l->v_ld, qm, km, vm, a, st)
+                   : window_attn_paged(l->q_ld, l->v_ld, qm, km, vm, a, st);
 }
 
 int grouped_attention(const bcg_stack* m, const bcg_stack_ws* ws, const bcg_step_batch* b, const bcg_layer* l, int mode,
@@ -574,8 +671,8 @@ int grouped_attention(const bcg_stack* m, const bcg_stack_ws* ws, const bcg_step
   const bool tensor = m->act_dtype == BCG_DT_BF16 && mode == 0 && m->page_size == kGdPage && padded_head(l->q_ld, l->v_ld);
   if (!tensor) return grouped_plain(m, l, ws, b, nullptr, b->T, st);
   if (b->n_tiles > 0) {
-    // the prompt kernel stores 16 bytes at a time and wants slopes
-    if (l->slopes && l->vdim % 8 == 0 && l->mix_ld % 8 == 0) BCG_TRY(grouped_prefill(l, ws, b, st));
+    // the prompt kernel stores 16 bytes at a time; without slopes it takes maxima in front of the scale
+    if ((l->slopes || l->scale > 0.f) && l->vdim % 8 == 0 && l->mix_ld % 8 == 0) BCG_TRY(grouped_prefill(l, ws, b, st));
     else BCG_TRY(grouped_plain(m, l, ws, b, nullptr, b->T, st));   // single tokens are recomputed below: harmless
   }
   if (n_single > 0) BCG_TRY(grouped_decode(m, l, ws, b, st));

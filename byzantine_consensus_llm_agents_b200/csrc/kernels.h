@@ -1,5 +1,6 @@
 // Internal C++ declarations shared by the .cu files; the public C ABI is include/bcg_b200.h.
 #pragma once
+#include <cuda_bf16.h>
 #include <cuda_runtime.h>
 #include <stdint.h>
 
@@ -15,6 +16,9 @@ int gemm_bf16_tn(const void* X, const void* W, void* out, int M, int N, int K, l
 int gemm_bf16_tn_fused(const void* X, const void* W, void* out, int M, int N, int K, long long ldx,
                        long long ldw, long long ld_out, int epi, int splits, int flags,
                        const bcg_gemm_fusion* fusion, cudaStream_t stream);
+// epilogue BCG_EPI_GLU: W rows interleaved [16 gate | 16 up], out bf16 [M, N / 2]
+int gemm_bf16_glu(const void* X, const void* W, void* out, int M, int N, int K, float limit, float alpha, int flags,
+                  cudaStream_t stream);
 int gemm_splits_for(int M, int N, int K);
 // Rows sorted by group (mixture of experts); internal epilogue BCG_EPI_GLU: columns interleaved [16 gate | 16 up],
 // each row's accumulators times its weight, clamped gated unit, bf16 [rows, N / 2]
@@ -32,7 +36,7 @@ int gemm_any_grouped(const void* X, int x_dtype, const void* W, float* out, int 
                      cudaStream_t stream);
 // Prefill shapes on CTA pairs (tcgen05.mma.cta_group::2); BCG_ERR_UNSUPPORTED = not a shape for it
 int gemm2sm_bf16_tn(const void* X, const void* W, void* out, int M, int N, int K, long long ldx, long long ldw,
-                    long long ld_out, int epi, cudaStream_t stream);
+                    long long ld_out, int epi, float glu_limit, float glu_alpha, cudaStream_t stream);
 // TMA descriptor of a row-major bf16 matrix (rows x K, pitch ld elements): boxes of box_rows x 64
 // elements land in shared memory 128B-swizzled, out-of-bounds elements read as zero.
 int make_tmap_bf16_sw128(CUtensorMap* m, const void* ptr, long long rows, long long K, long long ld,
@@ -84,10 +88,19 @@ struct NormExtra {
   int per_row = 0, n_partials = 1;
   long long partial_stride = 0;
 };
-// layer stacks (stack_*.cu, latent_*.cu, delta_scan.cu, gemm_simt.cu); act_dtype = BCG_DT_*
-// pos_embed (bf16 [n_pos, d]) may be NULL; zero[0..n_zero) is set to zero on the way
-int embed_norm(const int* ids, const void* embed, const int* positions, const void* pos_embed, int n_pos, const float* w,
-               float* residual, void* xn, int act_dtype, int T, int d, float eps, int* zero, int n_zero,
+// layer stacks (stack_*.cu, latent_*.cu, grouped_*.cu, delta_scan.cu, state_space.cu, moe.cu, gemm_simt.cu); act_dtype = BCG_DT_*
+// What the embedding kernel adds and multiplies; zero[0..n_zero) is set to zero on the way.
+struct EmbedArgs {
+  const int *ids, *positions;
+  const __nv_bfloat16* embed;
+  float scale;
+  const __nv_bfloat16* pos_embed;   // [n_pos, d] or NULL
+  int n_pos;
+  const double* pos_turns;          // [(d + 1) / 2] turns per position, or NULL: sin, cos in turn
+  int* zero;
+  int n_zero;
+};
+int embed_norm(const EmbedArgs& a, const float* w, float* residual, void* xn, int act_dtype, int T, int d, float eps,
                cudaStream_t stream);
 int rows_norm(const float* residual, const int* rows, const float* w, void* xn, int act_dtype, int n, int d,
               float eps, cudaStream_t stream);
@@ -123,6 +136,17 @@ int grouped_attention(const bcg_stack* m, const bcg_stack_ws* ws, const bcg_step
 // ws->xn through the layer's experts into ws->moe_out (*splits slabs), rows ws->moe_row
 int experts(const bcg_stack* m, const bcg_layer* l, const bcg_stack_ws* ws, int T, int* splits, cudaStream_t stream);
 int moe_splits(int T, int top, int N, int K);
+// clamped gated unit of slabs [rows][2 * ff_ld] (16 gate | 16 up); row_weight (NULL: 1) scales both
+int clamped_glu_rows(const float* z, int n_partials, long long pstride, const float* row_weight, void* out, int act_dtype,
+                     int rows, int ff_ld, float limit, float alpha, cudaStream_t stream);
+struct WindowAttn;
+// paged prompt attention without a distance bias (grouped_prefill.cu)
+int window_attn_paged(int q_ld, int v_ld, const CUtensorMap& qm, const CUtensorMap& km, const CUtensorMap& vm,
+                      const WindowAttn& a, cudaStream_t stream);
+int state_space(const bcg_stack* m, const bcg_layer* l, const bcg_stack_ws* ws, const bcg_step_batch* b, int n_partials,
+                long long pstride, long long ld, int mode, cudaStream_t stream);
+int state_space_step(const bcg_stack* m, const bcg_stack_ws* ws, const bcg_step_batch* b, int layer, int n_partials,
+                     long long pstride, long long ld, int mode, cudaStream_t stream);
 int grouped_in_step(const bcg_stack* m, const bcg_stack_ws* ws, const bcg_step_batch* b, int layer, int n_partials,
                     long long pstride, long long ld, int with_act, cudaStream_t stream);
 int grouped_attention_step(const bcg_stack* m, const bcg_stack_ws* ws, const bcg_step_batch* b, int layer, int mode,

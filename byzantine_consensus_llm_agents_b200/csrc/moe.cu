@@ -40,7 +40,7 @@ moe_glu_kernel(const float* __restrict__ z, int n_partials, long long pstride, c
   pdl_launch_dependents();
   pdl_wait();
   const long long row = blockIdx.x;
-  const float w = row_weight[row];
+  const float w = row_weight ? row_weight[row] : 1.f;
   const float* src = z + row * 2 * ff_ld;
   for (int c = (blockIdx.y * kMoeThreads + threadIdx.x) * 4; c < ff_ld; c += gridDim.y * kMoeThreads * 4) {
     const float* p = src + (c >> 4) * 32 + (c & 15);
@@ -50,6 +50,23 @@ moe_glu_kernel(const float* __restrict__ z, int n_partials, long long pstride, c
     for (int k = 0; k < 4; ++k) y.x[k] = clamped_glu(w * g.x[k], w * u.x[k], limit, alpha);
     store_vec<4>(out + row * ff_ld + c, y);
   }
+}
+
+int clamped_glu_rows(const float* z, int n_partials, long long pstride, const float* row_weight, void* out, int act_dtype,
+                     int rows, int ff_ld, float limit, float alpha, cudaStream_t st) {
+  if (!z || !out || rows <= 0 || ff_ld <= 0 || ff_ld % 16 || n_partials < 1) {
+    set_last_error("bcg_clamped_glu", "bad argument (ff % 16)");
+    return BCG_ERR_ARG;
+  }
+  const int per = rows <= 1024 ? (ff_ld + kMoeThreads * 4 - 1) / (kMoeThreads * 4) : 1;
+  const dim3 grid(rows, per);
+  if (act_dtype == BCG_DT_F32)
+    BCG_CUDA_CHECK(launch_k(moe_glu_kernel<float>, grid, dim3(kMoeThreads), 0, st, z, n_partials, pstride, row_weight,
+                            static_cast<float*>(out), ff_ld, limit, alpha));
+  else
+    BCG_CUDA_CHECK(launch_k(moe_glu_kernel<__nv_bfloat16>, grid, dim3(kMoeThreads), 0, st, z, n_partials, pstride, row_weight,
+                            static_cast<__nv_bfloat16*>(out), ff_ld, limit, alpha));
+  return BCG_OK;
 }
 
 static bool moe_tensor(const bcg_stack* m, const bcg_layer* l, int T, int N, int K) {
@@ -102,15 +119,8 @@ int experts(const bcg_stack* m, const bcg_layer* l, const bcg_stack_ws* ws, int 
     int s;
     BCG_TRY(expert_gemm(m, l, ws, T, ws->moe_x, l->w_experts_in, ws->moe_proj, ws->moe_proj_floats, 2 * ff, d, BCG_EPI_F32,
                         &s, st));
-    const int per = T <= 128 ? (ff + kMoeThreads * 4 - 1) / (kMoeThreads * 4) : 1;
-    const long long stride = static_cast<long long>(rows) * 2 * ff;
-    if (m->act_dtype == BCG_DT_F32)
-      BCG_CUDA_CHECK(launch_k(moe_glu_kernel<float>, dim3(rows, per), dim3(kMoeThreads), 0, st, ws->moe_proj, s, stride,
-                              ws->moe_row_weight, static_cast<float*>(ws->moe_h), ff, l->glu_limit, l->glu_alpha));
-    else
-      BCG_CUDA_CHECK(launch_k(moe_glu_kernel<__nv_bfloat16>, dim3(rows, per), dim3(kMoeThreads), 0, st, ws->moe_proj, s,
-                              stride, ws->moe_row_weight, static_cast<__nv_bfloat16*>(ws->moe_h), ff, l->glu_limit,
-                              l->glu_alpha));
+    BCG_TRY(clamped_glu_rows(ws->moe_proj, s, static_cast<long long>(rows) * 2 * ff, ws->moe_row_weight, ws->moe_h,
+                             m->act_dtype, rows, ff, l->glu_limit, l->glu_alpha, st));
   }
   return expert_gemm(m, l, ws, T, ws->moe_h, l->w_experts_out, ws->moe_out, ws->moe_out_floats, d, ff, BCG_EPI_F32, splits,
                      st);

@@ -1,5 +1,5 @@
 // Row-wise kernels of layer stacks:
-//   embed_norm      x = E[ids] (+ P[positions]);  xn = rmsnorm(x) * w
+//   embed_norm      x = scale * E[ids] (+ P[positions] or sinusoids);  xn = rmsnorm(x) * w
 //   sandwich_norm   x += rmsnorm(delta) * w_post (or += delta);  xn = rmsnorm(x) * w_next
 //                   delta may have a bias and rows of a second source (a token's experts) added
 //   rows_norm       xn[i] = rmsnorm(x[rows[i]]) * w
@@ -18,36 +18,38 @@ constexpr int kClusterMaxRows = 128;
 
 template <typename T, int V>
 __global__ void __launch_bounds__(kRowT)
-embed_norm_kernel(const int* __restrict__ ids, const __nv_bfloat16* __restrict__ embed,
-                  const int* __restrict__ positions, const __nv_bfloat16* __restrict__ pos_embed, int n_pos,
-                  const float* __restrict__ w, float* __restrict__ residual, T* __restrict__ xn, int d, float eps,
-                  int* __restrict__ zero, int n_zero) {
+embed_norm_kernel(const EmbedArgs a, const float* __restrict__ w, float* __restrict__ residual, T* __restrict__ xn, int d,
+                  float eps) {
   __shared__ RowSum<kRowT, 1, 1> sh;
   pdl_launch_dependents();
   pdl_wait();
-  const long long t = blockIdx.x, row = ids[t];
-  for (int i = blockIdx.x * kRowT + threadIdx.x; i < n_zero; i += gridDim.x * kRowT) zero[i] = 0;
+  const long long t = blockIdx.x, row = a.ids[t];
+  for (int i = blockIdx.x * kRowT + threadIdx.x; i < a.n_zero; i += gridDim.x * kRowT) a.zero[i] = 0;
   const __nv_bfloat16* pos = nullptr;
-  if (pos_embed) pos = pos_embed + static_cast<long long>(min(positions[t], n_pos - 1)) * d;
-  auto token = [&](int v) {
-    Vec<V> x = load_vec<V>(embed + row * d + v);
-    if (pos) {
-      const Vec<V> p = load_vec<V>(pos + v);
-#pragma unroll
-      for (int k = 0; k < V; ++k) x.x[k] += p.x[k];
-    }
-    return x;
-  };
+  if (a.pos_embed) pos = a.pos_embed + static_cast<long long>(min(a.positions[t], a.n_pos - 1)) * d;
+  const double at = a.pos_turns ? a.positions[t] : 0;
   float ss[1] = {0.f};
   for (int v = threadIdx.x * V; v < d; v += kRowT * V) {
-    const Vec<V> x = token(v);
-    store_vec<V>(residual + t * d + v, x);
+    Vec<V> x = load_vec<V>(a.embed + row * d + v);
+#pragma unroll
+    for (int k = 0; k < V; ++k) x.x[k] *= a.scale;
+    if (pos) x.add(load_vec<V>(pos + v));
+    if (a.pos_turns) {
+      // whole turns are taken off in double precision: the angle is exact at any position
+#pragma unroll
+      for (int k = 0; k < V; ++k) {
+        const double turns = at * a.pos_turns[(v + k) >> 1];
+        const float half = static_cast<float>(2.0 * (turns - rint(turns)));
+        x.x[k] += ((v + k) & 1) ? cospif(half) : sinpif(half);
+      }
+    }
+    store_vec<V>(residual + t * d + v, x);      // read again below by the same thread
     ss[0] += x.sumsq();
   }
   row_sum<kRowT, 1, 1>(sh, ss, 0);
   const float inv = rsqrtf(ss[0] / static_cast<float>(d) + eps);
   for (int v = threadIdx.x * V; v < d; v += kRowT * V) {
-    Vec<V> x = token(v);
+    Vec<V> x = load_vec<V>(residual + t * d + v);
     const Vec<V> ww = load_vec<V>(w + v);
 #pragma unroll
     for (int k = 0; k < V; ++k) x.x[k] *= inv * ww.x[k];
@@ -181,20 +183,15 @@ poly_norm_kernel(const float* __restrict__ z, int n_partials, long long partial_
   } while (0)
 
 template <typename T, int V>
-static int embed_t(const int* ids, const void* embed, const int* positions, const void* pos_embed, int n_pos,
-                   const float* w, float* residual, void* xn, int T_rows, int d, float eps, int* zero, int n_zero,
+static int embed_t(const EmbedArgs& a, const float* w, float* residual, void* xn, int T_rows, int d, float eps,
                    cudaStream_t st) {
-  BCG_CUDA_CHECK(launch_k(embed_norm_kernel<T, V>, dim3(T_rows), dim3(kRowT), 0, st, ids,
-                          static_cast<const __nv_bfloat16*>(embed), positions,
-                          static_cast<const __nv_bfloat16*>(pos_embed), n_pos, w, residual, static_cast<T*>(xn), d, eps,
-                          zero, n_zero));
+  BCG_CUDA_CHECK(launch_k(embed_norm_kernel<T, V>, dim3(T_rows), dim3(kRowT), 0, st, a, w, residual, static_cast<T*>(xn), d,
+                          eps));
   return BCG_OK;
 }
-int embed_norm(const int* ids, const void* embed, const int* positions, const void* pos_embed, int n_pos, const float* w,
-               float* residual, void* xn, int act_dtype, int T, int d, float eps, int* zero, int n_zero,
+int embed_norm(const EmbedArgs& a, const float* w, float* residual, void* xn, int act_dtype, int T, int d, float eps,
                cudaStream_t st) {
-  BCG_BY_TYPE(embed_t, d, act_dtype, ids, embed, positions, pos_embed, n_pos, w, residual, xn, T, d, eps, zero, n_zero,
-              st);
+  BCG_BY_TYPE(embed_t, d, act_dtype, a, w, residual, xn, T, d, eps, st);
 }
 
 template <typename T, int V>

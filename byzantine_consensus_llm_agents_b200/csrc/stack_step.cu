@@ -144,6 +144,28 @@ static int parallel_layer(const bcg_stack* m, const bcg_stack_ws* ws, const bcg_
                        extra, st);
 }
 
+// Gate and up products with the clamped unit: in the GEMM's epilogue where K is not split, else behind the slabs.
+static int glu_up(const bcg_stack* m, const bcg_stack_ws* ws, const bcg_layer* l, int T, cudaStream_t st) {
+  const int n = 2 * l->ff, d = m->d_model;
+  int s = stack_splits(m->act_dtype, T, n, d);
+  if (s == 1 && tensor_gemm(m->act_dtype, T, n, d))
+    return gemm_bf16_glu(ws->xn, l->w_up, ws->act, T, n, d, l->glu_limit, l->glu_alpha, launch_flags() & BCG_GEMM_PDL, st);
+  BCG_TRY(project(m, ws->xn, l->w_up, ws->proj, ws->proj_floats, T, n, d, &s, st));
+  return clamped_glu_rows(ws->proj, s, static_cast<long long>(T) * n, nullptr, ws->act, m->act_dtype, T, l->ff, l->glu_limit,
+                          l->glu_alpha, st);
+}
+
+int state_space_step(const bcg_stack* m, const bcg_stack_ws* ws, const bcg_step_batch* b, int layer, int n_partials,
+                     long long pstride, long long ld, int mode, cudaStream_t st) {
+  BCG_TRY(check_stack(m, ws));
+  if (!b || b->T <= 0 || b->T > ws->T_max || n_partials < 1 || layer < 0 || layer >= m->n_layers ||
+      m->layers[layer].ssm_heads <= 0) {
+    set_last_error("bcg_state_space", "not a state-space layer, or a bad batch");
+    return BCG_ERR_ARG;
+  }
+  return state_space(m, &m->layers[layer], ws, b, n_partials, pstride, ld, mode, st);
+}
+
 int stack_step(const bcg_stack* m, const bcg_stack_ws* ws, const bcg_step_batch* b, cudaStream_t st) {
   BCG_TRY(check_stack(m, ws));
   if (!b || b->T <= 0 || b->T > ws->T_max || b->n_seqs <= 0 || !b->ids || !b->positions || !b->slot_map ||
@@ -154,8 +176,10 @@ int stack_step(const bcg_stack* m, const bcg_stack_ws* ws, const bcg_step_batch*
   FlagScope scope(b->flags & BCG_GEMM_PDL);
   const int T = b->T, d = m->d_model, dt = m->act_dtype;
   const void* gathered = nullptr;
-  BCG_TRY(embed_norm(b->ids, m->embed, b->positions, m->pos_embed, m->n_pos, m->layers[0].norm1, ws->residual, ws->xn, dt,
-                     T, d, m->eps, ws->moe_counts, ws->moe_counts_n, st));
+  const EmbedArgs embed = {b->ids, b->positions, static_cast<const __nv_bfloat16*>(m->embed), m->embed_scale,
+                           static_cast<const __nv_bfloat16*>(m->pos_embed), m->n_pos, m->pos_turns, ws->moe_counts,
+                           ws->moe_counts_n};
+  BCG_TRY(embed_norm(embed, m->layers[0].norm1, ws->residual, ws->xn, dt, T, d, m->eps, st));
   for (int i = 0; i < m->n_layers; ++i) {
     const bcg_layer* l = &m->layers[i];
     const float* next = i + 1 < m->n_layers ? m->layers[i + 1].norm1 : m->final_norm;
@@ -183,16 +207,30 @@ int stack_step(const bcg_stack* m, const bcg_stack_ws* ws, const bcg_step_batch*
       BCG_TRY(delta_scan(l, ws->proj, s, in_stride, l->n_in, ws->decay, sd, static_cast<long long>(T) * mix_out,
                          b->positions, b->slot_map, b->seq_start, b->state_slots, b->n_seqs, T == b->n_seqs, ws->mix,
                          dt, m->eps, st));
+    } else if (l->mixer == BCG_MIXER_GROUPED_ATTN || (l->mixer == BCG_MIXER_STATE_SPACE && l->ssm_heads > 0)) {
+      // attention and a state-space mixer, or one of them, behind one input projection; their outputs lie side by side
+      mix_out = l->mix_ld;
+      if (l->mixer == BCG_MIXER_GROUPED_ATTN) {
+        BCG_TRY(grouped_in(m, l, ws, b, s, in_stride, l->n_in, false, st));
+        BCG_TRY(grouped_attention(m, ws, b, l, 0, st));
+      }
+      if (l->ssm_heads > 0) BCG_TRY(state_space(m, l, ws, b, s, in_stride, l->n_in, 0, st));
     } else {
       set_last_error("bcg_stack_step", "unknown mixer");
       return BCG_ERR_UNSUPPORTED;
     }
     BCG_TRY(project(m, ws->mix, l->w_out, ws->proj, ws->proj_floats, T, d, mix_out, &s, st));
+    NormExtra extra;
+    extra.bias = l->out_bias;
     BCG_TRY(sandwich_norm(ws->residual, ws->proj, s, static_cast<long long>(T) * d, l->norm1b, l->ff ? l->norm2 : next,
-                          ws->xn, dt, T, d, m->eps, {}, st));
+                          ws->xn, dt, T, d, m->eps, extra, st));
     if (l->ff) {
-      BCG_TRY(project(m, ws->xn, l->w_up, ws->proj, ws->proj_floats, T, l->ff, d, &s, st));
-      BCG_TRY(poly_norm(ws->proj, s, static_cast<long long>(T) * l->ff, l->act_coef, ws->act, dt, T, l->ff, m->eps, st));
+      if (l->ff_kind == BCG_FF_CLAMPED_GLU) {
+        BCG_TRY(glu_up(m, ws, l, T, st));
+      } else {
+        BCG_TRY(project(m, ws->xn, l->w_up, ws->proj, ws->proj_floats, T, l->ff, d, &s, st));
+        BCG_TRY(poly_norm(ws->proj, s, static_cast<long long>(T) * l->ff, l->act_coef, ws->act, dt, T, l->ff, m->eps, st));
+      }
       BCG_TRY(project(m, ws->act, l->w_down, ws->proj, ws->proj_floats, T, d, l->ff, &s, st));
       BCG_TRY(sandwich_norm(ws->residual, ws->proj, s, static_cast<long long>(T) * d, l->norm2b, next, ws->xn, dt, T, d,
                             m->eps, {}, st));

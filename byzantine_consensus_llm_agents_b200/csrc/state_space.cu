@@ -1,0 +1,767 @@
+// State-space mixer with one decay per head (state-space duality) over ragged sequences, state in fp32:
+//     S <- exp(-rate * step) S + step * B x^T,      y = S^T C + skip * x,      step = softplus(. + bias),
+// x, B and C behind a causal convolution per channel and silu; then  y * silu(z), an RMS norm in equal parts.
+// A state is stored as [vdim][n] per head, rows of its n entries.
+//
+//   ssm_conv    projection slabs -> convolved x | B | C (activations, heads and groups padded to multiples of 8 columns)
+//               and steps; the inputs ahead of a portion come from the convolution's state
+//   ssm_chunk   portions (bf16): chunks of 64 tokens on tensor cores.  Inside a chunk the recurrence is a product,
+//                   y_i = exp(c_i) S^T C_i + sum_{j <= i} exp(c_i - c_j) step_j (B_j . C_i) x_j,   c = running sum of -rate * step,
+//               and the state moves once per chunk.  Everything is held transposed (rows = entries of a head's output), so
+//               that the state stays in fp32 accumulators and becomes an operand without leaving the registers.  What is
+//               fp32 by nature - the state, decays, steps - enters a product as two bf16 halves (hi + lo).
+//   ssm_scan    portions token by token in fp32: the fp32 engine's kernel
+//   ssm_token   one token per sequence (decode): convolution, recurrence and gate in one kernel; the state is requested
+//               before the dependency wait
+//   ssm_norm    norm of the gated outputs; the convolution's state moves on
+#include "mma_sync.cuh"
+#include "attn_tcgen05.cuh"
+#include "stack_common.cuh"
+#include "kernels.h"
+
+namespace bcg {
+
+constexpr float kSsLog2e = 1.4426950408889634f;
+
+struct SsmArgs {
+  const float* proj;         // rows z | x | B | C | step from column col on, pitch ld
+  int n_partials;
+  long long pstride, ld;
+  int col;
+  const float *conv_w, *conv_b, *step_bias, *rate, *skip, *norm;
+  const int *positions, *slot_map, *row_seq, *seq_start, *state_slots;
+  float *state, *conv_state, *step;
+  void *x, *y;
+  int heads, vdim, n, groups, taps, parts, n_tokens;
+  float eps;
+
+  __host__ __device__ int inner() const { return heads * vdim; }
+  __host__ __device__ int channels() const { return heads * vdim + 2 * groups * n; }
+  __host__ __device__ int x_pad() const { return (vdim + 7) / 8 * 8; }
+  __host__ __device__ int n_pad() const { return (n + 7) / 8 * 8; }
+  __host__ __device__ int x_ld() const { return heads * x_pad() + 2 * groups * n_pad(); }
+  __device__ __forceinline__ int x_col(int c) const {        // place of channel c in x
+    if (c < inner()) return c / vdim * x_pad() + c % vdim;
+    c -= inner();
+    return heads * x_pad() + c / n * n_pad() + c % n;
+  }
+  __device__ __forceinline__ int b_col(int g) const { return heads * x_pad() + g * n_pad(); }
+  __device__ __forceinline__ int c_col(int g) const { return heads * x_pad() + (groups + g) * n_pad(); }
+  __device__ __forceinline__ const float* row(long long t) const { return proj + t * ld + col; }
+  __device__ __forceinline__ int seq_of(int t) const { return row_seq ? row_seq[t] : t; }
+  __device__ __forceinline__ int first_of(int s) const { return seq_start ? seq_start[s] : s; }
+  __device__ __forceinline__ int end_of(int s) const { return seq_start ? seq_start[s + 1] : s + 1; }
+};
+
+__device__ __forceinline__ float silu_f32(float x) { return x * sigmoid_f32(x); }
+__device__ __forceinline__ float softplus_f32(float x) { return fmaxf(x, 0.f) + log1pf(expf(-fabsf(x))); }
+// rounded once near 1: a state that decays slowly would drift with the error of exp
+__device__ __forceinline__ float decay_f32(float x) { return 1.0f + expm1f(x); }
+
+// ------------------------------------------------------------------------------------------- convolution
+constexpr int kConvThreads = 128;
+
+// V channels of the convolution's input at token t - k of the sequence that starts at token t0 of the step.
+template <int V>
+__device__ __forceinline__ Vec<V> conv_input(const SsmArgs& a, int c, int t, int k, int t0, int slot, bool fresh) {
+  if (t - k >= t0) return slab_sum_vec<V>(a.row(t - k) + a.inner() + c, a.n_partials, a.pstride);
+  Vec<V> x;
+#pragma unroll
+  for (int i = 0; i < V; ++i) x.x[i] = 0.f;
+  if (!fresh)
+    x = load_vec<V>(a.conv_state + (static_cast<long long>(slot) * (a.taps - 1) + (a.taps - 1) + (t - t0) - k) * a.channels() + c);
+  return x;
+}
+
+// TAPS: a window of inputs in registers; 0: any number of taps, every input loaded where it is used.
+template <typename T, int V, int TAPS>
+__global__ void __launch_bounds__(kConvThreads)
+ssm_conv_kernel(const SsmArgs a, int run, int conv_blocks) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const int r0 = blockIdx.y * run, r1 = min(a.n_tokens, r0 + run);
+  if (static_cast<int>(blockIdx.x) >= conv_blocks) {
+    const int h = (blockIdx.x - conv_blocks) * kConvThreads + threadIdx.x;
+    if (h >= a.heads) return;
+    for (int t = r0; t < r1; ++t)
+      a.step[static_cast<long long>(t) * a.heads + h] =
+          softplus_f32(slab_sum(a.row(t) + a.inner() + a.channels() + h, a.n_partials, a.pstride) + a.step_bias[h]);
+    return;
+  }
+  const int c = (blockIdx.x * kConvThreads + threadIdx.x) * V, ch = a.channels();
+  if (c >= ch) return;
+  T* out = static_cast<T*>(a.x) + a.x_col(c);
+  const Vec<V> bias = load_vec<V>(a.conv_b + c);
+  constexpr int W = TAPS > 0 ? TAPS : 1;
+  Vec<V> w[W], hist[W];            // hist[k - 1]: input of token t - k
+  if constexpr (TAPS > 0) {
+#pragma unroll
+    for (int k = 0; k < TAPS; ++k) w[k] = load_vec<V>(a.conv_w + static_cast<long long>(k) * ch + c);
+  }
+  int t_end = r0;                  // end of the current sequence
+  int t0 = 0, slot = 0;
+  bool fresh = false;
+  for (int t = r0; t < r1; ++t) {
+    if (t >= t_end) {
+      const int s = a.seq_of(t);
+      t0 = a.first_of(s);
+      t_end = a.end_of(s);
+      slot = a.state_slots[s];
+      fresh = a.positions[t0] == 0;
+      if constexpr (TAPS > 1) {
+#pragma unroll
+        for (int k = 1; k < TAPS; ++k) hist[k - 1] = conv_input<V>(a, c, t, k, t0, slot, fresh);
+      }
+    }
+    Vec<V> x = conv_input<V>(a, c, t, 0, t0, slot, fresh), y = bias;
+    if constexpr (TAPS > 0) {
+#pragma unroll
+      for (int i = 0; i < V; ++i) {
+#pragma unroll
+        for (int k = TAPS - 1; k > 0; --k) y.x[i] = fmaf(w[TAPS - 1 - k].x[i], hist[k - 1].x[i], y.x[i]);
+        y.x[i] = fmaf(w[TAPS - 1].x[i], x.x[i], y.x[i]);
+      }
+#pragma unroll
+      for (int k = TAPS - 1; k > 1; --k) hist[k - 1] = hist[k - 2];
+      if constexpr (TAPS > 1) hist[0] = x;
+    } else {
+      for (int k = a.taps - 1; k >= 0; --k) {
+        const Vec<V> in = k ? conv_input<V>(a, c, t, k, t0, slot, fresh) : x;
+        const Vec<V> wk = load_vec<V>(a.conv_w + static_cast<long long>(a.taps - 1 - k) * ch + c);
+#pragma unroll
+        for (int i = 0; i < V; ++i) y.x[i] = fmaf(wk.x[i], in.x[i], y.x[i]);
+      }
+    }
+#pragma unroll
+    for (int i = 0; i < V; ++i) y.x[i] = silu_f32(y.x[i]);
+    store_vec<V>(out + static_cast<long long>(t) * a.x_ld(), y);
+  }
+}
+
+template <typename T, int V>
+static int launch_conv(const SsmArgs& a, cudaStream_t st) {
+  const int run = a.n_tokens <= 256 ? 1 : a.n_tokens <= 4096 ? 8 : 16;
+  const int blocks = (a.channels() / V + kConvThreads - 1) / kConvThreads;
+  const dim3 grid(blocks + (a.heads + kConvThreads - 1) / kConvThreads, (a.n_tokens + run - 1) / run);
+  switch (a.taps) {
+    case 2: BCG_CUDA_CHECK(launch_k(ssm_conv_kernel<T, V, 2>, grid, dim3(kConvThreads), 0, st, a, run, blocks)); break;
+    case 3: BCG_CUDA_CHECK(launch_k(ssm_conv_kernel<T, V, 3>, grid, dim3(kConvThreads), 0, st, a, run, blocks)); break;
+    case 4: BCG_CUDA_CHECK(launch_k(ssm_conv_kernel<T, V, 4>, grid, dim3(kConvThreads), 0, st, a, run, blocks)); break;
+    default: BCG_CUDA_CHECK(launch_k(ssm_conv_kernel<T, V, 0>, grid, dim3(kConvThreads), 0, st, a, run, blocks));
+  }
+  return BCG_OK;
+}
+
+// ------------------------------------------------------------------------------------------- state in registers
+constexpr int kSsThreads = 256, kSsRows = 64;     // threads and state rows of a CTA
+
+// Rows of a head's state over groups of lanes: a group holds a row's entries, four (or twice four) per lane, and every
+// kPass-th row of the CTA's block.
+template <int NP>
+struct StateRows {
+  static constexpr int kLanes = NP / 4 < 32 ? NP / 4 : 32, kQ = NP / (4 * kLanes), kPass = kSsThreads / kLanes,
+                       kR = kSsRows / kPass;
+  static_assert(kR <= kLanes, "lane r of a group finishes its row r");
+  float s[kR][kQ][4];
+
+  static __device__ __forceinline__ int lane() { return threadIdx.x % kLanes; }
+  static __device__ __forceinline__ int row(int r) { return r * kPass + static_cast<int>(threadIdx.x) / kLanes; }
+  static __device__ __forceinline__ int entry(int q) { return (q * kLanes + lane()) * 4; }
+  __device__ __forceinline__ void zero() {
+#pragma unroll
+    for (int r = 0; r < kR; ++r)
+#pragma unroll
+      for (int q = 0; q < kQ; ++q)
+#pragma unroll
+        for (int i = 0; i < 4; ++i) s[r][q][i] = 0.f;
+  }
+  // st: [rows][n], `rows` of them valid
+  __device__ __forceinline__ void load(const float* st, int rows, int n) {
+#pragma unroll
+    for (int r = 0; r < kR; ++r)
+#pragma unroll
+      for (int q = 0; q < kQ; ++q) {
+        const int e = entry(q);
+        const float* p = st + static_cast<long long>(row(r)) * n + e;
+        if (row(r) < rows && e < n && n % 4 == 0) {
+          const float4 v = *reinterpret_cast<const float4*>(p);
+          s[r][q][0] = v.x; s[r][q][1] = v.y; s[r][q][2] = v.z; s[r][q][3] = v.w;
+        } else {
+#pragma unroll
+          for (int i = 0; i < 4; ++i) s[r][q][i] = row(r) < rows && e + i < n ? p[i] : 0.f;
+        }
+      }
+  }
+  __device__ __forceinline__ void store(float* st, int rows, int n) const {
+#pragma unroll
+    for (int r = 0; r < kR; ++r)
+#pragma unroll
+      for (int q = 0; q < kQ; ++q) {
+        const int e = entry(q);
+        float* p = st + static_cast<long long>(row(r)) * n + e;
+        if (row(r) >= rows) continue;
+        if (e < n && n % 4 == 0) {
+          *reinterpret_cast<float4*>(p) = make_float4(s[r][q][0], s[r][q][1], s[r][q][2], s[r][q][3]);
+        } else {
+#pragma unroll
+          for (int i = 0; i < 4; ++i)
+            if (e + i < n) p[i] = s[r][q][i];
+        }
+      }
+  }
+  // One token: v[r] = step * x of row r, b / c the lane's entries of B and C.  Returns S^T C of row lane(), valid in lanes
+  // below kR.
+  __device__ __forceinline__ float token(float keep, const float (&v)[kR], const float (&b)[kQ][4], const float (&c)[kQ][4]) {
+    float y[kR];
+#pragma unroll
+    for (int r = 0; r < kR; ++r) {
+      y[r] = 0.f;
+#pragma unroll
+      for (int q = 0; q < kQ; ++q)
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+          s[r][q][i] = fmaf(keep, s[r][q][i], v[r] * b[q][i]);
+          y[r] = fmaf(s[r][q][i], c[q][i], y[r]);
+        }
+    }
+#pragma unroll
+    for (int m = kLanes / 2; m > 0; m >>= 1)
+#pragma unroll
+      for (int r = 0; r < kR; ++r) y[r] += __shfl_xor_sync(0xffffffffu, y[r], m);
+    float mine = y[0];
+#pragma unroll
+    for (int r = 1; r < kR; ++r)
+      if (lane() == r) mine = y[r];
+    return mine;
+  }
+};
+
+template <typename T, int NP>
+__global__ void __launch_bounds__(kSsThreads)
+ssm_token_kernel(const SsmArgs a) {
+  using S = StateRows<NP>;
+  __shared__ float xs[kSsRows], zs[kSsRows], bs[NP], cs[NP], step_s;
+  const int h = blockIdx.x, p0 = blockIdx.y * kSsRows, t = blockIdx.z;
+  const int rows = min(kSsRows, a.vdim - p0), N = a.n, g = h / (a.heads / a.groups), inner = a.inner();
+  pdl_launch_dependents();
+  // Positions, slots and states were written by earlier steps, which are complete before any kernel of this step
+  // starts, so the state is on its way while the projections are finished.
+  const bool idle = a.slot_map[t] < 0, fresh = a.positions[t] == 0;
+  const int slot = a.state_slots[t];
+  float* st = a.state + ((static_cast<long long>(slot) * a.heads + h) * a.vdim + p0) * N;
+  S s;
+  if (idle || fresh) s.zero();
+  else s.load(st, rows, N);
+  pdl_wait();
+  if (idle) return;
+  const float* row = a.row(t);
+  // x, B, C through the convolution; z; the step
+  for (int i = threadIdx.x; i < 2 * kSsRows + 2 * NP + 1; i += kSsThreads) {
+    if (i < kSsRows) {
+      if (i < rows) zs[i] = silu_f32(slab_sum(row + h * a.vdim + p0 + i, a.n_partials, a.pstride));
+      continue;
+    }
+    if (i == 2 * kSsRows + 2 * NP) {
+      step_s = softplus_f32(slab_sum(row + inner + a.channels() + h, a.n_partials, a.pstride) + a.step_bias[h]);
+      continue;
+    }
+    const int e = i - kSsRows;
+    const int kind = e < kSsRows ? 0 : e < kSsRows + NP ? 1 : 2, k0 = kind == 0 ? e : kind == 1 ? e - kSsRows : e - kSsRows - NP;
+    float y = 0.f;
+    if (k0 < (kind == 0 ? rows : N)) {
+      const int c = kind == 0 ? h * a.vdim + p0 + k0 : inner + ((kind - 1) * a.groups + g) * N + k0, ch = a.channels();
+      y = fmaf(a.conv_w[static_cast<long long>(a.taps - 1) * ch + c], slab_sum(row + inner + c, a.n_partials, a.pstride), a.conv_b[c]);
+      if (!fresh)
+        for (int k = 0; k < a.taps - 1; ++k)
+          y = fmaf(a.conv_w[static_cast<long long>(k) * ch + c], a.conv_state[(static_cast<long long>(slot) * (a.taps - 1) + k) * ch + c], y);
+      y = silu_f32(y);
+    }
+    (kind == 0 ? xs : kind == 1 ? bs : cs)[k0] = y;
+  }
+  __syncthreads();
+  const float step = step_s, keep = decay_f32(-a.rate[h] * step);
+  float v[S::kR], b[S::kQ][4], c[S::kQ][4];
+#pragma unroll
+  for (int r = 0; r < S::kR; ++r) v[r] = S::row(r) < rows ? step * xs[S::row(r)] : 0.f;
+#pragma unroll
+  for (int q = 0; q < S::kQ; ++q)
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      b[q][i] = bs[S::entry(q) + i];
+      c[q][i] = cs[S::entry(q) + i];
+    }
+  const float y = s.token(keep, v, b, c);
+  s.store(st, rows, N);
+  if (S::lane() < S::kR) {
+    const int p = S::row(S::lane());
+    if (p < rows)
+      static_cast<T*>(a.y)[static_cast<long long>(t) * inner + h * a.vdim + p0 + p] = from_f32<T>(fmaf(a.skip[h], xs[p], y) * zs[p]);
+  }
+}
+
+// Token by token over a portion whose convolution is done.
+template <typename T, int NP>
+__global__ void __launch_bounds__(kSsThreads)
+ssm_scan_kernel(const SsmArgs a) {
+  using S = StateRows<NP>;
+  const int h = blockIdx.x, p0 = blockIdx.y * kSsRows, sq = blockIdx.z;
+  const int rows = min(kSsRows, a.vdim - p0), N = a.n, g = h / (a.heads / a.groups), inner = a.inner();
+  pdl_launch_dependents();
+  pdl_wait();
+  const int t0 = a.first_of(sq), t1 = a.end_of(sq);
+  if (t1 <= t0 || a.slot_map[t0] < 0) return;
+  float* st = a.state + ((static_cast<long long>(a.state_slots[sq]) * a.heads + h) * a.vdim + p0) * N;
+  S s;
+  if (a.positions[t0] == 0) s.zero();
+  else s.load(st, rows, N);
+  const T* base = static_cast<const T*>(a.x);
+  const float rate = a.rate[h], skip = a.skip[h];
+  float x[S::kR], b[S::kQ][4], c[S::kQ][4], step;
+  auto fetch = [&](int t) {
+    const T* tok = base + static_cast<long long>(t) * a.x_ld();
+    step = a.step[static_cast<long long>(t) * a.heads + h];
+#pragma unroll
+    for (int r = 0; r < S::kR; ++r) x[r] = S::row(r) < rows ? to_f32<T>(tok[h * a.x_pad() + p0 + S::row(r)]) : 0.f;
+#pragma unroll
+    for (int q = 0; q < S::kQ; ++q)
+#pragma unroll
+      for (int i = 0; i < 4; ++i) {
+        const int e = S::entry(q) + i;
+        b[q][i] = e < N ? to_f32<T>(tok[a.b_col(g) + e]) : 0.f;
+        c[q][i] = e < N ? to_f32<T>(tok[a.c_col(g) + e]) : 0.f;
+      }
+  };
+  fetch(t0);
+  for (int t = t0; t < t1; ++t) {
+    const float keep = decay_f32(-rate * step);
+    float v[S::kR], bb[S::kQ][4], cc[S::kQ][4], mine = x[0];
+#pragma unroll
+    for (int r = 0; r < S::kR; ++r) {
+      v[r] = step * x[r];
+      if (S::lane() == r) mine = x[r];
+    }
+#pragma unroll
+    for (int q = 0; q < S::kQ; ++q)
+#pragma unroll
+      for (int i = 0; i < 4; ++i) {
+        bb[q][i] = b[q][i];
+        cc[q][i] = c[q][i];
+      }
+    if (t + 1 < t1) fetch(t + 1);
+    const float y = s.token(keep, v, bb, cc);
+    if (S::lane() < S::kR) {
+      const int p = S::row(S::lane());
+      if (p < rows) {
+        const float z = slab_sum(a.row(t) + h * a.vdim + p0 + p, a.n_partials, a.pstride);
+        static_cast<T*>(a.y)[static_cast<long long>(t) * inner + h * a.vdim + p0 + p] = from_f32<T>(fmaf(skip, mine, y) * silu_f32(z));
+      }
+    }
+  }
+  s.store(st, rows, N);
+}
+
+// ------------------------------------------------------------------------------------------- chunks
+constexpr int kChTok = 64, kChWarps = 4, kChThreads = kChWarps * 32;
+
+template <int NP>
+struct ChCfg {
+  static constexpr int kBRow = NP + 8, kXRow = kSsRows + 8, kMRow = kChTok + 8;       // pitches, bf16
+  static constexpr int kBC = kChTok * kBRow, kX = kChTok * kXRow, kM = kChTok * kMRow;
+  static constexpr int kBuf = 2 * kBC + kX;                                             // B, C, x of a chunk
+  static constexpr int kSmem = (2 * kBuf + 2 * kM) * 2 + 2 * 4 * kChTok * 4;            // two chunks, M hi / lo, scalars
+};
+
+// hi + lo = v to about 2^-17
+__device__ __forceinline__ void split_bf16(float a, float b, uint32_t& hi, uint32_t& lo) {
+  hi = pack_bf16(a, b);
+  lo = pack_bf16(a - bf16lo(hi), b - bf16hi(hi));
+}
+__device__ __forceinline__ uint32_t transpose_8x8(uint32_t v) {
+  uint32_t r;
+  asm volatile("movmatrix.sync.aligned.m8n8.trans.b16 %0, %1;" : "=r"(r) : "r"(v));
+  return r;
+}
+
+// grid (heads, blocks of 64 head entries, sequences); warp w has entries 16 w .. 16 w + 15 of the block.
+template <int NP>
+__global__ void __launch_bounds__(kChThreads, NP <= 128 ? 2 : 1)
+ssm_chunk_kernel(const SsmArgs a) {
+  using C = ChCfg<NP>;
+  extern __shared__ __align__(16) uint8_t ch_raw[];
+  __nv_bfloat16* bufs = reinterpret_cast<__nv_bfloat16*>(ch_raw);
+  __nv_bfloat16* m_hi = bufs + 2 * C::kBuf;
+  __nv_bfloat16* m_lo = m_hi + C::kM;
+  float* scalars = reinterpret_cast<float*>(m_lo + C::kM);     // [2][4][64]: log2 decay sums, steps, e, w
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, n_warps = blockDim.x >> 5;
+  const int h = blockIdx.x, p0 = blockIdx.y * kSsRows, sq = blockIdx.z;
+  const int rows = min(kSsRows, a.vdim - p0), N = a.n, g = h / (a.heads / a.groups), inner = a.inner();
+  pdl_launch_dependents();
+  pdl_wait();
+  const int t0 = a.first_of(sq), t1 = a.end_of(sq);
+  if (t1 <= t0 || a.slot_map[t0] < 0) return;
+  const float rate = a.rate[h], skip = a.skip[h];
+  const __nv_bfloat16* xbc = static_cast<const __nv_bfloat16*>(a.x);
+  const int x_ld = a.x_ld(), xc = h * a.x_pad() + p0, bc = a.b_col(g), cc = a.c_col(g);
+
+  // B, C and x of a chunk; columns and tokens past the end are zero
+  auto copy_rows = [&](__nv_bfloat16* dst, int pitch, int col, int valid, int units, int first) {
+    for (int i = threadIdx.x; i < kChTok * units; i += blockDim.x) {
+      const int r = i / units, u = i - r * units;
+      const int bytes = first + r < t1 ? max(0, min(16, (valid - u * 8) * 2)) : 0;
+      const __nv_bfloat16* src = bytes ? xbc + static_cast<long long>(first + r) * x_ld + col + u * 8 : xbc;
+      asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(smem_u32(dst + r * pitch + u * 8)), "l"(src), "r"(bytes)
+                   : "memory");
+    }
+  };
+  auto fetch = [&](int c) {
+    __nv_bfloat16* b = bufs + (c & 1) * C::kBuf;
+    copy_rows(b, C::kBRow, bc, N, NP / 8, t0 + c * kChTok);
+    copy_rows(b + C::kBC, C::kBRow, cc, N, NP / 8, t0 + c * kChTok);
+    copy_rows(b + 2 * C::kBC, C::kXRow, xc, rows, kSsRows / 8, t0 + c * kChTok);
+    cp_async_commit();
+  };
+  auto step_at = [&](int t) { return t < t1 ? a.step[static_cast<long long>(t) * a.heads + h] : 0.f; };
+
+  const int n_chunks = (t1 - t0 + kChTok - 1) / kChTok;
+  const int pr = warp * 16 + (lane >> 2);       // this lane's rows of the state: pr, pr + 8; entries nt * 8 + 2 (lane & 3) ..
+  const int q2 = (lane & 3) * 2;
+  float* st = a.state + ((static_cast<long long>(a.state_slots[sq]) * a.heads + h) * a.vdim + p0) * N;
+  float S[NP / 8][4];
+  const bool fresh = a.positions[t0] == 0;
+#pragma unroll
+  for (int nt = 0; nt < NP / 8; ++nt)
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      const int p = pr + (i >> 1) * 8, n = nt * 8 + q2 + (i & 1);
+      S[nt][i] = !fresh && p < rows && n < N ? st[static_cast<long long>(p) * N + n] : 0.f;
+    }
+  fetch(0);
+  float s0 = 0.f, s1 = 0.f;                     // warp 0: steps of tokens 2 lane, 2 lane + 1 of the next chunk
+  if (warp == 0) {
+    s0 = step_at(t0 + 2 * lane);
+    s1 = step_at(t0 + 2 * lane + 1);
+  }
+
+  for (int c = 0; c < n_chunks; ++c) {
+    const int first = t0 + c * kChTok, nt_tok = min(kChTok, t1 - first);
+    const __nv_bfloat16* sB = bufs + (c & 1) * C::kBuf;
+    const __nv_bfloat16* sC = sB + C::kBC;
+    const __nv_bfloat16* sX = sC + C::kBC;
+    float* sum2 = scalars + (c & 1) * 4 * kChTok;
+    float *steps = sum2 + kChTok, *e_s = steps + kChTok, *w_s = e_s + kChTok;
+    if (warp == 0) {
+      const float a0 = -rate * s0, a1 = -rate * s1;
+      float run = a0 + a1;
+#pragma unroll
+      for (int o = 1; o < 32; o <<= 1) {
+        const float v = __shfl_up_sync(0xffffffffu, run, o);
+        if (lane >= o) run += v;
+      }
+      const float total = __shfl_sync(0xffffffffu, run, 31);
+      const float c1 = run, c0 = run - a1;
+      sum2[2 * lane] = c0 * kSsLog2e;
+      sum2[2 * lane + 1] = c1 * kSsLog2e;
+      steps[2 * lane] = s0;
+      steps[2 * lane + 1] = s1;
+      e_s[2 * lane] = expf(c0);
+      e_s[2 * lane + 1] = expf(c1);
+      w_s[2 * lane] = s0 * expf(total - c0);
+      w_s[2 * lane + 1] = s1 * expf(total - c1);
+      s0 = step_at(first + kChTok + 2 * lane);
+      s1 = step_at(first + kChTok + 2 * lane + 1);
+    }
+    cp_async_wait<0>();
+    __syncthreads();                            // the chunk is there; everybody is done with the previous one
+    if (c + 1 < n_chunks) fetch(c + 1);
+
+    // ---- M[i][j] = exp(c_i - c_j) step_j (C_i . B_j) for j <= i, 16 tokens i per turn
+    for (int rt = warp; rt * 16 < nt_tok; rt += n_warps) {
+      float acc[kChTok / 8][4] = {};
+#pragma unroll
+      for (int k = 0; k < NP / 16; ++k) {
+        uint32_t ca[4];
+        ldsm_x4(ca, sC + (rt * 16 + (lane & 15)) * C::kBRow + k * 16 + (lane >> 4) * 8);
+#pragma unroll
+        for (int jp = 0; jp < kChTok / 16; ++jp)
+          if (jp <= rt) {
+            uint32_t bb[4];
+            ldsm_x4(bb, sB + (jp * 16 + (lane & 7) + ((lane >> 4) << 3)) * C::kBRow + k * 16 + ((lane >> 3) & 1) * 8);
+            mma_bf16_16816(acc[2 * jp], ca, bb[0], bb[1]);
+            mma_bf16_16816(acc[2 * jp + 1], ca, bb[2], bb[3]);
+          }
+      }
+      const int i0 = rt * 16 + (lane >> 2);
+      const float ci[2] = {sum2[i0], sum2[i0 + 8]};
+#pragma unroll
+      for (int jt = 0; jt < kChTok / 8; ++jt)
+        if (jt <= 2 * rt + 1) {
+          const int j = jt * 8 + q2;
+          const float2 cj = *reinterpret_cast<const float2*>(sum2 + j), sj = *reinterpret_cast<const float2*>(steps + j);
+#pragma unroll
+          for (int e = 0; e < 2; ++e) {
+            const int i = i0 + e * 8;
+            const float m0 = j <= i ? acc[jt][2 * e] * (ex2_approx(ci[e] - cj.x) * sj.x) : 0.f;
+            const float m1 = j + 1 <= i ? acc[jt][2 * e + 1] * (ex2_approx(ci[e] - cj.y) * sj.y) : 0.f;
+            uint32_t hi, lo;
+            split_bf16(m0, m1, hi, lo);
+            *reinterpret_cast<uint32_t*>(m_hi + i * C::kMRow + j) = hi;
+            *reinterpret_cast<uint32_t*>(m_lo + i * C::kMRow + j) = lo;
+          }
+        }
+    }
+
+    // ---- Y^T = S^T C^T, columns (tokens) scaled by exp(c_i)
+    float Y[kChTok / 8][4] = {};
+#pragma unroll
+    for (int k = 0; k < NP / 16; ++k) {
+      uint32_t hi[4], lo[4];
+      split_bf16(S[2 * k][0], S[2 * k][1], hi[0], lo[0]);
+      split_bf16(S[2 * k][2], S[2 * k][3], hi[1], lo[1]);
+      split_bf16(S[2 * k + 1][0], S[2 * k + 1][1], hi[2], lo[2]);
+      split_bf16(S[2 * k + 1][2], S[2 * k + 1][3], hi[3], lo[3]);
+#pragma unroll
+      for (int ip = 0; ip < kChTok / 16; ++ip) {
+        uint32_t cb[4];
+        ldsm_x4(cb, sC + (ip * 16 + (lane & 7) + ((lane >> 4) << 3)) * C::kBRow + k * 16 + ((lane >> 3) & 1) * 8);
+        mma_bf16_16816(Y[2 * ip], hi, cb[0], cb[1]);
+        mma_bf16_16816(Y[2 * ip + 1], hi, cb[2], cb[3]);
+        mma_bf16_16816(Y[2 * ip], lo, cb[0], cb[1]);
+        mma_bf16_16816(Y[2 * ip + 1], lo, cb[2], cb[3]);
+      }
+    }
+#pragma unroll
+    for (int it = 0; it < kChTok / 8; ++it) {
+      const float2 e = *reinterpret_cast<const float2*>(e_s + it * 8 + q2);
+      Y[it][0] *= e.x;
+      Y[it][1] *= e.y;
+      Y[it][2] *= e.x;
+      Y[it][3] *= e.y;
+    }
+    const float keep = e_s[kChTok - 1];         // past the end steps are zero: the whole chunk's decay
+#pragma unroll
+    for (int nt = 0; nt < NP / 8; ++nt)
+#pragma unroll
+      for (int i = 0; i < 4; ++i) S[nt][i] *= keep;
+    __syncthreads();                            // M is complete
+
+    // ---- Y^T += x^T M^T + skip x^T;   S^T += (w x)^T B
+#pragma unroll
+    for (int jp = 0; jp < kChTok / 16; ++jp) {
+      uint32_t xa[4];
+      ldsm_x4_trans(xa, sX + (jp * 16 + (lane & 7) + ((lane >> 4) << 3)) * C::kXRow + warp * 16 + ((lane >> 3) & 1) * 8);
+#pragma unroll
+      for (int ip = jp; ip < kChTok / 16; ++ip)
+        if (ip * 16 < nt_tok) {
+          uint32_t mb[4];
+          const int at = (ip * 16 + (lane & 7) + ((lane >> 4) << 3)) * C::kMRow + jp * 16 + ((lane >> 3) & 1) * 8;
+          ldsm_x4(mb, m_hi + at);
+          mma_bf16_16816(Y[2 * ip], xa, mb[0], mb[1]);
+          mma_bf16_16816(Y[2 * ip + 1], xa, mb[2], mb[3]);
+          ldsm_x4(mb, m_lo + at);
+          mma_bf16_16816(Y[2 * ip], xa, mb[0], mb[1]);
+          mma_bf16_16816(Y[2 * ip + 1], xa, mb[2], mb[3]);
+        }
+      float xf[4][2];                           // rows pr, pr + 8 of tokens j, j + 1; the same of tokens j + 8, j + 9
+#pragma unroll
+      for (int i = 0; i < 4; ++i) {
+        xf[i][0] = bf16lo(xa[i]);
+        xf[i][1] = bf16hi(xa[i]);
+      }
+#pragma unroll
+      for (int e = 0; e < 2; ++e)
+#pragma unroll
+        for (int k = 0; k < 2; ++k) {
+          Y[2 * jp + e][k] = fmaf(skip, xf[2 * e][k], Y[2 * jp + e][k]);
+          Y[2 * jp + e][2 + k] = fmaf(skip, xf[2 * e + 1][k], Y[2 * jp + e][2 + k]);
+        }
+      const float2 w0 = *reinterpret_cast<const float2*>(w_s + jp * 16 + q2), w1 = *reinterpret_cast<const float2*>(w_s + jp * 16 + 8 + q2);
+      uint32_t hi[4], lo[4];
+      split_bf16(w0.x * xf[0][0], w0.y * xf[0][1], hi[0], lo[0]);
+      split_bf16(w0.x * xf[1][0], w0.y * xf[1][1], hi[1], lo[1]);
+      split_bf16(w1.x * xf[2][0], w1.y * xf[2][1], hi[2], lo[2]);
+      split_bf16(w1.x * xf[3][0], w1.y * xf[3][1], hi[3], lo[3]);
+#pragma unroll
+      for (int np = 0; np < NP / 16; ++np) {
+        uint32_t bb[4];
+        ldsm_x4_trans(bb, sB + (jp * 16 + (lane & 15)) * C::kBRow + np * 16 + (lane >> 4) * 8);
+        mma_bf16_16816(S[2 * np], hi, bb[0], bb[1]);
+        mma_bf16_16816(S[2 * np + 1], hi, bb[2], bb[3]);
+        mma_bf16_16816(S[2 * np], lo, bb[0], bb[1]);
+        mma_bf16_16816(S[2 * np + 1], lo, bb[2], bb[3]);
+      }
+    }
+
+    // ---- gate and store: z is read where the outputs are, pairs are transposed on the way out
+    __nv_bfloat16* out = static_cast<__nv_bfloat16*>(a.y) + static_cast<long long>(first) * inner + h * a.vdim + p0;
+#pragma unroll
+    for (int it = 0; it < kChTok / 8; ++it) {
+      if (it * 8 >= nt_tok) break;
+      float u[4];
+#pragma unroll
+      for (int i = 0; i < 4; ++i) {
+        const int tok = it * 8 + q2 + (i & 1), p = pr + (i >> 1) * 8;
+        float z = 0.f;
+        if (tok < nt_tok && p < rows) z = slab_sum(a.row(first + tok) + h * a.vdim + p0 + p, a.n_partials, a.pstride);
+        u[i] = Y[it][i] * silu_f32(z);
+      }
+#pragma unroll
+      for (int e = 0; e < 2; ++e) {
+        const uint32_t v = transpose_8x8(pack_bf16(u[2 * e], u[2 * e + 1]));     // token lane >> 2, entries q2, q2 + 1
+        const int tok = it * 8 + (lane >> 2), p = warp * 16 + e * 8 + q2;
+        __nv_bfloat16* dst = out + static_cast<long long>(tok) * inner + p;
+        if (tok < nt_tok && p + 1 < rows && (a.vdim & 1) == 0) {
+          *reinterpret_cast<uint32_t*>(dst) = v;
+        } else if (tok < nt_tok) {
+          if (p < rows) dst[0] = __ushort_as_bfloat16(static_cast<unsigned short>(v & 0xffffu));
+          if (p + 1 < rows) dst[1] = __ushort_as_bfloat16(static_cast<unsigned short>(v >> 16));
+        }
+        __syncwarp();
+      }
+    }
+  }
+#pragma unroll
+  for (int nt = 0; nt < NP / 8; ++nt)
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      const int p = pr + (i >> 1) * 8, n = nt * 8 + q2 + (i & 1);
+      if (p < rows && n < N) st[static_cast<long long>(p) * N + n] = S[nt][i];
+    }
+}
+
+// ------------------------------------------------------------------------------------------- norm
+constexpr int kSnThreads = 256;
+
+// A part of a token's outputs per CTA, or per cluster of CL.  The CTAs of a sequence's last token also move the
+// convolution's state on.
+template <typename T, int V, int CL>
+__global__ void __launch_bounds__(kSnThreads)
+ssm_norm_kernel(const SsmArgs a, T* __restrict__ out, long long out_ld) {
+  __shared__ RowSum<kSnThreads, CL, 1> sh;
+  pdl_launch_dependents();
+  pdl_wait();
+  const int unit = blockIdx.x % (a.parts * CL), t = blockIdx.x / (a.parts * CL);
+  const int part = unit / CL, inner = a.inner(), width = inner / a.parts;
+  const int per = (width / V + CL - 1) / CL * V, v0 = unit % CL * per, v1 = min(width, v0 + per);
+  const T* y = static_cast<const T*>(a.y) + static_cast<long long>(t) * inner + part * width;
+  float ss[1] = {0.f};
+  for (int v = v0 + threadIdx.x * V; v < v1; v += kSnThreads * V) ss[0] += load_vec<V>(y + v).sumsq();
+  row_sum<kSnThreads, CL, 1>(sh, ss, 0);
+  const float inv = rsqrtf(ss[0] / static_cast<float>(width) + a.eps);
+  for (int v = v0 + threadIdx.x * V; v < v1; v += kSnThreads * V) {
+    Vec<V> x = load_vec<V>(y + v);
+    const Vec<V> w = load_vec<V>(a.norm + part * width + v);
+#pragma unroll
+    for (int k = 0; k < V; ++k) x.x[k] *= inv * w.x[k];
+    store_vec<V>(out + t * out_ld + part * width + v, x);
+  }
+  const int s = a.seq_of(t), t0 = a.first_of(s), keep = a.taps - 1, ch = a.channels();
+  if (t == a.end_of(s) - 1 && keep > 0 && a.slot_map[t] >= 0) {
+    const bool fresh = a.positions[t0] == 0;
+    const int n = t + 1 - t0;
+    float* cs = a.conv_state + static_cast<long long>(a.state_slots[s]) * keep * ch;
+    for (int c = unit * kSnThreads + threadIdx.x; c < ch; c += a.parts * CL * kSnThreads)
+      for (int r = 0; r < keep; ++r) {          // row r <- input n + r - keep of this portion, or old row n + r
+        const int i = n + r - keep;
+        float x = 0.f;
+        if (i >= 0) x = slab_sum(a.row(t0 + i) + inner + c, a.n_partials, a.pstride);
+        else if (!fresh) x = cs[static_cast<long long>(n + r) * ch + c];
+        cs[static_cast<long long>(r) * ch + c] = x;
+      }
+  }
+  row_sum_exit<CL>();
+}
+
+template <typename T, int V>
+static int launch_norm(const SsmArgs& a, void* out, long long out_ld, cudaStream_t st) {
+  const long long units = static_cast<long long>(a.n_tokens) * a.parts;
+  if (a.n_tokens <= 128 && a.inner() / a.parts >= 1024)
+    BCG_CUDA_CHECK(launch_cluster(ssm_norm_kernel<T, V, 8>, dim3(static_cast<unsigned>(units * 8)), dim3(kSnThreads), 8, 0, st, a,
+                                  static_cast<T*>(out), out_ld));
+  else
+    BCG_CUDA_CHECK(launch_k(ssm_norm_kernel<T, V, 1>, dim3(static_cast<unsigned>(units)), dim3(kSnThreads), 0, st, a,
+                            static_cast<T*>(out), out_ld));
+  return BCG_OK;
+}
+
+// ------------------------------------------------------------------------------------------- launches
+template <typename T, int NP>
+static int run_np(const SsmArgs& a, int n_seqs, bool one_token, bool chunks, cudaStream_t st) {
+  const int blocks = (a.vdim + kSsRows - 1) / kSsRows;
+  const dim3 grid(a.heads, blocks, n_seqs);
+  if (one_token) {
+    BCG_CUDA_CHECK(launch_k(ssm_token_kernel<T, NP>, grid, dim3(kSsThreads), 0, st, a));
+  } else if (chunks) {
+    BCG_TRY(ensure_dynamic_smem(reinterpret_cast<const void*>(ssm_chunk_kernel<NP>), ChCfg<NP>::kSmem));
+    const int warps = (min(a.vdim, kSsRows) + 15) / 16;
+    BCG_CUDA_CHECK(launch_k(ssm_chunk_kernel<NP>, grid, dim3(warps * 32), ChCfg<NP>::kSmem, st, a));
+  } else {
+    BCG_CUDA_CHECK(launch_k(ssm_scan_kernel<T, NP>, grid, dim3(kSsThreads), 0, st, a));
+  }
+  return BCG_OK;
+}
+
+template <typename T>
+static int run_t(const SsmArgs& a, int n_seqs, bool one_token, int mode, void* out, long long out_ld, cudaStream_t st) {
+  const bool bf16 = sizeof(T) == 2;
+  const bool wide = ((a.vdim | a.n | a.col) & 3) == 0 && a.ld % 4 == 0 && a.pstride % 4 == 0;
+  const bool token = one_token && mode == 0, chunks = bf16 && mode == 0;
+  if (!token) {
+    if (wide) BCG_TRY((launch_conv<T, 4>(a, st)));
+    else BCG_TRY((launch_conv<T, 1>(a, st)));
+  }
+  if (a.n <= 32) BCG_TRY((run_np<T, 32>(a, n_seqs, token, chunks, st)));
+  else if (a.n <= 64) BCG_TRY((run_np<T, 64>(a, n_seqs, token, chunks, st)));
+  else if (a.n <= 128) BCG_TRY((run_np<T, 128>(a, n_seqs, token, chunks, st)));
+  else BCG_TRY((run_np<T, 256>(a, n_seqs, token, chunks, st)));
+  const int width = a.inner() / a.parts;
+  if (width % 4 == 0 && out_ld % 4 == 0 && reinterpret_cast<uintptr_t>(out) % 16 == 0) return launch_norm<T, 4>(a, out, out_ld, st);
+  return launch_norm<T, 1>(a, out, out_ld, st);
+}
+
+int state_space(const bcg_stack* m, const bcg_layer* l, const bcg_stack_ws* ws, const bcg_step_batch* b, int n_partials,
+                long long pstride, long long ld, int mode, cudaStream_t st) {
+  if (!l->conv_w || !l->conv_b || !l->step_bias || !l->decay_rate || !l->skip || !l->ssm_norm || !l->ssm_state ||
+      (l->ssm_taps > 1 && !l->conv_state) || !ws->ssm_x || !ws->ssm_step || !ws->ssm_y || !b->state_slots || l->ssm_n <= 0 ||
+      l->ssm_n > 256 || l->ssm_vdim <= 0 || l->ssm_taps < 1 || l->ssm_groups <= 0 || l->ssm_heads % l->ssm_groups ||
+      l->ssm_norm_parts <= 0 || (l->ssm_heads * l->ssm_vdim) % l->ssm_norm_parts || b->n_seqs > 65535) {
+    set_last_error("bcg_state_space", "bad layer (1..256 state entries, groups and parts that divide) or too many sequences");
+    return BCG_ERR_ARG;
+  }
+  SsmArgs a = {};
+  a.proj = ws->proj;
+  a.n_partials = n_partials;
+  a.pstride = pstride;
+  a.ld = ld;
+  a.col = l->ssm_col;
+  a.conv_w = l->conv_w;
+  a.conv_b = l->conv_b;
+  a.step_bias = l->step_bias;
+  a.rate = l->decay_rate;
+  a.skip = l->skip;
+  a.norm = l->ssm_norm;
+  a.positions = b->positions;
+  a.slot_map = b->slot_map;
+  a.row_seq = b->row_seq;
+  a.seq_start = b->seq_start;
+  a.state_slots = b->state_slots;
+  a.state = l->ssm_state;
+  a.conv_state = l->conv_state;
+  a.step = ws->ssm_step;
+  a.x = ws->ssm_x;
+  a.y = ws->ssm_y;
+  a.heads = l->ssm_heads;
+  a.vdim = l->ssm_vdim;
+  a.n = l->ssm_n;
+  a.groups = l->ssm_groups;
+  a.taps = l->ssm_taps;
+  a.parts = l->ssm_norm_parts;
+  a.n_tokens = b->T;
+  a.eps = m->eps;
+  const bool one = b->T == b->n_seqs;
+  const int size = m->act_dtype == BCG_DT_F32 ? 4 : 2;
+  void* out = static_cast<char*>(ws->mix) + static_cast<long long>(l->ssm_mix_col) * size;
+  return size == 4 ? run_t<float>(a, b->n_seqs, one, mode, out, l->mix_ld, st)
+                   : run_t<__nv_bfloat16>(a, b->n_seqs, one, mode, out, l->mix_ld, st);
+}
+
+}  // namespace bcg

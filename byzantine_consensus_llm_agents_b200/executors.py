@@ -24,7 +24,7 @@ import torch
 
 from . import lib as L
 from .model import ModelHandle
-from .stack import GeneralDelta, GroupedAttention, LatentAttention, MoeMlp, StackHandle
+from .stack import GeneralDelta, GroupedAttention, LatentAttention, MoeMlp, StackHandle, StateSpace
 
 PAGE = 16
 SPLIT_TOKENS = 256
@@ -191,9 +191,7 @@ class StackExecutor:
         self.B_max = max(max_rows, logit_rows)
         act, f32, bf = cfg.torch_dtype, torch.float32, torch.bfloat16
         T, D, d = T_max, max_rows, cfg.d_model
-        attn = [l.mixer for l in cfg.layers if isinstance(l.mixer, LatentAttention)]
-        grouped = [l.mixer for l in cfg.layers if isinstance(l.mixer, GroupedAttention)]
-        delta = [l.mixer for l in cfg.layers if isinstance(l.mixer, GeneralDelta)]
+        attn, grouped, delta, ssm = (cfg.mixers(k) for k in (LatentAttention, GroupedAttention, GeneralDelta, StateSpace))
         mlps = [l.mlp for l in cfg.layers if l.mlp and not l.parallel]
         moes = [l.mlp for l in cfg.layers if isinstance(l.mlp, MoeMlp)]
         top = lambda xs: max([8, *xs])
@@ -203,7 +201,7 @@ class StackExecutor:
         wide = act == bf
         shapes = [(cfg.in_rows(i), d) for i in range(cfg.n_layers)]
         for i, l in enumerate(cfg.layers):
-            shapes += [(d, cfg.mix_cols(i)[1])] + ([(l.mlp.ff, d), (d, l.mlp.ff)] if l.mlp in mlps else [])
+            shapes += [(d, cfg.mix_cols(i)[1])] + ([(l.mlp.up_rows, d), (d, l.mlp.ff_ld)] if l.mlp in mlps else [])
         slabs = lambda n, k: min(T, 128) * n * (L.splits_for(1, n, k) if wide else 1)
         proj = max([T * n for n, _ in shapes] + [slabs(n, k) for n, k in shapes])
         dec = max([8] + [max(T * m.out_dim, slabs(m.out_dim, m.rank_ld)) for m in delta])
@@ -227,7 +225,9 @@ class StackExecutor:
             moe_rank=z(T * choices + 8, torch.int32), moe_weight=z(T * choices + 8, f32),
             moe_row=z(T * choices + 8, torch.int32), moe_row_weight=z(T * choices + 8, f32),
             moe_counts=z(counts + 8, torch.int32),
-            act=z(T * top(m.ff for m in mlps), act), low=z(T * top(m.rank_ld for m in delta), act),
+            act=z(T * top(m.ff_ld for m in mlps), act), gates=z(T * top(m.heads for m in grouped if m.gate), f32),
+            ssm_x=z(T * top(m.x_ld for m in ssm) if ssm else 8, act), ssm_step=z(T * top(m.heads for m in ssm) if ssm else 8, f32),
+            ssm_y=z(T * top(m.out_dim for m in ssm) if ssm else 8, act), low=z(T * top(m.rank_ld for m in delta), act),
             latents=z(max(8, self.K_max * top(m.cache_row for m in expanded)), bf),
             expanded=z(max(8, self.K_max * top(m.heads * (m.q_ld + m.v_ld) for m in expanded)), bf),
             q_latent=z(D * top(m.heads * m.cache_row for m in attn) if wide else 8, bf),
@@ -250,12 +250,17 @@ class StackExecutor:
     def alloc_cache(self, pages: int, slots: int):
         self.caches = []
         for l in self.cfg.layers:
-            m = l.mixer
-            if isinstance(m, GeneralDelta):
+            m, att, ssm = l.mixer, l.one(GroupedAttention), l.one(StateSpace)
+            z = lambda *s, dt=torch.float32: torch.zeros(*s, dtype=dt, device=self.dev)
+            if att or ssm:
+                t = {}
+                if att:
+                    t.update({n: z(pages, att.kv_heads, PAGE, ld, dt=self.cfg.torch_dtype)
+                              for n, ld in (("cache", att.q_ld), ("cache_v", att.v_ld))})
+                if ssm:
+                    t.update(ssm_state=z(slots, ssm.heads, ssm.vdim, ssm.state), conv_state=z(slots, ssm.conv - 1, ssm.channels))
+            elif isinstance(m, GeneralDelta):
                 t = torch.zeros(slots, m.heads, m.dim, m.dim, dtype=torch.float32, device=self.dev)
-            elif isinstance(m, GroupedAttention):
-                t = tuple(torch.zeros(pages, m.kv_heads, PAGE, n, dtype=self.cfg.torch_dtype, device=self.dev)
-                          for n in (m.q_ld, m.v_ld))
             else:
                 t = torch.zeros(pages, PAGE, m.cache_row, dtype=self.cfg.torch_dtype, device=self.dev) \
                     if m.kv_from is None else None
@@ -335,6 +340,10 @@ class StackExecutor:
         for l in self.cfg.layers:
             if l.parallel:   # input projection, its split, attention, output projection, norm; scatter, two products, gate
                 n += 5 + (4 if isinstance(l.mlp, MoeMlp) else 0)
+                continue
+            if l.composed:   # input projection, attention's split and kernel, the state-space mixer's two (portions: three)
+                # kernels, output projection, norm; feed-forward: up with its unit (in its epilogue or not), down, norm
+                n += 3 + (2 if l.one(GroupedAttention) else 0) + (2 if l.one(StateSpace) else 0) + (3 if l.mlp else 0)
                 continue
             # input projection, mixer (delta: low rank, decay projection, scan; attention: qkv, absorb, decode,
             # combine, up), output projection, norm; feed-forward: up, activation, down, norm

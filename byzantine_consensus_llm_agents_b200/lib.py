@@ -19,7 +19,8 @@ STEP_FUSED_ROPE = 0x80000     # bcg_model_decode: qk-norm/RoPE/KV-write folded i
 STEP_DEFERRED_NORM = 0x40000  # bcg_model_decode: norm statistics kernel + 1/RMS in the next GEMM's epilogue
 
 DT_BF16, DT_F32 = 0, 1                          # activation dtype of a layer stack
-MIXER_LATENT_ATTN, MIXER_GENERAL_DELTA, MIXER_GROUPED_ATTN = 1, 2, 3
+MIXER_LATENT_ATTN, MIXER_GENERAL_DELTA, MIXER_GROUPED_ATTN, MIXER_STATE_SPACE = 1, 2, 3, 4
+FF_POLY_NORM, FF_CLAMPED_GLU = 0, 1             # Layer.ff_kind
 MAX_GROUPS = 512                                # experts the grouped tensor-core GEMM takes
 VALUES_FIRST, VALUES_MIX = 1, 2                 # Layer.v_role
 
@@ -96,6 +97,11 @@ class Layer(C.Structure):
         ("router_col", C.c_int), ("experts", C.c_int), ("top", C.c_int), ("expert_ld", C.c_int),
         ("glu_limit", C.c_float), ("glu_alpha", C.c_float), ("moe_counts_at", C.c_int), ("slopes", vp),
         ("in_bias", vp), ("out_bias", vp), ("w_experts_in", vp), ("w_experts_out", vp), ("cache_v", vp),
+        ("q_norm", vp), ("k_norm", vp), ("gated", C.c_int), ("gate_col", C.c_int), ("gate_scale", C.c_float),
+        ("ff_kind", C.c_int), ("ssm_heads", C.c_int), ("ssm_vdim", C.c_int), ("ssm_n", C.c_int), ("ssm_groups", C.c_int),
+        ("ssm_norm_parts", C.c_int), ("ssm_taps", C.c_int), ("ssm_col", C.c_int), ("ssm_mix_col", C.c_int),
+        ("conv_w", vp), ("conv_b", vp), ("step_bias", vp), ("decay_rate", vp), ("skip", vp), ("ssm_norm", vp),
+        ("ssm_state", vp), ("conv_state", vp),
     ]
 
 
@@ -104,6 +110,7 @@ class Stack(C.Structure):
         ("n_layers", C.c_int), ("d_model", C.c_int), ("vocab_ld", C.c_int), ("act_dtype", C.c_int),
         ("page_size", C.c_int), ("eps", C.c_float), ("embed", vp), ("lm_head", vp), ("final_norm", vp),
         ("layers", C.POINTER(Layer)), ("pos_embed", vp), ("n_pos", C.c_int),
+        ("embed_scale", C.c_float), ("pos_turns", vp),
     ]
 
 
@@ -116,7 +123,7 @@ class StackWs(C.Structure):
         ("D_max", C.c_int), ("B_max", C.c_int), ("v_first", vp), ("moe_x", vp), ("moe_h", vp), ("moe_proj", vp),
         ("moe_proj_floats", C.c_longlong), ("moe_out", vp), ("moe_out_floats", C.c_longlong), ("moe_expert", vp),
         ("moe_rank", vp), ("moe_weight", vp), ("moe_row", vp), ("moe_row_weight", vp), ("moe_counts", vp),
-        ("moe_counts_n", C.c_int), ("moe_rows_max", C.c_int),
+        ("moe_counts_n", C.c_int), ("moe_rows_max", C.c_int), ("gates", vp), ("ssm_x", vp), ("ssm_step", vp), ("ssm_y", vp),
     ]
 
 
@@ -188,6 +195,10 @@ _SIGS = {
                                         vp]),
     "bcg_gemm_grouped": (C.c_int, [vp, vp, vp, C.c_int, C.c_int, C.c_int, vp, C.c_int, C.c_int, C.c_int, vp, C.c_float,
                                    C.c_float, C.c_int, vp]),
+    "bcg_state_space": (C.c_int, [C.POINTER(Stack), C.POINTER(StackWs), C.POINTER(StepBatch), C.c_int, C.c_int,
+                                  C.c_longlong, C.c_longlong, C.c_int, vp]),
+    "bcg_clamped_glu": (C.c_int, [vp, C.c_int, C.c_longlong, vp, C.c_int, C.c_int, C.c_int, C.c_float, C.c_float, vp]),
+    "bcg_gemm_bf16_glu": (C.c_int, [vp, vp, vp, C.c_int, C.c_int, C.c_int, C.c_float, C.c_float, C.c_int, vp]),
     "bcg_experts": (C.c_int, [C.POINTER(Stack), C.POINTER(StackWs), C.c_int, C.c_int, c_int_p, vp]),
 }
 

@@ -1,8 +1,8 @@
 """Layer stacks: models whose layers differ in kind, described by composable specs.
 
-A `StackConfig` lists layers; each has a mixer spec (`LatentAttention`, `GeneralDelta`, `GroupedAttention`),
-optionally a feed-forward spec (`DenseMlp`, `MoeMlp`), and either norms before and after every sublayer or, in a
-parallel layer, one norm in front of both.  Which design a model directory
+A `StackConfig` lists layers; each has a mixer spec (`LatentAttention`, `GeneralDelta`, `GroupedAttention`, `StateSpace`,
+or two of them `SideBySide`), optionally a feed-forward spec (`DenseMlp`, `MoeMlp`), and norms before, or before and
+after, every sublayer or, in a parallel layer, one norm in front of both.  Which design a model directory
 holds is decided by config.json's "architecture" (`DESIGNS`, consulted by model.config_from_dir); a design is
 a reader from its config.json to specs, everything below the specs is shared.  `StackWeights` loads and packs
 the tensors for the kernels (include/bcg_b200.h, bcg_layer); there is nothing model-specific in the engine.
@@ -13,6 +13,7 @@ from __future__ import annotations
 
 import ctypes as C
 import json
+import math
 from dataclasses import dataclass, field, replace
 from pathlib import Path
 from typing import Callable, Dict, Optional, Tuple
@@ -113,8 +114,9 @@ class GeneralDelta:
 
 @dataclass(frozen=True)
 class GroupedAttention:
-    """Grouped-query attention without rotation: a linear distance bias per head, biased projections, queries
-    scaled by 1 + temp_coef * ln(floor((position + 1) / temp_every) + 1)."""
+    """Grouped-query attention without rotation: biased projections, queries scaled by 1 + temp_coef *
+    ln(floor((position + 1) / temp_every) + 1); optionally a linear distance bias per head, RMS norms of a token's
+    queries and of its keys over all heads at once, an output gate per head."""
     heads: int
     kv_heads: int
     dim: int
@@ -125,6 +127,9 @@ class GroupedAttention:
     temp_every: float = 1.0
     v_mix: bool = False             # the first such layer's values are mixed into the later ones'
     slopes: bool = True             # distance slope 2^(-8 (h + 1) / heads) of head h
+    qk_norm: bool = False
+    gate: bool = False              # head outputs times sigmoid of a projection
+    out_bias: bool = True
 
     @property
     def out_dim(self) -> int:
@@ -148,26 +153,103 @@ class GroupedAttention:
 
     @property
     def in_dim(self) -> int:
-        return self.heads * self.dim + self.kv_heads * (self.dim + self.vdim)
+        """Rows of the input projection: q | k | v | gate."""
+        return self.heads * self.dim + self.kv_heads * (self.dim + self.vdim) + (self.heads if self.gate else 0)
 
     def tensors(self, d: int) -> Dict[str, tuple]:
         out = {}
         for n, rows, cols in (("q", self.heads * self.dim, d), ("k", self.kv_heads * self.dim, d),
                               ("v", self.kv_heads * self.vdim, d), ("o", d, self.out_dim)):
-            out.update({n: (rows, cols), n + ".b": (rows,)})
+            out[n] = (rows, cols)
+            if n != "o" or self.out_bias:
+                out[n + ".b"] = (rows,)
+        if self.qk_norm:
+            out.update({"q.norm": (self.heads * self.dim,), "k.norm": (self.kv_heads * self.dim,)})
+        if self.gate:
+            out["g"] = (self.heads, d)
         if self.v_mix:
             out["vmix"] = ()
         return out
 
 
 @dataclass(frozen=True)
+class StateSpace:
+    """State-space mixer with one decay per head: x, B and C behind a causal convolution, a [vdim, state] fp32 state per
+    head, gated outputs normed in `norm_groups` equal parts."""
+    heads: int
+    vdim: int
+    state: int
+    groups: int                     # head h uses B and C of group h / (heads / groups)
+    norm_groups: int
+    conv: int                       # taps
+
+    @property
+    def out_dim(self) -> int:
+        return self.heads * self.vdim
+
+    @property
+    def channels(self) -> int:
+        """Channels of the convolution."""
+        return self.out_dim + 2 * self.groups * self.state
+
+    @property
+    def x_ld(self) -> int:
+        """Columns of the convolved channels, heads and groups padded."""
+        return self.heads * _up(self.vdim, 8) + 2 * self.groups * _up(self.state, 8)
+
+    @property
+    def in_dim(self) -> int:
+        """Rows of the input projection: z | x | B | C | step."""
+        return self.out_dim + self.channels + self.heads
+
+    @property
+    def state_floats(self) -> int:
+        return self.out_dim * self.state + (self.conv - 1) * self.channels
+
+    def tensors(self, d: int) -> Dict[str, tuple]:
+        n = self.out_dim
+        return {"in": (self.in_dim, d), "conv": (self.channels, self.conv), "conv.b": (self.channels,), "dt_bias": (self.heads,),
+                "A_log": (self.heads,), "D": (self.heads,), "norm": (n,), "o": (d, n)}
+
+
+@dataclass(frozen=True)
+class SideBySide:
+    """left_scale * left(h) + right_scale * right(h)."""
+    left: GroupedAttention
+    right: StateSpace
+    left_scale: float = 1.0
+    right_scale: float = 1.0
+
+    def tensors(self, d: int) -> Dict[str, tuple]:
+        return {f"{side}.{n}": s for side, m in (("left", self.left), ("right", self.right)) for n, s in m.tensors(d).items()}
+
+
+@dataclass(frozen=True)
 class DenseMlp:
-    """down(act(up(x))); act is PolyNorm, whose four numbers are weights, or the square of relu."""
+    """down(act(up(x))); act is PolyNorm, whose four numbers are weights, or the square of relu, or a gated unit: gate
+    clamped from above, linear part from both sides, gate * sigmoid(alpha * gate) * (linear + 1)."""
     ff: int
-    act: str = "poly_norm"          # or "relu2"
+    act: str = "poly_norm"          # or "relu2", "clamped_glu"
+    limit: float = 0.0
+    alpha: float = 1.702
+
+    @property
+    def glu(self) -> bool:
+        return self.act == "clamped_glu"
+
+    @property
+    def ff_ld(self) -> int:
+        """Columns of the activations."""
+        return _up(self.ff, 16) if self.glu else self.ff
+
+    @property
+    def up_rows(self) -> int:
+        return 2 * self.ff_ld if self.glu else self.ff
 
     def tensors(self, d: int) -> Dict[str, tuple]:
         t = {"up": (self.ff, d), "down": (d, self.ff)}
+        if self.glu:
+            t["gate"] = (self.ff, d)
         if self.act == "poly_norm":
             t["act"] = (4,)
         return t
@@ -199,6 +281,21 @@ class LayerSpec:
     mixer: object
     mlp: object = None
     parallel: bool = False          # x += mixer(h) + ff(h) with one norm h of x
+    post_norm: bool = True          # the sublayers' outputs are normed too (layers that are not parallel)
+
+    @property
+    def mixers(self) -> tuple:
+        """The mixers that read the layer's input: one, or two side by side."""
+        return (self.mixer.left, self.mixer.right) if isinstance(self.mixer, SideBySide) else (self.mixer,)
+
+    def one(self, kind):
+        """The mixer of this kind, or None."""
+        return next((m for m in self.mixers if isinstance(m, kind)), None)
+
+    @property
+    def composed(self) -> bool:
+        """Grouped attention and / or a state-space mixer behind one input projection."""
+        return not self.parallel and all(isinstance(m, (GroupedAttention, StateSpace)) for m in self.mixers)
 
 
 @dataclass(frozen=True)
@@ -212,24 +309,34 @@ class StackConfig:
     family: str = "qwen3"            # tokenizer / chat-template family
     max_pos: int = 131072
     learned_pos: bool = False        # max_pos position vectors are added to the embedding
+    sinusoid_pos: bool = False       # sines and cosines of position * 10000^(-2i / d_model) are added to the embedding
+    embed_scale: float = 1.0
+    norm_offset: float = 0.0         # added to the stored weights of the layers' and the final norm
 
     def __post_init__(self):
         if self.act_dtype not in ("bfloat16", "float32"):
             raise ValueError(f"act_dtype {self.act_dtype!r}")
         for i, l in enumerate(self.layers):
             m = l.mixer
-            if l.parallel != isinstance(m, GroupedAttention) or isinstance(l.mlp, MoeMlp) and not l.parallel:
-                raise ValueError(f"{self.name}: layer {i}: grouped attention and experts come in parallel layers, and only there")
+            att, ssm = l.one(GroupedAttention), l.one(StateSpace)
+            if l.parallel and not isinstance(m, GroupedAttention) or isinstance(l.mlp, MoeMlp) and not l.parallel:
+                raise ValueError(f"{self.name}: layer {i}: parallel layers have grouped attention, experts come in parallel layers")
             if l.mlp and isinstance(l.mlp, DenseMlp) and (l.mlp.act == "relu2") != l.parallel:
                 raise ValueError(f"{self.name}: layer {i}: activation {l.mlp.act!r} in this kind of layer")
+            if l.parallel and (att.qk_norm or att.gate):
+                raise ValueError(f"{self.name}: layer {i}: query and key norms and gates come in layers that are not parallel")
+            if isinstance(m, SideBySide) and (att is None or ssm is None or att.out_bias):
+                raise ValueError(f"{self.name}: layer {i}: side by side are grouped attention without output bias and a state-space mixer")
+            if ssm and (ssm.heads % ssm.groups or ssm.out_dim % ssm.norm_groups or not 0 < ssm.state <= 256 or ssm.conv < 1):
+                raise ValueError(f"{self.name}: layer {i}: state-space sizes (groups and parts that divide, up to 256 state entries)")
             if isinstance(l.mlp, MoeMlp) and not 0 < l.mlp.top <= l.mlp.experts <= 1024:
                 raise ValueError(f"{self.name}: layer {i}: {l.mlp.top} of {l.mlp.experts} experts (at most 1,024)")
-            if isinstance(m, GroupedAttention):
-                if m.heads % m.kv_heads:
-                    raise ValueError(f"{self.name}: layer {i}: {m.heads} query heads on {m.kv_heads} key/value heads")
-                if m.v_mix:
-                    f = self.layers[self.v_first].mixer
-                    if f.kv_heads * f.vdim != m.kv_heads * m.vdim:
+            if att:
+                if att.heads % att.kv_heads:
+                    raise ValueError(f"{self.name}: layer {i}: {att.heads} query heads on {att.kv_heads} key/value heads")
+                if att.v_mix:
+                    f = self.layers[self.v_first].one(GroupedAttention)
+                    if f.kv_heads * f.vdim != att.kv_heads * att.vdim:
                         raise ValueError(f"{self.name}: layer {i} cannot mix in values of layer {self.v_first}")
             if isinstance(m, GeneralDelta) and m.dim > 256:
                 raise ValueError(f"{self.name}: layer {i}: the delta-rule kernel takes up to 256 channels per head")
@@ -249,7 +356,11 @@ class StackConfig:
     @property
     def v_first(self) -> Optional[int]:
         """The layer whose values later layers mix in."""
-        return next((i for i, l in enumerate(self.layers) if getattr(l.mixer, "v_mix", False)), None)
+        return next((i for i, l in enumerate(self.layers) if any(getattr(m, "v_mix", False) for m in l.mixers)), None)
+
+    def mixers(self, *kinds) -> list:
+        """All mixers of these kinds."""
+        return [m for l in self.layers for m in l.mixers if isinstance(m, kinds)]
 
     @property
     def vocab_ld(self) -> int:
@@ -258,12 +369,12 @@ class StackConfig:
     @property
     def has_state(self) -> bool:
         """True when a prefix's cache pages alone do not restore it (recurrent layers)."""
-        return any(isinstance(l.mixer, GeneralDelta) for l in self.layers)
+        return bool(self.mixers(GeneralDelta, StateSpace))
 
     @property
     def max_window(self) -> int:
         """Largest attention window of the stack, 0 = unbounded."""
-        w = [l.mixer.window for l in self.layers if not isinstance(l.mixer, GeneralDelta)]
+        w = [m.window for m in self.mixers(LatentAttention, GroupedAttention)]
         return 0 if not w or 0 in w else max(w)
 
     @property
@@ -276,19 +387,34 @@ class StackConfig:
 
     @property
     def kv_bytes_per_token(self) -> int:
-        return sum(l.mixer.cache_row for l in self.layers
-                   if not isinstance(l.mixer, GeneralDelta) and getattr(l.mixer, "kv_from", None) is None) * self.itemsize
+        return sum(m.cache_row for m in self.mixers(LatentAttention, GroupedAttention)
+                   if getattr(m, "kv_from", None) is None) * self.itemsize
 
     @property
     def state_bytes_per_row(self) -> int:
-        return sum(4 * l.mixer.heads * l.mixer.dim ** 2 for l in self.layers if isinstance(l.mixer, GeneralDelta))
+        return sum(4 * m.heads * m.dim ** 2 for m in self.mixers(GeneralDelta)) + \
+            sum(4 * m.state_floats for m in self.mixers(StateSpace))
 
     def in_rows(self, i: int) -> int:
         """Rows of layer i's fused input projection, padded for the 256-wide GEMM tiles when it is large."""
         if self.layers[i].parallel:
             return self.qkv_rows(i) + self.up_rows(i)
-        n = self.layers[i].mixer.in_rows()
+        if self.layers[i].composed:
+            ssm = self.layers[i].one(StateSpace)
+            n = self.ssm_col(i) + (ssm.in_dim if ssm else 0)
+        else:
+            n = self.layers[i].mixer.in_rows()
         return _up(n, 256 if n >= 2048 else 16)
+
+    def ssm_col(self, i: int) -> int:
+        """Composed layers: first state-space row of the input projection, behind the attention's."""
+        att = self.layers[i].one(GroupedAttention)
+        return _up(att.in_dim, 16) if att else 0
+
+    def ssm_mix_col(self, i: int) -> int:
+        """Composed layers: first state-space column of what the output projection reads."""
+        att = self.layers[i].one(GroupedAttention)
+        return _up(att.out_dim, 8) if att else 0
 
     def qkv_rows(self, i: int) -> int:
         """Parallel layers: padded rows of q | k | v | router."""
@@ -303,6 +429,10 @@ class StackConfig:
 
     def mix_cols(self, i: int) -> Tuple[int, int]:
         """(first activation column, columns) of what layer i's output projection reads."""
+        if self.layers[i].composed:
+            ssm = self.layers[i].one(StateSpace)
+            n = _up(self.ssm_mix_col(i) + (ssm.out_dim if ssm else 0), 8)
+            return n, n
         n = self.layers[i].mixer.out_dim
         return (_up(n, 8), _up(n, 8) + self.up_rows(i)) if self.layers[i].parallel else (n, n)
 
@@ -314,6 +444,8 @@ class StackConfig:
             out["pos"] = (self.max_pos, d)
         for i, l in enumerate(self.layers):
             norms = ("norm1",) if l.parallel else ("norm1", "norm1b") + (("norm2", "norm2b") if l.mlp else ())
+            if not l.post_norm:
+                norms = tuple(n for n in norms if not n.endswith("b"))
             out.update({f"l{i}.{n}": (d,) for n in norms})
             out.update({f"l{i}.mix.{n}": s for n, s in l.mixer.tensors(d).items()})
             if l.mlp:
@@ -387,7 +519,38 @@ def _lerazen(c: dict, shape: Callable[[str], tuple], name: str) -> StackConfig:
                        rms_eps=float(c["norm"]["eps"]), max_pos=int(c["max_positions"]), learned_pos=True)
 
 
-DESIGNS: Dict[str, Callable] = {"Bekopel": _bekopel, "Lerazen": _lerazen}
+def _state_space(m: dict) -> StateSpace:
+    return StateSpace(heads=int(m["heads"]), vdim=int(m["vdim"]), state=int(m["state"]), groups=int(m["groups"]),
+                      norm_groups=int(m["norm_groups"]), conv=int(m["conv"]))
+
+
+def _merulorn(c: dict, shape: Callable[[str], tuple], name: str) -> StackConfig:
+    """config.json of the Merulorn design."""
+    layers = []
+    for i, e in enumerate(c["layers"]):
+        m, kind = e["mixer"], e["type"]
+        if kind == "parallel":
+            a = m["left"]
+            temp = a.get("q_temp") or {"coef": 0.0, "every": 1}
+            left = GroupedAttention(heads=int(a["heads"]), kv_heads=int(a["kv_heads"]), dim=int(a["dim"]), vdim=int(a["vdim"]),
+                                    scale=float(a["scale"]), temp_coef=float(temp["coef"]), temp_every=float(temp["every"]),
+                                    slopes=False, qk_norm=True, gate=True, out_bias=False)
+            mixer = SideBySide(left, _state_space(m["right"]), float(m["left_scale"]), float(m["right_scale"]))
+        elif kind == "mamba2":
+            mixer = _state_space(m)
+        else:
+            raise ValueError(f"{name}: layer {i}: unknown mixer {kind!r}")
+        f = e.get("mlp")
+        if f is not None and f.get("kind") != "dense":
+            raise ValueError(f"{name}: layer {i}: unknown feed-forward {f.get('kind')!r}")
+        mlp = DenseMlp(int(f["ff"]), "clamped_glu", float(f["limit"])) if f is not None else None
+        layers.append(LayerSpec(mixer, mlp, post_norm=False))
+    return StackConfig(name=name, d_model=int(c["width"]), vocab=int(c["vocab"]), layers=tuple(layers),
+                       rms_eps=float(c["norm"]["eps"]), sinusoid_pos=True, embed_scale=float(c["embedding"]["scale"]),
+                       norm_offset=1.0)
+
+
+DESIGNS: Dict[str, Callable] = {"Bekopel": _bekopel, "Lerazen": _lerazen, "Merulorn": _merulorn}
 
 
 def safetensors_shapes(path) -> Dict[str, tuple]:
@@ -439,11 +602,28 @@ def lerazen_preset(name: str, n_layers: int, d_model: int, ff: int, vocab: int, 
     return StackConfig(name, d_model, vocab, layers, max_pos=max_pos, learned_pos=True)
 
 
+def merulorn_preset(name: str, n_layers: int, d_model: int, ff: int, vocab: int, heads: int = 32, kv_heads: int = 8,
+                    dim: int = 128, vdim: int = 64, state: int = 128, groups: int = 8, max_pos: int = 32768) -> StackConfig:
+    """Merulorn at sizes of a real model's layers (random-init presets, bench): one layer in four has attention beside the
+    state-space mixer and a feed-forward."""
+    ssm = StateSpace(2 * d_model // vdim, vdim, state, groups, groups, 4)
+    att = GroupedAttention(heads, kv_heads, dim, dim, dim ** -0.5, 0, 0.1, 8192, slopes=False, qk_norm=True, gate=True, out_bias=False)
+    both = LayerSpec(SideBySide(att, ssm, 0.7, 0.7), DenseMlp(ff, "clamped_glu", 7.0), post_norm=False)
+    layers = tuple(LayerSpec(ssm, None, post_norm=False) if i % 4 in (1, 2, 3) else both for i in range(n_layers))
+    return StackConfig(name, d_model, vocab, layers, max_pos=max_pos, sinusoid_pos=True, embed_scale=d_model ** 0.5, norm_offset=1.0)
+
+
 # ------------------------------------------------------------------------------------------ weights
 def head_slopes(heads: int, device) -> torch.Tensor:
     """[heads] fp32 distance slopes 2^(-8 (h + 1) / heads)."""
     h = torch.arange(1, heads + 1, dtype=torch.float64)
     return torch.exp2(-8.0 * h / heads).float().to(device)
+
+
+def position_turns(width: int, device) -> torch.Tensor:
+    """[(width + 1) // 2] fp64: turns per position of the sinusoids, 10000^(-2i / width) / 2 pi."""
+    i = torch.arange((width + 1) // 2, dtype=torch.float64)
+    return (10000.0 ** (-2.0 * i / width) / (2.0 * math.pi)).to(device)
 
 
 def rope_table(rot: Rotary, n_pos: int, device) -> torch.Tensor:
@@ -463,6 +643,7 @@ class StackWeights:
     final_norm: torch.Tensor
     layers: list = field(default_factory=list)
     pos_embed: Optional[torch.Tensor] = None
+    pos_turns: Optional[torch.Tensor] = None
 
     @staticmethod
     def from_tensors(cfg: StackConfig, get: Callable[[str], torch.Tensor], device) -> "StackWeights":
@@ -481,16 +662,22 @@ class StackWeights:
         def rows(t, n):
             return t if t.shape[0] == n else torch.cat([t, t.new_zeros(n - t.shape[0], *t.shape[1:])])
 
-        w = StackWeights(cfg, bf(raw("embed")), bf(rows(raw("head"), cfg.vocab_ld)), f32(raw("final.norm")))
+        norm = lambda n: f32(raw(n)) + cfg.norm_offset
+        w = StackWeights(cfg, bf(raw("embed")), bf(rows(raw("head"), cfg.vocab_ld)), norm("final.norm"))
+        if cfg.sinusoid_pos:
+            w.pos_turns = position_turns(cfg.d_model, device)
         if cfg.learned_pos:
             w.pos_embed = bf(raw("pos"))
         for i, l in enumerate(cfg.layers):
             m, g = l.mixer, lambda n: raw(f"l{i}.mix.{n}")
             if l.parallel:
-                w.layers.append(StackWeights._parallel(cfg, i, raw, bf, f32, rows))
+                w.layers.append(StackWeights._parallel(cfg, i, raw, norm, bf, f32, rows))
                 continue
-            t = {"norm1": f32(raw(f"l{i}.norm1")), "norm1b": f32(raw(f"l{i}.norm1b")), "w_out": bf(g("o"))}
-            if isinstance(m, LatentAttention):
+            t = {n: norm(f"l{i}.{n}") for n in ("norm1", "norm1b", "norm2", "norm2b") if f"l{i}.{n}" in want}
+            if l.composed:
+                t.update(StackWeights._composed(cfg, i, raw, bf, f32, rows))
+            elif isinstance(m, LatentAttention):
+                t["w_out"] = bf(g("o"))
                 own = m.kv_from is None
                 t["w_in"] = bf(rows(torch.cat([g("q"), g("dkv")]) if own else g("q"), cfg.in_rows(i)))
                 if own:
@@ -501,19 +688,62 @@ class StackWeights:
                 if m.q_ld and cfg.act_dtype == "bfloat16":
                     t["w_expand"] = StackWeights.expansion(m, t["w_uk"], t["w_uv"])
             else:
+                t["w_out"] = bf(g("o"))
                 w1 = rows(g("w1"), m.rank_ld)
                 t["w_in"] = bf(rows(torch.cat([g("r"), g("k"), g("v"), g("g"), g("a"), w1]), cfg.in_rows(i)))
                 w2 = g("w2")
                 t["w_decay"] = bf(torch.cat([w2, w2.new_zeros(w2.shape[0], m.rank_ld - m.decay_rank)], dim=1))
                 t["decay_bias"], t["rate_bias"], t["out_norm"] = f32(g("w0")), f32(g("a.b")), f32(g("norm"))
-            if l.mlp:
-                t.update(norm2=f32(raw(f"l{i}.norm2")), norm2b=f32(raw(f"l{i}.norm2b")), w_up=bf(raw(f"l{i}.mlp.up")),
-                         w_down=bf(raw(f"l{i}.mlp.down")), act_coef=f32(raw(f"l{i}.mlp.act")))
+            if l.mlp and l.mlp.glu:
+                t["w_up"] = StackWeights.glu_rows(*(rows(bf(raw(f"l{i}.mlp.{n}")), l.mlp.ff_ld) for n in ("gate", "up")))
+                t["w_down"] = torch.zeros(cfg.d_model, l.mlp.ff_ld, dtype=torch.bfloat16, device=device)
+                t["w_down"][:, :l.mlp.ff] = bf(raw(f"l{i}.mlp.down"))
+            elif l.mlp:
+                t.update(w_up=bf(raw(f"l{i}.mlp.up")), w_down=bf(raw(f"l{i}.mlp.down")), act_coef=f32(raw(f"l{i}.mlp.act")))
             w.layers.append(t)
         return w
 
     @staticmethod
-    def _parallel(cfg: StackConfig, i: int, raw, bf, f32, rows) -> dict:
+    def glu_rows(gate: torch.Tensor, up: torch.Tensor) -> torch.Tensor:
+        """Gate and up rows (a multiple of 16 of each) interleaved by 16."""
+        n, d = gate.shape
+        return torch.stack([gate.view(n // 16, 16, d), up.view(n // 16, 16, d)], dim=1).reshape(2 * n, d)
+
+    @staticmethod
+    def _composed(cfg: StackConfig, i: int, raw, bf, f32, rows) -> dict:
+        """Grouped attention (q | k | v | gate) and a state-space mixer (z | x | B | C | step) in one input matrix, their
+        output matrices side by side.  Scales of the two join the gate and the state-space norm."""
+        l, d = cfg.layers[i], cfg.d_model
+        att, ssm, both = l.one(GroupedAttention), l.one(StateSpace), isinstance(l.mixer, SideBySide)
+        left = lambda n: raw(f"l{i}.mix." + ("left." if both else "") + n)
+        right = lambda n: raw(f"l{i}.mix." + ("right." if both else "") + n)
+        w_in, t = [], {}
+        some = left("o") if att else right("o")
+        w_out = torch.zeros(d, cfg.mix_cols(i)[1], dtype=torch.bfloat16, device=some.device)
+        if att:
+            w_in.append(rows(torch.cat([left(n) for n in ("q", "k", "v")] + ([left("g")] if att.gate else [])), cfg.ssm_col(i)))
+            w_out[:, :att.out_dim] = bf(left("o"))
+            t["in_bias"] = f32(torch.cat([left("q.b"), left("k.b"), left("v.b")]))
+            if att.out_bias:
+                t["out_bias"] = f32(left("o.b"))
+            if att.qk_norm:
+                t["q_norm"], t["k_norm"] = f32(left("q.norm")), f32(left("k.norm"))
+            if att.slopes:
+                t["slopes"] = head_slopes(att.heads, some.device)
+            if att.v_mix:
+                t["vmix"] = f32(left("vmix"))
+        if ssm:
+            w_in.append(right("in"))
+            at = cfg.ssm_mix_col(i)
+            w_out[:, at:at + ssm.out_dim] = bf(right("o"))
+            t.update(conv_w=f32(right("conv").T), conv_b=f32(right("conv.b")), step_bias=f32(right("dt_bias")),
+                     decay_rate=right("A_log").double().exp().float().contiguous(), skip=f32(right("D")),
+                     ssm_norm=f32(right("norm")) * (l.mixer.right_scale if both else 1.0))
+        t["w_in"], t["w_out"] = bf(rows(torch.cat(w_in), cfg.in_rows(i))), w_out
+        return t
+
+    @staticmethod
+    def _parallel(cfg: StackConfig, i: int, raw, norm, bf, f32, rows) -> dict:
         """A parallel layer: q | k | v | router, then the up rows, in one matrix; o and down side by side in another;
         experts one after another, gate and up rows interleaved by 16."""
         l, d = cfg.layers[i], cfg.d_model
@@ -527,7 +757,7 @@ class StackWeights:
         if dense:
             w_in = torch.cat([w_in, rows(ffn("up"), cfg.up_rows(i))])
             w_out[:, act_col:act_col + f.ff] = bf(ffn("down"))
-        t = {"norm1": f32(raw(f"l{i}.norm1")), "w_in": bf(w_in), "w_out": w_out, "out_bias": f32(g("o.b")),
+        t = {"norm1": norm(f"l{i}.norm1"), "w_in": bf(w_in), "w_out": w_out, "out_bias": f32(g("o.b")),
              "in_bias": f32(torch.cat([g("q.b"), g("k.b"), g("v.b")]))}
         if m.slopes:
             t["slopes"] = head_slopes(m.heads, w_in.device)
@@ -538,8 +768,7 @@ class StackWeights:
             t["w_experts_in"] = torch.zeros(f.experts, 2 * n, d, dtype=torch.bfloat16, device=w_in.device)
             t["w_experts_out"] = torch.zeros(f.experts, d, n, dtype=torch.bfloat16, device=w_in.device)
             for e in range(f.experts):
-                pair = torch.stack([rows(bf(ffn(f"e{e}.{x}")), n).view(n // 16, 16, d) for x in ("gate", "up")], dim=1)
-                t["w_experts_in"][e] = pair.reshape(2 * n, d)
+                t["w_experts_in"][e] = StackWeights.glu_rows(*(rows(bf(ffn(f"e{e}.{x}")), n) for x in ("gate", "up")))
                 t["w_experts_out"][e, :, :f.ff] = bf(ffn(f"e{e}.down"))
         return t
 
@@ -573,10 +802,17 @@ class StackWeights:
                 return torch.tensor([1.0, 0.5, 0.25, 0.0], device=device)
             if n.endswith(".vmix"):
                 return torch.tensor(0.5, device=device)
+            if n.endswith(".conv"):
+                return torch.empty(*s, device=device).normal_(0.0, s[1] ** -0.5, generator=g)
+            if n.endswith(".dt_bias"):      # steps around 0.02
+                return torch.full(s, -4.0, device=device)
+            if n.endswith(".D"):
+                return torch.ones(*s, device=device)
             if len(s) == 2:
                 return torch.empty(*s, dtype=torch.bfloat16, device=device).normal_(0.0, 0.02, generator=g)
             leaf = n.rsplit(".", 1)[-1]
-            return (torch.ones if leaf.startswith("norm") else torch.zeros)(*s, device=device)
+            one = leaf.startswith("norm") and not (cfg.norm_offset and ".mix." not in n)
+            return (torch.ones if one else torch.zeros)(*s, device=device)
         return StackWeights.from_tensors(cfg, get, device)
 
     def nbytes(self) -> int:
@@ -589,8 +825,9 @@ class StackHandle:
     """Host-side bcg_stack (include/bcg_b200.h) over StackWeights, caches and states.
 
     caches[i]: the latent pages [pages, page, cache_row] or the states [slots, heads, dim, dim] of layer i
-    (None where the layer reads another layer's cache); for grouped attention a pair (keys [pages, kv_heads, page,
-    q_ld], values [pages, kv_heads, page, v_ld])."""
+    (None where the layer reads another layer's cache); for grouped attention and state-space mixers a dict of what
+    there is of cache (keys [pages, kv_heads, page, q_ld]), cache_v (values [pages, kv_heads, page, v_ld]), ssm_state
+    [slots, heads, vdim, state] and conv_state [slots, taps - 1, channels]."""
 
     def __init__(self, w: StackWeights, caches: list, n_pos: int, page_size: int):
         cfg = w.cfg
@@ -601,19 +838,34 @@ class StackHandle:
         counts = 0
         for i, (spec, t) in enumerate(zip(cfg.layers, w.layers)):
             a, m = arr[i], spec.mixer
-            a.heads, a.dim, a.n_in = m.heads, m.dim, cfg.in_rows(i)
+            a.n_in = cfg.in_rows(i)
             src = i
-            if isinstance(m, GroupedAttention):
-                a.mixer, a.kv_heads, a.vdim, a.q_ld, a.v_ld = L.MIXER_GROUPED_ATTN, m.kv_heads, m.vdim, m.q_ld, m.v_ld
-                a.window, a.scale, a.owns_cache = m.window, m.scale, 1
-                a.temp_coef, a.temp_every = m.temp_coef, m.temp_every
-                if m.v_mix:
+            att, ssm = spec.one(GroupedAttention), spec.one(StateSpace)
+            if att:
+                a.mixer, a.heads, a.dim = L.MIXER_GROUPED_ATTN, att.heads, att.dim
+                a.kv_heads, a.vdim, a.q_ld, a.v_ld = att.kv_heads, att.vdim, att.q_ld, att.v_ld
+                a.window, a.scale, a.owns_cache = att.window, att.scale, 1
+                a.temp_coef, a.temp_every = att.temp_coef, att.temp_every
+                if att.v_mix:
                     a.v_role = L.VALUES_FIRST if i == cfg.v_first else L.VALUES_MIX
                     a.v_mix = float(t["vmix"])
-                a.parallel, a.n_qkv, a.router_col = 1, cfg.qkv_rows(i), m.in_dim
+                if spec.parallel:
+                    a.parallel, a.n_qkv, a.router_col = 1, cfg.qkv_rows(i), att.in_dim
+                if att.gate:
+                    a.gated, a.gate_col = 1, att.in_dim - att.heads
+                    a.gate_scale = m.left_scale if isinstance(m, SideBySide) else 1.0
                 a.act_col, a.mix_ld = cfg.mix_cols(i)
+            if ssm:
+                if not att:
+                    a.mixer = L.MIXER_STATE_SPACE
+                a.ssm_heads, a.ssm_vdim, a.ssm_n, a.ssm_groups = ssm.heads, ssm.vdim, ssm.state, ssm.groups
+                a.ssm_norm_parts, a.ssm_taps, a.ssm_col, a.ssm_mix_col = ssm.norm_groups, ssm.conv, cfg.ssm_col(i), cfg.ssm_mix_col(i)
+                a.mix_ld = cfg.mix_cols(i)[1]
+            if att or ssm:
+                for n, x in caches[i].items():
+                    setattr(a, n, x.data_ptr() if x.numel() else None)
             elif isinstance(m, LatentAttention):
-                a.mixer = L.MIXER_LATENT_ATTN
+                a.mixer, a.heads, a.dim = L.MIXER_LATENT_ATTN, m.heads, m.dim
                 a.rot_dim, a.rot_dims, a.vdim, a.kv_rank = m.rot_dim, m.rot.dims, m.vdim, m.kv_rank
                 a.window, a.scale, a.owns_cache = m.window, m.scale, int(m.kv_from is None)
                 if "w_expand" in t:
@@ -623,20 +875,21 @@ class StackHandle:
                     self._rope[m.rot] = rope_table(m.rot, n_pos, dev)
                 a.cos_sin = self._rope[m.rot].data_ptr()
             else:
-                a.mixer, a.decay_rank = L.MIXER_GENERAL_DELTA, m.rank_ld
+                a.mixer, a.heads, a.dim, a.decay_rank = L.MIXER_GENERAL_DELTA, m.heads, m.dim, m.rank_ld
             if isinstance(spec.mlp, MoeMlp):
                 f = spec.mlp
                 a.experts, a.top, a.expert_ld, a.glu_limit, a.glu_alpha = f.experts, f.top, f.ff_ld, f.limit, f.alpha
                 a.moe_counts_at = counts
                 counts += f.experts
             else:
-                a.ff = spec.mlp.ff if spec.mlp else 0
+                f = spec.mlp
+                a.ff = f.ff_ld if f else 0
+                if f and f.glu:
+                    a.ff_kind, a.glu_limit, a.glu_alpha = L.FF_CLAMPED_GLU, f.limit, f.alpha
             for n, x in t.items():
                 if n != "vmix":
                     setattr(a, n, x.data_ptr())
-            if isinstance(m, GroupedAttention):
-                a.cache, a.cache_v = (c.data_ptr() for c in caches[i])
-            else:
+            if not (att or ssm):
                 a.cache = caches[src].data_ptr()
         self._layers = arr
         s = L.Stack()
@@ -645,5 +898,8 @@ class StackHandle:
         s.embed, s.lm_head, s.final_norm = w.embed.data_ptr(), w.lm_head.data_ptr(), w.final_norm.data_ptr()
         if w.pos_embed is not None:
             s.pos_embed, s.n_pos = w.pos_embed.data_ptr(), w.pos_embed.shape[0]
+        s.embed_scale = cfg.embed_scale
+        if w.pos_turns is not None:
+            s.pos_turns = w.pos_turns.data_ptr()
         s.layers = C.cast(arr, C.POINTER(L.Layer))
         self.struct = s

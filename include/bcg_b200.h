@@ -22,7 +22,7 @@
 extern "C" {
 #endif
 
-#define BCG_ABI_VERSION 3
+#define BCG_ABI_VERSION 4
 
 /* status codes */
 #define BCG_STATUS_OK 0
@@ -359,8 +359,9 @@ int bcg_model_decode(const bcg_model* m, const bcg_workspace* ws, const int* ids
 /* ---------------------------------------------------------------------------------------------
  * Layer stacks: models whose layers differ in kind (the reference has no counterpart; its engine
  * only meets uniform dense decoders).  Every layer is a mixer and, optionally, a feed-forward, each
- * with a norm before and a norm after it:  x += norm1b(mixer(norm1(x))),  x += norm2b(ff(norm2(x))),
- * or, `parallel`, both behind one norm:  h = norm1(x),  x += mixer(h) + ff(h).
+ * with a norm before and (norm1b / norm2b not NULL) a norm after it:  x += norm1b(mixer(norm1(x))),
+ * x += norm2b(ff(norm2(x))), or, `parallel`, both behind one norm:  h = norm1(x),  x += mixer(h) + ff(h).
+ * A mixer may be two side by side, grouped attention and a state-space mixer, that read the same h.
  * `act_dtype` selects the activations that feed matrix products, the latent cache and the attention
  * operands: BCG_DT_BF16 (tensor-core kernels, fp32 accumulation) or BCG_DT_F32 (true fp32
  * throughout, CUDA-core kernels).  Weights are bf16 in both; the residual, norms, scores, gates and
@@ -370,6 +371,9 @@ int bcg_model_decode(const bcg_model* m, const bcg_workspace* ws, const int* ids
 #define BCG_MIXER_LATENT_ATTN 1
 #define BCG_MIXER_GENERAL_DELTA 2
 #define BCG_MIXER_GROUPED_ATTN 3
+#define BCG_MIXER_STATE_SPACE 4   /* alone; beside grouped attention: ssm_heads > 0 */
+#define BCG_FF_POLY_NORM 0   /* bcg_layer.ff_kind of layers that are not parallel */
+#define BCG_FF_CLAMPED_GLU 1 /* w_up rows interleaved [16 gate | 16 up], glu_limit, glu_alpha */
 #define BCG_VALUES_FIRST 1   /* bcg_layer.v_role: the layer's values are what later layers mix in */
 #define BCG_VALUES_MIX 2     /* values are (1 - v_mix) of its own and v_mix of those */
 
@@ -430,6 +434,26 @@ typedef struct bcg_layer {
   const void* w_experts_in;  /* bf16 [experts][2 * expert_ld][d], rows interleaved [16 gate | 16 up] */
   const void* w_experts_out; /* bf16 [experts][d][expert_ld] */
   void* cache_v;           /* values [pages][kv_heads][page_size][v_ld], columns past vdim zero */
+  /* grouped attention: RMS norms over all heads of a token's queries / keys at once, and an output gate per head */
+  const float* q_norm;     /* [heads * dim] or NULL */
+  const float* k_norm;     /* [kv_heads * dim] or NULL */
+  int gated, gate_col;     /* head outputs times gate_scale * sigmoid(column gate_col + head of the projection) */
+  float gate_scale;
+  int ff_kind;             /* BCG_FF_* */
+  /* state-space mixer: rows z | x | B | C | step of w_in from ssm_col on (ssm_heads * ssm_vdim, the same,
+     ssm_groups * ssm_n twice, ssm_heads rows); x, B and C pass a causal convolution of ssm_taps taps and silu */
+  int ssm_heads, ssm_vdim, ssm_n, ssm_groups;
+  int ssm_norm_parts;      /* equal parts of the output that are normed each by its own root mean square */
+  int ssm_taps, ssm_col;
+  int ssm_mix_col;         /* first column of ws->mix */
+  const float* conv_w;     /* [taps][channels], last row = current token */
+  const float* conv_b;     /* [channels] */
+  const float* step_bias;  /* [heads] */
+  const float* decay_rate; /* [heads] state decays by exp(-decay_rate * step) */
+  const float* skip;       /* [heads] */
+  const float* ssm_norm;   /* [heads * vdim] */
+  float* ssm_state;        /* fp32 [slots][heads][vdim][n] */
+  float* conv_state;       /* fp32 [slots][taps - 1][channels]: the last inputs of the convolution, oldest first */
 } bcg_layer;
 
 typedef struct bcg_stack {
@@ -442,6 +466,8 @@ typedef struct bcg_stack {
   const bcg_layer* layers;  /* host array */
   const void* pos_embed;    /* bf16 [n_pos, d] added to the embedding, or NULL */
   int n_pos;
+  float embed_scale;        /* factor of the embedding */
+  const double* pos_turns;  /* [(d + 1) / 2] turns per position: sin at entry 2i, cos at 2i + 1 are added; or NULL */
 } bcg_stack;
 
 typedef struct bcg_stack_ws {
@@ -452,7 +478,7 @@ typedef struct bcg_stack_ws {
   float* decay;     /* fp32 [T_max, heads * dim] slabs of w_decay */
   long long decay_floats;
   void* q;          /* act [T_max, heads * q_row] */
-  void* mix;        /* act [T_max, heads * (vdim or dim)] */
+  void* mix;        /* act [T_max, columns of w_out] */
   void* act;        /* act [T_max, ff] */
   void* low;        /* act [T_max, decay_rank] */
   void* latents;    /* bf16 [K_max, kv_rank + rot_dim] gathered cache rows */
@@ -480,6 +506,10 @@ typedef struct bcg_stack_ws {
   float* moe_row_weight; /* [rows] */
   int* moe_counts;       /* rows per expert, all layers' one after another; cleared at the start of a step */
   int moe_counts_n, moe_rows_max;
+  float* gates;     /* fp32 [T_max, heads]: factors of the head outputs */
+  void* ssm_x;      /* act [T_max, ssm_x_ld(layer)]: convolved x | B | C, heads and groups padded to multiples of 8 */
+  float* ssm_step;  /* fp32 [T_max, ssm_heads] */
+  void* ssm_y;      /* act [T_max, ssm_heads * ssm_vdim]: gated outputs in front of their norm */
 } bcg_stack_ws;
 
 /* A step: T new tokens of n_seqs sequences, portions of prompts beside single decoded tokens.  All
@@ -562,6 +592,19 @@ int bcg_gemm_grouped(const void* X, const void* W, void* out, int rows, int N, i
 /* No counterpart in the reference: ws->xn through the experts that bcg_grouped_in chose; ws->moe_out receives *splits
  * slabs of [T * top, d], row ws->moe_row[t * top + k] for choice k of token t. */
 int bcg_experts(const bcg_stack* m, const bcg_stack_ws* ws, int layer, int T, int* splits, void* stream);
+
+/* No counterpart in the reference: a state-space mixer behind its input projection (ws->proj, row pitch ld): convolution,
+ * recurrence, gate and norm; states advanced, ws->mix columns ssm_mix_col.. filled.  mode 0: what bcg_stack_step picks
+ * (tensor-core chunks or, one token each, the decode kernel); 1: token by token on CUDA cores. */
+int bcg_state_space(const bcg_stack* m, const bcg_stack_ws* ws, const bcg_step_batch* b, int layer, int n_partials,
+                    long long partial_stride, long long ld, int mode, void* stream);
+/* No counterpart in the reference: clamped gated unit of split-K slabs z [T, 2 * ff], columns interleaved [16 gate | 16 up],
+ * ff % 16 == 0:  out = g * sigmoid(alpha * g) * (u + 1), g = min(gate, limit), u clamped to +-limit. */
+int bcg_clamped_glu(const float* z, int n_partials, long long partial_stride, void* out, int act_dtype, int T, int ff,
+                    float limit, float alpha, void* stream);
+/* No counterpart in the reference: bcg_gemm_bf16_tn with that unit as its epilogue; out bf16 [M, N / 2], N % 32 == 0. */
+int bcg_gemm_bf16_glu(const void* X, const void* W, void* out, int M, int N, int K, float limit, float alpha, int flags,
+                      void* stream);
 
 #ifdef __cplusplus
 }

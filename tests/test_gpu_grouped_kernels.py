@@ -78,7 +78,7 @@ class Attention(OneLayer):
     def run(self, seqs, mode=0):
         """seqs: [(keys [n, G, dim], values [n, G, vdim], queries [k, H, dim] of its last k tokens)]."""
         m, e = self.m, self.eng
-        ck, cv = self.x.caches[0]
+        ck, cv = self.x.caches[0].values()
         junk = torch.randn(ck.shape[:3], generator=gen(1))[..., None].to(self.td).cuda() * 50
         ck[..., :m["dim"]] = junk             # rows nobody wrote must not matter
         cv[..., :m["vdim"]] = junk
@@ -218,7 +218,7 @@ def test_projection_is_split_biased_and_stored(dtype, heads, kv, dim, vdim, ff, 
     for role in (0, L.VALUES_FIRST, L.VALUES_MIX):
         l.v_role = role
         o.set("v_first", first)
-        for c in o.x.caches[0]:
+        for c in o.x.caches[0].values():
             c.zero_()
         o.set("moe_counts", torch.zeros(experts + 8))
         L.check(o.eng.lib.bcg_grouped_in(*o.args(C.byref(b), 0, parts, T * n_in, n_in, 1)))
@@ -233,7 +233,7 @@ def test_projection_is_split_biased_and_stored(dtype, heads, kv, dim, vdim, ff, 
         if role == L.VALUES_MIX:
             v = R.mix_values(v, first.double(), 0.3)
         close(o.get("v_first", T, nv), own if role == L.VALUES_FIRST else first, 2e-6)
-        ck, cv = (c.cpu() for c in o.x.caches[0])
+        ck, cv = (c.cpu() for c in o.x.caches[0].values())
         close(torch.stack([ck[pg, :, r, :dim] for pg, r in used]), k.view(T, kv, dim), tol)
         close(torch.stack([cv[pg, :, r, :vdim] for pg, r in used]), v.view(T, kv, vdim), tol)
         for c, n in ((ck, dim), (cv, vdim)):                # nothing else is touched
@@ -263,7 +263,7 @@ def test_finished_rows_write_nothing():
     o.set("proj", torch.ones(o.layer.n_in))
     L.check(o.eng.lib.bcg_grouped_in(*o.args(C.byref(b), 0, 1, 0, o.layer.n_in, 1)))
     torch.cuda.synchronize()
-    assert not any(c.any() for c in o.x.caches[0])
+    assert not any(c.any() for c in o.x.caches[0].values())
 
 
 def test_temperature_steps_at_multiples():

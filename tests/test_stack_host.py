@@ -130,7 +130,13 @@ def test_bad_parallel_configurations_are_refused(spoil, words):
 def test_mixed_kinds_of_layers_are_refused():
     g = S.GroupedAttention(2, 1, 8, 8, 1.0)
     with pytest.raises(ValueError, match="parallel"):
-        S.StackConfig("x", 16, 16, (S.LayerSpec(g),))
+        S.StackConfig("x", 16, 16, (S.LayerSpec(S.GeneralDelta(1, 8, 8), parallel=True),))
+    with pytest.raises(ValueError, match="not parallel"):
+        S.StackConfig("x", 16, 16, (S.LayerSpec(S.GroupedAttention(2, 1, 8, 8, 1.0, gate=True), parallel=True),))
+    with pytest.raises(ValueError, match="side by side"):
+        S.StackConfig("x", 16, 16, (S.LayerSpec(S.SideBySide(g, S.StateSpace(2, 8, 8, 1, 1, 2))),))
+    with pytest.raises(ValueError, match="state-space sizes"):
+        S.StackConfig("x", 16, 16, (S.LayerSpec(S.StateSpace(3, 8, 8, 2, 1, 2)),))
     with pytest.raises(ValueError, match="activation"):
         S.StackConfig("x", 16, 16, (S.LayerSpec(g, S.DenseMlp(8), True),))
 
