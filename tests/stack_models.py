@@ -1,4 +1,4 @@
-"""Small random layer-stack models for the tests: config.json dicts of the Bekopel and Lerazen designs, their
+"""Small random layer-stack models for the tests: config.json dicts of the Bekopel, Lerazen and Merulorn designs, their
 tensors, and model directories.  Weights are scaled so that every mechanism moves the logits: scores spread over
 several units, sinks that take a visible share, decays from fast to almost none, all four activation numbers set,
 biases and mixed values of the size of what they join.  Routers are decisive: a few coordinates of the stream hold
@@ -34,6 +34,64 @@ def gattn(heads=6, kv_heads=3, dim=24, vdim=40, window=20, coef=0.4, every=23, v
     return {"type": "attention", "mlp": mlp,
             "mixer": {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "mask": {"size": window},
                       "q_temp": {"coef": coef, "every": every}, "scale": scale or 2.0 * dim ** -0.5, "v_mix": v_mix}}
+
+
+def ssm(heads=4, vdim=24, state=20, groups=2, norm_groups=2, conv=4):
+    return {"heads": heads, "vdim": vdim, "state": state, "groups": groups, "norm_groups": norm_groups, "conv": conv}
+
+
+def glu(ff, limit=1.5):
+    return {"kind": "dense", "ff": ff, "limit": limit}
+
+
+def mamba(mlp=None, **kw):
+    return {"type": "mamba2", "mixer": ssm(**kw), "mlp": mlp}
+
+
+def both(heads=6, kv_heads=3, dim=24, vdim=40, coef=0.4, every=23, scale=None, left_scale=0.8, right_scale=1.3, mlp=None, heads_ssm=4,
+         vdim_ssm=24, **kw):
+    left = {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "q_temp": {"coef": coef, "every": every},
+            "scale": scale or 2.0 * dim ** -0.5}
+    return {"type": "parallel", "mlp": mlp,
+            "mixer": {"left": left, "left_scale": left_scale, "right": ssm(heads_ssm, vdim_ssm, **kw), "right_scale": right_scale}}
+
+
+def side_config(layers, width=80, vocab=200, eps=1e-5, scale=3.0):
+    return {"architecture": "Merulorn", "layers": layers, "norm": {"eps": eps}, "vocab": vocab, "width": width,
+            "embedding": {"scale": scale}}
+
+
+def side_tensors(cfg, seed=0):
+    g = torch.Generator().manual_seed(seed)
+    rnd = lambda *s, std=1.0, mean=0.0: torch.randn(*s, generator=g) * std + mean
+    d, V = cfg["width"], cfg["vocab"]
+    lin = lambda n, k, gain=1.0: rnd(n, k, std=gain * k ** -0.5)
+    t = {"embed": rnd(V, d, std=0.5), "final.norm": rnd(d, std=0.2), "head": lin(V, d)}
+
+    def state_space(p, m):
+        H, n = m["heads"], m["heads"] * m["vdim"]
+        ch = n + 2 * m["groups"] * m["state"]
+        # decays from a few tokens to thousands of them
+        t.update({p + "in": lin(n + ch + H, d), p + "conv": rnd(ch, m["conv"], std=m["conv"] ** -0.5), p + "conv.b": rnd(ch, std=0.2),
+                  p + "dt_bias": torch.linspace(-3.0, 0.5, H), p + "A_log": torch.linspace(-5.0, 0.5, H)[torch.randperm(H, generator=g)],
+                  p + "D": rnd(H, std=0.2, mean=0.8), p + "norm": rnd(n, std=0.2, mean=1.0), p + "o": lin(d, n)})
+    for i, l in enumerate(cfg["layers"]):
+        p, m, f = f"l{i}.", l["mixer"], l["mlp"]
+        t[p + "norm1"] = rnd(d, std=0.2)
+        if l["type"] == "parallel":
+            a, q = m["left"], p + "mix.left."
+            H, G = a["heads"], a["kv_heads"]
+            for n, rows in (("q", H * a["dim"]), ("k", G * a["dim"]), ("v", G * a["vdim"])):
+                t[q + n], t[q + n + ".b"] = lin(rows, d), rnd(rows, std=0.5)
+            t.update({q + "q.norm": rnd(H * a["dim"], std=0.3, mean=1.0), q + "k.norm": rnd(G * a["dim"], std=0.3, mean=1.0),
+                      q + "g": lin(H, d, 2.0), q + "o": lin(d, H * a["vdim"], 1.5)})
+            state_space(p + "mix.right.", m["right"])
+        else:
+            state_space(p + "mix.", m)
+        if f:
+            t[p + "norm2"] = rnd(d, std=0.2)
+            t.update({p + "mlp.gate": lin(f["ff"], d, 1.5), p + "mlp.up": lin(f["ff"], d, 1.5), p + "mlp.down": lin(d, f["ff"])})
+    return {n: x.to(torch.bfloat16) for n, x in t.items()}
 
 
 def parallel_config(layers, width=80, vocab=200, eps=1e-5, positions=512):
@@ -91,6 +149,8 @@ def tensors(cfg, seed=0, decay_rank=12):
     """name -> bf16 tensor, as a checkpoint of the design holds them."""
     if cfg["architecture"] == "Lerazen":
         return parallel_tensors(cfg, seed)
+    if cfg["architecture"] == "Merulorn":
+        return side_tensors(cfg, seed)
     g = torch.Generator().manual_seed(seed)
     rnd = lambda *s, std=1.0, mean=0.0: (torch.randn(*s, generator=g) * std + mean).to(torch.bfloat16)
     d, V = cfg["width"], cfg["vocab"]

@@ -47,8 +47,21 @@ CONFIGS = {
     "parallel-odd": SM.parallel_config([SM.gattn(3, 1, 7, 11, 19, mlp=SM.dense(45)), SM.gattn(5, 5, 9, 6, 40, v_mix=False, mlp=SM.moe(5, 3, 21)),
                                         SM.gattn(3, 1, 13, 11, 130, every=1, mlp=SM.dense(51))], width=61, vocab=83),
     "parallel-one": SM.parallel_config([SM.gattn(1, 1, 8, 8, 5, mlp=SM.dense(20))], width=36, vocab=36, positions=300),
+    # attention beside a state space, state spaces alone, with and without a feed-forward
+    "side": SM.side_config([SM.mamba(), SM.both(mlp=SM.glu(70)), SM.mamba(heads=2, vdim=40, state=33, groups=1, norm_groups=4, conv=2, mlp=SM.glu(48, 0.4)),
+                            SM.both(4, 1, 16, 24, every=64, coef=-0.1, conv=3)]),
+    # everything on the tensor-core kernels, two blocks of head entries, more parts than groups and fewer
+    "side-tensor": SM.side_config([SM.both(8, 2, 64, 32, mlp=SM.glu(320, 7.0), vdim_ssm=80, state=64), SM.mamba(heads=4, vdim=64, state=128, groups=1, norm_groups=8),
+                                   SM.both(2, 1, 128, 128, every=1, vdim_ssm=16, state=144, groups=4, norm_groups=1)], width=192, vocab=320),
+    # sizes no vector load or tile likes; one tap, five taps
+    "side-odd": SM.side_config([SM.both(3, 1, 7, 11, mlp=SM.glu(45), vdim_ssm=9, state=7, groups=1, norm_groups=3, conv=5),
+                                SM.mamba(heads=6, vdim=5, state=13, groups=3, norm_groups=5, conv=1), SM.both(5, 5, 9, 6, vdim_ssm=21, state=35, conv=2)],
+                               width=61, vocab=83, eps=1e-3, scale=1.0),
+    "side-wide": SM.side_config([SM.both(33, 1, 40, 8, heads_ssm=1, vdim_ssm=136, state=250, groups=1, norm_groups=1, mlp=SM.glu(16)),
+                                 SM.both(2, 2, 264, 264, heads_ssm=1, vdim_ssm=8, state=8, groups=1, norm_groups=1)], width=96, vocab=96),
+    "state-only": SM.side_config([SM.mamba(heads=1, vdim=8, state=16, groups=1, norm_groups=1), SM.mamba(heads=16, vdim=32, state=32, groups=8, norm_groups=16)], width=64, vocab=64),
 }
-ATTENTION_MIX = ["mixed", "tensor", "parallel", "parallel-tensor"]
+ATTENTION_MIX = ["mixed", "tensor", "parallel", "parallel-tensor", "side", "side-tensor"]
 
 
 class Model:
@@ -179,7 +192,7 @@ def test_pool_is_as_large_as_asked_and_says_when_it_is_full():
 
 
 @pytest.mark.parametrize("dtype", TOL)
-@pytest.mark.parametrize("name", ["mixed", "parallel"])
+@pytest.mark.parametrize("name", ["mixed", "parallel", "side"])
 def test_long_decoding(name, dtype):
     """Windows pass over decoded tokens many times over; the state is carried through every one of them."""
     m = Model(name, dtype)
@@ -188,10 +201,11 @@ def test_long_decoding(name, dtype):
 
 
 @pytest.mark.parametrize("dtype", ["float32"])
-def test_a_far_token_is_remembered(dtype):
+@pytest.mark.parametrize("name", ["mixed", "state-only"])
+def test_a_far_token_is_remembered(name, dtype):
     """Slow decays: logits hundreds of tokens later depend on the first ones (a lost state would show)."""
-    m = Model("mixed", dtype)
-    for n in ("l1.mix.w0", "l4.mix.w0"):
+    m = Model(name, dtype)
+    for n in ("l1.mix.w0", "l4.mix.w0") if name == "mixed" else ("l0.mix.A_log", "l1.mix.A_log"):
         m.t[n] -= 6.0
     m.eng = SM.engine(m.cfg, m.t, dtype)
     toks = m.tokens(300, 4)
@@ -213,9 +227,10 @@ def test_learned_positions_end_where_the_table_does():
 
 
 @pytest.mark.parametrize("dtype", TOL)
-def test_prompts_of_many_tiles(dtype):
-    """More tokens than one row tile of the experts' products, several prompt tiles, windows across them."""
-    m = Model("parallel-tensor", dtype, tokens=1024, max_model_len=512)
+@pytest.mark.parametrize("name", ["parallel-tensor", "side-tensor"])
+def test_prompts_of_many_tiles(name, dtype):
+    """More tokens than one row tile of the products, several prompt tiles and chunks, windows across them."""
+    m = Model(name, dtype, tokens=1024, max_model_len=512)
     a, b = m.tokens(500, 1), m.tokens(333, 2)
     sa, sb = m.eng.open(), m.eng.open()
     out = [m.eng.step([(sa, a[:400], list(range(400))), (sb, b[:3], [0, 1, 2])]),
@@ -245,7 +260,9 @@ GEN = SM.config([SM.delta(heads=2, dim=32), SM.attn(4, 32, 32, 32, 64, 24), SM.a
                 width=128, vocab=1024)
 GENS = {"Bekopel": GEN, "Lerazen": SM.parallel_config([SM.gattn(4, 2, 32, 32, 24, mlp=SM.dense(96)), SM.gattn(4, 1, 64, 64, 40, mlp=SM.moe(8, 2, 48)),
                                                        SM.gattn(2, 2, 40, 48, 1000, v_mix=False, mlp=SM.moe(4, 1, 32))],
-                                                      width=128, vocab=1024, positions=600)}
+                                                      width=128, vocab=1024, positions=600),
+        "Merulorn": SM.side_config([SM.mamba(heads=4, vdim=32, state=32), SM.both(4, 2, 32, 32, mlp=SM.glu(96)), SM.mamba(heads=2, vdim=64, state=40, norm_groups=1),
+                                    SM.both(2, 1, 64, 64, vdim_ssm=16, mlp=SM.glu(64, 0.7))], width=128, vocab=1024)}
 
 
 def _greedy(cfg, t, ids, out):
@@ -316,7 +333,7 @@ def test_adapter_generates_from_a_model_directory(design, tmp_path):
 
 # ------------------------------------------------------------------------------------------ trace replay
 @pytest.mark.parametrize("dtype", TOL)
-@pytest.mark.parametrize("name", ["tensor", "parallel-tensor"])
+@pytest.mark.parametrize("name", ["tensor", "parallel-tensor", "side-tensor"])
 def test_trace_replay_program(tmp_path, name, dtype):
     cfg = CONFIGS[name]
     t = SM.tensors(cfg, seed=11)

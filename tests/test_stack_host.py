@@ -168,7 +168,99 @@ def test_preset_resolves_by_name():
     with pytest.raises(ValueError, match="tensor parallelism"):
         c.shard(2)
     c = M.config_for("lerazen-30b-a3b")
+    assert M.config_for("merulorn-8b").layers[0].mixer.right.state == 128
     assert c.layers[0].mlp.act == "relu2" and c.layers[1].mlp.experts == 128 and c.v_first == 0
+
+
+# ---------------------------------------------------------------------------------------- mixers side by side
+SIDE = SM.side_config([SM.mamba(mlp=SM.glu(20, 0.5)), SM.both(heads=6, kv_heads=3, dim=7, vdim=9, mlp=None, conv=3), SM.mamba(heads=3, vdim=5, state=7, groups=1, norm_groups=5, conv=1)],
+                      width=60, eps=1e-3, scale=2.5)
+
+
+def test_side_config_comes_from_the_directory(tmp_path):
+    t = SM.tensors(SIDE)
+    c = M.config_from_dir(str(SM.save(SIDE, t, tmp_path / "m")))
+    assert isinstance(c, S.StackConfig) and set(c.tensor_shapes()) == set(t)
+    assert all(tuple(t[n].shape) == s for n, s in c.tensor_shapes().items())
+    assert c.sinusoid_pos and c.embed_scale == 2.5 and c.norm_offset == 1.0 and c.rms_eps == 1e-3 and c.has_state
+    assert c.layers[0].mixer == S.StateSpace(4, 24, 20, 2, 2, 4) and c.layers[0].mlp == S.DenseMlp(20, "clamped_glu", 0.5, 1.702)
+    m = c.layers[1].mixer
+    assert (m.left_scale, m.right_scale, m.right.conv) == (0.8, 1.3, 3) and c.layers[1].mlp is None
+    assert m.left == S.GroupedAttention(6, 3, 7, 9, 2.0 * 7 ** -0.5, 0, 0.4, 23.0, slopes=False, qk_norm=True, gate=True, out_bias=False)
+    assert c.kv_bytes_per_token == 2 * 3 * (64 + 64)
+    ch = (96 + 80, 96 + 80, 15 + 14)
+    assert c.state_bytes_per_row == 4 * (96 * 20 + 3 * ch[0] + 96 * 20 + 2 * ch[1] + 15 * 7)
+    w = S.StackWeights.from_safetensors_dir(c, tmp_path / "m", "cpu")
+    assert torch.equal(w.final_norm, 1 + t["final.norm"].float()) and torch.equal(w.layers[0]["norm2"], 1 + t["l0.norm2"].float())
+
+
+def test_side_layers_are_packed_side_by_side():
+    t = SM.tensors(SIDE)
+    c = SM.stack_config(SIDE, t)
+    w = S.StackWeights.from_tensors(c, t.__getitem__, "cpu")
+    a, b, m = w.layers[1], w.layers[0], c.layers[1].mixer
+    assert c.ssm_col(1) == 96 and m.left.in_dim == 42 + 21 + 27 + 6       # q | k | v | gate
+    assert torch.equal(a["w_in"][90:96], t["l1.mix.left.g"]) and torch.equal(a["w_in"][96:96 + m.right.in_dim], t["l1.mix.right.in"])
+    assert not a["w_in"][96 + m.right.in_dim:].any() and a["w_in"].shape[0] % 16 == 0
+    assert c.ssm_mix_col(1) == 56 and c.mix_cols(1) == (152, 152) and a["w_out"].shape == (60, 152)
+    assert torch.equal(a["w_out"][:, :54], t["l1.mix.left.o"]) and not a["w_out"][:, 54:56].any()
+    assert torch.equal(a["w_out"][:, 56:], t["l1.mix.right.o"]) and "slopes" not in a and "out_bias" not in a
+    assert torch.allclose(a["ssm_norm"], 1.3 * t["l1.mix.right.norm"].float()) and torch.equal(b["ssm_norm"], t["l0.mix.norm"].float())
+    assert torch.equal(a["conv_w"][2], t["l1.mix.right.conv"][:, 2].float()) and a["conv_w"].is_contiguous()
+    assert torch.allclose(b["decay_rate"], t["l0.mix.A_log"].float().exp())
+    gate, up = b["w_up"].view(2, 2, 16, 60).unbind(1)
+    for x, n in ((gate, "gate"), (up, "up")):
+        assert torch.equal(x.reshape(32, 60)[:20], t[f"l0.mlp.{n}"]) and not x.reshape(32, 60)[20:].any()
+    assert torch.equal(b["w_down"][:, :20], t["l0.mlp.down"]) and not b["w_down"][:, 20:].any()
+    # sizes of the third layer: one group, output columns padded for the product
+    assert c.mix_cols(2) == (16, 16) and c.layers[2].mixer.x_ld == 3 * 8 + 2 * 8
+
+
+@pytest.mark.parametrize("spoil, words", [
+    (lambda c: c["layers"][0].update(type="other"), "unknown mixer"),
+    (lambda c: c["layers"][0]["mlp"].update(kind="moe"), "unknown feed-forward"),
+    (lambda c: c["layers"][1]["mixer"]["left"].update(kv_heads=4), "key/value heads"),
+    (lambda c: c["layers"][0]["mixer"].update(groups=3), "state-space sizes"),
+    (lambda c: c["layers"][0]["mixer"].update(norm_groups=5), "state-space sizes"),
+    (lambda c: c["layers"][0]["mixer"].update(state=257), "state-space sizes"),
+])
+def test_bad_side_configurations_are_refused(spoil, words):
+    import copy
+    c = copy.deepcopy(SIDE)
+    spoil(c)
+    with pytest.raises(ValueError, match=words):
+        SM.stack_config(c, SM.tensors(SIDE))
+
+
+def test_position_turns_are_the_oracles_frequencies():
+    turns = S.position_turns(7, "cpu")
+    pos = torch.tensor([0, 1, 17, 90001])
+    ang = 2 * np.pi * pos.double()[:, None] * turns[None]
+    want = R.sinusoid(pos, 7)
+    assert torch.allclose(ang.sin(), want[:, 0::2], atol=1e-9) and torch.allclose(ang.cos()[:, :3], want[:, 1::2], atol=1e-9)
+
+
+def test_oracle_state_space_can_be_carried():
+    g = torch.Generator().manual_seed(3)
+    rnd = lambda *s: torch.randn(*s, generator=g, dtype=torch.float64)
+    x, B, C, dt, A, D = rnd(9, 4, 3), rnd(9, 2, 5), rnd(9, 2, 5), rnd(9, 4).abs(), rnd(4), rnd(4)
+    whole, s = R.ssm_scan(x, B, C, dt, A, D)
+    y1, s1 = R.ssm_scan(x[:4], B[:4], C[:4], dt[:4], A, D)
+    y2, s2 = R.ssm_scan(x[4:], B[4:], C[4:], dt[4:], A, D, s1)
+    assert torch.allclose(whole, torch.cat([y1, y2])) and torch.allclose(s, s2)
+    # head 2 uses group 1; one step by hand
+    want = torch.exp(-torch.exp(A[2]) * dt[4, 2]) * s1[2] + dt[4, 2] * B[4, 1][:, None] * x[4, 2][None]
+    assert torch.allclose(R.ssm_scan(x[4:5], B[4:5], C[4:5], dt[4:5], A, D, s1)[1][2], want)
+    assert torch.allclose(y2[0, 2], want.T @ C[4, 1] + D[2] * x[4, 2])
+
+
+def test_oracle_convolution_parts_and_heads():
+    x, w, b = torch.tensor([[1.0], [2.0], [4.0]]), torch.tensor([[10.0, 1.0]]), torch.tensor([0.5])
+    assert R.causal_conv(x, w, b).flatten().tolist() == [1.5, 12.5, 24.5]
+    assert R.causal_conv(x[1:], w, b, x[:1]).flatten().tolist() == [12.5, 24.5]
+    y = R.part_norm(torch.tensor([[3.0, 4.0, 0.0, 2.0]]), 2, 0.0, torch.tensor([1.0, 1.0, 1.0, 5.0]))
+    assert torch.allclose(y, torch.tensor([[3.0, 4.0, 0.0, 10.0]]) / torch.tensor([12.5 ** 0.5] * 2 + [2.0 ** 0.5] * 2))
+    assert torch.allclose(R.zero_norm(torch.tensor([[3.0, 4.0]]), 0.0, torch.tensor([0.0, -1.0])), torch.tensor([[3.0 / 12.5 ** 0.5, 0.0]]))
 
 
 # ---------------------------------------------------------------------------------------- work lists
