@@ -11,9 +11,11 @@
 //               that the state stays in fp32 accumulators and becomes an operand without leaving the registers.  What is
 //               fp32 by nature - the state, decays, steps - enters a product as two bf16 halves (hi + lo).
 //   ssm_scan    portions token by token in fp32: the fp32 engine's kernel
-//   ssm_token   one token per sequence (decode): convolution, recurrence and gate in one kernel; the state is requested
+//   ssm_token   one token per sequence (decode): convolution and recurrence in one kernel; the states are requested
 //               before the dependency wait
-//   ssm_norm    norm of the gated outputs; the convolution's state moves on
+//   ssm_norm    gate and norm of the outputs
+// The convolution's state moves on where nobody reads it any more: behind the chunks or the scan, and in ssm_norm for
+// single tokens (whose B and C every head of a group convolves for itself).
 #include "mma_sync.cuh"
 #include "attn_tcgen05.cuh"
 #include "stack_common.cuh"
@@ -73,8 +75,10 @@ __device__ __forceinline__ Vec<V> conv_input(const SsmArgs& a, int c, int t, int
   return x;
 }
 
-// TAPS: a window of inputs in registers; 0: any number of taps, every input loaded where it is used.
-template <typename T, int V, int TAPS>
+constexpr int kConvAhead = 4;     // inputs in flight per thread
+
+// TAPS: a window of inputs in registers; 0: any number of taps, every input loaded where it is used.  ONE: one slab.
+template <typename T, int V, int TAPS, bool ONE>
 __global__ void __launch_bounds__(kConvThreads)
 ssm_conv_kernel(const SsmArgs a, int run, int conv_blocks) {
   pdl_launch_dependents();
@@ -88,9 +92,10 @@ ssm_conv_kernel(const SsmArgs a, int run, int conv_blocks) {
           softplus_f32(slab_sum(a.row(t) + a.inner() + a.channels() + h, a.n_partials, a.pstride) + a.step_bias[h]);
     return;
   }
-  const int c = (blockIdx.x * kConvThreads + threadIdx.x) * V, ch = a.channels();
+  const int c = (blockIdx.x * kConvThreads + threadIdx.x) * V, ch = a.channels(), x_ld = a.x_ld();
   if (c >= ch) return;
   T* out = static_cast<T*>(a.x) + a.x_col(c);
+  const float* in = a.row(0) + a.inner() + c;
   const Vec<V> bias = load_vec<V>(a.conv_b + c);
   constexpr int W = TAPS > 0 ? TAPS : 1;
   Vec<V> w[W], hist[W];            // hist[k - 1]: input of token t - k
@@ -98,58 +103,87 @@ ssm_conv_kernel(const SsmArgs a, int run, int conv_blocks) {
 #pragma unroll
     for (int k = 0; k < TAPS; ++k) w[k] = load_vec<V>(a.conv_w + static_cast<long long>(k) * ch + c);
   }
-  int t_end = r0;                  // end of the current sequence
-  int t0 = 0, slot = 0;
-  bool fresh = false;
-  for (int t = r0; t < r1; ++t) {
-    if (t >= t_end) {
-      const int s = a.seq_of(t);
-      t0 = a.first_of(s);
-      t_end = a.end_of(s);
-      slot = a.state_slots[s];
-      fresh = a.positions[t0] == 0;
-      if constexpr (TAPS > 1) {
+  for (int t = r0; t < r1;) {      // a sequence's part of the run
+    const int s = a.seq_of(t), t0 = a.first_of(s), t_end = min(r1, a.end_of(s)), slot = a.state_slots[s];
+    const bool fresh = a.positions[t0] == 0;
+    if constexpr (TAPS > 1) {
 #pragma unroll
-        for (int k = 1; k < TAPS; ++k) hist[k - 1] = conv_input<V>(a, c, t, k, t0, slot, fresh);
+      for (int k = 1; k < TAPS; ++k) hist[k - 1] = conv_input<V>(a, c, t, k, t0, slot, fresh);
+    }
+    for (; t < t_end; t += kConvAhead) {
+      Vec<V> x[kConvAhead];
+#pragma unroll
+      for (int j = 0; j < kConvAhead; ++j) {
+        const float* p = in + static_cast<long long>(min(t + j, t_end - 1)) * a.ld;
+        x[j] = ONE ? load_vec<V>(p) : slab_sum_vec<V>(p, a.n_partials, a.pstride);
+      }
+#pragma unroll
+      for (int j = 0; j < kConvAhead; ++j) {
+        if (t + j >= t_end) break;
+        Vec<V> y = bias;
+        if constexpr (TAPS > 0) {
+#pragma unroll
+          for (int i = 0; i < V; ++i) {
+#pragma unroll
+            for (int k = TAPS - 1; k > 0; --k) y.x[i] = fmaf(w[TAPS - 1 - k].x[i], hist[k - 1].x[i], y.x[i]);
+            y.x[i] = fmaf(w[TAPS - 1].x[i], x[j].x[i], y.x[i]);
+          }
+#pragma unroll
+          for (int k = TAPS - 1; k > 1; --k) hist[k - 1] = hist[k - 2];
+          if constexpr (TAPS > 1) hist[0] = x[j];
+        } else {
+          for (int k = a.taps - 1; k >= 0; --k) {
+            const Vec<V> xk = k ? conv_input<V>(a, c, t + j, k, t0, slot, fresh) : x[j];
+            const Vec<V> wk = load_vec<V>(a.conv_w + static_cast<long long>(a.taps - 1 - k) * ch + c);
+#pragma unroll
+            for (int i = 0; i < V; ++i) y.x[i] = fmaf(wk.x[i], xk.x[i], y.x[i]);
+          }
+        }
+#pragma unroll
+        for (int i = 0; i < V; ++i) y.x[i] = silu_f32(y.x[i]);
+        store_vec<V>(out + static_cast<long long>(t + j) * x_ld, y);
       }
     }
-    Vec<V> x = conv_input<V>(a, c, t, 0, t0, slot, fresh), y = bias;
-    if constexpr (TAPS > 0) {
-#pragma unroll
-      for (int i = 0; i < V; ++i) {
-#pragma unroll
-        for (int k = TAPS - 1; k > 0; --k) y.x[i] = fmaf(w[TAPS - 1 - k].x[i], hist[k - 1].x[i], y.x[i]);
-        y.x[i] = fmaf(w[TAPS - 1].x[i], x.x[i], y.x[i]);
-      }
-#pragma unroll
-      for (int k = TAPS - 1; k > 1; --k) hist[k - 1] = hist[k - 2];
-      if constexpr (TAPS > 1) hist[0] = x;
-    } else {
-      for (int k = a.taps - 1; k >= 0; --k) {
-        const Vec<V> in = k ? conv_input<V>(a, c, t, k, t0, slot, fresh) : x;
-        const Vec<V> wk = load_vec<V>(a.conv_w + static_cast<long long>(a.taps - 1 - k) * ch + c);
-#pragma unroll
-        for (int i = 0; i < V; ++i) y.x[i] = fmaf(wk.x[i], in.x[i], y.x[i]);
-      }
-    }
-#pragma unroll
-    for (int i = 0; i < V; ++i) y.x[i] = silu_f32(y.x[i]);
-    store_vec<V>(out + static_cast<long long>(t) * a.x_ld(), y);
+    t = t_end;
   }
 }
 
-template <typename T, int V>
+template <typename T, int V, bool ONE>
 static int launch_conv(const SsmArgs& a, cudaStream_t st) {
-  const int run = a.n_tokens <= 256 ? 1 : a.n_tokens <= 4096 ? 8 : 16;
+  const int run = a.n_tokens <= 256 ? 1 : a.n_tokens <= 4096 ? 8 : 32;
   const int blocks = (a.channels() / V + kConvThreads - 1) / kConvThreads;
   const dim3 grid(blocks + (a.heads + kConvThreads - 1) / kConvThreads, (a.n_tokens + run - 1) / run);
   switch (a.taps) {
-    case 2: BCG_CUDA_CHECK(launch_k(ssm_conv_kernel<T, V, 2>, grid, dim3(kConvThreads), 0, st, a, run, blocks)); break;
-    case 3: BCG_CUDA_CHECK(launch_k(ssm_conv_kernel<T, V, 3>, grid, dim3(kConvThreads), 0, st, a, run, blocks)); break;
-    case 4: BCG_CUDA_CHECK(launch_k(ssm_conv_kernel<T, V, 4>, grid, dim3(kConvThreads), 0, st, a, run, blocks)); break;
-    default: BCG_CUDA_CHECK(launch_k(ssm_conv_kernel<T, V, 0>, grid, dim3(kConvThreads), 0, st, a, run, blocks));
+    case 2: BCG_CUDA_CHECK(launch_k(ssm_conv_kernel<T, V, 2, ONE>, grid, dim3(kConvThreads), 0, st, a, run, blocks)); break;
+    case 3: BCG_CUDA_CHECK(launch_k(ssm_conv_kernel<T, V, 3, ONE>, grid, dim3(kConvThreads), 0, st, a, run, blocks)); break;
+    case 4: BCG_CUDA_CHECK(launch_k(ssm_conv_kernel<T, V, 4, ONE>, grid, dim3(kConvThreads), 0, st, a, run, blocks)); break;
+    default: BCG_CUDA_CHECK(launch_k(ssm_conv_kernel<T, V, 0, ONE>, grid, dim3(kConvThreads), 0, st, a, run, blocks));
   }
   return BCG_OK;
+}
+
+// The convolution's state of channel c behind the last token of sequence s: row r <- input n + r - (taps - 1) of the
+// portion of n tokens, or old row n + r.
+__device__ __forceinline__ void advance_conv(const SsmArgs& a, int s, int t0, int t1, bool fresh, int c) {
+  const int keep = a.taps - 1, n = t1 - t0, ch = a.channels();
+  float* cs = a.conv_state + static_cast<long long>(a.state_slots[s]) * keep * ch + c;
+  for (int r = 0; r < keep; ++r) {
+    const int i = n + r - keep;
+    float x = 0.f;
+    if (i >= 0) x = slab_sum(a.row(t0 + i) + a.inner() + c, a.n_partials, a.pstride);
+    else if (!fresh) x = cs[static_cast<long long>(n + r) * ch];
+    cs[static_cast<long long>(r) * ch] = x;
+  }
+}
+// The channels that the CTA of head h and entries p0.. is in charge of: its own x, and its group's B and C where the head
+// is the group's first.
+__device__ __forceinline__ void advance_conv_of_head(const SsmArgs& a, int s, int t0, int t1, bool fresh, int h, int p0, int rows) {
+  const int per = a.heads / a.groups, g = h / per;
+  const int n = rows + (h % per == 0 && p0 == 0 ? 2 * a.n : 0);
+  for (int i = threadIdx.x; i < n; i += blockDim.x) {
+    const int e = i - rows;
+    advance_conv(a, s, t0, t1, fresh, i < rows ? h * a.vdim + p0 + i : a.inner() + (e / a.n * a.groups + g) * a.n + e % a.n);
+  }
 }
 
 // ------------------------------------------------------------------------------------------- state in registers
@@ -236,66 +270,94 @@ struct StateRows {
   }
 };
 
+constexpr int kTapsAhead = 4;     // taps whose past inputs are requested before the dependency wait
+
 template <typename T, int NP>
-__global__ void __launch_bounds__(kSsThreads)
+__global__ void __launch_bounds__(kSsThreads, NP <= 128 ? 3 : 2)
 ssm_token_kernel(const SsmArgs a) {
   using S = StateRows<NP>;
-  __shared__ float xs[kSsRows], zs[kSsRows], bs[NP], cs[NP], step_s;
+  constexpr int kItems = (kSsRows + 2 * NP + 1 + kSsThreads - 1) / kSsThreads;
+  __shared__ float xbc[kSsRows + 2 * NP], step_s;
   const int h = blockIdx.x, p0 = blockIdx.y * kSsRows, t = blockIdx.z;
-  const int rows = min(kSsRows, a.vdim - p0), N = a.n, g = h / (a.heads / a.groups), inner = a.inner();
+  const int rows = min(kSsRows, a.vdim - p0), N = a.n, g = h / (a.heads / a.groups), inner = a.inner(), ch = a.channels();
   pdl_launch_dependents();
   // Positions, slots and states were written by earlier steps, which are complete before any kernel of this step
-  // starts, so the state is on its way while the projections are finished.
+  // starts, so the states are on their way while the projections are finished.
   const bool idle = a.slot_map[t] < 0, fresh = a.positions[t] == 0;
   const int slot = a.state_slots[t];
   float* st = a.state + ((static_cast<long long>(slot) * a.heads + h) * a.vdim + p0) * N;
+  // items: x of the CTA's rows, B, C, the step; channel -1: padding, -2: the step
+  int chan[kItems];
+  float past[kItems][kTapsAhead - 1];
+  const float* cs = a.conv_state + static_cast<long long>(slot) * (a.taps - 1) * ch;
+#pragma unroll
+  for (int k = 0; k < kItems; ++k) {
+    const int i = threadIdx.x + k * kSsThreads, e = i - kSsRows;
+    chan[k] = -1;
+    if (i < rows) chan[k] = h * a.vdim + p0 + i;
+    else if (e >= 0 && e < 2 * NP && e % NP < N) chan[k] = inner + (e / NP * a.groups + g) * N + e % NP;
+    else if (e == 2 * NP) chan[k] = -2;
+#pragma unroll
+    for (int j = 0; j < kTapsAhead - 1; ++j)
+      past[k][j] = chan[k] >= 0 && !idle && !fresh && j < a.taps - 1 ? cs[static_cast<long long>(j) * ch + chan[k]] : 0.f;
+  }
   S s;
   if (idle || fresh) s.zero();
   else s.load(st, rows, N);
   pdl_wait();
   if (idle) return;
-  const float* row = a.row(t);
-  // x, B, C through the convolution; z; the step
-  for (int i = threadIdx.x; i < 2 * kSsRows + 2 * NP + 1; i += kSsThreads) {
-    if (i < kSsRows) {
-      if (i < rows) zs[i] = silu_f32(slab_sum(row + h * a.vdim + p0 + i, a.n_partials, a.pstride));
-      continue;
+  float in[kItems];
+#pragma unroll
+  for (int k = 0; k < kItems; ++k) in[k] = 0.f;
+  for (int p = 0; p < a.n_partials; p += 4) {       // slabs in index order, four per item in flight
+    float v[kItems][4];
+#pragma unroll
+    for (int k = 0; k < kItems; ++k) {
+      const float* src = a.row(t) + inner + (chan[k] == -2 ? ch + h : max(chan[k], 0));
+#pragma unroll
+      for (int q = 0; q < 4; ++q) v[k][q] = p + q < a.n_partials ? src[(p + q) * a.pstride] : 0.f;
     }
-    if (i == 2 * kSsRows + 2 * NP) {
-      step_s = softplus_f32(slab_sum(row + inner + a.channels() + h, a.n_partials, a.pstride) + a.step_bias[h]);
-      continue;
-    }
-    const int e = i - kSsRows;
-    const int kind = e < kSsRows ? 0 : e < kSsRows + NP ? 1 : 2, k0 = kind == 0 ? e : kind == 1 ? e - kSsRows : e - kSsRows - NP;
+#pragma unroll
+    for (int k = 0; k < kItems; ++k)
+#pragma unroll
+      for (int q = 0; q < 4; ++q) in[k] += v[k][q];
+  }
+#pragma unroll
+  for (int k = 0; k < kItems; ++k) {
+    const int i = threadIdx.x + k * kSsThreads, c = chan[k];
     float y = 0.f;
-    if (k0 < (kind == 0 ? rows : N)) {
-      const int c = kind == 0 ? h * a.vdim + p0 + k0 : inner + ((kind - 1) * a.groups + g) * N + k0, ch = a.channels();
-      y = fmaf(a.conv_w[static_cast<long long>(a.taps - 1) * ch + c], slab_sum(row + inner + c, a.n_partials, a.pstride), a.conv_b[c]);
+    if (c >= 0) {
+      const float* w = a.conv_w + c;
+      y = fmaf(w[static_cast<long long>(a.taps - 1) * ch], in[k], a.conv_b[c]);
+#pragma unroll
+      for (int j = 0; j < kTapsAhead - 1; ++j)
+        if (j < a.taps - 1) y = fmaf(w[static_cast<long long>(j) * ch], past[k][j], y);
       if (!fresh)
-        for (int k = 0; k < a.taps - 1; ++k)
-          y = fmaf(a.conv_w[static_cast<long long>(k) * ch + c], a.conv_state[(static_cast<long long>(slot) * (a.taps - 1) + k) * ch + c], y);
+        for (int j = kTapsAhead - 1; j < a.taps - 1; ++j)
+          y = fmaf(w[static_cast<long long>(j) * ch], cs[static_cast<long long>(j) * ch + c], y);
       y = silu_f32(y);
+    } else if (c == -2) {
+      step_s = softplus_f32(in[k] + a.step_bias[h]);
     }
-    (kind == 0 ? xs : kind == 1 ? bs : cs)[k0] = y;
+    if (i < kSsRows + 2 * NP) xbc[i] = y;
   }
   __syncthreads();
   const float step = step_s, keep = decay_f32(-a.rate[h] * step);
   float v[S::kR], b[S::kQ][4], c[S::kQ][4];
 #pragma unroll
-  for (int r = 0; r < S::kR; ++r) v[r] = S::row(r) < rows ? step * xs[S::row(r)] : 0.f;
+  for (int r = 0; r < S::kR; ++r) v[r] = step * xbc[S::row(r)];
 #pragma unroll
   for (int q = 0; q < S::kQ; ++q)
 #pragma unroll
     for (int i = 0; i < 4; ++i) {
-      b[q][i] = bs[S::entry(q) + i];
-      c[q][i] = cs[S::entry(q) + i];
+      b[q][i] = xbc[kSsRows + S::entry(q) + i];
+      c[q][i] = xbc[kSsRows + NP + S::entry(q) + i];
     }
   const float y = s.token(keep, v, b, c);
   s.store(st, rows, N);
   if (S::lane() < S::kR) {
     const int p = S::row(S::lane());
-    if (p < rows)
-      static_cast<T*>(a.y)[static_cast<long long>(t) * inner + h * a.vdim + p0 + p] = from_f32<T>(fmaf(a.skip[h], xs[p], y) * zs[p]);
+    if (p < rows) static_cast<T*>(a.y)[static_cast<long long>(t) * inner + h * a.vdim + p0 + p] = from_f32<T>(fmaf(a.skip[h], xbc[p], y));
   }
 }
 
@@ -312,7 +374,8 @@ ssm_scan_kernel(const SsmArgs a) {
   if (t1 <= t0 || a.slot_map[t0] < 0) return;
   float* st = a.state + ((static_cast<long long>(a.state_slots[sq]) * a.heads + h) * a.vdim + p0) * N;
   S s;
-  if (a.positions[t0] == 0) s.zero();
+  const bool fresh = a.positions[t0] == 0;
+  if (fresh) s.zero();
   else s.load(st, rows, N);
   const T* base = static_cast<const T*>(a.x);
   const float rate = a.rate[h], skip = a.skip[h];
@@ -351,13 +414,11 @@ ssm_scan_kernel(const SsmArgs a) {
     const float y = s.token(keep, v, bb, cc);
     if (S::lane() < S::kR) {
       const int p = S::row(S::lane());
-      if (p < rows) {
-        const float z = slab_sum(a.row(t) + h * a.vdim + p0 + p, a.n_partials, a.pstride);
-        static_cast<T*>(a.y)[static_cast<long long>(t) * inner + h * a.vdim + p0 + p] = from_f32<T>(fmaf(skip, mine, y) * silu_f32(z));
-      }
+      if (p < rows) static_cast<T*>(a.y)[static_cast<long long>(t) * inner + h * a.vdim + p0 + p] = from_f32<T>(fmaf(skip, mine, y));
     }
   }
   s.store(st, rows, N);
+  advance_conv_of_head(a, sq, t0, t1, fresh, h, p0, rows);
 }
 
 // ------------------------------------------------------------------------------------------- chunks
@@ -367,8 +428,8 @@ template <int NP>
 struct ChCfg {
   static constexpr int kBRow = NP + 8, kXRow = kSsRows + 8, kMRow = kChTok + 8;       // pitches, bf16
   static constexpr int kBC = kChTok * kBRow, kX = kChTok * kXRow, kM = kChTok * kMRow;
-  static constexpr int kBuf = 2 * kBC + kX;                                             // B, C, x of a chunk
-  static constexpr int kSmem = (2 * kBuf + 2 * kM) * 2 + 2 * 4 * kChTok * 4;            // two chunks, M hi / lo, scalars
+  static constexpr int kSmem = (2 * kBC + kX + 2 * kM) * 2 + 2 * 4 * kChTok * 4;        // B, C, x, M hi / lo, scalars
+  static constexpr int kCtasPerSm = NP <= 128 ? 3 : 2;
 };
 
 // hi + lo = v to about 2^-17
@@ -382,14 +443,60 @@ __device__ __forceinline__ uint32_t transpose_8x8(uint32_t v) {
   return r;
 }
 
+// M[i][j] = exp(c_i - c_j) step_j (C_i . B_j) for j <= i, tokens i = 16 RT .. 16 RT + 15, as two bf16 halves.
+template <int NP, int RT>
+__device__ __forceinline__ void chunk_matrix(const __nv_bfloat16* sB, const __nv_bfloat16* sC, const float* sum2,
+                                             const float* steps, __nv_bfloat16* m_hi, __nv_bfloat16* m_lo) {
+  using C = ChCfg<NP>;
+  const int lane = threadIdx.x & 31, q2 = (lane & 3) * 2;
+  float acc[2 * RT + 2][4] = {};
+  const __nv_bfloat16* pc = sC + (RT * 16 + (lane & 15)) * C::kBRow + (lane >> 4) * 8;
+  const __nv_bfloat16* pb = sB + ((lane & 7) + ((lane >> 4) << 3)) * C::kBRow + ((lane >> 3) & 1) * 8;
+#pragma unroll
+  for (int k = 0; k < NP / 16; ++k) {
+    uint32_t ca[4];
+    ldsm_x4(ca, pc + k * 16);
+#pragma unroll
+    for (int jp = 0; jp <= RT; ++jp) {
+      uint32_t bb[4];
+      ldsm_x4(bb, pb + jp * 16 * C::kBRow + k * 16);
+      mma_bf16_16816(acc[2 * jp], ca, bb[0], bb[1]);
+      mma_bf16_16816(acc[2 * jp + 1], ca, bb[2], bb[3]);
+    }
+  }
+  const int i0 = RT * 16 + (lane >> 2);
+  const float ci[2] = {sum2[i0], sum2[i0 + 8]};
+#pragma unroll
+  for (int jt = 0; jt < 2 * RT + 2; ++jt) {
+    const int j = jt * 8 + q2;
+    const float2 cj = *reinterpret_cast<const float2*>(sum2 + j), sj = *reinterpret_cast<const float2*>(steps + j);
+#pragma unroll
+    for (int e = 0; e < 2; ++e) {
+      const int i = i0 + e * 8;
+      float m0 = acc[jt][2 * e] * (ex2_approx(ci[e] - cj.x) * sj.x);
+      float m1 = acc[jt][2 * e + 1] * (ex2_approx(ci[e] - cj.y) * sj.y);
+      if (jt >= 2 * RT) {                       // the diagonal block
+        if (j > i) m0 = 0.f;
+        if (j + 1 > i) m1 = 0.f;
+      }
+      uint32_t hi, lo;
+      split_bf16(m0, m1, hi, lo);
+      *reinterpret_cast<uint32_t*>(m_hi + i * C::kMRow + j) = hi;
+      *reinterpret_cast<uint32_t*>(m_lo + i * C::kMRow + j) = lo;
+    }
+  }
+}
+
 // grid (heads, blocks of 64 head entries, sequences); warp w has entries 16 w .. 16 w + 15 of the block.
 template <int NP>
-__global__ void __launch_bounds__(kChThreads, NP <= 128 ? 2 : 1)
+__global__ void __launch_bounds__(kChThreads, ChCfg<NP>::kCtasPerSm)
 ssm_chunk_kernel(const SsmArgs a) {
   using C = ChCfg<NP>;
   extern __shared__ __align__(16) uint8_t ch_raw[];
-  __nv_bfloat16* bufs = reinterpret_cast<__nv_bfloat16*>(ch_raw);
-  __nv_bfloat16* m_hi = bufs + 2 * C::kBuf;
+  __nv_bfloat16* sB = reinterpret_cast<__nv_bfloat16*>(ch_raw);
+  __nv_bfloat16* sC = sB + C::kBC;
+  __nv_bfloat16* sX = sC + C::kBC;
+  __nv_bfloat16* m_hi = sX + C::kX;
   __nv_bfloat16* m_lo = m_hi + C::kM;
   float* scalars = reinterpret_cast<float*>(m_lo + C::kM);     // [2][4][64]: log2 decay sums, steps, e, w
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, n_warps = blockDim.x >> 5;
@@ -401,9 +508,9 @@ ssm_chunk_kernel(const SsmArgs a) {
   if (t1 <= t0 || a.slot_map[t0] < 0) return;
   const float rate = a.rate[h], skip = a.skip[h];
   const __nv_bfloat16* xbc = static_cast<const __nv_bfloat16*>(a.x);
-  const int x_ld = a.x_ld(), xc = h * a.x_pad() + p0, bc = a.b_col(g), cc = a.c_col(g);
+  const int x_ld = a.x_ld();
 
-  // B, C and x of a chunk; columns and tokens past the end are zero
+  // 64 tokens from `first` on, `valid` columns from `col` on; columns and tokens past the end are zero
   auto copy_rows = [&](__nv_bfloat16* dst, int pitch, int col, int valid, int units, int first) {
     for (int i = threadIdx.x; i < kChTok * units; i += blockDim.x) {
       const int r = i / units, u = i - r * units;
@@ -413,19 +520,16 @@ ssm_chunk_kernel(const SsmArgs a) {
                    : "memory");
     }
   };
-  auto fetch = [&](int c) {
-    __nv_bfloat16* b = bufs + (c & 1) * C::kBuf;
-    copy_rows(b, C::kBRow, bc, N, NP / 8, t0 + c * kChTok);
-    copy_rows(b + C::kBC, C::kBRow, cc, N, NP / 8, t0 + c * kChTok);
-    copy_rows(b + 2 * C::kBC, C::kXRow, xc, rows, kSsRows / 8, t0 + c * kChTok);
-    cp_async_commit();
-  };
   auto step_at = [&](int t) { return t < t1 ? a.step[static_cast<long long>(t) * a.heads + h] : 0.f; };
 
   const int n_chunks = (t1 - t0 + kChTok - 1) / kChTok;
   const int pr = warp * 16 + (lane >> 2);       // this lane's rows of the state: pr, pr + 8; entries nt * 8 + 2 (lane & 3) ..
   const int q2 = (lane & 3) * 2;
   float* st = a.state + ((static_cast<long long>(a.state_slots[sq]) * a.heads + h) * a.vdim + p0) * N;
+  copy_rows(sB, C::kBRow, a.b_col(g), N, NP / 8, t0);
+  copy_rows(sC, C::kBRow, a.c_col(g), N, NP / 8, t0);
+  copy_rows(sX, C::kXRow, h * a.x_pad() + p0, rows, kSsRows / 8, t0);
+  cp_async_commit();
   float S[NP / 8][4];
   const bool fresh = a.positions[t0] == 0;
 #pragma unroll
@@ -435,7 +539,6 @@ ssm_chunk_kernel(const SsmArgs a) {
       const int p = pr + (i >> 1) * 8, n = nt * 8 + q2 + (i & 1);
       S[nt][i] = !fresh && p < rows && n < N ? st[static_cast<long long>(p) * N + n] : 0.f;
     }
-  fetch(0);
   float s0 = 0.f, s1 = 0.f;                     // warp 0: steps of tokens 2 lane, 2 lane + 1 of the next chunk
   if (warp == 0) {
     s0 = step_at(t0 + 2 * lane);
@@ -444,9 +547,6 @@ ssm_chunk_kernel(const SsmArgs a) {
 
   for (int c = 0; c < n_chunks; ++c) {
     const int first = t0 + c * kChTok, nt_tok = min(kChTok, t1 - first);
-    const __nv_bfloat16* sB = bufs + (c & 1) * C::kBuf;
-    const __nv_bfloat16* sC = sB + C::kBC;
-    const __nv_bfloat16* sX = sC + C::kBC;
     float* sum2 = scalars + (c & 1) * 4 * kChTok;
     float *steps = sum2 + kChTok, *e_s = steps + kChTok, *w_s = e_s + kChTok;
     if (warp == 0) {
@@ -471,63 +571,31 @@ ssm_chunk_kernel(const SsmArgs a) {
       s1 = step_at(first + kChTok + 2 * lane + 1);
     }
     cp_async_wait<0>();
-    __syncthreads();                            // the chunk is there; everybody is done with the previous one
-    if (c + 1 < n_chunks) fetch(c + 1);
+    __syncthreads();                            // the chunk is there
 
-    // ---- M[i][j] = exp(c_i - c_j) step_j (C_i . B_j) for j <= i, 16 tokens i per turn
     for (int rt = warp; rt * 16 < nt_tok; rt += n_warps) {
-      float acc[kChTok / 8][4] = {};
-#pragma unroll
-      for (int k = 0; k < NP / 16; ++k) {
-        uint32_t ca[4];
-        ldsm_x4(ca, sC + (rt * 16 + (lane & 15)) * C::kBRow + k * 16 + (lane >> 4) * 8);
-#pragma unroll
-        for (int jp = 0; jp < kChTok / 16; ++jp)
-          if (jp <= rt) {
-            uint32_t bb[4];
-            ldsm_x4(bb, sB + (jp * 16 + (lane & 7) + ((lane >> 4) << 3)) * C::kBRow + k * 16 + ((lane >> 3) & 1) * 8);
-            mma_bf16_16816(acc[2 * jp], ca, bb[0], bb[1]);
-            mma_bf16_16816(acc[2 * jp + 1], ca, bb[2], bb[3]);
-          }
-      }
-      const int i0 = rt * 16 + (lane >> 2);
-      const float ci[2] = {sum2[i0], sum2[i0 + 8]};
-#pragma unroll
-      for (int jt = 0; jt < kChTok / 8; ++jt)
-        if (jt <= 2 * rt + 1) {
-          const int j = jt * 8 + q2;
-          const float2 cj = *reinterpret_cast<const float2*>(sum2 + j), sj = *reinterpret_cast<const float2*>(steps + j);
-#pragma unroll
-          for (int e = 0; e < 2; ++e) {
-            const int i = i0 + e * 8;
-            const float m0 = j <= i ? acc[jt][2 * e] * (ex2_approx(ci[e] - cj.x) * sj.x) : 0.f;
-            const float m1 = j + 1 <= i ? acc[jt][2 * e + 1] * (ex2_approx(ci[e] - cj.y) * sj.y) : 0.f;
-            uint32_t hi, lo;
-            split_bf16(m0, m1, hi, lo);
-            *reinterpret_cast<uint32_t*>(m_hi + i * C::kMRow + j) = hi;
-            *reinterpret_cast<uint32_t*>(m_lo + i * C::kMRow + j) = lo;
-          }
-        }
+      if (rt == 0) chunk_matrix<NP, 0>(sB, sC, sum2, steps, m_hi, m_lo);
+      else if (rt == 1) chunk_matrix<NP, 1>(sB, sC, sum2, steps, m_hi, m_lo);
+      else if (rt == 2) chunk_matrix<NP, 2>(sB, sC, sum2, steps, m_hi, m_lo);
+      else chunk_matrix<NP, 3>(sB, sC, sum2, steps, m_hi, m_lo);
     }
 
     // ---- Y^T = S^T C^T, columns (tokens) scaled by exp(c_i)
     float Y[kChTok / 8][4] = {};
+    const __nv_bfloat16* pc = sC + ((lane & 7) + ((lane >> 4) << 3)) * C::kBRow + ((lane >> 3) & 1) * 8;
 #pragma unroll
     for (int k = 0; k < NP / 16; ++k) {
-      uint32_t hi[4], lo[4];
+      uint32_t hi[4], lo[4], cb[kChTok / 16][4];
+#pragma unroll
+      for (int ip = 0; ip < kChTok / 16; ++ip) ldsm_x4(cb[ip], pc + ip * 16 * C::kBRow + k * 16);
       split_bf16(S[2 * k][0], S[2 * k][1], hi[0], lo[0]);
       split_bf16(S[2 * k][2], S[2 * k][3], hi[1], lo[1]);
       split_bf16(S[2 * k + 1][0], S[2 * k + 1][1], hi[2], lo[2]);
       split_bf16(S[2 * k + 1][2], S[2 * k + 1][3], hi[3], lo[3]);
 #pragma unroll
-      for (int ip = 0; ip < kChTok / 16; ++ip) {
-        uint32_t cb[4];
-        ldsm_x4(cb, sC + (ip * 16 + (lane & 7) + ((lane >> 4) << 3)) * C::kBRow + k * 16 + ((lane >> 3) & 1) * 8);
-        mma_bf16_16816(Y[2 * ip], hi, cb[0], cb[1]);
-        mma_bf16_16816(Y[2 * ip + 1], hi, cb[2], cb[3]);
-        mma_bf16_16816(Y[2 * ip], lo, cb[0], cb[1]);
-        mma_bf16_16816(Y[2 * ip + 1], lo, cb[2], cb[3]);
-      }
+      for (int it = 0; it < kChTok / 8; ++it) mma_bf16_16816(Y[it], hi, cb[it >> 1][(it & 1) * 2], cb[it >> 1][(it & 1) * 2 + 1]);
+#pragma unroll
+      for (int it = 0; it < kChTok / 8; ++it) mma_bf16_16816(Y[it], lo, cb[it >> 1][(it & 1) * 2], cb[it >> 1][(it & 1) * 2 + 1]);
     }
 #pragma unroll
     for (int it = 0; it < kChTok / 8; ++it) {
@@ -542,24 +610,27 @@ ssm_chunk_kernel(const SsmArgs a) {
     for (int nt = 0; nt < NP / 8; ++nt)
 #pragma unroll
       for (int i = 0; i < 4; ++i) S[nt][i] *= keep;
-    __syncthreads();                            // M is complete
+    __syncthreads();                            // M is complete, C has been read
+    if (c + 1 < n_chunks) copy_rows(sC, C::kBRow, a.c_col(g), N, NP / 8, first + kChTok);
 
     // ---- Y^T += x^T M^T + skip x^T;   S^T += (w x)^T B
+    const __nv_bfloat16* px = sX + ((lane & 7) + ((lane >> 4) << 3)) * C::kXRow + warp * 16 + ((lane >> 3) & 1) * 8;
+    const __nv_bfloat16* pb = sB + (lane & 15) * C::kBRow + (lane >> 4) * 8;
+    const int pm = ((lane & 7) + ((lane >> 4) << 3)) * C::kMRow + ((lane >> 3) & 1) * 8;
 #pragma unroll
     for (int jp = 0; jp < kChTok / 16; ++jp) {
       uint32_t xa[4];
-      ldsm_x4_trans(xa, sX + (jp * 16 + (lane & 7) + ((lane >> 4) << 3)) * C::kXRow + warp * 16 + ((lane >> 3) & 1) * 8);
+      ldsm_x4_trans(xa, px + jp * 16 * C::kXRow);
 #pragma unroll
       for (int ip = jp; ip < kChTok / 16; ++ip)
         if (ip * 16 < nt_tok) {
-          uint32_t mb[4];
-          const int at = (ip * 16 + (lane & 7) + ((lane >> 4) << 3)) * C::kMRow + jp * 16 + ((lane >> 3) & 1) * 8;
-          ldsm_x4(mb, m_hi + at);
-          mma_bf16_16816(Y[2 * ip], xa, mb[0], mb[1]);
-          mma_bf16_16816(Y[2 * ip + 1], xa, mb[2], mb[3]);
-          ldsm_x4(mb, m_lo + at);
-          mma_bf16_16816(Y[2 * ip], xa, mb[0], mb[1]);
-          mma_bf16_16816(Y[2 * ip + 1], xa, mb[2], mb[3]);
+          uint32_t mh[4], ml[4];
+          ldsm_x4(mh, m_hi + pm + ip * 16 * C::kMRow + jp * 16);
+          ldsm_x4(ml, m_lo + pm + ip * 16 * C::kMRow + jp * 16);
+          mma_bf16_16816(Y[2 * ip], xa, mh[0], mh[1]);
+          mma_bf16_16816(Y[2 * ip + 1], xa, mh[2], mh[3]);
+          mma_bf16_16816(Y[2 * ip], xa, ml[0], ml[1]);
+          mma_bf16_16816(Y[2 * ip + 1], xa, ml[2], ml[3]);
         }
       float xf[4][2];                           // rows pr, pr + 8 of tokens j, j + 1; the same of tokens j + 8, j + 9
 #pragma unroll
@@ -581,32 +652,35 @@ ssm_chunk_kernel(const SsmArgs a) {
       split_bf16(w1.x * xf[2][0], w1.y * xf[2][1], hi[2], lo[2]);
       split_bf16(w1.x * xf[3][0], w1.y * xf[3][1], hi[3], lo[3]);
 #pragma unroll
-      for (int np = 0; np < NP / 16; ++np) {
-        uint32_t bb[4];
-        ldsm_x4_trans(bb, sB + (jp * 16 + (lane & 15)) * C::kBRow + np * 16 + (lane >> 4) * 8);
-        mma_bf16_16816(S[2 * np], hi, bb[0], bb[1]);
-        mma_bf16_16816(S[2 * np + 1], hi, bb[2], bb[3]);
-        mma_bf16_16816(S[2 * np], lo, bb[0], bb[1]);
-        mma_bf16_16816(S[2 * np + 1], lo, bb[2], bb[3]);
+      for (int np = 0; np < NP / 16; np += 2) {
+        uint32_t b0[4], b1[4];
+        ldsm_x4_trans(b0, pb + jp * 16 * C::kBRow + np * 16);
+        ldsm_x4_trans(b1, pb + jp * 16 * C::kBRow + np * 16 + 16);
+        mma_bf16_16816(S[2 * np], hi, b0[0], b0[1]);
+        mma_bf16_16816(S[2 * np + 1], hi, b0[2], b0[3]);
+        mma_bf16_16816(S[2 * np + 2], hi, b1[0], b1[1]);
+        mma_bf16_16816(S[2 * np + 3], hi, b1[2], b1[3]);
+        mma_bf16_16816(S[2 * np], lo, b0[0], b0[1]);
+        mma_bf16_16816(S[2 * np + 1], lo, b0[2], b0[3]);
+        mma_bf16_16816(S[2 * np + 2], lo, b1[0], b1[1]);
+        mma_bf16_16816(S[2 * np + 3], lo, b1[2], b1[3]);
       }
     }
+    __syncthreads();                            // B and x have been read
+    if (c + 1 < n_chunks) {
+      copy_rows(sB, C::kBRow, a.b_col(g), N, NP / 8, first + kChTok);
+      copy_rows(sX, C::kXRow, h * a.x_pad() + p0, rows, kSsRows / 8, first + kChTok);
+      cp_async_commit();
+    }
 
-    // ---- gate and store: z is read where the outputs are, pairs are transposed on the way out
+    // ---- store: pairs are transposed on the way out
     __nv_bfloat16* out = static_cast<__nv_bfloat16*>(a.y) + static_cast<long long>(first) * inner + h * a.vdim + p0;
 #pragma unroll
     for (int it = 0; it < kChTok / 8; ++it) {
       if (it * 8 >= nt_tok) break;
-      float u[4];
-#pragma unroll
-      for (int i = 0; i < 4; ++i) {
-        const int tok = it * 8 + q2 + (i & 1), p = pr + (i >> 1) * 8;
-        float z = 0.f;
-        if (tok < nt_tok && p < rows) z = slab_sum(a.row(first + tok) + h * a.vdim + p0 + p, a.n_partials, a.pstride);
-        u[i] = Y[it][i] * silu_f32(z);
-      }
 #pragma unroll
       for (int e = 0; e < 2; ++e) {
-        const uint32_t v = transpose_8x8(pack_bf16(u[2 * e], u[2 * e + 1]));     // token lane >> 2, entries q2, q2 + 1
+        const uint32_t v = transpose_8x8(pack_bf16(Y[it][2 * e], Y[it][2 * e + 1]));     // token lane >> 2, entries q2, q2 + 1
         const int tok = it * 8 + (lane >> 2), p = warp * 16 + e * 8 + q2;
         __nv_bfloat16* dst = out + static_cast<long long>(tok) * inner + p;
         if (tok < nt_tok && p + 1 < rows && (a.vdim & 1) == 0) {
@@ -626,16 +700,18 @@ ssm_chunk_kernel(const SsmArgs a) {
       const int p = pr + (i >> 1) * 8, n = nt * 8 + q2 + (i & 1);
       if (p < rows && n < N) st[static_cast<long long>(p) * N + n] = S[nt][i];
     }
+  advance_conv_of_head(a, sq, t0, t1, fresh, h, p0, rows);
 }
 
 // ------------------------------------------------------------------------------------------- norm
 constexpr int kSnThreads = 256;
 
-// A part of a token's outputs per CTA, or per cluster of CL.  The CTAs of a sequence's last token also move the
-// convolution's state on.
-template <typename T, int V, int CL>
+// A part of a token's outputs per CTA, or per cluster of CL.  ADVANCE: single tokens, the convolution's state moves on.
+template <typename T, int V, int CL, bool ADVANCE>
 __global__ void __launch_bounds__(kSnThreads)
 ssm_norm_kernel(const SsmArgs a, T* __restrict__ out, long long out_ld) {
+  extern __shared__ float4 stage_raw[];
+  float* stage = reinterpret_cast<float*>(stage_raw);
   __shared__ RowSum<kSnThreads, CL, 1> sh;
   pdl_launch_dependents();
   pdl_wait();
@@ -643,44 +719,100 @@ ssm_norm_kernel(const SsmArgs a, T* __restrict__ out, long long out_ld) {
   const int part = unit / CL, inner = a.inner(), width = inner / a.parts;
   const int per = (width / V + CL - 1) / CL * V, v0 = unit % CL * per, v1 = min(width, v0 + per);
   const T* y = static_cast<const T*>(a.y) + static_cast<long long>(t) * inner + part * width;
+  const float* z = a.row(t) + part * width;
   float ss[1] = {0.f};
-  for (int v = v0 + threadIdx.x * V; v < v1; v += kSnThreads * V) ss[0] += load_vec<V>(y + v).sumsq();
+  for (int v = v0 + threadIdx.x * V; v < v1; v += kSnThreads * V) {
+    Vec<V> u = load_vec<V>(y + v);
+    const Vec<V> g = slab_sum_vec<V>(z + v, a.n_partials, a.pstride);
+#pragma unroll
+    for (int k = 0; k < V; ++k) u.x[k] *= silu_f32(g.x[k]);
+    store_vec<V>(stage + v - v0, u);
+    ss[0] += u.sumsq();
+  }
   row_sum<kSnThreads, CL, 1>(sh, ss, 0);
   const float inv = rsqrtf(ss[0] / static_cast<float>(width) + a.eps);
   for (int v = v0 + threadIdx.x * V; v < v1; v += kSnThreads * V) {
-    Vec<V> x = load_vec<V>(y + v);
+    Vec<V> x = load_vec<V>(stage + v - v0);
     const Vec<V> w = load_vec<V>(a.norm + part * width + v);
 #pragma unroll
     for (int k = 0; k < V; ++k) x.x[k] *= inv * w.x[k];
     store_vec<V>(out + t * out_ld + part * width + v, x);
   }
-  const int s = a.seq_of(t), t0 = a.first_of(s), keep = a.taps - 1, ch = a.channels();
-  if (t == a.end_of(s) - 1 && keep > 0 && a.slot_map[t] >= 0) {
-    const bool fresh = a.positions[t0] == 0;
-    const int n = t + 1 - t0;
-    float* cs = a.conv_state + static_cast<long long>(a.state_slots[s]) * keep * ch;
-    for (int c = unit * kSnThreads + threadIdx.x; c < ch; c += a.parts * CL * kSnThreads)
-      for (int r = 0; r < keep; ++r) {          // row r <- input n + r - keep of this portion, or old row n + r
-        const int i = n + r - keep;
-        float x = 0.f;
-        if (i >= 0) x = slab_sum(a.row(t0 + i) + inner + c, a.n_partials, a.pstride);
-        else if (!fresh) x = cs[static_cast<long long>(n + r) * ch + c];
-        cs[static_cast<long long>(r) * ch + c] = x;
-      }
+  if constexpr (ADVANCE) {
+    if (a.taps > 1 && a.slot_map[t] >= 0) {
+      const int ch = a.channels();
+      const bool fresh = a.positions[t] == 0;
+      for (int c = unit * kSnThreads + threadIdx.x; c < ch; c += a.parts * CL * kSnThreads) advance_conv(a, t, t, t + 1, fresh, c);
+    }
   }
   row_sum_exit<CL>();
 }
 
-template <typename T, int V>
-static int launch_norm(const SsmArgs& a, void* out, long long out_ld, cudaStream_t st) {
-  const long long units = static_cast<long long>(a.n_tokens) * a.parts;
-  if (a.n_tokens <= 128 && a.inner() / a.parts >= 1024)
-    BCG_CUDA_CHECK(launch_cluster(ssm_norm_kernel<T, V, 8>, dim3(static_cast<unsigned>(units * 8)), dim3(kSnThreads), 8, 0, st, a,
-                                  static_cast<T*>(out), out_ld));
-  else
-    BCG_CUDA_CHECK(launch_k(ssm_norm_kernel<T, V, 1>, dim3(static_cast<unsigned>(units)), dim3(kSnThreads), 0, st, a,
-                            static_cast<T*>(out), out_ld));
+// Prompts, one slab: a part of a token's outputs per warp, NV vectors of four per lane.
+template <typename T, int NV>
+__global__ void __launch_bounds__(kSnThreads)
+ssm_norm_warp_kernel(const SsmArgs a, T* __restrict__ out, long long out_ld) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const int lane = threadIdx.x & 31;
+  const long long unit = blockIdx.x * static_cast<long long>(kSnThreads / 32) + (threadIdx.x >> 5);
+  if (unit >= static_cast<long long>(a.n_tokens) * a.parts) return;
+  const long long t = unit / a.parts;
+  const int inner = a.inner(), width = inner / a.parts, c0 = static_cast<int>(unit % a.parts) * width;
+  const T* y = static_cast<const T*>(a.y) + t * inner + c0;
+  const float* z = a.row(t) + c0;
+  Vec<4> u[NV], g[NV];
+#pragma unroll
+  for (int i = 0; i < NV; ++i) {
+    const int v = min((i * 32 + lane) * 4, width - 4);
+    u[i] = load_vec<4>(y + v);
+    g[i] = load_vec<4>(z + v);
+  }
+  float ss = 0.f;
+#pragma unroll
+  for (int i = 0; i < NV; ++i) {
+#pragma unroll
+    for (int k = 0; k < 4; ++k) u[i].x[k] *= silu_f32(g[i].x[k]);
+    if ((i * 32 + lane) * 4 < width) ss += u[i].sumsq();
+  }
+  const float inv = rsqrtf(warp_sum(ss) / static_cast<float>(width) + a.eps);
+#pragma unroll
+  for (int i = 0; i < NV; ++i) {
+    const int v = (i * 32 + lane) * 4;
+    if (v >= width) break;
+    const Vec<4> w = load_vec<4>(a.norm + c0 + v);
+#pragma unroll
+    for (int k = 0; k < 4; ++k) u[i].x[k] *= inv * w.x[k];
+    store_vec<4>(out + t * out_ld + c0 + v, u[i]);
+  }
+}
+
+template <typename T, int V, int CL, bool ADVANCE>
+static int launch_norm_cl(const SsmArgs& a, void* out, long long out_ld, cudaStream_t st) {
+  const int width = a.inner() / a.parts;
+  const dim3 grid(static_cast<unsigned>(static_cast<long long>(a.n_tokens) * a.parts * CL));
+  const size_t sm = static_cast<size_t>((width / V + CL - 1) / CL * V) * 4;
+  BCG_TRY(ensure_dynamic_smem(reinterpret_cast<const void*>(ssm_norm_kernel<T, V, CL, ADVANCE>), 200 * 1024));
+  BCG_CUDA_CHECK(launch_cluster(ssm_norm_kernel<T, V, CL, ADVANCE>, grid, dim3(kSnThreads), CL, sm, st, a, static_cast<T*>(out), out_ld));
   return BCG_OK;
+}
+
+template <typename T, int V>
+static int launch_norm(const SsmArgs& a, bool advance, void* out, long long out_ld, cudaStream_t st) {
+  const int width = a.inner() / a.parts;
+  if constexpr (V == 4) {
+    if (!advance && a.n_partials == 1 && width <= 2048 && a.n_tokens > 128) {
+      const dim3 grid(static_cast<unsigned>((static_cast<long long>(a.n_tokens) * a.parts + kSnThreads / 32 - 1) / (kSnThreads / 32)));
+      T* o = static_cast<T*>(out);
+      if (width <= 256) BCG_CUDA_CHECK(launch_k(ssm_norm_warp_kernel<T, 2>, grid, dim3(kSnThreads), 0, st, a, o, out_ld));
+      else if (width <= 1024) BCG_CUDA_CHECK(launch_k(ssm_norm_warp_kernel<T, 8>, grid, dim3(kSnThreads), 0, st, a, o, out_ld));
+      else BCG_CUDA_CHECK(launch_k(ssm_norm_warp_kernel<T, 16>, grid, dim3(kSnThreads), 0, st, a, o, out_ld));
+      return BCG_OK;
+    }
+  }
+  if (a.n_tokens <= 128 && width >= 1024)
+    return advance ? launch_norm_cl<T, V, 8, true>(a, out, out_ld, st) : launch_norm_cl<T, V, 8, false>(a, out, out_ld, st);
+  return advance ? launch_norm_cl<T, V, 1, true>(a, out, out_ld, st) : launch_norm_cl<T, V, 1, false>(a, out, out_ld, st);
 }
 
 // ------------------------------------------------------------------------------------------- launches
@@ -706,16 +838,18 @@ static int run_t(const SsmArgs& a, int n_seqs, bool one_token, int mode, void* o
   const bool wide = ((a.vdim | a.n | a.col) & 3) == 0 && a.ld % 4 == 0 && a.pstride % 4 == 0;
   const bool token = one_token && mode == 0, chunks = bf16 && mode == 0;
   if (!token) {
-    if (wide) BCG_TRY((launch_conv<T, 4>(a, st)));
-    else BCG_TRY((launch_conv<T, 1>(a, st)));
+    if (!wide) BCG_TRY((launch_conv<T, 1, false>(a, st)));
+    else if (a.n_partials == 1) BCG_TRY((launch_conv<T, 4, true>(a, st)));
+    else BCG_TRY((launch_conv<T, 4, false>(a, st)));
   }
   if (a.n <= 32) BCG_TRY((run_np<T, 32>(a, n_seqs, token, chunks, st)));
   else if (a.n <= 64) BCG_TRY((run_np<T, 64>(a, n_seqs, token, chunks, st)));
   else if (a.n <= 128) BCG_TRY((run_np<T, 128>(a, n_seqs, token, chunks, st)));
   else BCG_TRY((run_np<T, 256>(a, n_seqs, token, chunks, st)));
   const int width = a.inner() / a.parts;
-  if (width % 4 == 0 && out_ld % 4 == 0 && reinterpret_cast<uintptr_t>(out) % 16 == 0) return launch_norm<T, 4>(a, out, out_ld, st);
-  return launch_norm<T, 1>(a, out, out_ld, st);
+  if (width % 4 == 0 && out_ld % 4 == 0 && a.col % 4 == 0 && a.ld % 4 == 0 && a.pstride % 4 == 0)
+    return launch_norm<T, 4>(a, token, out, out_ld, st);
+  return launch_norm<T, 1>(a, token, out, out_ld, st);
 }
 
 int state_space(const bcg_stack* m, const bcg_layer* l, const bcg_stack_ws* ws, const bcg_step_batch* b, int n_partials,
@@ -723,7 +857,7 @@ int state_space(const bcg_stack* m, const bcg_layer* l, const bcg_stack_ws* ws, 
   if (!l->conv_w || !l->conv_b || !l->step_bias || !l->decay_rate || !l->skip || !l->ssm_norm || !l->ssm_state ||
       (l->ssm_taps > 1 && !l->conv_state) || !ws->ssm_x || !ws->ssm_step || !ws->ssm_y || !b->state_slots || l->ssm_n <= 0 ||
       l->ssm_n > 256 || l->ssm_vdim <= 0 || l->ssm_taps < 1 || l->ssm_groups <= 0 || l->ssm_heads % l->ssm_groups ||
-      l->ssm_norm_parts <= 0 || (l->ssm_heads * l->ssm_vdim) % l->ssm_norm_parts || b->n_seqs > 65535) {
+      l->ssm_norm_parts <= 0 || (l->ssm_heads * l->ssm_vdim) % l->ssm_norm_parts || l->ssm_heads * l->ssm_vdim / l->ssm_norm_parts > 51200 || b->n_seqs > 65535) {
     set_last_error("bcg_state_space", "bad layer (1..256 state entries, groups and parts that divide) or too many sequences");
     return BCG_ERR_ARG;
   }

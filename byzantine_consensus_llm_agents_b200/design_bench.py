@@ -28,10 +28,12 @@ from .tokenizer import get_tokenizer
 SIZES = {"2k": (2048, 6144, 8), "4k": (4096, 12288, 8)}
 # a stack's ff makes its layers (no gate matrix, other mixer projections) the dense layers' size
 BEKOPEL_FF = {"2k": 7424, "4k": 14592}
+MERULORN_FF = {"2k": 11520, "4k": 23680}       # of one layer in four; the others have none
 EXPERTS, TOP = 64, 8
 VOCAB, CTX, PROMPT, PROMPTS = 32768, 1600, 1536, 8
 FP32_FMA = 148 * 128 * 1.965e9       # nominal
-KINDS = {"bekopel": ("qwen3", "bekopel"), "lerazen": ("qwen3", "lerazen", "lerazen-moe")}
+KINDS = {"bekopel": ("qwen3", "bekopel"), "lerazen": ("qwen3", "lerazen", "lerazen-moe"),
+         "merulorn": ("qwen3", "bekopel", "merulorn")}
 
 
 def _config(kind: str, size: str):
@@ -39,6 +41,8 @@ def _config(kind: str, size: str):
     name, heads = f"{kind}-{size}", d // 128
     if kind == "bekopel":
         return S.bekopel_preset(name, layers, d, BEKOPEL_FF[size], VOCAB, heads=heads)
+    if kind == "merulorn":
+        return S.merulorn_preset(name, layers, d, MERULORN_FF[size], VOCAB, heads=heads)
     if kind.startswith("lerazen"):      # two matrices instead of three; experts: three matrices, TOP of them active
         return S.lerazen_preset(name, layers, d, ff * 3 // 2, VOCAB, heads=heads, kv_heads=8,
                                 experts=EXPERTS if kind.endswith("moe") else 0, top=TOP, expert_ff=ff // TOP)
@@ -277,9 +281,48 @@ def _lerazen_kernels(k: _Bench, what: str, B: int, T: int, shape: str, v, plan) 
         b["xn"].data_ptr(), L.DT_BF16, T, d, 1e-5, st()), nbytes=T * d * (10.0 + 4 * s3 + 4 * extra[2] * extra[3]))
 
 
+def _merulorn_kernels(k: _Bench, what: str, B: int, T: int, shape: str, v, plan) -> None:
+    e, b, cfg, lib, x, st = k.e, k.e.buf, k.e.cfg, k.e.lib, k.e.exec, L.stream_ptr
+    d, layer = cfg.d_model, next(i for i, l in enumerate(cfg.layers) if l.one(S.GroupedAttention))
+    spec, w, prefill = cfg.layers[layer], e.w.layers[layer], what == "prefill"
+    m, ssm, f = spec.one(S.GroupedAttention), spec.one(S.StateSpace), spec.mlp
+    bt = _step_batch(e, what, T, B, v, plan)
+    model, ws = C.byref(x.model.struct), C.byref(x.ws)
+    n_in, cols = cfg.in_rows(layer), cfg.mix_cols(layer)[1]
+    splits = lambda n, kk: 1 if prefill else L.splits_for(B, n, kk)
+    s = splits(n_in, d)
+    keys = PROMPT * (PROMPT + 1) // 2
+    k.gemm("input product", shape, b["xn"], w["w_in"], b["proj"], T, n_in, d, L.EPI_F32, s)
+    k.add("attention", shape, lambda: lib.bcg_grouped_attention(model, ws, C.byref(bt), layer, 0, st()),
+          **(dict(flops=2.0 * B * keys * m.heads * (m.dim + m.vdim)) if prefill
+             else dict(nbytes=B * CTX * m.kv_heads * (m.dim + m.vdim) * 2.0)))
+    k.add("input split", shape, lambda: lib.bcg_grouped_in(model, ws, C.byref(bt), layer, s, T * n_in, n_in, 0, st()),
+          nbytes=T * m.in_dim * (4.0 * s + 2))
+    # the projection in, outputs out, states in and out; the products of 64-token chunks
+    k.add("state space, all launches", shape, lambda: lib.bcg_state_space(model, ws, C.byref(bt), layer, s, T * n_in, n_in, 0, st()),
+          nbytes=T * (ssm.in_dim * 4.0 * s + ssm.out_dim * 2) + B * ssm.state_floats * 8.0,
+          flops=2.0 * T * (ssm.heads * ssm.vdim * (32 + 2 * ssm.state) + ssm.groups * 32 * ssm.state) if prefill else 0.0)
+    n_up = f.up_rows
+    if prefill or splits(n_up, d) == 1:
+        k.add("up product", shape, lambda: lib.bcg_gemm_bf16_glu(
+            b["xn"].data_ptr(), w["w_up"].data_ptr(), b["act"].data_ptr(), T, n_up, d, f.limit, f.alpha, 0, st()),
+            nbytes=2.0 * n_up * d + 2.0 * T * d + T * n_up, flops=2.0 * T * n_up * d)
+    else:
+        k.gemm("up product", shape, b["xn"], w["w_up"], b["proj"], T, n_up, d, L.EPI_F32, splits(n_up, d))
+        k.add("activation", shape, lambda: lib.bcg_clamped_glu(
+            b["proj"].data_ptr(), splits(n_up, d), T * n_up, b["act"].data_ptr(), L.DT_BF16, T, f.ff_ld, f.limit, f.alpha, st()),
+            nbytes=T * f.ff_ld * (8.0 * splits(n_up, d) + 2))
+    k.gemm("down product", shape, b["act"], w["w_down"], b["proj"], T, d, f.ff_ld, L.EPI_F32, splits(d, f.ff_ld))
+    s3 = splits(d, cols)
+    k.gemm("output product", shape, b["mix"], w["w_out"], b["proj"], T, d, cols, L.EPI_F32, s3)
+    k.add("norm", shape, lambda: lib.bcg_sandwich_norm(
+        b["residual"].data_ptr(), b["proj"].data_ptr(), s3, T * d, None, w["norm2"].data_ptr(), b["xn"].data_ptr(), L.DT_BF16, T, d,
+        1e-5, st()), nbytes=T * d * (10.0 + 4 * s3))
+
+
 def _kernels(e: Engine, kind: str, hbm: float, tf: float) -> list:
     k = _Bench(e, hbm, tf)
-    run = {"qwen3": _dense_kernels, "bekopel": _bekopel_kernels}.get(kind, _lerazen_kernels)
+    run = {"qwen3": _dense_kernels, "bekopel": _bekopel_kernels, "merulorn": _merulorn_kernels}.get(kind, _lerazen_kernels)
     for what, B in (("prefill", PROMPTS), ("decode", 8), ("decode", 64)):
         T = B * PROMPT if what == "prefill" else B
         plan, v = _prefill(e, B) if what == "prefill" else (None, None)
@@ -310,6 +353,8 @@ def _run(kind: str, size: str, tokenizer, hbm: float, tf: float, kernels: bool) 
             own = sum(isinstance(l.mixer, S.LatentAttention) for l in e.cfg.layers)
             has = sum(isinstance(l.mixer, S.LatentAttention) and l.mixer.kv_from is None for l in e.cfg.layers)
             cache = cache * own // max(has, 1) + 2 * e.cfg.state_bytes_per_row
+        if kind == "merulorn":
+            cache += 2 * e.cfg.state_bytes_per_row
         out[f"decode_ms_{B}"] = round(ms, 4)
         out[f"decode_tok_s_{B}"] = round(B / ms * 1e3)
         out[f"decode_of_hbm_roofline_{B}"] = round((weights + B * cache) / hbm / ms * 1e-6, 3)

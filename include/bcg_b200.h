@@ -509,7 +509,7 @@ typedef struct bcg_stack_ws {
   float* gates;     /* fp32 [T_max, heads]: factors of the head outputs */
   void* ssm_x;      /* act [T_max, ssm_x_ld(layer)]: convolved x | B | C, heads and groups padded to multiples of 8 */
   float* ssm_step;  /* fp32 [T_max, ssm_heads] */
-  void* ssm_y;      /* act [T_max, ssm_heads * ssm_vdim]: gated outputs in front of their norm */
+  void* ssm_y;      /* act [T_max, ssm_heads * ssm_vdim]: outputs in front of gate and norm */
 } bcg_stack_ws;
 
 /* A step: T new tokens of n_seqs sequences, portions of prompts beside single decoded tokens.  All

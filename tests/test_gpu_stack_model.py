@@ -48,7 +48,7 @@ CONFIGS = {
                                         SM.gattn(3, 1, 13, 11, 130, every=1, mlp=SM.dense(51))], width=61, vocab=83),
     "parallel-one": SM.parallel_config([SM.gattn(1, 1, 8, 8, 5, mlp=SM.dense(20))], width=36, vocab=36, positions=300),
     # attention beside a state space, state spaces alone, with and without a feed-forward
-    "side": SM.side_config([SM.mamba(), SM.both(mlp=SM.glu(70)), SM.mamba(heads=2, vdim=40, state=33, groups=1, norm_groups=4, conv=2, mlp=SM.glu(48, 0.4)),
+    "side": SM.side_config([SM.mamba(), SM.both(mlp=SM.glu(70)), SM.mamba(heads=2, vdim=40, state=33, groups=1, norm_groups=1, conv=2, mlp=SM.glu(48, 0.4)),
                             SM.both(4, 1, 16, 24, every=64, coef=-0.1, conv=3)]),
     # everything on the tensor-core kernels, two blocks of head entries, more parts than groups and fewer
     "side-tensor": SM.side_config([SM.both(8, 2, 64, 32, mlp=SM.glu(320, 7.0), vdim_ssm=80, state=64), SM.mamba(heads=4, vdim=64, state=128, groups=1, norm_groups=8),
