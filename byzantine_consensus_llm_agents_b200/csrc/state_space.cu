@@ -8,8 +8,9 @@
 //   ssm_chunk   portions (bf16): chunks of 64 tokens on tensor cores.  Inside a chunk the recurrence is a product,
 //                   y_i = exp(c_i) S^T C_i + sum_{j <= i} exp(c_i - c_j) step_j (B_j . C_i) x_j,   c = running sum of -rate * step,
 //               and the state moves once per chunk.  Everything is held transposed (rows = entries of a head's output), so
-//               that the state stays in fp32 accumulators and becomes an operand without leaving the registers.  What is
-//               fp32 by nature - the state, decays, steps - enters a product as two bf16 halves (hi + lo).
+//               that the state stays in fp32 accumulators and becomes an operand without leaving the registers.  Weights (decays,
+//               steps) are formed in fp32; what they add to the state enters its product as two bf16 halves (hi + lo),
+//               what is only read out is rounded like any activation.
 //   ssm_scan    portions token by token in fp32: the fp32 engine's kernel
 //   ssm_token   one token per sequence (decode): convolution and recurrence in one kernel; the states are requested
 //               before the dependency wait
@@ -243,18 +244,20 @@ struct StateRows {
         }
       }
   }
-  // One token: v[r] = step * x of row r, b / c the lane's entries of B and C.  Returns S^T C of row lane(), valid in lanes
+  // One token: v(r) = step * x of row r, b / c the lane's entries of B and C.  Returns S^T C of row lane(), valid in lanes
   // below kR.
-  __device__ __forceinline__ float token(float keep, const float (&v)[kR], const float (&b)[kQ][4], const float (&c)[kQ][4]) {
+  template <typename F>
+  __device__ __forceinline__ float token(float keep, F v, const float (&b)[kQ][4], const float (&c)[kQ][4]) {
     float y[kR];
 #pragma unroll
     for (int r = 0; r < kR; ++r) {
+      const float vr = v(r);
       y[r] = 0.f;
 #pragma unroll
       for (int q = 0; q < kQ; ++q)
 #pragma unroll
         for (int i = 0; i < 4; ++i) {
-          s[r][q][i] = fmaf(keep, s[r][q][i], v[r] * b[q][i]);
+          s[r][q][i] = fmaf(keep, s[r][q][i], vr * b[q][i]);
           y[r] = fmaf(s[r][q][i], c[q][i], y[r]);
         }
     }
@@ -273,7 +276,7 @@ struct StateRows {
 constexpr int kTapsAhead = 4;     // taps whose past inputs are requested before the dependency wait
 
 template <typename T, int NP>
-__global__ void __launch_bounds__(kSsThreads, NP <= 128 ? 3 : 2)
+__global__ void __launch_bounds__(kSsThreads, NP <= 128 ? 4 : 2)
 ssm_token_kernel(const SsmArgs a) {
   using S = StateRows<NP>;
   constexpr int kItems = (kSsRows + 2 * NP + 1 + kSsThreads - 1) / kSsThreads;
@@ -343,9 +346,7 @@ ssm_token_kernel(const SsmArgs a) {
   }
   __syncthreads();
   const float step = step_s, keep = decay_f32(-a.rate[h] * step);
-  float v[S::kR], b[S::kQ][4], c[S::kQ][4];
-#pragma unroll
-  for (int r = 0; r < S::kR; ++r) v[r] = step * xbc[S::row(r)];
+  float b[S::kQ][4], c[S::kQ][4];
 #pragma unroll
   for (int q = 0; q < S::kQ; ++q)
 #pragma unroll
@@ -353,7 +354,7 @@ ssm_token_kernel(const SsmArgs a) {
       b[q][i] = xbc[kSsRows + S::entry(q) + i];
       c[q][i] = xbc[kSsRows + NP + S::entry(q) + i];
     }
-  const float y = s.token(keep, v, b, c);
+  const float y = s.token(keep, [&](int r) { return step * xbc[S::row(r)]; }, b, c);
   s.store(st, rows, N);
   if (S::lane() < S::kR) {
     const int p = S::row(S::lane());
@@ -411,7 +412,7 @@ ssm_scan_kernel(const SsmArgs a) {
         cc[q][i] = c[q][i];
       }
     if (t + 1 < t1) fetch(t + 1);
-    const float y = s.token(keep, v, bb, cc);
+    const float y = s.token(keep, [&](int r) { return v[r]; }, bb, cc);
     if (S::lane() < S::kR) {
       const int p = S::row(S::lane());
       if (p < rows) static_cast<T*>(a.y)[static_cast<long long>(t) * inner + h * a.vdim + p0 + p] = from_f32<T>(fmaf(skip, mine, y));
@@ -428,7 +429,7 @@ template <int NP>
 struct ChCfg {
   static constexpr int kBRow = NP + 8, kXRow = kSsRows + 8, kMRow = kChTok + 8;       // pitches, bf16
   static constexpr int kBC = kChTok * kBRow, kX = kChTok * kXRow, kM = kChTok * kMRow;
-  static constexpr int kSmem = (2 * kBC + kX + 2 * kM) * 2 + 2 * 4 * kChTok * 4;        // B, C, x, M hi / lo, scalars
+  static constexpr int kSmem = (2 * kBC + kX + kM) * 2 + 2 * 4 * kChTok * 4;            // B, C, x, M, scalars
   static constexpr int kCtasPerSm = NP <= 128 ? 3 : 2;
 };
 
@@ -443,10 +444,10 @@ __device__ __forceinline__ uint32_t transpose_8x8(uint32_t v) {
   return r;
 }
 
-// M[i][j] = exp(c_i - c_j) step_j (C_i . B_j) for j <= i, tokens i = 16 RT .. 16 RT + 15, as two bf16 halves.
+// M[i][j] = exp(c_i - c_j) step_j (C_i . B_j) for j <= i, tokens i = 16 RT .. 16 RT + 15.
 template <int NP, int RT>
 __device__ __forceinline__ void chunk_matrix(const __nv_bfloat16* sB, const __nv_bfloat16* sC, const float* sum2,
-                                             const float* steps, __nv_bfloat16* m_hi, __nv_bfloat16* m_lo) {
+                                             const float* steps, __nv_bfloat16* sM) {
   using C = ChCfg<NP>;
   const int lane = threadIdx.x & 31, q2 = (lane & 3) * 2;
   float acc[2 * RT + 2][4] = {};
@@ -479,10 +480,7 @@ __device__ __forceinline__ void chunk_matrix(const __nv_bfloat16* sB, const __nv
         if (j > i) m0 = 0.f;
         if (j + 1 > i) m1 = 0.f;
       }
-      uint32_t hi, lo;
-      split_bf16(m0, m1, hi, lo);
-      *reinterpret_cast<uint32_t*>(m_hi + i * C::kMRow + j) = hi;
-      *reinterpret_cast<uint32_t*>(m_lo + i * C::kMRow + j) = lo;
+      *reinterpret_cast<uint32_t*>(sM + i * C::kMRow + j) = pack_bf16(m0, m1);
     }
   }
 }
@@ -496,9 +494,8 @@ ssm_chunk_kernel(const SsmArgs a) {
   __nv_bfloat16* sB = reinterpret_cast<__nv_bfloat16*>(ch_raw);
   __nv_bfloat16* sC = sB + C::kBC;
   __nv_bfloat16* sX = sC + C::kBC;
-  __nv_bfloat16* m_hi = sX + C::kX;
-  __nv_bfloat16* m_lo = m_hi + C::kM;
-  float* scalars = reinterpret_cast<float*>(m_lo + C::kM);     // [2][4][64]: log2 decay sums, steps, e, w
+  __nv_bfloat16* sM = sX + C::kX;
+  float* scalars = reinterpret_cast<float*>(sM + C::kM);     // [2][4][64]: log2 decay sums, steps, e, w
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, n_warps = blockDim.x >> 5;
   const int h = blockIdx.x, p0 = blockIdx.y * kSsRows, sq = blockIdx.z;
   const int rows = min(kSsRows, a.vdim - p0), N = a.n, g = h / (a.heads / a.groups), inner = a.inner();
@@ -574,10 +571,10 @@ ssm_chunk_kernel(const SsmArgs a) {
     __syncthreads();                            // the chunk is there
 
     for (int rt = warp; rt * 16 < nt_tok; rt += n_warps) {
-      if (rt == 0) chunk_matrix<NP, 0>(sB, sC, sum2, steps, m_hi, m_lo);
-      else if (rt == 1) chunk_matrix<NP, 1>(sB, sC, sum2, steps, m_hi, m_lo);
-      else if (rt == 2) chunk_matrix<NP, 2>(sB, sC, sum2, steps, m_hi, m_lo);
-      else chunk_matrix<NP, 3>(sB, sC, sum2, steps, m_hi, m_lo);
+      if (rt == 0) chunk_matrix<NP, 0>(sB, sC, sum2, steps, sM);
+      else if (rt == 1) chunk_matrix<NP, 1>(sB, sC, sum2, steps, sM);
+      else if (rt == 2) chunk_matrix<NP, 2>(sB, sC, sum2, steps, sM);
+      else chunk_matrix<NP, 3>(sB, sC, sum2, steps, sM);
     }
 
     // ---- Y^T = S^T C^T, columns (tokens) scaled by exp(c_i)
@@ -585,17 +582,15 @@ ssm_chunk_kernel(const SsmArgs a) {
     const __nv_bfloat16* pc = sC + ((lane & 7) + ((lane >> 4) << 3)) * C::kBRow + ((lane >> 3) & 1) * 8;
 #pragma unroll
     for (int k = 0; k < NP / 16; ++k) {
-      uint32_t hi[4], lo[4], cb[kChTok / 16][4];
+      const uint32_t sa[4] = {pack_bf16(S[2 * k][0], S[2 * k][1]), pack_bf16(S[2 * k][2], S[2 * k][3]),
+                              pack_bf16(S[2 * k + 1][0], S[2 * k + 1][1]), pack_bf16(S[2 * k + 1][2], S[2 * k + 1][3])};
 #pragma unroll
-      for (int ip = 0; ip < kChTok / 16; ++ip) ldsm_x4(cb[ip], pc + ip * 16 * C::kBRow + k * 16);
-      split_bf16(S[2 * k][0], S[2 * k][1], hi[0], lo[0]);
-      split_bf16(S[2 * k][2], S[2 * k][3], hi[1], lo[1]);
-      split_bf16(S[2 * k + 1][0], S[2 * k + 1][1], hi[2], lo[2]);
-      split_bf16(S[2 * k + 1][2], S[2 * k + 1][3], hi[3], lo[3]);
-#pragma unroll
-      for (int it = 0; it < kChTok / 8; ++it) mma_bf16_16816(Y[it], hi, cb[it >> 1][(it & 1) * 2], cb[it >> 1][(it & 1) * 2 + 1]);
-#pragma unroll
-      for (int it = 0; it < kChTok / 8; ++it) mma_bf16_16816(Y[it], lo, cb[it >> 1][(it & 1) * 2], cb[it >> 1][(it & 1) * 2 + 1]);
+      for (int ip = 0; ip < kChTok / 16; ++ip) {
+        uint32_t cb[4];
+        ldsm_x4(cb, pc + ip * 16 * C::kBRow + k * 16);
+        mma_bf16_16816(Y[2 * ip], sa, cb[0], cb[1]);
+        mma_bf16_16816(Y[2 * ip + 1], sa, cb[2], cb[3]);
+      }
     }
 #pragma unroll
     for (int it = 0; it < kChTok / 8; ++it) {
@@ -624,13 +619,10 @@ ssm_chunk_kernel(const SsmArgs a) {
 #pragma unroll
       for (int ip = jp; ip < kChTok / 16; ++ip)
         if (ip * 16 < nt_tok) {
-          uint32_t mh[4], ml[4];
-          ldsm_x4(mh, m_hi + pm + ip * 16 * C::kMRow + jp * 16);
-          ldsm_x4(ml, m_lo + pm + ip * 16 * C::kMRow + jp * 16);
-          mma_bf16_16816(Y[2 * ip], xa, mh[0], mh[1]);
-          mma_bf16_16816(Y[2 * ip + 1], xa, mh[2], mh[3]);
-          mma_bf16_16816(Y[2 * ip], xa, ml[0], ml[1]);
-          mma_bf16_16816(Y[2 * ip + 1], xa, ml[2], ml[3]);
+          uint32_t mb[4];
+          ldsm_x4(mb, sM + pm + ip * 16 * C::kMRow + jp * 16);
+          mma_bf16_16816(Y[2 * ip], xa, mb[0], mb[1]);
+          mma_bf16_16816(Y[2 * ip + 1], xa, mb[2], mb[3]);
         }
       float xf[4][2];                           // rows pr, pr + 8 of tokens j, j + 1; the same of tokens j + 8, j + 9
 #pragma unroll
@@ -810,7 +802,7 @@ static int launch_norm(const SsmArgs& a, bool advance, void* out, long long out_
       return BCG_OK;
     }
   }
-  if (a.n_tokens <= 128 && width >= 1024)
+  if (static_cast<long long>(a.n_tokens) * a.parts <= 64 && width >= 1024)      // few of them: a cluster each
     return advance ? launch_norm_cl<T, V, 8, true>(a, out, out_ld, st) : launch_norm_cl<T, V, 8, false>(a, out, out_ld, st);
   return advance ? launch_norm_cl<T, V, 1, true>(a, out, out_ld, st) : launch_norm_cl<T, V, 1, false>(a, out, out_ld, st);
 }
