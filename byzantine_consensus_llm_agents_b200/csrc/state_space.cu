@@ -12,8 +12,10 @@
 //               steps) are formed in fp32; what they add to the state enters its product as two bf16 halves (hi + lo),
 //               what is only read out is rounded like any activation.
 //   ssm_scan    portions token by token in fp32: the fp32 engine's kernel
-//   ssm_token   one token per sequence (decode): convolution and recurrence in one kernel; the states are requested
-//               before the dependency wait
+//   ssm_token   one token per sequence (decode): convolution and recurrence in one kernel, a head per CTA; the states are
+//               requested before the dependency wait
+//   ssm_stream  the same with the states streamed through shared memory: a CTA has a list of heads, bulk copies of the
+//               next ones' states in flight both ways, and the next one's operands requested a turn ahead
 //   ssm_norm    gate and norm of the outputs
 // The convolution's state moves on where nobody reads it any more: behind the chunks or the scan, and in ssm_norm for
 // single tokens (whose B and C every head of a group convolves for itself).
@@ -261,6 +263,10 @@ struct StateRows {
           y[r] = fmaf(s[r][q][i], c[q][i], y[r]);
         }
     }
+    return gather(y);
+  }
+  // The sums over a group's lanes; lane r gets row r's.
+  static __device__ __forceinline__ float gather(float (&y)[kR]) {
 #pragma unroll
     for (int m = kLanes / 2; m > 0; m >>= 1)
 #pragma unroll
@@ -271,79 +277,138 @@ struct StateRows {
       if (lane() == r) mine = y[r];
     return mine;
   }
+  // token() on a state in (shared) memory, row by row, n a multiple of 4.
+  template <typename F>
+  static __device__ __forceinline__ float token_in_place(float* st, int rows, int n, bool fresh, float keep, F v,
+                                                         const float (&b)[kQ][4], const float (&c)[kQ][4]) {
+    float y[kR];
+#pragma unroll
+    for (int r = 0; r < kR; ++r) {
+      y[r] = 0.f;
+      if (row(r) >= rows) continue;
+      const float vr = v(r);
+#pragma unroll
+      for (int q = 0; q < kQ; ++q) {
+        if (entry(q) >= n) continue;
+        float4* p = reinterpret_cast<float4*>(st + row(r) * n + entry(q));
+        float4 s = fresh ? make_float4(0.f, 0.f, 0.f, 0.f) : *p;
+        s.x = fmaf(keep, s.x, vr * b[q][0]);
+        s.y = fmaf(keep, s.y, vr * b[q][1]);
+        s.z = fmaf(keep, s.z, vr * b[q][2]);
+        s.w = fmaf(keep, s.w, vr * b[q][3]);
+        *p = s;
+        y[r] = fmaf(s.w, c[q][3], fmaf(s.z, c[q][2], fmaf(s.y, c[q][1], fmaf(s.x, c[q][0], y[r]))));
+      }
+    }
+    return gather(y);
+  }
 };
 
-constexpr int kTapsAhead = 4;     // taps whose past inputs are requested before the dependency wait
+constexpr int kTapsAhead = 4;     // taps whose past inputs are requested ahead of time
+
+// What is known of a token before its projections are.
+struct TokenPlace {
+  int t, h, slot;
+  bool idle, fresh;
+  __device__ __forceinline__ void load(const SsmArgs& a, int t_, int h_) {
+    t = t_;
+    h = h_;
+    idle = a.slot_map[t] < 0;
+    fresh = a.positions[t] == 0;
+    slot = a.state_slots[t];
+  }
+};
+
+// What one token's head needs: x of the block's rows, B and C behind the convolution, and the step.  begin() requests
+// weights and what earlier steps left, arrive() the projections (up to four slabs), finish() writes floats
+// [kSsRows | NP | NP] and the step.
+template <int NP>
+struct TokenInputs {
+  static constexpr int kItems = (kSsRows + 2 * NP + 1 + kSsThreads - 1) / kSsThreads;
+  TokenPlace at;
+  int chan[kItems];     // channel -1: padding, -2: the step
+  float past[kItems][kTapsAhead - 1], w[kItems][kTapsAhead], bias[kItems], v[kItems][4];
+
+  __device__ __forceinline__ void begin(const SsmArgs& a, const TokenPlace& place, int p0, int rows) {
+    at = place;
+    const int g = at.h / (a.heads / a.groups), ch = a.channels();
+    const float* cs = a.conv_state + static_cast<long long>(at.slot) * (a.taps - 1) * ch;
+#pragma unroll
+    for (int k = 0; k < kItems; ++k) {
+      const int i = threadIdx.x + k * kSsThreads, e = i - kSsRows;
+      chan[k] = -1;
+      if (i < rows) chan[k] = at.h * a.vdim + p0 + i;
+      else if (e >= 0 && e < 2 * NP && e % NP < a.n) chan[k] = a.inner() + (e / NP * a.groups + g) * a.n + e % NP;
+      else if (e == 2 * NP) chan[k] = -2;
+      const bool some = chan[k] >= 0;
+      // tap j of the last kTapsAhead: w[kTapsAhead - 1] is the current token's
+#pragma unroll
+      for (int j = 0; j < kTapsAhead; ++j) {
+        const int tap = a.taps - kTapsAhead + j;
+        w[k][j] = some && tap >= 0 ? a.conv_w[static_cast<long long>(tap) * ch + chan[k]] : 0.f;
+        if (j < kTapsAhead - 1)
+          past[k][j] = some && tap >= 0 && !at.idle && !at.fresh ? cs[static_cast<long long>(tap) * ch + chan[k]] : 0.f;
+      }
+      bias[k] = some ? a.conv_b[chan[k]] : chan[k] == -2 ? a.step_bias[at.h] : 0.f;
+    }
+  }
+  __device__ __forceinline__ const float* source(const SsmArgs& a, int k) const {
+    return a.row(at.t) + a.inner() + (chan[k] == -2 ? a.channels() + at.h : max(chan[k], 0));
+  }
+  __device__ __forceinline__ void arrive(const SsmArgs& a) {
+#pragma unroll
+    for (int k = 0; k < kItems; ++k)
+#pragma unroll
+      for (int q = 0; q < 4; ++q) v[k][q] = q < a.n_partials ? source(a, k)[q * a.pstride] : 0.f;
+  }
+  __device__ __forceinline__ void finish(const SsmArgs& a, float* xbc, float* step) const {
+    const int ch = a.channels();
+#pragma unroll
+    for (int k = 0; k < kItems; ++k) {
+      const int i = threadIdx.x + k * kSsThreads, c = chan[k];
+      float in = 0.f, y = 0.f;
+#pragma unroll
+      for (int q = 0; q < 4; ++q) in += v[k][q];
+      for (int q = 4; q < a.n_partials; ++q) in += source(a, k)[q * a.pstride];
+      if (c >= 0) {
+        y = fmaf(w[k][kTapsAhead - 1], in, bias[k]);
+#pragma unroll
+        for (int j = 0; j < kTapsAhead - 1; ++j) y = fmaf(w[k][j], past[k][j], y);
+        if (!at.fresh)
+          for (int j = 0; j < a.taps - kTapsAhead; ++j)
+            y = fmaf(a.conv_w[static_cast<long long>(j) * ch + c],
+                     a.conv_state[(static_cast<long long>(at.slot) * (a.taps - 1) + j) * ch + c], y);
+        y = silu_f32(y);
+      } else if (c == -2) {
+        *step = softplus_f32(in + bias[k]);
+      }
+      if (i < kSsRows + 2 * NP) xbc[i] = y;
+    }
+  }
+};
 
 template <typename T, int NP>
 __global__ void __launch_bounds__(kSsThreads, NP <= 128 ? 4 : 2)
 ssm_token_kernel(const SsmArgs a) {
   using S = StateRows<NP>;
-  constexpr int kItems = (kSsRows + 2 * NP + 1 + kSsThreads - 1) / kSsThreads;
   __shared__ float xbc[kSsRows + 2 * NP], step_s;
   const int h = blockIdx.x, p0 = blockIdx.y * kSsRows, t = blockIdx.z;
-  const int rows = min(kSsRows, a.vdim - p0), N = a.n, g = h / (a.heads / a.groups), inner = a.inner(), ch = a.channels();
+  const int rows = min(kSsRows, a.vdim - p0), N = a.n;
   pdl_launch_dependents();
   // Positions, slots and states were written by earlier steps, which are complete before any kernel of this step
   // starts, so the states are on their way while the projections are finished.
-  const bool idle = a.slot_map[t] < 0, fresh = a.positions[t] == 0;
-  const int slot = a.state_slots[t];
-  float* st = a.state + ((static_cast<long long>(slot) * a.heads + h) * a.vdim + p0) * N;
-  // items: x of the CTA's rows, B, C, the step; channel -1: padding, -2: the step
-  int chan[kItems];
-  float past[kItems][kTapsAhead - 1];
-  const float* cs = a.conv_state + static_cast<long long>(slot) * (a.taps - 1) * ch;
-#pragma unroll
-  for (int k = 0; k < kItems; ++k) {
-    const int i = threadIdx.x + k * kSsThreads, e = i - kSsRows;
-    chan[k] = -1;
-    if (i < rows) chan[k] = h * a.vdim + p0 + i;
-    else if (e >= 0 && e < 2 * NP && e % NP < N) chan[k] = inner + (e / NP * a.groups + g) * N + e % NP;
-    else if (e == 2 * NP) chan[k] = -2;
-#pragma unroll
-    for (int j = 0; j < kTapsAhead - 1; ++j)
-      past[k][j] = chan[k] >= 0 && !idle && !fresh && j < a.taps - 1 ? cs[static_cast<long long>(j) * ch + chan[k]] : 0.f;
-  }
+  TokenPlace place;
+  place.load(a, t, h);
+  float* st = a.state + ((static_cast<long long>(place.slot) * a.heads + h) * a.vdim + p0) * N;
   S s;
-  if (idle || fresh) s.zero();
+  if (place.idle || place.fresh) s.zero();
   else s.load(st, rows, N);
+  TokenInputs<NP> in;
+  in.begin(a, place, p0, rows);
   pdl_wait();
-  if (idle) return;
-  float in[kItems];
-#pragma unroll
-  for (int k = 0; k < kItems; ++k) in[k] = 0.f;
-  for (int p = 0; p < a.n_partials; p += 4) {       // slabs in index order, four per item in flight
-    float v[kItems][4];
-#pragma unroll
-    for (int k = 0; k < kItems; ++k) {
-      const float* src = a.row(t) + inner + (chan[k] == -2 ? ch + h : max(chan[k], 0));
-#pragma unroll
-      for (int q = 0; q < 4; ++q) v[k][q] = p + q < a.n_partials ? src[(p + q) * a.pstride] : 0.f;
-    }
-#pragma unroll
-    for (int k = 0; k < kItems; ++k)
-#pragma unroll
-      for (int q = 0; q < 4; ++q) in[k] += v[k][q];
-  }
-#pragma unroll
-  for (int k = 0; k < kItems; ++k) {
-    const int i = threadIdx.x + k * kSsThreads, c = chan[k];
-    float y = 0.f;
-    if (c >= 0) {
-      const float* w = a.conv_w + c;
-      y = fmaf(w[static_cast<long long>(a.taps - 1) * ch], in[k], a.conv_b[c]);
-#pragma unroll
-      for (int j = 0; j < kTapsAhead - 1; ++j)
-        if (j < a.taps - 1) y = fmaf(w[static_cast<long long>(j) * ch], past[k][j], y);
-      if (!fresh)
-        for (int j = kTapsAhead - 1; j < a.taps - 1; ++j)
-          y = fmaf(w[static_cast<long long>(j) * ch], cs[static_cast<long long>(j) * ch + c], y);
-      y = silu_f32(y);
-    } else if (c == -2) {
-      step_s = softplus_f32(in[k] + a.step_bias[h]);
-    }
-    if (i < kSsRows + 2 * NP) xbc[i] = y;
-  }
+  if (place.idle) return;
+  in.arrive(a);
+  in.finish(a, xbc, &step_s);
   __syncthreads();
   const float step = step_s, keep = decay_f32(-a.rate[h] * step);
   float b[S::kQ][4], c[S::kQ][4];
@@ -358,7 +423,133 @@ ssm_token_kernel(const SsmArgs a) {
   s.store(st, rows, N);
   if (S::lane() < S::kR) {
     const int p = S::row(S::lane());
-    if (p < rows) static_cast<T*>(a.y)[static_cast<long long>(t) * inner + h * a.vdim + p0 + p] = from_f32<T>(fmaf(a.skip[h], xbc[p], y));
+    if (p < rows)
+      static_cast<T*>(a.y)[static_cast<long long>(t) * a.inner() + h * a.vdim + p0 + p] = from_f32<T>(fmaf(a.skip[h], xbc[p], y));
+  }
+}
+
+__device__ __forceinline__ void bulk_store_1d(void* gdst, const void* smem_src, uint32_t bytes) {
+  asm volatile("cp.async.bulk.global.shared::cta.bulk_group [%0], [%1], %2;" ::"l"(gdst), "r"(smem_u32(smem_src)), "r"(bytes) : "memory");
+  asm volatile("cp.async.bulk.commit_group;" ::: "memory");
+}
+
+// State rows of 16 bytes' multiple, up to 128 entries.  A unit is 64 rows of a token's head (fewer at a head's end).  Warps
+// 0-7 compute, warp 8 moves states: a stage is filled, worked on in place, stored, and filled again once it has been read.
+constexpr int kStStages = 3, kStThreads = kSsThreads + 32;
+template <int NP>
+struct StCfg {
+  static constexpr int kStage = kSsRows * NP;      // floats
+  static constexpr int kOps = kSsRows + 2 * NP;
+  static constexpr int kSmem = kStStages * kStage * 4 + 2 * kOps * 4 + 64;
+};
+
+template <typename T, int NP>
+__global__ void __launch_bounds__(kStThreads, 2)
+ssm_stream_kernel(const SsmArgs a, int n_units) {
+  using S = StateRows<NP>;
+  using C = StCfg<NP>;
+  extern __shared__ __align__(128) float st_raw[];
+  float* xbc = st_raw + kStStages * C::kStage;                  // [2][rows | B | C]
+  float* steps = xbc + 2 * C::kOps;                             // [2]
+  uint64_t* full = reinterpret_cast<uint64_t*>(steps + 2);      // [stages] a state has arrived
+  uint64_t* done = full + kStStages;                            // [stages] it has been worked on
+  const int N = a.n, blocks = (a.vdim + kSsRows - 1) / kSsRows;
+  const int n = (n_units - static_cast<int>(blockIdx.x) + static_cast<int>(gridDim.x) - 1) / static_cast<int>(gridDim.x);
+  pdl_launch_dependents();
+  if (threadIdx.x == 0) {
+    for (int i = 0; i < kStStages; ++i) {
+      mbar_init(&full[i], 1);
+      mbar_init(&done[i], kSsThreads);
+    }
+    fence_barrier_init();
+  }
+  struct Unit {
+    int t, h, p0, rows;
+  };
+  auto unit = [&](int i) {          // heads are the fastest index: neighbours share a token's inputs
+    const int u = static_cast<int>(blockIdx.x) + i * static_cast<int>(gridDim.x), r = u / a.heads;
+    const int p0 = r % blocks * kSsRows;
+    return Unit{r / blocks, u % a.heads, p0, min(kSsRows, a.vdim - p0)};
+  };
+  __syncthreads();
+  // States, slots and positions were written by earlier steps (see ssm_token).
+  if (threadIdx.x >= kSsThreads) {
+    if (threadIdx.x == kSsThreads) {
+      auto state_of = [&](const Unit& u) {
+        return a.state + ((static_cast<long long>(a.state_slots[u.t]) * a.heads + u.h) * a.vdim + u.p0) * N;
+      };
+      for (int i = 0; i < n + kStStages - 1; ++i) {
+        if (i < n) {
+          const Unit u = unit(i);
+          const uint32_t bytes = static_cast<uint32_t>(u.rows * N * 4);
+          float* src = state_of(u);
+          // the stage's previous state (unit i - stages) was stored a turn ago
+          if (i >= kStStages) asm volatile("cp.async.bulk.wait_group.read 0;" ::: "memory");
+          mbar_arrive_expect_tx(&full[i % kStStages], bytes);
+          bulk_load_1d(st_raw + (i % kStStages) * C::kStage, src, bytes, &full[i % kStStages]);
+        }
+        const int j = i - (kStStages - 1);
+        if (j >= 0) {
+          const Unit u = unit(j);
+          float* dst = state_of(u);
+          const bool idle = a.slot_map[u.t] < 0;
+          mbar_wait(&done[j % kStStages], (j / kStStages) & 1);
+          if (!idle) bulk_store_1d(dst, st_raw + (j % kStStages) * C::kStage, static_cast<uint32_t>(u.rows * N * 4));
+        }
+      }
+      asm volatile("cp.async.bulk.wait_group 0;" ::: "memory");
+    }
+    return;
+  }
+  TokenInputs<NP> in;
+  TokenPlace next;
+  Unit u = unit(0);
+  next.load(a, u.t, u.h);
+  in.begin(a, next, u.p0, u.rows);
+  if (n > 1) {
+    const Unit v = unit(1);
+    next.load(a, v.t, v.h);
+  }
+  pdl_wait();
+  in.arrive(a);
+  for (int i = 0; i < n; ++i) {
+    float* ops = xbc + (i & 1) * C::kOps;
+    in.finish(a, ops, &steps[i & 1]);
+    const bool idle = in.at.idle, fresh = in.at.fresh;
+    const float rate = a.rate[u.h], skip = a.skip[u.h];
+    Unit v = u;
+    if (i + 1 < n) {                // requested now, used a turn later
+      v = unit(i + 1);
+      in.begin(a, next, v.p0, v.rows);
+      in.arrive(a);
+      if (i + 2 < n) {
+        const Unit w = unit(i + 2);
+        next.load(a, w.t, w.h);
+      }
+    }
+    asm volatile("bar.sync 1, %0;" ::"n"(kSsThreads) : "memory");     // operands are there
+    mbar_wait(&full[i % kStStages], (i / kStStages) & 1);
+    if (!idle) {
+      float* st = st_raw + (i % kStStages) * C::kStage;
+      const float step = steps[i & 1], keep = decay_f32(-rate * step);
+      float b[S::kQ][4], c[S::kQ][4];
+#pragma unroll
+      for (int q = 0; q < S::kQ; ++q)
+#pragma unroll
+        for (int k = 0; k < 4; ++k) {
+          b[q][k] = ops[kSsRows + S::entry(q) + k];
+          c[q][k] = ops[kSsRows + NP + S::entry(q) + k];
+        }
+      const float y = S::token_in_place(st, u.rows, N, fresh, keep, [&](int r) { return step * ops[S::row(r)]; }, b, c);
+      if (S::lane() < S::kR) {
+        const int p = S::row(S::lane());
+        if (p < u.rows)
+          static_cast<T*>(a.y)[static_cast<long long>(u.t) * a.inner() + u.h * a.vdim + u.p0 + p] = from_f32<T>(fmaf(skip, ops[p], y));
+      }
+      fence_proxy_async();
+    }
+    mbar_arrive(&done[i % kStStages]);
+    u = v;
   }
 }
 
@@ -812,7 +1003,13 @@ template <typename T, int NP>
 static int run_np(const SsmArgs& a, int n_seqs, bool one_token, bool chunks, cudaStream_t st) {
   const int blocks = (a.vdim + kSsRows - 1) / kSsRows;
   const dim3 grid(a.heads, blocks, n_seqs);
-  if (one_token) {
+  if (one_token && NP <= 128 && a.n % 4 == 0) {
+    constexpr int P = NP <= 128 ? NP : 128;
+    const long long units = static_cast<long long>(n_seqs) * a.heads * blocks;
+    const int ctas = static_cast<int>(units < 2 * 148 ? units : 2 * 148);
+    BCG_TRY(ensure_dynamic_smem(reinterpret_cast<const void*>(ssm_stream_kernel<T, P>), StCfg<P>::kSmem));
+    BCG_CUDA_CHECK(launch_k(ssm_stream_kernel<T, P>, dim3(ctas), dim3(kStThreads), StCfg<P>::kSmem, st, a, static_cast<int>(units)));
+  } else if (one_token) {
     BCG_CUDA_CHECK(launch_k(ssm_token_kernel<T, NP>, grid, dim3(kSsThreads), 0, st, a));
   } else if (chunks) {
     BCG_TRY(ensure_dynamic_smem(reinterpret_cast<const void*>(ssm_chunk_kernel<NP>), ChCfg<NP>::kSmem));

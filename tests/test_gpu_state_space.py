@@ -57,7 +57,7 @@ class OneLayer:
         for i, e in enumerate(entries):
             if not isinstance(e, Entry):
                 bt = np.zeros(self.eng.max_blocks, np.int32)
-                bt[:4] = np.arange(4) + 4 * i
+                bt[:4] = np.arange(4) + 4 * (i % 8)
                 e = Entry([0] * e[0], e[1], bt, e[2])
             out.append(e)
         p = self.x.plan(out)
@@ -77,7 +77,8 @@ class OneLayer:
 # ------------------------------------------------------------------------------------------ state space
 SIZES = {  # heads, vdim, state, groups, norm_groups, conv
     "usual": (4, 64, 128, 2, 2, 4), "small": (4, 16, 16, 4, 1, 4), "blocks": (2, 136, 64, 1, 2, 3), "wide": (2, 64, 256, 1, 1, 2),
-    "odd": (3, 11, 13, 3, 3, 4), "halves": (2, 66, 50, 1, 4, 5), "one": (1, 8, 8, 1, 1, 1), "parts": (8, 24, 36, 2, 48, 4), "row": (2, 1, 200, 2, 2, 3)}
+    "odd": (3, 11, 13, 3, 3, 4), "halves": (2, 66, 50, 1, 4, 5), "one": (1, 8, 8, 1, 1, 1), "parts": (8, 24, 36, 2, 48, 4), "row": (2, 1, 200, 2, 2, 3),
+    "many": (72, 16, 20, 8, 4, 3), "many-blocks": (40, 72, 24, 4, 1, 5)}
 
 
 class StateSpace(OneLayer):
@@ -196,6 +197,40 @@ def test_single_tokens_in_one_launch_and_idle_rows():
         close(a.state[3 - s], S, a.tol)
         close(a.conv[3 - s], last, 1e-5)
     assert torch.equal(a.state[2], before[0][2]) and torch.equal(a.conv[2], before[1][2])
+
+
+@pytest.mark.parametrize("dtype", DT)
+@pytest.mark.parametrize("size", ["many", "many-blocks", "row"])
+def test_more_single_tokens_than_ctas(size, dtype):
+    """Several steps of fifteen sequences: long ones, one that starts, one that is finished."""
+    n = 15
+    a = StateSpace(size, dtype, rows=16)
+    proj = [_proj(a, 6 if s == 4 else 12, s) for s in range(n)]
+    a.junk()
+    for s in range(n):
+        if s != 4:
+            a.run([(6, 0, s)], proj[s][:6])
+    idle = a.state[9].clone(), a.conv[9].clone()
+    got = [[] for _ in range(n)]
+    for step in range(6):
+        starts = [step if s == 4 else 6 + step for s in range(n)]
+        p, b = a.batch([(1, starts[s], s) for s in range(n)])
+        a.keep["slots"][9] = -1
+        full = torch.zeros(n, a.ld)
+        full[:, :a.rows] = torch.stack([proj[s][starts[s]] for s in range(n)])
+        a.set("proj", full)
+        L.check(a.eng.lib.bcg_state_space(*a.args(C.byref(b), 0, 1, 0, a.ld, 0)))
+        out = a.get("mix", n, a.layer.mix_ld)[:, :a.inner]
+        for s in range(n):
+            got[s].append(out[s])
+    for s in range(n):
+        if s == 9:
+            continue
+        want, S, last = a.oracle(proj[s])
+        a.check(torch.stack(got[s]), want[-6:], a.tol)
+        close(a.state[s], S, a.tol)
+        close(a.conv[s], last, 1e-5)
+    assert torch.equal(a.state[9], idle[0]) and torch.equal(a.conv[9], idle[1])
 
 
 @pytest.mark.parametrize("dtype", DT)
