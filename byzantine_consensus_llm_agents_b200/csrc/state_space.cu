@@ -246,8 +246,10 @@ struct StateRows {
         }
       }
   }
-  // One token: v(r) = step * x of row r, b / c the lane's entries of B and C.  Returns S^T C of row lane(), valid in lanes
-  // below kR.
+  // The row of the group whose output a lane ends up with, and whether it is the lane to write it.
+  static __device__ __forceinline__ int mine() { return lane() / (kLanes / kR); }
+  static __device__ __forceinline__ bool writes() { return lane() % (kLanes / kR) == 0; }
+  // One token: v(r) = step * x of row r, b / c the lane's entries of B and C.  Returns S^T C of row mine().
   template <typename F>
   __device__ __forceinline__ float token(float keep, F v, const float (&b)[kQ][4], const float (&c)[kQ][4]) {
     float y[kR];
@@ -265,32 +267,37 @@ struct StateRows {
     }
     return gather(y);
   }
-  // The sums over a group's lanes; lane r gets row r's.
+  // The sums over a group's lanes; every lane gets row mine()'s.  Half of the rows change sides at every exchange.
   static __device__ __forceinline__ float gather(float (&y)[kR]) {
+    int m = kLanes / 2;
 #pragma unroll
-    for (int m = kLanes / 2; m > 0; m >>= 1)
+    for (int w = kR / 2; w > 0; w >>= 1, m >>= 1) {
+      const bool up = lane() & m;
 #pragma unroll
-      for (int r = 0; r < kR; ++r) y[r] += __shfl_xor_sync(0xffffffffu, y[r], m);
-    float mine = y[0];
+      for (int r = 0; r < w; ++r) {
+        const float other = __shfl_xor_sync(0xffffffffu, up ? y[r] : y[r + w], m);
+        y[r] = (up ? y[r + w] : y[r]) + other;
+      }
+    }
 #pragma unroll
-    for (int r = 1; r < kR; ++r)
-      if (lane() == r) mine = y[r];
-    return mine;
+    for (; m > 0; m >>= 1) y[0] += __shfl_xor_sync(0xffffffffu, y[0], m);
+    return y[0];
   }
-  // token() on a state in (shared) memory, row by row, n a multiple of 4.
-  template <typename F>
+  // token() on a state in shared memory, row by row, n a multiple of 4.  FULL: all rows, n = NP.
+  template <bool FULL, typename F>
   static __device__ __forceinline__ float token_in_place(float* st, int rows, int n, bool fresh, float keep, F v,
                                                          const float (&b)[kQ][4], const float (&c)[kQ][4]) {
+    const int pitch = FULL ? NP : n;
     float y[kR];
 #pragma unroll
     for (int r = 0; r < kR; ++r) {
       y[r] = 0.f;
-      if (row(r) >= rows) continue;
+      if (!FULL && row(r) >= rows) continue;
       const float vr = v(r);
 #pragma unroll
       for (int q = 0; q < kQ; ++q) {
-        if (entry(q) >= n) continue;
-        float4* p = reinterpret_cast<float4*>(st + row(r) * n + entry(q));
+        if (!FULL && entry(q) >= n) continue;
+        float4* p = reinterpret_cast<float4*>(st + row(r) * pitch + entry(q));
         float4 s = fresh ? make_float4(0.f, 0.f, 0.f, 0.f) : *p;
         s.x = fmaf(keep, s.x, vr * b[q][0]);
         s.y = fmaf(keep, s.y, vr * b[q][1]);
@@ -319,98 +326,88 @@ struct TokenPlace {
   }
 };
 
-// What one token's head needs: x of the block's rows, B and C behind the convolution, and the step.  begin() requests
-// weights and what earlier steps left, arrive() the projections (up to four slabs), finish() writes floats
-// [kSsRows | NP | NP] and the step.
-template <int NP>
-struct TokenInputs {
-  static constexpr int kItems = (kSsRows + 2 * NP + 1 + kSsThreads - 1) / kSsThreads;
-  TokenPlace at;
-  int chan[kItems];     // channel -1: padding, -2: the step
-  float past[kItems][kTapsAhead - 1], w[kItems][kTapsAhead], bias[kItems], v[kItems][4];
+// One channel of a single token's convolution (or its step) on the way: begin() requests weights and what earlier steps
+// left, arrive() the projection (up to four slabs), value() is the sum behind its activation.
+constexpr int kPadChannel = -1, kStepChannel = -2;
+struct TokenChannel {
+  int c;
+  float past[kTapsAhead - 1], w[kTapsAhead], bias, v[4];
 
-  __device__ __forceinline__ void begin(const SsmArgs& a, const TokenPlace& place, int p0, int rows) {
-    at = place;
-    const int g = at.h / (a.heads / a.groups), ch = a.channels();
-    const float* cs = a.conv_state + static_cast<long long>(at.slot) * (a.taps - 1) * ch;
+  __device__ __forceinline__ void begin(const SsmArgs& a, const TokenPlace& at, int c_) {
+    c = c_;
+    const int ch = a.channels(), tap0 = a.taps - kTapsAhead;     // w[kTapsAhead - 1] is the current token's
+    const float* cw = a.conv_w + c;
+    const float* cs = a.conv_state + static_cast<long long>(at.slot) * (a.taps - 1) * ch + c;
+    const bool old = c >= 0 && !at.idle && !at.fresh;
 #pragma unroll
-    for (int k = 0; k < kItems; ++k) {
-      const int i = threadIdx.x + k * kSsThreads, e = i - kSsRows;
-      chan[k] = -1;
-      if (i < rows) chan[k] = at.h * a.vdim + p0 + i;
-      else if (e >= 0 && e < 2 * NP && e % NP < a.n) chan[k] = a.inner() + (e / NP * a.groups + g) * a.n + e % NP;
-      else if (e == 2 * NP) chan[k] = -2;
-      const bool some = chan[k] >= 0;
-      // tap j of the last kTapsAhead: w[kTapsAhead - 1] is the current token's
-#pragma unroll
-      for (int j = 0; j < kTapsAhead; ++j) {
-        const int tap = a.taps - kTapsAhead + j;
-        w[k][j] = some && tap >= 0 ? a.conv_w[static_cast<long long>(tap) * ch + chan[k]] : 0.f;
-        if (j < kTapsAhead - 1)
-          past[k][j] = some && tap >= 0 && !at.idle && !at.fresh ? cs[static_cast<long long>(tap) * ch + chan[k]] : 0.f;
-      }
-      bias[k] = some ? a.conv_b[chan[k]] : chan[k] == -2 ? a.step_bias[at.h] : 0.f;
+    for (int j = 0; j < kTapsAhead; ++j) {
+      w[j] = c >= 0 && tap0 + j >= 0 ? cw[(tap0 + j) * ch] : 0.f;
+      if (j < kTapsAhead - 1) past[j] = old && tap0 + j >= 0 ? cs[(tap0 + j) * ch] : 0.f;
     }
+    bias = c >= 0 ? a.conv_b[c] : c == kStepChannel ? a.step_bias[at.h] : 0.f;
   }
-  __device__ __forceinline__ const float* source(const SsmArgs& a, int k) const {
-    return a.row(at.t) + a.inner() + (chan[k] == -2 ? a.channels() + at.h : max(chan[k], 0));
+  __device__ __forceinline__ const float* source(const SsmArgs& a, const TokenPlace& at) const {
+    return a.row(at.t) + a.inner() + (c == kStepChannel ? a.channels() + at.h : max(c, 0));
   }
-  __device__ __forceinline__ void arrive(const SsmArgs& a) {
+  __device__ __forceinline__ void arrive(const SsmArgs& a, const TokenPlace& at) {
+    const float* src = source(a, at);
 #pragma unroll
-    for (int k = 0; k < kItems; ++k)
-#pragma unroll
-      for (int q = 0; q < 4; ++q) v[k][q] = q < a.n_partials ? source(a, k)[q * a.pstride] : 0.f;
+    for (int q = 0; q < 4; ++q) v[q] = c != kPadChannel && q < a.n_partials ? src[q * a.pstride] : 0.f;
   }
-  __device__ __forceinline__ void finish(const SsmArgs& a, float* xbc, float* step) const {
-    const int ch = a.channels();
+  __device__ __forceinline__ float value(const SsmArgs& a, const TokenPlace& at) const {
+    float in = (v[0] + v[1]) + (v[2] + v[3]);
+    if (c == kPadChannel) return 0.f;
+    for (int q = 4; q < a.n_partials; ++q) in += source(a, at)[q * a.pstride];
+    if (c == kStepChannel) return softplus_f32(in + bias);
+    float y = fmaf(w[kTapsAhead - 1], in, bias);
 #pragma unroll
-    for (int k = 0; k < kItems; ++k) {
-      const int i = threadIdx.x + k * kSsThreads, c = chan[k];
-      float in = 0.f, y = 0.f;
-#pragma unroll
-      for (int q = 0; q < 4; ++q) in += v[k][q];
-      for (int q = 4; q < a.n_partials; ++q) in += source(a, k)[q * a.pstride];
-      if (c >= 0) {
-        y = fmaf(w[k][kTapsAhead - 1], in, bias[k]);
-#pragma unroll
-        for (int j = 0; j < kTapsAhead - 1; ++j) y = fmaf(w[k][j], past[k][j], y);
-        if (!at.fresh)
-          for (int j = 0; j < a.taps - kTapsAhead; ++j)
-            y = fmaf(a.conv_w[static_cast<long long>(j) * ch + c],
-                     a.conv_state[(static_cast<long long>(at.slot) * (a.taps - 1) + j) * ch + c], y);
-        y = silu_f32(y);
-      } else if (c == -2) {
-        *step = softplus_f32(in + bias[k]);
-      }
-      if (i < kSsRows + 2 * NP) xbc[i] = y;
-    }
+    for (int j = 0; j < kTapsAhead - 1; ++j) y = fmaf(w[j], past[j], y);
+    if (!at.fresh)
+      for (int j = 0; j < a.taps - kTapsAhead; ++j)
+        y = fmaf(a.conv_w[static_cast<long long>(j) * a.channels() + c],
+                 a.conv_state[(static_cast<long long>(at.slot) * (a.taps - 1) + j) * a.channels() + c], y);
+    return silu_f32(y);
   }
 };
+// Channel of entry e of [B: NP | C: NP] of group g.
+template <int NP>
+__device__ __forceinline__ int bc_channel(const SsmArgs& a, int g, int e) {
+  const int which = e / NP, k = e % NP;
+  return e < 2 * NP && k < a.n ? a.inner() + (which * a.groups + g) * a.n + k : kPadChannel;
+}
 
 template <typename T, int NP>
-__global__ void __launch_bounds__(kSsThreads, NP <= 128 ? 4 : 2)
+__global__ void __launch_bounds__(kSsThreads, NP <= 128 ? 2 : 1)
 ssm_token_kernel(const SsmArgs a) {
   using S = StateRows<NP>;
-  __shared__ float xbc[kSsRows + 2 * NP], step_s;
+  constexpr int kItems = (kSsRows + 2 * NP + 1 + kSsThreads - 1) / kSsThreads;
+  __shared__ float xbc[kItems * kSsThreads];        // x of the CTA's rows | B | C | step
   const int h = blockIdx.x, p0 = blockIdx.y * kSsRows, t = blockIdx.z;
   const int rows = min(kSsRows, a.vdim - p0), N = a.n;
   pdl_launch_dependents();
   // Positions, slots and states were written by earlier steps, which are complete before any kernel of this step
   // starts, so the states are on their way while the projections are finished.
-  TokenPlace place;
-  place.load(a, t, h);
-  float* st = a.state + ((static_cast<long long>(place.slot) * a.heads + h) * a.vdim + p0) * N;
+  TokenPlace at;
+  at.load(a, t, h);
+  float* st = a.state + ((static_cast<long long>(at.slot) * a.heads + h) * a.vdim + p0) * N;
   S s;
-  if (place.idle || place.fresh) s.zero();
+  if (at.idle || at.fresh) s.zero();
   else s.load(st, rows, N);
-  TokenInputs<NP> in;
-  in.begin(a, place, p0, rows);
+  TokenChannel in[kItems];
+#pragma unroll
+  for (int k = 0; k < kItems; ++k) {
+    const int i = threadIdx.x + k * kSsThreads, e = i - kSsRows;
+    in[k].begin(a, at, e < 0 ? (i < rows ? h * a.vdim + p0 + i : kPadChannel)
+                             : e == 2 * NP ? kStepChannel : bc_channel<NP>(a, h / (a.heads / a.groups), e));
+  }
   pdl_wait();
-  if (place.idle) return;
-  in.arrive(a);
-  in.finish(a, xbc, &step_s);
+  if (at.idle) return;
+#pragma unroll
+  for (int k = 0; k < kItems; ++k) in[k].arrive(a, at);
+#pragma unroll
+  for (int k = 0; k < kItems; ++k) xbc[threadIdx.x + k * kSsThreads] = in[k].value(a, at);
   __syncthreads();
-  const float step = step_s, keep = decay_f32(-a.rate[h] * step);
+  const float step = xbc[kSsRows + 2 * NP], keep = decay_f32(-a.rate[h] * step);
   float b[S::kQ][4], c[S::kQ][4];
 #pragma unroll
   for (int q = 0; q < S::kQ; ++q)
@@ -421,11 +418,9 @@ ssm_token_kernel(const SsmArgs a) {
     }
   const float y = s.token(keep, [&](int r) { return step * xbc[S::row(r)]; }, b, c);
   s.store(st, rows, N);
-  if (S::lane() < S::kR) {
-    const int p = S::row(S::lane());
-    if (p < rows)
-      static_cast<T*>(a.y)[static_cast<long long>(t) * a.inner() + h * a.vdim + p0 + p] = from_f32<T>(fmaf(a.skip[h], xbc[p], y));
-  }
+  const int p = S::row(S::mine());
+  if (S::writes() && p < rows)
+    static_cast<T*>(a.y)[static_cast<long long>(t) * a.inner() + h * a.vdim + p0 + p] = from_f32<T>(fmaf(a.skip[h], xbc[p], y));
 }
 
 __device__ __forceinline__ void bulk_store_1d(void* gdst, const void* smem_src, uint32_t bytes) {
@@ -433,14 +428,43 @@ __device__ __forceinline__ void bulk_store_1d(void* gdst, const void* smem_src, 
   asm volatile("cp.async.bulk.commit_group;" ::: "memory");
 }
 
-// State rows of 16 bytes' multiple, up to 128 entries.  A unit is 64 rows of a token's head (fewer at a head's end).  Warps
-// 0-7 compute, warp 8 moves states: a stage is filled, worked on in place, stored, and filled again once it has been read.
+// State rows of 16 bytes' multiple, up to 128 entries.  A unit is 64 rows of a token's head (fewer at a head's end), a CTA
+// has consecutive ones: B and C are made once per group.  Warps 0-7 compute, warp 8 moves states: a stage is filled, worked
+// on in place, stored, and filled again once it has been read.
 constexpr int kStStages = 3, kStThreads = kSsThreads + 32;
 template <int NP>
 struct StCfg {
-  static constexpr int kStage = kSsRows * NP;      // floats
-  static constexpr int kOps = kSsRows + 2 * NP;
-  static constexpr int kSmem = kStStages * kStage * 4 + 2 * kOps * 4 + 64;
+  static constexpr int kStage = kSsRows * NP;                             // floats
+  static constexpr int kX = kSsRows + 4, kBC = 2 * NP;                    // x and the step (16-byte multiple); B and C; two of each
+  static constexpr int kSmem = (kStStages * kStage + 2 * kX + 2 * kBC) * 4 + 64;
+};
+
+// A walk over units: heads first, then blocks of rows, then tokens.
+struct UnitWalk {
+  int t, pb, h, in_group, g;
+  __device__ __forceinline__ UnitWalk(const SsmArgs& a, int blocks, int u) {
+    const int r = u / a.heads, per = a.heads / a.groups;
+    h = u - r * a.heads;
+    t = r / blocks;
+    pb = r - t * blocks;
+    g = h / per;
+    in_group = h - g * per;
+  }
+  __device__ __forceinline__ void next(const SsmArgs& a, int blocks) {
+    ++h;
+    if (++in_group == a.heads / a.groups) {
+      in_group = 0;
+      ++g;
+    }
+    if (h == a.heads) {
+      h = g = 0;
+      if (++pb == blocks) {
+        pb = 0;
+        ++t;
+      }
+    }
+  }
+  __device__ __forceinline__ int rows(const SsmArgs& a) const { return min(kSsRows, a.vdim - pb * kSsRows); }
 };
 
 template <typename T, int NP>
@@ -448,13 +472,15 @@ __global__ void __launch_bounds__(kStThreads, 2)
 ssm_stream_kernel(const SsmArgs a, int n_units) {
   using S = StateRows<NP>;
   using C = StCfg<NP>;
+  constexpr int kItems = (C::kBC + kSsThreads - 1) / kSsThreads;
   extern __shared__ __align__(128) float st_raw[];
-  float* xbc = st_raw + kStStages * C::kStage;                  // [2][rows | B | C]
-  float* steps = xbc + 2 * C::kOps;                             // [2]
-  uint64_t* full = reinterpret_cast<uint64_t*>(steps + 2);      // [stages] a state has arrived
+  float* xs = st_raw + kStStages * C::kStage;                   // [2][rows | step]
+  float* bc = xs + 2 * C::kX;                                   // [2][B | C]
+  uint64_t* full = reinterpret_cast<uint64_t*>(bc + 2 * C::kBC);   // [stages] a state has arrived
   uint64_t* done = full + kStStages;                            // [stages] it has been worked on
   const int N = a.n, blocks = (a.vdim + kSsRows - 1) / kSsRows;
-  const int n = (n_units - static_cast<int>(blockIdx.x) + static_cast<int>(gridDim.x) - 1) / static_cast<int>(gridDim.x);
+  const int u0 = static_cast<int>(static_cast<long long>(n_units) * blockIdx.x / gridDim.x);
+  const int n = static_cast<int>(static_cast<long long>(n_units) * (blockIdx.x + 1) / gridDim.x) - u0;
   pdl_launch_dependents();
   if (threadIdx.x == 0) {
     for (int i = 0; i < kStStages; ++i) {
@@ -463,93 +489,121 @@ ssm_stream_kernel(const SsmArgs a, int n_units) {
     }
     fence_barrier_init();
   }
-  struct Unit {
-    int t, h, p0, rows;
-  };
-  auto unit = [&](int i) {          // heads are the fastest index: neighbours share a token's inputs
-    const int u = static_cast<int>(blockIdx.x) + i * static_cast<int>(gridDim.x), r = u / a.heads;
-    const int p0 = r % blocks * kSsRows;
-    return Unit{r / blocks, u % a.heads, p0, min(kSsRows, a.vdim - p0)};
-  };
   __syncthreads();
   // States, slots and positions were written by earlier steps (see ssm_token).
   if (threadIdx.x >= kSsThreads) {
     if (threadIdx.x == kSsThreads) {
-      auto state_of = [&](const Unit& u) {
-        return a.state + ((static_cast<long long>(a.state_slots[u.t]) * a.heads + u.h) * a.vdim + u.p0) * N;
+      UnitWalk in(a, blocks, u0), out = in;
+      auto state_of = [&](const UnitWalk& u) {
+        return a.state + ((static_cast<long long>(a.state_slots[u.t]) * a.heads + u.h) * a.vdim + u.pb * kSsRows) * N;
       };
       for (int i = 0; i < n + kStStages - 1; ++i) {
         if (i < n) {
-          const Unit u = unit(i);
-          const uint32_t bytes = static_cast<uint32_t>(u.rows * N * 4);
-          float* src = state_of(u);
+          const uint32_t bytes = static_cast<uint32_t>(in.rows(a) * N * 4);
+          const float* src = state_of(in);
           // the stage's previous state (unit i - stages) was stored a turn ago
           if (i >= kStStages) asm volatile("cp.async.bulk.wait_group.read 0;" ::: "memory");
           mbar_arrive_expect_tx(&full[i % kStStages], bytes);
           bulk_load_1d(st_raw + (i % kStStages) * C::kStage, src, bytes, &full[i % kStStages]);
+          in.next(a, blocks);
         }
         const int j = i - (kStStages - 1);
         if (j >= 0) {
-          const Unit u = unit(j);
-          float* dst = state_of(u);
-          const bool idle = a.slot_map[u.t] < 0;
+          float* dst = state_of(out);
+          const bool idle = a.slot_map[out.t] < 0;
           mbar_wait(&done[j % kStStages], (j / kStStages) & 1);
-          if (!idle) bulk_store_1d(dst, st_raw + (j % kStStages) * C::kStage, static_cast<uint32_t>(u.rows * N * 4));
+          if (!idle) bulk_store_1d(dst, st_raw + (j % kStStages) * C::kStage, static_cast<uint32_t>(out.rows(a) * N * 4));
+          out.next(a, blocks);
         }
       }
       asm volatile("cp.async.bulk.wait_group 0;" ::: "memory");
     }
     return;
   }
-  TokenInputs<NP> in;
-  TokenPlace next;
-  Unit u = unit(0);
-  next.load(a, u.t, u.h);
-  in.begin(a, next, u.p0, u.rows);
-  if (n > 1) {
-    const Unit v = unit(1);
-    next.load(a, v.t, v.h);
-  }
+  UnitWalk u(a, blocks, u0);
+  TokenPlace at, ahead;             // of this unit, of the next one
+  TokenChannel x, group[kItems];    // threads up to kSsRows have an x channel or the step, all have some of B and C
+  auto x_begin = [&](const UnitWalk& w, const TokenPlace& place) {
+    const int tid = static_cast<int>(threadIdx.x);
+    if (tid <= kSsRows)
+      x.begin(a, place, tid == kSsRows ? kStepChannel : tid < w.rows(a) ? w.h * a.vdim + w.pb * kSsRows + tid : kPadChannel);
+  };
+  auto x_arrive = [&](const TokenPlace& place) {
+    if (threadIdx.x <= kSsRows) x.arrive(a, place);
+  };
+  auto group_begin = [&](const UnitWalk& w, const TokenPlace& place) {
+#pragma unroll
+    for (int k = 0; k < kItems; ++k) group[k].begin(a, place, bc_channel<NP>(a, w.g, threadIdx.x + k * kSsThreads));
+  };
+  auto group_arrive = [&](const TokenPlace& place) {
+#pragma unroll
+    for (int k = 0; k < kItems; ++k) group[k].arrive(a, place);
+  };
+  at.load(a, u.t, u.h);
+  x_begin(u, at);
+  group_begin(u, at);
+  float rate = a.rate[u.h], skip = a.skip[u.h];
   pdl_wait();
-  in.arrive(a);
+  x_arrive(at);
+  group_arrive(at);
+  bool new_group = true;
+  int side = 1;                     // of bc
   for (int i = 0; i < n; ++i) {
-    float* ops = xbc + (i & 1) * C::kOps;
-    in.finish(a, ops, &steps[i & 1]);
-    const bool idle = in.at.idle, fresh = in.at.fresh;
-    const float rate = a.rate[u.h], skip = a.skip[u.h];
-    Unit v = u;
-    if (i + 1 < n) {                // requested now, used a turn later
-      v = unit(i + 1);
-      in.begin(a, next, v.p0, v.rows);
-      in.arrive(a);
-      if (i + 2 < n) {
-        const Unit w = unit(i + 2);
-        next.load(a, w.t, w.h);
+    float* xi = xs + (i & 1) * C::kX;
+    if (threadIdx.x <= kSsRows) xi[threadIdx.x] = x.value(a, at);
+    if (new_group) {
+      side ^= 1;
+#pragma unroll
+      for (int k = 0; k < kItems; ++k) {
+        const int e = threadIdx.x + k * kSsThreads;
+        if (e < C::kBC) bc[side * C::kBC + e] = group[k].value(a, at);
       }
+    }
+    UnitWalk w = u;
+    float rate1 = rate, skip1 = skip;
+    ahead = at;
+    new_group = false;
+    if (i + 1 < n) {                // requested now, used a turn later
+      w.next(a, blocks);
+      if (w.t != u.t) ahead.load(a, w.t, w.h);
+      ahead.h = w.h;
+      new_group = w.t != u.t || w.g != u.g;
+      x_begin(w, ahead);
+      x_arrive(ahead);
+      if (new_group) {
+        group_begin(w, ahead);
+        group_arrive(ahead);
+      }
+      rate1 = a.rate[w.h];
+      skip1 = a.skip[w.h];
     }
     asm volatile("bar.sync 1, %0;" ::"n"(kSsThreads) : "memory");     // operands are there
     mbar_wait(&full[i % kStStages], (i / kStStages) & 1);
-    if (!idle) {
+    if (!at.idle) {
       float* st = st_raw + (i % kStStages) * C::kStage;
-      const float step = steps[i & 1], keep = decay_f32(-rate * step);
+      const float step = xi[kSsRows], keep = decay_f32(-rate * step);
       float b[S::kQ][4], c[S::kQ][4];
 #pragma unroll
-      for (int q = 0; q < S::kQ; ++q)
-#pragma unroll
-        for (int k = 0; k < 4; ++k) {
-          b[q][k] = ops[kSsRows + S::entry(q) + k];
-          c[q][k] = ops[kSsRows + NP + S::entry(q) + k];
-        }
-      const float y = S::token_in_place(st, u.rows, N, fresh, keep, [&](int r) { return step * ops[S::row(r)]; }, b, c);
-      if (S::lane() < S::kR) {
-        const int p = S::row(S::lane());
-        if (p < u.rows)
-          static_cast<T*>(a.y)[static_cast<long long>(u.t) * a.inner() + u.h * a.vdim + u.p0 + p] = from_f32<T>(fmaf(skip, ops[p], y));
+      for (int q = 0; q < S::kQ; ++q) {
+        const float4 bv = *reinterpret_cast<const float4*>(bc + side * C::kBC + S::entry(q));
+        const float4 cv = *reinterpret_cast<const float4*>(bc + side * C::kBC + NP + S::entry(q));
+        b[q][0] = bv.x; b[q][1] = bv.y; b[q][2] = bv.z; b[q][3] = bv.w;
+        c[q][0] = cv.x; c[q][1] = cv.y; c[q][2] = cv.z; c[q][3] = cv.w;
       }
+      const int rows = u.rows(a);
+      auto v = [&](int r) { return step * xi[S::row(r)]; };
+      const float y = rows == kSsRows && N == NP ? S::template token_in_place<true>(st, rows, N, at.fresh, keep, v, b, c)
+                                                 : S::template token_in_place<false>(st, rows, N, at.fresh, keep, v, b, c);
+      const int p = S::row(S::mine());
+      if (S::writes() && p < rows)
+        static_cast<T*>(a.y)[static_cast<long long>(u.t) * a.inner() + u.h * a.vdim + u.pb * kSsRows + p] = from_f32<T>(fmaf(skip, xi[p], y));
       fence_proxy_async();
     }
     mbar_arrive(&done[i % kStStages]);
-    u = v;
+    u = w;
+    at = ahead;
+    rate = rate1;
+    skip = skip1;
   }
 }
 
@@ -593,7 +647,7 @@ ssm_scan_kernel(const SsmArgs a) {
 #pragma unroll
     for (int r = 0; r < S::kR; ++r) {
       v[r] = step * x[r];
-      if (S::lane() == r) mine = x[r];
+      if (S::mine() == r) mine = x[r];
     }
 #pragma unroll
     for (int q = 0; q < S::kQ; ++q)
@@ -604,10 +658,9 @@ ssm_scan_kernel(const SsmArgs a) {
       }
     if (t + 1 < t1) fetch(t + 1);
     const float y = s.token(keep, [&](int r) { return v[r]; }, bb, cc);
-    if (S::lane() < S::kR) {
-      const int p = S::row(S::lane());
-      if (p < rows) static_cast<T*>(a.y)[static_cast<long long>(t) * inner + h * a.vdim + p0 + p] = from_f32<T>(fmaf(skip, mine, y));
-    }
+    const int p = S::row(S::mine());
+    if (S::writes() && p < rows)
+      static_cast<T*>(a.y)[static_cast<long long>(t) * inner + h * a.vdim + p0 + p] = from_f32<T>(fmaf(skip, mine, y));
   }
   s.store(st, rows, N);
   advance_conv_of_head(a, sq, t0, t1, fresh, h, p0, rows);
