@@ -19,6 +19,8 @@
 //   ssm_norm    gate and norm of the outputs
 // The convolution's state moves on where nobody reads it any more: behind the chunks or the scan, and in ssm_norm for
 // single tokens (whose B and C every head of a group convolves for itself).
+#include <type_traits>
+
 #include "mma_sync.cuh"
 #include "attn_tcgen05.cuh"
 #include "stack_common.cuh"
@@ -677,10 +679,24 @@ struct ChCfg {
   static constexpr int kCtasPerSm = NP <= 128 ? 3 : 2;
 };
 
+// matrix loads from shared-memory addresses: offsets that are constants cost no instruction
+__device__ __forceinline__ void ldsm_at(uint32_t (&r)[4], uint32_t p) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0, %1, %2, %3}, [%4];"
+               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3])
+               : "r"(p));
+}
+__device__ __forceinline__ void ldsm_trans_at(uint32_t (&r)[4], uint32_t p) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0, %1, %2, %3}, [%4];"
+               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3])
+               : "r"(p));
+}
 // hi + lo = v to about 2^-17
 __device__ __forceinline__ void split_bf16(float a, float b, uint32_t& hi, uint32_t& lo) {
   hi = pack_bf16(a, b);
   lo = pack_bf16(a - bf16lo(hi), b - bf16hi(hi));
+}
+__device__ __forceinline__ void scale2(float& a, float& b, float fa, float fb) {
+  unpack_f32x2(mul_f32x2(pack_f32x2(__float_as_uint(a), __float_as_uint(b)), pack_f32x2(__float_as_uint(fa), __float_as_uint(fb))), a, b);
 }
 __device__ __forceinline__ uint32_t transpose_8x8(uint32_t v) {
   uint32_t r;
@@ -695,16 +711,16 @@ __device__ __forceinline__ void chunk_matrix(const __nv_bfloat16* sB, const __nv
   using C = ChCfg<NP>;
   const int lane = threadIdx.x & 31, q2 = (lane & 3) * 2;
   float acc[2 * RT + 2][4] = {};
-  const __nv_bfloat16* pc = sC + (RT * 16 + (lane & 15)) * C::kBRow + (lane >> 4) * 8;
-  const __nv_bfloat16* pb = sB + ((lane & 7) + ((lane >> 4) << 3)) * C::kBRow + ((lane >> 3) & 1) * 8;
+  const uint32_t pc = smem_u32(sC + (RT * 16 + (lane & 15)) * C::kBRow + (lane >> 4) * 8);
+  const uint32_t pb = smem_u32(sB + ((lane & 7) + ((lane >> 4) << 3)) * C::kBRow + ((lane >> 3) & 1) * 8);
 #pragma unroll
   for (int k = 0; k < NP / 16; ++k) {
     uint32_t ca[4];
-    ldsm_x4(ca, pc + k * 16);
+    ldsm_at(ca, pc + k * 32);
 #pragma unroll
     for (int jp = 0; jp <= RT; ++jp) {
       uint32_t bb[4];
-      ldsm_x4(bb, pb + jp * 16 * C::kBRow + k * 16);
+      ldsm_at(bb, pb + (jp * 16 * C::kBRow + k * 16) * 2);
       mma_bf16_16816(acc[2 * jp], ca, bb[0], bb[1]);
       mma_bf16_16816(acc[2 * jp + 1], ca, bb[2], bb[3]);
     }
@@ -740,7 +756,7 @@ ssm_chunk_kernel(const SsmArgs a) {
   __nv_bfloat16* sX = sC + C::kBC;
   __nv_bfloat16* sM = sX + C::kX;
   float* scalars = reinterpret_cast<float*>(sM + C::kM);     // [2][4][64]: log2 decay sums, steps, e, w
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, n_warps = blockDim.x >> 5;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int h = blockIdx.x, p0 = blockIdx.y * kSsRows, sq = blockIdx.z;
   const int rows = min(kSsRows, a.vdim - p0), N = a.n, g = h / (a.heads / a.groups), inner = a.inner();
   pdl_launch_dependents();
@@ -749,27 +765,33 @@ ssm_chunk_kernel(const SsmArgs a) {
   if (t1 <= t0 || a.slot_map[t0] < 0) return;
   const float rate = a.rate[h], skip = a.skip[h];
   const __nv_bfloat16* xbc = static_cast<const __nv_bfloat16*>(a.x);
-  const int x_ld = a.x_ld();
+  const int x_ld = a.x_ld(), b_col = a.b_col(g), c_col = a.c_col(g), x_col = h * a.x_pad() + p0;
 
-  // 64 tokens from `first` on, `valid` columns from `col` on; columns and tokens past the end are zero
-  auto copy_rows = [&](__nv_bfloat16* dst, int pitch, int col, int valid, int units, int first) {
-    for (int i = threadIdx.x; i < kChTok * units; i += blockDim.x) {
-      const int r = i / units, u = i - r * units;
-      const int bytes = first + r < t1 ? max(0, min(16, (valid - u * 8) * 2)) : 0;
-      const __nv_bfloat16* src = bytes ? xbc + static_cast<long long>(first + r) * x_ld + col + u * 8 : xbc;
-      asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(smem_u32(dst + r * pitch + u * 8)), "l"(src), "r"(bytes)
+  // 64 tokens from `first` on, up to 8 UNITS columns from `col` on, `valid` of them; the rest and tokens past the end are zero
+  auto copy_rows = [&](auto units, __nv_bfloat16* dst, int pitch, int col, int valid, int first) {
+    constexpr int kUnits = decltype(units)::value, kPass = kChThreads / kUnits;
+    const int u = threadIdx.x % kUnits, r = threadIdx.x / kUnits, wide = max(0, min(16, (valid - u * 8) * 2));
+    const __nv_bfloat16* src = xbc + static_cast<long long>(first + r) * x_ld + col + u * 8;
+    const uint32_t to = smem_u32(dst + r * pitch + u * 8);
+#pragma unroll
+    for (int i = 0; i < kChTok / kPass; ++i) {
+      const int bytes = first + r + i * kPass < t1 ? wide : 0;
+      asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(to + i * kPass * pitch * 2), "l"(bytes ? src : xbc), "r"(bytes)
                    : "memory");
+      src += static_cast<long long>(kPass) * x_ld;
     }
   };
+  using BCUnits = std::integral_constant<int, NP / 8>;
+  using XUnits = std::integral_constant<int, kSsRows / 8>;
   auto step_at = [&](int t) { return t < t1 ? a.step[static_cast<long long>(t) * a.heads + h] : 0.f; };
 
   const int n_chunks = (t1 - t0 + kChTok - 1) / kChTok;
   const int pr = warp * 16 + (lane >> 2);       // this lane's rows of the state: pr, pr + 8; entries nt * 8 + 2 (lane & 3) ..
   const int q2 = (lane & 3) * 2;
   float* st = a.state + ((static_cast<long long>(a.state_slots[sq]) * a.heads + h) * a.vdim + p0) * N;
-  copy_rows(sB, C::kBRow, a.b_col(g), N, NP / 8, t0);
-  copy_rows(sC, C::kBRow, a.c_col(g), N, NP / 8, t0);
-  copy_rows(sX, C::kXRow, h * a.x_pad() + p0, rows, kSsRows / 8, t0);
+  copy_rows(BCUnits{}, sB, C::kBRow, b_col, N, t0);
+  copy_rows(BCUnits{}, sC, C::kBRow, c_col, N, t0);
+  copy_rows(XUnits{}, sX, C::kXRow, x_col, rows, t0);
   cp_async_commit();
   float S[NP / 8][4];
   const bool fresh = a.positions[t0] == 0;
@@ -781,49 +803,50 @@ ssm_chunk_kernel(const SsmArgs a) {
       S[nt][i] = !fresh && p < rows && n < N ? st[static_cast<long long>(p) * N + n] : 0.f;
     }
   float s0 = 0.f, s1 = 0.f;                     // warp 0: steps of tokens 2 lane, 2 lane + 1 of the next chunk
+  // warp 0: the scalars of chunk c from s0 and s1, then the steps of the chunk behind it
+  auto scalars_of = [&](int c) {
+    float* sum2 = scalars + (c & 1) * 4 * kChTok;
+    float *steps = sum2 + kChTok, *e_s = steps + kChTok, *w_s = e_s + kChTok;
+    const float a0 = -rate * s0, a1 = -rate * s1;
+    float run = a0 + a1;
+#pragma unroll
+    for (int o = 1; o < 32; o <<= 1) {
+      const float v = __shfl_up_sync(0xffffffffu, run, o);
+      if (lane >= o) run += v;
+    }
+    const float total = __shfl_sync(0xffffffffu, run, 31);
+    const float c1 = run, c0 = run - a1;
+    *reinterpret_cast<float2*>(sum2 + 2 * lane) = make_float2(c0 * kSsLog2e, c1 * kSsLog2e);
+    *reinterpret_cast<float2*>(steps + 2 * lane) = make_float2(s0, s1);
+    *reinterpret_cast<float2*>(e_s + 2 * lane) = make_float2(expf(c0), expf(c1));
+    *reinterpret_cast<float2*>(w_s + 2 * lane) = make_float2(s0 * expf(total - c0), s1 * expf(total - c1));
+    s0 = step_at(t0 + (c + 1) * kChTok + 2 * lane);
+    s1 = step_at(t0 + (c + 1) * kChTok + 2 * lane + 1);
+  };
   if (warp == 0) {
     s0 = step_at(t0 + 2 * lane);
     s1 = step_at(t0 + 2 * lane + 1);
+    scalars_of(0);
   }
 
   for (int c = 0; c < n_chunks; ++c) {
     const int first = t0 + c * kChTok, nt_tok = min(kChTok, t1 - first);
-    float* sum2 = scalars + (c & 1) * 4 * kChTok;
-    float *steps = sum2 + kChTok, *e_s = steps + kChTok, *w_s = e_s + kChTok;
-    if (warp == 0) {
-      const float a0 = -rate * s0, a1 = -rate * s1;
-      float run = a0 + a1;
-#pragma unroll
-      for (int o = 1; o < 32; o <<= 1) {
-        const float v = __shfl_up_sync(0xffffffffu, run, o);
-        if (lane >= o) run += v;
-      }
-      const float total = __shfl_sync(0xffffffffu, run, 31);
-      const float c1 = run, c0 = run - a1;
-      sum2[2 * lane] = c0 * kSsLog2e;
-      sum2[2 * lane + 1] = c1 * kSsLog2e;
-      steps[2 * lane] = s0;
-      steps[2 * lane + 1] = s1;
-      e_s[2 * lane] = expf(c0);
-      e_s[2 * lane + 1] = expf(c1);
-      w_s[2 * lane] = s0 * expf(total - c0);
-      w_s[2 * lane + 1] = s1 * expf(total - c1);
-      s0 = step_at(first + kChTok + 2 * lane);
-      s1 = step_at(first + kChTok + 2 * lane + 1);
-    }
+    const float* sum2 = scalars + (c & 1) * 4 * kChTok;
+    const float *steps = sum2 + kChTok, *e_s = steps + kChTok, *w_s = e_s + kChTok;
     cp_async_wait<0>();
     __syncthreads();                            // the chunk is there
 
-    for (int rt = warp; rt * 16 < nt_tok; rt += n_warps) {
-      if (rt == 0) chunk_matrix<NP, 0>(sB, sC, sum2, steps, sM);
-      else if (rt == 1) chunk_matrix<NP, 1>(sB, sC, sum2, steps, sM);
-      else if (rt == 2) chunk_matrix<NP, 2>(sB, sC, sum2, steps, sM);
+    if (warp * 16 < nt_tok) {
+      if (warp == 0) chunk_matrix<NP, 0>(sB, sC, sum2, steps, sM);
+      else if (warp == 1) chunk_matrix<NP, 1>(sB, sC, sum2, steps, sM);
+      else if (warp == 2) chunk_matrix<NP, 2>(sB, sC, sum2, steps, sM);
       else chunk_matrix<NP, 3>(sB, sC, sum2, steps, sM);
     }
+    if (warp == 0) scalars_of(c + 1);           // the warp with the smallest share of M
 
     // ---- Y^T = S^T C^T, columns (tokens) scaled by exp(c_i)
     float Y[kChTok / 8][4] = {};
-    const __nv_bfloat16* pc = sC + ((lane & 7) + ((lane >> 4) << 3)) * C::kBRow + ((lane >> 3) & 1) * 8;
+    const uint32_t pc = smem_u32(sC + ((lane & 7) + ((lane >> 4) << 3)) * C::kBRow + ((lane >> 3) & 1) * 8);
 #pragma unroll
     for (int k = 0; k < NP / 16; ++k) {
       const uint32_t sa[4] = {pack_bf16(S[2 * k][0], S[2 * k][1]), pack_bf16(S[2 * k][2], S[2 * k][3]),
@@ -831,7 +854,7 @@ ssm_chunk_kernel(const SsmArgs a) {
 #pragma unroll
       for (int ip = 0; ip < kChTok / 16; ++ip) {
         uint32_t cb[4];
-        ldsm_x4(cb, pc + ip * 16 * C::kBRow + k * 16);
+        ldsm_at(cb, pc + (ip * 16 * C::kBRow + k * 16) * 2);
         mma_bf16_16816(Y[2 * ip], sa, cb[0], cb[1]);
         mma_bf16_16816(Y[2 * ip + 1], sa, cb[2], cb[3]);
       }
@@ -839,32 +862,31 @@ ssm_chunk_kernel(const SsmArgs a) {
 #pragma unroll
     for (int it = 0; it < kChTok / 8; ++it) {
       const float2 e = *reinterpret_cast<const float2*>(e_s + it * 8 + q2);
-      Y[it][0] *= e.x;
-      Y[it][1] *= e.y;
-      Y[it][2] *= e.x;
-      Y[it][3] *= e.y;
+      scale2(Y[it][0], Y[it][1], e.x, e.y);
+      scale2(Y[it][2], Y[it][3], e.x, e.y);
     }
     const float keep = e_s[kChTok - 1];         // past the end steps are zero: the whole chunk's decay
 #pragma unroll
-    for (int nt = 0; nt < NP / 8; ++nt)
-#pragma unroll
-      for (int i = 0; i < 4; ++i) S[nt][i] *= keep;
+    for (int nt = 0; nt < NP / 8; ++nt) {
+      scale2(S[nt][0], S[nt][1], keep, keep);
+      scale2(S[nt][2], S[nt][3], keep, keep);
+    }
     __syncthreads();                            // M is complete, C has been read
-    if (c + 1 < n_chunks) copy_rows(sC, C::kBRow, a.c_col(g), N, NP / 8, first + kChTok);
+    if (c + 1 < n_chunks) copy_rows(BCUnits{}, sC, C::kBRow, c_col, N, first + kChTok);
 
     // ---- Y^T += x^T M^T + skip x^T;   S^T += (w x)^T B
-    const __nv_bfloat16* px = sX + ((lane & 7) + ((lane >> 4) << 3)) * C::kXRow + warp * 16 + ((lane >> 3) & 1) * 8;
-    const __nv_bfloat16* pb = sB + (lane & 15) * C::kBRow + (lane >> 4) * 8;
-    const int pm = ((lane & 7) + ((lane >> 4) << 3)) * C::kMRow + ((lane >> 3) & 1) * 8;
+    const uint32_t px = smem_u32(sX + ((lane & 7) + ((lane >> 4) << 3)) * C::kXRow + warp * 16 + ((lane >> 3) & 1) * 8);
+    const uint32_t pb = smem_u32(sB + (lane & 15) * C::kBRow + (lane >> 4) * 8);
+    const uint32_t pm = smem_u32(sM + ((lane & 7) + ((lane >> 4) << 3)) * C::kMRow + ((lane >> 3) & 1) * 8);
 #pragma unroll
     for (int jp = 0; jp < kChTok / 16; ++jp) {
       uint32_t xa[4];
-      ldsm_x4_trans(xa, px + jp * 16 * C::kXRow);
+      ldsm_trans_at(xa, px + jp * 16 * C::kXRow * 2);
 #pragma unroll
       for (int ip = jp; ip < kChTok / 16; ++ip)
         if (ip * 16 < nt_tok) {
           uint32_t mb[4];
-          ldsm_x4(mb, sM + pm + ip * 16 * C::kMRow + jp * 16);
+          ldsm_at(mb, pm + (ip * 16 * C::kMRow + jp * 16) * 2);
           mma_bf16_16816(Y[2 * ip], xa, mb[0], mb[1]);
           mma_bf16_16816(Y[2 * ip + 1], xa, mb[2], mb[3]);
         }
@@ -890,8 +912,8 @@ ssm_chunk_kernel(const SsmArgs a) {
 #pragma unroll
       for (int np = 0; np < NP / 16; np += 2) {
         uint32_t b0[4], b1[4];
-        ldsm_x4_trans(b0, pb + jp * 16 * C::kBRow + np * 16);
-        ldsm_x4_trans(b1, pb + jp * 16 * C::kBRow + np * 16 + 16);
+        ldsm_trans_at(b0, pb + (jp * 16 * C::kBRow + np * 16) * 2);
+        ldsm_trans_at(b1, pb + (jp * 16 * C::kBRow + np * 16 + 16) * 2);
         mma_bf16_16816(S[2 * np], hi, b0[0], b0[1]);
         mma_bf16_16816(S[2 * np + 1], hi, b0[2], b0[3]);
         mma_bf16_16816(S[2 * np + 2], hi, b1[0], b1[1]);
@@ -904,29 +926,32 @@ ssm_chunk_kernel(const SsmArgs a) {
     }
     __syncthreads();                            // B and x have been read
     if (c + 1 < n_chunks) {
-      copy_rows(sB, C::kBRow, a.b_col(g), N, NP / 8, first + kChTok);
-      copy_rows(sX, C::kXRow, h * a.x_pad() + p0, rows, kSsRows / 8, first + kChTok);
+      copy_rows(BCUnits{}, sB, C::kBRow, b_col, N, first + kChTok);
+      copy_rows(XUnits{}, sX, C::kXRow, x_col, rows, first + kChTok);
       cp_async_commit();
     }
 
-    // ---- store: pairs are transposed on the way out
-    __nv_bfloat16* out = static_cast<__nv_bfloat16*>(a.y) + static_cast<long long>(first) * inner + h * a.vdim + p0;
+    // ---- store: pairs are transposed on the way out (token lane >> 2, entries q2, q2 + 1)
+    __nv_bfloat16* out = static_cast<__nv_bfloat16*>(a.y) + static_cast<long long>(first + (lane >> 2)) * inner + h * a.vdim + p0 +
+                         warp * 16 + q2;
+    const bool whole = nt_tok == kChTok && warp * 16 + 16 <= rows && (a.vdim & 1) == 0;
 #pragma unroll
     for (int it = 0; it < kChTok / 8; ++it) {
       if (it * 8 >= nt_tok) break;
 #pragma unroll
       for (int e = 0; e < 2; ++e) {
-        const uint32_t v = transpose_8x8(pack_bf16(Y[it][2 * e], Y[it][2 * e + 1]));     // token lane >> 2, entries q2, q2 + 1
-        const int tok = it * 8 + (lane >> 2), p = warp * 16 + e * 8 + q2;
-        __nv_bfloat16* dst = out + static_cast<long long>(tok) * inner + p;
-        if (tok < nt_tok && p + 1 < rows && (a.vdim & 1) == 0) {
+        const uint32_t v = transpose_8x8(pack_bf16(Y[it][2 * e], Y[it][2 * e + 1]));
+        __nv_bfloat16* dst = out + e * 8;
+        const int p = warp * 16 + e * 8 + q2;
+        if (whole) {
           *reinterpret_cast<uint32_t*>(dst) = v;
-        } else if (tok < nt_tok) {
+        } else if (it * 8 + (lane >> 2) < nt_tok) {
           if (p < rows) dst[0] = __ushort_as_bfloat16(static_cast<unsigned short>(v & 0xffffu));
           if (p + 1 < rows) dst[1] = __ushort_as_bfloat16(static_cast<unsigned short>(v >> 16));
         }
         __syncwarp();
       }
+      out += 8ll * inner;
     }
   }
 #pragma unroll
@@ -1066,8 +1091,7 @@ static int run_np(const SsmArgs& a, int n_seqs, bool one_token, bool chunks, cud
     BCG_CUDA_CHECK(launch_k(ssm_token_kernel<T, NP>, grid, dim3(kSsThreads), 0, st, a));
   } else if (chunks) {
     BCG_TRY(ensure_dynamic_smem(reinterpret_cast<const void*>(ssm_chunk_kernel<NP>), ChCfg<NP>::kSmem));
-    const int warps = (min(a.vdim, kSsRows) + 15) / 16;
-    BCG_CUDA_CHECK(launch_k(ssm_chunk_kernel<NP>, grid, dim3(warps * 32), ChCfg<NP>::kSmem, st, a));
+    BCG_CUDA_CHECK(launch_k(ssm_chunk_kernel<NP>, grid, dim3(kChThreads), ChCfg<NP>::kSmem, st, a));
   } else {
     BCG_CUDA_CHECK(launch_k(ssm_scan_kernel<T, NP>, grid, dim3(kSsThreads), 0, st, a));
   }

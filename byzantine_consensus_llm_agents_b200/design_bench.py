@@ -290,9 +290,8 @@ def _merulorn_kernels(k: _Bench, what: str, B: int, T: int, shape: str, v, plan)
     model, ws = C.byref(x.model.struct), C.byref(x.ws)
     n_in, cols = cfg.in_rows(layer), cfg.mix_cols(layer)[1]
     splits = lambda n, kk: 1 if prefill else L.splits_for(B, n, kk)
-    s = splits(n_in, d)
+    s, s3 = splits(n_in, d), splits(d, cols)
     keys = PROMPT * (PROMPT + 1) // 2
-    k.gemm("input product", shape, b["xn"], w["w_in"], b["proj"], T, n_in, d, L.EPI_F32, s)
     k.add("attention", shape, lambda: lib.bcg_grouped_attention(model, ws, C.byref(bt), layer, 0, st()),
           **(dict(flops=2.0 * B * keys * m.heads * (m.dim + m.vdim)) if prefill
              else dict(nbytes=B * CTX * m.kv_heads * (m.dim + m.vdim) * 2.0)))
@@ -302,6 +301,10 @@ def _merulorn_kernels(k: _Bench, what: str, B: int, T: int, shape: str, v, plan)
     k.add("state space, all launches", shape, lambda: lib.bcg_state_space(model, ws, C.byref(bt), layer, s, T * n_in, n_in, 0, st()),
           nbytes=T * (ssm.in_dim * 4.0 * s + ssm.out_dim * 2) + B * ssm.state_floats * 8.0,
           flops=2.0 * T * (ssm.heads * ssm.vdim * (32 + 2 * ssm.state) + ssm.groups * 32 * ssm.state) if prefill else 0.0)
+    k.add("norm", shape, lambda: lib.bcg_sandwich_norm(
+        b["residual"].data_ptr(), b["proj"].data_ptr(), s3, T * d, None, w["norm2"].data_ptr(), b["xn"].data_ptr(), L.DT_BF16, T, d,
+        1e-5, st()), nbytes=T * d * (10.0 + 4 * s3))
+    k.gemm("input product", shape, b["xn"], w["w_in"], b["proj"], T, n_in, d, L.EPI_F32, s)
     n_up = f.up_rows
     if prefill or splits(n_up, d) == 1:
         k.add("up product", shape, lambda: lib.bcg_gemm_bf16_glu(
@@ -313,11 +316,7 @@ def _merulorn_kernels(k: _Bench, what: str, B: int, T: int, shape: str, v, plan)
             b["proj"].data_ptr(), splits(n_up, d), T * n_up, b["act"].data_ptr(), L.DT_BF16, T, f.ff_ld, f.limit, f.alpha, st()),
             nbytes=T * f.ff_ld * (8.0 * splits(n_up, d) + 2))
     k.gemm("down product", shape, b["act"], w["w_down"], b["proj"], T, d, f.ff_ld, L.EPI_F32, splits(d, f.ff_ld))
-    s3 = splits(d, cols)
     k.gemm("output product", shape, b["mix"], w["w_out"], b["proj"], T, d, cols, L.EPI_F32, s3)
-    k.add("norm", shape, lambda: lib.bcg_sandwich_norm(
-        b["residual"].data_ptr(), b["proj"].data_ptr(), s3, T * d, None, w["norm2"].data_ptr(), b["xn"].data_ptr(), L.DT_BF16, T, d,
-        1e-5, st()), nbytes=T * d * (10.0 + 4 * s3))
 
 
 def _kernels(e: Engine, kind: str, hbm: float, tf: float) -> list:
