@@ -671,11 +671,12 @@ ssm_scan_kernel(const SsmArgs a) {
 // ------------------------------------------------------------------------------------------- chunks
 constexpr int kChTok = 64, kChWarps = 4, kChThreads = kChWarps * 32;
 
+// Tiles in shared memory are rows of 16-byte pieces, piece p of row r at place p ^ (r & 7).  B and x are there for two chunks.
 template <int NP>
 struct ChCfg {
-  static constexpr int kBRow = NP + 8, kXRow = kSsRows + 8, kMRow = kChTok + 8;       // pitches, bf16
-  static constexpr int kBC = kChTok * kBRow, kX = kChTok * kXRow, kM = kChTok * kMRow;
-  static constexpr int kSmem = (2 * kBC + kX + kM) * 2 + 2 * 4 * kChTok * 4;            // B, C, x, M, scalars
+  static constexpr int kBC = kChTok * NP * 2, kX = kChTok * kSsRows * 2, kM = kChTok * kChTok * 2;     // bytes
+  static constexpr int kOffC = 2 * kBC, kOffX = kOffC + kBC, kOffM = kOffX + 2 * kX, kOffS = kOffM + kM;
+  static constexpr int kSmem = kOffS + 2 * 4 * kChTok * 4 + 128;
   static constexpr int kCtasPerSm = NP <= 128 ? 3 : 2;
 };
 
@@ -704,23 +705,22 @@ __device__ __forceinline__ uint32_t transpose_8x8(uint32_t v) {
   return r;
 }
 
-// M[i][j] = exp(c_i - c_j) step_j (C_i . B_j) for j <= i, tokens i = 16 RT .. 16 RT + 15.
+// M[i][j] = exp(c_i - c_j) step_j (C_i . B_j) for j <= i, tokens i = 16 RT .. 16 RT + 15.  sB, sC, sM: addresses.
 template <int NP, int RT>
-__device__ __forceinline__ void chunk_matrix(const __nv_bfloat16* sB, const __nv_bfloat16* sC, const float* sum2,
-                                             const float* steps, __nv_bfloat16* sM) {
-  using C = ChCfg<NP>;
+__device__ __forceinline__ void chunk_matrix(uint32_t sB, uint32_t sC, const float* sum2, const float* steps, uint32_t sM) {
   const int lane = threadIdx.x & 31, q2 = (lane & 3) * 2;
   float acc[2 * RT + 2][4] = {};
-  const uint32_t pc = smem_u32(sC + (RT * 16 + (lane & 15)) * C::kBRow + (lane >> 4) * 8);
-  const uint32_t pb = smem_u32(sB + ((lane & 7) + ((lane >> 4) << 3)) * C::kBRow + ((lane >> 3) & 1) * 8);
+  const uint32_t pc = sC + (RT * 16 + (lane & 15)) * NP * 2, xc = ((lane >> 4) ^ (lane & 7)) << 4;
+  const uint32_t pb = sB + ((lane & 7) + ((lane >> 4) << 3)) * NP * 2, xb = (((lane >> 3) & 1) ^ (lane & 7)) << 4;
 #pragma unroll
   for (int k = 0; k < NP / 16; ++k) {
     uint32_t ca[4];
-    ldsm_at(ca, pc + k * 32);
+    ldsm_at(ca, pc + (xc ^ (k << 5)));
+    const uint32_t at = pb + (xb ^ (k << 5));
 #pragma unroll
     for (int jp = 0; jp <= RT; ++jp) {
       uint32_t bb[4];
-      ldsm_at(bb, pb + (jp * 16 * C::kBRow + k * 16) * 2);
+      ldsm_at(bb, at + jp * 16 * NP * 2);
       mma_bf16_16816(acc[2 * jp], ca, bb[0], bb[1]);
       mma_bf16_16816(acc[2 * jp + 1], ca, bb[2], bb[3]);
     }
@@ -740,7 +740,8 @@ __device__ __forceinline__ void chunk_matrix(const __nv_bfloat16* sB, const __nv
         if (j > i) m0 = 0.f;
         if (j + 1 > i) m1 = 0.f;
       }
-      *reinterpret_cast<uint32_t*>(sM + i * C::kMRow + j) = pack_bf16(m0, m1);
+      asm volatile("st.shared.b32 [%0], %1;" ::"r"(sM + i * kChTok * 2 + ((jt ^ (lane >> 2)) << 4) + q2 * 2), "r"(pack_bf16(m0, m1))
+                   : "memory");
     }
   }
 }
@@ -750,12 +751,10 @@ template <int NP>
 __global__ void __launch_bounds__(kChThreads, ChCfg<NP>::kCtasPerSm)
 ssm_chunk_kernel(const SsmArgs a) {
   using C = ChCfg<NP>;
-  extern __shared__ __align__(16) uint8_t ch_raw[];
-  __nv_bfloat16* sB = reinterpret_cast<__nv_bfloat16*>(ch_raw);
-  __nv_bfloat16* sC = sB + C::kBC;
-  __nv_bfloat16* sX = sC + C::kBC;
-  __nv_bfloat16* sM = sX + C::kX;
-  float* scalars = reinterpret_cast<float*>(sM + C::kM);     // [2][4][64]: log2 decay sums, steps, e, w
+  extern __shared__ __align__(128) uint8_t ch_raw[];
+  const uint32_t base = (smem_u32(ch_raw) + 127u) & ~127u;
+  float* scalars = reinterpret_cast<float*>(ch_raw + (base - smem_u32(ch_raw)) + C::kOffS);     // [2][4][64]: log2 decay sums, steps, e, w
+  const uint32_t sC = base + C::kOffC, sM = base + C::kOffM;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int h = blockIdx.x, p0 = blockIdx.y * kSsRows, sq = blockIdx.z;
   const int rows = min(kSsRows, a.vdim - p0), N = a.n, g = h / (a.heads / a.groups), inner = a.inner();
@@ -767,16 +766,17 @@ ssm_chunk_kernel(const SsmArgs a) {
   const __nv_bfloat16* xbc = static_cast<const __nv_bfloat16*>(a.x);
   const int x_ld = a.x_ld(), b_col = a.b_col(g), c_col = a.c_col(g), x_col = h * a.x_pad() + p0;
 
-  // 64 tokens from `first` on, up to 8 UNITS columns from `col` on, `valid` of them; the rest and tokens past the end are zero
-  auto copy_rows = [&](auto units, __nv_bfloat16* dst, int pitch, int col, int valid, int first) {
+  // 64 tokens from `first` on, up to 8 `units` columns from `col` on, `valid` of them; the rest and tokens past the end are
+  // zero
+  auto copy_rows = [&](auto units, uint32_t dst, int col, int valid, int first) {
     constexpr int kUnits = decltype(units)::value, kPass = kChThreads / kUnits;
     const int u = threadIdx.x % kUnits, r = threadIdx.x / kUnits, wide = max(0, min(16, (valid - u * 8) * 2));
     const __nv_bfloat16* src = xbc + static_cast<long long>(first + r) * x_ld + col + u * 8;
-    const uint32_t to = smem_u32(dst + r * pitch + u * 8);
 #pragma unroll
     for (int i = 0; i < kChTok / kPass; ++i) {
-      const int bytes = first + r + i * kPass < t1 ? wide : 0;
-      asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(to + i * kPass * pitch * 2), "l"(bytes ? src : xbc), "r"(bytes)
+      const int row = r + i * kPass, bytes = first + row < t1 ? wide : 0;
+      asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst + row * kUnits * 16 + ((u ^ (row & 7)) << 4)),
+                   "l"(bytes ? src : xbc), "r"(bytes)
                    : "memory");
       src += static_cast<long long>(kPass) * x_ld;
     }
@@ -789,9 +789,9 @@ ssm_chunk_kernel(const SsmArgs a) {
   const int pr = warp * 16 + (lane >> 2);       // this lane's rows of the state: pr, pr + 8; entries nt * 8 + 2 (lane & 3) ..
   const int q2 = (lane & 3) * 2;
   float* st = a.state + ((static_cast<long long>(a.state_slots[sq]) * a.heads + h) * a.vdim + p0) * N;
-  copy_rows(BCUnits{}, sB, C::kBRow, b_col, N, t0);
-  copy_rows(BCUnits{}, sC, C::kBRow, c_col, N, t0);
-  copy_rows(XUnits{}, sX, C::kXRow, x_col, rows, t0);
+  copy_rows(BCUnits{}, base, b_col, N, t0);
+  copy_rows(BCUnits{}, sC, c_col, N, t0);
+  copy_rows(XUnits{}, base + C::kOffX, x_col, rows, t0);
   cp_async_commit();
   float S[NP / 8][4];
   const bool fresh = a.positions[t0] == 0;
@@ -834,7 +834,12 @@ ssm_chunk_kernel(const SsmArgs a) {
     const float* sum2 = scalars + (c & 1) * 4 * kChTok;
     const float *steps = sum2 + kChTok, *e_s = steps + kChTok, *w_s = e_s + kChTok;
     cp_async_wait<0>();
-    __syncthreads();                            // the chunk is there
+    __syncthreads();                            // the chunk is there, everybody is done with the previous one
+    const uint32_t sB = base + (c & 1) * C::kBC, sX = base + C::kOffX + (c & 1) * C::kX;
+    if (c + 1 < n_chunks) {
+      copy_rows(BCUnits{}, base + ((c + 1) & 1) * C::kBC, b_col, N, first + kChTok);
+      copy_rows(XUnits{}, base + C::kOffX + ((c + 1) & 1) * C::kX, x_col, rows, first + kChTok);
+    }
 
     if (warp * 16 < nt_tok) {
       if (warp == 0) chunk_matrix<NP, 0>(sB, sC, sum2, steps, sM);
@@ -846,7 +851,8 @@ ssm_chunk_kernel(const SsmArgs a) {
 
     // ---- Y^T = S^T C^T, columns (tokens) scaled by exp(c_i)
     float Y[kChTok / 8][4] = {};
-    const uint32_t pc = smem_u32(sC + ((lane & 7) + ((lane >> 4) << 3)) * C::kBRow + ((lane >> 3) & 1) * 8);
+    const uint32_t r8 = (lane & 7) + ((lane >> 4) << 3), x8 = (((lane >> 3) & 1) ^ (lane & 7)) << 4;
+    const uint32_t pc = sC + r8 * NP * 2;
 #pragma unroll
     for (int k = 0; k < NP / 16; ++k) {
       const uint32_t sa[4] = {pack_bf16(S[2 * k][0], S[2 * k][1]), pack_bf16(S[2 * k][2], S[2 * k][3]),
@@ -854,7 +860,7 @@ ssm_chunk_kernel(const SsmArgs a) {
 #pragma unroll
       for (int ip = 0; ip < kChTok / 16; ++ip) {
         uint32_t cb[4];
-        ldsm_at(cb, pc + (ip * 16 * C::kBRow + k * 16) * 2);
+        ldsm_at(cb, pc + (x8 ^ (k << 5)) + ip * 16 * NP * 2);
         mma_bf16_16816(Y[2 * ip], sa, cb[0], cb[1]);
         mma_bf16_16816(Y[2 * ip + 1], sa, cb[2], cb[3]);
       }
@@ -872,21 +878,22 @@ ssm_chunk_kernel(const SsmArgs a) {
       scale2(S[nt][2], S[nt][3], keep, keep);
     }
     __syncthreads();                            // M is complete, C has been read
-    if (c + 1 < n_chunks) copy_rows(BCUnits{}, sC, C::kBRow, c_col, N, first + kChTok);
+    if (c + 1 < n_chunks) copy_rows(BCUnits{}, sC, c_col, N, first + kChTok);
+    cp_async_commit();
 
     // ---- Y^T += x^T M^T + skip x^T;   S^T += (w x)^T B
-    const uint32_t px = smem_u32(sX + ((lane & 7) + ((lane >> 4) << 3)) * C::kXRow + warp * 16 + ((lane >> 3) & 1) * 8);
-    const uint32_t pb = smem_u32(sB + (lane & 15) * C::kBRow + (lane >> 4) * 8);
-    const uint32_t pm = smem_u32(sM + ((lane & 7) + ((lane >> 4) << 3)) * C::kMRow + ((lane >> 3) & 1) * 8);
+    const uint32_t px = sX + r8 * kSsRows * 2 + (x8 ^ (warp << 5));
+    const uint32_t pb = sB + (lane & 15) * NP * 2, xb = ((lane >> 4) ^ (lane & 7)) << 4;
+    const uint32_t pm = sM + r8 * kChTok * 2;
 #pragma unroll
     for (int jp = 0; jp < kChTok / 16; ++jp) {
       uint32_t xa[4];
-      ldsm_trans_at(xa, px + jp * 16 * C::kXRow * 2);
+      ldsm_trans_at(xa, px + jp * 16 * kSsRows * 2);
 #pragma unroll
       for (int ip = jp; ip < kChTok / 16; ++ip)
         if (ip * 16 < nt_tok) {
           uint32_t mb[4];
-          ldsm_at(mb, pm + (ip * 16 * C::kMRow + jp * 16) * 2);
+          ldsm_at(mb, pm + (x8 ^ (jp << 5)) + ip * 16 * kChTok * 2);
           mma_bf16_16816(Y[2 * ip], xa, mb[0], mb[1]);
           mma_bf16_16816(Y[2 * ip + 1], xa, mb[2], mb[3]);
         }
@@ -912,8 +919,8 @@ ssm_chunk_kernel(const SsmArgs a) {
 #pragma unroll
       for (int np = 0; np < NP / 16; np += 2) {
         uint32_t b0[4], b1[4];
-        ldsm_trans_at(b0, pb + (jp * 16 * C::kBRow + np * 16) * 2);
-        ldsm_trans_at(b1, pb + (jp * 16 * C::kBRow + np * 16 + 16) * 2);
+        ldsm_trans_at(b0, pb + (xb ^ (np << 5)) + jp * 16 * NP * 2);
+        ldsm_trans_at(b1, pb + (xb ^ ((np + 1) << 5)) + jp * 16 * NP * 2);
         mma_bf16_16816(S[2 * np], hi, b0[0], b0[1]);
         mma_bf16_16816(S[2 * np + 1], hi, b0[2], b0[3]);
         mma_bf16_16816(S[2 * np + 2], hi, b1[0], b1[1]);
@@ -923,12 +930,6 @@ ssm_chunk_kernel(const SsmArgs a) {
         mma_bf16_16816(S[2 * np + 2], lo, b1[0], b1[1]);
         mma_bf16_16816(S[2 * np + 3], lo, b1[2], b1[3]);
       }
-    }
-    __syncthreads();                            // B and x have been read
-    if (c + 1 < n_chunks) {
-      copy_rows(BCUnits{}, sB, C::kBRow, b_col, N, first + kChTok);
-      copy_rows(XUnits{}, sX, C::kXRow, x_col, rows, first + kChTok);
-      cp_async_commit();
     }
 
     // ---- store: pairs are transposed on the way out (token lane >> 2, entries q2, q2 + 1)
@@ -1090,8 +1091,9 @@ static int run_np(const SsmArgs& a, int n_seqs, bool one_token, bool chunks, cud
   } else if (one_token) {
     BCG_CUDA_CHECK(launch_k(ssm_token_kernel<T, NP>, grid, dim3(kSsThreads), 0, st, a));
   } else if (chunks) {
-    BCG_TRY(ensure_dynamic_smem(reinterpret_cast<const void*>(ssm_chunk_kernel<NP>), ChCfg<NP>::kSmem));
-    BCG_CUDA_CHECK(launch_k(ssm_chunk_kernel<NP>, grid, dim3(kChThreads), ChCfg<NP>::kSmem, st, a));
+    constexpr int P = NP < 64 ? 64 : NP;
+    BCG_TRY(ensure_dynamic_smem(reinterpret_cast<const void*>(ssm_chunk_kernel<P>), ChCfg<P>::kSmem));
+    BCG_CUDA_CHECK(launch_k(ssm_chunk_kernel<P>, grid, dim3(kChThreads), ChCfg<P>::kSmem, st, a));
   } else {
     BCG_CUDA_CHECK(launch_k(ssm_scan_kernel<T, NP>, grid, dim3(kSsThreads), 0, st, a));
   }
