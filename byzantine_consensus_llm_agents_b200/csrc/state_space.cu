@@ -1012,7 +1012,7 @@ ssm_norm_kernel(const SsmArgs a, T* __restrict__ out, long long out_ld) {
 
 // Prompts, one slab: a part of a token's outputs per warp, NV vectors of four per lane.
 template <typename T, int NV>
-__global__ void __launch_bounds__(kSnThreads)
+__global__ void __launch_bounds__(kSnThreads, NV <= 8 ? 4 : 2)
 ssm_norm_warp_kernel(const SsmArgs a, T* __restrict__ out, long long out_ld) {
   pdl_launch_dependents();
   pdl_wait();

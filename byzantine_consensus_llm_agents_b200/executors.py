@@ -335,15 +335,18 @@ class StackExecutor:
         L.check(self.lib.bcg_stack_head(C.byref(self.model.struct), C.byref(self.ws), v["rows"].data_ptr() + 4 * first, n,
                                         row0, self.flags & L.GEMM_PDL, L.stream_ptr()), "bcg_stack_head")
 
-    def _launches_per_step(self) -> int:
-        n = 1
+    def _launches_per_step(self, decode: bool) -> int:
+        n, d = 1, self.cfg.d_model
         for l in self.cfg.layers:
             if l.parallel:   # input projection, its split, attention, output projection, norm; scatter, two products, gate
                 n += 5 + (4 if isinstance(l.mlp, MoeMlp) else 0)
                 continue
-            if l.composed:   # input projection, attention's split and kernel, the state-space mixer's two (portions: three)
-                # kernels, output projection, norm; feed-forward: up with its unit (in its epilogue or not), down, norm
-                n += 3 + (2 if l.one(GroupedAttention) else 0) + (2 if l.one(StateSpace) else 0) + (3 if l.mlp else 0)
+            if l.composed:
+                # input projection, attention's split and kernel, state space (convolution,) recurrence and norm, output
+                # projection, norm; feed-forward: up, its unit where K is split, down, norm
+                n += 3 + (2 if l.one(GroupedAttention) else 0) + ((2 if decode else 3) if l.one(StateSpace) else 0)
+                if l.mlp:
+                    n += 3 + int(not l.mlp.glu or decode and L.splits_for(1, l.mlp.up_rows, d) > 1)
                 continue
             # input projection, mixer (delta: low rank, decay projection, scan; attention: qkv, absorb, decode,
             # combine, up), output projection, norm; feed-forward: up, activation, down, norm
@@ -351,7 +354,7 @@ class StackExecutor:
         return n
 
     def launches_prefill(self) -> int:
-        return self._launches_per_step() + 2
+        return self._launches_per_step(False) + 2
 
     def decode(self, row: dict, B: int, max_splits: int) -> None:
         b = self._batch(B, B)
@@ -363,7 +366,7 @@ class StackExecutor:
                                         self.flags & L.GEMM_PDL, L.stream_ptr()), "bcg_stack_head")
 
     def launches_per_decode_step(self, B: int) -> int:
-        return self._launches_per_step() + 1
+        return self._launches_per_step(True) + 1
 
 
 def make_executor(cfg, lcfg, weights, dev, **kw):
