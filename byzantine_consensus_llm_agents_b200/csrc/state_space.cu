@@ -61,6 +61,11 @@ struct SsmArgs {
 };
 
 __device__ __forceinline__ float silu_f32(float x) { return x * sigmoid_f32(x); }
+// silu of what becomes an activation of type T: the short exponential where that is rounded to bf16
+template <typename T>
+__device__ __forceinline__ float silu_act(float x) {
+  return sizeof(T) == 2 ? __fdividef(x, 1.0f + __expf(-x)) : silu_f32(x);
+}
 __device__ __forceinline__ float softplus_f32(float x) { return fmaxf(x, 0.f) + log1pf(expf(-fabsf(x))); }
 // rounded once near 1: a state that decays slowly would drift with the error of exp
 __device__ __forceinline__ float decay_f32(float x) { return 1.0f + expm1f(x); }
@@ -84,7 +89,7 @@ constexpr int kConvAhead = 4;     // inputs in flight per thread
 
 // TAPS: a window of inputs in registers; 0: any number of taps, every input loaded where it is used.  ONE: one slab.
 template <typename T, int V, int TAPS, bool ONE>
-__global__ void __launch_bounds__(kConvThreads)
+__global__ void __launch_bounds__(kConvThreads, V == 4 ? 8 : 12)
 ssm_conv_kernel(const SsmArgs a, int run, int conv_blocks) {
   pdl_launch_dependents();
   pdl_wait();
@@ -145,7 +150,7 @@ ssm_conv_kernel(const SsmArgs a, int run, int conv_blocks) {
           }
         }
 #pragma unroll
-        for (int i = 0; i < V; ++i) y.x[i] = silu_f32(y.x[i]);
+        for (int i = 0; i < V; ++i) y.x[i] = silu_act<T>(y.x[i]);
         store_vec<V>(out + static_cast<long long>(t + j) * x_ld, y);
       }
     }
@@ -987,7 +992,7 @@ ssm_norm_kernel(const SsmArgs a, T* __restrict__ out, long long out_ld) {
     Vec<V> u = load_vec<V>(y + v);
     const Vec<V> g = slab_sum_vec<V>(z + v, a.n_partials, a.pstride);
 #pragma unroll
-    for (int k = 0; k < V; ++k) u.x[k] *= silu_f32(g.x[k]);
+    for (int k = 0; k < V; ++k) u.x[k] *= silu_act<T>(g.x[k]);
     store_vec<V>(stage + v - v0, u);
     ss[0] += u.sumsq();
   }
@@ -1034,7 +1039,7 @@ ssm_norm_warp_kernel(const SsmArgs a, T* __restrict__ out, long long out_ld) {
 #pragma unroll
   for (int i = 0; i < NV; ++i) {
 #pragma unroll
-    for (int k = 0; k < 4; ++k) u[i].x[k] *= silu_f32(g[i].x[k]);
+    for (int k = 0; k < 4; ++k) u[i].x[k] *= silu_act<T>(g[i].x[k]);
     if ((i * 32 + lane) * 4 < width) ss += u[i].sumsq();
   }
   const float inv = rsqrtf(warp_sum(ss) / static_cast<float>(width) + a.eps);
