@@ -78,7 +78,8 @@ class OneLayer:
 SIZES = {  # heads, vdim, state, groups, norm_groups, conv
     "usual": (4, 64, 128, 2, 2, 4), "small": (4, 16, 16, 4, 1, 4), "blocks": (2, 136, 64, 1, 2, 3), "wide": (2, 64, 256, 1, 1, 2),
     "odd": (3, 11, 13, 3, 3, 4), "halves": (2, 66, 50, 1, 4, 5), "one": (1, 8, 8, 1, 1, 1), "parts": (8, 24, 36, 2, 48, 4), "row": (2, 1, 200, 2, 2, 3),
-    "many": (72, 16, 20, 8, 4, 3), "many-blocks": (40, 72, 24, 4, 1, 5)}
+    "many": (72, 16, 20, 8, 4, 3), "many-blocks": (40, 72, 24, 4, 1, 5),
+    "large-part": (16, 72, 16, 2, 1, 2), "larger-part": (40, 56, 8, 1, 1, 3)}
 
 
 class StateSpace(OneLayer):
