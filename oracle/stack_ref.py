@@ -5,7 +5,10 @@ attention with a sliding window and a sink, generalized delta rule, PolyNorm fee
 both sides of each sublayer; Lerazen: grouped-query attention with a linear distance bias, a query
 temperature and values mixed with an earlier layer's, squared-relu and mixture-of-experts
 feed-forwards, parallel sublayers, learned positions; Merulorn: attention with whole-projection query and key
-norms and a gate per head beside a selective state-space mixer, clamped gated units, sinusoidal positions).  One function per mechanism; torch on the CPU, in the dtype of its
+norms and a gate per head beside a selective state-space mixer, clamped gated units, sinusoidal positions;
+Vosolorn: attention with rotated values over a window and means of the blocks in front of it, a matrix memory with
+exponential gates, gelu units, a mixture of plain experts with a shared one, norms and scales on the sublayers'
+outputs only).  One function per mechanism; torch on the CPU, in the dtype of its
 inputs (the tests use float64, rounding weights only).  A whole sequence is computed at once, token by
 token where there is a recurrence, with no cache: what a cache, a batch or a cut of the prompt could get
 wrong is absent here by construction.
@@ -308,6 +311,136 @@ def _merulorn(config, T, tokens, collect):
     return zero_norm(x, eps, T["final.norm"]) @ T["head"].T
 
 
+def rotate_pairs(x, positions, dims, base, back=False):
+    """Pairs (2i, 2i + 1) of the first `dims` entries of the last axis turn by position * base^(-2i / dims), or back."""
+    y = x.clone()
+    for i in range(dims // 2):
+        a = positions.to(torch.float64) * float(base) ** (-2.0 * i / dims)
+        if back:
+            a = -a
+        shape = (x.shape[0],) + (1,) * (x.dim() - 2)
+        cos, sin = a.cos().to(x.dtype).view(shape), a.sin().to(x.dtype).view(shape)
+        u, v = x[..., 2 * i], x[..., 2 * i + 1]
+        y[..., 2 * i], y[..., 2 * i + 1] = u * cos - v * sin, v * cos + u * sin
+    return y
+
+
+def block_means(x, pool):
+    """[t // pool, ...]: means of whole blocks of `pool` tokens."""
+    n = x.shape[0] // pool
+    return x[:n * pool].reshape(n, pool, *x.shape[1:]).mean(1)
+
+
+def blocks_visible(n, n_blocks, size, pool):
+    """[query, block] boolean: the whole block has left the window of `size` tokens."""
+    i, b = torch.arange(n)[:, None], torch.arange(n_blocks)[None, :]
+    return b * pool + pool - 1 <= i - size
+
+
+def pooled_attention(h, w, m, positions, eps):
+    """m: dict(heads, kv_heads, dim, vdim, scale, size, pool, dims, base).  Query and key norms per head, rotated queries,
+    keys and values; tokens of a window and means of the blocks in front of it share one softmax."""
+    t, H, G = h.shape[0], m["heads"], m["kv_heads"]
+    q = rotate_pairs(rms_norm((h @ w["q"].T).view(t, H, m["dim"]), eps, w["q.norm"]), positions, m["dims"], m["base"])
+    k = rotate_pairs(rms_norm((h @ w["k"].T).view(t, G, m["dim"]), eps, w["k.norm"]), positions, m["dims"], m["base"])
+    v = rotate_pairs((h @ w["v"].T).view(t, G, m["vdim"]), positions, m["vdim"], m["base"])
+    ok = window_visible(t, m["size"])
+    if m["pool"]:
+        kb, vb = block_means(k, m["pool"]), block_means(v, m["pool"])
+        ok = torch.cat([ok, blocks_visible(t, kb.shape[0], m["size"], m["pool"])], dim=1)
+        k, v = torch.cat([k, kb]), torch.cat([v, vb])
+    mine = torch.arange(H) // (H // G)
+    s = torch.einsum("ihd,jhd->hij", q, k[:, mine]) * m["scale"]
+    o = torch.einsum("hij,jhd->ihd", softmax_with_sink(s, ok), v[:, mine])
+    return rotate_pairs(o, positions, m["vdim"], m["base"], back=True).reshape(t, H * m["vdim"]) @ w["o"].T
+
+
+def memory_gates(h, w, cap):
+    """(log input gate, log forget gate), both [t, heads]."""
+    soft = lambda z: cap * torch.tanh(z / cap)
+    return soft(h @ w["i"].T + w["i.b"]), torch.nn.functional.logsigmoid(soft(h @ w["f"].T + w["f.b"]))
+
+
+def memory_scan(q, k, v, log_i, log_f, state=None):
+    """q (scaled) and k [t, heads, dim], v [t, heads, vdim], gates [t, heads].  Token by token with a running maximum m of
+    the gates, which starts at 0.  Returns (o [t, heads, vdim], (S [heads, dim, vdim], n [heads, dim], m [heads]))."""
+    t, H, D = k.shape
+    S, n, m = (torch.zeros(H, D, v.shape[2], dtype=q.dtype), torch.zeros(H, D, dtype=q.dtype),
+               torch.zeros(H, dtype=q.dtype)) if state is None else state
+    out = []
+    for i in range(t):
+        top = torch.maximum(log_f[i] + m, log_i[i])
+        keep, add, m = torch.exp(log_f[i] + m - top), torch.exp(log_i[i] - top), top
+        S = keep[:, None, None] * S + add[:, None, None] * k[i][:, :, None] * v[i][:, None, :]
+        n = keep[:, None] * n + add[:, None] * k[i]
+        den = torch.maximum((n * q[i]).sum(-1).abs(), torch.exp(-m)) + 1e-6
+        out.append(torch.einsum("hde,hd->he", S, q[i]) / den[:, None])
+    return torch.stack(out), (S, n, m)
+
+
+def matrix_memory(h, w, m, eps):
+    """m: dict(heads, dim, vdim, cap)."""
+    t, H = h.shape[0], m["heads"]
+    q, k = (h @ w["q"].T).view(t, H, -1) * m["dim"] ** -0.5, (h @ w["k"].T).view(t, H, -1)
+    log_i, log_f = memory_gates(h, w, m["cap"])
+    o, _ = memory_scan(q, k, (h @ w["v"].T).view(t, H, -1), log_i, log_f)
+    o = rms_norm(o, eps).reshape(t, H * m["vdim"]) * w["norm"]
+    return (o * torch.sigmoid(h @ w["g"].T)) @ w["o"].T
+
+
+def gelu_tanh(z):
+    return 0.5 * z * (1 + torch.tanh(math.sqrt(2 / math.pi) * (z + 0.044715 * z ** 3)))
+
+
+def gelu_erf(z):
+    return 0.5 * z * (1 + torch.erf(z / math.sqrt(2)))
+
+
+def route_softmax(h, router, bias, top):
+    """(experts [t, top], weights [t, top]): the largest logits and the softmax over just them."""
+    best = torch.topk(h @ router.T + bias, top, dim=-1)
+    e = torch.exp(best.values - best.values.max(-1, keepdim=True).values)
+    return best.indices, e / e.sum(-1, keepdim=True)
+
+
+def plain_mixture(h, w, top):
+    """Experts without gates, weighted outputs, and a shared expert where there is one."""
+    experts, weights = route_softmax(h, w["router"], w["router.b"], top)
+    unit = lambda x, p: w[p + "down"] @ gelu_erf(w[p + "up"] @ x)
+    out = torch.zeros_like(h)
+    for t in range(h.shape[0]):
+        for e, s in zip(experts[t].tolist(), weights[t]):
+            out[t] += s * unit(h[t], f"e{e}.")
+        if "shared.up" in w:
+            out[t] += unit(h[t], "shared.")
+    return out
+
+
+def _vosolorn(config, T, tokens, collect):
+    eps, pos = float(config["norm"]["eps"]), torch.arange(len(tokens))
+    x = rms_norm(T["embed"][torch.as_tensor(tokens, dtype=torch.long)], eps, T["embed.norm"])
+    for i, layer in enumerate(config["layers"]):
+        p, mix, mlp = f"l{i}.", layer["mixer"], layer.get("mlp")
+        sub = lambda kind: {n[len(p + kind) + 1:]: t for n, t in T.items() if n.startswith(p + kind + ".")}
+        if layer["type"] == "attention":
+            mask, rot = mix.get("mask") or {"size": 0}, mix["rot"]
+            m = {**mix, "size": mask["size"], "pool": mask.get("pool", 0), "dims": rot["dims"], "base": rot["base"]}
+            y = pooled_attention(x, sub("mix"), m, pos, eps)
+        elif layer["type"] == "mlstm":
+            y = matrix_memory(x, sub("mix"), {**mix, "cap": mix["gate_cap"]}, eps)
+        else:
+            raise ValueError(f"unknown mixer {layer['type']!r}")
+        x = x + rms_norm(y, eps, T[p + "norm1"]) * T[p + "ls1"]
+        if mlp:
+            w = sub("mlp")
+            y = plain_mixture(x, w, mlp["router"]["top"]) if mlp["kind"] == "moe" \
+                else (gelu_tanh(x @ w["gate"].T) * (x @ w["up"].T)) @ w["down"].T
+            x = x + rms_norm(y, eps, T[p + "norm2"]) * T[p + "ls2"]
+        if collect is not None:
+            collect.append(x.clone())
+    return rms_norm(x, eps, T["final.norm"]) @ T["embed"].T * config["logit_scale"]
+
+
 def forward(config, tensors, tokens, collect=None, dtype=torch.float64):
     """Logits [tokens, vocab] of one sequence.  `config` is the parsed config.json, `tensors` name -> tensor.
     `collect`: a list that receives the residual stream after every layer."""
@@ -317,6 +450,8 @@ def forward(config, tensors, tokens, collect=None, dtype=torch.float64):
         return _lerazen(config, T, tokens, collect)
     if config["architecture"] == "Merulorn":
         return _merulorn(config, T, tokens, collect)
+    if config["architecture"] == "Vosolorn":
+        return _vosolorn(config, T, tokens, collect)
     pos = torch.arange(len(tokens))
     x = T["embed"][torch.as_tensor(tokens, dtype=torch.long)]
     kv = {}
