@@ -38,6 +38,7 @@ SOURCES = [
     "grouped_attn.cu",
     "grouped_prefill.cu",
     "state_space.cu",
+    "matrix_memory.cu",
     "moe.cu",
     "delta_scan.cu",
     "stack_step.cu",

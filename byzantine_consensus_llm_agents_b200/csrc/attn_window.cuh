@@ -1,6 +1,7 @@
 // Prompt attention on tcgen05: 128 query rows of one head against keys in blocks of 64, causal with an optional
 // sliding window.  Options: a softmax sink, a linear distance bias per head (SLOPES), keys and values read from
-// contiguous rows or through a block table of 16-token pages (PAGED).
+// contiguous rows or through a block table of 16-token pages (PAGED); with pages and without a bias, blocks of means
+// of the tokens in front of the window, which have pages of their own, and outputs turned back by the query's position.
 //
 //   grid (heads, tiles), 192 threads; keys from the first one any row of the tile sees.
 //     warp 0      TMA producer: Q tile once, then K and V blocks (64-column boxes of 64 rows, or of the 16 rows
@@ -55,6 +56,15 @@ __device__ __forceinline__ void load_block(uint8_t* dst, const CUtensorMap* map,
   }
 }
 
+// Means of blocks of `pool` tokens that a query sees beside its window: block b from position b * pool + pool - 1 + window on.
+struct PooledKeys {
+  int pool, col;            // col: first column of their pages in the block table; pool = 0: none
+  __device__ __forceinline__ int visible(int pos, int window) const {
+    const int gone = pos - window + 1;             // tokens in front of the window
+    return pool > 0 && gone >= pool ? gone / pool : 0;
+  }
+};
+
 struct WindowAttn {
   const int* tiles;
   int n_tiles;
@@ -65,11 +75,41 @@ struct WindowAttn {
   int k_col, v_col;         // contiguous rows: columns per head of a key / first column of the values
   int group;                // query heads per key/value head
   const float* gates;       // [tokens][heads] factors of the outputs, or NULL
+  PooledKeys pooled;        // PAGED without SLOPES only
+  const float* v_cos_sin;   // outputs turn back in pairs of neighbours, or NULL
+  int v_rot_dims;
   __nv_bfloat16* out;
   long long out_ld;         // row pitch
   int heads, vdim, window;
   float scale_log2e;
 };
+
+// Columns c0 .. c0 + 31 of an output row turned back: pairs (2m, 2m + 1), cosines at m of the table's row, sines at dims / 2 + m.
+__device__ __forceinline__ void turn_back(uint32_t (&o)[32], const float* row, int dims, int c0) {
+  const int half = dims / 2;
+#pragma unroll
+  for (int i = 0; i < 16; i += 4) {
+    const int m = c0 / 2 + i;
+    float cs[4], sn[4];
+    if (m + 4 <= half && dims % 8 == 0) {
+      const float4 c = __ldg(reinterpret_cast<const float4*>(row + m)), s = __ldg(reinterpret_cast<const float4*>(row + half + m));
+      cs[0] = c.x; cs[1] = c.y; cs[2] = c.z; cs[3] = c.w;
+      sn[0] = s.x; sn[1] = s.y; sn[2] = s.z; sn[3] = s.w;
+    } else {
+#pragma unroll
+      for (int k = 0; k < 4; ++k) {
+        cs[k] = m + k < half ? row[m + k] : 1.f;
+        sn[k] = m + k < half ? row[half + m + k] : 0.f;
+      }
+    }
+#pragma unroll
+    for (int k = 0; k < 4; ++k) {
+      const float u = __uint_as_float(o[2 * (i + k)]), v = __uint_as_float(o[2 * (i + k) + 1]);
+      o[2 * (i + k)] = __float_as_uint(u * cs[k] + v * sn[k]);
+      o[2 * (i + k) + 1] = __float_as_uint(v * cs[k] - u * sn[k]);
+    }
+  }
+}
 
 template <int QD, int VD, bool PAGED, bool SLOPES>
 __global__ void __launch_bounds__(kWaThreads, WaCfg<QD, VD>::kCtasPerSm)
@@ -130,7 +170,10 @@ window_attn_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_const
   const int first = max(window > 0 ? pos0 - window + 1 : 0, PAGED ? 0 : ti[4]);
   const int kb = PAGED ? first & ~(kWaPage - 1) : first;
   const int kv_row = ti[3] + kb - ti[4];
-  const int nb = (pos0 + n_rows - kb + kWaBN - 1) / kWaBN;
+  const int nb_tok = (pos0 + n_rows - kb + kWaBN - 1) / kWaBN;
+  constexpr bool kPools = PAGED && !SLOPES;
+  const int n_pooled = kPools ? a.pooled.visible(pos0 + n_rows - 1, window) : 0;    // pooled blocks come behind the tokens
+  const int nb = nb_tok + (n_pooled + kWaBN - 1) / kWaBN;
   // With a distance bias the newest keys usually hold the maximum: they come first, so that O is rarely rescaled.
   auto block_at = [&](int j) { return SLOPES ? nb - 1 - j : j; };
   tc_fence_before();
@@ -154,8 +197,12 @@ window_attn_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_const
         int prow[kWaBN / kWaPage];      // PAGED: first row of every page of the block
         if constexpr (PAGED) {
 #pragma unroll
-          for (int pg = 0; pg < kWaBN / kWaPage; ++pg)
-            prow[pg] = (bt[min((kb + jb * kWaBN) / kWaPage + pg, last_page)] * a.page_heads + kvh) * kWaPage;
+          for (int pg = 0; pg < kWaBN / kWaPage; ++pg) {
+            int at = min((kb + jb * kWaBN) / kWaPage + pg, last_page);
+            if (kPools && jb >= nb_tok)
+              at = a.pooled.col + min((jb - nb_tok) * (kWaBN / kWaPage) + pg, (n_pooled - 1) / kWaPage);
+            prow[pg] = (bt[at] * a.page_heads + kvh) * kWaPage;
+          }
         }
         uint8_t* dk = smem + C::kOffK + st * C::kK;
         mbar_wait(&k_empty[st], par ^ 1);
@@ -213,8 +260,8 @@ window_attn_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_const
     const int q4 = warp & 3;
     const int r = q4 * 32 + lane;
     const uint32_t lane_addr = static_cast<uint32_t>(q4 * 32) << 16;
-    const int limit = pos0 + r - kb;                                   // last visible key, counted from kb
-    const int low = window > 0 ? max(0, pos0 + r - window + 1 - kb) : 0;   // first visible key
+    const int tok_limit = pos0 + r - kb;                                   // last visible key, counted from kb
+    const int tok_low = window > 0 ? max(0, pos0 + r - window + 1 - kb) : 0;   // first visible key
     uint8_t* p_row = smem + C::kOffP + r * 128;
     const int sw = r & 7;
     float m_run = a.sink ? a.sink[head] * 1.4426950408889634f : kWaNoSink;
@@ -222,7 +269,9 @@ window_attn_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_const
     const float slope = SLOPES ? a.slopes[head] * 1.4426950408889634f : 0.f;
     const uint64_t scale2 = pack_f32x2(__float_as_uint(a.scale_log2e), __float_as_uint(a.scale_log2e));
     for (int j = 0; j < nb; ++j) {
-      const int col0 = block_at(j) * kWaBN;
+      const bool pooled = kPools && j >= nb_tok;
+      const int col0 = pooled ? (j - nb_tok) * kWaBN : block_at(j) * kWaBN;
+      const int limit = pooled ? a.pooled.visible(pos0 + r, window) - 1 : tok_limit, low = pooled ? 0 : tok_low;
       const bool need_mask = col0 + kWaBN - 1 > limit || col0 < low;
       mbar_wait(&s_full[j & 1], (j >> 1) & 1);
       tc_fence_after();
@@ -313,6 +362,9 @@ window_attn_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_const
       tmem_ld_x32(tmem_o + lane_addr + c * 32, o);
       tmem_ld_wait();
       if (r < n_rows) {
+        if constexpr (kPools) {
+          if (a.v_cos_sin) turn_back(o, a.v_cos_sin + static_cast<long long>(pos0 + r) * a.v_rot_dims, a.v_rot_dims, c * 32);
+        }
 #pragma unroll
         for (int g = 0; g < 4; ++g)
           if (c * 32 + g * 8 < a.vdim) {

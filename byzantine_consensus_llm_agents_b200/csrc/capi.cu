@@ -229,16 +229,18 @@ int bcg_sandwich_norm(float* residual, const float* delta, int n_partials, long 
 }
 
 int bcg_residual_norm(float* residual, const float* delta, int n_partials, long long partial_stride, const float* bias,
-                      const float* rows, const int* index, int per_row, int row_partials, long long row_stride,
-                      const float* w_next, void* xn, int act_dtype, int T, int d, float eps, void* stream) {
+                      const float* rows, const int* index, const float* weight, int per_row, int row_partials,
+                      long long row_stride, const float* w_post, const float* w_next, void* xn, int act_dtype, int T, int d,
+                      float eps, void* stream) {
   NormExtra extra;
+  extra.weight = weight;
   extra.bias = bias;
   extra.rows = rows;
   extra.index = index;
   extra.per_row = rows && index ? per_row : 0;
   extra.n_partials = row_partials;
   extra.partial_stride = row_stride;
-  return sandwich_norm(residual, delta, n_partials, partial_stride, nullptr, w_next, xn, act_dtype, T, d, eps, extra,
+  return sandwich_norm(residual, delta, n_partials, partial_stride, w_post, w_next, xn, act_dtype, T, d, eps, extra,
                        S(stream));
 }
 
@@ -293,12 +295,46 @@ int bcg_state_space(const bcg_stack* m, const bcg_stack_ws* ws, const bcg_step_b
 
 int bcg_clamped_glu(const float* z, int n_partials, long long partial_stride, void* out, int act_dtype, int T, int ff,
                     float limit, float alpha, void* stream) {
-  return clamped_glu_rows(z, n_partials, partial_stride, nullptr, out, act_dtype, T, ff, limit, alpha, S(stream));
+  return unit_rows(z, n_partials, partial_stride, nullptr, out, act_dtype, T, ff, BCG_EPI_GLU, limit, alpha, S(stream));
 }
 
 int bcg_gemm_bf16_glu(const void* X, const void* W, void* out, int M, int N, int K, float limit, float alpha, int flags,
                       void* stream) {
-  return gemm_bf16_glu(X, W, out, M, N, K, limit, alpha, flags, S(stream));
+  return gemm_bf16_glu(X, W, out, M, N, K, BCG_EPI_GLU, limit, alpha, flags, S(stream));
+}
+
+int bcg_gelu_unit(const float* z, int n_partials, long long partial_stride, void* out, int act_dtype, int T, int ff, int gated,
+                  void* stream) {
+  return unit_rows(z, n_partials, partial_stride, nullptr, out, act_dtype, T, ff, gated ? BCG_EPI_GELU_GLU : BCG_EPI_GELU, 0.f, 0.f,
+                   S(stream));
+}
+
+int bcg_gemm_bf16_gelu(const void* X, const void* W, void* out, int M, int N, int K, int gated, int flags, void* stream) {
+  return gated ? gemm_bf16_glu(X, W, out, M, N, K, BCG_EPI_GELU_GLU, 0.f, 0.f, flags, S(stream))
+               : gemm_bf16_gelu(X, W, out, M, N, K, flags, S(stream));
+}
+
+int bcg_gemm_grouped_gelu(const void* X, const void* W, void* out, int rows, int N, int K, const int* counts, int n_groups, int max_rows,
+                          int flags, void* stream) {
+  GemmGroups g = {};
+  g.counts = counts;
+  g.n_groups = n_groups;
+  g.max_rows = max_rows;
+  const int saved = launch_flags();
+  launch_flags() = flags & BCG_GEMM_PDL;
+  const int rc = gemm_grouped(X, W, out, rows, N, K, BCG_EPI_GELU, 1, g, S(stream));
+  launch_flags() = saved;
+  return rc;
+}
+
+int bcg_expert_in(const bcg_stack* m, const bcg_stack_ws* ws, int layer, int T, int n_partials, long long partial_stride, long long ld,
+                  int with_act, void* stream) {
+  return expert_in_step(m, ws, layer, T, n_partials, partial_stride, ld, with_act, S(stream));
+}
+
+int bcg_matrix_memory(const bcg_stack* m, const bcg_stack_ws* ws, const bcg_step_batch* b, int layer, int n_partials,
+                      long long partial_stride, long long ld, int mode, void* stream) {
+  return matrix_memory_step(m, ws, b, layer, n_partials, partial_stride, ld, mode, S(stream));
 }
 
 int bcg_experts(const bcg_stack* m, const bcg_stack_ws* ws, int layer, int T, int* splits, void* stream) {

@@ -299,6 +299,14 @@ __device__ __forceinline__ void st_v8(void* p, const uint32_t* v) {
 
 __device__ __forceinline__ float bf16lo(uint32_t w) { return __uint_as_float(w << 16); }
 __device__ __forceinline__ float bf16hi(uint32_t w) { return __uint_as_float(w & 0xffff0000u); }
+// gelu of bf16 outputs: short exponential in the tanh form z / (1 + exp(-2 y)), y = sqrt(2 / pi) (z + 0.044715 z^3)
+__device__ __forceinline__ float gelu_tanh_mul(float g, float u) {
+  return __fdividef(g, 1.0f + __expf(-1.5957691216057308f * fmaf(0.044715f * g * g, g, g))) * u;
+}
+__device__ __forceinline__ uint32_t gelu_erf_bits(uint32_t v) {
+  const float z = __uint_as_float(v);
+  return __float_as_uint(0.5f * z * (1.0f + erff(z * 0.70710678118654752f)));
+}
 __device__ __forceinline__ uint32_t pack_bf16(float lo, float hi) {
   __nv_bfloat162 v = __floats2bfloat162_rn(lo, hi);
   return *reinterpret_cast<uint32_t*>(&v);

@@ -249,7 +249,7 @@ gemm2sm_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_
       const uint32_t taddr = tmem_base + (static_cast<uint32_t>(q * 32) << 16) + static_cast<uint32_t>(acc * k2BlockN);
       const int m = tm * 256 + static_cast<int>(rank) * k2BlockM + row;
       const int n0 = tn * k2BlockN;
-      if (args.epi == BCG_EPI_SWIGLU || args.epi == BCG_EPI_GLU) {
+      if (args.epi == BCG_EPI_SWIGLU || args.epi == BCG_EPI_GLU || args.epi == BCG_EPI_GELU_GLU) {
         __nv_bfloat16* o = reinterpret_cast<__nv_bfloat16*>(args.out);
 #pragma unroll 1
         for (int c = 0; c < k2BlockN; c += 32) {
@@ -264,6 +264,11 @@ gemm2sm_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_
               p[j] = pack_bf16(glu_clamp2(__uint_as_float(g[2 * j]), __uint_as_float(u[2 * j]), args.glu_limit, args.glu_alpha),
                                glu_clamp2(__uint_as_float(g[2 * j + 1]), __uint_as_float(u[2 * j + 1]), args.glu_limit,
                                           args.glu_alpha));
+          } else if (args.epi == BCG_EPI_GELU_GLU) {
+#pragma unroll
+            for (int j = 0; j < 8; ++j)
+              p[j] = pack_bf16(gelu_tanh_mul(__uint_as_float(g[2 * j]), __uint_as_float(u[2 * j])),
+                               gelu_tanh_mul(__uint_as_float(g[2 * j + 1]), __uint_as_float(u[2 * j + 1])));
           } else {
 #pragma unroll
             for (int j = 0; j < 8; ++j)
@@ -312,6 +317,12 @@ gemm2sm_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_
                 const float x0 = fmaxf(__uint_as_float(v0[j]), 0.f), x1 = fmaxf(__uint_as_float(v1[j]), 0.f);
                 v0[j] = __float_as_uint(x0 * x0);
                 v1[j] = __float_as_uint(x1 * x1);
+              }
+            } else if (args.epi == BCG_EPI_GELU) {
+#pragma unroll
+              for (int j = 0; j < 16; ++j) {
+                v0[j] = gelu_erf_bits(v0[j]);
+                v1[j] = gelu_erf_bits(v1[j]);
               }
             }
 #pragma unroll

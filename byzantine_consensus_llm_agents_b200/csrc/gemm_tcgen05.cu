@@ -373,7 +373,8 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_a,
               const float u = __shfl_down_sync(0xffffffffu, g, 16);
               const int m = m0 + c + j;
               if (lane < 16 && m < M && n < N) o[m * ld + nb] = __float2bfloat16_rn(
-                  args.epi == BCG_EPI_GLU ? glu_clamp(g, u, args.glu_limit, args.glu_alpha) : silu_mul(g, u));
+                  args.epi == BCG_EPI_GLU ? glu_clamp(g, u, args.glu_limit, args.glu_alpha)
+                                          : args.epi == BCG_EPI_GELU_GLU ? gelu_tanh_mul(g, u) : silu_mul(g, u));
             }
           }
         }
@@ -381,7 +382,7 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_a,
         // lanes = activation rows (m), columns = weight rows (n)
         const int m = ta * kBlockA + row;
         const int n0 = tb * BN;
-        if (args.epi == BCG_EPI_SWIGLU || args.epi == BCG_EPI_GLU) {
+        if (args.epi == BCG_EPI_SWIGLU || args.epi == BCG_EPI_GLU || args.epi == BCG_EPI_GELU_GLU) {
           __nv_bfloat16* o = reinterpret_cast<__nv_bfloat16*>(args.out) + base;
           float weight = 1.f;
           if (GROUPED && m < M) weight = args.groups.row_weight[first_row[e] + m];
@@ -399,6 +400,8 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_a,
               if (GROUPED || args.epi == BCG_EPI_GLU)
                 p[j] = pack_bf16(glu_clamp(weight * g0, weight * u0, args.glu_limit, args.glu_alpha),
                                  glu_clamp(weight * g1, weight * u1, args.glu_limit, args.glu_alpha));
+              else if (args.epi == BCG_EPI_GELU_GLU)
+                p[j] = pack_bf16(gelu_tanh_mul(g0, u0), gelu_tanh_mul(g1, u1));
               else
                 p[j] = pack_bf16(silu_mul(g0, u0), silu_mul(g1, u1));
             }
@@ -451,6 +454,12 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_a,
                 for (int j = 0; j < 16; ++j) {
                   v0[j] = relu_squared(v0[j]);
                   v1[j] = relu_squared(v1[j]);
+                }
+              } else if (args.epi == BCG_EPI_GELU) {
+#pragma unroll
+                for (int j = 0; j < 16; ++j) {
+                  v0[j] = gelu_erf_bits(v0[j]);
+                  v1[j] = gelu_erf_bits(v1[j]);
                 }
               }
 #pragma unroll
@@ -659,9 +668,13 @@ int gemm_bf16_tn_fused(const void* X, const void* W, void* out, int M, int N, in
   return gemm_dense(X, W, out, M, N, K, ldx, ldw, ld_out, epi, splits, flags, fu, 0.f, 0.f, stream);
 }
 
-int gemm_bf16_glu(const void* X, const void* W, void* out, int M, int N, int K, float limit, float alpha, int flags,
+int gemm_bf16_glu(const void* X, const void* W, void* out, int M, int N, int K, int epi, float limit, float alpha, int flags,
                   cudaStream_t stream) {
-  return gemm_dense(X, W, out, M, N, K, K, K, N / 2, BCG_EPI_GLU, 1, flags, nullptr, limit, alpha, stream);
+  return gemm_dense(X, W, out, M, N, K, K, K, N / 2, epi, 1, flags, nullptr, limit, alpha, stream);
+}
+
+int gemm_bf16_gelu(const void* X, const void* W, void* out, int M, int N, int K, int flags, cudaStream_t stream) {
+  return gemm_dense(X, W, out, M, N, K, K, K, N, BCG_EPI_GELU, 1, flags, nullptr, 0.f, 0.f, stream);
 }
 
 static int gemm_dense(const void* X, const void* W, void* out, int M, int N, int K, long long ldx, long long ldw,
@@ -681,14 +694,14 @@ static int gemm_dense(const void* X, const void* W, void* out, int M, int N, int
     set_last_error("bcg_gemm_bf16_tn", "split-K needs the fp32 partial epilogue");
     return BCG_ERR_ARG;
   }
-  const bool paired = epi == BCG_EPI_SWIGLU || epi == BCG_EPI_GLU;
+  const bool paired = epi == BCG_EPI_SWIGLU || epi == BCG_EPI_GLU || epi == BCG_EPI_GELU_GLU;
   if (paired && (N % 32)) {
     set_last_error("bcg_gemm_bf16_tn", "gated epilogues need N % 32 == 0");
     return BCG_ERR_ARG;
   }
   const bool swap = (M <= 128);
-  if (epi == BCG_EPI_RELU2 && (swap || N % 16)) {
-    set_last_error("bcg_gemm_bf16_tn", "squared relu with M <= 128 or N % 16");
+  if ((epi == BCG_EPI_RELU2 || epi == BCG_EPI_GELU) && (swap || N % 16)) {
+    set_last_error("bcg_gemm_bf16_tn", "squared relu or gelu with M <= 128 or N % 16");
     return BCG_ERR_ARG;
   }
   if (!swap && ((epi == BCG_EPI_F32 ? (ld_out % 4) : (ld_out % 8)))) {
@@ -790,7 +803,8 @@ int gemm_grouped(const void* X, const void* W, void* out, int rows, int N, int K
                  cudaStream_t stream) {
   const bool swap = g.max_rows <= 128;
   if (!X || !W || !out || rows <= 0 || N <= 0 || K <= 0 || K % 8 || g.n_groups <= 0 || g.n_groups > kMaxGroups ||
-      !g.counts || splits < 1 || (splits > 1 && !swap) || (epi != BCG_EPI_F32 && (epi != BCG_EPI_GLU || swap || N % 32)) ||
+      !g.counts || splits < 1 || (splits > 1 && !swap) ||
+      (epi != BCG_EPI_F32 && (swap || (epi != BCG_EPI_GELU && (epi != BCG_EPI_GLU || N % 32)))) ||
       (!swap && N % 16) || (epi == BCG_EPI_GLU && !g.row_weight) ||
       ((reinterpret_cast<uintptr_t>(X) | reinterpret_cast<uintptr_t>(W) | reinterpret_cast<uintptr_t>(out)) & 15)) {
     set_last_error("bcg_gemm_grouped", "bad argument (K % 8, N % 16 beyond 128 rows, at most 512 groups, alignment)");

@@ -1,11 +1,15 @@
 // Grouped-query attention over paged keys and values, with what a layer has of: a linear distance bias, a sliding
-// window, a query temperature, query and key norms over all heads at once, an output gate per head.
+// window, a query temperature, query and key norms over all heads at once or head by head, rotated queries, keys and
+// values, means of blocks of tokens in front of the window, an output gate per head.
 //
 // A layer's cache is two pools of 16-token pages, keys [page][kv head][16][q_ld] and values [page][kv head][16][v_ld];
 // heads are padded to q_ld / v_ld columns, the padding is zero and stays so.
 //   grouped_in      projection slabs -> queries (bias, temperature), keys and values (bias, value mixing) into the
 //                   pages, squared-relu activations of a parallel feed-forward, routing of a parallel mixture;
-//                   where there are norms or gates, a CTA or a cluster has a whole token (grouped_norm_in)
+//                   where there are norms or gates, a CTA or a cluster has a whole token (grouped_norm_in); where
+//                   heads are normed or rotated one by one, a warp has a head (head_in)
+//   pool_blocks     means of the blocks of tokens that a ragged step completes, into their own pages (single tokens:
+//                   head_in makes them)
 //   grouped_plain   one CTA per (token, head), any sizes, fp32 or bf16: the fp32 engine's kernel, and the bf16
 //                   one's for head sizes the kernels below do not take
 //   grouped_decode  single tokens: a cluster per (token, kv head) shares the key pages, a ring of TMA loads and a
@@ -43,6 +47,12 @@ struct GroupedIn {
   float* gates;               // [T][heads] or NULL; logits are columns gate_col.. of proj
   int gate_col;
   float gate_scale, eps;
+  // heads one by one (head_in): q_norm and k_norm are [dim]
+  const float *cos_sin, *v_cos_sin;   // [positions][dims]: cosines of the dims / 2 angles, then sines
+  int rot_dims, rot_pairs, v_rot_dims;
+  int pool, pool_col;         // pool > 0: single tokens that complete a block write its means
+  const int* block_table;
+  int max_blocks;
 };
 
 // Where a token's columns go.
@@ -184,6 +194,134 @@ static int norm_in_t(const GroupedIn& a, cudaStream_t st) {
   return BCG_OK;
 }
 
+// Row of a key/value head in the pages: entry i of logical page j0 + i / page_size of a sequence's row of the block table.
+__device__ __forceinline__ long long page_row(const int* bt, int j0, int i, int kv_heads, int g, int page_size) {
+  return (static_cast<long long>(bt[j0 + i / page_size]) * kv_heads + g) * page_size + i % page_size;
+}
+
+// Mean of `pool` rows of a cache, the cached ones of positions p0 .. and `last`, added in their order.
+template <typename T, int V>
+__device__ __forceinline__ Vec<V> block_mean(const T* cache, const int* bt, int kv_heads, int g, int page_size, int ld, int c, int p0,
+                                             int pool, const Vec<V>* last) {
+  Vec<V> sum;
+#pragma unroll
+  for (int k = 0; k < V; ++k) sum.x[k] = 0.f;
+  const int n = last ? pool - 1 : pool;
+#pragma unroll 4
+  for (int j = 0; j < n; ++j) sum.add(load_vec<V>(cache + page_row(bt, 0, p0 + j, kv_heads, g, page_size) * ld + c));
+  if (last) sum.add(*last);
+#pragma unroll
+  for (int k = 0; k < V; ++k) sum.x[k] /= static_cast<float>(pool);
+  return sum;
+}
+
+// One head of a token (queries, then keys, then values) per warp: norm, rotation, destination.  blocks: the step has one token per
+// sequence, so whoever writes the last row of a block also writes its mean.
+template <typename T, int V>
+__global__ void __launch_bounds__(kInThreads)
+head_in_kernel(const GroupedIn a, int pitch, bool blocks) {
+  extern __shared__ float4 stage_raw[];
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  float* x = reinterpret_cast<float*>(stage_raw) + warp * pitch;
+  pdl_launch_dependents();
+  pdl_wait();
+  const int per = a.heads + 2 * a.kv_heads;
+  const long long unit = blockIdx.x * static_cast<long long>(kInThreads / 32) + warp;
+  const long long t = unit / per;
+  if (t >= a.n_tokens) return;
+  const int s = static_cast<int>(unit - t * per);
+  const bool is_q = s < a.heads, is_v = s >= a.heads + a.kv_heads;
+  const int g = is_q ? s : s - a.heads - (is_v ? a.kv_heads : 0);
+  const int width = is_v ? a.vdim : a.dim, dims = is_v ? a.v_rot_dims : a.rot_dims, half = dims / 2;
+  const int col = is_q ? g * a.dim : is_v ? (a.heads + a.kv_heads) * a.dim + g * a.vdim : (a.heads + g) * a.dim;
+  const bool pairs = is_v || a.rot_pairs;
+  const int pos = a.positions[t], slot = a.slot_map[t];
+  const float* row = a.proj + t * a.ld + col;
+  float ss = 0.f;
+  for (int c = lane * V; c < width; c += 32 * V) {
+    Vec<V> v = slab_sum_vec<V>(row + c, a.n_partials, a.pstride);
+    if (a.bias) v.add(load_vec<V>(a.bias + col + c));
+    store_vec<V>(x + c, v);
+    ss += v.sumsq();
+  }
+  const float* w = is_q ? a.q_norm : is_v ? nullptr : a.k_norm;
+  const float inv = w ? rsqrtf(warp_sum(ss) / static_cast<float>(width) + a.eps) : 1.0f;
+  __syncwarp();
+  const float* angle = (is_v ? a.v_cos_sin : a.cos_sin) + static_cast<long long>(pos) * dims;
+  const int ld = is_v ? a.v_ld : a.q_ld;
+  T* cache = static_cast<T*>(is_v ? a.v_cache : a.k_cache);
+  T* dst = nullptr;
+  if (is_q) dst = static_cast<T*>(a.q) + (t * a.heads + g) * a.q_ld;
+  else if (slot >= 0) dst = cache + ((static_cast<long long>(slot / a.page_size) * a.kv_heads + g) * a.page_size + slot % a.page_size) * ld;
+  const bool whole = blocks && a.pool > 0 && !is_q && slot >= 0 && (pos + 1) % a.pool == 0;
+  const int* bt = a.block_table + t * a.max_blocks;
+  for (int c = lane * V; c < width; c += 32 * V) {
+    Vec<V> y;
+#pragma unroll
+    for (int k = 0; k < V; ++k) {
+      const int e = c + k;
+      const float own = x[e] * (w ? inv * w[e] : 1.0f);
+      y.x[k] = own;
+      if (e < dims) {
+        const bool first = pairs ? !(e & 1) : e < half;
+        const int p = pairs ? e ^ 1 : first ? e + half : e - half, i = pairs ? e >> 1 : first ? e : e - half;
+        const float other = x[p] * (w ? inv * w[p] : 1.0f), cs = angle[i], sn = angle[half + i];
+        y.x[k] = first ? own * cs - other * sn : own * cs + other * sn;
+      }
+      if (sizeof(T) == 2) y.x[k] = to_f32<T>(from_f32<T>(y.x[k]));      // as the cache holds it
+    }
+    if (dst) store_vec<V>(dst + c, y);
+    if (whole) {
+      const int b = pos / a.pool;
+      const Vec<V> mean = block_mean<T, V>(cache, bt, a.kv_heads, g, a.page_size, ld, c, b * a.pool, a.pool, &y);
+      store_vec<V>(cache + page_row(bt, a.pool_col, b, a.kv_heads, g, a.page_size) * ld + c, mean);
+    }
+  }
+}
+
+// A warp has a run of 32 tokens and a key or value head: the means of the blocks that end there.
+template <typename T, int V>
+__global__ void __launch_bounds__(kInThreads)
+pool_blocks_kernel(const GroupedIn a, const int* __restrict__ row_seq) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const int lane = threadIdx.x & 31;
+  const long long unit = blockIdx.x * static_cast<long long>(kInThreads / 32) + (threadIdx.x >> 5);
+  const int s = static_cast<int>(unit % (2 * a.kv_heads));
+  const long long t0 = unit / (2 * a.kv_heads) * 32;
+  if (t0 >= a.n_tokens) return;
+  const bool is_v = s >= a.kv_heads, mine = t0 + lane < a.n_tokens;
+  const int g = is_v ? s - a.kv_heads : s, width = is_v ? a.vdim : a.dim, ld = is_v ? a.v_ld : a.q_ld;
+  T* cache = static_cast<T*>(is_v ? a.v_cache : a.k_cache);
+  const int pos = mine ? a.positions[t0 + lane] : 0;
+  unsigned ends = __ballot_sync(0xffffffffu, mine && a.slot_map[t0 + lane] >= 0 && (pos + 1) % a.pool == 0);
+  for (; ends; ends &= ends - 1) {
+    const int i = __ffs(ends) - 1, b = __shfl_sync(0xffffffffu, pos, i) / a.pool;
+    const int* bt = a.block_table + static_cast<long long>(row_seq ? row_seq[t0 + i] : t0 + i) * a.max_blocks;
+    T* dst = cache + page_row(bt, a.pool_col, b, a.kv_heads, g, a.page_size) * ld;
+    for (int c = lane * V; c < width; c += 32 * V)
+      store_vec<V>(dst + c, block_mean<T, V>(cache, bt, a.kv_heads, g, a.page_size, ld, c, b * a.pool, a.pool, nullptr));
+  }
+}
+
+template <typename T, int V>
+static int head_in_t(const GroupedIn& a, const int* row_seq, bool one_token, cudaStream_t st) {
+  const int pitch = (max(a.dim, a.vdim) + 3) / 4 * 4;
+  const size_t sm = static_cast<size_t>(kInThreads / 32) * pitch * 4;
+  if (sm > 200 * 1024) {
+    set_last_error("bcg_grouped_in", "heads are too large");
+    return BCG_ERR_UNSUPPORTED;
+  }
+  if (sm > 48 * 1024) BCG_TRY(ensure_dynamic_smem(reinterpret_cast<const void*>(head_in_kernel<T, V>), 200 * 1024));
+  const long long units = static_cast<long long>(a.n_tokens) * (a.heads + 2 * a.kv_heads);
+  BCG_CUDA_CHECK(launch_k(head_in_kernel<T, V>, dim3(static_cast<unsigned>((units + 7) / 8)), dim3(kInThreads), sm, st, a, pitch, one_token));
+  if (a.pool > 0 && !one_token) {
+    const long long runs = static_cast<long long>((a.n_tokens + 31) / 32) * 2 * a.kv_heads;
+    BCG_CUDA_CHECK(launch_k(pool_blocks_kernel<T, V>, dim3(static_cast<unsigned>((runs + 7) / 8)), dim3(kInThreads), 0, st, a, row_seq));
+  }
+  return BCG_OK;
+}
+
 template <typename T>
 static int grouped_in_t(const GroupedIn& a, cudaStream_t st) {
   const bool wide = ((a.dim | a.vdim | a.ff | a.act_from) & 3) == 0 && a.ld % 4 == 0 && a.pstride % 4 == 0;
@@ -242,6 +380,31 @@ int grouped_in(const bcg_stack* m, const bcg_layer* l, const bcg_stack_ws* ws, c
   a.gate_col = l->gate_col;
   a.gate_scale = l->gate_scale;
   a.eps = m->eps;
+  if (l->by_head) {
+    if ((l->rot_dims && !l->cos_sin) || (l->v_rot_dims && !l->v_cos_sin) || l->rot_dims % 2 || l->rot_dims > l->dim || l->v_rot_dims % 2 ||
+        l->v_rot_dims > l->vdim || l->gated || l->v_role || l->slopes || l->temp_coef != 0.f || with_act || l->pool < 0) {
+      set_last_error("bcg_grouped_in", "heads one by one: even rotary sizes with tables; no gates, mixed values, bias or temperature");
+      return BCG_ERR_ARG;
+    }
+    a.cos_sin = l->cos_sin;
+    a.v_cos_sin = l->v_cos_sin;
+    a.rot_dims = l->rot_dims;
+    a.rot_pairs = l->rot_pairs;
+    a.v_rot_dims = l->v_rot_dims;
+    a.pool = l->pool;
+    a.pool_col = l->pool_col;
+    a.block_table = b->block_table;
+    a.max_blocks = b->max_blocks;
+    a.n_tokens = b->T;
+    const bool wide = ((a.dim | a.vdim) & 3) == 0 && a.ld % 4 == 0 && a.pstride % 4 == 0, one = b->T == b->n_seqs;
+    if (m->act_dtype == BCG_DT_F32)
+      return wide ? head_in_t<float, 4>(a, b->row_seq, one, st) : head_in_t<float, 1>(a, b->row_seq, one, st);
+    return wide ? head_in_t<__nv_bfloat16, 4>(a, b->row_seq, one, st) : head_in_t<__nv_bfloat16, 1>(a, b->row_seq, one, st);
+  }
+  if (!l->in_bias) {
+    set_last_error("bcg_grouped_in", "projections without bias: heads one by one");
+    return BCG_ERR_UNSUPPORTED;
+  }
   if (l->experts > 0) a.route = moe_route(l, ws);
   const int cols = l->heads * l->dim + l->kv_heads * (l->dim + l->vdim);
   a.blocks = b->T <= 128 ? max(1, ((cols > a.ff ? cols : a.ff) + kInThreads * 4 - 1) / (kInThreads * 4)) : 1;
@@ -262,6 +425,17 @@ struct GroupedAttn {
   long long out_ld;
   int heads, kv_heads, dim, vdim, q_ld, v_ld, window;
   float scale;
+  PooledKeys pooled;
+  const float* v_cos_sin;     // outputs turn back in pairs of neighbours, or NULL
+  int v_rot_dims;
+  // Output columns c (even) and c + 1 of a token at position pos.
+  __device__ __forceinline__ void turn_back(int pos, int c, float& u, float& v) const {
+    if (!v_cos_sin || c >= v_rot_dims) return;
+    const float* row = v_cos_sin + static_cast<long long>(pos) * v_rot_dims + c / 2;
+    const float cs = row[0], sn = row[v_rot_dims / 2], x = u;
+    u = x * cs + v * sn;
+    v = v * cs - x * sn;
+  }
 };
 
 template <typename T>
@@ -281,23 +455,24 @@ grouped_plain_kernel(const GroupedAttn a) {
   const int* bt = a.block_table + static_cast<long long>(a.row_seq ? a.row_seq[t] : t) * a.max_blocks;
   const T* qh = static_cast<const T*>(a.q) + (t * a.heads + h) * a.q_ld;
   const float slope = a.slopes ? a.slopes[h] : 0.f;
-  auto row_of = [&](int key) {
-    return (static_cast<long long>(bt[key / a.page_size]) * a.kv_heads + g) * a.page_size + key % a.page_size;
-  };
   for (int i = threadIdx.x; i < a.dim; i += kGpThreads) qs[i] = to_f32<T>(qh[i]);
   for (int i = threadIdx.x; i < a.vdim; i += kGpThreads) oc[i] = 0.f;
   float m = -INFINITY, l = 0.f;
   const int lo = a.window > 0 ? max(0, pos - a.window + 1) : 0;
-  for (int j0 = lo; j0 <= pos; j0 += kGpKeys) {
-    const int n = min(kGpKeys, pos + 1 - j0);
+  // tokens lo .. pos, then the pooled blocks that are seen
+  const int n_tok = pos + 1 - lo, n_all = n_tok + a.pooled.visible(pos, a.window);
+  auto row_of = [&](int u) {
+    return u < n_tok ? page_row(bt, 0, lo + u, a.kv_heads, g, a.page_size) : page_row(bt, a.pooled.col, u - n_tok, a.kv_heads, g, a.page_size);
+  };
+  for (int j0 = 0; j0 < n_all; j0 += kGpKeys) {
+    const int n = min(kGpKeys, n_all - j0);
     __syncthreads();
     float mx = -INFINITY;
     for (int j = warp; j < n; j += kGpThreads / 32) {
-      const int key = j0 + j;
-      const T* k = static_cast<const T*>(a.k_cache) + row_of(key) * a.q_ld;
+      const T* k = static_cast<const T*>(a.k_cache) + row_of(j0 + j) * a.q_ld;
       float s = 0.f;
       for (int i = lane; i < a.dim; i += 32) s = fmaf(qs[i], to_f32<T>(k[i]), s);
-      s = warp_sum(s) * a.scale - slope * static_cast<float>(pos - key);
+      s = warp_sum(s) * a.scale - slope * static_cast<float>(pos - lo - (j0 + j));
       if (lane == 0) p[j] = s;
       mx = fmaxf(mx, s);
     }
@@ -332,7 +507,12 @@ grouped_plain_kernel(const GroupedAttn a) {
   __syncthreads();
   const float inv = (a.gates ? a.gates[t * a.heads + h] : 1.0f) / l;
   T* dst = static_cast<T*>(a.out) + t * a.out_ld + static_cast<long long>(h) * a.vdim;
-  for (int r = threadIdx.x; r < a.vdim; r += kGpThreads) dst[r] = from_f32<T>(oc[r] * inv);
+  for (int r = threadIdx.x * 2; r < a.vdim; r += kGpThreads * 2) {
+    float u = oc[r] * inv, v = r + 1 < a.vdim ? oc[r + 1] * inv : 0.f;
+    a.turn_back(pos, r, u, v);
+    dst[r] = from_f32<T>(u);
+    if (r + 1 < a.vdim) dst[r + 1] = from_f32<T>(v);
+  }
 }
 
 static GroupedAttn attn_args(const bcg_stack* m, const bcg_layer* l, const bcg_stack_ws* ws, const bcg_step_batch* b,
@@ -359,6 +539,9 @@ static GroupedAttn attn_args(const bcg_stack* m, const bcg_layer* l, const bcg_s
   a.v_ld = l->v_ld;
   a.window = l->window;
   a.scale = l->scale;
+  a.pooled = {l->pool, l->pool_col};
+  a.v_cos_sin = l->v_rot_dims > 0 ? l->v_cos_sin : nullptr;
+  a.v_rot_dims = l->v_rot_dims;
   return a;
 }
 
@@ -432,11 +615,15 @@ grouped_decode_kernel(const __grid_constant__ CUtensorMap k_map, const __grid_co
   const int pos = a.positions[t];
   const int lo = a.window > 0 ? max(0, pos - a.window + 1) : 0;
   const int* bt = a.block_table + static_cast<long long>(a.row_seq ? a.row_seq[t] : t) * a.max_blocks;
-  const int first = lo / kGdPage + rank * kGdWarps + warp, stride = n_cta * kGdWarps;
-  const int n = pos / kGdPage >= first ? (pos / kGdPage - first) / stride + 1 : 0;
+  // the token's pages, then those of the pooled blocks it sees: the warp has first, first + stride, ...
+  const int n_pooled = a.pooled.visible(pos, a.window), tok_pages = pos / kGdPage - lo / kGdPage + 1;
+  const int n_pages = tok_pages + (n_pooled + kGdPage - 1) / kGdPage;
+  const int first = rank * kGdWarps + warp, stride = n_cta * kGdWarps;
+  const int n = n_pages > first ? (n_pages - 1 - first) / stride + 1 : 0;
   auto load = [&](int i) {    // lane 0
     const int st = i % C::kStages;
-    const int row = (bt[first + i * stride] * a.kv_heads + g) * kGdPage;
+    const int u = first + i * stride;
+    const int row = (bt[u < tok_pages ? lo / kGdPage + u : a.pooled.col + u - tok_pages] * a.kv_heads + g) * kGdPage;
     uint8_t* dst = ring + st * C::kStage;
     mbar_arrive_expect_tx(&full[st], C::kStage);
 #pragma unroll
@@ -477,7 +664,10 @@ grouped_decode_kernel(const __grid_constant__ CUtensorMap k_map, const __grid_co
       mma_bf16_16816(s[0], qa, kb[0], kb[1]);
       mma_bf16_16816(s[1], qa, kb[2], kb[3]);
     }
-    const int key0 = (first + i * stride) * kGdPage + (lane & 3) * 2;
+    const int page = first + i * stride;
+    const bool pooled = page >= tok_pages;
+    const int key0 = (pooled ? page - tok_pages : lo / kGdPage + page) * kGdPage + (lane & 3) * 2;
+    const int key_lo = pooled ? 0 : lo, key_hi = pooled ? n_pooled - 1 : pos;
     float corr[2];
 #pragma unroll
     for (int e = 0; e < 2; ++e) {
@@ -486,7 +676,7 @@ grouped_decode_kernel(const __grid_constant__ CUtensorMap k_map, const __grid_co
       for (int c = 0; c < 4; ++c) {      // keys key0, key0 + 1, key0 + 8, key0 + 9
         const int key = key0 + (c >> 1) * 8 + (c & 1);
         float& x = s[c >> 1][2 * e + (c & 1)];
-        x = key >= lo && key <= pos ? fmaf(x, scale2, slope[e] * static_cast<float>(key - pos)) : -INFINITY;
+        x = key >= key_lo && key <= key_hi ? fmaf(x, scale2, slope[e] * static_cast<float>(key - pos)) : -INFINITY;
         mx = fmaxf(mx, x);
       }
       mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 1));
@@ -556,21 +746,30 @@ grouped_decode_kernel(const __grid_constant__ CUtensorMap k_map, const __grid_co
   if (n_cta > 1) cluster.sync();
   else __syncthreads();
   auto* dst = static_cast<__nv_bfloat16*>(a.out) + static_cast<long long>(t) * a.out_ld + static_cast<long long>(h0) * a.vdim;
-  for (int i = rank * kGdThreads + threadIdx.x; i < nh * VD; i += n_cta * kGdThreads) {
+  for (int i = (rank * kGdThreads + threadIdx.x) * 2; i < nh * VD; i += n_cta * kGdThreads * 2) {
     const int r = i / VD, c = i % VD;
     if (c >= a.vdim) continue;
-    float top = -INFINITY, x = 0.f, den = 0.f;
+    float top = -INFINITY, x0 = 0.f, x1 = 0.f, den = 0.f;
     for (int q = 0; q < n_cta; ++q) {
       const float2 other = *cluster.map_shared_rank(ml + kGdWarps * kGdHeads + r, q);
-      const float val = cluster.map_shared_rank(mine, q)[i];
+      const float2 val = *reinterpret_cast<const float2*>(cluster.map_shared_rank(mine, q) + i);
       const float up = fmaxf(top, other.x);
       const float f0 = weight(top, up), f1 = weight(other.x, up);
-      x = x * f0 + val * f1;
+      x0 = x0 * f0 + val.x * f1;
+      x1 = x1 * f0 + val.y * f1;
       den = den * f0 + other.y * f1;
       top = up;
     }
-    if (a.gates) x *= a.gates[static_cast<long long>(t) * a.heads + h0 + r];
-    dst[static_cast<long long>(r) * a.vdim + c] = __float2bfloat16(x / den);
+    if (a.gates) {
+      const float gate = a.gates[static_cast<long long>(t) * a.heads + h0 + r];
+      x0 *= gate;
+      x1 *= gate;
+    }
+    x0 /= den;
+    x1 /= den;
+    a.turn_back(pos, c, x0, x1);
+    dst[static_cast<long long>(r) * a.vdim + c] = __float2bfloat16(x0);
+    if (c + 1 < a.vdim) dst[static_cast<long long>(r) * a.vdim + c + 1] = __float2bfloat16(x1);
   }
   if (n_cta > 1) cluster.sync();                     // nobody leaves while its shared memory is being read
 }
@@ -609,7 +808,8 @@ static int grouped_decode(const bcg_stack* m, const bcg_layer* l, const bcg_stac
                           cudaStream_t st) {
   const int n = b->single_rows ? b->n_single : b->T;
   const int reach = l->window > 0 && l->window < b->max_context ? l->window + kGdPage - 1 : b->max_context;
-  const int pages = (reach + kGdPage - 1) / kGdPage;
+  const int blocks = l->pool > 0 && b->max_context > l->window ? (b->max_context - l->window) / l->pool : 0;
+  const int pages = (reach + kGdPage - 1) / kGdPage + (blocks + kGdPage - 1) / kGdPage;
   const int groups = l->kv_heads * ((l->heads / l->kv_heads + kGdHeads - 1) / kGdHeads);
   if (n > 65535 || groups > 65535) {
     set_last_error("bcg_grouped_attention", "too many single tokens or heads");
@@ -660,6 +860,9 @@ static int grouped_prefill(const bcg_layer* l, const bcg_stack_ws* ws, const bcg
   a.heads = l->heads;
   a.vdim = l->vdim;
   a.window = l->window;
+  a.pooled = {l->pool, l->pool_col};
+  a.v_cos_sin = l->v_rot_dims > 0 ? l->v_cos_sin : nullptr;
+  a.v_rot_dims = l->v_rot_dims;
   a.scale_log2e = l->scale * kLog2e;
   return l->slopes ? window_attn<true, true>(l->q_ld, l->v_ld, qm, km, vm, a, st)
                    : window_attn_paged(l->q_ld, l->v_ld, qm, km, vm, a, st);
@@ -667,6 +870,10 @@ static int grouped_prefill(const bcg_layer* l, const bcg_stack_ws* ws, const bcg
 
 int grouped_attention(const bcg_stack* m, const bcg_stack_ws* ws, const bcg_step_batch* b, const bcg_layer* l, int mode,
                       cudaStream_t st) {
+  if (l->slopes && (l->pool > 0 || l->v_rot_dims > 0)) {
+    set_last_error("bcg_grouped_attention", "a distance bias does not come with pooled blocks or rotated values");
+    return BCG_ERR_UNSUPPORTED;
+  }
   const int n_single = b->single_rows ? b->n_single : (b->n_tiles > 0 ? 0 : b->T);
   const bool tensor = m->act_dtype == BCG_DT_BF16 && mode == 0 && m->page_size == kGdPage && padded_head(l->q_ld, l->v_ld);
   if (!tensor) return grouped_plain(m, l, ws, b, nullptr, b->T, st);

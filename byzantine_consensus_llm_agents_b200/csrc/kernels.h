@@ -16,13 +16,16 @@ int gemm_bf16_tn(const void* X, const void* W, void* out, int M, int N, int K, l
 int gemm_bf16_tn_fused(const void* X, const void* W, void* out, int M, int N, int K, long long ldx,
                        long long ldw, long long ld_out, int epi, int splits, int flags,
                        const bcg_gemm_fusion* fusion, cudaStream_t stream);
-// epilogue BCG_EPI_GLU: W rows interleaved [16 gate | 16 up], out bf16 [M, N / 2]
-int gemm_bf16_glu(const void* X, const void* W, void* out, int M, int N, int K, float limit, float alpha, int flags,
+// epilogue BCG_EPI_GLU or BCG_EPI_GELU_GLU: W rows interleaved [16 gate | 16 up], out bf16 [M, N / 2]
+int gemm_bf16_glu(const void* X, const void* W, void* out, int M, int N, int K, int epi, float limit, float alpha, int flags,
                   cudaStream_t stream);
+// epilogue BCG_EPI_GELU: out bf16 [M, N], M > 128, N % 16 == 0
+int gemm_bf16_gelu(const void* X, const void* W, void* out, int M, int N, int K, int flags, cudaStream_t stream);
 int gemm_splits_for(int M, int N, int K);
-// Rows sorted by group (mixture of experts); internal epilogue BCG_EPI_GLU: columns interleaved [16 gate | 16 up],
-// each row's accumulators times its weight, clamped gated unit, bf16 [rows, N / 2]
-constexpr int BCG_EPI_GLU = 16;
+// Rows sorted by group (mixture of experts).  Internal epilogues: BCG_EPI_GLU, columns interleaved [16 gate | 16 up], each
+// row's accumulators times its weight (groups only), clamped gated unit, bf16 [rows, N / 2]; BCG_EPI_GELU_GLU, the same columns,
+// gelu(gate) * up with gelu's tanh form (no groups); BCG_EPI_GELU, gelu's erf form, bf16 [rows, N]
+constexpr int BCG_EPI_GLU = 16, BCG_EPI_GELU_GLU = 17, BCG_EPI_GELU = 18;
 constexpr int kMaxGroups = 512;
 struct GemmGroups {
   const int* counts;         // device [n_groups]: rows of every group
@@ -85,6 +88,7 @@ struct NormExtra {
   const float* bias = nullptr;      // [d]
   const float* rows = nullptr;      // [n_partials][any][d]
   const int* index = nullptr;       // [T][per_row] rows of it
+  const float* weight = nullptr;    // [T][per_row] their factors, or NULL
   int per_row = 0, n_partials = 1;
   long long partial_stride = 0;
 };
@@ -99,6 +103,7 @@ struct EmbedArgs {
   const double* pos_turns;          // [(d + 1) / 2] turns per position, or NULL: sin, cos in turn
   int* zero;
   int n_zero;
+  const float* norm;                // [d] weight of a norm of the embedding, or NULL
 };
 int embed_norm(const EmbedArgs& a, const float* w, float* residual, void* xn, int act_dtype, int T, int d, float eps,
                cudaStream_t stream);
@@ -136,9 +141,20 @@ int grouped_attention(const bcg_stack* m, const bcg_stack_ws* ws, const bcg_step
 // ws->xn through the layer's experts into ws->moe_out (*splits slabs), rows ws->moe_row
 int experts(const bcg_stack* m, const bcg_layer* l, const bcg_stack_ws* ws, int T, int* splits, cudaStream_t stream);
 int moe_splits(int T, int top, int N, int K);
-// clamped gated unit of slabs [rows][2 * ff_ld] (16 gate | 16 up); row_weight (NULL: 1) scales both
-int clamped_glu_rows(const float* z, int n_partials, long long pstride, const float* row_weight, void* out, int act_dtype,
-                     int rows, int ff_ld, float limit, float alpha, cudaStream_t stream);
+// A feed-forward's unit (BCG_EPI_GLU, BCG_EPI_GELU_GLU or BCG_EPI_GELU) of slabs [rows][2 * ff_ld] (16 gate | 16 up) or
+// [rows][ff_ld]; row_weight (NULL: 1) scales its input
+int unit_rows(const float* z, int n_partials, long long pstride, const float* row_weight, void* out, int act_dtype, int rows,
+              int ff_ld, int unit, float limit, float alpha, cudaStream_t stream);
+// Routing of a layer with experts that is not parallel (logits are the first columns of ws->proj) and, with_act, gelu of the
+// columns behind them into ws->act
+int expert_in(const bcg_stack* m, const bcg_layer* l, const bcg_stack_ws* ws, int T, int n_partials, long long pstride, long long ld,
+              bool with_act, cudaStream_t stream);
+int expert_in_step(const bcg_stack* m, const bcg_stack_ws* ws, int layer, int T, int n_partials, long long pstride, long long ld,
+                   int with_act, cudaStream_t stream);
+int matrix_memory(const bcg_stack* m, const bcg_layer* l, const bcg_stack_ws* ws, const bcg_step_batch* b, int n_partials,
+                  long long pstride, long long ld, int mode, cudaStream_t stream);
+int matrix_memory_step(const bcg_stack* m, const bcg_stack_ws* ws, const bcg_step_batch* b, int layer, int n_partials,
+                       long long pstride, long long ld, int mode, cudaStream_t stream);
 struct WindowAttn;
 // paged prompt attention without a distance bias (grouped_prefill.cu)
 int window_attn_paged(int q_ld, int v_ld, const CUtensorMap& qm, const CUtensorMap& km, const CUtensorMap& vm,

@@ -12,6 +12,8 @@ struct MoeRoute {
   int* rank;                 // [T][top] place among the expert's rows
   float* weight;             // [T][top]
   int* counts;               // [experts] rows per expert, zero before the step
+  const float* bias;         // [experts] added to the logits, or NULL
+  bool softmax;              // weights are the softmax over the chosen logits, else their sigmoids
 };
 
 __host__ inline MoeRoute moe_route(const bcg_layer* l, const bcg_stack_ws* ws) {
@@ -23,6 +25,8 @@ __host__ inline MoeRoute moe_route(const bcg_layer* l, const bcg_stack_ws* ws) {
   r.rank = ws->moe_rank;
   r.weight = ws->moe_weight;
   r.counts = ws->moe_counts + l->moe_counts_at;
+  r.bias = l->router_bias;
+  r.softmax = l->ff_kind == BCG_FF_EXPERTS;
   return r;
 }
 
@@ -39,11 +43,11 @@ __device__ __forceinline__ float from_ordered(uint32_t k) {
 __host__ __device__ constexpr int route_words(int experts, int threads) { return experts * (threads / 32 + 2); }
 
 // One warp, one token: the `top` experts with the largest logits (the sigmoid is monotone; ties go to the lower
-// index), weighted by their sigmoid scores.  keys: the warp's shared memory, one word per expert.
+// index), weighted by their sigmoid scores or by the softmax over the chosen ones.  keys: the warp's shared memory, one word per expert.
 // counters: rows of every expert so far.
 __device__ __forceinline__ void route_token(const MoeRoute& r, const float* row, int n_partials, long long pstride, int t,
                                             uint32_t* keys, int* counters, int lane) {
-  for (int e = lane; e < r.experts; e += 32) keys[e] = ordered_bits(slab_sum(row + r.col + e, n_partials, pstride));
+  for (int e = lane; e < r.experts; e += 32) keys[e] = ordered_bits(slab_sum(row + r.col + e, n_partials, pstride) + (r.bias ? r.bias[e] : 0.f));
   uint32_t best;      // the lane's best expert that is still free (key 0: none)
   int at;
   auto scan = [&]() {
@@ -59,8 +63,10 @@ __device__ __forceinline__ void route_token(const MoeRoute& r, const float* row,
   scan();
   int mine = 0;              // lane k keeps choice k: the counters are then touched side by side
   uint32_t key = 0;
+  float first = 0.f, sum = 0.f;      // largest logit, this lane's exponentials
   for (int k = 0; k < r.top; ++k) {
     const uint32_t top = __reduce_max_sync(0xffffffffu, best);
+    if (k == 0) first = from_ordered(top);
     const int e = __reduce_min_sync(0xffffffffu, best == top ? at : 0x7fffffff);
     if (e % 32 == lane) {
       keys[e] = 0;
@@ -74,10 +80,16 @@ __device__ __forceinline__ void route_token(const MoeRoute& r, const float* row,
       const int i = t * r.top + (k & ~31) + lane;
       if (lane <= k % 32) {
         r.expert[i] = mine;
-        r.weight[i] = 1.0f / (1.0f + expf(-from_ordered(key)));
+        const float z = from_ordered(key), w = r.softmax ? expf(z - first) : 1.0f / (1.0f + expf(-z));
+        r.weight[i] = w;
+        sum += w;
         r.rank[i] = atomicAdd(counters + mine, 1);
       }
     }
+  }
+  if (r.softmax) {
+    sum = warp_sum(sum);
+    for (int k = lane; k < r.top; k += 32) r.weight[t * r.top + k] /= sum;
   }
 }
 
@@ -119,5 +131,10 @@ __device__ __forceinline__ float clamped_glu(float g, float u, float limit, floa
   u = fminf(fmaxf(u, -limit), limit);
   return g / (1.0f + expf(-alpha * g)) * (u + 1.0f);
 }
+// 0.5 z (1 + tanh(y)) = z / (1 + exp(-2 y)), y = sqrt(2 / pi) (z + 0.044715 z^3)
+__device__ __forceinline__ float gelu_tanh(float z) {
+  return z / (1.0f + expf(-1.5957691216057308f * fmaf(0.044715f * z * z, z, z)));
+}
+__device__ __forceinline__ float gelu_erf(float z) { return 0.5f * z * (1.0f + erff(z * 0.70710678118654752f)); }
 
 }  // namespace bcg

@@ -1,7 +1,7 @@
 // Row-wise kernels of layer stacks:
-//   embed_norm      x = scale * E[ids] (+ P[positions] or sinusoids);  xn = rmsnorm(x) * w
-//   sandwich_norm   x += rmsnorm(delta) * w_post (or += delta);  xn = rmsnorm(x) * w_next
-//                   delta may have a bias and rows of a second source (a token's experts) added
+//   embed_norm      x = scale * E[ids] (+ P[positions] or sinusoids), normed or not;  xn = rmsnorm(x) * w (or x)
+//   sandwich_norm   x += rmsnorm(delta) * w_post (or += delta);  xn = rmsnorm(x) * w_next (or x)
+//                   delta may have a bias and rows of a second source (a token's experts, weighted or not) added
 //   rows_norm       xn[i] = rmsnorm(x[rows[i]]) * w
 //   poly_norm       PolyNorm activation: a N(z) + b N(z^2) + c N(z^3) + e, N = division by the row's RMS
 // `delta` and `z` arrive as fp32 split-K slabs of the projection in front.  Decode-sized launches spread a
@@ -47,12 +47,27 @@ embed_norm_kernel(const EmbedArgs a, const float* __restrict__ w, float* __restr
     ss[0] += x.sumsq();
   }
   row_sum<kRowT, 1, 1>(sh, ss, 0);
-  const float inv = rsqrtf(ss[0] / static_cast<float>(d) + eps);
+  float inv = rsqrtf(ss[0] / static_cast<float>(d) + eps);
+  if (a.norm) {
+    ss[0] = 0.f;
+    for (int v = threadIdx.x * V; v < d; v += kRowT * V) {
+      Vec<V> x = load_vec<V>(residual + t * d + v);
+      const Vec<V> ww = load_vec<V>(a.norm + v);
+#pragma unroll
+      for (int k = 0; k < V; ++k) x.x[k] *= inv * ww.x[k];
+      store_vec<V>(residual + t * d + v, x);
+      ss[0] += x.sumsq();
+    }
+    row_sum<kRowT, 1, 1>(sh, ss, 1);
+    inv = rsqrtf(ss[0] / static_cast<float>(d) + eps);
+  }
   for (int v = threadIdx.x * V; v < d; v += kRowT * V) {
     Vec<V> x = load_vec<V>(residual + t * d + v);
-    const Vec<V> ww = load_vec<V>(w + v);
+    if (w) {
+      const Vec<V> ww = load_vec<V>(w + v);
 #pragma unroll
-    for (int k = 0; k < V; ++k) x.x[k] *= inv * ww.x[k];
+      for (int k = 0; k < V; ++k) x.x[k] *= inv * ww.x[k];
+    }
     store_vec<V>(xn + t * d + v, x);
   }
 }
@@ -73,11 +88,21 @@ sandwich_norm_kernel(float* __restrict__ residual, const float* __restrict__ del
   const float inv_d = 1.0f / static_cast<float>(d);
   float ss[1] = {0.f};
   for (int v = v0 + threadIdx.x * V; v < v1; v += kRowT * V) {
-    Vec<V> y = slab_sum_vec<V>(delta + t * d + v, n_partials, partial_stride);
+    Vec<V> y;
+    if (delta) {
+      y = slab_sum_vec<V>(delta + t * d + v, n_partials, partial_stride);
+    } else {
+#pragma unroll
+      for (int k = 0; k < V; ++k) y.x[k] = 0.f;
+    }
     if (extra.bias) y.add(load_vec<V>(extra.bias + v));
-    for (int k = 0; k < extra.per_row; ++k)
-      y.add(slab_sum_vec<V>(extra.rows + static_cast<long long>(extra.index[t * extra.per_row + k]) * d + v,
-                            extra.n_partials, extra.partial_stride));
+    for (int k = 0; k < extra.per_row; ++k) {
+      const Vec<V> row = slab_sum_vec<V>(extra.rows + static_cast<long long>(extra.index[t * extra.per_row + k]) * d + v,
+                                         extra.n_partials, extra.partial_stride);
+      const float f = extra.weight ? extra.weight[t * extra.per_row + k] : 1.0f;
+#pragma unroll
+      for (int j = 0; j < V; ++j) y.x[j] = fmaf(f, row.x[j], y.x[j]);
+    }
     store_vec<V>(stage + v - v0, y);
     ss[0] += y.sumsq();
   }
@@ -100,6 +125,7 @@ sandwich_norm_kernel(float* __restrict__ residual, const float* __restrict__ del
     }
     store_vec<V>(residual + t * d + v, x);
     store_vec<V>(stage + v - v0, x);
+    if (!w_next && xn) store_vec<V>(xn + t * d + v, x);
     ss[0] += x.sumsq();
   }
   if (w_next) {
@@ -232,7 +258,7 @@ static int sandwich_t(float* residual, const float* delta, int n_partials, long 
 int sandwich_norm(float* residual, const float* delta, int n_partials, long long partial_stride,
                   const float* w_post, const float* w_next, void* xn, int act_dtype, int T, int d, float eps,
                   const NormExtra& extra, cudaStream_t st) {
-  if (!residual || !delta || T <= 0 || d <= 0 || d > 51200 || n_partials < 1 || (w_next && !xn)) {
+  if (!residual || (!delta && extra.per_row <= 0) || T <= 0 || d <= 0 || d > 51200 || n_partials < 1 || (w_next && !xn)) {
     set_last_error("bcg_sandwich_norm", "bad argument (d <= 51200)");
     return BCG_ERR_ARG;
   }

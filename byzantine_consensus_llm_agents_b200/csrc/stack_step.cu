@@ -104,11 +104,25 @@ int grouped_attention_step(const bcg_stack* m, const bcg_stack_ws* ws, const bcg
   return l ? grouped_attention(m, ws, b, l, mode, st) : static_cast<int>(BCG_ERR_ARG);
 }
 
+static const bcg_layer* expert_layer(const bcg_stack* m, int layer, bool fits) {
+  if (!fits || layer < 0 || layer >= m->n_layers || m->layers[layer].experts <= 0) {
+    set_last_error("bcg_experts", "the layer has no experts, or a bad batch");
+    return nullptr;
+  }
+  return &m->layers[layer];
+}
+
 int experts_step(const bcg_stack* m, const bcg_stack_ws* ws, int layer, int T, int* splits, cudaStream_t st) {
   BCG_TRY(check_stack(m, ws));
-  const bcg_layer* l = layer_of(m, layer, T > 0 && T <= ws->T_max && splits, "bcg_experts");
-  if (l && l->experts <= 0) set_last_error("bcg_experts", "the layer has no experts");
-  return l && l->experts > 0 ? experts(m, l, ws, T, splits, st) : static_cast<int>(BCG_ERR_ARG);
+  const bcg_layer* l = expert_layer(m, layer, T > 0 && T <= ws->T_max && splits);
+  return l ? experts(m, l, ws, T, splits, st) : static_cast<int>(BCG_ERR_ARG);
+}
+
+int expert_in_step(const bcg_stack* m, const bcg_stack_ws* ws, int layer, int T, int n_partials, long long pstride, long long ld,
+                   int with_act, cudaStream_t st) {
+  BCG_TRY(check_stack(m, ws));
+  const bcg_layer* l = expert_layer(m, layer, T > 0 && T <= ws->T_max && n_partials > 0);
+  return l ? expert_in(m, l, ws, T, n_partials, pstride, ld, with_act != 0, st) : static_cast<int>(BCG_ERR_ARG);
 }
 
 // A parallel layer: attention and feed-forward read one norm, their outputs meet in one residual addition.  The
@@ -144,15 +158,50 @@ static int parallel_layer(const bcg_stack* m, const bcg_stack_ws* ws, const bcg_
                        extra, st);
 }
 
-// Gate and up products with the clamped unit: in the GEMM's epilogue where K is not split, else behind the slabs.
+// Gate and up products with their unit: in the GEMM's epilogue where K is not split, else behind the slabs.
 static int glu_up(const bcg_stack* m, const bcg_stack_ws* ws, const bcg_layer* l, int T, cudaStream_t st) {
-  const int n = 2 * l->ff, d = m->d_model;
+  const int n = 2 * l->ff, d = m->d_model, unit = l->ff_kind == BCG_FF_GELU_GLU ? BCG_EPI_GELU_GLU : BCG_EPI_GLU;
   int s = stack_splits(m->act_dtype, T, n, d);
   if (s == 1 && tensor_gemm(m->act_dtype, T, n, d))
-    return gemm_bf16_glu(ws->xn, l->w_up, ws->act, T, n, d, l->glu_limit, l->glu_alpha, launch_flags() & BCG_GEMM_PDL, st);
+    return gemm_bf16_glu(ws->xn, l->w_up, ws->act, T, n, d, unit, l->glu_limit, l->glu_alpha, launch_flags() & BCG_GEMM_PDL, st);
   BCG_TRY(project(m, ws->xn, l->w_up, ws->proj, ws->proj_floats, T, n, d, &s, st));
-  return clamped_glu_rows(ws->proj, s, static_cast<long long>(T) * n, nullptr, ws->act, m->act_dtype, T, l->ff, l->glu_limit,
-                          l->glu_alpha, st);
+  return unit_rows(ws->proj, s, static_cast<long long>(T) * n, nullptr, ws->act, m->act_dtype, T, l->ff, unit, l->glu_limit,
+                   l->glu_alpha, st);
+}
+
+// Router, experts and the shared expert of a layer that is not parallel, up to their sum with the stream: the router's rows and
+// the shared expert's first matrix are one product; *splits slabs of the shared expert's output are left in ws->proj (0: none).
+static int expert_ff(const bcg_stack* m, const bcg_stack_ws* ws, const bcg_layer* l, int T, NormExtra* extra, int* splits,
+                     cudaStream_t st) {
+  const int d = m->d_model, dt = m->act_dtype, n_all = l->n_router + l->ff;
+  // long launches: the gelu is the shared product's epilogue
+  const bool apart = l->ff > 0 && T > 128 && tensor_gemm(dt, T, l->ff, d) && tensor_gemm(dt, T, l->n_router, d);
+  const int n = apart ? l->n_router : n_all;
+  int s = 1;
+  BCG_TRY(project(m, ws->xn, l->w_up, ws->proj, ws->proj_floats, T, n, d, &s, st));
+  BCG_TRY(expert_in(m, l, ws, T, s, static_cast<long long>(T) * n, n, !apart, st));
+  if (apart)
+    BCG_TRY(gemm_bf16_gelu(ws->xn, static_cast<const char*>(l->w_up) + static_cast<size_t>(l->n_router) * d * 2, ws->act, T, l->ff, d,
+                           launch_flags() & BCG_GEMM_PDL, st));
+  BCG_TRY(experts(m, l, ws, T, &extra->n_partials, st));
+  extra->rows = ws->moe_out;
+  extra->index = ws->moe_row;
+  extra->weight = ws->moe_weight;
+  extra->per_row = l->top;
+  extra->partial_stride = static_cast<long long>(T) * l->top * d;
+  *splits = 0;
+  return l->ff > 0 ? project(m, ws->act, l->w_down, ws->proj, ws->proj_floats, T, d, l->ff, splits, st) : static_cast<int>(BCG_OK);
+}
+
+int matrix_memory_step(const bcg_stack* m, const bcg_stack_ws* ws, const bcg_step_batch* b, int layer, int n_partials,
+                       long long pstride, long long ld, int mode, cudaStream_t st) {
+  BCG_TRY(check_stack(m, ws));
+  if (!b || b->T <= 0 || b->T > ws->T_max || n_partials < 1 || layer < 0 || layer >= m->n_layers ||
+      m->layers[layer].mixer != BCG_MIXER_MATRIX_MEMORY) {
+    set_last_error("bcg_matrix_memory", "not a matrix memory layer, or a bad batch");
+    return BCG_ERR_ARG;
+  }
+  return matrix_memory(m, &m->layers[layer], ws, b, n_partials, pstride, ld, mode, st);
 }
 
 int state_space_step(const bcg_stack* m, const bcg_stack_ws* ws, const bcg_step_batch* b, int layer, int n_partials,
@@ -178,7 +227,7 @@ int stack_step(const bcg_stack* m, const bcg_stack_ws* ws, const bcg_step_batch*
   const void* gathered = nullptr;
   const EmbedArgs embed = {b->ids, b->positions, static_cast<const __nv_bfloat16*>(m->embed), m->embed_scale,
                            static_cast<const __nv_bfloat16*>(m->pos_embed), m->n_pos, m->pos_turns, ws->moe_counts,
-                           ws->moe_counts_n};
+                           ws->moe_counts_n, m->embed_norm};
   BCG_TRY(embed_norm(embed, m->layers[0].norm1, ws->residual, ws->xn, dt, T, d, m->eps, st));
   for (int i = 0; i < m->n_layers; ++i) {
     const bcg_layer* l = &m->layers[i];
@@ -215,6 +264,9 @@ int stack_step(const bcg_stack* m, const bcg_stack_ws* ws, const bcg_step_batch*
         BCG_TRY(grouped_attention(m, ws, b, l, 0, st));
       }
       if (l->ssm_heads > 0) BCG_TRY(state_space(m, l, ws, b, s, in_stride, l->n_in, 0, st));
+    } else if (l->mixer == BCG_MIXER_MATRIX_MEMORY) {
+      mix_out = l->mix_ld;
+      BCG_TRY(matrix_memory(m, l, ws, b, s, in_stride, l->n_in, 0, st));
     } else {
       set_last_error("bcg_stack_step", "unknown mixer");
       return BCG_ERR_UNSUPPORTED;
@@ -222,10 +274,16 @@ int stack_step(const bcg_stack* m, const bcg_stack_ws* ws, const bcg_step_batch*
     BCG_TRY(project(m, ws->mix, l->w_out, ws->proj, ws->proj_floats, T, d, mix_out, &s, st));
     NormExtra extra;
     extra.bias = l->out_bias;
-    BCG_TRY(sandwich_norm(ws->residual, ws->proj, s, static_cast<long long>(T) * d, l->norm1b, l->ff ? l->norm2 : next,
+    const bool has_ff = l->ff > 0 || l->ff_kind == BCG_FF_EXPERTS;
+    BCG_TRY(sandwich_norm(ws->residual, ws->proj, s, static_cast<long long>(T) * d, l->norm1b, has_ff ? l->norm2 : next,
                           ws->xn, dt, T, d, m->eps, extra, st));
-    if (l->ff) {
-      if (l->ff_kind == BCG_FF_CLAMPED_GLU) {
+    if (l->ff_kind == BCG_FF_EXPERTS) {
+      NormExtra rows;
+      BCG_TRY(expert_ff(m, ws, l, T, &rows, &s, st));
+      BCG_TRY(sandwich_norm(ws->residual, s ? ws->proj : nullptr, s ? s : 1, static_cast<long long>(T) * d, l->norm2b, next, ws->xn, dt,
+                            T, d, m->eps, rows, st));
+    } else if (l->ff) {
+      if (l->ff_kind == BCG_FF_CLAMPED_GLU || l->ff_kind == BCG_FF_GELU_GLU) {
         BCG_TRY(glu_up(m, ws, l, T, st));
       } else {
         BCG_TRY(project(m, ws->xn, l->w_up, ws->proj, ws->proj_floats, T, l->ff, d, &s, st));

@@ -263,7 +263,7 @@ def _lerazen_kernels(k: _Bench, what: str, B: int, T: int, shape: str, v, plan) 
         k.add("down product", shape, lambda: lib.bcg_gemm_grouped(
             b["moe_h"].data_ptr(), w["w_experts_out"].data_ptr(), b["moe_out"].data_ptr(), rows, d, ff, cp, f.experts, T, s2, None, 0.0,
             0.0, 0, st()), nbytes=used * 2.0 * ff * d + rows * (2.0 * ff + 4.0 * s2 * d), flops=2.0 * rows * ff * d)
-        extra = (b["moe_out"].data_ptr(), b["moe_row"].data_ptr(), top, s2, rows * d)
+        extra = (b["moe_out"].data_ptr(), b["moe_row"].data_ptr(), None, top, s2, rows * d)
     else:
         act_col, cols = cfg.mix_cols(layer)
         out = b["mix"][act_col:]
@@ -272,13 +272,13 @@ def _lerazen_kernels(k: _Bench, what: str, B: int, T: int, shape: str, v, plan) 
             k.gemm("up product", shape, b["xn"], up, out[:T * (cols - act_col)], T, cols - act_col, d, L.EPI_RELU2, 1)
         else:
             k.gemm("up product", shape, b["xn"], w["w_in"], b["proj"], B, n_in, d, L.EPI_F32, s)
-        extra = (None, None, 0, 1, 0)
+        extra = (None, None, None, 0, 1, 0)
     cols = cfg.mix_cols(layer)[1]
     s3 = 1 if prefill else L.splits_for(B, d, cols)
     k.gemm("output product" if moe else "down product", shape, b["mix"], w["w_out"], b["proj"], T, d, cols, L.EPI_F32, s3)
     k.add("norm", shape, lambda: lib.bcg_residual_norm(
-        b["residual"].data_ptr(), b["proj"].data_ptr(), s3, T * d, w["out_bias"].data_ptr(), *extra, w["norm1"].data_ptr(),
-        b["xn"].data_ptr(), L.DT_BF16, T, d, 1e-5, st()), nbytes=T * d * (10.0 + 4 * s3 + 4 * extra[2] * extra[3]))
+        b["residual"].data_ptr(), b["proj"].data_ptr(), s3, T * d, w["out_bias"].data_ptr(), *extra, None, w["norm1"].data_ptr(),
+        b["xn"].data_ptr(), L.DT_BF16, T, d, 1e-5, st()), nbytes=T * d * (10.0 + 4 * s3 + 4 * extra[3] * extra[4]))
 
 
 def _merulorn_kernels(k: _Bench, what: str, B: int, T: int, shape: str, v, plan) -> None:

@@ -33,7 +33,7 @@ import torch
 
 from . import grammar as G
 from . import lib as L
-from .executors import PAGE, PREFILL_TILE, SPLIT_TOKENS, Entry, make_executor
+from .executors import PAGE, PREFILL_TILE, SPLIT_TOKENS, Entry, block_pages_for, make_executor
 from .model import ModelConfig, Weights
 from .tokenizer import CachedEncoder
 
@@ -164,6 +164,7 @@ class LiveSequence:
     """A live sequence of the step interface (Engine.open / step / close)."""
     length: int = 0
     pages: List[int] = field(default_factory=list)
+    blocks: List[List[int]] = field(default_factory=list)      # pages of pooled blocks, one list per block size
     slot: int = 0
 
 
@@ -234,16 +235,19 @@ class Engine:
                 t = torch.tensor([kv_pages], dtype=torch.int64)
                 dist.all_reduce(t, op=dist.ReduceOp.MIN, group=tp_group)
                 kv_pages = int(t.item())
-        self.exec.alloc_cache(kv_pages, self.slots.n)
+        # pages of pooled blocks: as many as the tokens of all pages can fill, and a part of one per sequence
+        block_pages = [kv_pages // p + max(self.slots.n, B) for p, _ in self.exec.block_pools]
+        self.exec.alloc_cache(kv_pages, self.slots.n, block_pages)
         self.kv_layers, self.model = self.exec.kv_layers, self.exec.model
         self.pool = PagePool(kv_pages)
-        # pages alone restore a prefix only where no layer carries a recurrent state
-        self.enable_prefix_cache = enable_prefix_cache and not self.exec.has_state
+        self.block_pools = [PagePool(n) for n in block_pages]
+        # pages alone restore a prefix only where no layer carries a recurrent state or pools blocks of tokens
+        self.enable_prefix_cache = enable_prefix_cache and not self.exec.has_state and not block_pages
         # ---- per-row device state (bcg_sampler_args).  Everything the host writes at the start of a
         # call lives in ONE int32 block with a pinned host mirror, so a call costs one H2D copy
         # instead of one per field.
         fields = [("grammar_id", 1), ("state", 1), ("temperature", 1), ("seed", 2), ("max_tokens", 1),
-                  ("n_out", 1), ("finished", 1), ("seq_lens", 1), ("state_slot", 1), ("block_table", self.max_blocks)]
+                  ("n_out", 1), ("finished", 1), ("seq_lens", 1), ("state_slot", 1), ("block_table", self.exec.table_cols)]
         words = sum(w for _, w in fields) * B
         self._state_dev = z(words, dt=i32)
         self._state_host = torch.zeros(words, dtype=i32).pin_memory()
@@ -319,7 +323,7 @@ class Engine:
         a.B, a.V, a.mask_words, a.max_steps = B, self.lcfg.vocab, self.mask_words, self.max_steps
         stops = list(self.tk.stop_ids) + [-1]
         a.eos_id0, a.eos_id1 = stops[0], stops[1]
-        a.page_size, a.max_blocks_per_seq = PAGE, self.max_blocks
+        a.page_size, a.max_blocks_per_seq = PAGE, self.exec.table_cols
         a.grammar_id = r["grammar_id"].data_ptr()
         a.mask_tables, a.trans_tables = self.mask_ptrs.data_ptr(), self.trans_ptrs.data_ptr()
         a.tok_bytes, a.tok_offsets = self.tok_bytes.data_ptr(), self.tok_offsets.data_ptr()
@@ -374,7 +378,7 @@ class Engine:
         t_host0 = time.perf_counter()
         cfg, B = self.cfg, len(reqs)
         r = self.row
-        ids_list, cached, pages_of, hashes_of, slots_of = [], [], [], [], []
+        ids_list, cached, pages_of, hashes_of, slots_of, blocks_of = [], [], [], [], [], []
         use_forced = any(q.forced is not None for q in reqs)
         for q in reqs:
             ids = list(q.prompt_ids) if q.prompt_ids is not None else self._encode(q.prompt)
@@ -407,33 +411,51 @@ class Engine:
                 while len(pages) < total_pages:
                     pages.append(self.pool.alloc())
                 pages_of.append(pages)
+                blocks_of.append([[] for _ in self.block_pools])
+                self._grow_blocks(blocks_of[-1], len(ids) + q.max_tokens)
                 hashes_of.append(hs)
                 cached.append(hit * PAGE)
                 slots_of.append(self.slots.alloc() if self.exec.has_state else 0)
         except Exception:
-            self._release(pages_of, slots_of)
+            self._release(pages_of, slots_of, blocks_of)
             raise
 
         try:
-            results = self._run(reqs, ids_list, cached, pages_of, hashes_of, slots_of, use_forced, row0, t_host0)
+            results = self._run(reqs, ids_list, cached, pages_of, blocks_of, hashes_of, slots_of, use_forced, row0, t_host0)
         finally:
-            self._release(pages_of, slots_of)
+            self._release(pages_of, slots_of, blocks_of)
         return results
 
-    def _release(self, pages_of, slots_of) -> None:
+    def _grow_blocks(self, blocks: List[List[int]], tokens: int) -> None:
+        """Gives a sequence the pages of pooled blocks that `tokens` tokens fill."""
+        for (size, _), pool, mine in zip(self.exec.block_pools, self.block_pools, blocks):
+            while len(mine) < block_pages_for(tokens, size):
+                mine.append(pool.alloc())
+
+    def _table_row(self, row: np.ndarray, pages: List[int], blocks: List[List[int]]) -> None:
+        """A sequence's row of the block table.  Pages of pooled blocks are numbered behind the tokens' pages."""
+        row[:len(pages)] = pages
+        for (_, col), mine in zip(self.exec.block_pools, blocks):
+            row[col:col + len(mine)] = [self.pool.n_pages + p for p in mine]
+
+    def _release(self, pages_of, slots_of, blocks_of) -> None:
         for pages in pages_of:
             for p in pages:
                 self.pool.release(p)
+        for blocks in blocks_of:
+            for pool, mine in zip(self.block_pools, blocks):
+                for p in mine:
+                    pool.release(p)
         if self.exec.has_state:
             for s in slots_of:
                 self.slots.release(s)
 
-    def _run(self, reqs, ids_list, cached, pages_of, hashes_of, slots_of, use_forced, row0, t_host0):
+    def _run(self, reqs, ids_list, cached, pages_of, blocks_of, hashes_of, slots_of, use_forced, row0, t_host0):
         cfg, B, r, dev = self.cfg, len(reqs), self.row, self.dev
         i32 = torch.int32
-        bt = np.zeros((B, self.max_blocks), np.int32)
+        bt = np.zeros((B, self.exec.table_cols), np.int32)
         for b, pages in enumerate(pages_of):
-            bt[b, :len(pages)] = pages
+            self._table_row(bt[b], pages, blocks_of[b])
         gids = [self.grammar_index(q.schema) for q in reqs]
         seeds = np.array([tuple(q.seed) if q.seed is not None else row_seed(self.base_seed, self.calls, row0 + b)
                           for b, q in enumerate(reqs)], np.uint32)
@@ -618,12 +640,12 @@ class Engine:
     # The step interface: the caller brings the tokens, the engine keeps pages and states.  The same launches
     # as generate(): a batch of single tokens is a decode step, anything else a ragged step.
     def open(self) -> LiveSequence:
-        return LiveSequence(slot=self.slots.alloc() if self.exec.has_state else 0)
+        return LiveSequence(blocks=[[] for _ in self.block_pools], slot=self.slots.alloc() if self.exec.has_state else 0)
 
     def close_sequence(self, seq: LiveSequence) -> None:
         """Gives a sequence's pages and state slot back."""
-        self._release([seq.pages], [seq.slot])
-        seq.pages, seq.length = [], 0
+        self._release([seq.pages], [seq.slot], [seq.blocks])
+        seq.pages, seq.blocks, seq.length = [], [[] for _ in self.block_pools], 0
 
     def step(self, work) -> torch.Tensor:
         """work: [(LiveSequence, token ids, places among them whose logits are wanted)], one batch.  Returns the
@@ -637,8 +659,9 @@ class Engine:
                 raise L.BcgError(f"sequence of {end} tokens exceeds max_model_len ({self.max_model_len})")
             while len(seq.pages) * PAGE < end:
                 seq.pages.append(self.pool.alloc())
-            row = np.zeros(self.max_blocks, np.int32)
-            row[:len(seq.pages)] = seq.pages
+            self._grow_blocks(seq.blocks, end)
+            row = np.zeros(self.exec.table_cols, np.int32)
+            self._table_row(row, seq.pages, seq.blocks)
             done = 0
             while done < len(tokens):           # a portion longer than a launch takes is cut
                 n = min(len(tokens) - done, self.exec.max_tokens_of(seq.length + done))

@@ -3,7 +3,9 @@
 The engine owns scheduling, pages, state slots, row state and sampling; an executor owns the device buffers of
 a model's forward pass and knows how to launch it.  Both kinds offer the same interface:
 
-  buf, page_bytes, state_slot_bytes, alloc_cache(pages, slots)
+  buf, page_bytes, state_slot_bytes, table_cols (columns of the block table)
+  block_pools                   pooled blocks of tokens: [(tokens of a block, first column of the block table)]
+  alloc_cache(pages, slots, block_pages)
   plan(entries)                 host arrays (int32) describing one ragged step over `entries`
   launch(plan, views, row0)     the step: every entry's tokens through the model, the wanted logits into rows
                                 row0.. of buf["logits"]
@@ -24,12 +26,17 @@ import torch
 
 from . import lib as L
 from .model import ModelHandle
-from .stack import GeneralDelta, GroupedAttention, LatentAttention, MoeMlp, StackHandle, StateSpace
+from .stack import GeneralDelta, GroupedAttention, LatentAttention, MatrixMemory, MoeMlp, StackHandle, StateSpace
 
 PAGE = 16
 SPLIT_TOKENS = 256
 PREFILL_TILE = 128      # query rows per prefill-attention CTA
 SINGLE_MAX = 4          # portions up to this long are attended token by token (latent attention)
+
+
+def block_pages_for(tokens: int, pool: int) -> int:
+    """Pages that the whole blocks of `pool` tokens of a sequence fill."""
+    return -(-(tokens // pool) // PAGE)
 
 
 @dataclass
@@ -76,7 +83,8 @@ class DenseExecutor:
         bf, f32, i32 = torch.bfloat16, torch.float32, torch.int32
         z = lambda *s, dt=bf: torch.zeros(*s, dtype=dt, device=dev)
         self.max_splits_cap = (max_model_len + SPLIT_TOKENS - 1) // SPLIT_TOKENS
-        self.max_blocks = (max_model_len + PAGE - 1) // PAGE
+        self.max_blocks = self.table_cols = (max_model_len + PAGE - 1) // PAGE
+        self.block_pools = []
         self.B_max, self.T_max = max(B, logit_rows), T
         lc = lcfg
         splits = [L.splits_for(1, n, k) for n, k in ((lc.qkv_dim, d), (d, lc.n_heads * 128),
@@ -118,7 +126,7 @@ class DenseExecutor:
         # ids | positions | slots | wanted rows | tiles | block table
         self.staging_words = 4 * T + self.B_max + 4 * (T // PREFILL_TILE + B) + B * self.max_blocks + 32
 
-    def alloc_cache(self, pages: int, slots: int):
+    def alloc_cache(self, pages: int, slots: int, block_pages: Sequence[int] = ()):
         self.kv_layers = [torch.zeros(pages, 2, self.lcfg.n_kv_heads, PAGE, 128, dtype=torch.bfloat16, device=self.dev)
                           for _ in range(self.cfg.n_layers)]
         self.model = ModelHandle(self.weights, self.kv_layers, PAGE, self.tp_size)
@@ -186,22 +194,31 @@ class StackExecutor:
     def __init__(self, cfg, weights, dev, *, max_rows: int, T_max: int, max_model_len: int, logit_rows: int, flags: int):
         self.lib, self.cfg, self.lcfg, self.dev, self.flags = L.load(), cfg, cfg, dev, flags
         self.weights, self.has_state = weights, cfg.has_state
-        self.max_blocks = (max_model_len + PAGE - 1) // PAGE
+        self.max_blocks = self.table_cols = (max_model_len + PAGE - 1) // PAGE
+        self.block_pools = []
+        for pool in cfg.pools:
+            self.block_pools.append((pool, self.table_cols))
+            self.table_cols += block_pages_for(max_model_len, pool)
         self.max_model_len, self.T_max, self.D_max = max_model_len, T_max, max_rows
         self.B_max = max(max_rows, logit_rows)
         act, f32, bf = cfg.torch_dtype, torch.float32, torch.bfloat16
         T, D, d = T_max, max_rows, cfg.d_model
-        attn, grouped, delta, ssm = (cfg.mixers(k) for k in (LatentAttention, GroupedAttention, GeneralDelta, StateSpace))
-        mlps = [l.mlp for l in cfg.layers if l.mlp and not l.parallel]
+        attn, grouped, delta, ssm, mem = (cfg.mixers(k) for k in (LatentAttention, GroupedAttention, GeneralDelta, StateSpace,
+                                                                  MatrixMemory))
         moes = [l.mlp for l in cfg.layers if isinstance(l.mlp, MoeMlp)]
+        # rows of the first and columns of the second matrix of feed-forwards of their own
+        mlps = [(l.mlp.router_rows + l.mlp.shared_ld, l.mlp.shared_ld) if isinstance(l.mlp, MoeMlp) else (l.mlp.up_rows, l.mlp.ff_ld)
+                for l in cfg.layers if l.mlp and not l.parallel]
         top = lambda xs: max([8, *xs])
         self.history = min(cfg.max_window - 1 if cfg.max_window else max_model_len, max_model_len)
         expanded = [m for m in attn if m.q_ld and cfg.act_dtype == "bfloat16"]
         self.K_max = T + min(T, max_rows * self.history) if expanded else 0
         wide = act == bf
         shapes = [(cfg.in_rows(i), d) for i in range(cfg.n_layers)]
-        for i, l in enumerate(cfg.layers):
-            shapes += [(d, cfg.mix_cols(i)[1])] + ([(l.mlp.up_rows, d), (d, l.mlp.ff_ld)] if l.mlp in mlps else [])
+        for i in range(cfg.n_layers):
+            shapes.append((d, cfg.mix_cols(i)[1]))
+        for up, down in mlps:
+            shapes += [(up, d)] + ([(d, down)] if down else [])
         slabs = lambda n, k: min(T, 128) * n * (L.splits_for(1, n, k) if wide else 1)
         proj = max([T * n for n, _ in shapes] + [slabs(n, k) for n, k in shapes])
         dec = max([8] + [max(T * m.out_dim, slabs(m.out_dim, m.rank_ld)) for m in delta])
@@ -210,7 +227,7 @@ class StackExecutor:
         # experts: rows are (token, choice) pairs; long bf16 launches keep gate and up in the GEMM's epilogue
         choices = max([m.top for m in moes], default=0)
         cut = lambda m, n, k: min(T, 128) * m.top * n * (L.splits_for(1, m.top * n, k) if wide else 1)
-        moe_in = top([cut(m, 2 * m.ff_ld, d) for m in moes] + [T * m.top * 2 * m.ff_ld for m in moes
+        moe_in = top([cut(m, m.in_rows, d) for m in moes] + [T * m.top * m.in_rows for m in moes
                                                              if not (wide and d % 8 == 0 and m.experts <= L.MAX_GROUPS)])
         moe_out = top([max(T * m.top * d, cut(m, d, m.ff_ld)) for m in moes])
         counts = sum(m.experts for m in moes)
@@ -225,9 +242,11 @@ class StackExecutor:
             moe_rank=z(T * choices + 8, torch.int32), moe_weight=z(T * choices + 8, f32),
             moe_row=z(T * choices + 8, torch.int32), moe_row_weight=z(T * choices + 8, f32),
             moe_counts=z(counts + 8, torch.int32),
-            act=z(T * top(m.ff_ld for m in mlps), act), gates=z(T * top(m.heads for m in grouped if m.gate), f32),
-            ssm_x=z(T * top(m.x_ld for m in ssm) if ssm else 8, act), ssm_step=z(T * top(m.heads for m in ssm) if ssm else 8, f32),
-            ssm_y=z(T * top(m.out_dim for m in ssm) if ssm else 8, act), low=z(T * top(m.rank_ld for m in delta), act),
+            act=z(T * top(down for _, down in mlps), act), gates=z(T * top(m.heads for m in grouped if m.gate), f32),
+            ssm_x=z(T * top(m.x_ld for m in ssm + mem) if ssm or mem else 8, act),
+            ssm_step=z(T * top(m.heads for m in ssm) if ssm else 8, f32),
+            ssm_y=z(T * top(m.out_dim for m in ssm + mem) if ssm or mem else 8, act),
+            mem_den=z(T * top(m.heads for m in mem) if mem else 8, f32), low=z(T * top(m.rank_ld for m in delta), act),
             latents=z(max(8, self.K_max * top(m.cache_row for m in expanded)), bf),
             expanded=z(max(8, self.K_max * top(m.heads * (m.q_ld + m.v_ld) for m in expanded)), bf),
             q_latent=z(D * top(m.heads * m.cache_row for m in attn) if wide else 8, bf),
@@ -241,21 +260,25 @@ class StackExecutor:
         ws.moe_proj_floats, ws.moe_out_floats, ws.moe_counts_n, ws.moe_rows_max = moe_in, moe_out, counts, T * choices
         ws.T_max, ws.K_max, ws.D_max, ws.B_max = T, self.K_max, D, self.B_max
         self.ws = ws
-        self.page_bytes = PAGE * cfg.kv_bytes_per_token
+        self.page_bytes = PAGE * cfg.kv_bytes_per_token + sum(-(-PAGE * cfg.pool_bytes_per_block(p) // p) for p in cfg.pools)
         self.state_slot_bytes = cfg.state_bytes_per_row
         # ids | positions | slots | row_seq | wanted rows (<= T) | seq_start, state slots | singles | tiles | gather | bt
         self.staging_words = 5 * T + 4 * (2 * max_rows + 2) + 8 * (T // PREFILL_TILE + max_rows + 1) + T + self.K_max + \
-            max_rows * self.max_blocks + 64
+            max_rows * self.table_cols + 64
 
-    def alloc_cache(self, pages: int, slots: int):
+    def alloc_cache(self, pages: int, slots: int, block_pages: Sequence[int] = ()):
+        """block_pages: pages of every entry of block_pools, numbered from `pages` on."""
         self.caches = []
+        extra = {pool: n for (pool, _), n in zip(self.block_pools, block_pages)}
         for l in self.cfg.layers:
-            m, att, ssm = l.mixer, l.one(GroupedAttention), l.one(StateSpace)
+            m, att, ssm, mem = l.mixer, l.one(GroupedAttention), l.one(StateSpace), l.one(MatrixMemory)
             z = lambda *s, dt=torch.float32: torch.zeros(*s, dtype=dt, device=self.dev)
-            if att or ssm:
+            if att or ssm or mem:
                 t = {}
+                if mem:
+                    t.update(mem_state=z(slots, mem.heads, mem.vdim + 1, mem.dim), mem_max=z(slots, mem.heads, mem.blocks))
                 if att:
-                    t.update({n: z(pages, att.kv_heads, PAGE, ld, dt=self.cfg.torch_dtype)
+                    t.update({n: z(pages + (extra[att.pool] if att.pool else 0), att.kv_heads, PAGE, ld, dt=self.cfg.torch_dtype)
                               for n, ld in (("cache", att.q_ld), ("cache_v", att.v_ld))})
                 if ssm:
                     t.update(ssm_state=z(slots, ssm.heads, ssm.vdim, ssm.state), conv_state=z(slots, ssm.conv - 1, ssm.channels))
@@ -266,7 +289,7 @@ class StackExecutor:
                     if m.kv_from is None else None
             self.caches.append(t)
         self.kv_layers = [c for c in self.caches if c is not None]
-        self.model = StackHandle(self.weights, self.caches, self.max_model_len, PAGE)
+        self.model = StackHandle(self.weights, self.caches, self.max_model_len, PAGE, dict(self.block_pools))
 
     def max_tokens_of(self, start: int) -> int:
         if not self.K_max:
@@ -308,7 +331,7 @@ class StackExecutor:
     def _batch(self, T, n_seqs) -> L.StepBatch:
         b = L.StepBatch()
         # programmatic dependent launch pays for short kernels; long ones only occupy SMs while they wait
-        b.T, b.n_seqs, b.max_blocks, b.flags = T, n_seqs, self.max_blocks, self.flags & L.GEMM_PDL if T <= 128 else 0
+        b.T, b.n_seqs, b.max_blocks, b.flags = T, n_seqs, self.table_cols, self.flags & L.GEMM_PDL if T <= 128 else 0
         return b
 
     def _run(self, b: L.StepBatch) -> None:
@@ -342,10 +365,15 @@ class StackExecutor:
                 n += 5 + (4 if isinstance(l.mlp, MoeMlp) else 0)
                 continue
             if l.composed:
-                # input projection, attention's split and kernel, state space (convolution,) recurrence and norm, output
-                # projection, norm; feed-forward: up, its unit where K is split, down, norm
-                n += 3 + (2 if l.one(GroupedAttention) else 0) + ((2 if decode else 3) if l.one(StateSpace) else 0)
-                if l.mlp:
+                # input projection, attention's split (, pooled blocks) and kernel, state space or matrix memory (convolution or
+                # split,) recurrence and norm, output projection, norm; feed-forward: up, its unit where K is split, down, norm;
+                # experts: router and shared rows, routing, scatter, two products, unit, shared output, norm
+                att = l.one(GroupedAttention)
+                n += 3 + (2 if att else 0) + int(bool(att and att.pool and not decode))
+                n += (2 if decode else 3) if l.one(StateSpace) or l.one(MatrixMemory) else 0
+                if isinstance(l.mlp, MoeMlp):
+                    n += 6 + int(decode) + int(l.mlp.shared > 0) * (1 if decode else 2)
+                elif l.mlp:
                     n += 3 + int(not l.mlp.glu or decode and L.splits_for(1, l.mlp.up_rows, d) > 1)
                 continue
             # input projection, mixer (delta: low rank, decay projection, scan; attention: qkv, absorb, decode,

@@ -19,8 +19,8 @@ STEP_FUSED_ROPE = 0x80000     # bcg_model_decode: qk-norm/RoPE/KV-write folded i
 STEP_DEFERRED_NORM = 0x40000  # bcg_model_decode: norm statistics kernel + 1/RMS in the next GEMM's epilogue
 
 DT_BF16, DT_F32 = 0, 1                          # activation dtype of a layer stack
-MIXER_LATENT_ATTN, MIXER_GENERAL_DELTA, MIXER_GROUPED_ATTN, MIXER_STATE_SPACE = 1, 2, 3, 4
-FF_POLY_NORM, FF_CLAMPED_GLU = 0, 1             # Layer.ff_kind
+MIXER_LATENT_ATTN, MIXER_GENERAL_DELTA, MIXER_GROUPED_ATTN, MIXER_STATE_SPACE, MIXER_MATRIX_MEMORY = 1, 2, 3, 4, 5
+FF_POLY_NORM, FF_CLAMPED_GLU, FF_GELU_GLU, FF_EXPERTS = 0, 1, 2, 3      # Layer.ff_kind
 MAX_GROUPS = 512                                # experts the grouped tensor-core GEMM takes
 VALUES_FIRST, VALUES_MIX = 1, 2                 # Layer.v_role
 
@@ -102,6 +102,9 @@ class Layer(C.Structure):
         ("ssm_norm_parts", C.c_int), ("ssm_taps", C.c_int), ("ssm_col", C.c_int), ("ssm_mix_col", C.c_int),
         ("conv_w", vp), ("conv_b", vp), ("step_bias", vp), ("decay_rate", vp), ("skip", vp), ("ssm_norm", vp),
         ("ssm_state", vp), ("conv_state", vp),
+        ("by_head", C.c_int), ("rot_pairs", C.c_int), ("v_rot_dims", C.c_int), ("v_cos_sin", vp), ("pool", C.c_int),
+        ("pool_col", C.c_int), ("gate_cap", C.c_float), ("mem_bias", vp), ("mem_norm", vp), ("mem_state", vp), ("mem_max", vp),
+        ("n_router", C.c_int), ("router_bias", vp),
     ]
 
 
@@ -110,7 +113,7 @@ class Stack(C.Structure):
         ("n_layers", C.c_int), ("d_model", C.c_int), ("vocab_ld", C.c_int), ("act_dtype", C.c_int),
         ("page_size", C.c_int), ("eps", C.c_float), ("embed", vp), ("lm_head", vp), ("final_norm", vp),
         ("layers", C.POINTER(Layer)), ("pos_embed", vp), ("n_pos", C.c_int),
-        ("embed_scale", C.c_float), ("pos_turns", vp),
+        ("embed_scale", C.c_float), ("pos_turns", vp), ("embed_norm", vp),
     ]
 
 
@@ -124,6 +127,7 @@ class StackWs(C.Structure):
         ("moe_proj_floats", C.c_longlong), ("moe_out", vp), ("moe_out_floats", C.c_longlong), ("moe_expert", vp),
         ("moe_rank", vp), ("moe_weight", vp), ("moe_row", vp), ("moe_row_weight", vp), ("moe_counts", vp),
         ("moe_counts_n", C.c_int), ("moe_rows_max", C.c_int), ("gates", vp), ("ssm_x", vp), ("ssm_step", vp), ("ssm_y", vp),
+        ("mem_den", vp),
     ]
 
 
@@ -182,7 +186,7 @@ _SIGS = {
                                C.c_longlong, vp]),
     "bcg_sandwich_norm": (C.c_int, [vp, vp, C.c_int, C.c_longlong, vp, vp, vp, C.c_int, C.c_int, C.c_int, C.c_float,
                                     vp]),
-    "bcg_residual_norm": (C.c_int, [vp, vp, C.c_int, C.c_longlong, vp, vp, vp, C.c_int, C.c_int, C.c_longlong, vp, vp,
+    "bcg_residual_norm": (C.c_int, [vp, vp, C.c_int, C.c_longlong, vp, vp, vp, vp, C.c_int, C.c_int, C.c_longlong, vp, vp, vp,
                                     C.c_int, C.c_int, C.c_int, C.c_float, vp]),
     "bcg_poly_norm": (C.c_int, [vp, C.c_int, C.c_longlong, vp, vp, C.c_int, C.c_int, C.c_int, C.c_float, vp]),
     "bcg_delta_scan": (C.c_int, [C.POINTER(Layer), vp, C.c_int, C.c_longlong, C.c_longlong, vp, C.c_int,
@@ -199,6 +203,13 @@ _SIGS = {
                                   C.c_longlong, C.c_longlong, C.c_int, vp]),
     "bcg_clamped_glu": (C.c_int, [vp, C.c_int, C.c_longlong, vp, C.c_int, C.c_int, C.c_int, C.c_float, C.c_float, vp]),
     "bcg_gemm_bf16_glu": (C.c_int, [vp, vp, vp, C.c_int, C.c_int, C.c_int, C.c_float, C.c_float, C.c_int, vp]),
+    "bcg_gelu_unit": (C.c_int, [vp, C.c_int, C.c_longlong, vp, C.c_int, C.c_int, C.c_int, C.c_int, vp]),
+    "bcg_gemm_bf16_gelu": (C.c_int, [vp, vp, vp, C.c_int, C.c_int, C.c_int, C.c_int, C.c_int, vp]),
+    "bcg_gemm_grouped_gelu": (C.c_int, [vp, vp, vp, C.c_int, C.c_int, C.c_int, vp, C.c_int, C.c_int, C.c_int, vp]),
+    "bcg_expert_in": (C.c_int, [C.POINTER(Stack), C.POINTER(StackWs), C.c_int, C.c_int, C.c_int, C.c_longlong, C.c_longlong, C.c_int,
+                                vp]),
+    "bcg_matrix_memory": (C.c_int, [C.POINTER(Stack), C.POINTER(StackWs), C.POINTER(StepBatch), C.c_int, C.c_int,
+                                    C.c_longlong, C.c_longlong, C.c_int, vp]),
     "bcg_experts": (C.c_int, [C.POINTER(Stack), C.POINTER(StackWs), C.c_int, C.c_int, c_int_p, vp]),
 }
 

@@ -1,8 +1,8 @@
 """Layer stacks: models whose layers differ in kind, described by composable specs.
 
 A `StackConfig` lists layers; each has a mixer spec (`LatentAttention`, `GeneralDelta`, `GroupedAttention`, `StateSpace`,
-or two of them `SideBySide`), optionally a feed-forward spec (`DenseMlp`, `MoeMlp`), and norms before, or before and
-after, every sublayer or, in a parallel layer, one norm in front of both.  Which design a model directory
+`MatrixMemory`, or two of them `SideBySide`), optionally a feed-forward spec (`DenseMlp`, `MoeMlp`), and norms before, after,
+or before and after every sublayer or, in a parallel layer, one norm in front of both.  Which design a model directory
 holds is decided by config.json's "architecture" (`DESIGNS`, consulted by model.config_from_dir); a design is
 a reader from its config.json to specs, everything below the specs is shared.  `StackWeights` loads and packs
 the tensors for the kernels (include/bcg_b200.h, bcg_layer); there is nothing model-specific in the engine.
@@ -30,9 +30,11 @@ def _up(n: int, m: int) -> int:
 # ------------------------------------------------------------------------------------------ specs
 @dataclass(frozen=True)
 class Rotary:
-    """Rotate-half over the first `dims` entries of the rotated part, frequencies base^(-2i/dims)."""
+    """The first `dims` entries of the rotated part turn, frequencies base^(-2i/dims): entry i with dims / 2 + i or, with
+    `pairs`, 2i with 2i + 1."""
     base: float
     dims: int
+    pairs: bool = False
 
 
 @dataclass(frozen=True)
@@ -114,9 +116,10 @@ class GeneralDelta:
 
 @dataclass(frozen=True)
 class GroupedAttention:
-    """Grouped-query attention without rotation: biased projections, queries scaled by 1 + temp_coef *
-    ln(floor((position + 1) / temp_every) + 1); optionally a linear distance bias per head, RMS norms of a token's
-    queries and of its keys over all heads at once, an output gate per head."""
+    """Grouped-query attention: queries scaled by 1 + temp_coef * ln(floor((position + 1) / temp_every) + 1); optionally
+    biased projections, a linear distance bias per head, RMS norms of a token's queries and of its keys over all heads at
+    once or head by head, rotated queries and keys, rotated values whose sum is turned back, an output gate per head.
+    Behind a window, means of whole blocks of `pool` tokens may stand for the tokens that have left it."""
     heads: int
     kv_heads: int
     dim: int
@@ -130,6 +133,11 @@ class GroupedAttention:
     qk_norm: bool = False
     gate: bool = False              # head outputs times sigmoid of a projection
     out_bias: bool = True
+    in_bias: bool = True
+    head_norm: bool = False         # every head by its own root mean square, one weight for all heads
+    rot: Optional[Rotary] = None    # queries and keys
+    v_rot: Optional[Rotary] = None  # values; outputs are turned back by the query's position
+    pool: int = 0                   # tokens of a block; 0: what has left the window is not seen
 
     @property
     def out_dim(self) -> int:
@@ -147,6 +155,11 @@ class GroupedAttention:
     q_row = q_ld
 
     @property
+    def by_head(self) -> bool:
+        """Heads are normed or rotated one by one on the way from the projection."""
+        return self.head_norm or self.rot is not None or self.v_rot is not None
+
+    @property
     def cache_row(self) -> int:
         """Cache elements of one token."""
         return self.kv_heads * (self.q_ld + self.v_ld)
@@ -161,8 +174,10 @@ class GroupedAttention:
         for n, rows, cols in (("q", self.heads * self.dim, d), ("k", self.kv_heads * self.dim, d),
                               ("v", self.kv_heads * self.vdim, d), ("o", d, self.out_dim)):
             out[n] = (rows, cols)
-            if n != "o" or self.out_bias:
+            if self.out_bias if n == "o" else self.in_bias:
                 out[n + ".b"] = (rows,)
+        if self.head_norm:
+            out.update({"q.norm": (self.dim,), "k.norm": (self.dim,)})
         if self.qk_norm:
             out.update({"q.norm": (self.heads * self.dim,), "k.norm": (self.kv_heads * self.dim,)})
         if self.gate:
@@ -213,6 +228,48 @@ class StateSpace:
 
 
 @dataclass(frozen=True)
+class MatrixMemory:
+    """Matrix memory with exponential gates: a [vdim, dim] fp32 state, a normalizer row and a running maximum of the log
+    gates per head; log gates are limited softly to +-gate_cap."""
+    heads: int
+    dim: int
+    vdim: int
+    gate_cap: float
+
+    @property
+    def out_dim(self) -> int:
+        return self.heads * self.vdim
+
+    @property
+    def gate_col(self) -> int:
+        """First gate row of the input projection q | k | v | output gate | input and forget gates."""
+        return _up(2 * self.heads * (self.dim + self.vdim), 16)
+
+    @property
+    def in_dim(self) -> int:
+        return self.gate_col + 2 * self.heads
+
+    @property
+    def x_ld(self) -> int:
+        """Columns of the projections as activations, heads padded: q | k | v | output gate."""
+        return 2 * self.heads * (_up(self.dim, 8) + _up(self.vdim, 8))
+
+    @property
+    def blocks(self) -> int:
+        """Blocks of a head's state rows; each keeps the running maximum."""
+        return (self.vdim + 63) // 64
+
+    @property
+    def state_floats(self) -> int:
+        return self.heads * ((self.vdim + 1) * self.dim + self.blocks)
+
+    def tensors(self, d: int) -> Dict[str, tuple]:
+        nk, n, H = self.heads * self.dim, self.out_dim, self.heads
+        return {"q": (nk, d), "k": (nk, d), "v": (n, d), "g": (n, d), "i": (H, d), "i.b": (H,), "f": (H, d), "f.b": (H,),
+                "norm": (n,), "o": (d, n)}
+
+
+@dataclass(frozen=True)
 class SideBySide:
     """left_scale * left(h) + right_scale * right(h)."""
     left: GroupedAttention
@@ -227,15 +284,16 @@ class SideBySide:
 @dataclass(frozen=True)
 class DenseMlp:
     """down(act(up(x))); act is PolyNorm, whose four numbers are weights, or the square of relu, or a gated unit: gate
-    clamped from above, linear part from both sides, gate * sigmoid(alpha * gate) * (linear + 1)."""
+    clamped from above, linear part from both sides, gate * sigmoid(alpha * gate) * (linear + 1), or the tanh form of
+    gelu of the gate times the linear part."""
     ff: int
-    act: str = "poly_norm"          # or "relu2", "clamped_glu"
+    act: str = "poly_norm"          # or "relu2", "clamped_glu", "gelu_glu"
     limit: float = 0.0
     alpha: float = 1.702
 
     @property
     def glu(self) -> bool:
-        return self.act == "clamped_glu"
+        return self.act in ("clamped_glu", "gelu_glu")
 
     @property
     def ff_ld(self) -> int:
@@ -257,22 +315,50 @@ class DenseMlp:
 
 @dataclass(frozen=True)
 class MoeMlp:
-    """`experts` gated units (gate clamped from above, linear part from both sides, sigmoid(alpha * gate)), of which
-    a token uses the `top` with the largest sigmoid scores; a score scales its expert's input."""
+    """`experts` units of which a token uses the `top` with the largest router logits.  "clamped_glu" (parallel layers): gated
+    units (gate clamped from above, linear part from both sides, sigmoid(alpha * gate)), a sigmoid score scales its expert's
+    input.  "gelu" (other layers): down(gelu(up(x))) with the erf form, biased logits, the softmax over the chosen ones scales
+    the outputs; beside them an expert of `shared` inner size that every token uses."""
     experts: int
     top: int
     ff: int
-    limit: float
+    limit: float = 0.0
     alpha: float = 1.702
+    act: str = "clamped_glu"        # or "gelu"
+    shared: int = 0                 # 0: none
 
     @property
     def ff_ld(self) -> int:
         return _up(self.ff, 16)
 
+    @property
+    def glu(self) -> bool:
+        return self.act == "clamped_glu"
+
+    @property
+    def in_rows(self) -> int:
+        """Rows of an expert's first matrix."""
+        return 2 * self.ff_ld if self.glu else self.ff_ld
+
+    @property
+    def router_rows(self) -> int:
+        """Layers that are not parallel: rows of the router in front of the shared expert's."""
+        return _up(self.experts, 16)
+
+    @property
+    def shared_ld(self) -> int:
+        return _up(self.shared, 16)
+
     def tensors(self, d: int) -> Dict[str, tuple]:
         t = {"router": (self.experts, d)}
+        names = ("gate", "up", "down") if self.glu else ("up", "down")
+        each = lambda p, ff: {f"{p}.{n}": (d, ff) if n == "down" else (ff, d) for n in names}
+        if not self.glu:
+            t["router.b"] = (self.experts,)
         for e in range(self.experts):
-            t.update({f"e{e}.gate": (self.ff, d), f"e{e}.up": (self.ff, d), f"e{e}.down": (d, self.ff)})
+            t.update(each(f"e{e}", self.ff))
+        if self.shared:
+            t.update(each("shared", self.shared))
         return t
 
 
@@ -282,6 +368,8 @@ class LayerSpec:
     mlp: object = None
     parallel: bool = False          # x += mixer(h) + ff(h) with one norm h of x
     post_norm: bool = True          # the sublayers' outputs are normed too (layers that are not parallel)
+    pre_norm: bool = True           # False: the sublayers read the stream itself; norm1 and norm2 are their outputs' norms
+    layer_scale: bool = False       # the sublayers' outputs are multiplied by ls1 and ls2 (behind their norms)
 
     @property
     def mixers(self) -> tuple:
@@ -294,8 +382,19 @@ class LayerSpec:
 
     @property
     def composed(self) -> bool:
-        """Grouped attention and / or a state-space mixer behind one input projection."""
-        return not self.parallel and all(isinstance(m, (GroupedAttention, StateSpace)) for m in self.mixers)
+        """Grouped attention and / or a state-space mixer, or a matrix memory, behind one input projection."""
+        return not self.parallel and all(isinstance(m, (GroupedAttention, StateSpace, MatrixMemory)) for m in self.mixers)
+
+    @property
+    def norms(self) -> tuple:
+        """Checkpoint names of the norms and scales."""
+        if self.parallel:
+            return ("norm1",)
+        parts = ("1", "2") if self.mlp else ("1",)
+        out = tuple(f"norm{p}" for p in parts)
+        if self.pre_norm and self.post_norm:
+            out += tuple(f"norm{p}b" for p in parts)
+        return out + (tuple(f"ls{p}" for p in parts) if self.layer_scale else ())
 
 
 @dataclass(frozen=True)
@@ -312,6 +411,9 @@ class StackConfig:
     sinusoid_pos: bool = False       # sines and cosines of position * 10000^(-2i / d_model) are added to the embedding
     embed_scale: float = 1.0
     norm_offset: float = 0.0         # added to the stored weights of the layers' and the final norm
+    embed_norm: bool = False         # the embedding is normed
+    tied_head: bool = False          # logits are products with the embedding
+    logit_scale: float = 1.0
 
     def __post_init__(self):
         if self.act_dtype not in ("bfloat16", "float32"):
@@ -319,12 +421,19 @@ class StackConfig:
         for i, l in enumerate(self.layers):
             m = l.mixer
             att, ssm = l.one(GroupedAttention), l.one(StateSpace)
-            if l.parallel and not isinstance(m, GroupedAttention) or isinstance(l.mlp, MoeMlp) and not l.parallel:
-                raise ValueError(f"{self.name}: layer {i}: parallel layers have grouped attention, experts come in parallel layers")
+            if l.parallel and not isinstance(m, GroupedAttention):
+                raise ValueError(f"{self.name}: layer {i}: parallel layers have grouped attention")
+            if isinstance(l.mlp, MoeMlp) and l.mlp.glu != l.parallel:
+                raise ValueError(f"{self.name}: layer {i}: gated experts come in parallel layers, plain ones in the others")
             if l.mlp and isinstance(l.mlp, DenseMlp) and (l.mlp.act == "relu2") != l.parallel:
                 raise ValueError(f"{self.name}: layer {i}: activation {l.mlp.act!r} in this kind of layer")
-            if l.parallel and (att.qk_norm or att.gate):
-                raise ValueError(f"{self.name}: layer {i}: query and key norms and gates come in layers that are not parallel")
+            if l.parallel and (att.qk_norm or att.gate or att.by_head):
+                raise ValueError(f"{self.name}: layer {i}: query and key norms, rotation and gates come in layers that are not parallel")
+            if not l.pre_norm and (l.parallel or not l.post_norm):
+                raise ValueError(f"{self.name}: layer {i}: norms in front of the sublayers, behind them, or both")
+            mem = l.one(MatrixMemory)
+            if mem and (isinstance(m, SideBySide) or not 0 < mem.dim <= 256 or mem.gate_cap <= 0):
+                raise ValueError(f"{self.name}: layer {i}: a matrix memory stands alone and takes up to 256 key channels per head")
             if isinstance(m, SideBySide) and (att is None or ssm is None or att.out_bias):
                 raise ValueError(f"{self.name}: layer {i}: side by side are grouped attention without output bias and a state-space mixer")
             if ssm and (ssm.heads % ssm.groups or ssm.out_dim % ssm.norm_groups or not 0 < ssm.state <= 256 or ssm.conv < 1):
@@ -332,6 +441,15 @@ class StackConfig:
             if isinstance(l.mlp, MoeMlp) and not 0 < l.mlp.top <= l.mlp.experts <= 1024:
                 raise ValueError(f"{self.name}: layer {i}: {l.mlp.top} of {l.mlp.experts} experts (at most 1,024)")
             if att:
+                if att.by_head and (att.qk_norm or att.gate or att.v_mix or att.slopes or att.temp_coef):
+                    raise ValueError(f"{self.name}: layer {i}: norms by head and rotation do not come with norms over all heads, "
+                                     "gates, mixed values, distance bias or query temperature")
+                if att.rot and (att.rot.dims % 2 or not 0 <= att.rot.dims <= att.dim):
+                    raise ValueError(f"{self.name}: layer {i}: rotary dims {att.rot.dims} of {att.dim}")
+                if att.v_rot and (not att.v_rot.pairs or att.v_rot.dims % 2 or not 0 <= att.v_rot.dims <= att.vdim):
+                    raise ValueError(f"{self.name}: layer {i}: values rotate in pairs of neighbours")
+                if att.pool and (att.window <= 0 or att.pool < 0 or att.slopes):
+                    raise ValueError(f"{self.name}: layer {i}: pooled blocks stand behind a window, without distance bias")
                 if att.heads % att.kv_heads:
                     raise ValueError(f"{self.name}: layer {i}: {att.heads} query heads on {att.kv_heads} key/value heads")
                 if att.v_mix:
@@ -369,7 +487,12 @@ class StackConfig:
     @property
     def has_state(self) -> bool:
         """True when a prefix's cache pages alone do not restore it (recurrent layers)."""
-        return bool(self.mixers(GeneralDelta, StateSpace))
+        return bool(self.mixers(GeneralDelta, StateSpace, MatrixMemory))
+
+    @property
+    def pools(self) -> Tuple[int, ...]:
+        """Block sizes of pooled keys; each has pages and columns of the block table of its own."""
+        return tuple(sorted({m.pool for m in self.mixers(GroupedAttention) if m.pool}))
 
     @property
     def max_window(self) -> int:
@@ -390,18 +513,22 @@ class StackConfig:
         return sum(m.cache_row for m in self.mixers(LatentAttention, GroupedAttention)
                    if getattr(m, "kv_from", None) is None) * self.itemsize
 
+    def pool_bytes_per_block(self, pool: int) -> int:
+        """Bytes of one pooled block of `pool` tokens, all layers that have such blocks."""
+        return sum(m.cache_row for m in self.mixers(GroupedAttention) if m.pool == pool) * self.itemsize
+
     @property
     def state_bytes_per_row(self) -> int:
         return sum(4 * m.heads * m.dim ** 2 for m in self.mixers(GeneralDelta)) + \
-            sum(4 * m.state_floats for m in self.mixers(StateSpace))
+            sum(4 * m.state_floats for m in self.mixers(StateSpace, MatrixMemory))
 
     def in_rows(self, i: int) -> int:
         """Rows of layer i's fused input projection, padded for the 256-wide GEMM tiles when it is large."""
         if self.layers[i].parallel:
             return self.qkv_rows(i) + self.up_rows(i)
         if self.layers[i].composed:
-            ssm = self.layers[i].one(StateSpace)
-            n = self.ssm_col(i) + (ssm.in_dim if ssm else 0)
+            ssm, mem = self.layers[i].one(StateSpace), self.layers[i].one(MatrixMemory)
+            n = mem.in_dim if mem else self.ssm_col(i) + (ssm.in_dim if ssm else 0)
         else:
             n = self.layers[i].mixer.in_rows()
         return _up(n, 256 if n >= 2048 else 16)
@@ -430,8 +557,8 @@ class StackConfig:
     def mix_cols(self, i: int) -> Tuple[int, int]:
         """(first activation column, columns) of what layer i's output projection reads."""
         if self.layers[i].composed:
-            ssm = self.layers[i].one(StateSpace)
-            n = _up(self.ssm_mix_col(i) + (ssm.out_dim if ssm else 0), 8)
+            own = self.layers[i].one(StateSpace) or self.layers[i].one(MatrixMemory)
+            n = _up(self.ssm_mix_col(i) + (own.out_dim if own else 0), 8)
             return n, n
         n = self.layers[i].mixer.out_dim
         return (_up(n, 8), _up(n, 8) + self.up_rows(i)) if self.layers[i].parallel else (n, n)
@@ -439,14 +566,15 @@ class StackConfig:
     def tensor_shapes(self) -> Dict[str, tuple]:
         """Every tensor of the checkpoint, name -> shape."""
         d = self.d_model
-        out = {"embed": (self.vocab, d), "final.norm": (d,), "head": (self.vocab, d)}
+        out = {"embed": (self.vocab, d), "final.norm": (d,)}
+        if not self.tied_head:
+            out["head"] = (self.vocab, d)
+        if self.embed_norm:
+            out["embed.norm"] = (d,)
         if self.learned_pos:
             out["pos"] = (self.max_pos, d)
         for i, l in enumerate(self.layers):
-            norms = ("norm1",) if l.parallel else ("norm1", "norm1b") + (("norm2", "norm2b") if l.mlp else ())
-            if not l.post_norm:
-                norms = tuple(n for n in norms if not n.endswith("b"))
-            out.update({f"l{i}.{n}": (d,) for n in norms})
+            out.update({f"l{i}.{n}": (d,) for n in l.norms})
             out.update({f"l{i}.mix.{n}": s for n, s in l.mixer.tensors(d).items()})
             if l.mlp:
                 out.update({f"l{i}.mlp.{n}": s for n, s in l.mlp.tensors(d).items()})
@@ -457,7 +585,7 @@ class StackConfig:
         use on average when they choose at random (None: all of them)."""
         total = 0.0
         for n, s in self.tensor_shapes().items():
-            if len(s) == 2 and n not in ("embed", "pos"):
+            if len(s) == 2 and n not in (("pos",) if self.tied_head else ("embed", "pos")):
                 f = self.layers[int(n[1:n.index(".")])].mlp if ".mlp.e" in n else None
                 used = 1.0 - (1.0 - f.top / f.experts) ** rows if f and rows is not None else 1.0
                 total += 2 * s[0] * s[1] * used
@@ -550,7 +678,37 @@ def _merulorn(c: dict, shape: Callable[[str], tuple], name: str) -> StackConfig:
                        norm_offset=1.0)
 
 
-DESIGNS: Dict[str, Callable] = {"Bekopel": _bekopel, "Lerazen": _lerazen, "Merulorn": _merulorn}
+def _vosolorn(c: dict, shape: Callable[[str], tuple], name: str) -> StackConfig:
+    """config.json of the Vosolorn design."""
+    layers = []
+    for i, e in enumerate(c["layers"]):
+        m, kind = e["mixer"], e["type"]
+        if kind == "attention":
+            mask, rot, vdim = m.get("mask") or {"size": 0}, m["rot"], int(m["vdim"])
+            mixer = GroupedAttention(heads=int(m["heads"]), kv_heads=int(m["kv_heads"]), dim=int(m["dim"]), vdim=vdim,
+                                     scale=float(m["scale"]), window=int(mask["size"]), slopes=False, out_bias=False, in_bias=False,
+                                     head_norm=True, rot=Rotary(float(rot["base"]), int(rot["dims"]), True),
+                                     v_rot=Rotary(float(rot["base"]), vdim, True), pool=int(mask.get("pool") or 0))
+        elif kind == "mlstm":
+            mixer = MatrixMemory(heads=int(m["heads"]), dim=int(m["dim"]), vdim=int(m["vdim"]), gate_cap=float(m["gate_cap"]))
+        else:
+            raise ValueError(f"{name}: layer {i}: unknown mixer {kind!r}")
+        f = e.get("mlp")
+        if f is None:
+            mlp = None
+        elif f.get("kind") == "dense":
+            mlp = DenseMlp(int(f["ff"]), "gelu_glu")
+        elif f.get("kind") == "moe":
+            mlp = MoeMlp(int(f["router"]["experts"]), int(f["router"]["top"]), int(f["expert"]["ff"]), act="gelu",
+                         shared=int((f.get("shared") or {"ff": 0})["ff"]))
+        else:
+            raise ValueError(f"{name}: layer {i}: unknown feed-forward {f.get('kind')!r}")
+        layers.append(LayerSpec(mixer, mlp, pre_norm=False, layer_scale=True))
+    return StackConfig(name=name, d_model=int(c["width"]), vocab=int(c["vocab"]), layers=tuple(layers),
+                       rms_eps=float(c["norm"]["eps"]), embed_norm=True, tied_head=True, logit_scale=float(c["logit_scale"]))
+
+
+DESIGNS: Dict[str, Callable] = {"Bekopel": _bekopel, "Lerazen": _lerazen, "Merulorn": _merulorn, "Vosolorn": _vosolorn}
 
 
 def safetensors_shapes(path) -> Dict[str, tuple]:
@@ -644,6 +802,7 @@ class StackWeights:
     layers: list = field(default_factory=list)
     pos_embed: Optional[torch.Tensor] = None
     pos_turns: Optional[torch.Tensor] = None
+    embed_norm: Optional[torch.Tensor] = None
 
     @staticmethod
     def from_tensors(cfg: StackConfig, get: Callable[[str], torch.Tensor], device) -> "StackWeights":
@@ -663,7 +822,12 @@ class StackWeights:
             return t if t.shape[0] == n else torch.cat([t, t.new_zeros(n - t.shape[0], *t.shape[1:])])
 
         norm = lambda n: f32(raw(n)) + cfg.norm_offset
-        w = StackWeights(cfg, bf(raw("embed")), bf(rows(raw("head"), cfg.vocab_ld)), norm("final.norm"))
+        embed = bf(raw("embed"))
+        head = rows(embed, cfg.vocab_ld) if cfg.tied_head else bf(rows(raw("head"), cfg.vocab_ld))
+        # the factor of the logits joins the final norm's weight
+        w = StackWeights(cfg, embed, head, norm("final.norm") * cfg.logit_scale)
+        if cfg.embed_norm:
+            w.embed_norm = norm("embed.norm")
         if cfg.sinusoid_pos:
             w.pos_turns = position_turns(cfg.d_model, device)
         if cfg.learned_pos:
@@ -673,7 +837,13 @@ class StackWeights:
             if l.parallel:
                 w.layers.append(StackWeights._parallel(cfg, i, raw, norm, bf, f32, rows))
                 continue
-            t = {n: norm(f"l{i}.{n}") for n in ("norm1", "norm1b", "norm2", "norm2b") if f"l{i}.{n}" in want}
+            t = {}
+            for part in ("1", "2") if l.mlp else ("1",):        # a scale joins the weight of the norm in front of it
+                scale = f32(raw(f"l{i}.ls{part}")) if l.layer_scale else 1.0
+                if l.pre_norm:
+                    t[f"norm{part}"] = norm(f"l{i}.norm{part}")
+                if l.post_norm:
+                    t[f"norm{part}b"] = norm(f"l{i}.norm{part}" + ("b" if l.pre_norm else "")) * scale
             if l.composed:
                 t.update(StackWeights._composed(cfg, i, raw, bf, f32, rows))
             elif isinstance(m, LatentAttention):
@@ -694,7 +864,9 @@ class StackWeights:
                 w2 = g("w2")
                 t["w_decay"] = bf(torch.cat([w2, w2.new_zeros(w2.shape[0], m.rank_ld - m.decay_rank)], dim=1))
                 t["decay_bias"], t["rate_bias"], t["out_norm"] = f32(g("w0")), f32(g("a.b")), f32(g("norm"))
-            if l.mlp and l.mlp.glu:
+            if isinstance(l.mlp, MoeMlp):
+                t.update(StackWeights._experts(cfg, i, raw, bf, f32, rows))
+            elif l.mlp and l.mlp.glu:
                 t["w_up"] = StackWeights.glu_rows(*(rows(bf(raw(f"l{i}.mlp.{n}")), l.mlp.ff_ld) for n in ("gate", "up")))
                 t["w_down"] = torch.zeros(cfg.d_model, l.mlp.ff_ld, dtype=torch.bfloat16, device=device)
                 t["w_down"][:, :l.mlp.ff] = bf(raw(f"l{i}.mlp.down"))
@@ -717,16 +889,19 @@ class StackWeights:
         att, ssm, both = l.one(GroupedAttention), l.one(StateSpace), isinstance(l.mixer, SideBySide)
         left = lambda n: raw(f"l{i}.mix." + ("left." if both else "") + n)
         right = lambda n: raw(f"l{i}.mix." + ("right." if both else "") + n)
+        if l.one(MatrixMemory):
+            return StackWeights._memory(cfg, i, right, bf, f32, rows)
         w_in, t = [], {}
         some = left("o") if att else right("o")
         w_out = torch.zeros(d, cfg.mix_cols(i)[1], dtype=torch.bfloat16, device=some.device)
         if att:
             w_in.append(rows(torch.cat([left(n) for n in ("q", "k", "v")] + ([left("g")] if att.gate else [])), cfg.ssm_col(i)))
             w_out[:, :att.out_dim] = bf(left("o"))
-            t["in_bias"] = f32(torch.cat([left("q.b"), left("k.b"), left("v.b")]))
+            if att.in_bias:
+                t["in_bias"] = f32(torch.cat([left("q.b"), left("k.b"), left("v.b")]))
             if att.out_bias:
                 t["out_bias"] = f32(left("o.b"))
-            if att.qk_norm:
+            if att.qk_norm or att.head_norm:
                 t["q_norm"], t["k_norm"] = f32(left("q.norm")), f32(left("k.norm"))
             if att.slopes:
                 t["slopes"] = head_slopes(att.heads, some.device)
@@ -740,6 +915,33 @@ class StackWeights:
                      decay_rate=right("A_log").double().exp().float().contiguous(), skip=f32(right("D")),
                      ssm_norm=f32(right("norm")) * (l.mixer.right_scale if both else 1.0))
         t["w_in"], t["w_out"] = bf(rows(torch.cat(w_in), cfg.in_rows(i))), w_out
+        return t
+
+    @staticmethod
+    def _memory(cfg: StackConfig, i: int, get, bf, f32, rows) -> dict:
+        """q | k | v | output gate, then the input and forget gates, in one input matrix."""
+        m = cfg.layers[i].mixer
+        w_in = torch.cat([rows(torch.cat([get(n) for n in ("q", "k", "v", "g")]), m.gate_col), get("i"), get("f")])
+        w_out = torch.zeros(cfg.d_model, cfg.mix_cols(i)[1], dtype=torch.bfloat16, device=w_in.device)
+        w_out[:, :m.out_dim] = bf(get("o"))
+        return {"w_in": bf(rows(w_in, cfg.in_rows(i))), "w_out": w_out, "mem_bias": f32(torch.cat([get("i.b"), get("f.b")])),
+                "mem_norm": f32(get("norm"))}
+
+    @staticmethod
+    def _experts(cfg: StackConfig, i: int, raw, bf, f32, rows) -> dict:
+        """Plain experts: the router and the shared expert's rows in one matrix, the others' one after another."""
+        f, d = cfg.layers[i].mlp, cfg.d_model
+        g = lambda n: raw(f"l{i}.mlp.{n}")
+        up = [rows(g("router"), f.router_rows)] + ([rows(g("shared.up"), f.shared_ld)] if f.shared else [])
+        t = {"w_up": bf(torch.cat(up)), "router_bias": f32(g("router.b"))}
+        z = lambda *s: torch.zeros(*s, dtype=torch.bfloat16, device=t["w_up"].device)
+        if f.shared:
+            t["w_down"] = z(d, f.shared_ld)
+            t["w_down"][:, :f.shared] = bf(g("shared.down"))
+        t["w_experts_in"], t["w_experts_out"] = z(f.experts, f.ff_ld, d), z(f.experts, d, f.ff_ld)
+        for e in range(f.experts):
+            t["w_experts_in"][e, :f.ff] = bf(g(f"e{e}.up"))
+            t["w_experts_out"][e, :, :f.ff] = bf(g(f"e{e}.down"))
         return t
 
     @staticmethod
@@ -808,15 +1010,17 @@ class StackWeights:
                 return torch.full(s, -4.0, device=device)
             if n.endswith(".D"):
                 return torch.ones(*s, device=device)
+            if n.endswith(".f.b"):          # memories of a few dozen tokens and more
+                return torch.linspace(3.0, 6.0, s[0], device=device)
             if len(s) == 2:
                 return torch.empty(*s, dtype=torch.bfloat16, device=device).normal_(0.0, 0.02, generator=g)
             leaf = n.rsplit(".", 1)[-1]
-            one = leaf.startswith("norm") and not (cfg.norm_offset and ".mix." not in n)
+            one = leaf.startswith(("norm", "ls")) and not (cfg.norm_offset and ".mix." not in n)
             return (torch.ones if one else torch.zeros)(*s, device=device)
         return StackWeights.from_tensors(cfg, get, device)
 
     def nbytes(self) -> int:
-        ts = [self.embed, self.lm_head] + ([self.pos_embed] if self.pos_embed is not None else []) + [t for l in self.layers for t in l.values()]
+        ts = [self.embed] + ([] if self.lm_head.data_ptr() == self.embed.data_ptr() else [self.lm_head]) + ([self.pos_embed] if self.pos_embed is not None else []) + [t for l in self.layers for t in l.values()]
         return sum(t.numel() * t.element_size() for t in ts)
 
 
@@ -827,21 +1031,36 @@ class StackHandle:
     caches[i]: the latent pages [pages, page, cache_row] or the states [slots, heads, dim, dim] of layer i
     (None where the layer reads another layer's cache); for grouped attention and state-space mixers a dict of what
     there is of cache (keys [pages, kv_heads, page, q_ld]), cache_v (values [pages, kv_heads, page, v_ld]), ssm_state
-    [slots, heads, vdim, state] and conv_state [slots, taps - 1, channels]."""
+    [slots, heads, vdim, state] and conv_state [slots, taps - 1, channels]; for matrix memories mem_state [slots, heads,
+    vdim + 1, dim] and mem_max [slots, heads, blocks].  Pages of pooled blocks follow the others; pool_cols: block size ->
+    first column of their page numbers in the block table."""
 
-    def __init__(self, w: StackWeights, caches: list, n_pos: int, page_size: int):
+    def __init__(self, w: StackWeights, caches: list, n_pos: int, page_size: int, pool_cols: Optional[Dict[int, int]] = None):
         cfg = w.cfg
         self.w, self.caches = w, caches
         dev = w.embed.device
         self._rope: Dict[Rotary, torch.Tensor] = {}
         arr = (L.Layer * cfg.n_layers)()
         counts = 0
+
+        def table(rot: Rotary) -> int:
+            if rot not in self._rope:
+                self._rope[rot] = rope_table(rot, n_pos, dev)
+            return self._rope[rot].data_ptr()
         for i, (spec, t) in enumerate(zip(cfg.layers, w.layers)):
             a, m = arr[i], spec.mixer
             a.n_in = cfg.in_rows(i)
             src = i
-            att, ssm = spec.one(GroupedAttention), spec.one(StateSpace)
+            att, ssm, mem = spec.one(GroupedAttention), spec.one(StateSpace), spec.one(MatrixMemory)
             if att:
+                if att.by_head:
+                    a.by_head, a.rot_dims, a.v_rot_dims = 1, att.rot.dims if att.rot else 0, att.v_rot.dims if att.v_rot else 0
+                    if a.rot_dims:
+                        a.cos_sin, a.rot_pairs = table(att.rot), int(att.rot.pairs)
+                    if a.v_rot_dims:
+                        a.v_cos_sin = table(att.v_rot)
+                if att.pool:
+                    a.pool, a.pool_col = att.pool, pool_cols[att.pool]
                 a.mixer, a.heads, a.dim = L.MIXER_GROUPED_ATTN, att.heads, att.dim
                 a.kv_heads, a.vdim, a.q_ld, a.v_ld = att.kv_heads, att.vdim, att.q_ld, att.v_ld
                 a.window, a.scale, a.owns_cache = att.window, att.scale, 1
@@ -861,7 +1080,10 @@ class StackHandle:
                 a.ssm_heads, a.ssm_vdim, a.ssm_n, a.ssm_groups = ssm.heads, ssm.vdim, ssm.state, ssm.groups
                 a.ssm_norm_parts, a.ssm_taps, a.ssm_col, a.ssm_mix_col = ssm.norm_groups, ssm.conv, cfg.ssm_col(i), cfg.ssm_mix_col(i)
                 a.mix_ld = cfg.mix_cols(i)[1]
-            if att or ssm:
+            if mem:
+                a.mixer, a.heads, a.dim, a.vdim = L.MIXER_MATRIX_MEMORY, mem.heads, mem.dim, mem.vdim
+                a.gate_col, a.gate_cap, a.mix_ld = mem.gate_col, mem.gate_cap, cfg.mix_cols(i)[1]
+            if att or ssm or mem:
                 for n, x in caches[i].items():
                     setattr(a, n, x.data_ptr() if x.numel() else None)
             elif isinstance(m, LatentAttention):
@@ -871,9 +1093,7 @@ class StackHandle:
                 if "w_expand" in t:
                     a.q_ld, a.v_ld = m.q_ld, m.v_ld
                 src = i if m.kv_from is None else m.kv_from
-                if m.rot not in self._rope:
-                    self._rope[m.rot] = rope_table(m.rot, n_pos, dev)
-                a.cos_sin = self._rope[m.rot].data_ptr()
+                a.cos_sin = table(m.rot)
             else:
                 a.mixer, a.heads, a.dim, a.decay_rank = L.MIXER_GENERAL_DELTA, m.heads, m.dim, m.rank_ld
             if isinstance(spec.mlp, MoeMlp):
@@ -881,15 +1101,18 @@ class StackHandle:
                 a.experts, a.top, a.expert_ld, a.glu_limit, a.glu_alpha = f.experts, f.top, f.ff_ld, f.limit, f.alpha
                 a.moe_counts_at = counts
                 counts += f.experts
+                if not f.glu:
+                    a.ff_kind, a.ff, a.n_router = L.FF_EXPERTS, f.shared_ld, f.router_rows
             else:
                 f = spec.mlp
                 a.ff = f.ff_ld if f else 0
                 if f and f.glu:
-                    a.ff_kind, a.glu_limit, a.glu_alpha = L.FF_CLAMPED_GLU, f.limit, f.alpha
+                    a.ff_kind = L.FF_GELU_GLU if f.act == "gelu_glu" else L.FF_CLAMPED_GLU
+                    a.glu_limit, a.glu_alpha = f.limit, f.alpha
             for n, x in t.items():
                 if n != "vmix":
                     setattr(a, n, x.data_ptr())
-            if not (att or ssm):
+            if not (att or ssm or mem):
                 a.cache = caches[src].data_ptr()
         self._layers = arr
         s = L.Stack()
@@ -899,6 +1122,8 @@ class StackHandle:
         if w.pos_embed is not None:
             s.pos_embed, s.n_pos = w.pos_embed.data_ptr(), w.pos_embed.shape[0]
         s.embed_scale = cfg.embed_scale
+        if w.embed_norm is not None:
+            s.embed_norm = w.embed_norm.data_ptr()
         if w.pos_turns is not None:
             s.pos_turns = w.pos_turns.data_ptr()
         s.layers = C.cast(arr, C.POINTER(L.Layer))

@@ -22,7 +22,7 @@
 extern "C" {
 #endif
 
-#define BCG_ABI_VERSION 4
+#define BCG_ABI_VERSION 5
 
 /* status codes */
 #define BCG_STATUS_OK 0
@@ -361,7 +361,8 @@ int bcg_model_decode(const bcg_model* m, const bcg_workspace* ws, const int* ids
  * only meets uniform dense decoders).  Every layer is a mixer and, optionally, a feed-forward, each
  * with a norm before and (norm1b / norm2b not NULL) a norm after it:  x += norm1b(mixer(norm1(x))),
  * x += norm2b(ff(norm2(x))), or, `parallel`, both behind one norm:  h = norm1(x),  x += mixer(h) + ff(h).
- * A mixer may be two side by side, grouped attention and a state-space mixer, that read the same h.
+ * norm1 / norm2 NULL: the sublayers read x itself.  A mixer may be two side by side, grouped attention and a state-space
+ * mixer, that read the same h.
  * `act_dtype` selects the activations that feed matrix products, the latent cache and the attention
  * operands: BCG_DT_BF16 (tensor-core kernels, fp32 accumulation) or BCG_DT_F32 (true fp32
  * throughout, CUDA-core kernels).  Weights are bf16 in both; the residual, norms, scores, gates and
@@ -372,8 +373,12 @@ int bcg_model_decode(const bcg_model* m, const bcg_workspace* ws, const int* ids
 #define BCG_MIXER_GENERAL_DELTA 2
 #define BCG_MIXER_GROUPED_ATTN 3
 #define BCG_MIXER_STATE_SPACE 4   /* alone; beside grouped attention: ssm_heads > 0 */
+#define BCG_MIXER_MATRIX_MEMORY 5
 #define BCG_FF_POLY_NORM 0   /* bcg_layer.ff_kind of layers that are not parallel */
 #define BCG_FF_CLAMPED_GLU 1 /* w_up rows interleaved [16 gate | 16 up], glu_limit, glu_alpha */
+#define BCG_FF_GELU_GLU 2    /* the same rows; gelu(gate) * up, gelu in its tanh form */
+#define BCG_FF_EXPERTS 3     /* experts without gates, gelu in its erf form; w_up: n_router router rows, then the ff rows of a
+                                shared expert (ff = 0: none), whose output matrix is w_down */
 #define BCG_VALUES_FIRST 1   /* bcg_layer.v_role: the layer's values are what later layers mix in */
 #define BCG_VALUES_MIX 2     /* values are (1 - v_mix) of its own and v_mix of those */
 
@@ -454,6 +459,24 @@ typedef struct bcg_layer {
   const float* ssm_norm;   /* [heads * vdim] */
   float* ssm_state;        /* fp32 [slots][heads][vdim][n] */
   float* conv_state;       /* fp32 [slots][taps - 1][channels]: the last inputs of the convolution, oldest first */
+  /* grouped attention whose heads are normed (q_norm, k_norm: [dim], or NULL) and rotated one by one */
+  int by_head;
+  int rot_pairs;           /* entries 2i and 2i + 1 turn together, else i and rot_dims / 2 + i */
+  int v_rot_dims;          /* entries of the values that turn, in pairs 2i, 2i + 1; outputs are turned back; 0 = none */
+  const float* v_cos_sin;  /* [max_pos][v_rot_dims] as cos_sin */
+  int pool;                /* tokens of a pooled block; 0 = none.  Block b's key and value are the means of the cached ones of
+                              tokens b * pool .. + pool - 1; query i sees it if b * pool + pool - 1 <= i - window */
+  int pool_col;            /* column of the block table with the page of pooled blocks 0 .. page_size - 1, and so on */
+  /* matrix memory: rows q | k (heads * dim each) | v | output gate (heads * vdim each) of w_in, from gate_col on input and
+     forget gates (heads each); log gates cap * tanh((z + bias) / cap), the forget gate's logsigmoid of that */
+  float gate_cap;
+  const float* mem_bias;   /* [2 * heads] */
+  const float* mem_norm;   /* [heads * vdim] */
+  float* mem_state;        /* fp32 [slots][heads][vdim + 1][dim], last row = normalizer */
+  float* mem_max;          /* fp32 [slots][heads][(vdim + 63) / 64]: running maximum of the log gates, one copy per 64 rows */
+  /* BCG_FF_EXPERTS */
+  int n_router;
+  const float* router_bias; /* [experts] */
 } bcg_layer;
 
 typedef struct bcg_stack {
@@ -468,6 +491,7 @@ typedef struct bcg_stack {
   int n_pos;
   float embed_scale;        /* factor of the embedding */
   const double* pos_turns;  /* [(d + 1) / 2] turns per position: sin at entry 2i, cos at 2i + 1 are added; or NULL */
+  const float* embed_norm;  /* [d] weight of a norm of the embedding, or NULL */
 } bcg_stack;
 
 typedef struct bcg_stack_ws {
@@ -510,6 +534,7 @@ typedef struct bcg_stack_ws {
   void* ssm_x;      /* act [T_max, ssm_x_ld(layer)]: convolved x | B | C, heads and groups padded to multiples of 8 */
   float* ssm_step;  /* fp32 [T_max, ssm_heads] */
   void* ssm_y;      /* act [T_max, ssm_heads * ssm_vdim]: outputs in front of gate and norm */
+  float* mem_den;   /* fp32 [T_max, heads]: denominators of a matrix memory's outputs (ssm_x and ssm_y are its other buffers) */
 } bcg_stack_ws;
 
 /* A step: T new tokens of n_seqs sequences, portions of prompts beside single decoded tokens.  All
@@ -521,7 +546,7 @@ typedef struct bcg_step_batch {
   const int* slot_map;     /* [T] cache row of each token (< 0: writes nothing, keeps the state) */
   const int* row_seq;      /* [T] sequence of each token, NULL = token t belongs to sequence t */
   const int* seq_start;    /* [n_seqs + 1] first token of each sequence, NULL = one token each */
-  const int* block_table;  /* [n_seqs, max_blocks] */
+  const int* block_table;  /* [n_seqs, max_blocks]: pages of the tokens, then, from bcg_layer.pool_col on, of pooled blocks */
   int max_blocks;
   const int* state_slots;  /* [n_seqs] */
   int max_context;         /* upper bound on positions + 1 of the single tokens (sizes the grid) */
@@ -551,15 +576,16 @@ int bcg_stack_head(const bcg_stack* m, const bcg_stack_ws* ws, const int* rows, 
 int bcg_gemm_any(const void* X, int x_dtype, const void* W, float* out, int M, int N, int K, long long ldx,
                  long long ldw, long long ldo, void* stream);
 /* No counterpart in the reference: residual += w_post ? rmsnorm(delta) * w_post : delta, then
- * xn = rmsnorm(residual) * w_next (NULL: skipped). */
+ * xn = rmsnorm(residual) * w_next (w_next NULL: xn = residual; xn NULL: skipped). */
 int bcg_sandwich_norm(float* residual, const float* delta, int n_partials, long long partial_stride,
                       const float* w_post, const float* w_next, void* xn, int act_dtype, int T, int d, float eps,
                       void* stream);
-/* No counterpart in the reference: the same with further summands and no norm of delta: residual += delta + bias (may be
- * NULL) + sum over k < per_row of rows[index[t * per_row + k]] (fp32 slabs too); xn = rmsnorm(residual) * w_next. */
+/* No counterpart in the reference: the same with further summands: delta (may be NULL when per_row > 0) + bias (may be NULL) +
+ * sum over k < per_row of rows[index[t * per_row + k]] (fp32 slabs too) times weight[t * per_row + k] (NULL: 1). */
 int bcg_residual_norm(float* residual, const float* delta, int n_partials, long long partial_stride, const float* bias,
-                      const float* rows, const int* index, int per_row, int row_partials, long long row_stride,
-                      const float* w_next, void* xn, int act_dtype, int T, int d, float eps, void* stream);
+                      const float* rows, const int* index, const float* weight, int per_row, int row_partials,
+                      long long row_stride, const float* w_post, const float* w_next, void* xn, int act_dtype, int T, int d,
+                      float eps, void* stream);
 /* No counterpart in the reference: a N(z) + b N(z^2) + c N(z^3) + e with N = division by the row's RMS. */
 int bcg_poly_norm(const float* z, int n_partials, long long partial_stride, const float* coef, void* out,
                   int act_dtype, int T, int ff, float eps, void* stream);
@@ -605,6 +631,26 @@ int bcg_clamped_glu(const float* z, int n_partials, long long partial_stride, vo
 /* No counterpart in the reference: bcg_gemm_bf16_tn with that unit as its epilogue; out bf16 [M, N / 2], N % 32 == 0. */
 int bcg_gemm_bf16_glu(const void* X, const void* W, void* out, int M, int N, int K, float limit, float alpha, int flags,
                       void* stream);
+
+/* No counterpart in the reference: gelu of split-K slabs; gated: z [T, 2 * ff], columns interleaved [16 gate | 16 up], out =
+ * gelu(gate) * up with the tanh form; else z [T, ff], the erf form.  ff % 16 == 0. */
+int bcg_gelu_unit(const float* z, int n_partials, long long partial_stride, void* out, int act_dtype, int T, int ff, int gated,
+                  void* stream);
+/* No counterpart in the reference: bcg_gemm_bf16_tn with that unit as its epilogue: gated, out bf16 [M, N / 2], N % 32 == 0; else
+ * out bf16 [M, N], N % 16 == 0, M > 128. */
+int bcg_gemm_bf16_gelu(const void* X, const void* W, void* out, int M, int N, int K, int gated, int flags, void* stream);
+/* No counterpart in the reference: bcg_gemm_grouped with gelu (erf form) as its epilogue, out bf16 [rows, N], max_rows > 128. */
+int bcg_gemm_grouped_gelu(const void* X, const void* W, void* out, int rows, int N, int K, const int* counts, int n_groups, int max_rows,
+                          int flags, void* stream);
+/* No counterpart in the reference: routing of a BCG_FF_EXPERTS layer whose logits are the first columns of ws->proj (row pitch ld;
+ * ws->moe_counts must be zero) and, with_act, gelu of the columns behind n_router into ws->act. */
+int bcg_expert_in(const bcg_stack* m, const bcg_stack_ws* ws, int layer, int T, int n_partials, long long partial_stride, long long ld,
+                  int with_act, void* stream);
+/* No counterpart in the reference: a matrix memory behind its input projection (ws->proj, row pitch ld): recurrence, norm and output
+ * gate; states advanced, ws->mix filled.  mode 0: what bcg_stack_step picks (tensor-core chunks or, one token each, the decode
+ * kernel); 1: token by token on CUDA cores. */
+int bcg_matrix_memory(const bcg_stack* m, const bcg_stack_ws* ws, const bcg_step_batch* b, int layer, int n_partials,
+                      long long partial_stride, long long ld, int mode, void* stream);
 
 #ifdef __cplusplus
 }

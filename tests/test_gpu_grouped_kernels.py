@@ -348,14 +348,24 @@ def test_residual_norm_adds_bias_and_expert_rows(dtype, T, d, parts, per_row, ro
     x, y, bias, wn = (torch.randn(*s, generator=g) for s in ((T, d), (parts, T, d), (d,), (d,)))
     n = max(T * per_row, 1)
     rows, index = torch.randn(row_parts, n, d, generator=g), torch.randperm(n, generator=g)[:T * per_row].view(T, per_row)
-    R_, Y, B, W, E, I = (v.cuda() for v in (x, y, bias, wn, rows, index.int()))
-    xn = torch.zeros(T, d, dtype=td, device="cuda")
-    L.check(L.load().bcg_residual_norm(R_.data_ptr(), Y.data_ptr(), parts, T * d, B.data_ptr(), E.data_ptr() if per_row else None,
-                                       I.data_ptr() if per_row else None, per_row, row_parts, n * d, W.data_ptr(), xn.data_ptr(),
-                                       code, T, d, 1e-3, L.stream_ptr()))
-    want = x.double() + y.double().sum(0) + bias.double() + rows.double().sum(0)[index].sum(1)
-    close(R_, want, 2e-6)
-    close(xn, R.rms_norm(want, 1e-3, wn.double()), tol)
+    weight, wp = torch.rand(T, max(per_row, 1), generator=g)[:, :per_row], torch.randn(d, generator=g)
+    Y, B, W, E, I, F, P = (v.cuda() for v in (y, bias, wn, rows, index.int(), weight.contiguous(), wp))
+    ptr = lambda v, there=True: v.data_ptr() if there else None
+    # as it stands; weighted rows behind a norm of their own, the stream itself passed on; weighted rows alone
+    for weighted, with_delta, post, nxt in ((False, True, False, True), (True, True, True, False), (True, False, True, True)):
+        if not with_delta and not per_row:
+            continue
+        R_, xn = x.cuda(), torch.zeros(T, d, dtype=td, device="cuda")
+        L.check(L.load().bcg_residual_norm(R_.data_ptr(), ptr(Y, with_delta), parts, T * d, ptr(B, with_delta), ptr(E, per_row),
+                                           ptr(I, per_row), ptr(F, per_row and weighted), per_row, row_parts, n * d, ptr(P, post),
+                                           ptr(W, nxt), xn.data_ptr(), code, T, d, 1e-3, L.stream_ptr()))
+        factor = weight.double()[..., None] if weighted else 1.0
+        add = (factor * rows.double().sum(0)[index]).sum(1)
+        if with_delta:
+            add = add + y.double().sum(0) + bias.double()
+        want = x.double() + (R.rms_norm(add, 1e-3, wp.double()) if post else add)
+        close(R_, want, 3e-6)
+        close(xn, R.rms_norm(want, 1e-3, wn.double()) if nxt else want, tol)
 
 
 @pytest.mark.parametrize("M,N,K", [(129, 48, 64), (300, 96, 200), (700, 256, 128), (600, 2080, 192), (513, 2048, 64)])
