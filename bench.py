@@ -364,7 +364,7 @@ def main():
     ap.add_argument("--pdl", type=int, default=int(os.environ.get("BCG_B200_PDL", "1")),
                     help="programmatic dependent launch for the decode step (1 = on)")
     ap.add_argument("--design", default=None,
-                    help="instead of the default workload: throughput of a layer-stack design (bekopel, lerazen, merulorn) beside a "
+                    help="instead of the default workload: throughput of a layer-stack design (bekopel, lerazen, merulorn, vosolorn) beside a "
                          "dense model of equal size, one JSON line")
     ap.add_argument("--design-sizes", default=None, help="comma-separated subset of the sizes of --design")
     a = ap.parse_args()

@@ -12,6 +12,11 @@ __device__ __forceinline__ float softplus_f32(float x) { return fmaxf(x, 0.f) + 
 // rounded once near 1: a state that decays slowly would drift with the error of exp
 __device__ __forceinline__ float decay_f32(float x) { return 1.0f + expm1f(x); }
 
+__device__ __forceinline__ void bulk_store_1d(void* gdst, const void* smem_src, uint32_t bytes) {
+  asm volatile("cp.async.bulk.global.shared::cta.bulk_group [%0], [%1], %2;" ::"l"(gdst), "r"(smem_u32(smem_src)), "r"(bytes) : "memory");
+  asm volatile("cp.async.bulk.commit_group;" ::: "memory");
+}
+
 constexpr int kSsThreads = 256, kSsRows = 64;     // threads and state rows of a CTA
 
 // Rows of a head's state over groups of lanes: a group holds a row's entries, four (or twice four) per lane, and every

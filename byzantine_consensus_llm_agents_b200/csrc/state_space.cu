@@ -5,7 +5,7 @@
 //
 //   ssm_conv    projection slabs -> convolved x | B | C (activations, heads and groups padded to multiples of 8 columns)
 //               and steps; the inputs ahead of a portion come from the convolution's state
-//   ssm_chunk   portions (bf16): chunks of 64 tokens on tensor cores.  Inside a chunk the recurrence is a product,
+//   chunks      portions (bf16): chunks of 64 tokens on tensor cores (state_chunk.cuh).  Inside a chunk the recurrence is a product,
 //                   y_i = exp(c_i) S^T C_i + sum_{j <= i} exp(c_i - c_j) step_j (B_j . C_i) x_j,   c = running sum of -rate * step,
 //               and the state moves once per chunk.  Everything is held transposed (rows = entries of a head's output), so
 //               that the state stays in fp32 accumulators and becomes an operand without leaving the registers.  Weights (decays,
@@ -19,9 +19,7 @@
 //   ssm_norm    gate and norm of the outputs
 // The convolution's state moves on where nobody reads it any more: behind the chunks or the scan, and in ssm_norm for
 // single tokens (whose B and C every head of a group convolves for itself).
-#include <type_traits>
-
-#include "state_rows.cuh"
+#include "state_chunk.cuh"
 #include "kernels.h"
 
 namespace bcg {
@@ -50,6 +48,12 @@ struct SsmArgs {
   }
   __device__ __forceinline__ int b_col(int g) const { return heads * x_pad() + g * n_pad(); }
   __device__ __forceinline__ int c_col(int g) const { return heads * x_pad() + (groups + g) * n_pad(); }
+  // what state_chunk.cuh asks for: columns of a head, entries of a state row, a head's state
+  __device__ __forceinline__ int in_col(int h) const { return b_col(h / (heads / groups)); }
+  __device__ __forceinline__ int out_col(int h) const { return c_col(h / (heads / groups)); }
+  __device__ __forceinline__ int row_col(int h) const { return h * x_pad(); }
+  __device__ __forceinline__ int entries() const { return n; }
+  __device__ __forceinline__ float* state_of(int slot, int h) const { return state + (static_cast<long long>(slot) * heads + h) * vdim * n; }
   __device__ __forceinline__ const float* row(long long t) const { return proj + t * ld + col; }
   __device__ __forceinline__ int seq_of(int t) const { return row_seq ? row_seq[t] : t; }
   __device__ __forceinline__ int first_of(int s) const { return seq_start ? seq_start[s] : s; }
@@ -301,11 +305,6 @@ ssm_token_kernel(const SsmArgs a) {
     static_cast<T*>(a.y)[static_cast<long long>(t) * a.inner() + h * a.vdim + p0 + p] = from_f32<T>(fmaf(a.skip[h], xbc[p], y));
 }
 
-__device__ __forceinline__ void bulk_store_1d(void* gdst, const void* smem_src, uint32_t bytes) {
-  asm volatile("cp.async.bulk.global.shared::cta.bulk_group [%0], [%1], %2;" ::"l"(gdst), "r"(smem_u32(smem_src)), "r"(bytes) : "memory");
-  asm volatile("cp.async.bulk.commit_group;" ::: "memory");
-}
-
 // State rows of 16 bytes' multiple, up to 128 entries.  A unit is 64 rows of a token's head (fewer at a head's end), a CTA
 // has consecutive ones: B and C are made once per group.  Warps 0-7 compute, warp 8 moves states: a stage is filled, worked
 // on in place, stored, and filled again once it has been read.
@@ -545,143 +544,22 @@ ssm_scan_kernel(const SsmArgs a) {
 }
 
 // ------------------------------------------------------------------------------------------- chunks
-constexpr int kChTok = 64, kChWarps = 4, kChThreads = kChWarps * 32;
-
-// Tiles in shared memory are rows of 16-byte pieces, piece p of row r at place p ^ (r & 7).  B and x are there for two chunks.
-template <int NP>
-struct ChCfg {
-  static constexpr int kBC = kChTok * NP * 2, kX = kChTok * kSsRows * 2, kM = kChTok * kChTok * 2;     // bytes
-  static constexpr int kOffC = 2 * kBC, kOffX = kOffC + kBC, kOffM = kOffX + 2 * kX, kOffS = kOffM + kM;
-  static constexpr int kSmem = kOffS + 2 * 4 * kChTok * 4 + 128;
-  static constexpr int kCtasPerSm = NP <= 128 ? 3 : 2;
-};
-
-// matrix loads from shared-memory addresses: offsets that are constants cost no instruction
-__device__ __forceinline__ void ldsm_at(uint32_t (&r)[4], uint32_t p) {
-  asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0, %1, %2, %3}, [%4];"
-               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3])
-               : "r"(p));
-}
-__device__ __forceinline__ void ldsm_trans_at(uint32_t (&r)[4], uint32_t p) {
-  asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0, %1, %2, %3}, [%4];"
-               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3])
-               : "r"(p));
-}
-// hi + lo = v to about 2^-17
-__device__ __forceinline__ void split_bf16(float a, float b, uint32_t& hi, uint32_t& lo) {
-  hi = pack_bf16(a, b);
-  lo = pack_bf16(a - bf16lo(hi), b - bf16hi(hi));
-}
-__device__ __forceinline__ void scale2(float& a, float& b, float fa, float fb) {
-  unpack_f32x2(mul_f32x2(pack_f32x2(__float_as_uint(a), __float_as_uint(b)), pack_f32x2(__float_as_uint(fa), __float_as_uint(fb))), a, b);
-}
-__device__ __forceinline__ uint32_t transpose_8x8(uint32_t v) {
-  uint32_t r;
-  asm volatile("movmatrix.sync.aligned.m8n8.trans.b16 %0, %1;" : "=r"(r) : "r"(v));
-  return r;
-}
-
-// M[i][j] = exp(c_i - c_j) step_j (C_i . B_j) for j <= i, tokens i = 16 RT .. 16 RT + 15.  sB, sC, sM: addresses.
-template <int NP, int RT>
-__device__ __forceinline__ void chunk_matrix(uint32_t sB, uint32_t sC, const float* sum2, const float* steps, uint32_t sM) {
-  const int lane = threadIdx.x & 31, q2 = (lane & 3) * 2;
-  float acc[2 * RT + 2][4] = {};
-  const uint32_t pc = sC + (RT * 16 + (lane & 15)) * NP * 2, xc = ((lane >> 4) ^ (lane & 7)) << 4;
-  const uint32_t pb = sB + ((lane & 7) + ((lane >> 4) << 3)) * NP * 2, xb = (((lane >> 3) & 1) ^ (lane & 7)) << 4;
-#pragma unroll
-  for (int k = 0; k < NP / 16; ++k) {
-    uint32_t ca[4];
-    ldsm_at(ca, pc + (xc ^ (k << 5)));
-    const uint32_t at = pb + (xb ^ (k << 5));
-#pragma unroll
-    for (int jp = 0; jp <= RT; ++jp) {
-      uint32_t bb[4];
-      ldsm_at(bb, at + jp * 16 * NP * 2);
-      mma_bf16_16816(acc[2 * jp], ca, bb[0], bb[1]);
-      mma_bf16_16816(acc[2 * jp + 1], ca, bb[2], bb[3]);
-    }
+// Scalars of a chunk: running sums of -rate * step in log2 units | steps | exp(sum) | step * exp(total - sum).
+struct SsdRule {
+  using Args = SsmArgs;
+  static constexpr bool kNormalized = false;
+  static constexpr int kScalars = 4 * kChTok;
+  const SsmArgs& a;
+  const int h, t0, t1;
+  const float rate;
+  float s0, s1;               // steps of tokens 2 lane, 2 lane + 1 of the next chunk
+  __device__ __forceinline__ SsdRule(const SsmArgs& a_, int h_, int t0_, int t1_, int, bool) : a(a_), h(h_), t0(t0_), t1(t1_), rate(a_.rate[h_]), s0(0.f), s1(0.f) {}
+  __device__ __forceinline__ float step_at(int t) const { return t < t1 ? a.step[static_cast<long long>(t) * a.heads + h] : 0.f; }
+  __device__ __forceinline__ void request(int chunk, int lane) {
+    s0 = step_at(t0 + chunk * kChTok + 2 * lane);
+    s1 = step_at(t0 + chunk * kChTok + 2 * lane + 1);
   }
-  const int i0 = RT * 16 + (lane >> 2);
-  const float ci[2] = {sum2[i0], sum2[i0 + 8]};
-#pragma unroll
-  for (int jt = 0; jt < 2 * RT + 2; ++jt) {
-    const int j = jt * 8 + q2;
-    const float2 cj = *reinterpret_cast<const float2*>(sum2 + j), sj = *reinterpret_cast<const float2*>(steps + j);
-#pragma unroll
-    for (int e = 0; e < 2; ++e) {
-      const int i = i0 + e * 8;
-      float m0 = acc[jt][2 * e] * (ex2_approx(ci[e] - cj.x) * sj.x);
-      float m1 = acc[jt][2 * e + 1] * (ex2_approx(ci[e] - cj.y) * sj.y);
-      if (jt >= 2 * RT) {                       // the diagonal block
-        if (j > i) m0 = 0.f;
-        if (j + 1 > i) m1 = 0.f;
-      }
-      asm volatile("st.shared.b32 [%0], %1;" ::"r"(sM + i * kChTok * 2 + ((jt ^ (lane >> 2)) << 4) + q2 * 2), "r"(pack_bf16(m0, m1))
-                   : "memory");
-    }
-  }
-}
-
-// grid (heads, blocks of 64 head entries, sequences); warp w has entries 16 w .. 16 w + 15 of the block.
-template <int NP>
-__global__ void __launch_bounds__(kChThreads, ChCfg<NP>::kCtasPerSm)
-ssm_chunk_kernel(const SsmArgs a) {
-  using C = ChCfg<NP>;
-  extern __shared__ __align__(128) uint8_t ch_raw[];
-  const uint32_t base = (smem_u32(ch_raw) + 127u) & ~127u;
-  float* scalars = reinterpret_cast<float*>(ch_raw + (base - smem_u32(ch_raw)) + C::kOffS);     // [2][4][64]: log2 decay sums, steps, e, w
-  const uint32_t sC = base + C::kOffC, sM = base + C::kOffM;
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const int h = blockIdx.x, p0 = blockIdx.y * kSsRows, sq = blockIdx.z;
-  const int rows = min(kSsRows, a.vdim - p0), N = a.n, g = h / (a.heads / a.groups), inner = a.inner();
-  pdl_launch_dependents();
-  pdl_wait();
-  const int t0 = a.first_of(sq), t1 = a.end_of(sq);
-  if (t1 <= t0 || a.slot_map[t0] < 0) return;
-  const float rate = a.rate[h], skip = a.skip[h];
-  const __nv_bfloat16* xbc = static_cast<const __nv_bfloat16*>(a.x);
-  const int x_ld = a.x_ld(), b_col = a.b_col(g), c_col = a.c_col(g), x_col = h * a.x_pad() + p0;
-
-  // 64 tokens from `first` on, up to 8 `units` columns from `col` on, `valid` of them; the rest and tokens past the end are
-  // zero
-  auto copy_rows = [&](auto units, uint32_t dst, int col, int valid, int first) {
-    constexpr int kUnits = decltype(units)::value, kPass = kChThreads / kUnits;
-    const int u = threadIdx.x % kUnits, r = threadIdx.x / kUnits, wide = max(0, min(16, (valid - u * 8) * 2));
-    const __nv_bfloat16* src = xbc + static_cast<long long>(first + r) * x_ld + col + u * 8;
-#pragma unroll
-    for (int i = 0; i < kChTok / kPass; ++i) {
-      const int row = r + i * kPass, bytes = first + row < t1 ? wide : 0;
-      asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst + row * kUnits * 16 + ((u ^ (row & 7)) << 4)),
-                   "l"(bytes ? src : xbc), "r"(bytes)
-                   : "memory");
-      src += static_cast<long long>(kPass) * x_ld;
-    }
-  };
-  using BCUnits = std::integral_constant<int, NP / 8>;
-  using XUnits = std::integral_constant<int, kSsRows / 8>;
-  auto step_at = [&](int t) { return t < t1 ? a.step[static_cast<long long>(t) * a.heads + h] : 0.f; };
-
-  const int n_chunks = (t1 - t0 + kChTok - 1) / kChTok;
-  const int pr = warp * 16 + (lane >> 2);       // this lane's rows of the state: pr, pr + 8; entries nt * 8 + 2 (lane & 3) ..
-  const int q2 = (lane & 3) * 2;
-  float* st = a.state + ((static_cast<long long>(a.state_slots[sq]) * a.heads + h) * a.vdim + p0) * N;
-  copy_rows(BCUnits{}, base, b_col, N, t0);
-  copy_rows(BCUnits{}, sC, c_col, N, t0);
-  copy_rows(XUnits{}, base + C::kOffX, x_col, rows, t0);
-  cp_async_commit();
-  float S[NP / 8][4];
-  const bool fresh = a.positions[t0] == 0;
-#pragma unroll
-  for (int nt = 0; nt < NP / 8; ++nt)
-#pragma unroll
-    for (int i = 0; i < 4; ++i) {
-      const int p = pr + (i >> 1) * 8, n = nt * 8 + q2 + (i & 1);
-      S[nt][i] = !fresh && p < rows && n < N ? st[static_cast<long long>(p) * N + n] : 0.f;
-    }
-  float s0 = 0.f, s1 = 0.f;                     // warp 0: steps of tokens 2 lane, 2 lane + 1 of the next chunk
-  // warp 0: the scalars of chunk c from s0 and s1, then the steps of the chunk behind it
-  auto scalars_of = [&](int c) {
-    float* sum2 = scalars + (c & 1) * 4 * kChTok;
+  __device__ __forceinline__ void scalars(float* sum2, int, int lane) {
     float *steps = sum2 + kChTok, *e_s = steps + kChTok, *w_s = e_s + kChTok;
     const float a0 = -rate * s0, a1 = -rate * s1;
     float run = a0 + a1;
@@ -696,150 +574,20 @@ ssm_chunk_kernel(const SsmArgs a) {
     *reinterpret_cast<float2*>(steps + 2 * lane) = make_float2(s0, s1);
     *reinterpret_cast<float2*>(e_s + 2 * lane) = make_float2(expf(c0), expf(c1));
     *reinterpret_cast<float2*>(w_s + 2 * lane) = make_float2(s0 * expf(total - c0), s1 * expf(total - c1));
-    s0 = step_at(t0 + (c + 1) * kChTok + 2 * lane);
-    s1 = step_at(t0 + (c + 1) * kChTok + 2 * lane + 1);
-  };
-  if (warp == 0) {
-    s0 = step_at(t0 + 2 * lane);
-    s1 = step_at(t0 + 2 * lane + 1);
-    scalars_of(0);
   }
-
-  for (int c = 0; c < n_chunks; ++c) {
-    const int first = t0 + c * kChTok, nt_tok = min(kChTok, t1 - first);
-    const float* sum2 = scalars + (c & 1) * 4 * kChTok;
-    const float *steps = sum2 + kChTok, *e_s = steps + kChTok, *w_s = e_s + kChTok;
-    cp_async_wait<0>();
-    __syncthreads();                            // the chunk is there, everybody is done with the previous one
-    const uint32_t sB = base + (c & 1) * C::kBC, sX = base + C::kOffX + (c & 1) * C::kX;
-    if (c + 1 < n_chunks) {
-      copy_rows(BCUnits{}, base + ((c + 1) & 1) * C::kBC, b_col, N, first + kChTok);
-      copy_rows(XUnits{}, base + C::kOffX + ((c + 1) & 1) * C::kX, x_col, rows, first + kChTok);
-    }
-
-    if (warp * 16 < nt_tok) {
-      if (warp == 0) chunk_matrix<NP, 0>(sB, sC, sum2, steps, sM);
-      else if (warp == 1) chunk_matrix<NP, 1>(sB, sC, sum2, steps, sM);
-      else if (warp == 2) chunk_matrix<NP, 2>(sB, sC, sum2, steps, sM);
-      else chunk_matrix<NP, 3>(sB, sC, sum2, steps, sM);
-    }
-    if (warp == 0) scalars_of(c + 1);           // the warp with the smallest share of M
-
-    // ---- Y^T = S^T C^T, columns (tokens) scaled by exp(c_i)
-    float Y[kChTok / 8][4] = {};
-    const uint32_t r8 = (lane & 7) + ((lane >> 4) << 3), x8 = (((lane >> 3) & 1) ^ (lane & 7)) << 4;
-    const uint32_t pc = sC + r8 * NP * 2;
-#pragma unroll
-    for (int k = 0; k < NP / 16; ++k) {
-      const uint32_t sa[4] = {pack_bf16(S[2 * k][0], S[2 * k][1]), pack_bf16(S[2 * k][2], S[2 * k][3]),
-                              pack_bf16(S[2 * k + 1][0], S[2 * k + 1][1]), pack_bf16(S[2 * k + 1][2], S[2 * k + 1][3])};
-#pragma unroll
-      for (int ip = 0; ip < kChTok / 16; ++ip) {
-        uint32_t cb[4];
-        ldsm_at(cb, pc + (x8 ^ (k << 5)) + ip * 16 * NP * 2);
-        mma_bf16_16816(Y[2 * ip], sa, cb[0], cb[1]);
-        mma_bf16_16816(Y[2 * ip + 1], sa, cb[2], cb[3]);
-      }
-    }
-#pragma unroll
-    for (int it = 0; it < kChTok / 8; ++it) {
-      const float2 e = *reinterpret_cast<const float2*>(e_s + it * 8 + q2);
-      scale2(Y[it][0], Y[it][1], e.x, e.y);
-      scale2(Y[it][2], Y[it][3], e.x, e.y);
-    }
-    const float keep = e_s[kChTok - 1];         // past the end steps are zero: the whole chunk's decay
-#pragma unroll
-    for (int nt = 0; nt < NP / 8; ++nt) {
-      scale2(S[nt][0], S[nt][1], keep, keep);
-      scale2(S[nt][2], S[nt][3], keep, keep);
-    }
-    __syncthreads();                            // M is complete, C has been read
-    if (c + 1 < n_chunks) copy_rows(BCUnits{}, sC, c_col, N, first + kChTok);
-    cp_async_commit();
-
-    // ---- Y^T += x^T M^T + skip x^T;   S^T += (w x)^T B
-    const uint32_t px = sX + r8 * kSsRows * 2 + (x8 ^ (warp << 5));
-    const uint32_t pb = sB + (lane & 15) * NP * 2, xb = ((lane >> 4) ^ (lane & 7)) << 4;
-    const uint32_t pm = sM + r8 * kChTok * 2;
-#pragma unroll
-    for (int jp = 0; jp < kChTok / 16; ++jp) {
-      uint32_t xa[4];
-      ldsm_trans_at(xa, px + jp * 16 * kSsRows * 2);
-#pragma unroll
-      for (int ip = jp; ip < kChTok / 16; ++ip)
-        if (ip * 16 < nt_tok) {
-          uint32_t mb[4];
-          ldsm_at(mb, pm + (x8 ^ (jp << 5)) + ip * 16 * kChTok * 2);
-          mma_bf16_16816(Y[2 * ip], xa, mb[0], mb[1]);
-          mma_bf16_16816(Y[2 * ip + 1], xa, mb[2], mb[3]);
-        }
-      float xf[4][2];                           // rows pr, pr + 8 of tokens j, j + 1; the same of tokens j + 8, j + 9
-#pragma unroll
-      for (int i = 0; i < 4; ++i) {
-        xf[i][0] = bf16lo(xa[i]);
-        xf[i][1] = bf16hi(xa[i]);
-      }
-#pragma unroll
-      for (int e = 0; e < 2; ++e)
-#pragma unroll
-        for (int k = 0; k < 2; ++k) {
-          Y[2 * jp + e][k] = fmaf(skip, xf[2 * e][k], Y[2 * jp + e][k]);
-          Y[2 * jp + e][2 + k] = fmaf(skip, xf[2 * e + 1][k], Y[2 * jp + e][2 + k]);
-        }
-      const float2 w0 = *reinterpret_cast<const float2*>(w_s + jp * 16 + q2), w1 = *reinterpret_cast<const float2*>(w_s + jp * 16 + 8 + q2);
-      uint32_t hi[4], lo[4];
-      split_bf16(w0.x * xf[0][0], w0.y * xf[0][1], hi[0], lo[0]);
-      split_bf16(w0.x * xf[1][0], w0.y * xf[1][1], hi[1], lo[1]);
-      split_bf16(w1.x * xf[2][0], w1.y * xf[2][1], hi[2], lo[2]);
-      split_bf16(w1.x * xf[3][0], w1.y * xf[3][1], hi[3], lo[3]);
-#pragma unroll
-      for (int np = 0; np < NP / 16; np += 2) {
-        uint32_t b0[4], b1[4];
-        ldsm_trans_at(b0, pb + (xb ^ (np << 5)) + jp * 16 * NP * 2);
-        ldsm_trans_at(b1, pb + (xb ^ ((np + 1) << 5)) + jp * 16 * NP * 2);
-        mma_bf16_16816(S[2 * np], hi, b0[0], b0[1]);
-        mma_bf16_16816(S[2 * np + 1], hi, b0[2], b0[3]);
-        mma_bf16_16816(S[2 * np + 2], hi, b1[0], b1[1]);
-        mma_bf16_16816(S[2 * np + 3], hi, b1[2], b1[3]);
-        mma_bf16_16816(S[2 * np], lo, b0[0], b0[1]);
-        mma_bf16_16816(S[2 * np + 1], lo, b0[2], b0[3]);
-        mma_bf16_16816(S[2 * np + 2], lo, b1[0], b1[1]);
-        mma_bf16_16816(S[2 * np + 3], lo, b1[2], b1[3]);
-      }
-    }
-
-    // ---- store: pairs are transposed on the way out (token lane >> 2, entries q2, q2 + 1)
-    __nv_bfloat16* out = static_cast<__nv_bfloat16*>(a.y) + static_cast<long long>(first + (lane >> 2)) * inner + h * a.vdim + p0 +
-                         warp * 16 + q2;
-    const bool whole = nt_tok == kChTok && warp * 16 + 16 <= rows && (a.vdim & 1) == 0;
-#pragma unroll
-    for (int it = 0; it < kChTok / 8; ++it) {
-      if (it * 8 >= nt_tok) break;
-#pragma unroll
-      for (int e = 0; e < 2; ++e) {
-        const uint32_t v = transpose_8x8(pack_bf16(Y[it][2 * e], Y[it][2 * e + 1]));
-        __nv_bfloat16* dst = out + e * 8;
-        const int p = warp * 16 + e * 8 + q2;
-        if (whole) {
-          *reinterpret_cast<uint32_t*>(dst) = v;
-        } else if (it * 8 + (lane >> 2) < nt_tok) {
-          if (p < rows) dst[0] = __ushort_as_bfloat16(static_cast<unsigned short>(v & 0xffffu));
-          if (p + 1 < rows) dst[1] = __ushort_as_bfloat16(static_cast<unsigned short>(v >> 16));
-        }
-        __syncwarp();
-      }
-      out += 8ll * inner;
-    }
+  // exp(c_i - c_j) step_j of tokens j, j + 1; ci: entry i of the scalars
+  __device__ __forceinline__ float2 weights(const float* sc, float ci, int j) const {
+    const float2 cj = *reinterpret_cast<const float2*>(sc + j), sj = *reinterpret_cast<const float2*>(sc + kChTok + j);
+    return make_float2(ex2_approx(ci - cj.x) * sj.x, ex2_approx(ci - cj.y) * sj.y);
   }
-#pragma unroll
-  for (int nt = 0; nt < NP / 8; ++nt)
-#pragma unroll
-    for (int i = 0; i < 4; ++i) {
-      const int p = pr + (i >> 1) * 8, n = nt * 8 + q2 + (i & 1);
-      if (p < rows && n < N) st[static_cast<long long>(p) * N + n] = S[nt][i];
-    }
-  advance_conv_of_head(a, sq, t0, t1, fresh, h, p0, rows);
-}
+  __device__ __forceinline__ float2 readout(const float* sc, int i) const { return *reinterpret_cast<const float2*>(sc + 2 * kChTok + i); }
+  // past the end steps are zero: the whole chunk's decay
+  __device__ __forceinline__ float keep(const float* sc) const { return sc[3 * kChTok - 1]; }
+  __device__ __forceinline__ float skip() const { return a.skip[h]; }
+  __device__ __forceinline__ void finish(int sq, int p0, int rows, bool fresh) const {
+    advance_conv_of_head(a, sq, t0, t1, fresh, h, p0, rows);
+  }
+};
 
 // ------------------------------------------------------------------------------------------- norm
 constexpr int kSnThreads = 256;
@@ -968,8 +716,7 @@ static int run_np(const SsmArgs& a, int n_seqs, bool one_token, bool chunks, cud
     BCG_CUDA_CHECK(launch_k(ssm_token_kernel<T, NP>, grid, dim3(kSsThreads), 0, st, a));
   } else if (chunks) {
     constexpr int P = NP < 64 ? 64 : NP;
-    BCG_TRY(ensure_dynamic_smem(reinterpret_cast<const void*>(ssm_chunk_kernel<P>), ChCfg<P>::kSmem));
-    BCG_CUDA_CHECK(launch_k(ssm_chunk_kernel<P>, grid, dim3(kChThreads), ChCfg<P>::kSmem, st, a));
+    BCG_TRY((launch_chunks<P, SsdRule>(a, grid, st)));
   } else {
     BCG_CUDA_CHECK(launch_k(ssm_scan_kernel<T, NP>, grid, dim3(kSsThreads), 0, st, a));
   }

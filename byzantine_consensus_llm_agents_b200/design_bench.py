@@ -29,11 +29,13 @@ SIZES = {"2k": (2048, 6144, 8), "4k": (4096, 12288, 8)}
 # a stack's ff makes its layers (no gate matrix, other mixer projections) the dense layers' size
 BEKOPEL_FF = {"2k": 7424, "4k": 14592}
 MERULORN_FF = {"2k": 11520, "4k": 23680}       # of one layer in four; the others have none
+VOSOLORN_FF, VOSOLORN_EXPERT_FF = {"2k": 5632, "4k": 10752}, {"2k": 960, "4k": 1792}     # one expert in TOP + 1 is the shared one
 EXPERTS, TOP = 64, 8
 VOCAB, CTX, PROMPT, PROMPTS = 32768, 1600, 1536, 8
 FP32_FMA = 148 * 128 * 1.965e9       # nominal
 KINDS = {"bekopel": ("qwen3", "bekopel"), "lerazen": ("qwen3", "lerazen", "lerazen-moe"),
-         "merulorn": ("qwen3", "bekopel", "merulorn")}
+         "merulorn": ("qwen3", "bekopel", "merulorn"),
+         "vosolorn": ("qwen3", "merulorn", "lerazen-moe", "vosolorn", "vosolorn-moe")}
 
 
 def _config(kind: str, size: str):
@@ -43,6 +45,9 @@ def _config(kind: str, size: str):
         return S.bekopel_preset(name, layers, d, BEKOPEL_FF[size], VOCAB, heads=heads)
     if kind == "merulorn":
         return S.merulorn_preset(name, layers, d, MERULORN_FF[size], VOCAB, heads=heads)
+    if kind.startswith("vosolorn"):
+        return S.vosolorn_preset(name, layers, d, VOSOLORN_FF[size], VOCAB, heads=heads, experts=EXPERTS if kind.endswith("moe") else 0,
+                                 top=TOP, expert_ff=VOSOLORN_EXPERT_FF[size])
     if kind.startswith("lerazen"):      # two matrices instead of three; experts: three matrices, TOP of them active
         return S.lerazen_preset(name, layers, d, ff * 3 // 2, VOCAB, heads=heads, kv_heads=8,
                                 experts=EXPERTS if kind.endswith("moe") else 0, top=TOP, expert_ff=ff // TOP)
@@ -222,6 +227,22 @@ def _bekopel_kernels(k: _Bench, what: str, B: int, T: int, shape: str, v, plan) 
         st()), nbytes=T * ff * (2.0 + 4 * min(parts, 2)))
 
 
+def _route_at_random(k: _Bench, layer: int, T: int) -> int:
+    """The routing buffers of a layer as T tokens with random experts fill them; returns how many experts are used."""
+    b, f = k.e.buf, k.e.cfg.layers[layer].mlp
+    rows = T * f.top
+    pick = torch.rand(T, f.experts, generator=torch.Generator().manual_seed(0)).topk(f.top).indices.cuda()
+    counts = torch.bincount(pick.flatten(), minlength=f.experts)
+    order = pick.flatten().argsort(stable=True)
+    rank = torch.empty(rows, dtype=torch.int64, device="cuda")
+    rank[order] = torch.arange(rows, device="cuda")
+    rank -= (counts.cumsum(0) - counts)[pick.flatten()]
+    at = k.e.exec.model.struct.layers[layer].moe_counts_at
+    b["moe_counts"][at:at + f.experts], b["moe_expert"][:rows], b["moe_rank"][:rows] = counts.int(), pick.flatten().int(), rank.int()
+    b["moe_weight"][:rows] = 0.7
+    return int((counts > 0).sum())
+
+
 def _lerazen_kernels(k: _Bench, what: str, B: int, T: int, shape: str, v, plan) -> None:
     e, b, cfg, lib, x, st = k.e, k.e.buf, k.e.cfg, k.e.lib, k.e.exec, L.stream_ptr
     d, layer = cfg.d_model, cfg.n_layers - 1
@@ -240,18 +261,8 @@ def _lerazen_kernels(k: _Bench, what: str, B: int, T: int, shape: str, v, plan) 
           nbytes=T * n_in * (4.0 * s + 2) + T * m.kv_heads * m.vdim * 4.0)
     if moe:
         top, ff, rows = f.top, f.ff_ld, T * f.top
-        g = torch.Generator().manual_seed(0)
-        pick = torch.rand(T, f.experts, generator=g).topk(top).indices.cuda()
-        counts = torch.bincount(pick.flatten(), minlength=f.experts)
-        order = pick.flatten().argsort(stable=True)
-        rank = torch.empty(rows, dtype=torch.int64, device="cuda")
-        rank[order] = torch.arange(rows, device="cuda")
-        rank -= (counts.cumsum(0) - counts)[pick.flatten()]
-        at = x.model.struct.layers[layer].moe_counts_at
-        b["moe_counts"][at:at + f.experts], b["moe_expert"][:rows], b["moe_rank"][:rows] = counts.int(), pick.flatten().int(), rank.int()
-        b["moe_weight"][:rows] = 0.7
-        used, splits = int((counts > 0).sum()), C.c_int()
-        cp = b["moe_counts"].data_ptr() + 4 * at
+        used, splits = _route_at_random(k, layer, T), C.c_int()
+        cp = b["moe_counts"].data_ptr() + 4 * x.model.struct.layers[layer].moe_counts_at
         s1, s2 = (1, 1) if prefill else (L.splits_for(1, top * 2 * ff, d), L.splits_for(1, top * d, ff))
         size = 2.0 if prefill else 8.0 * s1
         k.add("experts, all launches", shape, lambda: lib.bcg_experts(model, ws, layer, T, C.byref(splits), st()),
@@ -319,9 +330,63 @@ def _merulorn_kernels(k: _Bench, what: str, B: int, T: int, shape: str, v, plan)
     k.gemm("output product", shape, b["mix"], w["w_out"], b["proj"], T, d, cols, L.EPI_F32, s3)
 
 
+def _vosolorn_kernels(k: _Bench, what: str, B: int, T: int, shape: str, v, plan) -> None:
+    e, b, cfg, lib, x, st = k.e, k.e.buf, k.e.cfg, k.e.lib, k.e.exec, L.stream_ptr
+    d, prefill = cfg.d_model, what == "prefill"
+    i_att = max(i for i, l in enumerate(cfg.layers) if l.one(S.GroupedAttention))
+    i_mem = max(i for i, l in enumerate(cfg.layers) if l.one(S.MatrixMemory))
+    m, mem, f, w = cfg.layers[i_att].mixer, cfg.layers[i_mem].mixer, cfg.layers[i_mem].mlp, e.w.layers[i_mem]
+    bt = _step_batch(e, what, T, B, v, plan)
+    model, ws = C.byref(x.model.struct), C.byref(x.ws)
+    splits = lambda n, kk: 1 if prefill else L.splits_for(B, n, kk)
+    blocks = lambda ctx: max(0, ctx - m.window) // m.pool
+    n_in, n_mem, s_out = cfg.in_rows(i_att), cfg.in_rows(i_mem), splits(d, mem.out_dim)
+    s, s_mem = splits(n_in, d), splits(n_mem, d)
+    pairs = _window_keys(m.window) + sum(blocks(p + 1) for p in range(PROMPT))
+    k.add("attention", shape, lambda: lib.bcg_grouped_attention(model, ws, C.byref(bt), i_att, 0, st()),
+          **(dict(flops=2.0 * B * pairs * m.heads * (m.dim + m.vdim)) if prefill
+             else dict(nbytes=B * (min(m.window, CTX) + blocks(CTX)) * m.kv_heads * (m.dim + m.vdim) * 2.0)))
+    k.add("input split", shape, lambda: lib.bcg_grouped_in(model, ws, C.byref(bt), i_att, s, T * n_in, n_in, 0, st()),
+          nbytes=T * m.in_dim * (4.0 * s + 2))
+    # the projection in, outputs out, states in and out; the products of 64-token chunks
+    k.add("matrix memory, all launches", shape, lambda: lib.bcg_matrix_memory(model, ws, C.byref(bt), i_mem, s_mem, T * n_mem, n_mem, 0, st()),
+          nbytes=T * (mem.in_dim * 4.0 * s_mem + mem.out_dim * 2) + B * mem.state_floats * 8.0,
+          flops=2.0 * T * mem.heads * (mem.vdim * (32 + 2 * mem.dim) + 32 * mem.dim) if prefill else 0.0)
+    k.add("norm", shape, lambda: lib.bcg_sandwich_norm(
+        b["residual"].data_ptr(), b["proj"].data_ptr(), s_out, T * d, w["norm1b"].data_ptr(), None, b["xn"].data_ptr(), L.DT_BF16, T, d,
+        1e-5, st()), nbytes=T * d * (10.0 + 4 * s_out))
+    k.gemm("input product", shape, b["xn"], w["w_in"], b["proj"], T, n_mem, d, L.EPI_F32, s_mem)
+    k.gemm("output product", shape, b["mix"], w["w_out"], b["proj"], T, d, mem.out_dim, L.EPI_F32, s_out)
+    if isinstance(f, S.MoeMlp):
+        used, rows, ff = _route_at_random(k, i_mem, T), T * f.top, f.ff_ld
+        out = C.c_int()
+        k.add("experts, all launches", shape, lambda: lib.bcg_experts(model, ws, i_mem, T, C.byref(out), st()),
+              nbytes=used * 4.0 * ff * d + rows * d * 4.0, flops=4.0 * rows * ff * d)
+        n = f.router_rows + f.shared_ld
+        k.gemm("router and shared product", shape, b["xn"], w["w_up"], b["proj"], T, n, d, L.EPI_F32, splits(n, d))
+        s_sh = splits(d, f.shared_ld)
+        k.add("norm with experts", shape, lambda: lib.bcg_residual_norm(
+            b["residual"].data_ptr(), b["proj"].data_ptr(), s_sh, T * d, None, b["moe_out"].data_ptr(), b["moe_row"].data_ptr(),
+            b["moe_weight"].data_ptr(), f.top, out.value, rows * d, w["norm2b"].data_ptr(), None, b["xn"].data_ptr(), L.DT_BF16, T, d, 1e-5,
+            st()), nbytes=T * d * (10.0 + 4 * s_sh + 4 * f.top * out.value))
+        return
+    n_up = f.up_rows
+    if splits(n_up, d) == 1:
+        k.add("up product", shape, lambda: lib.bcg_gemm_bf16_gelu(
+            b["xn"].data_ptr(), w["w_up"].data_ptr(), b["act"].data_ptr(), T, n_up, d, 1, 0, st()),
+            nbytes=2.0 * n_up * d + 2.0 * T * d + T * n_up, flops=2.0 * T * n_up * d)
+    else:
+        k.gemm("up product", shape, b["xn"], w["w_up"], b["proj"], T, n_up, d, L.EPI_F32, splits(n_up, d))
+        k.add("activation", shape, lambda: lib.bcg_gelu_unit(
+            b["proj"].data_ptr(), splits(n_up, d), T * n_up, b["act"].data_ptr(), L.DT_BF16, T, f.ff_ld, 1, st()),
+            nbytes=T * f.ff_ld * (8.0 * splits(n_up, d) + 2))
+    k.gemm("down product", shape, b["act"], w["w_down"], b["proj"], T, d, f.ff_ld, L.EPI_F32, splits(d, f.ff_ld))
+
+
 def _kernels(e: Engine, kind: str, hbm: float, tf: float) -> list:
     k = _Bench(e, hbm, tf)
-    run = {"qwen3": _dense_kernels, "bekopel": _bekopel_kernels, "merulorn": _merulorn_kernels}.get(kind, _lerazen_kernels)
+    run = {"qwen3": _dense_kernels, "bekopel": _bekopel_kernels, "merulorn": _merulorn_kernels, "vosolorn": _vosolorn_kernels,
+           "vosolorn-moe": _vosolorn_kernels}.get(kind, _lerazen_kernels)
     for what, B in (("prefill", PROMPTS), ("decode", 8), ("decode", 64)):
         T = B * PROMPT if what == "prefill" else B
         plan, v = _prefill(e, B) if what == "prefill" else (None, None)
@@ -343,16 +408,18 @@ def _run(kind: str, size: str, tokenizer, hbm: float, tf: float, kernels: bool) 
         ms = _events(_graph(lambda: e.exec.decode(e.row, B, (CTX + 255) // 256), 4), 20) / 4
         cache = e.cfg.kv_bytes_per_token * (CTX if kind == "qwen3" else min(CTX, e.cfg.max_window or CTX))
         weights = e.cfg.decode_weight_bytes()
-        if kind == "lerazen-moe":           # the experts that the step's tokens used
+        if kind.endswith("-moe"):           # the experts that the step's tokens used
             f = e.cfg.layers[-1].mlp
             used = int((e.buf["moe_counts"][:e.ws.moe_counts_n] > 0).sum())
-            weights = e.cfg.decode_weight_bytes(0) + used * 6 * f.ff * e.cfg.d_model
+            weights = e.cfg.decode_weight_bytes(0) + used * (6 if f.glu else 4) * f.ff * e.cfg.d_model
             out[f"experts_used_per_layer_{B}"] = round(used * f.experts / e.ws.moe_counts_n, 1)
         if kind == "bekopel":     # layers that share a cache read it once each; states are read and written
             own = sum(isinstance(l.mixer, S.LatentAttention) for l in e.cfg.layers)
             has = sum(isinstance(l.mixer, S.LatentAttention) and l.mixer.kv_from is None for l in e.cfg.layers)
             cache = cache * own // max(has, 1) + 2 * e.cfg.state_bytes_per_row
-        if kind == "merulorn":
+        if kind.startswith("vosolorn"):     # the blocks behind the window, too
+            cache += sum(e.cfg.pool_bytes_per_block(p) * max(0, CTX - e.cfg.max_window) // p for p in e.cfg.pools)
+        if kind == "merulorn" or kind.startswith("vosolorn"):
             cache += 2 * e.cfg.state_bytes_per_row
         out[f"decode_ms_{B}"] = round(ms, 4)
         out[f"decode_tok_s_{B}"] = round(B / ms * 1e3)

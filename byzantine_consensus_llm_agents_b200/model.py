@@ -83,6 +83,7 @@ PRESETS = {
     "lerazen-30b-a3b": stack.lerazen_preset("lerazen-30b-a3b", 48, 2048, 6144, 151936, kv_heads=4, experts=128, top=8,
                                             expert_ff=768),
     "merulorn-8b": stack.merulorn_preset("merulorn-8b", 48, 4096, 12288, 151936),
+    "vosolorn-8b": stack.vosolorn_preset("vosolorn-8b", 36, 4096, 10752, 151936),
 }
 
 _HF_NAMES = {

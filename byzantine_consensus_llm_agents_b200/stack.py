@@ -771,6 +771,21 @@ def merulorn_preset(name: str, n_layers: int, d_model: int, ff: int, vocab: int,
     return StackConfig(name, d_model, vocab, layers, max_pos=max_pos, sinusoid_pos=True, embed_scale=d_model ** 0.5, norm_offset=1.0)
 
 
+def vosolorn_preset(name: str, n_layers: int, d_model: int, ff: int, vocab: int, heads: int = 32, kv_heads: int = 8, dim: int = 128,
+                    window: int = 512, pool: int = 16, mem_dim: int = 128, mem_vdim: int = 256, experts: int = 0, top: int = 8,
+                    expert_ff: int = 1024, max_pos: int = 32768) -> StackConfig:
+    """Vosolorn at sizes of a real model's layers (random-init presets, bench): one layer in four has attention, the others a
+    matrix memory; dense feed-forwards, or, with `experts`, a dense one in the first layer and experts, one of them shared, in
+    the others."""
+    att = GroupedAttention(heads, kv_heads, dim, dim, dim ** -0.5, window, slopes=False, out_bias=False, in_bias=False, head_norm=True,
+                           rot=Rotary(1e6, dim, True), v_rot=Rotary(1e6, dim, True), pool=pool)
+    mem = MatrixMemory(d_model // mem_vdim, mem_dim, mem_vdim, 15.0)
+    dense = DenseMlp(ff, "gelu_glu")
+    moe = MoeMlp(experts, top, expert_ff, act="gelu", shared=expert_ff) if experts else dense
+    layers = tuple(LayerSpec(mem if i % 4 else att, moe if i else dense, pre_norm=False, layer_scale=True) for i in range(n_layers))
+    return StackConfig(name, d_model, vocab, layers, max_pos=max_pos, embed_norm=True, tied_head=True, logit_scale=d_model ** -0.5)
+
+
 # ------------------------------------------------------------------------------------------ weights
 def head_slopes(heads: int, device) -> torch.Tensor:
     """[heads] fp32 distance slopes 2^(-8 (h + 1) / heads)."""

@@ -1,5 +1,5 @@
-"""Small random layer-stack models for the tests: config.json dicts of the Bekopel, Lerazen and Merulorn designs, their
-tensors, and model directories.  Weights are scaled so that every mechanism moves the logits: scores spread over
+"""Small random layer-stack models for the tests: config.json dicts of the Bekopel, Lerazen, Merulorn and Vosolorn designs,
+their tensors, and model directories.  Weights are scaled so that every mechanism moves the logits: scores spread over
 several units, sinks that take a visible share, decays from fast to almost none, all four activation numbers set,
 biases and mixed values of the size of what they join.  Routers are decisive: a few coordinates of the stream hold
 a code of the token that no layer touches, and the router reads mostly those, so that rounding does not choose
@@ -141,6 +141,83 @@ def parallel_tensors(cfg, seed=0):
     return {n: x.to(torch.bfloat16) for n, x in t.items()}
 
 
+def pattn(heads=6, kv_heads=3, dim=24, vdim=40, size=20, pool=6, dims=16, base=1e4, scale=None, mlp=None):
+    return {"type": "attention", "mlp": mlp,
+            "mixer": {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "mask": {"size": size, "pool": pool},
+                      "rot": {"base": base, "dims": dims}, "scale": scale or 2.0 * dim ** -0.5}}
+
+
+def mlstm(heads=3, dim=24, vdim=40, cap=9.0, mlp=None):
+    return {"type": "mlstm", "mlp": mlp, "mixer": {"heads": heads, "dim": dim, "vdim": vdim, "gate_cap": cap}}
+
+
+def plain_moe(experts=6, top=2, ff=40, shared=24):
+    return {"kind": "moe", "expert": {"ff": ff}, "router": {"experts": experts, "top": top}, **({"shared": {"ff": shared}} if shared else {})}
+
+
+def output_norm_config(layers, width=80, vocab=200, eps=1e-5, scale=0.4):
+    return {"architecture": "Vosolorn", "layers": layers, "norm": {"eps": eps}, "vocab": vocab, "width": width, "logit_scale": scale}
+
+
+def output_norm_tensors(cfg, seed=0):
+    g = torch.Generator().manual_seed(seed)
+    rnd = lambda *s, std=1.0, mean=0.0: torch.randn(*s, generator=g) * std + mean
+    d, V = cfg["width"], cfg["vocab"]
+    lin = lambda n, k, gain=1.0: rnd(n, k, std=gain * k ** -0.5)
+    routers = [l["mlp"]["router"]["experts"] for l in cfg["layers"] if l["mlp"] and l["mlp"]["kind"] == "moe"]
+    # the last coordinates of the stream: a constant, then the code
+    code = max(routers, default=0)
+    own = code + 1
+
+    def out(*s, gain=1.0):                        # output matrices leave them alone
+        w = lin(*s, gain)
+        w[d - own:] = 0
+        return w
+    t = {"embed": rnd(V, d), "embed.norm": rnd(d, std=0.2, mean=1.0), "final.norm": rnd(d, std=0.2, mean=1.0)}
+    t["embed.norm"][d - own:] = 1
+    t["embed"][:, d - own] = 2
+    if code:
+        for v in range(V):
+            t["embed"][v, d - code:] = torch.linspace(-3, 3, code)[torch.randperm(code, generator=g)]
+    step = 12.0 / max(code - 1, 1) / (1 + 2.0 * code / d) ** 0.5        # between two neighbouring logits of a router
+    for i, l in enumerate(cfg["layers"]):
+        p, m, f = f"l{i}.", l["mixer"], l["mlp"]
+        for n in ("norm1", "ls1") + (("norm2", "ls2") if f else ()):
+            t[p + n] = rnd(d, std=0.2, mean=1.0 if n.startswith("norm") else 0.8)
+        H = m["heads"]
+        if l["type"] == "attention":
+            G = m["kv_heads"]
+            t.update({p + "mix.q": lin(H * m["dim"], d), p + "mix.k": lin(G * m["dim"], d), p + "mix.v": lin(G * m["vdim"], d),
+                      p + "mix.q.norm": rnd(m["dim"], std=0.4, mean=1.2), p + "mix.k.norm": rnd(m["dim"], std=0.4, mean=1.2),
+                      p + "mix.o": out(d, H * m["vdim"], gain=1.5)})
+        else:
+            n = H * m["vdim"]
+            # Forget gates from a few tokens to thousands of them; input gates above and below the running maximum.  Keys and
+            # queries share a part that every token has: a head's output, which is divided by its own root mean square, is a sum
+            # with positive weights and does not cancel, so that rounding does not choose its sign.
+            k, q, same = lin(H * m["dim"], d), lin(H * m["dim"], d), rnd(H * m["dim"])
+            k[:, d - own], q[:, d - own] = same, same
+            t.update({p + "mix.q": q, p + "mix.k": k, p + "mix.v": lin(n, d), p + "mix.g": lin(n, d),
+                      p + "mix.i": lin(H, d, 1.5), p + "mix.i.b": torch.linspace(1.0, -2.0, H), p + "mix.f": lin(H, d),
+                      p + "mix.f.b": torch.linspace(0.0, 8.0, H)[torch.randperm(H, generator=g)], p + "mix.norm": rnd(n, std=0.2, mean=1.0),
+                      p + "mix.o": out(d, n)})
+        if f and f["kind"] == "dense":
+            t.update({p + "mlp.gate": lin(f["ff"], d, 1.5), p + "mlp.up": lin(f["ff"], d, 1.5), p + "mlp.down": out(d, f["ff"])})
+        elif f:
+            E, n = f["router"]["experts"], f["expert"]["ff"]
+            router = lin(E, d, 0.02)
+            router[:, d - code:] = 0
+            for e, c in enumerate(torch.randperm(code, generator=g)[:E]):
+                router[e, d - code + c] = 2.0
+            # logits stay apart: every other expert is lifted by about a third of the distance between two neighbours
+            t.update({p + "mlp.router": router, p + "mlp.router.b": 0.37 * step * (torch.arange(E) % 2)})
+            for e in range(E):
+                t.update({p + f"mlp.e{e}.up": lin(n, d, 2.0), p + f"mlp.e{e}.down": out(d, n, gain=1.5)})
+            if "shared" in f:
+                t.update({p + "mlp.shared.up": lin(f["shared"]["ff"], d, 2.0), p + "mlp.shared.down": out(d, f["shared"]["ff"])})
+    return {n: x.to(torch.bfloat16) for n, x in t.items()}
+
+
 def config(layers, width=80, vocab=200, eps=1e-5):
     return {"architecture": "Bekopel", "layers": layers, "norm": {"eps": eps}, "vocab": vocab, "width": width}
 
@@ -151,6 +228,8 @@ def tensors(cfg, seed=0, decay_rank=12):
         return parallel_tensors(cfg, seed)
     if cfg["architecture"] == "Merulorn":
         return side_tensors(cfg, seed)
+    if cfg["architecture"] == "Vosolorn":
+        return output_norm_tensors(cfg, seed)
     g = torch.Generator().manual_seed(seed)
     rnd = lambda *s, std=1.0, mean=0.0: (torch.randn(*s, generator=g) * std + mean).to(torch.bfloat16)
     d, V = cfg["width"], cfg["vocab"]

@@ -60,8 +60,21 @@ CONFIGS = {
     "side-wide": SM.side_config([SM.both(33, 1, 40, 8, heads_ssm=1, vdim_ssm=136, state=250, groups=1, norm_groups=1, mlp=SM.glu(16)),
                                  SM.both(2, 2, 264, 264, heads_ssm=1, vdim_ssm=8, state=8, groups=1, norm_groups=1)], width=96, vocab=96),
     "state-only": SM.side_config([SM.mamba(heads=1, vdim=8, state=16, groups=1, norm_groups=1), SM.mamba(heads=16, vdim=32, state=32, groups=8, norm_groups=16)], width=64, vocab=64),
+    # pooled blocks of several sizes, longer than the window and shorter than a page's part, beside matrix memories
+    "pooled": SM.output_norm_config([SM.pattn(mlp=SM.plain_moe()), SM.mlstm(mlp=SM.dense(70)), SM.pattn(4, 1, 16, 24, 5, 9, 8, base=100.0),
+                                     SM.mlstm(2, 16, 72, 4.0, mlp=SM.plain_moe(5, 3, 24, 0)), SM.pattn(3, 3, 40, 16, 1, 1, 40, mlp=SM.plain_moe(4, 1, 20, 40))]),
+    # everything on the tensor-core kernels
+    "pooled-tensor": SM.output_norm_config([SM.mlstm(4, 64, 128, 15.0, mlp=SM.plain_moe(8, 3, 64, 96)), SM.pattn(8, 2, 64, 64, 33, 4, 64, mlp=SM.dense(320)),
+                                            SM.mlstm(3, 128, 80, mlp=SM.dense(64)), SM.pattn(4, 4, 128, 128, 70, 16, 32, mlp=SM.plain_moe(8, 1, 128, 64)),
+                                            SM.pattn(2, 1, 200, 248, 17, 3, 24), SM.mlstm(1, 200, 24)], width=192, vocab=320),
+    # sizes no vector load or tile likes, groups of more than 16 query heads, heads beyond the tiles
+    "pooled-odd": SM.output_norm_config([SM.pattn(3, 1, 7, 10, 19, 5, 6, mlp=SM.dense(45)), SM.mlstm(5, 9, 13, 1.5, mlp=SM.plain_moe(5, 3, 21, 11)),
+                                         SM.pattn(33, 1, 13, 6, 40, 7, 0), SM.pattn(2, 2, 264, 260, 50, 24, 100), SM.mlstm(1, 250, 7)],
+                                        width=61, vocab=83, eps=1e-3, scale=1.0),
+    "pooled-one": SM.output_norm_config([SM.pattn(1, 1, 8, 8, 5, 2, 8, mlp=SM.dense(20))], width=36, vocab=36),
+    "memory-only": SM.output_norm_config([SM.mlstm(1, 8, 16), SM.mlstm(2, 32, 64, 20.0, mlp=SM.plain_moe(9, 9, 8, 8))], width=64, vocab=64),
 }
-ATTENTION_MIX = ["mixed", "tensor", "parallel", "parallel-tensor", "side", "side-tensor"]
+ATTENTION_MIX = ["mixed", "tensor", "parallel", "parallel-tensor", "side", "side-tensor", "pooled", "pooled-tensor"]
 
 
 class Model:
@@ -79,7 +92,7 @@ class Model:
 
     def given_back(self):
         e = self.eng
-        return len(e.pool.free) == e.pool.n_pages and len(e.slots.free) == e.slots.n
+        return all(len(p.free) == p.n_pages for p in [e.pool, *e.block_pools]) and len(e.slots.free) == e.slots.n
 
     def check(self, got, want):
         got, want = got.double().cpu(), want.double()
@@ -192,7 +205,7 @@ def test_pool_is_as_large_as_asked_and_says_when_it_is_full():
 
 
 @pytest.mark.parametrize("dtype", TOL)
-@pytest.mark.parametrize("name", ["mixed", "parallel", "side"])
+@pytest.mark.parametrize("name", ["mixed", "parallel", "side", "pooled", "pooled-tensor"])
 def test_long_decoding(name, dtype):
     """Windows pass over decoded tokens many times over; the state is carried through every one of them."""
     m = Model(name, dtype)
@@ -201,12 +214,14 @@ def test_long_decoding(name, dtype):
 
 
 @pytest.mark.parametrize("dtype", ["float32"])
-@pytest.mark.parametrize("name", ["mixed", "state-only"])
+@pytest.mark.parametrize("name", ["mixed", "state-only", "memory-only"])
 def test_a_far_token_is_remembered(name, dtype):
     """Slow decays: logits hundreds of tokens later depend on the first ones (a lost state would show)."""
     m = Model(name, dtype)
-    for n in ("l1.mix.w0", "l4.mix.w0") if name == "mixed" else ("l0.mix.A_log", "l1.mix.A_log"):
-        m.t[n] -= 6.0
+    shift = {"mixed": {"l1.mix.w0": -6.0, "l4.mix.w0": -6.0}, "state-only": {"l0.mix.A_log": -6.0, "l1.mix.A_log": -6.0},
+             "memory-only": {"l0.mix.f.b": 8.0, "l1.mix.f.b": 8.0, "l0.mix.i.b": -3.0, "l1.mix.i.b": -3.0}}
+    for n, by in shift[name].items():
+        m.t[n] += by
     m.eng = SM.engine(m.cfg, m.t, dtype)
     toks = m.tokens(300, 4)
     want = m.oracle(toks)
@@ -227,7 +242,7 @@ def test_learned_positions_end_where_the_table_does():
 
 
 @pytest.mark.parametrize("dtype", TOL)
-@pytest.mark.parametrize("name", ["parallel-tensor", "side-tensor"])
+@pytest.mark.parametrize("name", ["parallel-tensor", "side-tensor", "pooled-tensor"])
 def test_prompts_of_many_tiles(name, dtype):
     """More tokens than one row tile of the products, several prompt tiles and chunks, windows across them."""
     m = Model(name, dtype, tokens=1024, max_model_len=512)
@@ -262,7 +277,9 @@ GENS = {"Bekopel": GEN, "Lerazen": SM.parallel_config([SM.gattn(4, 2, 32, 32, 24
                                                        SM.gattn(2, 2, 40, 48, 1000, v_mix=False, mlp=SM.moe(4, 1, 32))],
                                                       width=128, vocab=1024, positions=600),
         "Merulorn": SM.side_config([SM.mamba(heads=4, vdim=32, state=32), SM.both(4, 2, 32, 32, mlp=SM.glu(96)), SM.mamba(heads=2, vdim=64, state=40, norm_groups=1),
-                                    SM.both(2, 1, 64, 64, vdim_ssm=16, mlp=SM.glu(64, 0.7))], width=128, vocab=1024)}
+                                    SM.both(2, 1, 64, 64, vdim_ssm=16, mlp=SM.glu(64, 0.7))], width=128, vocab=1024),
+        "Vosolorn": SM.output_norm_config([SM.pattn(4, 2, 32, 32, 24, 3, 16, mlp=SM.plain_moe(8, 2, 48, 32)), SM.mlstm(2, 32, 48, mlp=SM.dense(96)),
+                                           SM.mlstm(4, 16, 64), SM.pattn(2, 1, 64, 64, 16, 8, 64, mlp=SM.plain_moe(4, 1, 32, 16))], width=128, vocab=1024)}
 
 
 def _greedy(cfg, t, ids, out):
@@ -299,6 +316,7 @@ def test_greedy_generation_through_the_scheduler(design, dtype, graph):
         assert again.token_ids == res[3].token_ids
     # a prefix is taken from its pages where they are all there is to it
     assert again.cached_tokens == (0 if eng.exec.has_state else 32)
+    assert all(len(p.free) == p.n_pages for p in eng.block_pools)
     assert len(eng.slots.free) == eng.slots.n and len(eng.pool.free) + len(eng.pool.cached) == eng.pool.n_pages
 
 
@@ -333,7 +351,7 @@ def test_adapter_generates_from_a_model_directory(design, tmp_path):
 
 # ------------------------------------------------------------------------------------------ trace replay
 @pytest.mark.parametrize("dtype", TOL)
-@pytest.mark.parametrize("name", ["tensor", "parallel-tensor", "side-tensor"])
+@pytest.mark.parametrize("name", ["tensor", "parallel-tensor", "side-tensor", "pooled-tensor"])
 def test_trace_replay_program(tmp_path, name, dtype):
     cfg = CONFIGS[name]
     t = SM.tensors(cfg, seed=11)

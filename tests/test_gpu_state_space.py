@@ -30,9 +30,10 @@ def close(got, want, tol):
 
 class OneLayer:
     """A one-layer model inside an engine; its buffers are set and read by hand."""
+    make = staticmethod(SM.side_config)
 
     def __init__(self, layer, dtype, width=64, seed=0, tokens=512, rows=6, **kw):
-        self.cfg = SM.side_config([layer], width=width, vocab=16)
+        self.cfg = self.make([layer], width=width, vocab=16)
         self.t = SM.tensors(self.cfg, seed=seed)
         self.t.update(kw.pop("tensors", {}))
         self.eng = SM.engine(self.cfg, self.t, dtype, tokens=tokens, rows=rows, **kw)

@@ -168,6 +168,7 @@ def test_preset_resolves_by_name():
     with pytest.raises(ValueError, match="tensor parallelism"):
         c.shard(2)
     c = M.config_for("lerazen-30b-a3b")
+    assert M.config_for("vosolorn-8b").pools == (16,)
     assert M.config_for("merulorn-8b").layers[0].mixer.right.state == 128
     assert c.layers[0].mlp.act == "relu2" and c.layers[1].mlp.experts == 128 and c.v_first == 0
 
@@ -230,6 +231,108 @@ def test_bad_side_configurations_are_refused(spoil, words):
     spoil(c)
     with pytest.raises(ValueError, match=words):
         SM.stack_config(c, SM.tensors(SIDE))
+
+
+# ---------------------------------------------------------------------------------------- norms on outputs only
+POOLED = SM.output_norm_config([SM.pattn(6, 2, 10, 14, 33, 5, 6, mlp=SM.plain_moe(5, 2, 21, 11)), SM.mlstm(3, 7, 9, 4.5, mlp=SM.dense(20)),
+                                SM.pattn(2, 2, 8, 8, 7, 40, 8), SM.mlstm(2, 24, 70, mlp=SM.plain_moe(3, 1, 16, 0))], width=60, eps=1e-3, scale=0.3)
+
+
+def test_pooled_config_comes_from_the_directory(tmp_path):
+    t = SM.tensors(POOLED)
+    c = M.config_from_dir(str(SM.save(POOLED, t, tmp_path / "m")))
+    assert isinstance(c, S.StackConfig) and set(c.tensor_shapes()) == set(t)
+    assert all(tuple(t[n].shape) == s for n, s in c.tensor_shapes().items())
+    assert c.embed_norm and c.tied_head and c.rms_eps == 1e-3 and c.has_state and c.pools == (5, 40) and c.max_window == 33
+    m = c.layers[0].mixer
+    assert m == S.GroupedAttention(6, 2, 10, 14, 2.0 * 10 ** -0.5, 33, slopes=False, out_bias=False, in_bias=False, head_norm=True,
+                                   rot=S.Rotary(1e4, 6, True), v_rot=S.Rotary(1e4, 14, True), pool=5)
+    assert c.layers[1].mixer == S.MatrixMemory(3, 7, 9, 4.5) and c.layers[1].mlp == S.DenseMlp(20, "gelu_glu")
+    assert c.layers[0].mlp == S.MoeMlp(5, 2, 21, act="gelu", shared=11) and c.layers[3].mlp.shared == 0 and c.layers[2].mlp is None
+    assert c.state_bytes_per_row == 4 * (3 * (10 * 7 + 1) + 2 * (71 * 24 + 2))
+    w = S.StackWeights.from_safetensors_dir(c, tmp_path / "m", "cpu")
+    # factors join the norms in front of them; the head is the embedding
+    assert torch.allclose(w.final_norm, 0.3 * t["final.norm"].float()) and torch.equal(w.embed_norm, t["embed.norm"].float())
+    assert torch.equal(w.lm_head[:200], t["embed"]) and "norm1" not in w.layers[0]
+    assert torch.allclose(w.layers[0]["norm1b"], t["l0.norm1"].float() * t["l0.ls1"].float())
+    assert torch.allclose(w.layers[3]["norm2b"], t["l3.norm2"].float() * t["l3.ls2"].float()) and "norm2b" not in w.layers[2]
+
+
+def test_memory_and_plain_expert_rows_are_packed():
+    t = SM.tensors(POOLED)
+    c = SM.stack_config(POOLED, t)
+    w = S.StackWeights.from_tensors(c, t.__getitem__, "cpu")
+    a, b = w.layers[0], w.layers[1]
+    m = c.layers[1].mixer
+    assert m.gate_col == 96 and c.in_rows(1) == 112 and b["w_in"].shape == (112, 60)          # 2 * 3 * (7 + 9) rows, then the gates
+    assert torch.equal(b["w_in"][21:42], t["l1.mix.k"]) and torch.equal(b["w_in"][69:96], t["l1.mix.g"])
+    assert torch.equal(b["w_in"][96:102], torch.cat([t["l1.mix.i"], t["l1.mix.f"]])) and not b["w_in"][102:].any()
+    assert torch.equal(b["w_out"][:, :27], t["l1.mix.o"]) and not b["w_out"][:, 27:].any()
+    assert torch.equal(b["mem_bias"], torch.cat([t["l1.mix.i.b"], t["l1.mix.f.b"]]).float())
+    f = c.layers[0].mlp
+    assert (f.router_rows, f.shared_ld, f.ff_ld, f.in_rows) == (16, 16, 32, 32) and a["w_up"].shape == (32, 60)
+    assert torch.equal(a["w_up"][:5], t["l0.mlp.router"]) and torch.equal(a["w_up"][16:27], t["l0.mlp.shared.up"])
+    assert not a["w_up"][5:16].any() and not a["w_up"][27:].any() and torch.equal(a["w_down"][:, :11], t["l0.mlp.shared.down"])
+    assert torch.equal(a["w_experts_in"][3, :21], t["l0.mlp.e3.up"]) and torch.equal(a["w_experts_out"][4, :, :21], t["l0.mlp.e4.down"])
+    assert not a["w_experts_in"][:, 21:].any() and not a["w_experts_out"][:, :, 21:].any() and "w_down" not in w.layers[3]
+
+
+@pytest.mark.parametrize("spoil, words", [
+    (lambda c: c["layers"][0].update(type="other"), "unknown mixer"),
+    (lambda c: c["layers"][1]["mlp"].update(kind="other"), "unknown feed-forward"),
+    (lambda c: c["layers"][0]["mixer"].update(kv_heads=4), "key/value heads"),
+    (lambda c: c["layers"][0]["mixer"]["rot"].update(dims=12), "rotary dims 12 of 10"),
+    (lambda c: c["layers"][0]["mixer"]["mask"].update(size=0), "pooled blocks"),
+    (lambda c: c["layers"][1]["mixer"].update(dim=257), "256 key channels"),
+    (lambda c: c["layers"][0]["mlp"]["router"].update(top=6), "6 of 5 experts"),
+])
+def test_bad_pooled_configurations_are_refused(spoil, words):
+    import copy
+    c = copy.deepcopy(POOLED)
+    spoil(c)
+    with pytest.raises(ValueError, match=words):
+        SM.stack_config(c, SM.tensors(POOLED))
+
+
+def test_pages_of_pooled_blocks():
+    from byzantine_consensus_llm_agents_b200.executors import PAGE, block_pages_for
+    assert [block_pages_for(n, 5) for n in (0, 4, 5, 5 * PAGE, 5 * PAGE + 4, 5 * PAGE + 5)] == [0, 0, 1, 1, 1, 2]
+
+
+def test_oracle_matrix_memory_can_be_carried():
+    g = torch.Generator().manual_seed(4)
+    rnd = lambda *s: torch.randn(*s, generator=g, dtype=torch.float64)
+    q, k, v, i, f = rnd(9, 2, 3), rnd(9, 2, 3), rnd(9, 2, 5), 3 * rnd(9, 2), -rnd(9, 2).abs()
+    whole, (S_, n, m) = R.memory_scan(q, k, v, i, f)
+    y1, s1 = R.memory_scan(q[:4], k[:4], v[:4], i[:4], f[:4])
+    y2, s2 = R.memory_scan(q[4:], k[4:], v[4:], i[4:], f[4:], s1)
+    assert torch.allclose(whole, torch.cat([y1, y2])) and all(torch.allclose(a, b) for a, b in zip((S_, n, m), s2))
+    # without a running maximum: the plain sums, scaled
+    c = torch.cumsum(f, 0)
+    w = torch.exp(i + c[-1] - c)[:, :, None]                # weight of token j at the end
+    assert torch.allclose(n * m.exp()[:, None], (w * k).sum(0)) and (m >= c[-1]).all()
+    nq = ((w * k).sum(0) * q[-1]).sum(-1)
+    o = torch.einsum("jhd,jhe,hd->he", w * k, v, q[-1])
+    want = o / (torch.maximum(nq.abs(), torch.ones_like(nq)) + 1e-6 * m.exp())[:, None]
+    assert torch.allclose(whole[-1], want)
+    assert torch.allclose(R.memory_gates(torch.ones(1, 1), {"i": torch.ones(1, 1), "i.b": torch.zeros(1), "f": torch.ones(1, 1) * 50,
+                                                            "f.b": torch.zeros(1)}, 2.0)[0], torch.tensor(2 * np.tanh(0.5)).float())
+
+
+def test_oracle_blocks_rotation_and_experts():
+    # 3-token blocks behind a window of 4: block b is seen from position 3b + 6 on
+    seen = R.blocks_visible(12, 4, 4, 3)
+    assert [int(seen[:, b].float().argmax()) for b in range(2)] == [6, 9] and not seen[:, 2:].any()
+    assert R.block_means(torch.arange(8.0)[:, None], 3).flatten().tolist() == [1.0, 4.0]
+    x, pos = torch.randn(5, 2, 7, dtype=torch.float64), torch.tensor([0, 3, 4, 90, 7])
+    y = R.rotate_pairs(x, pos, 4, 100.0)
+    a = 3 * 100.0 ** -0.5
+    assert torch.allclose(y[1, 0, 2:4], torch.stack([x[1, 0, 2] * np.cos(a) - x[1, 0, 3] * np.sin(a), x[1, 0, 3] * np.cos(a) + x[1, 0, 2] * np.sin(a)]))
+    assert torch.equal(y[..., 4:], x[..., 4:]) and torch.allclose(R.rotate_pairs(y, pos, 4, 100.0, back=True), x)
+    e, w = R.route_softmax(torch.tensor([[1.0, 2.0, 0.0]]), torch.eye(3), torch.tensor([0.0, -5.0, 2.0]), 2)
+    assert e.tolist() == [[2, 0]] and torch.allclose(w, torch.softmax(torch.tensor([[2.0, 1.0]]), -1))
+    z = torch.tensor([-1.5, 0.0, 2.0], dtype=torch.float64)
+    assert torch.allclose(R.gelu_erf(z), torch.nn.functional.gelu(z)) and torch.allclose(R.gelu_tanh(z), torch.nn.functional.gelu(z, approximate="tanh"))
 
 
 def test_position_turns_are_the_oracles_frequencies():
