@@ -199,24 +199,155 @@ __device__ __forceinline__ long long page_row(const int* bt, int j0, int i, int 
   return (static_cast<long long>(bt[j0 + i / page_size]) * kv_heads + g) * page_size + i % page_size;
 }
 
-// Mean of `pool` rows of a cache, the cached ones of positions p0 .. and `last`, added in their order.
+// Sum of n rows of a cache from position p0 on, in their order; a whole warp, every lane with columns c .. c + V - 1 of `width`.
 template <typename T, int V>
-__device__ __forceinline__ Vec<V> block_mean(const T* cache, const int* bt, int kv_heads, int g, int page_size, int ld, int c, int p0,
-                                             int pool, const Vec<V>* last) {
+__device__ __forceinline__ Vec<V> rows_sum(const T* cache, const int* bt, int kv_heads, int g, int page_size, int ld, int c, int width,
+                                           int p0, int n) {
+  const int lane = threadIdx.x & 31;
   Vec<V> sum;
 #pragma unroll
   for (int k = 0; k < V; ++k) sum.x[k] = 0.f;
-  const int n = last ? pool - 1 : pool;
-#pragma unroll 4
-  for (int j = 0; j < n; ++j) sum.add(load_vec<V>(cache + page_row(bt, 0, p0 + j, kv_heads, g, page_size) * ld + c));
-  if (last) sum.add(*last);
+  for (int j0 = 0; j0 < n; j0 += 32) {
+    const int mine = static_cast<int>(page_row(bt, 0, p0 + min(j0 + lane, n - 1), kv_heads, g, page_size));
+    const int m = min(32, n - j0);
+    for (int j1 = 0; j1 < m; j1 += 8) {
+      Vec<V> v[8];
 #pragma unroll
-  for (int k = 0; k < V; ++k) sum.x[k] /= static_cast<float>(pool);
+      for (int j = 0; j < 8; ++j) {
+        const long long row = __shfl_sync(0xffffffffu, mine, min(j1 + j, m - 1));
+        if (c < width) v[j] = load_vec<V>(cache + row * ld + c);
+      }
+#pragma unroll
+      for (int j = 0; j < 8; ++j)
+        if (j1 + j < m && c < width) sum.add(v[j]);
+    }
+  }
+  return sum;
+}
+template <int V>
+__device__ __forceinline__ Vec<V> divided(Vec<V> sum, int n) {
+#pragma unroll
+  for (int k = 0; k < V; ++k) sum.x[k] /= static_cast<float>(n);
   return sum;
 }
 
-// One head of a token (queries, then keys, then values) per warp: norm, rotation, destination.  blocks: the step has one token per
-// sequence, so whoever writes the last row of a block also writes its mean.
+// What a warp needs of one head of a token: queries, then keys, then values.
+struct HeadUnit {
+  long long t;
+  int g, width, dims, col, ld, pos, slot;
+  bool is_q, is_v, there;
+  __device__ __forceinline__ HeadUnit(const GroupedIn& a, long long unit) {
+    const int per = a.heads + 2 * a.kv_heads;
+    there = unit < static_cast<long long>(a.n_tokens) * per;
+    if (!there) unit = 0;
+    t = unit / per;
+    const int s = static_cast<int>(unit - t * per);
+    is_q = s < a.heads;
+    is_v = s >= a.heads + a.kv_heads;
+    g = is_q ? s : s - a.heads - (is_v ? a.kv_heads : 0);
+    width = is_v ? a.vdim : a.dim;
+    dims = is_v ? a.v_rot_dims : a.rot_dims;
+    col = is_q ? g * a.dim : is_v ? (a.heads + a.kv_heads) * a.dim + g * a.vdim : (a.heads + g) * a.dim;
+    ld = is_v ? a.v_ld : a.q_ld;
+    pos = a.positions[t];
+    slot = a.slot_map[t];
+  }
+  template <typename T>
+  __device__ __forceinline__ T* cache(const GroupedIn& a) const { return static_cast<T*>(is_v ? a.v_cache : a.k_cache); }
+  // row of the queries or of the cache, NULL: the token is not stored
+  template <typename T>
+  __device__ __forceinline__ T* destination(const GroupedIn& a) const {
+    if (!there) return nullptr;
+    if (is_q) return static_cast<T*>(a.q) + (t * a.heads + g) * a.q_ld;
+    return slot < 0 ? nullptr : cache<T>(a) + ((static_cast<long long>(slot / a.page_size) * a.kv_heads + g) * a.page_size + slot % a.page_size) * ld;
+  }
+  __device__ __forceinline__ const float* norm(const GroupedIn& a) const { return is_q ? a.q_norm : is_v ? nullptr : a.k_norm; }
+  // cosines, sines dims / 2 behind them
+  __device__ __forceinline__ const float* angles(const GroupedIn& a) const {
+    return (is_v ? a.v_cos_sin : a.cos_sin) + static_cast<long long>(pos) * dims;
+  }
+  __device__ __forceinline__ bool ends_block(const GroupedIn& a) const { return a.pool > 0 && there && !is_q && slot >= 0 && (pos + 1) % a.pool == 0; }
+  template <typename T>
+  __device__ __forceinline__ T* block_row(const GroupedIn& a) const {
+    return cache<T>(a) + page_row(a.block_table + t * a.max_blocks, a.pool_col, pos / a.pool, a.kv_heads, g, a.page_size) * ld;
+  }
+};
+
+// Heads in registers: rotation in pairs of neighbours, up to 128 * NC entries, multiples of four.  A warp has U heads.  blocks: the
+// step has one token per sequence, so whoever writes the last row of a block also writes its mean.
+template <typename T, int NC, int U>
+__global__ void __launch_bounds__(kInThreads)
+head_pairs_kernel(const GroupedIn a, bool blocks) {
+  const int lane = threadIdx.x & 31;
+  const long long first = (blockIdx.x * static_cast<long long>(kInThreads / 32) + (threadIdx.x >> 5)) * U;
+  pdl_launch_dependents();
+  if constexpr (U > 1) pdl_wait();
+  Vec<4> x[U][NC], sum[NC];
+#pragma unroll
+  for (int i = 0; i < U; ++i) {
+    const HeadUnit u(a, first + i);
+    if constexpr (U == 1) {         // the block's other rows and the positions were there before this step
+      if (blocks && u.ends_block(a)) {
+#pragma unroll
+        for (int n = 0; n < NC; ++n)
+          sum[n] = rows_sum<T, 4>(u.cache<T>(a), a.block_table + u.t * a.max_blocks, a.kv_heads, u.g, a.page_size, u.ld, (n * 32 + lane) * 4,
+                                  u.width, u.pos + 1 - a.pool, a.pool - 1);
+      }
+      pdl_wait();
+    }
+    const float* row = a.proj + u.t * a.ld + u.col;
+#pragma unroll
+    for (int n = 0; n < NC; ++n) {
+      const int c = (n * 32 + lane) * 4;
+      if (c < u.width) x[i][n] = slab_sum_vec<4>(row + c, a.n_partials, a.pstride);
+      else x[i][n] = Vec<4>{};
+      if (a.bias && c < u.width) x[i][n].add(load_vec<4>(a.bias + u.col + c));
+    }
+  }
+#pragma unroll
+  for (int i = 0; i < U; ++i) {
+    const HeadUnit u(a, first + i);
+    if (!u.there) return;
+    const float* w = u.norm(a);
+    float inv = 1.f;
+    if (w) {
+      float ss = 0.f;
+#pragma unroll
+      for (int n = 0; n < NC; ++n) ss += x[i][n].sumsq();
+      inv = rsqrtf(warp_sum(ss) / static_cast<float>(u.width) + a.eps);
+    }
+    const float* angle = u.angles(a);
+    const int half = u.dims / 2;
+    T* dst = u.destination<T>(a);
+    const bool whole = U == 1 && blocks && u.ends_block(a);
+#pragma unroll
+    for (int n = 0; n < NC; ++n) {
+      const int c = (n * 32 + lane) * 4;
+      if (c >= u.width) break;
+      Vec<4> y = x[i][n];
+      if (w) {
+        const Vec<4> ww = load_vec<4>(w + c);
+#pragma unroll
+        for (int k = 0; k < 4; ++k) y.x[k] *= inv * ww.x[k];
+      }
+#pragma unroll
+      for (int k = 0; k < 4; k += 2)
+        if (c + k < u.dims) {
+          const float cs = angle[(c + k) / 2], sn = angle[half + (c + k) / 2], p = y.x[k], q = y.x[k + 1];
+          y.x[k] = p * cs - q * sn;
+          y.x[k + 1] = q * cs + p * sn;
+        }
+      if (dst) store_vec<4>(dst + c, y);
+      if (whole) {
+#pragma unroll
+        for (int k = 0; k < 4; ++k) sum[n].x[k] += sizeof(T) == 2 ? to_f32<T>(from_f32<T>(y.x[k])) : y.x[k];      // as the cache holds it
+        store_vec<4>(u.block_row<T>(a) + c, divided(sum[n], a.pool));
+      }
+    }
+  }
+}
+
+// Any head: a warp has one, through shared memory.
 template <typename T, int V>
 __global__ void __launch_bounds__(kInThreads)
 head_in_kernel(const GroupedIn a, int pitch, bool blocks) {
@@ -225,44 +356,34 @@ head_in_kernel(const GroupedIn a, int pitch, bool blocks) {
   float* x = reinterpret_cast<float*>(stage_raw) + warp * pitch;
   pdl_launch_dependents();
   pdl_wait();
-  const int per = a.heads + 2 * a.kv_heads;
-  const long long unit = blockIdx.x * static_cast<long long>(kInThreads / 32) + warp;
-  const long long t = unit / per;
-  if (t >= a.n_tokens) return;
-  const int s = static_cast<int>(unit - t * per);
-  const bool is_q = s < a.heads, is_v = s >= a.heads + a.kv_heads;
-  const int g = is_q ? s : s - a.heads - (is_v ? a.kv_heads : 0);
-  const int width = is_v ? a.vdim : a.dim, dims = is_v ? a.v_rot_dims : a.rot_dims, half = dims / 2;
-  const int col = is_q ? g * a.dim : is_v ? (a.heads + a.kv_heads) * a.dim + g * a.vdim : (a.heads + g) * a.dim;
-  const bool pairs = is_v || a.rot_pairs;
-  const int pos = a.positions[t], slot = a.slot_map[t];
-  const float* row = a.proj + t * a.ld + col;
+  const HeadUnit u(a, blockIdx.x * static_cast<long long>(kInThreads / 32) + warp);
+  if (!u.there) return;
+  const int half = u.dims / 2;
+  const bool pairs = u.is_v || a.rot_pairs;
+  const float* row = a.proj + u.t * a.ld + u.col;
   float ss = 0.f;
-  for (int c = lane * V; c < width; c += 32 * V) {
+  for (int c = lane * V; c < u.width; c += 32 * V) {
     Vec<V> v = slab_sum_vec<V>(row + c, a.n_partials, a.pstride);
-    if (a.bias) v.add(load_vec<V>(a.bias + col + c));
+    if (a.bias) v.add(load_vec<V>(a.bias + u.col + c));
     store_vec<V>(x + c, v);
     ss += v.sumsq();
   }
-  const float* w = is_q ? a.q_norm : is_v ? nullptr : a.k_norm;
-  const float inv = w ? rsqrtf(warp_sum(ss) / static_cast<float>(width) + a.eps) : 1.0f;
+  const float* w = u.norm(a);
+  const float inv = w ? rsqrtf(warp_sum(ss) / static_cast<float>(u.width) + a.eps) : 1.0f;
   __syncwarp();
-  const float* angle = (is_v ? a.v_cos_sin : a.cos_sin) + static_cast<long long>(pos) * dims;
-  const int ld = is_v ? a.v_ld : a.q_ld;
-  T* cache = static_cast<T*>(is_v ? a.v_cache : a.k_cache);
-  T* dst = nullptr;
-  if (is_q) dst = static_cast<T*>(a.q) + (t * a.heads + g) * a.q_ld;
-  else if (slot >= 0) dst = cache + ((static_cast<long long>(slot / a.page_size) * a.kv_heads + g) * a.page_size + slot % a.page_size) * ld;
-  const bool whole = blocks && a.pool > 0 && !is_q && slot >= 0 && (pos + 1) % a.pool == 0;
-  const int* bt = a.block_table + t * a.max_blocks;
-  for (int c = lane * V; c < width; c += 32 * V) {
+  const float* angle = u.angles(a);
+  T* dst = u.destination<T>(a);
+  const bool whole = blocks && u.ends_block(a);
+  for (int c0 = 0; c0 < u.width; c0 += 32 * V) {
+    const int c = c0 + lane * V;
     Vec<V> y;
 #pragma unroll
     for (int k = 0; k < V; ++k) {
       const int e = c + k;
+      if (e >= u.width) continue;
       const float own = x[e] * (w ? inv * w[e] : 1.0f);
       y.x[k] = own;
-      if (e < dims) {
+      if (e < u.dims) {
         const bool first = pairs ? !(e & 1) : e < half;
         const int p = pairs ? e ^ 1 : first ? e + half : e - half, i = pairs ? e >> 1 : first ? e : e - half;
         const float other = x[p] * (w ? inv * w[p] : 1.0f), cs = angle[i], sn = angle[half + i];
@@ -270,27 +391,30 @@ head_in_kernel(const GroupedIn a, int pitch, bool blocks) {
       }
       if (sizeof(T) == 2) y.x[k] = to_f32<T>(from_f32<T>(y.x[k]));      // as the cache holds it
     }
-    if (dst) store_vec<V>(dst + c, y);
+    if (dst && c < u.width) store_vec<V>(dst + c, y);
     if (whole) {
-      const int b = pos / a.pool;
-      const Vec<V> mean = block_mean<T, V>(cache, bt, a.kv_heads, g, a.page_size, ld, c, b * a.pool, a.pool, &y);
-      store_vec<V>(cache + page_row(bt, a.pool_col, b, a.kv_heads, g, a.page_size) * ld + c, mean);
+      Vec<V> sum = rows_sum<T, V>(u.cache<T>(a), a.block_table + u.t * a.max_blocks, a.kv_heads, u.g, a.page_size, u.ld, c, u.width,
+                                  u.pos + 1 - a.pool, a.pool - 1);
+      if (c < u.width) {
+        sum.add(y);
+        store_vec<V>(u.block_row<T>(a) + c, divided(sum, a.pool));
+      }
     }
   }
 }
 
-// A warp has a run of 32 tokens and a key or value head: the means of the blocks that end there.
+// A warp has a run of `run` tokens (up to 32) and a key or value head: the means of the blocks that end there.
 template <typename T, int V>
 __global__ void __launch_bounds__(kInThreads)
-pool_blocks_kernel(const GroupedIn a, const int* __restrict__ row_seq) {
+pool_blocks_kernel(const GroupedIn a, const int* __restrict__ row_seq, int run) {
   pdl_launch_dependents();
   pdl_wait();
   const int lane = threadIdx.x & 31;
   const long long unit = blockIdx.x * static_cast<long long>(kInThreads / 32) + (threadIdx.x >> 5);
   const int s = static_cast<int>(unit % (2 * a.kv_heads));
-  const long long t0 = unit / (2 * a.kv_heads) * 32;
+  const long long t0 = unit / (2 * a.kv_heads) * run;
   if (t0 >= a.n_tokens) return;
-  const bool is_v = s >= a.kv_heads, mine = t0 + lane < a.n_tokens;
+  const bool is_v = s >= a.kv_heads, mine = lane < run && t0 + lane < a.n_tokens;
   const int g = is_v ? s - a.kv_heads : s, width = is_v ? a.vdim : a.dim, ld = is_v ? a.v_ld : a.q_ld;
   T* cache = static_cast<T*>(is_v ? a.v_cache : a.k_cache);
   const int pos = mine ? a.positions[t0 + lane] : 0;
@@ -299,25 +423,45 @@ pool_blocks_kernel(const GroupedIn a, const int* __restrict__ row_seq) {
     const int i = __ffs(ends) - 1, b = __shfl_sync(0xffffffffu, pos, i) / a.pool;
     const int* bt = a.block_table + static_cast<long long>(row_seq ? row_seq[t0 + i] : t0 + i) * a.max_blocks;
     T* dst = cache + page_row(bt, a.pool_col, b, a.kv_heads, g, a.page_size) * ld;
-    for (int c = lane * V; c < width; c += 32 * V)
-      store_vec<V>(dst + c, block_mean<T, V>(cache, bt, a.kv_heads, g, a.page_size, ld, c, b * a.pool, a.pool, nullptr));
+    for (int c0 = 0; c0 < width; c0 += 32 * V) {
+      const int c = c0 + lane * V;
+      const Vec<V> sum = rows_sum<T, V>(cache, bt, a.kv_heads, g, a.page_size, ld, c, width, b * a.pool, a.pool);
+      if (c < width) store_vec<V>(dst + c, divided(sum, a.pool));
+    }
   }
+}
+
+template <typename T, int NC>
+static int head_pairs_t(const GroupedIn& a, bool one_token, cudaStream_t st) {
+  const long long units = static_cast<long long>(a.n_tokens) * (a.heads + 2 * a.kv_heads);
+  constexpr int kFew = 4096, kPer = NC == 1 ? 4 : 2;
+  const long long per = (units <= kFew || one_token ? 1 : kPer) * (kInThreads / 32);
+  const dim3 grid(static_cast<unsigned>((units + per - 1) / per));
+  if (units <= kFew || one_token) BCG_CUDA_CHECK(launch_k(head_pairs_kernel<T, NC, 1>, grid, dim3(kInThreads), 0, st, a, one_token));
+  else BCG_CUDA_CHECK(launch_k(head_pairs_kernel<T, NC, kPer>, grid, dim3(kInThreads), 0, st, a, false));
+  return BCG_OK;
 }
 
 template <typename T, int V>
 static int head_in_t(const GroupedIn& a, const int* row_seq, bool one_token, cudaStream_t st) {
-  const int pitch = (max(a.dim, a.vdim) + 3) / 4 * 4;
-  const size_t sm = static_cast<size_t>(kInThreads / 32) * pitch * 4;
-  if (sm > 200 * 1024) {
-    set_last_error("bcg_grouped_in", "heads are too large");
-    return BCG_ERR_UNSUPPORTED;
+  const int wide = max(a.dim, a.vdim);
+  if (V == 4 && a.rot_pairs && wide <= 256) {
+    BCG_TRY(wide <= 128 ? (head_pairs_t<T, 1>(a, one_token, st)) : (head_pairs_t<T, 2>(a, one_token, st)));
+  } else {
+    const int pitch = (wide + 3) / 4 * 4;
+    const size_t sm = static_cast<size_t>(kInThreads / 32) * pitch * 4;
+    if (sm > 200 * 1024) {
+      set_last_error("bcg_grouped_in", "heads are too large");
+      return BCG_ERR_UNSUPPORTED;
+    }
+    if (sm > 48 * 1024) BCG_TRY(ensure_dynamic_smem(reinterpret_cast<const void*>(head_in_kernel<T, V>), 200 * 1024));
+    const long long units = static_cast<long long>(a.n_tokens) * (a.heads + 2 * a.kv_heads);
+    BCG_CUDA_CHECK(launch_k(head_in_kernel<T, V>, dim3(static_cast<unsigned>((units + 7) / 8)), dim3(kInThreads), sm, st, a, pitch, one_token));
   }
-  if (sm > 48 * 1024) BCG_TRY(ensure_dynamic_smem(reinterpret_cast<const void*>(head_in_kernel<T, V>), 200 * 1024));
-  const long long units = static_cast<long long>(a.n_tokens) * (a.heads + 2 * a.kv_heads);
-  BCG_CUDA_CHECK(launch_k(head_in_kernel<T, V>, dim3(static_cast<unsigned>((units + 7) / 8)), dim3(kInThreads), sm, st, a, pitch, one_token));
   if (a.pool > 0 && !one_token) {
-    const long long runs = static_cast<long long>((a.n_tokens + 31) / 32) * 2 * a.kv_heads;
-    BCG_CUDA_CHECK(launch_k(pool_blocks_kernel<T, V>, dim3(static_cast<unsigned>((runs + 7) / 8)), dim3(kInThreads), 0, st, a, row_seq));
+    const int run = min(max(a.pool, 4), 32);
+    const long long runs = static_cast<long long>((a.n_tokens + run - 1) / run) * 2 * a.kv_heads;
+    BCG_CUDA_CHECK(launch_k(pool_blocks_kernel<T, V>, dim3(static_cast<unsigned>((runs + 7) / 8)), dim3(kInThreads), 0, st, a, row_seq, run));
   }
   return BCG_OK;
 }

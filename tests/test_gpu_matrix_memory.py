@@ -38,7 +38,7 @@ class Memory(OneLayer):
         """Rows q | k | v | g and gates of t tokens; keys and queries share a part, so that outputs do not cancel."""
         H, D, V = self.dims
         x, g = torch.randn(t, self.rows, generator=gen(seed)), torch.randn(t, 2 * H, generator=gen(seed + 1)) * gates
-        same = torch.randn(H * D, generator=gen(99))
+        same = 1.5 * torch.randn(H * D, generator=gen(99))
         x[:, :H * D] += same
         x[:, H * D:2 * H * D] += same
         return torch.cat([x, g], dim=1)
@@ -130,7 +130,7 @@ def test_the_maximum_starts_at_zero_and_bounds_the_denominator(dtype):
     H, D, V = a.dims
     proj[:, a.rows:a.rows + H] -= 6.0
     want = a.oracle(proj)
-    assert (want[1][:3] <= 2.5).all() and (want[1] > 0.99).all()
+    assert (want[1] > 0.99).all() and (want[2][2] < -1.0).any()
     for slot, sizes in enumerate(([100], [1], [64, 2, 1])):
         a.junk()
         a.check(a.feed(proj, sizes, slot), want, slot, loose=3.0)
