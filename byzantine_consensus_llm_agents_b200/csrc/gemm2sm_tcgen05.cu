@@ -360,7 +360,8 @@ gemm2sm_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_
 int gemm2sm_bf16_tn(const void* X, const void* W, void* out, int M, int N, int K, long long ldx, long long ldw,
                     long long ld_out, int epi, float glu_limit, float glu_alpha, cudaStream_t stream) {
   // the last column tile may be partial (the epilogue stores 32 columns at a time), where that wastes little
-  if (M < 512 || (N % 32) != 0 || (N % k2BlockN != 0 && N < 8 * k2BlockN)) return BCG_ERR_UNSUPPORTED;
+  const int idle = (N + k2BlockN - 1) / k2BlockN * k2BlockN - N;
+  if (M < 512 || (N % 32) != 0 || idle * 8ll > N) return BCG_ERR_UNSUPPORTED;
   static const bool off = getenv("BCG_GEMM_2SM") && atoi(getenv("BCG_GEMM_2SM")) == 0;   // tuning knob
   if (off) return BCG_ERR_UNSUPPORTED;
   Gemm2Args a = {};

@@ -648,6 +648,9 @@ int gemm_splits_for(int M, int N, int K) {
   return best;
 }
 
+// Tiles of 256 columns where they cover no more than tiles of 128 would.
+static bool wide_tiles(int N) { return (N + 255) / 256 * 2 == (N + 127) / 128; }
+
 static int gemm_dense(const void* X, const void* W, void* out, int M, int N, int K, long long ldx, long long ldw,
                       long long ld_out, int epi, int splits, int flags, const bcg_gemm_fusion* fu, float glu_limit,
                       float glu_alpha, cudaStream_t stream);
@@ -768,7 +771,7 @@ static int gemm_dense(const void* X, const void* W, void* out, int M, int N, int
     a.hint_a = kEvictFirst;  // weights are streamed exactly once per step
     a.hint_b = kEvictLast;
   } else {
-    bn = (N % 256 == 0) ? 256 : 128;
+    bn = wide_tiles(N) ? 256 : 128;
     if (epi == BCG_EPI_F32 && bn == 256 && N < 2048) bn = 128;
     a.tiles_a = (M + kBlockA - 1) / kBlockA;
     a.tiles_b = (N + bn - 1) / bn;
@@ -826,7 +829,7 @@ int gemm_grouped(const void* X, const void* W, void* out, int rows, int N, int K
   a.glu_alpha = g.glu_alpha;
   a.pdl_wait_b = (launch_flags() & BCG_GEMM_PDL) ? 1 : 0;
   const int bn = swap ? (g.max_rows <= 16 ? 16 : g.max_rows <= 32 ? 32 : g.max_rows <= 64 ? 64 : 128)
-                      : (N % 256 == 0 ? 256 : 128);
+                      : (wide_tiles(N) ? 256 : 128);
   const int tile_rows = swap ? bn : kBlockA, w_tiles = swap ? (N + kBlockA - 1) / kBlockA : (N + bn - 1) / bn;
   a.tiles_a = swap ? w_tiles : 1;
   a.tiles_b = swap ? 1 : w_tiles;

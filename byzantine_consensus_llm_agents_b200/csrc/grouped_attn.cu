@@ -199,30 +199,33 @@ __device__ __forceinline__ long long page_row(const int* bt, int j0, int i, int 
   return (static_cast<long long>(bt[j0 + i / page_size]) * kv_heads + g) * page_size + i % page_size;
 }
 
-// Sum of n rows of a cache from position p0 on, in their order; a whole warp, every lane with columns c .. c + V - 1 of `width`.
-template <typename T, int V>
-__device__ __forceinline__ Vec<V> rows_sum(const T* cache, const int* bt, int kv_heads, int g, int page_size, int ld, int c, int width,
-                                           int p0, int n) {
-  const int lane = threadIdx.x & 31;
-  Vec<V> sum;
+// Sum of n rows of a cache from position p0 on, in their order: NV vectors of V columns per lane, the first at column c, for the lanes
+// that want it.  Groups of L lanes share the look-ups; n is the warp's.
+template <typename T, int V, int NV, int L>
+__device__ __forceinline__ void rows_sum(Vec<V> (&sum)[NV], const T* cache, const int* bt, int kv_heads, int g, int page_size, int ld, int c,
+                                         bool want, int p0, int n) {
+  const int lane = threadIdx.x % L;
 #pragma unroll
-  for (int k = 0; k < V; ++k) sum.x[k] = 0.f;
-  for (int j0 = 0; j0 < n; j0 += 32) {
+  for (int i = 0; i < NV; ++i) sum[i] = Vec<V>{};
+  for (int j0 = 0; j0 < n; j0 += L) {
     const int mine = static_cast<int>(page_row(bt, 0, p0 + min(j0 + lane, n - 1), kv_heads, g, page_size));
-    const int m = min(32, n - j0);
+    const int m = min(L, n - j0);
     for (int j1 = 0; j1 < m; j1 += 8) {
-      Vec<V> v[8];
+      Vec<V> v[8][NV];
 #pragma unroll
       for (int j = 0; j < 8; ++j) {
-        const long long row = __shfl_sync(0xffffffffu, mine, min(j1 + j, m - 1));
-        if (c < width) v[j] = load_vec<V>(cache + row * ld + c);
+        const T* row = cache + static_cast<long long>(__shfl_sync(0xffffffffu, mine, min(j1 + j, m - 1), L)) * ld + c;
+#pragma unroll
+        for (int i = 0; i < NV; ++i)
+          if (want) v[j][i] = load_vec<V>(row + i * V);
       }
 #pragma unroll
       for (int j = 0; j < 8; ++j)
-        if (j1 + j < m && c < width) sum.add(v[j]);
+#pragma unroll
+        for (int i = 0; i < NV; ++i)
+          if (j1 + j < m && want) sum[i].add(v[j][i]);
     }
   }
-  return sum;
 }
 template <int V>
 __device__ __forceinline__ Vec<V> divided(Vec<V> sum, int n) {
@@ -231,117 +234,154 @@ __device__ __forceinline__ Vec<V> divided(Vec<V> sum, int n) {
   return sum;
 }
 
-// What a warp needs of one head of a token: queries, then keys, then values.
+// A token whose heads (queries, then keys, then values) warps take one by one.
+struct HeadToken {
+  int t, pos, slot, n_heads;
+  bool ends_block;             // of pooled keys
+  __device__ __forceinline__ HeadToken(const GroupedIn& a, int t_) : t(t_), pos(a.positions[t_]), slot(a.slot_map[t_]), n_heads(a.heads + 2 * a.kv_heads) {
+    ends_block = a.pool > 0 && slot >= 0 && (pos + 1) % a.pool == 0;
+  }
+};
 struct HeadUnit {
-  long long t;
-  int g, width, dims, col, ld, pos, slot;
-  bool is_q, is_v, there;
-  __device__ __forceinline__ HeadUnit(const GroupedIn& a, long long unit) {
-    const int per = a.heads + 2 * a.kv_heads;
-    there = unit < static_cast<long long>(a.n_tokens) * per;
-    if (!there) unit = 0;
-    t = unit / per;
-    const int s = static_cast<int>(unit - t * per);
+  int g, width, dims, col, ld;
+  bool is_q, is_v;
+  __device__ __forceinline__ HeadUnit(const GroupedIn& a, int s) {
     is_q = s < a.heads;
     is_v = s >= a.heads + a.kv_heads;
     g = is_q ? s : s - a.heads - (is_v ? a.kv_heads : 0);
     width = is_v ? a.vdim : a.dim;
     dims = is_v ? a.v_rot_dims : a.rot_dims;
-    col = is_q ? g * a.dim : is_v ? (a.heads + a.kv_heads) * a.dim + g * a.vdim : (a.heads + g) * a.dim;
+    col = is_v ? (a.heads + a.kv_heads) * a.dim + g * a.vdim : s * a.dim;
     ld = is_v ? a.v_ld : a.q_ld;
-    pos = a.positions[t];
-    slot = a.slot_map[t];
   }
   template <typename T>
   __device__ __forceinline__ T* cache(const GroupedIn& a) const { return static_cast<T*>(is_v ? a.v_cache : a.k_cache); }
   // row of the queries or of the cache, NULL: the token is not stored
   template <typename T>
-  __device__ __forceinline__ T* destination(const GroupedIn& a) const {
-    if (!there) return nullptr;
-    if (is_q) return static_cast<T*>(a.q) + (t * a.heads + g) * a.q_ld;
-    return slot < 0 ? nullptr : cache<T>(a) + ((static_cast<long long>(slot / a.page_size) * a.kv_heads + g) * a.page_size + slot % a.page_size) * ld;
+  __device__ __forceinline__ T* destination(const GroupedIn& a, const HeadToken& at) const {
+    if (is_q) return static_cast<T*>(a.q) + (static_cast<long long>(at.t) * a.heads + g) * ld;
+    if (at.slot < 0) return nullptr;
+    const int page = at.slot / a.page_size;
+    return cache<T>(a) + ((static_cast<long long>(page) * a.kv_heads + g) * a.page_size + at.slot - page * a.page_size) * ld;
   }
   __device__ __forceinline__ const float* norm(const GroupedIn& a) const { return is_q ? a.q_norm : is_v ? nullptr : a.k_norm; }
   // cosines, sines dims / 2 behind them
-  __device__ __forceinline__ const float* angles(const GroupedIn& a) const {
+  __device__ __forceinline__ const float* angles(const GroupedIn& a, int pos) const {
     return (is_v ? a.v_cos_sin : a.cos_sin) + static_cast<long long>(pos) * dims;
   }
-  __device__ __forceinline__ bool ends_block(const GroupedIn& a) const { return a.pool > 0 && there && !is_q && slot >= 0 && (pos + 1) % a.pool == 0; }
   template <typename T>
-  __device__ __forceinline__ T* block_row(const GroupedIn& a) const {
-    return cache<T>(a) + page_row(a.block_table + t * a.max_blocks, a.pool_col, pos / a.pool, a.kv_heads, g, a.page_size) * ld;
+  __device__ __forceinline__ T* block_row(const GroupedIn& a, const HeadToken& at) const {
+    return cache<T>(a) +
+           page_row(a.block_table + static_cast<long long>(at.t) * a.max_blocks, a.pool_col, at.pos / a.pool, a.kv_heads, g, a.page_size) * ld;
   }
 };
 
-// Heads in registers: rotation in pairs of neighbours, up to 128 * NC entries, multiples of four.  A warp has U heads.  blocks: the
-// step has one token per sequence, so whoever writes the last row of a block also writes its mean.
-template <typename T, int NC, int U>
-__global__ void __launch_bounds__(kInThreads)
-head_pairs_kernel(const GroupedIn a, bool blocks) {
-  const int lane = threadIdx.x & 31;
-  const long long first = (blockIdx.x * static_cast<long long>(kInThreads / 32) + (threadIdx.x >> 5)) * U;
-  pdl_launch_dependents();
-  if constexpr (U > 1) pdl_wait();
-  Vec<4> x[U][NC], sum[NC];
+// Cosines and sines of the four pairs from column c (a multiple of eight) on; pairs behind `dims` do not turn.
+struct PairAngles {
+  float cs[4], sn[4];
+  __device__ __forceinline__ void load(const float* row, int dims, int c) {
+    const int m = c / 2, half = dims / 2;
+    if (c + 8 <= dims && dims % 8 == 0) {
+      const float4 a = __ldg(reinterpret_cast<const float4*>(row + m)), b = __ldg(reinterpret_cast<const float4*>(row + half + m));
+      cs[0] = a.x; cs[1] = a.y; cs[2] = a.z; cs[3] = a.w;
+      sn[0] = b.x; sn[1] = b.y; sn[2] = b.z; sn[3] = b.w;
+    } else {
 #pragma unroll
-  for (int i = 0; i < U; ++i) {
-    const HeadUnit u(a, first + i);
-    if constexpr (U == 1) {         // the block's other rows and the positions were there before this step
-      if (blocks && u.ends_block(a)) {
-#pragma unroll
-        for (int n = 0; n < NC; ++n)
-          sum[n] = rows_sum<T, 4>(u.cache<T>(a), a.block_table + u.t * a.max_blocks, a.kv_heads, u.g, a.page_size, u.ld, (n * 32 + lane) * 4,
-                                  u.width, u.pos + 1 - a.pool, a.pool - 1);
+      for (int k = 0; k < 4; ++k) {
+        cs[k] = m + k < half ? row[m + k] : 1.f;
+        sn[k] = m + k < half ? row[half + m + k] : 0.f;
       }
-      pdl_wait();
-    }
-    const float* row = a.proj + u.t * a.ld + u.col;
-#pragma unroll
-    for (int n = 0; n < NC; ++n) {
-      const int c = (n * 32 + lane) * 4;
-      if (c < u.width) x[i][n] = slab_sum_vec<4>(row + c, a.n_partials, a.pstride);
-      else x[i][n] = Vec<4>{};
-      if (a.bias && c < u.width) x[i][n].add(load_vec<4>(a.bias + u.col + c));
     }
   }
+  __device__ __forceinline__ void turn(Vec<4>& v, int first) const {
+#pragma unroll
+    for (int k = 0; k < 2; ++k) {
+      const float p = v.x[2 * k], q = v.x[2 * k + 1];
+      v.x[2 * k] = p * cs[first + k] - q * sn[first + k];
+      v.x[2 * k + 1] = q * cs[first + k] + p * sn[first + k];
+    }
+  }
+};
+
+// Heads in registers: rotation in pairs of neighbours, multiples of eight entries up to 8 * L.  L lanes have a head, a warp has 32 / L
+// at a time and U times that; `groups` CTAs per token.  blocks: the step has one token per sequence, so whoever writes the last row
+// of a block also writes its mean.
+template <typename T, int L, int U>
+__global__ void __launch_bounds__(kInThreads)
+head_pairs_kernel(const GroupedIn a, int groups, bool blocks) {
+  constexpr int kAtOnce = 32 / L, kPerCta = kInThreads / 32 * kAtOnce * U;
+  const int t = blockIdx.x / groups, c = threadIdx.x % L * 8;
+  const int warp_first = (blockIdx.x - t * groups) * kPerCta + static_cast<int>(threadIdx.x >> 5) * kAtOnce * U;
+  const int first = warp_first + static_cast<int>(threadIdx.x & 31) / L;
+  pdl_launch_dependents();
+  const HeadToken at(a, t);
+  if (warp_first >= at.n_heads) return;
+  auto unit = [&](int i) { return HeadUnit(a, min(first + i * kAtOnce, at.n_heads - 1)); };
+  Vec<4> x[U][2], sum[2];
+  const bool whole = U == 1 && blocks && at.ends_block;
+  if constexpr (U == 1) {         // the block's other rows and the positions were there before this step
+    if (whole && warp_first + kAtOnce > a.heads) {
+      const HeadUnit u = unit(0);
+      rows_sum<T, 4, 2, L>(sum, u.cache<T>(a), a.block_table + static_cast<long long>(t) * a.max_blocks, a.kv_heads, u.is_q ? 0 : u.g, a.page_size,
+                           u.ld, c, !u.is_q && c < u.width, at.pos + 1 - a.pool, a.pool - 1);
+    }
+  }
+  pdl_wait();
+  const float* row = a.proj + t * a.ld;
 #pragma unroll
   for (int i = 0; i < U; ++i) {
-    const HeadUnit u(a, first + i);
-    if (!u.there) return;
-    const float* w = u.norm(a);
-    float inv = 1.f;
-    if (w) {
-      float ss = 0.f;
+    const HeadUnit u = unit(i);
 #pragma unroll
-      for (int n = 0; n < NC; ++n) ss += x[i][n].sumsq();
-      inv = rsqrtf(warp_sum(ss) / static_cast<float>(u.width) + a.eps);
-    }
-    const float* angle = u.angles(a);
-    const int half = u.dims / 2;
-    T* dst = u.destination<T>(a);
-    const bool whole = U == 1 && blocks && u.ends_block(a);
-#pragma unroll
-    for (int n = 0; n < NC; ++n) {
-      const int c = (n * 32 + lane) * 4;
-      if (c >= u.width) break;
-      Vec<4> y = x[i][n];
-      if (w) {
-        const Vec<4> ww = load_vec<4>(w + c);
-#pragma unroll
-        for (int k = 0; k < 4; ++k) y.x[k] *= inv * ww.x[k];
+    for (int n = 0; n < 2; ++n) {
+      x[i][n] = Vec<4>{};
+      if (c < u.width) {
+        const float* src = row + u.col + c + n * 4;
+        x[i][n] = U > 1 && a.n_partials == 1 ? load_vec<4>(src) : slab_sum_vec<4>(src, a.n_partials, a.pstride);
+        if (a.bias) x[i][n].add(load_vec<4>(a.bias + u.col + c + n * 4));
       }
+    }
+  }
+  PairAngles of_qk = {}, of_v = {};
+  if (a.rot_dims > 0 && warp_first < a.heads + a.kv_heads) of_qk.load(a.cos_sin + static_cast<long long>(at.pos) * a.rot_dims, a.rot_dims, c);
+  if (a.v_rot_dims > 0 && warp_first + kAtOnce * U > a.heads + a.kv_heads)
+    of_v.load(a.v_cos_sin + static_cast<long long>(at.pos) * a.v_rot_dims, a.v_rot_dims, c);
+  const float inv_dim = 1.0f / static_cast<float>(a.dim);
 #pragma unroll
-      for (int k = 0; k < 4; k += 2)
-        if (c + k < u.dims) {
-          const float cs = angle[(c + k) / 2], sn = angle[half + (c + k) / 2], p = y.x[k], q = y.x[k + 1];
-          y.x[k] = p * cs - q * sn;
-          y.x[k + 1] = q * cs + p * sn;
-        }
-      if (dst) store_vec<4>(dst + c, y);
-      if (whole) {
+  for (int i = 0; i < U; ++i) {
+    const HeadUnit u = unit(i);
+    float ss = x[i][0].sumsq() + x[i][1].sumsq();
 #pragma unroll
-        for (int k = 0; k < 4; ++k) sum[n].x[k] += sizeof(T) == 2 ? to_f32<T>(from_f32<T>(y.x[k])) : y.x[k];      // as the cache holds it
-        store_vec<4>(u.block_row<T>(a) + c, divided(sum[n], a.pool));
+    for (int o = L / 2; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+    if (first + i * kAtOnce >= at.n_heads || c >= u.width) continue;
+    if (const float* w = u.norm(a)) {
+      const float inv = rsqrtf(ss * inv_dim + a.eps);
+#pragma unroll
+      for (int n = 0; n < 2; ++n) {
+        const Vec<4> ww = load_vec<4>(w + c + n * 4);
+#pragma unroll
+        for (int k = 0; k < 4; ++k) x[i][n].x[k] *= inv * ww.x[k];
+      }
+    }
+    if (u.dims > 0) {
+      PairAngles an;
+#pragma unroll
+      for (int k = 0; k < 4; ++k) {
+        an.cs[k] = u.is_v ? of_v.cs[k] : of_qk.cs[k];
+        an.sn[k] = u.is_v ? of_v.sn[k] : of_qk.sn[k];
+      }
+      an.turn(x[i][0], 0);
+      an.turn(x[i][1], 2);
+    }
+    if (T* dst = u.destination<T>(a, at)) {
+      store_vec<4>(dst + c, x[i][0]);
+      store_vec<4>(dst + c + 4, x[i][1]);
+    }
+    if (whole && !u.is_q) {
+#pragma unroll
+      for (int n = 0; n < 2; ++n) {
+#pragma unroll
+        for (int k = 0; k < 4; ++k) sum[n].x[k] += sizeof(T) == 2 ? to_f32<T>(from_f32<T>(x[i][n].x[k])) : x[i][n].x[k];   // as the cache holds it
+        store_vec<4>(u.block_row<T>(a, at) + c + n * 4, divided(sum[n], a.pool));
       }
     }
   }
@@ -350,17 +390,19 @@ head_pairs_kernel(const GroupedIn a, bool blocks) {
 // Any head: a warp has one, through shared memory.
 template <typename T, int V>
 __global__ void __launch_bounds__(kInThreads)
-head_in_kernel(const GroupedIn a, int pitch, bool blocks) {
+head_in_kernel(const GroupedIn a, int groups, int pitch, bool blocks) {
   extern __shared__ float4 stage_raw[];
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   float* x = reinterpret_cast<float*>(stage_raw) + warp * pitch;
   pdl_launch_dependents();
   pdl_wait();
-  const HeadUnit u(a, blockIdx.x * static_cast<long long>(kInThreads / 32) + warp);
-  if (!u.there) return;
+  const int t = blockIdx.x / groups, s = (blockIdx.x - t * groups) * (kInThreads / 32) + warp;
+  const HeadToken at(a, t);
+  if (s >= at.n_heads) return;
+  const HeadUnit u(a, s);
   const int half = u.dims / 2;
   const bool pairs = u.is_v || a.rot_pairs;
-  const float* row = a.proj + u.t * a.ld + u.col;
+  const float* row = a.proj + t * a.ld + u.col;
   float ss = 0.f;
   for (int c = lane * V; c < u.width; c += 32 * V) {
     Vec<V> v = slab_sum_vec<V>(row + c, a.n_partials, a.pstride);
@@ -371,9 +413,9 @@ head_in_kernel(const GroupedIn a, int pitch, bool blocks) {
   const float* w = u.norm(a);
   const float inv = w ? rsqrtf(warp_sum(ss) / static_cast<float>(u.width) + a.eps) : 1.0f;
   __syncwarp();
-  const float* angle = u.angles(a);
-  T* dst = u.destination<T>(a);
-  const bool whole = blocks && u.ends_block(a);
+  const float* angle = u.angles(a, at.pos);
+  T* dst = u.destination<T>(a, at);
+  const bool whole = blocks && at.ends_block && !u.is_q;
   for (int c0 = 0; c0 < u.width; c0 += 32 * V) {
     const int c = c0 + lane * V;
     Vec<V> y;
@@ -393,11 +435,12 @@ head_in_kernel(const GroupedIn a, int pitch, bool blocks) {
     }
     if (dst && c < u.width) store_vec<V>(dst + c, y);
     if (whole) {
-      Vec<V> sum = rows_sum<T, V>(u.cache<T>(a), a.block_table + u.t * a.max_blocks, a.kv_heads, u.g, a.page_size, u.ld, c, u.width,
-                                  u.pos + 1 - a.pool, a.pool - 1);
+      Vec<V> sum[1];
+      rows_sum<T, V, 1, 32>(sum, u.cache<T>(a), a.block_table + static_cast<long long>(t) * a.max_blocks, a.kv_heads, u.g, a.page_size, u.ld, c,
+                            c < u.width, at.pos + 1 - a.pool, a.pool - 1);
       if (c < u.width) {
-        sum.add(y);
-        store_vec<V>(u.block_row<T>(a) + c, divided(sum, a.pool));
+        sum[0].add(y);
+        store_vec<V>(u.block_row<T>(a, at) + c, divided(sum[0], a.pool));
       }
     }
   }
@@ -405,14 +448,13 @@ head_in_kernel(const GroupedIn a, int pitch, bool blocks) {
 
 // A warp has a run of `run` tokens (up to 32) and a key or value head: the means of the blocks that end there.
 template <typename T, int V>
-__global__ void __launch_bounds__(kInThreads)
+__global__ void __launch_bounds__(kInThreads, 3)
 pool_blocks_kernel(const GroupedIn a, const int* __restrict__ row_seq, int run) {
   pdl_launch_dependents();
   pdl_wait();
   const int lane = threadIdx.x & 31;
-  const long long unit = blockIdx.x * static_cast<long long>(kInThreads / 32) + (threadIdx.x >> 5);
-  const int s = static_cast<int>(unit % (2 * a.kv_heads));
-  const long long t0 = unit / (2 * a.kv_heads) * run;
+  const int unit = blockIdx.x * (kInThreads / 32) + (threadIdx.x >> 5), r = unit / (2 * a.kv_heads), s = unit - r * 2 * a.kv_heads;
+  const long long t0 = static_cast<long long>(r) * run;
   if (t0 >= a.n_tokens) return;
   const bool is_v = s >= a.kv_heads, mine = lane < run && t0 + lane < a.n_tokens;
   const int g = is_v ? s - a.kv_heads : s, width = is_v ? a.vdim : a.dim, ld = is_v ? a.v_ld : a.q_ld;
@@ -425,28 +467,28 @@ pool_blocks_kernel(const GroupedIn a, const int* __restrict__ row_seq, int run) 
     T* dst = cache + page_row(bt, a.pool_col, b, a.kv_heads, g, a.page_size) * ld;
     for (int c0 = 0; c0 < width; c0 += 32 * V) {
       const int c = c0 + lane * V;
-      const Vec<V> sum = rows_sum<T, V>(cache, bt, a.kv_heads, g, a.page_size, ld, c, width, b * a.pool, a.pool);
-      if (c < width) store_vec<V>(dst + c, divided(sum, a.pool));
+      Vec<V> sum[1];
+      rows_sum<T, V, 1, 32>(sum, cache, bt, a.kv_heads, g, a.page_size, ld, c, c < width, b * a.pool, a.pool);
+      if (c < width) store_vec<V>(dst + c, divided(sum[0], a.pool));
     }
   }
 }
 
-template <typename T, int NC>
+template <typename T, int L>
 static int head_pairs_t(const GroupedIn& a, bool one_token, cudaStream_t st) {
-  const long long units = static_cast<long long>(a.n_tokens) * (a.heads + 2 * a.kv_heads);
-  constexpr int kFew = 4096, kPer = NC == 1 ? 4 : 2;
-  const long long per = (units <= kFew || one_token ? 1 : kPer) * (kInThreads / 32);
-  const dim3 grid(static_cast<unsigned>((units + per - 1) / per));
-  if (units <= kFew || one_token) BCG_CUDA_CHECK(launch_k(head_pairs_kernel<T, NC, 1>, grid, dim3(kInThreads), 0, st, a, one_token));
-  else BCG_CUDA_CHECK(launch_k(head_pairs_kernel<T, NC, kPer>, grid, dim3(kInThreads), 0, st, a, false));
+  const bool few = one_token || a.n_tokens <= 128;
+  const int per = (few ? 1 : 2) * (kInThreads / L), groups = (a.heads + 2 * a.kv_heads + per - 1) / per;
+  const dim3 grid(static_cast<unsigned>(a.n_tokens * groups));
+  if (few) BCG_CUDA_CHECK(launch_k(head_pairs_kernel<T, L, 1>, grid, dim3(kInThreads), 0, st, a, groups, one_token));
+  else BCG_CUDA_CHECK(launch_k(head_pairs_kernel<T, L, 2>, grid, dim3(kInThreads), 0, st, a, groups, false));
   return BCG_OK;
 }
 
 template <typename T, int V>
 static int head_in_t(const GroupedIn& a, const int* row_seq, bool one_token, cudaStream_t st) {
   const int wide = max(a.dim, a.vdim);
-  if (V == 4 && a.rot_pairs && wide <= 256) {
-    BCG_TRY(wide <= 128 ? (head_pairs_t<T, 1>(a, one_token, st)) : (head_pairs_t<T, 2>(a, one_token, st)));
+  if (V == 4 && a.rot_pairs && wide <= 256 && a.dim % 8 == 0 && a.vdim % 8 == 0) {
+    BCG_TRY(wide <= 128 ? (head_pairs_t<T, 16>(a, one_token, st)) : (head_pairs_t<T, 32>(a, one_token, st)));
   } else {
     const int pitch = (wide + 3) / 4 * 4;
     const size_t sm = static_cast<size_t>(kInThreads / 32) * pitch * 4;
@@ -455,8 +497,9 @@ static int head_in_t(const GroupedIn& a, const int* row_seq, bool one_token, cud
       return BCG_ERR_UNSUPPORTED;
     }
     if (sm > 48 * 1024) BCG_TRY(ensure_dynamic_smem(reinterpret_cast<const void*>(head_in_kernel<T, V>), 200 * 1024));
-    const long long units = static_cast<long long>(a.n_tokens) * (a.heads + 2 * a.kv_heads);
-    BCG_CUDA_CHECK(launch_k(head_in_kernel<T, V>, dim3(static_cast<unsigned>((units + 7) / 8)), dim3(kInThreads), sm, st, a, pitch, one_token));
+    const int groups = (a.heads + 2 * a.kv_heads + kInThreads / 32 - 1) / (kInThreads / 32);
+    BCG_CUDA_CHECK(launch_k(head_in_kernel<T, V>, dim3(static_cast<unsigned>(a.n_tokens * groups)), dim3(kInThreads), sm, st, a, groups, pitch,
+                            one_token));
   }
   if (a.pool > 0 && !one_token) {
     const int run = min(max(a.pool, 4), 32);

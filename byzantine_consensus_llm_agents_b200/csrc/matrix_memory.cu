@@ -465,34 +465,60 @@ memory_stream_kernel(const MemArgs a, int n_units) {
 // ------------------------------------------------------------------------------------------- norm
 constexpr int kMnThreads = 256;
 
-// A head of a token per warp.  SLABS: output gates are columns of the projection, else of a.x.
-template <typename T, int V, bool SLABS>
+__device__ __forceinline__ float sigmoid_fast(float x) { return __fdividef(1.0f, 1.0f + __expf(-x)); }
+
+// A head of a token per warp.  SLABS: output gates are columns of the projection, else of a.x.  Up to NV vectors per lane stay in
+// registers between the sum of squares and the output (NV = 0: any number, read twice).
+template <typename T, int V, bool SLABS, int NV>
 __global__ void __launch_bounds__(kMnThreads)
 memory_norm_kernel(const MemArgs a, T* __restrict__ out, long long out_ld) {
   pdl_launch_dependents();
   pdl_wait();
-  const int lane = threadIdx.x & 31;
-  const long long unit = blockIdx.x * static_cast<long long>(kMnThreads / 32) + (threadIdx.x >> 5);
-  if (unit >= static_cast<long long>(a.n_tokens) * a.heads) return;
-  const long long t = unit / a.heads;
-  const int h = static_cast<int>(unit % a.heads);
+  const int lane = threadIdx.x & 31, unit = blockIdx.x * (kMnThreads / 32) + (threadIdx.x >> 5);
+  const int tok = unit / a.heads, h = unit - tok * a.heads;
+  if (tok >= a.n_tokens) return;
+  const long long t = tok;
   const T* y = static_cast<const T*>(a.y) + t * a.inner() + h * a.vdim;
   const T* g = static_cast<const T*>(a.x) + t * a.x_ld() + a.g_col(h);
   const float* slabs = a.proj + t * a.ld + 2 * a.heads * a.dim + (a.heads + h) * a.vdim;
   const float* w = a.norm + h * a.vdim;
-  float ss = 0.f;
-  for (int c = lane * V; c < a.vdim; c += 32 * V) ss += load_vec<V>(y + c).sumsq();
-  const float den = 1.0f / a.den[unit];
-  const float f = den * rsqrtf(warp_sum(ss) * den * den / static_cast<float>(a.vdim) + a.eps);
   T* dst = out + t * out_ld + h * a.vdim;
-  for (int c = lane * V; c < a.vdim; c += 32 * V) {
-    Vec<V> o = load_vec<V>(y + c), gate;
-    if constexpr (SLABS) gate = slab_sum_vec<V>(slabs + c, a.n_partials, a.pstride);
-    else gate = load_vec<V>(g + c);
+  const float den = 1.0f / a.den[unit];
+  auto gate_of = [&](int c) {
+    if constexpr (SLABS) return slab_sum_vec<V>(slabs + c, a.n_partials, a.pstride);
+    else return load_vec<V>(g + c);
+  };
+  auto finish = [&](Vec<V> o, const Vec<V>& gate, float f, int c) {
     const Vec<V> ww = load_vec<V>(w + c);
 #pragma unroll
-    for (int k = 0; k < V; ++k) o.x[k] *= f * ww.x[k] * sigmoid_f32(gate.x[k]);
+    for (int k = 0; k < V; ++k) o.x[k] *= f * ww.x[k] * (sizeof(T) == 2 ? sigmoid_fast(gate.x[k]) : sigmoid_f32(gate.x[k]));
     store_vec<V>(dst + c, o);
+  };
+  float ss = 0.f;
+  Vec<V> o[NV > 0 ? NV : 1], gate[NV > 0 ? NV : 1];
+  if constexpr (NV > 0) {
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+      const int c = (i * 32 + lane) * V;
+      if (c < a.vdim) {
+        o[i] = load_vec<V>(y + c);
+        gate[i] = gate_of(c);
+      } else {
+        o[i] = Vec<V>{};
+      }
+    }
+#pragma unroll
+    for (int i = 0; i < NV; ++i) ss += o[i].sumsq();
+  } else {
+    for (int c = lane * V; c < a.vdim; c += 32 * V) ss += load_vec<V>(y + c).sumsq();
+  }
+  const float f = den * rsqrtf(warp_sum(ss) * den * den / static_cast<float>(a.vdim) + a.eps);
+  if constexpr (NV > 0) {
+#pragma unroll
+    for (int i = 0; i < NV; ++i)
+      if ((i * 32 + lane) * V < a.vdim) finish(o[i], gate[i], f, (i * 32 + lane) * V);
+  } else {
+    for (int c = lane * V; c < a.vdim; c += 32 * V) finish(load_vec<V>(y + c), gate_of(c), f, c);
   }
 }
 
@@ -523,7 +549,11 @@ static int run_np(const MemArgs& a, int n_seqs, bool stream, bool chunks, cudaSt
 template <typename T, int V, bool SLABS>
 static int launch_norm(const MemArgs& a, void* out, long long out_ld, cudaStream_t st) {
   const dim3 grid(static_cast<unsigned>((static_cast<long long>(a.n_tokens) * a.heads + kMnThreads / 32 - 1) / (kMnThreads / 32)));
-  BCG_CUDA_CHECK(launch_k(memory_norm_kernel<T, V, SLABS>, grid, dim3(kMnThreads), 0, st, a, static_cast<T*>(out), out_ld));
+  T* o = static_cast<T*>(out);
+  const dim3 block(kMnThreads);
+  if (V == 4 && a.vdim <= 256) BCG_CUDA_CHECK(launch_k(memory_norm_kernel<T, V, SLABS, 2>, grid, block, 0, st, a, o, out_ld));
+  else if (V == 4 && a.vdim <= 512) BCG_CUDA_CHECK(launch_k(memory_norm_kernel<T, V, SLABS, 4>, grid, block, 0, st, a, o, out_ld));
+  else BCG_CUDA_CHECK(launch_k(memory_norm_kernel<T, V, SLABS, 0>, grid, block, 0, st, a, o, out_ld));
   return BCG_OK;
 }
 

@@ -117,7 +117,7 @@ int expert_in(const bcg_stack* m, const bcg_layer* l, const bcg_stack_ws* ws, in
               bool with_act, cudaStream_t st) {
   const int ff = with_act ? l->ff : 0;
   const int blocks = ff == 0 ? 0 : T <= 128 ? (ff + kExpertInThreads * 4 - 1) / (kExpertInThreads * 4) : 1;
-  const int per = T <= 128 ? kExpertInThreads / 32 : kExpertInThreads / 4;
+  const int per = T <= 128 ? kExpertInThreads / 32 : kExpertInThreads / 8;
   const dim3 grid(T * blocks + (T + per - 1) / per);
   const size_t sm = static_cast<size_t>(route_words(l->experts, kExpertInThreads)) * 4;
   if (sm > 48 * 1024 || l->top > l->experts || l->n_router < l->experts || l->n_router % 4 || l->ff % 16 || !l->router_bias) {
