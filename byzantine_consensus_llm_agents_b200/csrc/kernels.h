@@ -151,8 +151,9 @@ int expert_in(const bcg_stack* m, const bcg_layer* l, const bcg_stack_ws* ws, in
               bool with_act, cudaStream_t stream);
 int expert_in_step(const bcg_stack* m, const bcg_stack_ws* ws, int layer, int T, int n_partials, long long pstride, long long ld,
                    int with_act, cudaStream_t stream);
+// split: the operands are activations in ws->ssm_x already, ws->proj has just the gates
 int matrix_memory(const bcg_stack* m, const bcg_layer* l, const bcg_stack_ws* ws, const bcg_step_batch* b, int n_partials,
-                  long long pstride, long long ld, int mode, cudaStream_t stream);
+                  long long pstride, long long ld, int mode, bool split, cudaStream_t stream);
 int matrix_memory_step(const bcg_stack* m, const bcg_stack_ws* ws, const bcg_step_batch* b, int layer, int n_partials,
                        long long pstride, long long ld, int mode, cudaStream_t stream);
 struct WindowAttn;

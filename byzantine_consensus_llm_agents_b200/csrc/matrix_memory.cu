@@ -7,6 +7,7 @@
 // [vdim + 1][dim] per head, n behind S; every block of 64 rows keeps its own copy of m, so that no CTA waits for another's.
 //
 //   memory_in      projection slabs -> q | k | v | output gate as activations, heads padded to multiples of 8 columns
+//                  (long bf16 launches: the product writes them itself where no head needs padding)
 //   chunks         portions (bf16): chunks of 64 tokens on tensor cores (state_chunk.cuh).  With c_t the running sum of f in a chunk,
 //                  a_t = i_t - c_t and M_t the running maximum of a and the chunk's first m, m_t = c_t + M_t, so that all
 //                  weights are exp(a_j - M_i), exp(m - M_i) and exp(a_j - M_last): no difference of large sums
@@ -558,10 +559,10 @@ static int launch_norm(const MemArgs& a, void* out, long long out_ld, cudaStream
 }
 
 template <typename T>
-static int run_t(const MemArgs& a, int n_seqs, bool one_token, int mode, void* out, long long out_ld, cudaStream_t st) {
-  const bool wide = ((a.dim | a.vdim) & 3) == 0 && a.ld % 4 == 0 && a.pstride % 4 == 0 && out_ld % 4 == 0;
-  const bool stream = one_token && mode == 0 && a.dim % 4 == 0, chunks = sizeof(T) == 2 && mode == 0;
-  if (!stream) {
+static int run_t(const MemArgs& a, int n_seqs, bool one_token, int mode, bool split, void* out, long long out_ld, cudaStream_t st) {
+  const bool wide = ((a.dim | a.vdim) & 3) == 0 && (split || a.ld % 4 == 0) && a.pstride % 4 == 0 && out_ld % 4 == 0;
+  const bool stream = one_token && mode == 0 && !split && a.dim % 4 == 0, chunks = sizeof(T) == 2 && mode == 0;
+  if (!stream && !split) {
     const int n = 2 * a.heads * (a.dim + a.vdim);
     const int blocks = a.n_tokens <= 128 ? (n + kMiThreads * 4 - 1) / (kMiThreads * 4) : 1;
     const dim3 grid(static_cast<unsigned>(a.n_tokens * blocks));
@@ -577,7 +578,7 @@ static int run_t(const MemArgs& a, int n_seqs, bool one_token, int mode, void* o
 }
 
 int matrix_memory(const bcg_stack* m, const bcg_layer* l, const bcg_stack_ws* ws, const bcg_step_batch* b, int n_partials,
-                  long long pstride, long long ld, int mode, cudaStream_t st) {
+                  long long pstride, long long ld, int mode, bool split, cudaStream_t st) {
   if (!l->mem_bias || !l->mem_norm || !l->mem_state || !l->mem_max || !ws->ssm_x || !ws->ssm_y || !ws->mem_den || !b->state_slots ||
       l->heads <= 0 || l->dim <= 0 || l->dim > 256 || l->vdim <= 0 || l->vdim > 65535 * kSsRows || l->gate_cap <= 0.f || b->n_seqs > 65535) {
     set_last_error("bcg_matrix_memory", "bad layer (1..256 key channels) or too many sequences");
@@ -588,7 +589,7 @@ int matrix_memory(const bcg_stack* m, const bcg_layer* l, const bcg_stack_ws* ws
   a.n_partials = n_partials;
   a.pstride = pstride;
   a.ld = ld;
-  a.gate_col = l->gate_col;
+  a.gate_col = split ? 0 : l->gate_col;
   a.bias = l->mem_bias;
   a.norm = l->mem_norm;
   a.positions = b->positions;
@@ -608,8 +609,8 @@ int matrix_memory(const bcg_stack* m, const bcg_layer* l, const bcg_stack_ws* ws
   a.scale = 1.0f / sqrtf(static_cast<float>(l->dim));
   a.eps = m->eps;
   const bool one = b->T == b->n_seqs;
-  return m->act_dtype == BCG_DT_F32 ? run_t<float>(a, b->n_seqs, one, mode, ws->mix, l->mix_ld, st)
-                                    : run_t<__nv_bfloat16>(a, b->n_seqs, one, mode, ws->mix, l->mix_ld, st);
+  return m->act_dtype == BCG_DT_F32 ? run_t<float>(a, b->n_seqs, one, mode, split, ws->mix, l->mix_ld, st)
+                                    : run_t<__nv_bfloat16>(a, b->n_seqs, one, mode, split, ws->mix, l->mix_ld, st);
 }
 
 }  // namespace bcg

@@ -193,6 +193,24 @@ static int expert_ff(const bcg_stack* m, const bcg_stack_ws* ws, const bcg_layer
   return l->ff > 0 ? project(m, ws->act, l->w_down, ws->proj, ws->proj_floats, T, d, l->ff, splits, st) : static_cast<int>(BCG_OK);
 }
 
+// Long launches: queries, keys, values and output gates leave their product as the activations that the matrix memory reads; the
+// input and forget gates, a product of their own, stay fp32.
+static bool memory_splits(const bcg_stack* m, const bcg_layer* l, int T) {
+  return m->act_dtype == BCG_DT_BF16 && T > 128 && l->dim % 8 == 0 && l->vdim % 8 == 0 && tensor_gemm(m->act_dtype, T, l->gate_col, m->d_model) &&
+         tensor_gemm(m->act_dtype, T, l->n_in - l->gate_col, m->d_model);
+}
+static int memory_products(const bcg_stack* m, const bcg_stack_ws* ws, const bcg_layer* l, int T, cudaStream_t st) {
+  const int d = m->d_model, n = l->gate_col;
+  int s;
+  if (!ws->ssm_x) {
+    set_last_error("bcg_stack_step", "incomplete workspace");
+    return BCG_ERR_ARG;
+  }
+  BCG_TRY(gemm_bf16_tn(ws->xn, l->w_in, ws->ssm_x, T, n, d, d, d, n, BCG_EPI_BF16, 1, launch_flags() & BCG_GEMM_PDL, st));
+  return project(m, ws->xn, static_cast<const char*>(l->w_in) + static_cast<size_t>(n) * d * 2, ws->proj, ws->proj_floats, T, l->n_in - n, d,
+                 &s, st);
+}
+
 int matrix_memory_step(const bcg_stack* m, const bcg_stack_ws* ws, const bcg_step_batch* b, int layer, int n_partials,
                        long long pstride, long long ld, int mode, cudaStream_t st) {
   BCG_TRY(check_stack(m, ws));
@@ -201,7 +219,12 @@ int matrix_memory_step(const bcg_stack* m, const bcg_stack_ws* ws, const bcg_ste
     set_last_error("bcg_matrix_memory", "not a matrix memory layer, or a bad batch");
     return BCG_ERR_ARG;
   }
-  return matrix_memory(m, &m->layers[layer], ws, b, n_partials, pstride, ld, mode, st);
+  const bcg_layer* l = &m->layers[layer];
+  if (mode == 2 && (l->dim % 8 || l->vdim % 8 || n_partials != 1)) {
+    set_last_error("bcg_matrix_memory", "operands that are activations already: heads in multiples of 8 columns, one slab of gates");
+    return BCG_ERR_ARG;
+  }
+  return matrix_memory(m, l, ws, b, n_partials, pstride, ld, mode == 2 ? 0 : mode, mode == 2, st);
 }
 
 int state_space_step(const bcg_stack* m, const bcg_stack_ws* ws, const bcg_step_batch* b, int layer, int n_partials,
@@ -241,7 +264,9 @@ int stack_step(const bcg_stack* m, const bcg_stack_ws* ws, const bcg_step_batch*
       continue;
     }
     int s = 1, mix_out = 0;
-    BCG_TRY(project(m, ws->xn, l->w_in, ws->proj, ws->proj_floats, T, l->n_in, d, &s, st));
+    const bool split = l->mixer == BCG_MIXER_MATRIX_MEMORY && T != b->n_seqs && memory_splits(m, l, T);
+    if (split) BCG_TRY(memory_products(m, ws, l, T, st));
+    else BCG_TRY(project(m, ws->xn, l->w_in, ws->proj, ws->proj_floats, T, l->n_in, d, &s, st));
     const long long in_stride = static_cast<long long>(T) * l->n_in;
     if (l->mixer == BCG_MIXER_LATENT_ATTN) {
       mix_out = l->heads * l->vdim;
@@ -266,7 +291,7 @@ int stack_step(const bcg_stack* m, const bcg_stack_ws* ws, const bcg_step_batch*
       if (l->ssm_heads > 0) BCG_TRY(state_space(m, l, ws, b, s, in_stride, l->n_in, 0, st));
     } else if (l->mixer == BCG_MIXER_MATRIX_MEMORY) {
       mix_out = l->mix_ld;
-      BCG_TRY(matrix_memory(m, l, ws, b, s, in_stride, l->n_in, 0, st));
+      BCG_TRY(matrix_memory(m, l, ws, b, s, in_stride, split ? l->n_in - l->gate_col : l->n_in, 0, split, st));
     } else {
       set_last_error("bcg_stack_step", "unknown mixer");
       return BCG_ERR_UNSUPPORTED;

@@ -348,14 +348,20 @@ def _vosolorn_kernels(k: _Bench, what: str, B: int, T: int, shape: str, v, plan)
              else dict(nbytes=B * (min(m.window, CTX) + blocks(CTX)) * m.kv_heads * (m.dim + m.vdim) * 2.0)))
     k.add("input split", shape, lambda: lib.bcg_grouped_in(model, ws, C.byref(bt), i_att, s, T * n_in, n_in, 0, st()),
           nbytes=T * m.in_dim * (4.0 * s + 2))
-    # the projection in, outputs out, states in and out; the products of 64-token chunks
-    k.add("matrix memory, all launches", shape, lambda: lib.bcg_matrix_memory(model, ws, C.byref(bt), i_mem, s_mem, T * n_mem, n_mem, 0, st()),
-          nbytes=T * (mem.in_dim * 4.0 * s_mem + mem.out_dim * 2) + B * mem.state_floats * 8.0,
+    # operands in (prompts: activations and fp32 gates), outputs out, states in and out; the products of 64-token chunks
+    ld, mode = (n_mem - mem.gate_col, 2) if prefill else (n_mem, 0)
+    operands = mem.x_ld * 2.0 + 8.0 * mem.heads if prefill else mem.in_dim * 4.0 * s_mem
+    k.add("matrix memory, all launches", shape, lambda: lib.bcg_matrix_memory(model, ws, C.byref(bt), i_mem, s_mem, T * ld, ld, mode, st()),
+          nbytes=T * (operands + mem.out_dim * 2) + B * mem.state_floats * 8.0,
           flops=2.0 * T * mem.heads * (mem.vdim * (32 + 2 * mem.dim) + 32 * mem.dim) if prefill else 0.0)
     k.add("norm", shape, lambda: lib.bcg_sandwich_norm(
         b["residual"].data_ptr(), b["proj"].data_ptr(), s_out, T * d, w["norm1b"].data_ptr(), None, b["xn"].data_ptr(), L.DT_BF16, T, d,
         1e-5, st()), nbytes=T * d * (10.0 + 4 * s_out))
-    k.gemm("input product", shape, b["xn"], w["w_in"], b["proj"], T, n_mem, d, L.EPI_F32, s_mem)
+    if prefill:
+        k.gemm("input product", shape, b["xn"], w["w_in"], b["ssm_x"], T, mem.gate_col, d, L.EPI_BF16, 1)
+        k.gemm("gate product", shape, b["xn"], w["w_in"][mem.gate_col:], b["proj"], T, n_mem - mem.gate_col, d, L.EPI_F32, 1)
+    else:
+        k.gemm("input product", shape, b["xn"], w["w_in"], b["proj"], T, n_mem, d, L.EPI_F32, s_mem)
     k.gemm("output product", shape, b["mix"], w["w_out"], b["proj"], T, d, mem.out_dim, L.EPI_F32, s_out)
     if isinstance(f, S.MoeMlp):
         used, rows, ff = _route_at_random(k, i_mem, T), T * f.top, f.ff_ld

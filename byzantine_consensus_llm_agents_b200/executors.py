@@ -365,8 +365,8 @@ class StackExecutor:
                 n += 5 + (4 if isinstance(l.mlp, MoeMlp) else 0)
                 continue
             if l.composed:
-                # input projection, attention's split (, pooled blocks) and kernel, state space or matrix memory (convolution or
-                # split,) recurrence and norm, output projection, norm; feed-forward: up, its unit where K is split, down, norm;
+                # input projection, attention's split (, pooled blocks) and kernel, state space or matrix memory (convolution,
+                # split or gates' product,) recurrence and norm, output projection, norm; feed-forward: up, its unit where K is split, down, norm;
                 # experts: router and shared rows, routing, scatter, two products, unit, shared output, norm
                 att = l.one(GroupedAttention)
                 n += 3 + (2 if att else 0) + int(bool(att and att.pool and not decode))

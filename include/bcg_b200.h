@@ -647,8 +647,9 @@ int bcg_gemm_grouped_gelu(const void* X, const void* W, void* out, int rows, int
 int bcg_expert_in(const bcg_stack* m, const bcg_stack_ws* ws, int layer, int T, int n_partials, long long partial_stride, long long ld,
                   int with_act, void* stream);
 /* No counterpart in the reference: a matrix memory behind its input projection (ws->proj, row pitch ld): recurrence, norm and output
- * gate; states advanced, ws->mix filled.  mode 0: what bcg_stack_step picks (tensor-core chunks or, one token each, the decode
- * kernel); 1: token by token on CUDA cores. */
+ * gate; states advanced, ws->mix filled.  mode 0: tensor-core chunks or, one token each, the decode kernel; 1: token by token on CUDA
+ * cores; 2: as 0 with queries, keys, values and output gates in ws->ssm_x as activations already (heads in multiples of 8 columns),
+ * ws->proj just the input and forget gates: what bcg_stack_step does in launches of more than 128 tokens. */
 int bcg_matrix_memory(const bcg_stack* m, const bcg_stack_ws* ws, const bcg_step_batch* b, int layer, int n_partials,
                       long long partial_stride, long long ld, int mode, void* stream);
 

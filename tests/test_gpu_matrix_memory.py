@@ -110,6 +110,30 @@ def test_portions_and_tokens(size, dtype):
 
 
 @pytest.mark.parametrize("dtype", TOL)
+@pytest.mark.parametrize("size", ["usual", "small", "even"])
+def test_operands_that_are_activations_already(size, dtype):
+    """What a product with bf16 output leaves: rows q | k | v | g, and a narrow matrix of gates."""
+    a = Memory(size, dtype)
+    H, n = a.dims[0], 140
+    proj = a.proj(n, 11)
+    assert a.gate_col == a.rows and a.eng.cfg.layers[0].mixer.x_ld == a.rows
+    gates = torch.zeros(n, a.ld - a.gate_col)
+    gates[:, :2 * H] = proj[:, a.rows:]
+    a.junk()
+    out, at = [], 0
+    for t in (90, 50):
+        p, b = a.batch([(t, at, 3)])
+        a.set("ssm_x", proj[at:at + t, :a.rows])
+        a.set("proj", gates[at:at + t])
+        L.check(a.eng.lib.bcg_matrix_memory(*a.args(C.byref(b), 0, 1, 0, gates.shape[1], 2)))
+        out.append((a.get("mix", t, a.layer.mix_ld)[:, :H * a.dims[2]], a.get("mem_den", t, H)))
+        at += t
+    a.check(tuple(torch.cat(x) for x in zip(*out)), a.oracle(proj), 3)
+    p, b = a.batch([(2, 0, 0)])
+    assert a.eng.lib.bcg_matrix_memory(*a.args(C.byref(b), 0, 2, 0, gates.shape[1], 2)) != 0
+
+
+@pytest.mark.parametrize("dtype", TOL)
 @pytest.mark.parametrize("cap", [1.5, 30.0])
 @pytest.mark.parametrize("sizes", [[140], [1], [70, 1]])
 def test_gates_far_above_and_below_the_maximum(sizes, cap, dtype):
