@@ -64,7 +64,7 @@ CONFIGS = {
     "pooled": SM.output_norm_config([SM.pattn(mlp=SM.plain_moe()), SM.mlstm(mlp=SM.dense(70)), SM.pattn(4, 1, 16, 24, 5, 9, 8, base=100.0),
                                      SM.mlstm(2, 16, 72, 4.0, mlp=SM.plain_moe(5, 3, 24, 0)), SM.pattn(3, 3, 40, 16, 1, 1, 40, mlp=SM.plain_moe(4, 1, 20, 40))]),
     # everything on the tensor-core kernels
-    "pooled-tensor": SM.output_norm_config([SM.mlstm(4, 64, 128, 15.0, mlp=SM.plain_moe(8, 3, 64, 96)), SM.pattn(8, 2, 64, 64, 33, 4, 64, mlp=SM.dense(320)),
+    "pooled-tensor": SM.output_norm_config([SM.mlstm(4, 64, 128, 12.0, mlp=SM.plain_moe(8, 3, 64, 80)), SM.pattn(8, 2, 64, 64, 33, 4, 64, mlp=SM.dense(320)),
                                             SM.mlstm(3, 128, 80, mlp=SM.dense(64)), SM.pattn(4, 4, 128, 128, 70, 16, 32, mlp=SM.plain_moe(8, 1, 128, 64)),
                                             SM.pattn(2, 1, 200, 248, 17, 3, 24), SM.mlstm(1, 200, 24)], width=192, vocab=320),
     # sizes no vector load or tile likes, groups of more than 16 query heads, heads beyond the tiles
